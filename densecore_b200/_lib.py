@@ -27,6 +27,13 @@ class DcError(RuntimeError):
 
 
 _lib = None
+_partial = bool(os.environ.get("DC_B200_LIB"))   # entry points may be missing from the named library
+
+
+def use(path: str) -> None:
+    """Loads another build of the library, possibly a part of it (before the first call)."""
+    global LIB_PATH, _partial
+    LIB_PATH, _partial = path, True
 
 
 def lib() -> C.CDLL:
@@ -128,6 +135,9 @@ def _signatures() -> dict:
         "dc_b200_decode_step": (i32, [vp, vp, i32, vp, vp, vp]),
         "dc_b200_decode_run": (i32, [vp, vp, i32, vp, i32, vp, C.POINTER(f32)]),
         "dc_b200_forward_chunk": (i32, [vp, i32, vp, i32, vp]),
+        "dc_b200_forward_batch": (i32, [vp, i32, vp, vp, vp, i32, vp, vp, vp]),
+        "dc_b200_model_from_dir": (i32, [vp, cstr, i32, i32, i32, i32, pp]),
+        "dc_b200_model_from_config": (i32, [vp, cstr, cstr, i32, i32, i32, i32, pp]),
         "dc_b200_model_logits_dev": (vp, [vp]),
         "dc_b200_model_phase_timing": (i32, [vp, vp, i32]),
         "dc_b200_model_step_stats": (i32, [vp, pi, C.POINTER(C.c_double), C.POINTER(C.c_double)]),
@@ -148,8 +158,8 @@ def _signatures() -> dict:
 
 def _declare(l: C.CDLL) -> None:
     for name, (res, args) in _signatures().items():
-        if os.environ.get("DC_B200_LIB") and not hasattr(l, name):
-            continue   # an older build named for A/B timing may lack the newest entry points
+        if _partial and not hasattr(l, name):
+            continue
         fn = getattr(l, name)
         fn.restype = res
         fn.argtypes = args

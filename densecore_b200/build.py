@@ -25,14 +25,19 @@ NVCC_FLAGS = [
 ]
 
 
+# Sources of the layer-list decoders alone (no K-quant kernels): what a process that serves only such a model compiles.
+PARTS = {"layers": ["api", "kv", "linear", "linear_tc", "misc", "mix_latent", "mix_recur", "model", "norm_act", "stack", "stack_config",
+                    "stack_load"]}
+
+
 def sources() -> list[str]:
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")))
 
 
-def _stale() -> bool:
-    if not os.path.exists(LIB):
+def _stale(lib: str = LIB) -> bool:
+    if not os.path.exists(lib):
         return True
-    t = os.path.getmtime(LIB)
+    t = os.path.getmtime(lib)
     deps = sources() + glob.glob(os.path.join(CSRC, "*.h")) + glob.glob(os.path.join(CSRC, "*.cuh"))
     deps += glob.glob(os.path.join(ROOT, "include", "*.h"))
     return any(os.path.getmtime(d) > t for d in deps)
@@ -75,11 +80,31 @@ def build(force: bool = False, verbose: bool = False, out: str | None = None, ex
     return LIB
 
 
-def _build_variant(out: str, extra: list[str]) -> str:
+def build_part(part: str) -> str:
+    """The whole library if it is built and up to date, else a library of one part's sources."""
+    if not _stale():
+        return LIB
+    out = os.path.join(PKG, f"libdc_b200_{part}.so")
+    if _stale(out):
+        tmp = f"{out}.{os.getpid()}"
+        _build_variant(tmp, [], [os.path.join(CSRC, f"{n}.cu") for n in PARTS[part]])
+        os.replace(tmp, out)     # a process that starts meanwhile sees the old file or the finished one
+    return out
+
+
+def _build_variant(out: str, extra: list[str], srcs: list[str] | None = None) -> str:
+    import shutil
     import tempfile
     tmp = tempfile.mkdtemp(prefix="dcb200_")
+    try:
+        return _compile(out, extra, srcs or sources(), tmp)
+    finally:
+        shutil.rmtree(tmp, ignore_errors=True)
+
+
+def _compile(out: str, extra: list[str], srcs: list[str], tmp: str) -> str:
     objs, procs = [], []
-    for src in sources():
+    for src in srcs:
         obj = os.path.join(tmp, os.path.basename(src)[:-3] + ".o")
         cmd = [nvcc(), *NVCC_FLAGS, *extra, "-I", os.path.join(ROOT, "include"), "-c", src, "-o", obj]
         procs.append(subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True))

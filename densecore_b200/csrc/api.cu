@@ -204,6 +204,7 @@ int dc_b200_upload_weight(dc_ctx* ctx, int ggml_type, const int64_t ne[4], const
     const bool kq = ggml_type == DC_TYPE_Q4_K || ggml_type == DC_TYPE_Q6_K;
     if (!kq && ggml_type != DC_TYPE_F32 && ggml_type != DC_TYPE_F16)
         return dc_fail(ctx, DC_B200_UNSUPPORTED, "upload_weight: ggml type %d is not supported", ggml_type);
+    if (kq && !dc_launch_gemv) return dc_fail(ctx, DC_B200_UNSUPPORTED, "upload_weight: this library was built without the K-quant kernels");
     if (kq && (K % DC_QK_K))
         return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "upload_weight: K=%lld is not a multiple of 256", (long long)K);
     cudaSetDevice(ctx->device);
@@ -254,6 +255,7 @@ void* dc_b200_weight_data(const dc_weight* w, size_t* bytes) {
 int dc_b200_quantize_q8k_dev(dc_ctx* ctx, const float* x_dev, int rows, int K, void* q8_dev) {
     if (!ctx || !x_dev || !q8_dev || rows <= 0 || K <= 0 || (K % DC_QK_K))
         return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "quantize_q8k: bad argument (rows=%d K=%d)", rows, K);
+    if (!dc_launch_quantize_q8k) return dc_fail(ctx, DC_B200_UNSUPPORTED, "quantize_q8k: this library was built without the K-quant kernels");
     cudaSetDevice(ctx->device);
     return dc_launch_quantize_q8k(ctx, x_dev, rows, K, (uint8_t*)q8_dev);
 }
@@ -261,6 +263,7 @@ int dc_b200_quantize_q8k_dev(dc_ctx* ctx, const float* x_dev, int rows, int K, v
 int dc_b200_quantize_q8k(dc_ctx* ctx, const float* x_host, int rows, int K, void* q8_host) {
     if (!ctx || !x_host || !q8_host || rows <= 0 || K <= 0 || (K % DC_QK_K))
         return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "quantize_q8k: bad argument (rows=%d K=%d)", rows, K);
+    if (!dc_launch_quantize_q8k) return dc_fail(ctx, DC_B200_UNSUPPORTED, "quantize_q8k: this library was built without the K-quant kernels");
     cudaSetDevice(ctx->device);
     const size_t xb = (size_t)rows * K * 4, qb = (size_t)rows * (K / DC_QK_K) * DC_Q8K_BYTES;
     uint8_t* s = dc_scratch(ctx, xb + qb + 256);

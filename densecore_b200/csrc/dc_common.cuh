@@ -2,6 +2,7 @@
 // block layouts, exact scalar helpers, the per-warp bulk-copy pipeline that
 // streams weight rows HBM -> shared memory, and the K-quant row-dot decoders.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -16,6 +17,7 @@
 #define DC_TYPE_F16 1
 #define DC_TYPE_Q4_K 12
 #define DC_TYPE_Q6_K 14
+#define DC_TYPE_BF16 30
 
 // Hot bodies (row dots, stream loops, phases of the persistent kernel) are inlined into their callers;
 // the callers that several sites share are the ones kept out of line (measured: outlining per row costs

@@ -1,5 +1,6 @@
 // Host-side structures shared by the translation units of libdc_b200.so.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
 
@@ -12,6 +13,10 @@
 #define DC_NSTAGE 4
 #define DC_WARPS 8
 #define DC_STAGE_TARGET 4608  // bytes of weight rows one pipeline stage aims to hold: one warp pass of Q4_K rows
+
+// Launchers of the K-quant decoders.  Weak, so that a build of only the layer-list decoders (build.py, part "layers")
+// links without those kernels; entry points that need them check for their presence first.
+#define DC_PART __attribute__((weak))
 
 struct dc_weight {
     int type;        // ggml type id
@@ -68,20 +73,20 @@ enum { DC_EPI_STORE = 0, DC_EPI_ACC = 1, DC_EPI_SWIGLU = 2 };
 // zeroed by the caller) receives the packed (value,row) maximum of the stored rows.
 // dump_I / dump_M (parity checks, single segment): receive the exact int32 block sums the kernel forms,
 // [T][n_rows][K/256] (M for Q4_K only).
-int dc_launch_gemv(dc_ctx* ctx, const dc_gemv_seg* segs, int n_seg, int epi, const uint8_t* act_q8, int T, int K,
+DC_PART int dc_launch_gemv(dc_ctx* ctx, const dc_gemv_seg* segs, int n_seg, int epi, const uint8_t* act_q8, int T, int K,
                    unsigned long long* argmax, int32_t* dump_I = nullptr, int32_t* dump_M = nullptr);
 // rows x K f32 -> native Q8_K blocks (row stride K/256*292)
-int dc_launch_quantize_q8k(dc_ctx* ctx, const float* x, int rows, int K, uint8_t* out);
+DC_PART int dc_launch_quantize_q8k(dc_ctx* ctx, const float* x, int rows, int K, uint8_t* out);
 // Tensor-core MUL_MAT for many token rows (gemm_tc.cu): activations quantised into 64-token tiles, then
 // out[slot * ldo + row] for every weight row; tile_expert (optional, device) picks an expert matrix per tile.
-size_t dc_gemm_tc_act_bytes(int n_slots, int K);
-int dc_gemm_tc_tiles(int n_slots);
-bool dc_gemm_tc_supports(const dc_weight* w);
-int dc_launch_quantize_q8k_tiled(dc_ctx* ctx, const float* x, int ldx, int n_rows, int K, uint8_t* act, int n_tt,
+DC_PART size_t dc_gemm_tc_act_bytes(int n_slots, int K);
+DC_PART int dc_gemm_tc_tiles(int n_slots);
+DC_PART bool dc_gemm_tc_supports(const dc_weight* w);
+DC_PART int dc_launch_quantize_q8k_tiled(dc_ctx* ctx, const float* x, int ldx, int n_rows, int K, uint8_t* act, int n_tt,
                                  const int* slot_token);
 // pair_tile0 / pair_nset (device, n_pairs entries; needed with tile_expert): the pairs of neighbouring tiles of
 // one expert that a CTA works on
-int dc_launch_gemm_tc(dc_ctx* ctx, const dc_weight* w, const uint8_t* act, int n_slots, float* out, int ldo,
+DC_PART int dc_launch_gemm_tc(dc_ctx* ctx, const dc_weight* w, const uint8_t* act, int n_slots, float* out, int ldo,
                       const int* tile_expert = nullptr, const int* slot_row = nullptr, bool accumulate = false,
                       const int* pair_tile0 = nullptr, const int* pair_nset = nullptr, int n_pairs = 0);
 // up to three matrices of one type, K and row length in one launch (Q | K | V, gate | up)
@@ -92,7 +97,8 @@ int dc_launch_gemm_tc_multi(dc_ctx* ctx, const dc_weight* const* ws, const int* 
 
 
 // ---- misc.cu ----
-int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x);
+// ldx (0: the row length) and xb (a bf16 copy) are optional
+int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x, int ldx = 0, __nv_bfloat16* xb = nullptr);
 // x (+= add) -> RMSNorm * w -> optional f32 copy and Q8_K blocks
 int dc_launch_rmsnorm_q8k(dc_ctx* ctx, float* x, const float* add, const float* w, int T, int H, float eps,
                           float* xn_out, uint8_t* q8_out);
@@ -112,9 +118,9 @@ struct dc_attn_scratch {
     float* part_d;    // [T][n_head][nsplit]
     int* tickets;     // [T][n_kv], zeroed once
 };
-size_t dc_attention_scratch_bytes(int T, int n_head, int n_kv, int max_blocks, int nsplit);
-void dc_attn_scratch_bind(dc_attn_scratch* sc, uint8_t* base, int T, int n_head, int n_kv, int max_blocks, int nsplit);
-int dc_launch_attention(dc_ctx* ctx, const float* q, const void* k_arena, const void* v_arena,
+DC_PART size_t dc_attention_scratch_bytes(int T, int n_head, int n_kv, int max_blocks, int nsplit);
+DC_PART void dc_attn_scratch_bind(dc_attn_scratch* sc, uint8_t* base, int T, int n_head, int n_kv, int max_blocks, int nsplit);
+DC_PART int dc_launch_attention(dc_ctx* ctx, const float* q, const void* k_arena, const void* v_arena,
                         const int32_t* block_tables, int max_blocks, const int32_t* seq_ids, const int32_t* positions,
                         int T, int n_head, int n_kv, float scale, int nsplit, const dc_attn_scratch* sc, float* out,
                         uint8_t* q8_out);
@@ -138,16 +144,16 @@ struct dc_moe_route {
 // (core/src/llm/moe/native.cpp:610-676); DC_ROUTE_SOFTMAX = softmax over all experts, top-k on the
 // probabilities with strict '>', renormalise (core/src/moe/moe_routing.cpp:53-101).
 enum { DC_ROUTE_STABLE = 0, DC_ROUTE_SOFTMAX = 1 };
-int dc_launch_router(dc_ctx* ctx, const dc_weight* wr, const float* xn, int n_expert, int T, int top_k, float scale,
+DC_PART int dc_launch_router(dc_ctx* ctx, const dc_weight* wr, const float* xn, int n_expert, int T, int top_k, float scale,
                      int ep_lo, int ep_hi, const dc_moe_route* rt, int mode = DC_ROUTE_STABLE);
 // the same routing for any number of tokens (prompt chunks): logits [T][E], ids and weights [T][top_k]
 int dc_launch_router_batched(dc_ctx* ctx, const dc_weight* wr, const float* xn, int T, int top_k, float scale, float* logits,
                              int32_t* ids, float* weights, int mode);
 // carves a dc_moe_route for (T, E, top_k) out of a byte buffer; returns bytes used
-size_t dc_moe_route_bind(dc_moe_route* rt, uint8_t* base, int T, int E, int top_k);
-int dc_launch_moe_mm(dc_ctx* ctx, bool pair, const dc_weight* w0, const dc_weight* w1, const uint8_t* act_q8,
+DC_PART size_t dc_moe_route_bind(dc_moe_route* rt, uint8_t* base, int T, int E, int top_k);
+DC_PART int dc_launch_moe_mm(dc_ctx* ctx, bool pair, const dc_weight* w0, const dc_weight* w1, const uint8_t* act_q8,
                      int act_rows, int T, int top_k, int e_base, const dc_moe_route* rt, float* out);
-int dc_launch_moe_combine(dc_ctx* ctx, const float* dn, const int32_t* ids, const float* weights, int T, int top_k,
+DC_PART int dc_launch_moe_combine(dc_ctx* ctx, const float* dn, const int32_t* ids, const float* weights, int T, int top_k,
                           int H, int ep_lo, int ep_hi, float* out);
 
 // ---- sample.cu ----

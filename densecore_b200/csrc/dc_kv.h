@@ -22,6 +22,13 @@ struct dc_kv_cache {
     __half* k_arena = nullptr;
     __half* v_arena = nullptr;
     int32_t* d_tables = nullptr; // [max_seqs][max_blocks_per_seq]
+    // Caches of other shapes: planes of `row_bytes` per token, [block][16 slots][row_bytes], sharing the block tables;
+    // and one fixed-size state slot per sequence for recurrent layers (copied by a fork; a state cannot be
+    // truncated and is not shared through the prefix cache).
+    struct plane { size_t row_bytes = 0; uint8_t* arena = nullptr; };
+    std::vector<plane> planes;
+    uint8_t* state = nullptr;    // [max_seqs][state_bytes]
+    size_t state_bytes = 0;
     std::vector<int> free_list;
     std::vector<int> ref;        // references per physical block (sequences sharing it after a fork)
     std::vector<dc_kv_seq> seqs;
@@ -39,6 +46,8 @@ struct dc_kv_cache {
 
 int dc_kv_init(dc_ctx* ctx, dc_kv_cache* kv, int n_layer, int n_kv_head, int head_dim, int max_blocks, int max_seqs,
                int max_blocks_per_seq);
+int dc_kv_init_planes(dc_ctx* ctx, dc_kv_cache* kv, const std::vector<size_t>& row_bytes, size_t state_bytes, int max_blocks, int max_seqs,
+                      int max_blocks_per_seq);
 void dc_kv_release(dc_kv_cache* kv);
 int dc_kv_seq_alloc(dc_kv_cache* kv, int* out_seq);
 int dc_kv_seq_free(dc_kv_cache* kv, int seq);

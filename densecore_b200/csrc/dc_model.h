@@ -12,6 +12,7 @@
 enum {
     DC_K_EMBED = 0, DC_K_RMSNORM, DC_K_GEMV_QKV, DC_K_QKROPE, DC_K_ATTENTION, DC_K_GEMV_O, DC_K_ROUTER, DC_K_MOE_GATEUP,
     DC_K_QUANT_H, DC_K_MOE_DOWN, DC_K_COMBINE, DC_K_ALLREDUCE, DC_K_FFN_GATEUP, DC_K_FFN_DOWN, DC_K_LM_HEAD, DC_K_ARGMAX,
+    DC_K_MIX_IN, DC_K_MIX_OUT, DC_K_MIX_DELTA, DC_K_MIX_SSD, DC_K_MIX_LATENT, DC_K_POST_NORM,
     DC_K_COUNT
 };
 
@@ -41,6 +42,7 @@ struct dc_graph {
 };
 
 struct dc_prefill_buffers;
+struct dc_stack;
 
 struct dc_model {
     dc_ctx* ctx = nullptr;
@@ -83,6 +85,7 @@ struct dc_model {
     int prefill_chunk = 2048;
     bool prefill_flash = true;            // option "prefill_attention": 1 tensor-core flash attention, 0 the decode kernels' exact chain
     dc_prefill_buffers* prefill = nullptr;
+    dc_stack* stack = nullptr;            // layer-list decoders (dc_stack.h); null for the K-quant decoders of this file
     bool prefix_cache = false;            // option "prefix_cache": prefill looks up and registers block prefixes
     uint64_t prefill_tokens_run = 0;      // prompt tokens that went through the decoder (cached ones do not)
     // expert parallel
@@ -99,23 +102,26 @@ struct dc_model {
 };
 
 // ---- synth.cu ----
-int dc_launch_synth_quantized(dc_ctx* ctx, int type, uint64_t seed, int64_t first_row, int64_t rows, int64_t K, float sigma,
+DC_PART int dc_launch_synth_quantized(dc_ctx* ctx, int type, uint64_t seed, int64_t first_row, int64_t rows, int64_t K, float sigma,
                               uint8_t* out);
-int dc_launch_synth_f32(dc_ctx* ctx, uint64_t seed, int64_t n, float sigma, float offset, float* out);
+DC_PART int dc_launch_synth_f32(dc_ctx* ctx, uint64_t seed, int64_t n, float sigma, float offset, float* out);
 // ---- mega.cu ----
-void dc_mega_release_xch(dc_model* m);
-int dc_mega_test_loopback(dc_model* m);
+DC_PART void dc_mega_release_xch(dc_model* m);
+DC_PART int dc_mega_test_loopback(dc_model* m);
 struct MegaParams;
-bool dc_mega_plan(dc_model* m, int T, MegaParams* out, const char** why);
-int dc_mega_run(dc_model* m, int T, int n_steps, bool feedback);
+DC_PART bool dc_mega_plan(dc_model* m, int T, MegaParams* out, const char** why);
+DC_PART int dc_mega_run(dc_model* m, int T, int n_steps, bool feedback);
 // Appends tokens[0..n) to a sequence in chunks; if `final`, the last chunk also picks the next token (and leaves
 // its logits in the step buffer) and *next_token receives it after a synchronize.
 int dc_model_prefill_range(dc_model* m, int seq, const int32_t* tokens_host, int n, bool final, int32_t* next_token);
-int dc_mega_prepare(dc_model* m);
+int dc_model_check_entry(dc_model* m, int seq, const int32_t* tokens, int n);
+int dc_model_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, int n_rows, const int32_t* rows,
+                   float* logits_host, int32_t* picks_host);
+DC_PART int dc_mega_prepare(dc_model* m);
 // ---- prefill.cu ----
-bool dc_prefill_tc_ok(dc_model* m, int n);
-int dc_prefill_chunk_tc(dc_model* m, int seq, const int32_t* tokens, int n, bool lm);
-void dc_prefill_release(dc_model* m);
+DC_PART bool dc_prefill_tc_ok(dc_model* m, int n);
+DC_PART int dc_prefill_chunk_tc(dc_model* m, int seq, const int32_t* tokens, int n, bool lm);
+DC_PART void dc_prefill_release(dc_model* m);
 // ---- ep.cu ----
-int dc_ep_allreduce(dc_model* m, float* buf, size_t n);
-void dc_ep_destroy(dc_model* m);
+DC_PART int dc_ep_allreduce(dc_model* m, float* buf, size_t n);
+DC_PART void dc_ep_destroy(dc_model* m);

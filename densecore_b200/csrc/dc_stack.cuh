@@ -1,0 +1,43 @@
+// Scalar device functions of the layer-list decoders' kernels (f32 throughout).
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+namespace dc {
+
+__device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ unsigned long long argmax_key(float f, int row) {
+    uint32_t u = __float_as_uint(f);
+    u = (f != f) ? 0u : ((u & 0x80000000u) ? ~u : (u | 0x80000000u));
+    return ((unsigned long long)u << 32) | (0xFFFFFFFFu - (uint32_t)row);
+}
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+// Sum over a CTA of up to 1024 threads; red: 33 floats of shared memory.  Every thread gets the result.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    if (threadIdx.x < 32) {
+        float s = threadIdx.x < (blockDim.x >> 5) ? red[threadIdx.x] : 0.0f;
+        s = warp_sum(s);
+        if (threadIdx.x == 0) red[32] = s;
+    }
+    __syncthreads();
+    return red[32];
+}
+__device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float load_as(const float* p) { return *p; }
+__device__ __forceinline__ float load_as(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+
+}  // namespace dc

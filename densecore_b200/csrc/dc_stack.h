@@ -1,0 +1,218 @@
+// Layer-list decoders: models whose config.json names the mixer and the feed-forward of every layer.  A model
+// is a list of layers built from the mechanisms below; every size and constant is a field, so that a design is
+// a line in the architecture table (stack_config.cu) and not a forward pass of its own.
+//
+// Numbers: weights are bf16 in HBM; the residual, norms, decays, gates, recurrent state and attention scores are
+// f32.  Steps of up to DC_MAX_T tokens, and every step of an f32 model, keep activations in f32 all the way
+// (row-streaming products); larger steps of a bf16 model round the inputs of matrix products to bf16 and run
+// them on the tensor cores.
+#pragma once
+#include <cuda.h>
+#include <cuda_bf16.h>
+
+#include <map>
+#include <string>
+#include <vector>
+
+#include "dc_internal.h"
+#include "dc_json.h"
+#include "dc_kv.h"
+
+struct dc_model;
+
+enum { DC_MIX_DELTA = 0, DC_MIX_LATENT = 1, DC_MIX_SSD = 2 };
+enum { DC_DTYPE_BF16 = 0, DC_DTYPE_F32 = 1 };
+enum { DC_LIN_STORE = 0, DC_LIN_GELU_PAIR = 1 };
+
+static inline int dc_pad8(int n) { return (n + 7) & ~7; }
+
+// Rows of one or more weight matrices that share their input, bf16, every row padded with zeros to `ld`
+// elements.  Segments start at row offsets that are multiples of eight (unused rows are zero).
+struct dc_lin {
+    __nv_bfloat16* w = nullptr;
+    int N = 0, K = 0, ld = 0;
+    CUtensorMap map;            // [N rows][K], box 128 x 64, 128-byte swizzle
+};
+
+// Input of a tensor-core product: a bf16 buffer [rows][ld] with the tensor map that reads its first K columns.
+struct dc_tc_in {
+    const __nv_bfloat16* x = nullptr;
+    int K = 0, ld = 0;
+    CUtensorMap map;            // box 128 x 64
+};
+
+struct dc_delta_mixer {         // gated delta rule with one decay per key channel
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 0, a_rank = 0, g_rank = 0;
+    float unit_eps = 1e-6f, q_scale = 1.0f;
+    dc_lin in, a2, g2, o;       // in: q | k | v | b | a1 | g1
+    int off_q = 0, off_k = 0, off_v = 0, off_b = 0, off_a = 0, off_g = 0;
+    float *conv = nullptr;      // [C][taps], C = q, k and v channels
+    float *neg_a = nullptr;     // [heads]: -exp(A_log)
+    float *dt_bias = nullptr;   // [heads * dim]
+    float *norm = nullptr;      // [vdim]
+};
+
+struct dc_ssd_mixer {           // Mamba-2
+    int heads = 0, vdim = 0, state = 0, groups = 0, norm_groups = 0, taps = 0;
+    dc_lin in, o;               // in: z | x B C | dt
+    int off_z = 0, off_x = 0, off_dt = 0;
+    float *conv = nullptr, *conv_b = nullptr, *neg_a = nullptr, *dt_bias = nullptr, *D = nullptr, *norm = nullptr;
+};
+
+struct dc_latent_mixer {        // attention over a compressed key/value latent with a shared rotated key part
+    int heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0, window = 0;   // window 0: every earlier token
+    int kv_from = -1;           // layer whose cached latent this layer reads (-1: its own)
+    float scale = 1.0f;
+    double rot_base = 10000.0;
+    dc_lin in, ukv, o;          // in: q | c and rotated key part;  ukv: per head uk, then per head uv (rows padded to 8)
+    int off_q = 0, off_kv = 0, dim_p = 0, vdim_p = 0, uv_row = 0;
+    float* kv_norm = nullptr;   // [kv_rank]
+    const float* cos_sin = nullptr;   // [max_ctx][rot_dim / 2][2]
+    int plane = -1;             // cache plane read (and, without kv_from, written)
+    int row = 0;                // elements per cached token
+    int range = 0;              // which of the step's key ranges (distinct windows)
+};
+
+struct dc_stack_layer {
+    int kind = DC_MIX_DELTA;
+    dc_delta_mixer dl;
+    dc_ssd_mixer ssd;
+    dc_latent_mixer la;
+    size_t state_off = 0, ring_off = 0;   // byte offsets in a sequence's state slot
+    int ff = 0;                 // 0: no feed-forward
+    dc_lin gate_up, down;       // gate_up: rows 2i = gate row i, 2i + 1 = up row i
+    float *norm1 = nullptr, *norm2 = nullptr;
+};
+
+// Where a named tensor goes: rows of a dc_lin, or a vector of floats.
+struct dc_stack_tensor {
+    std::string name;
+    std::vector<int64_t> shape;
+    dc_lin* lin = nullptr;
+    int row0 = 0, row_step = 1; // destination row of tensor row i: row0 + i * row_step (head_rows 0) ...
+    int head_rows = 0, head_pad = 0;      // ... or row0 + (i / head_rows) * head_pad + i % head_rows
+    float** vec = nullptr;
+    int64_t vec_off = 0, vec_len = 0;     // destination range and the vector's whole length
+    bool neg_exp = false;       // stored as -exp(value)
+    bool loaded = false;
+    int synth = 0;              // random-weight kind: 0 matrix, 1 norm weight, 2 decay exponent, 3 step bias, 4 small vector
+};
+
+struct dc_stack_config {
+    std::string arch;
+    int vocab = 0, width = 0;
+    float eps = 1e-5f;
+};
+
+// One step's tokens on the device.  Entry e is tokens starts[e] .. starts[e + 1] - 1, consecutive positions of one
+// sequence.
+struct dc_step {
+    int T = 0, E = 0;
+    const int32_t *tokens = nullptr, *seq_ids = nullptr, *positions = nullptr, *starts = nullptr;
+    bool tc = false;            // matrix products on the tensor cores (bf16 inputs)
+    bool single = false;        // every entry is one token
+};
+
+struct dc_stack_buffers {
+    int cap = 0;                // tokens of a step
+    int key_cap = 0;            // gathered keys of a step
+    int32_t* meta = nullptr;    // device copy of one step's metadata
+    int32_t* h_meta = nullptr;  // pinned, DC_STACK_META_SLOTS slots
+    int meta_ints = 0, meta_slot = 0;
+    int32_t *iota = nullptr, *chunk = nullptr;   // constant entry starts: one token each; one entry of n tokens at chunk + 2 n
+    float *x = nullptr, *y = nullptr, *proj = nullptr, *act = nullptr, *scan = nullptr, *low = nullptr, *gate = nullptr, *small = nullptr;
+    float *mix = nullptr, *ff = nullptr, *lm_x = nullptr;
+    __nv_bfloat16 *xb = nullptr, *mixb = nullptr, *ffb = nullptr, *lowb = nullptr;
+    __nv_bfloat16 *keys_c = nullptr, *keys_r = nullptr, *keys_kv = nullptr;
+    float *qa = nullptr, *part = nullptr, *part_ml = nullptr;
+    std::vector<void*> owned;
+};
+#define DC_STACK_META_SLOTS 4
+
+struct dc_stack {
+    dc_stack_config cfg;
+    int dtype = DC_DTYPE_BF16;
+    std::vector<dc_stack_layer> layers;
+    dc_weight* embed = nullptr;
+    dc_lin head;
+    float* final_norm = nullptr;
+    std::vector<dc_stack_tensor> tensors;
+    std::map<std::string, int> index;
+    std::vector<void*> owned;   // weight memory
+    size_t weight_bytes = 0;
+    std::map<std::pair<double, int>, float*> rot;    // (base, dims) -> cos/sin table
+    std::vector<int> windows;   // distinct windows of the attention layers
+    int splits = 1;             // key splits of a decode step's attention
+    dc_stack_buffers b;
+    std::map<std::pair<const void*, int>, dc_tc_in> ins;
+};
+
+// ---- stack_config.cu: architecture table, config.json -> layers and tensor slots
+int dc_stack_parse(dc_model* m, const dc_json& config, const std::map<std::string, std::vector<int64_t>>& shapes);
+// ---- stack.cu
+int dc_stack_finalize(dc_model* m);
+void dc_stack_release(dc_model* m);
+int dc_stack_set_tensor(dc_model* m, const char* name, int type, const int64_t ne[4], const void* data);
+int dc_stack_init_synthetic(dc_model* m, uint64_t seed, float sigma);
+int dc_stack_create_cache(dc_model* m, int pool_tokens);
+// a step of up to DC_MAX_T tokens whose inputs are in the model's step buffers: one token per sequence, or (chunk)
+// consecutive tokens of one sequence
+int dc_stack_enqueue_small(dc_model* m, int T, bool chunk, int lm_mode, bool feedback);
+// entries of any length as one batch: counts[e] next tokens of seqs[e].  rows: places (flat token index, ascending)
+// whose logits are wanted; logits_host / picks_host may be null.
+int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, int n_rows,
+                   const int32_t* rows, float* logits_host, int32_t* picks_host);
+void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token);
+
+// ---- linear.cu / linear_tc.cu: y = W x
+// T <= DC_MAX_T tokens, f32 inputs: one pass over the weights.  keys: packed greedy picks per token.
+int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo,
+                          unsigned long long* keys = nullptr);
+// any T, f32 inputs (f32 models)
+int dc_launch_linear_f32(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo);
+// any T, bf16 inputs on the tensor cores; exactly one of out / outb is used
+int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, int epi, float* out, __nv_bfloat16* outb, int ldo);
+int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int rows, int K, int ld);
+
+// ---- norm_act.cu
+// x += rms(y) * w per token; xb (optional): bf16 copy of the new x
+int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, int T, int H, int ld, float eps, __nv_bfloat16* xb);
+// out[r] = rms(x[rows ? rows[r] : first + r]) * w
+int dc_launch_norm_rows(dc_ctx* ctx, const float* x, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps,
+                        float* out, int ldo);
+
+// ---- mix_recur.cu
+struct dc_state_ref {           // per-sequence state in the cache manager's slots
+    uint8_t* base = nullptr;
+    size_t slot_bytes = 0, state_off = 0, ring_off = 0;
+};
+int dc_launch_delta_prep(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp,
+                         float* act, int lda, float* small, __nv_bfloat16* lowb, int ldl);
+int dc_launch_delta_scan(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act, int lda,
+                         const float* small, float* decay, int ldd, const float* raw_g, int ldg, float eps, float* o,
+                         float* mix, __nv_bfloat16* mixb, int ldm);
+int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp,
+                           float eps, float* mix, int ldm);
+int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* act,
+                  int lda, float* small, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
+int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y,
+                         float eps, float* mix, int ldm);
+int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps);
+
+// ---- mix_latent.cu
+struct dc_latent_cache {
+    void* arena = nullptr;      // [block][DC_KV_BLOCK][row], bf16 or f32
+    bool f32 = false;
+    const int32_t* tables = nullptr;
+    int max_blocks = 0;
+};
+int dc_launch_latent_prep(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, float* proj, int ldp, float eps,
+                          int max_pos);
+int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const float* proj, int ldp,
+                              int splits, float* qa, float* part, float* part_ml, float* mix, int ldm);
+int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const int32_t* key_base,
+                            int n_keys, __nv_bfloat16* keys_c, int ldc, __nv_bfloat16* keys_r, int ldr);
+int dc_launch_latent_prefill(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const int32_t* key_base, const int32_t* tiles,
+                             int n_tiles, const float* proj, int ldp, const __nv_bfloat16* keys_kv, int ldkv, const __nv_bfloat16* keys_r,
+                             int ldr, __nv_bfloat16* mixb, int ldm);
+#define DC_LATENT_QTILE 64      // queries per tile of the prompt attention

@@ -35,6 +35,7 @@
 #include "dc_common.cuh"
 #include "dc_gemm_tc.h"
 #include "dc_internal.h"
+#include "dc_tcgen05.cuh"
 
 #define DC_TRY(expr)                       \
     do {                                   \
@@ -72,20 +73,6 @@ struct GemmTcParams {
     int* err;
 };
 
-// ---- tcgen05 wrappers -------------------------------------------------------------------------------
-__device__ __forceinline__ void tmem_alloc(uint32_t smem_slot, uint32_t ncols) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_slot), "r"(ncols) : "memory");
-}
-__device__ __forceinline__ void tmem_relinquish() { asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t ncols) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-__device__ __forceinline__ void umma_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
 // D[128 x N] (+)= A[128 x 32] * B[32 x N], 8-bit operands from shared memory, int32 accumulators in TMEM.
 __device__ __forceinline__ void umma_i8(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
     asm volatile(
@@ -94,26 +81,9 @@ __device__ __forceinline__ void umma_i8(uint32_t tmem_d, uint64_t desc_a, uint64
         ::"r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
         : "memory");
 }
-// Shared-memory operand descriptor, K-major rows of 128 bytes with the 128-byte swizzle (8-row groups of 1024
-// bytes, 1024-byte aligned; chunk c of row r at chunk position c ^ (r % 8)).  saddr = the tile's base plus the
-// K offset of the instruction in bytes (32 per K-step); sbo = byte distance between 8-row groups.
-__device__ __forceinline__ uint64_t umma_desc_sw128(uint32_t saddr, uint32_t sbo) {
-    const uint32_t lo = ((saddr >> 4) & 0x3FFFu) | (1u << 16);                 // leading byte offset: unused with a swizzle
-    const uint32_t hi = ((sbo >> 4) & 0x3FFFu) | (1u << 14) | (2u << 29);      // version 1 (sm_100), SWIZZLE_128B
-    return ((uint64_t)hi << 32) | lo;
-}
 // Instruction descriptor: int32 accumulate, A unsigned or signed 8-bit, B signed 8-bit, both K-major.
 __host__ __device__ constexpr uint32_t umma_idesc_i8(int a_signed, int M, int N) {
     return (2u << 4) | ((uint32_t)a_signed << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
-}
-// 16 consecutive 32-bit columns of this thread's TMEM lane.
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, int (&v)[16]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
-        : "r"(taddr)
-        : "memory");
 }
 // Packed single precision (two lanes per instruction), each lane rounded to nearest like the scalar
 // instruction, never contracted with a neighbouring operation.
@@ -139,14 +109,6 @@ __device__ __forceinline__ float2 fma2_rn(float2 a, float2 b, float2 c) {
         : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
     return r;
 }
-// 8 consecutive 32-bit columns of this thread's TMEM lane.
-__device__ __forceinline__ void tmem_ld8(uint32_t taddr, int (&v)[8]) {
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
-                 : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7])
-                 : "r"(taddr)
-                 : "memory");
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void sts128(uint32_t a, uint32_t x, uint32_t y, uint32_t z, uint32_t w) {
     asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(a), "r"(x), "r"(y), "r"(z), "r"(w) : "memory");
 }
@@ -221,15 +183,6 @@ constexpr int TC_N = 128;                  // tokens per CTA
 // indexed with run-time values)
 enum TcBar { A_FULL = 0, A_FREE = 4, B_FULL = 8, B_FREE = 10, S_FULL = 12, D_FULL = 16, ACC_FULL = 20, ACC_FREE = 22, TC_NBARS = 24 };
 
-__device__ __forceinline__ bool tc_wait_raw(uint32_t bar, uint32_t parity, volatile int* give_up, int* err) {
-    for (uint32_t i = 0; i < DC_WAIT_LIMIT; ++i) {
-        if (mbar_try_wait(bar, parity)) return true;
-        if ((i & 63u) == 63u && *give_up) return false;
-    }
-    *give_up = 1;
-    if (err) atomicExch(err, DC_ERR_MBAR_TIMEOUT);
-    return false;
-}
 #ifdef DC_TC_TIMING
 // instrumented build: cycles one thread of every role spends in each kind of wait, summed over CTAs
 // 0 a_free (expander)  1 b_full  2 a_full  3 acc_free (issuer)  4 b_free (loader)  5 d/s_full  6 acc_full (read-out)
@@ -244,10 +197,6 @@ __device__ __forceinline__ bool tc_wait_k(int kind, uint32_t bar, uint32_t parit
 #else
 #define tc_wait_k(kind, bar, parity, give_up, err) tc_wait_raw(bar, parity, give_up, err)
 #endif
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-
 template <int TYPE>
 constexpr size_t tc_smem_bytes() {
     using T = TcTraits<TYPE>;

@@ -9,25 +9,15 @@
 #include "dc_internal.h"
 #include "dc_kv.h"
 
-int dc_kv_init(dc_ctx* ctx, dc_kv_cache* kv, int n_layer, int n_kv_head, int head_dim, int max_blocks, int max_seqs,
-               int max_blocks_per_seq) {
-    if (n_layer <= 0 || n_kv_head <= 0 || head_dim != 128 || max_blocks <= 0 || max_seqs <= 0 || max_blocks_per_seq <= 0)
-        return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "kv_create: bad shape (head_dim must be 128)");
+// Block manager and device block tables.
+static int init_manager(dc_ctx* ctx, dc_kv_cache* kv, int max_blocks, int max_seqs, int max_blocks_per_seq) {
     kv->ctx = ctx;
-    kv->n_layer = n_layer;
-    kv->n_kv = n_kv_head;
-    kv->head_dim = head_dim;
     kv->max_blocks = max_blocks;
     kv->max_seqs = max_seqs;
     kv->max_blocks_per_seq = max_blocks_per_seq;
-    kv->layer_elems = (size_t)max_blocks * DC_KV_BLOCK * n_kv_head * head_dim;
-    const size_t bytes = kv->layer_elems * n_layer * sizeof(__half);
-    cudaError_t e = cudaMalloc(&kv->k_arena, bytes);
-    if (e == cudaSuccess) e = cudaMalloc(&kv->v_arena, bytes);
-    if (e == cudaSuccess) e = cudaMalloc(&kv->d_tables, (size_t)max_seqs * max_blocks_per_seq * sizeof(int32_t));
-    if (e == cudaSuccess) e = cudaMemsetAsync(kv->k_arena, 0, bytes, ctx->stream);
-    if (e == cudaSuccess) e = cudaMemsetAsync(kv->v_arena, 0, bytes, ctx->stream);
-    if (e == cudaSuccess) e = cudaMemsetAsync(kv->d_tables, 0, (size_t)max_seqs * max_blocks_per_seq * sizeof(int32_t), ctx->stream);
+    const size_t table_bytes = (size_t)max_seqs * max_blocks_per_seq * sizeof(int32_t);
+    cudaError_t e = cudaMalloc(&kv->d_tables, table_bytes);
+    if (e == cudaSuccess) e = cudaMemsetAsync(kv->d_tables, 0, table_bytes, ctx->stream);
     if (e != cudaSuccess) return dc_check_cuda(ctx, e, "kv_create");
     kv->free_list.clear();
     for (int b = max_blocks - 1; b >= 0; --b) kv->free_list.push_back(b);
@@ -38,6 +28,43 @@ int dc_kv_init(dc_ctx* ctx, dc_kv_cache* kv, int n_layer, int n_kv_head, int hea
     kv->block_tokens.assign(max_blocks, std::array<int32_t, 16>());
     kv->block_used.assign(max_blocks, 0);
     return DC_B200_OK;
+}
+
+int dc_kv_init(dc_ctx* ctx, dc_kv_cache* kv, int n_layer, int n_kv_head, int head_dim, int max_blocks, int max_seqs,
+               int max_blocks_per_seq) {
+    if (n_layer <= 0 || n_kv_head <= 0 || head_dim != 128 || max_blocks <= 0 || max_seqs <= 0 || max_blocks_per_seq <= 0)
+        return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "kv_create: bad shape (head_dim must be 128)");
+    kv->n_layer = n_layer;
+    kv->n_kv = n_kv_head;
+    kv->head_dim = head_dim;
+    kv->layer_elems = (size_t)max_blocks * DC_KV_BLOCK * n_kv_head * head_dim;
+    const size_t bytes = kv->layer_elems * n_layer * sizeof(__half);
+    cudaError_t e = cudaMalloc(&kv->k_arena, bytes);
+    if (e == cudaSuccess) e = cudaMalloc(&kv->v_arena, bytes);
+    if (e == cudaSuccess) e = cudaMemsetAsync(kv->k_arena, 0, bytes, ctx->stream);
+    if (e == cudaSuccess) e = cudaMemsetAsync(kv->v_arena, 0, bytes, ctx->stream);
+    if (e != cudaSuccess) return dc_check_cuda(ctx, e, "kv_create");
+    return init_manager(ctx, kv, max_blocks, max_seqs, max_blocks_per_seq);
+}
+
+int dc_kv_init_planes(dc_ctx* ctx, dc_kv_cache* kv, const std::vector<size_t>& row_bytes, size_t state_bytes, int max_blocks, int max_seqs,
+                      int max_blocks_per_seq) {
+    if (max_blocks <= 0 || max_seqs <= 0 || max_blocks_per_seq <= 0) return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "kv: bad pool size");
+    kv->planes.resize(row_bytes.size());
+    for (size_t i = 0; i < row_bytes.size(); ++i) {
+        const size_t bytes = row_bytes[i] * max_blocks * DC_KV_BLOCK;
+        kv->planes[i].row_bytes = row_bytes[i];
+        cudaError_t e = cudaMalloc(&kv->planes[i].arena, bytes);
+        if (e == cudaSuccess) e = cudaMemsetAsync(kv->planes[i].arena, 0, bytes, ctx->stream);
+        if (e != cudaSuccess) return dc_check_cuda(ctx, e, "kv plane");
+    }
+    kv->state_bytes = state_bytes;
+    if (state_bytes) {
+        cudaError_t e = cudaMalloc(&kv->state, state_bytes * max_seqs);
+        if (e == cudaSuccess) e = cudaMemsetAsync(kv->state, 0, state_bytes * max_seqs, ctx->stream);
+        if (e != cudaSuccess) return dc_check_cuda(ctx, e, "kv state slots");
+    }
+    return init_manager(ctx, kv, max_blocks, max_seqs, max_blocks_per_seq);
 }
 
 // Blocks an allocation can get: the free list plus cached blocks that only the prefix cache still holds.
@@ -73,6 +100,11 @@ void dc_kv_release(dc_kv_cache* kv) {
     if (kv->k_arena) cudaFree(kv->k_arena);
     if (kv->v_arena) cudaFree(kv->v_arena);
     if (kv->d_tables) cudaFree(kv->d_tables);
+    for (auto& p : kv->planes)
+        if (p.arena) cudaFree(p.arena);
+    kv->planes.clear();
+    if (kv->state) cudaFree(kv->state);
+    kv->state = nullptr;
     kv->k_arena = kv->v_arena = nullptr;
     kv->d_tables = nullptr;
 }
@@ -141,6 +173,9 @@ int dc_kv_seq_fork(dc_kv_cache* kv, int src_seq, int* out_seq) {
     kv->seqs[dst].len = kv->seqs[src_seq].len;
     for (int b : kv->seqs[dst].blocks) ++kv->ref[b];
     st = upload_table(kv, dst, 0, (int)kv->seqs[dst].blocks.size());
+    if (st == DC_B200_OK && kv->state_bytes)
+        st = dc_check_cuda(kv->ctx, cudaMemcpyAsync(kv->state + (size_t)dst * kv->state_bytes, kv->state + (size_t)src_seq * kv->state_bytes,
+                                                    kv->state_bytes, cudaMemcpyDeviceToDevice, kv->ctx->stream), "kv: state copy");
     if (st != DC_B200_OK) {
         dc_kv_seq_free(kv, dst);
         return st;
@@ -169,8 +204,14 @@ int dc_kv_seq_reserve(dc_kv_cache* kv, int seq, int n_tokens) {
         if (fresh < 0) return dc_fail(kv->ctx, DC_B200_OUT_OF_MEMORY, "kv: out of blocks (copy-on-write)");
         --kv->ref[old];
         const size_t be = (size_t)DC_KV_BLOCK * kv->n_kv * kv->head_dim;
-        k_kv_copy_block<<<dim3(kv->n_layer, 2), 256, 0, kv->ctx->stream>>>(kv->k_arena, kv->v_arena, kv->layer_elems, be, old, fresh);
+        if (kv->n_layer > 0)
+            k_kv_copy_block<<<dim3(kv->n_layer, 2), 256, 0, kv->ctx->stream>>>(kv->k_arena, kv->v_arena, kv->layer_elems, be, old, fresh);
         int st = dc_check_cuda(kv->ctx, cudaGetLastError(), "k_kv_copy_block");
+        for (auto& p : kv->planes) {
+            const size_t b = p.row_bytes * DC_KV_BLOCK;
+            if (st == DC_B200_OK)
+                st = dc_check_cuda(kv->ctx, cudaMemcpyAsync(p.arena + b * fresh, p.arena + b * old, b, cudaMemcpyDeviceToDevice, kv->ctx->stream), "kv: block copy");
+        }
         if (st != DC_B200_OK) return st;
         s.blocks[lb] = fresh;
         st = upload_table(kv, seq, lb, 1);
@@ -207,6 +248,7 @@ int dc_kv_prefix_attach(dc_kv_cache* kv, int seq, const int32_t* tokens, int n_t
     if (s.len != 0 || !s.blocks.empty())
         return dc_fail(kv->ctx, DC_B200_INVALID_ARGUMENT, "kv: prefix lookup needs an empty sequence (sequence %d holds %d tokens)", seq, s.len);
     ++kv->prefix_lookups;
+    if (kv->state_bytes) return DC_B200_OK;     // cached blocks alone do not bring a recurrent state back
     if (!tokens || n_tokens <= DC_KV_BLOCK) return DC_B200_OK;
     int reusable = (n_tokens - 1) / DC_KV_BLOCK * DC_KV_BLOCK;
     if (reusable > kv->max_blocks_per_seq * DC_KV_BLOCK) reusable = kv->max_blocks_per_seq * DC_KV_BLOCK;
@@ -234,6 +276,7 @@ int dc_kv_prefix_attach(dc_kv_cache* kv, int seq, const int32_t* tokens, int n_t
 int dc_kv_prefix_register(dc_kv_cache* kv, int seq, const int32_t* tokens, int n_tokens) {
     if (seq < 0 || seq >= kv->max_seqs || !kv->seqs[seq].used || !tokens)
         return dc_fail(kv->ctx, DC_B200_INVALID_ARGUMENT, "kv: sequence %d is not allocated", seq);
+    if (kv->state_bytes) return DC_B200_OK;
     dc_kv_seq& s = kv->seqs[seq];
     if (n_tokens > s.len) n_tokens = s.len;
     uint64_t h = 14695981039346656037ULL;

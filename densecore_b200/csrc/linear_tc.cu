@@ -1,0 +1,167 @@
+// bf16 products y = W x for prompt-sized steps on the 5th-generation tensor cores.
+//
+// One CTA per 128 weight rows x 128 tokens: one thread keeps a ring of shared-memory stages full with tiled TMA
+// loads (64 columns of both operands, 128-byte swizzle), one thread issues the UMMAs (128 x 128 x 16, f32
+// accumulators in tensor memory), four warps read the accumulators out.  A weight row is a tensor-memory lane, so
+// a warp's stores of one token are 32 consecutive outputs.  Two CTAs share an SM: one's read-out overlaps the
+// other's products.  Columns beyond K and rows beyond the matrix are the zeros that TMA fills in.  Every wait is
+// bounded; a CTA that gives up drains its copies, frees its tensor memory and leaves.
+#include "dc_common.cuh"
+#include "dc_launch.cuh"
+#include "dc_stack.h"
+#include "dc_stack.cuh"
+#include "dc_tcgen05.cuh"
+
+using namespace dc;
+
+namespace {
+
+constexpr int LT_STAGES = 3, LT_TILE = 128 * 128;   // bytes of one operand of a stage: 128 rows of 64 bf16
+constexpr int LT_THREADS = 192;
+constexpr size_t LT_SMEM = (size_t)LT_STAGES * 2 * LT_TILE + 1024;
+
+struct LtParams {
+    int K, T, n_out, ldo, epi;
+    float* out;
+    __nv_bfloat16* outb;
+    int* err;
+};
+
+__global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_constant__ CUtensorMap wmap,
+                                                             const __grid_constant__ CUtensorMap xmap, const LtParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t s_bar[2 * LT_STAGES + 1];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_give_up;
+    pdl_launch_dependents();
+    const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+    const uint32_t full = smem_u32(s_bar), empty = full + 8 * LT_STAGES, acc = empty + 8 * LT_STAGES;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int row0 = blockIdx.x * 128, t0 = blockIdx.y * 128;
+    const int nk = (p.K + 63) / 64;
+    volatile int* give_up = &s_give_up;
+    if (warp == 1) {
+        tmem_alloc(smem_u32(&s_tmem), 128);
+        tmem_relinquish();
+    }
+    if (tid == 0) {
+        s_give_up = 0;
+        for (int i = 0; i < LT_STAGES; ++i) {
+            mbar_init(full + 8 * i, 1);
+            mbar_init(empty + 8 * i, 1);
+        }
+        mbar_init(acc, 1);
+        mbar_fence_init();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s_tmem;
+    pdl_wait();
+    if (warp == 0) {
+        if (lane == 0) {
+            int issued = 0;
+            for (; issued < nk; ++issued) {
+                const int s = issued % LT_STAGES, use = issued / LT_STAGES;
+                if (use > 0 && !tc_wait_raw(empty + 8 * s, (use - 1) & 1, give_up, p.err)) break;
+                mbar_expect_tx(full + 8 * s, 2 * LT_TILE);
+                tma_load_2d(base + s * 2 * LT_TILE, &wmap, issued * 64, row0, full + 8 * s);
+                tma_load_2d(base + s * 2 * LT_TILE + LT_TILE, &xmap, issued * 64, t0, full + 8 * s);
+            }
+            // no copy may still be in flight when the CTA leaves (at once unless someone gave up)
+            for (int s = 0; s < LT_STAGES; ++s) {
+                const int uses = (issued - s + LT_STAGES - 1) / LT_STAGES;
+                if (issued > s)
+                    for (uint32_t i = 0; i < DC_WAIT_LIMIT && !mbar_try_wait(full + 8 * s, (uses - 1) & 1); ++i) {}
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc = umma_idesc_bf16(128, 128);
+            for (int k = 0; k < nk; ++k) {
+                const int s = k % LT_STAGES;
+                if (!tc_wait_raw(full + 8 * s, (k / LT_STAGES) & 1, give_up, p.err)) break;
+                tc_fence_after();
+                const uint32_t a = base + s * 2 * LT_TILE, b = a + LT_TILE;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) umma_f16(tmem, umma_desc_sw128(a + 32 * j, 1024), umma_desc_sw128(b + 32 * j, 1024), idesc, k > 0 || j > 0);
+                umma_commit(empty + 8 * s);
+            }
+            umma_commit(acc);
+        }
+    } else {
+        const bool ok = tc_wait_raw(acc, 0, give_up, p.err) && !*give_up;
+        tc_fence_after();
+        if (__all_sync(0xffffffffu, ok)) {
+            const int quarter = warp & 3, row = row0 + 32 * quarter + lane;
+            for (int c0 = 0; c0 < 128 && t0 + c0 < p.T; c0 += 16) {
+                int v[16];
+                tmem_ld16(tmem + ((uint32_t)(32 * quarter) << 16) + c0, v);
+                tmem_ld_wait();
+                if (p.epi == DC_LIN_GELU_PAIR) {
+                    // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
+                    const bool up = lane & 1;
+                    const int o = row >> 1;
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
+                        const float mine = __int_as_float(up ? v[i + 8] : v[i]);
+                        const float h = up ? gelu_tanh(got) * mine : gelu_tanh(mine) * got;
+                        const int t = t0 + c0 + i + (up ? 8 : 0);
+                        if (t < p.T && o < p.n_out) {
+                            if (p.outb) p.outb[(size_t)t * p.ldo + o] = __float2bfloat16_rn(h);
+                            else p.out[(size_t)t * p.ldo + o] = h;
+                        }
+                    }
+                } else if (row < p.n_out) {
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) {
+                        const int t = t0 + c0 + i;
+                        if (t >= p.T) break;
+                        if (p.outb) p.outb[(size_t)t * p.ldo + row] = __float2bfloat16_rn(__int_as_float(v[i]));
+                        else p.out[(size_t)t * p.ldo + row] = __int_as_float(v[i]);
+                    }
+                }
+            }
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 1) tmem_dealloc(tmem, 128);
+}
+
+typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                             const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+EncodeFn encode_fn() {
+    static EncodeFn fn = [] {
+        void* f = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &f, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) f = nullptr;
+        return (EncodeFn)f;
+    }();
+    return fn;
+}
+
+}  // namespace
+
+// Tensor map of a bf16 matrix [rows][ld] whose first K columns count: boxes of 128 rows x 64 columns.
+int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int rows, int K, int ld) {
+    EncodeFn f = encode_fn();
+    if (!f) return dc_fail(ctx, DC_B200_BACKEND_ERROR, "the driver has no cuTensorMapEncodeTiled");
+    const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {64, 128}, es[2] = {1, 1};
+    const CUresult r = f(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void*)base, dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? DC_B200_OK : dc_fail(ctx, DC_B200_BACKEND_ERROR, "cuTensorMapEncodeTiled failed (%d) for %d x %d, pitch %d", (int)r, rows, K, ld);
+}
+
+int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, int epi, float* out, __nv_bfloat16* outb, int ldo) {
+    if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: inner sizes %d and %d differ", w.K, x.K);
+    int st = dc_kernel_setup(ctx, (const void*)k_linear_tc, (int)LT_SMEM, "k_linear_tc");
+    if (st != DC_B200_OK) return st;
+    LtParams p = {w.K, T, epi == DC_LIN_GELU_PAIR ? w.N / 2 : w.N, ldo, epi, out, outb, ctx->d_err};
+    if (p.n_out > ldo) p.n_out = ldo;
+    return dc_launch(ctx, "k_linear_tc", k_linear_tc, dim3((w.N + 127) / 128, (T + 127) / 128), dim3(LT_THREADS), LT_SMEM, w.map, x.map, p);
+}

@@ -12,14 +12,14 @@ using namespace dc;
 // d*scale*(q-32) with the order of core/src/llm/matmul/q6_small_batch.h:52-74.
 __global__ void __launch_bounds__(256) k_embed(const uint8_t* __restrict__ w, int type, int row_bytes, int H,
                                                const int32_t* __restrict__ tokens, int vocab,
-                                               float* __restrict__ x) {
+                                               float* __restrict__ x, int ldx, __nv_bfloat16* __restrict__ xb) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
     int tok = tokens[t];
     if (tok < 0 || tok >= vocab) tok = 0;
     const uint8_t* row = w + (size_t)tok * row_bytes;
-    float* o = x + (size_t)t * H;
+    float* o = x + (size_t)t * ldx;
     for (int e = threadIdx.x; e < H; e += blockDim.x) {
         const int b = e >> 8, i = e & 255;
         float v;
@@ -51,15 +51,18 @@ __global__ void __launch_bounds__(256) k_embed(const uint8_t* __restrict__ w, in
             v = __fmul_rn(__fmul_rn(d, (float)sc), (float)q);
         } else if (type == DC_TYPE_F16) {
             v = fp16_bits_to_float(reinterpret_cast<const uint16_t*>(row)[e]);
+        } else if (type == DC_TYPE_BF16) {
+            v = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(row)[e]);
         } else {
             v = reinterpret_cast<const float*>(row)[e];
         }
         o[e] = v;
+        if (xb) xb[(size_t)t * ldx + e] = __float2bfloat16_rn(v);
     }
 }
 
-int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x) {
-    k_embed<<<T, 256, 0, ctx->stream>>>(w->dev, w->type, (int)w->row_bytes, (int)w->K, tokens, (int)w->N, x);
+int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x, int ldx, __nv_bfloat16* xb) {
+    k_embed<<<T, 256, 0, ctx->stream>>>(w->dev, w->type, (int)w->row_bytes, (int)w->K, tokens, (int)w->N, x, ldx ? ldx : (int)w->K, xb);
     return dc_check_cuda(ctx, cudaGetLastError(), "k_embed");
 }
 

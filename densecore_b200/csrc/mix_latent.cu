@@ -1,0 +1,551 @@
+// Attention over a compressed key/value latent (one row per token: the normed latent c and a rotated key part that
+// all heads share), with an optional sliding window.
+//
+// Decode-sized steps and f32 models use the absorbed form: a head's unrotated query is taken through its W_uk once
+// (q' = W_uk^T q), scores are q' . c + q_rot . k_rot, the softmax-weighted sum of latents goes through W_uv at the
+// end; the cache row is the key and the value of every head.  Prompt-sized steps of bf16 models gather the visible
+// rows of each entry, expand them to per-head keys and values with one tensor-core product, and run a tiled
+// attention over them.  Scores and softmax are f32 in both.
+#include "dc_common.cuh"
+#include "dc_launch.cuh"
+#include "dc_stack.h"
+#include "dc_stack.cuh"
+
+#define DC_TRY(expr)                       \
+    do {                                   \
+        int st_ = (expr);                  \
+        if (st_ != DC_B200_OK) return st_; \
+    } while (0)
+
+using namespace dc;
+
+namespace {
+
+__device__ __forceinline__ int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
+
+struct CacheRef {
+    void* arena;
+    const int32_t* tables;
+    int max_blocks, row;     // row: elements per cached token
+    __device__ size_t at(int seq, int pos) const {
+        return ((size_t)tables[(size_t)seq * max_blocks + pos / DC_KV_BLOCK] * DC_KV_BLOCK + pos % DC_KV_BLOCK) * row;
+    }
+};
+
+// ---------------------------------------------------------------- rotation, latent norm, cache write
+struct PrepParams {
+    float* proj;             // queries are turned in place
+    int ldp, off_q, off_kv, heads, dim, rot, rank, max_pos;
+    const float* norm;       // null: another layer writes the cache
+    const float* cos_sin;
+    float eps;
+    const int32_t *seq_ids, *positions;
+    CacheRef c;
+};
+
+template <typename TC>
+__global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int pos = min(max(p.positions[t], 0), p.max_pos - 1);
+    const float* cs = p.cos_sin + (size_t)pos * p.rot;
+    float* row = p.proj + (size_t)t * p.ldp;
+    const int half = p.rot / 2;
+    if (p.norm && warp == 0) {
+        const float* src = row + p.off_kv;
+        TC* dst = reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos);
+        float ss = 0.0f;
+        for (int i = lane; i < p.rank; i += 32) ss = fmaf(src[i], src[i], ss);
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.rank + p.eps);
+        for (int i = lane; i < p.rank; i += 32) store_as(dst + i, src[i] * inv * p.norm[i]);
+        for (int i = lane; i < half; i += 32) {
+            const float u = src[p.rank + 2 * i], v = src[p.rank + 2 * i + 1], c = cs[2 * i], s = cs[2 * i + 1];
+            store_as(dst + p.rank + 2 * i, u * c - v * s);
+            store_as(dst + p.rank + 2 * i + 1, v * c + u * s);
+        }
+        for (int i = p.rank + p.rot + lane; i < p.c.row; i += 32) store_as(dst + i, 0.0f);
+    }
+    for (int i = threadIdx.x; i < p.heads * half; i += 256) {
+        const int h = i / half, j = i - h * half;
+        float* q = row + p.off_q + h * (p.dim + p.rot) + p.dim + 2 * j;
+        const float u = q[0], v = q[1], c = cs[2 * j], s = cs[2 * j + 1];
+        q[0] = u * c - v * s;
+        q[1] = v * c + u * s;
+    }
+}
+
+// ---------------------------------------------------------------- absorbed form
+// qa[t][h][r] = sum_d q[t][h][d] * uk[h][d][r].  CTA: one head, 256 columns, up to NT tokens.
+template <int NT>
+__global__ void __launch_bounds__(128) k_latent_absorb(const float* __restrict__ proj, int ldp, int off_q, int heads, int dim, int rot,
+                                                       const __nv_bfloat16* __restrict__ uk, int ldw, int dim_p, int rank, int T,
+                                                       float* __restrict__ qa, int ldq) {
+    extern __shared__ float sq[];    // [NT][dim]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, tb = blockIdx.z * NT, nt = min(NT, T - tb), r = blockIdx.y * 256 + 2 * threadIdx.x;
+    for (int i = threadIdx.x; i < NT * dim; i += 128) {
+        const int t = i / dim, d = i - t * dim;
+        sq[i] = t < nt ? proj[(size_t)(tb + t) * ldp + off_q + h * (dim + rot) + d] : 0.0f;
+    }
+    __syncthreads();
+    if (r >= rank) return;
+    float a[NT][2];
+#pragma unroll
+    for (int t = 0; t < NT; ++t) a[t][0] = a[t][1] = 0.0f;
+    const __nv_bfloat16* w = uk + (size_t)h * dim_p * ldw + r;
+#pragma unroll 8
+    for (int d = 0; d < dim; ++d) {
+        const float2 wf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + (size_t)d * ldw));
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            a[t][0] = fmaf(sq[t * dim + d], wf.x, a[t][0]);
+            a[t][1] = fmaf(sq[t * dim + d], wf.y, a[t][1]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+        if (t < nt) {
+            float* o = qa + ((size_t)(tb + t) * heads + h) * ldq + r;
+            o[0] = a[t][0];
+            if (r + 1 < rank) o[1] = a[t][1];
+        }
+}
+
+__device__ __forceinline__ void unpack16(const uint4& v, float (&f)[8], __nv_bfloat16) {
+    const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        f[2 * i] = __uint_as_float(u[i] << 16);
+        f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void unpack16(const uint4& v, float (&f)[4], float) {
+    f[0] = __uint_as_float(v.x), f[1] = __uint_as_float(v.y), f[2] = __uint_as_float(v.z), f[3] = __uint_as_float(v.w);
+}
+
+struct AbsorbedParams {
+    const float* qa;         // [T][heads][ldq]
+    int ldq;
+    const float* proj;
+    int ldp, off_q, heads, dim, rot, rank, window, splits;
+    float scale;
+    const int32_t *seq_ids, *positions;
+    CacheRef c;
+    float *part, *part_ml;   // [T][heads][splits][rank], [T][heads][splits][2]
+};
+
+constexpr int AB_KEYS = 32, AB_HEADS = 8;
+
+// One CTA per (key split, group of eight heads, token): a warp is a head.  Scores: a lane is a key; sums: a lane owns
+// column pairs lane, lane + 32, ... of the latent.
+template <typename TC, int RP>
+__global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const AbsorbedParams p) {
+    constexpr int EPC = 16 / sizeof(TC);      // elements of a 16-byte chunk
+    extern __shared__ __align__(16) uint8_t sm[];
+    float* sq = reinterpret_cast<float*>(sm);                              // [AB_HEADS][row]
+    const int row = p.c.row, ldk = row + EPC;
+    TC* sk = reinterpret_cast<TC*>(sm + (size_t)AB_HEADS * row * 4);       // [AB_KEYS][ldk]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int s = blockIdx.x, h0 = blockIdx.y * AB_HEADS, t = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = h0 + warp, pos = p.positions[t], seq = p.seq_ids[t];
+    const bool live = h < p.heads;
+    for (int i = tid; i < AB_HEADS * row; i += AB_HEADS * 32) {
+        const int hh = i / row, c = i - hh * row;
+        float v = 0.0f;
+        if (h0 + hh < p.heads) {
+            if (c < p.rank) v = p.qa[((size_t)t * p.heads + h0 + hh) * p.ldq + c];
+            else if (c < p.rank + p.rot) v = p.proj[(size_t)t * p.ldp + p.off_q + (h0 + hh) * (p.dim + p.rot) + p.dim + c - p.rank];
+        }
+        sq[i] = v * p.scale;
+    }
+    const int first = first_key(pos, p.window), nk = pos - first + 1;
+    const int per = ((nk + p.splits - 1) / p.splits + AB_KEYS - 1) / AB_KEYS * AB_KEYS;
+    const int kb = first + s * per, ke = min(first + nk, kb + per);
+    float m = -INFINITY, l = 0.0f, acc[RP][2];
+#pragma unroll
+    for (int j = 0; j < RP; ++j) acc[j][0] = acc[j][1] = 0.0f;
+    const int chunks = row / EPC;
+    for (int k0 = kb; k0 < ke; k0 += AB_KEYS) {
+        __syncthreads();
+        for (int i = tid; i < AB_KEYS * chunks; i += AB_HEADS * 32) {
+            const int kk = i / chunks, c = i - kk * chunks;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (k0 + kk < ke) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const TC*>(p.c.arena) + p.c.at(seq, k0 + kk) + c * EPC);
+            *reinterpret_cast<uint4*>(sk + kk * ldk + c * EPC) = v;
+        }
+        __syncthreads();
+        if (!live) continue;
+        float sc = 0.0f;
+        const float* q = sq + warp * row;
+        for (int c = 0; c < chunks; ++c) {
+            float f[EPC];
+            unpack16(*reinterpret_cast<const uint4*>(sk + lane * ldk + c * EPC), f, TC());
+#pragma unroll
+            for (int i = 0; i < EPC; ++i) sc = fmaf(f[i], q[c * EPC + i], sc);
+        }
+        if (k0 + lane >= ke) sc = -INFINITY;
+        float mx = sc;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float mn = fmaxf(m, mx), corr = expf(m - mn), pr = expf(sc - mn);
+        m = mn;
+        l = l * corr + warp_sum(pr);
+#pragma unroll
+        for (int j = 0; j < RP; ++j) {
+            acc[j][0] *= corr;
+            acc[j][1] *= corr;
+        }
+        for (int kk = 0; kk < AB_KEYS; ++kk) {
+            const float w = __shfl_sync(0xffffffffu, pr, kk);
+            const TC* kr = sk + kk * ldk;
+#pragma unroll
+            for (int j = 0; j < RP; ++j) {
+                const int r = 2 * (lane + 32 * j);
+                if (r < p.rank) {
+                    acc[j][0] = fmaf(w, load_as(kr + r), acc[j][0]);
+                    acc[j][1] = fmaf(w, load_as(kr + r + 1), acc[j][1]);     // rank odd: the neighbour's value, never stored
+                }
+            }
+        }
+    }
+    if (!live) return;
+    const size_t o = ((size_t)t * p.heads + h) * p.splits + s;
+    if (lane == 0) {
+        p.part_ml[2 * o] = m;
+        p.part_ml[2 * o + 1] = l;
+    }
+#pragma unroll
+    for (int j = 0; j < RP; ++j) {
+        const int r = 2 * (lane + 32 * j);
+        if (r < p.rank) p.part[o * p.rank + r] = acc[j][0];
+        if (r + 1 < p.rank) p.part[o * p.rank + r + 1] = acc[j][1];
+    }
+}
+
+// Splits of one (head, token) joined, then taken through the head's W_uv.
+__global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits,
+                                                    int rank, const __nv_bfloat16* __restrict__ uv, int ldw, int vdim_p, int vdim,
+                                                    float* __restrict__ mix, int ldm) {
+    extern __shared__ __align__(16) float lat[];      // [rank padded to 8]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const size_t o = ((size_t)t * heads + h) * splits;
+    float M = -INFINITY;
+    for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[2 * (o + s)]);
+    float L = 0.0f;
+    for (int s = 0; s < splits; ++s) L += part_ml[2 * (o + s) + 1] * expf(part_ml[2 * (o + s)] - M);
+    const float inv = 1.0f / L;
+    const int rank8 = (rank + 7) & ~7;
+    for (int r = threadIdx.x; r < rank8; r += 256) {
+        float v = 0.0f;
+        if (r < rank)
+            for (int s = 0; s < splits; ++s) {
+                const float w = expf(part_ml[2 * (o + s)] - M);
+                if (w > 0.0f) v = fmaf(part[(o + s) * rank + r], w, v);     // an empty split holds nothing readable
+            }
+        lat[r] = v * inv;
+    }
+    __syncthreads();
+    for (int e = warp; e < vdim; e += 8) {
+        const uint4* w = reinterpret_cast<const uint4*>(uv + (size_t)(h * vdim_p + e) * ldw);
+        float a = 0.0f;
+        for (int c = lane; c < rank8 / 8; c += 32) {
+            float f[8];
+            unpack16(w[c], f, __nv_bfloat16());
+#pragma unroll
+            for (int i = 0; i < 8; ++i) a = fmaf(f[i], lat[8 * c + i], a);
+        }
+        a = warp_sum(a);
+        if (lane == 0) mix[(size_t)t * ldm + (size_t)h * vdim + e] = a;
+    }
+}
+
+template <typename TC>
+int launch_absorbed(dc_ctx* ctx, const AbsorbedParams& p, int T) {
+    const size_t smem = (size_t)AB_HEADS * p.c.row * 4 + (size_t)AB_KEYS * (p.c.row * sizeof(TC) + 16);
+    const dim3 grid(p.splits, (p.heads + AB_HEADS - 1) / AB_HEADS, T), block(AB_HEADS * 32);
+#define DC_AB(RP)                                                                                                     \
+    do {                                                                                                              \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_absorbed<TC, RP>, (int)smem, "k_latent_absorbed"));         \
+        return dc_launch(ctx, "k_latent_absorbed", k_latent_absorbed<TC, RP>, grid, block, smem, p);                  \
+    } while (0)
+    if (p.rank <= 64) DC_AB(1);
+    if (p.rank <= 128) DC_AB(2);
+    if (p.rank <= 256) DC_AB(4);
+    if (p.rank <= 512) DC_AB(8);
+    DC_AB(16);
+#undef DC_AB
+}
+
+// ---------------------------------------------------------------- prompt form
+// Row i of the gathered keys: the cached latent and rotated part of an entry's visible positions (from the first key
+// that its first token sees to its last token).
+__global__ void __launch_bounds__(256) k_latent_gather(CacheRef c, const int32_t* __restrict__ seq_ids, const int32_t* __restrict__ positions,
+                                                       const int32_t* __restrict__ starts, const int32_t* __restrict__ key_base, int E, int n_keys,
+                                                       int window, int rank, int rot, __nv_bfloat16* __restrict__ kc, int ldc,
+                                                       __nv_bfloat16* __restrict__ kr, int ldr) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (i >= n_keys) return;
+    int e = 0;
+    while (e + 1 < E && key_base[e + 1] <= i) ++e;
+    const int t0 = starts[e], pos = first_key(positions[t0], window) + i - key_base[e];
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(c.arena) + c.at(seq_ids[t0], pos);
+    if (rank % 8 == 0) {
+        for (int j = lane; j < rank / 8; j += 32) reinterpret_cast<uint4*>(kc + (size_t)i * ldc)[j] = reinterpret_cast<const uint4*>(src)[j];
+    } else {
+        for (int j = lane; j < rank; j += 32) kc[(size_t)i * ldc + j] = src[j];
+    }
+    for (int j = lane; j < ldr; j += 32) kr[(size_t)i * ldr + j] = j < rot ? src[rank + j] : __float2bfloat16_rn(0.0f);
+}
+
+__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool valid) {
+    const int bytes = valid ? 16 : 0;   // 0: the 16 bytes are zero-filled, the address is not read
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+
+struct PromptParams {
+    const float* proj;
+    int ldp, off_q, dim, rot, dim_p, vdim, vdim_p, uv_row, window;
+    float scale;
+    const int32_t *positions, *starts, *key_base, *tiles;    // tiles: (entry, first query of the entry) pairs
+    const __nv_bfloat16* kv;
+    int ldkv;
+    const __nv_bfloat16* kr;
+    int ldr, dq;             // dq: padded key length (dim_p + ldr, up to a multiple of 16)
+    __nv_bfloat16* out;
+    int ldm;
+};
+
+constexpr int PQ = DC_LATENT_QTILE, PK = 64;
+
+// One CTA per (64 queries of one entry, head).  VD: value columns, padded.
+template <int VD>
+__global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
+    constexpr int LDV = VD + 8;
+    extern __shared__ __align__(16) uint8_t smem[];
+    const int ldk = p.dq + 8;
+    __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);     // [PQ][ldk]
+    __nv_bfloat16* sK = sQ + PQ * ldk;                              // [2][PK][ldk]
+    __nv_bfloat16* sV = sK + 2 * PK * ldk;                          // [2][PK][LDV]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, head = blockIdx.y;
+    const int e = p.tiles[2 * blockIdx.x], q0 = p.tiles[2 * blockIdx.x + 1];
+    const int t0 = p.starts[e], n = p.starts[e + 1] - t0, pos0 = p.positions[t0];
+    const int key0 = first_key(pos0, p.window);                     // position of the entry's first gathered key
+    const int first = first_key(pos0 + q0, p.window), last = pos0 + min(q0 + PQ, n) - 1;
+    const int n_tiles = (last - first) / PK + 1;
+    const __nv_bfloat16* kv = p.kv + (size_t)(p.key_base[e] - key0) * p.ldkv;      // indexed by position
+    const __nv_bfloat16* kr = p.kr + (size_t)(p.key_base[e] - key0) * p.ldr;
+    const int kc = p.dim_p / 8, rc = p.ldr / 8, pad = p.dq / 8, vc = p.vdim_p / 8;
+
+    auto load = [&](int tile, int buf) {
+        const int k0 = first + tile * PK;
+        for (int i = tid; i < PK * pad; i += 128) {
+            const int key = i / pad, c = i - key * pad, pos = k0 + key;
+            const bool ok = pos <= last && c < kc + rc;
+            const __nv_bfloat16* src = !ok ? p.kv : c < kc ? kv + (ptrdiff_t)pos * p.ldkv + head * p.dim_p + c * 8 : kr + (ptrdiff_t)pos * p.ldr + (c - kc) * 8;
+            cp_async16z(smem_u32(sK + (buf * PK + key) * ldk + c * 8), src, ok);
+        }
+        for (int i = tid; i < PK * (VD / 8); i += 128) {
+            const int key = i / (VD / 8), c = i - key * (VD / 8), pos = k0 + key;
+            const bool ok = pos <= last && c < vc;
+            const __nv_bfloat16* src = ok ? kv + (ptrdiff_t)pos * p.ldkv + p.uv_row + head * p.vdim_p + c * 8 : p.kv;
+            cp_async16z(smem_u32(sV + (buf * PK + key) * LDV + c * 8), src, ok);
+        }
+        cp_async_commit();
+    };
+    load(0, 0);
+    for (int i = tid; i < PQ * p.dq; i += 128) {
+        const int r = i / p.dq, c = i - r * p.dq;
+        float v = 0.0f;
+        if (q0 + r < n) {
+            const float* q = p.proj + (size_t)(t0 + q0 + r) * p.ldp + p.off_q + head * (p.dim + p.rot);
+            if (c < p.dim) v = q[c];
+            else if (c >= p.dim_p && c < p.dim_p + p.rot) v = q[p.dim + c - p.dim_p];
+        }
+        sQ[r * ldk + c] = __float2bfloat16_rn(v);
+    }
+    float o[VD / 8][4];
+#pragma unroll
+    for (int i = 0; i < VD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    float m_run[2] = {-1e30f, -1e30f}, l_run[2] = {0.0f, 0.0f};
+    const float sl2 = p.scale * 1.4426950408889634f;
+    const int g = lane >> 2, t4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
+    const int qpos0 = pos0 + q0 + 16 * warp + g;
+    const int window = p.window > 0 ? p.window : 0x7fffffff;
+
+    for (int tile = 0; tile < n_tiles; ++tile) {
+        const int buf = tile & 1, k0 = first + tile * PK;
+        if (tile + 1 < n_tiles) {
+            load(tile + 1, buf ^ 1);
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
+        __syncthreads();
+        float s[8][4];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+        const uint32_t qa = smem_u32(sQ + (16 * warp + (mi & 1) * 8 + r8) * ldk + (mi >> 1) * 8);
+        const uint32_t ka = smem_u32(sK + (buf * PK + (mi >> 1) * 8 + r8) * ldk + (mi & 1) * 8);
+#pragma unroll 2
+        for (int kk = 0; kk < p.dq; kk += 16) {
+            uint32_t a[4];
+            ldsm_x4(qa + 2 * kk, a);
+#pragma unroll
+            for (int np = 0; np < 4; ++np) {
+                uint32_t b[4];
+                ldsm_x4(ka + 2 * (16 * np * ldk + kk), b);
+                mma_bf16(s[2 * np], a, b[0], b[1]);
+                mma_bf16(s[2 * np + 1], a, b[2], b[3]);
+            }
+        }
+        float mx[2] = {-1e30f, -1e30f};
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int kp = k0 + 8 * nt + 2 * t4 + (j & 1), qp = qpos0 + (j >> 1) * 8;
+                const float v = kp <= qp && qp - kp < window ? s[nt][j] * sl2 : -INFINITY;
+                s[nt][j] = v;
+                mx[j >> 1] = fmaxf(mx[j >> 1], v);
+            }
+        float corr[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+            const float m_new = fmaxf(m_run[h], mx[h]);
+            corr[h] = exp2f(m_run[h] - m_new);
+            m_run[h] = m_new;
+            l_run[h] *= corr[h];
+        }
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float w = exp2f(s[nt][j] - m_run[j >> 1]);
+                s[nt][j] = w;
+                l_run[j >> 1] += w;
+            }
+#pragma unroll
+        for (int i = 0; i < VD / 8; ++i) {
+            o[i][0] *= corr[0];
+            o[i][1] *= corr[0];
+            o[i][2] *= corr[1];
+            o[i][3] *= corr[1];
+        }
+        const uint32_t va = smem_u32(sV + (buf * PK + (mi & 1) * 8 + r8) * LDV + (mi >> 1) * 8);
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            uint32_t a[4];
+            a[0] = pack_bf2(s[2 * ks][0], s[2 * ks][1]);
+            a[1] = pack_bf2(s[2 * ks][2], s[2 * ks][3]);
+            a[2] = pack_bf2(s[2 * ks + 1][0], s[2 * ks + 1][1]);
+            a[3] = pack_bf2(s[2 * ks + 1][2], s[2 * ks + 1][3]);
+#pragma unroll
+            for (int dp = 0; dp < VD / 16; ++dp) {
+                uint32_t b[4];
+                ldsm_x4_t(va + 2 * (16 * ks * LDV + 16 * dp), b);
+                mma_bf16(o[2 * dp], a, b[0], b[1]);
+                mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
+            }
+        }
+        __syncthreads();     // every warp is done with this buffer before the next load overwrites it
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
+        const int row = q0 + 16 * warp + g + 8 * h;
+        if (row >= n) continue;
+        const float inv = 1.0f / l_run[h];
+        __nv_bfloat16* dst = p.out + (size_t)(t0 + row) * p.ldm + (size_t)head * p.vdim;
+#pragma unroll
+        for (int nt = 0; nt < VD / 8; ++nt)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const int c = 8 * nt + 2 * t4 + j;
+                if (c < p.vdim) dst[c] = __float2bfloat16_rn(o[nt][2 * h + j] * inv);
+            }
+    }
+}
+
+CacheRef cache_ref(const dc_latent_cache& c, int row) { return CacheRef{c.arena, c.tables, c.max_blocks, row}; }
+
+}  // namespace
+
+int dc_launch_latent_prep(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, float* proj, int ldp, float eps,
+                          int max_pos) {
+    PrepParams p = {proj, ldp, m.off_q, m.off_kv, m.heads, m.dim, m.rot_dim, m.kv_rank, max_pos, m.kv_from < 0 ? m.kv_norm : nullptr,
+                    m.cos_sin, eps, st.seq_ids, st.positions, cache_ref(c, m.row)};
+    if (c.f32) return dc_launch(ctx, "k_latent_prep", k_latent_prep<float>, dim3(st.T), dim3(256), 0, p);
+    return dc_launch(ctx, "k_latent_prep", k_latent_prep<__nv_bfloat16>, dim3(st.T), dim3(256), 0, p);
+}
+
+int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const float* proj, int ldp,
+                              int splits, float* qa, float* part, float* part_ml, float* mix, int ldm) {
+    const int ldq = dc_pad8(m.kv_rank), rb = (m.kv_rank + 255) / 256;
+#define DC_ABSORB(NT)                                                                                                                        \
+    DC_TRY(dc_launch(ctx, "k_latent_absorb", k_latent_absorb<NT>, dim3(m.heads, rb, (st.T + NT - 1) / NT), dim3(128), (size_t)NT * m.dim * 4, \
+                     proj, ldp, m.off_q, m.heads, m.dim, m.rot_dim, m.ukv.w, m.ukv.ld, m.dim_p, m.kv_rank, st.T, qa, ldq))
+    if (st.T == 1) DC_ABSORB(1);
+    else if (st.T <= 4) DC_ABSORB(4);
+    else DC_ABSORB(16);
+#undef DC_ABSORB
+    AbsorbedParams p = {qa, ldq, proj, ldp, m.off_q, m.heads, m.dim, m.rot_dim, m.kv_rank, m.window, splits, m.scale, st.seq_ids, st.positions,
+                        cache_ref(c, m.row), part, part_ml};
+    DC_TRY(c.f32 ? launch_absorbed<float>(ctx, p, st.T) : launch_absorbed<__nv_bfloat16>(ctx, p, st.T));
+    return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T), dim3(256), (size_t)dc_pad8(m.kv_rank) * 4, part, part_ml, m.heads, splits,
+                     m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim, mix, ldm);
+}
+
+int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const int32_t* key_base,
+                            int n_keys, __nv_bfloat16* keys_c, int ldc, __nv_bfloat16* keys_r, int ldr) {
+    return dc_launch(ctx, "k_latent_gather", k_latent_gather, dim3((n_keys + 7) / 8), dim3(256), 0, cache_ref(c, m.row), st.seq_ids, st.positions,
+                     st.starts, key_base, st.E, n_keys, m.window, m.kv_rank, m.rot_dim, keys_c, ldc, keys_r, ldr);
+}
+
+int dc_launch_latent_prefill(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const int32_t* key_base, const int32_t* tiles,
+                             int n_tiles, const float* proj, int ldp, const __nv_bfloat16* keys_kv, int ldkv, const __nv_bfloat16* keys_r,
+                             int ldr, __nv_bfloat16* mixb, int ldm) {
+    PromptParams p = {proj, ldp, m.off_q, m.dim, m.rot_dim, m.dim_p, m.vdim, m.vdim_p, m.uv_row, m.window, m.scale, st.positions, st.starts,
+                      key_base, tiles, keys_kv, ldkv, keys_r, ldr, (m.dim_p + ldr + 15) & ~15, mixb, ldm};
+    const dim3 grid(n_tiles, m.heads), block(128);
+#define DC_PROMPT(VD)                                                                                                       \
+    do {                                                                                                                    \
+        const size_t smem = ((size_t)(PQ + 2 * PK) * (p.dq + 8) + (size_t)2 * PK * (VD + 8)) * 2;                           \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_prompt<VD>, (int)smem, "k_latent_prompt"));                       \
+        return dc_launch(ctx, "k_latent_prompt", k_latent_prompt<VD>, grid, block, smem, p);                                \
+    } while (0)
+    if (m.vdim <= 32) DC_PROMPT(32);
+    if (m.vdim <= 64) DC_PROMPT(64);
+    if (m.vdim <= 128) DC_PROMPT(128);
+    DC_PROMPT(256);
+#undef DC_PROMPT
+}

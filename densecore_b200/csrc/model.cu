@@ -18,6 +18,7 @@
 #include "dc_kv.h"
 #include "dc_mega.h"
 #include "dc_model.h"
+#include "dc_stack.h"
 
 #define DC_TRY(expr)                       \
     do {                                   \
@@ -110,6 +111,11 @@ static bool find_slot(dc_model* m, const std::string& name, TensorSlot* out) {
 
 static std::vector<std::string> tensor_names(const dc_model* m) {
     const dc_model_config& c = m->cfg;
+    if (m->stack) {
+        std::vector<std::string> names;
+        for (const dc_stack_tensor& t : m->stack->tensors) names.push_back(t.name);
+        return names;
+    }
     std::vector<std::string> v = {"token_embd.weight", "output_norm.weight"};
     if (!c.tie_embeddings) v.push_back("output.weight");
     for (int il = 0; il < c.n_layer; ++il) {
@@ -299,21 +305,23 @@ static int enqueue_forward(dc_model* m, int T, int lm_mode, bool feedback) {
 }
 
 // Captured once per (T, lm_mode, feedback); replayed afterwards.
-static int run_forward(dc_model* m, int T, int lm_mode, bool feedback) {
+// chunk: the T tokens are consecutive positions of one sequence (otherwise one token each of T sequences).
+static int run_forward(dc_model* m, int T, int lm_mode, bool feedback, bool chunk = false) {
     dc_ctx* ctx = m->ctx;
-    if (!m->use_graphs || m->dbg_x) return enqueue_forward(m, T, lm_mode, feedback);
-    const int key = T * 8 + lm_mode * 2 + (feedback ? 1 : 0);
+    auto enqueue = [&]() { return m->stack ? dc_stack_enqueue_small(m, T, chunk, lm_mode, feedback) : enqueue_forward(m, T, lm_mode, feedback); };
+    if (!m->use_graphs || m->dbg_x) return enqueue();
+    const int key = T * 8 + lm_mode * 2 + (feedback ? 1 : 0) + (m->stack && chunk ? 1024 : 0);
     auto it = m->graphs.find(key);
     if (it == m->graphs.end()) {
         // one eager pass first: it sets kernel attributes, which is not allowed while capturing
         if (!m->warmed[key]) {
             m->warmed[key] = true;
-            return enqueue_forward(m, T, lm_mode, feedback);
+            return enqueue();
         }
         cudaGraph_t g = nullptr;
         cudaGraphExec_t ge = nullptr;
         DC_TRY(dc_check_cuda(ctx, cudaStreamBeginCapture(ctx->stream, cudaStreamCaptureModeThreadLocal), "begin capture"));
-        int st = enqueue_forward(m, T, lm_mode, feedback);
+        int st = enqueue();
         cudaError_t e = cudaStreamEndCapture(ctx->stream, &g);
         if (st != DC_B200_OK) {
             if (g) cudaGraphDestroy(g);
@@ -351,13 +359,21 @@ static int upload_step_inputs(dc_model* m, const int32_t* tokens, const int32_t*
 // by instruction issue and the per-op kernels (more resident warps per SM) are faster (measured: 1116 vs
 // 1284 us per step at 2 streams, 1546 vs 2059 at 4, 8-layer cut), so the default sends one stream to it.
 static bool mega_ok(dc_model* m, int T) {
-    if (!m->use_mega || (m->use_mega == 1 && T > 1)) return false;
+    if (m->stack || !m->use_mega || (m->use_mega == 1 && T > 1)) return false;
     MegaParams p;
     const char* why = "";
     return dc_mega_plan(m, T, &p, &why);
 }
 
 static bool model_complete(dc_model* m, std::string* missing) {
+    if (m->stack) {
+        for (const dc_stack_tensor& t : m->stack->tensors)
+            if (!t.loaded) {
+                *missing = t.name;
+                return false;
+            }
+        return true;
+    }
     for (const std::string& n : tensor_names(m)) {
         TensorSlot s;
         if (!find_slot(m, n, &s) || !*s.slot) {
@@ -386,7 +402,7 @@ static int forward_chunk(dc_model* m, int seq, const int32_t* tokens, int n, int
         pos[i] = s.len + i;
     }
     DC_TRY(upload_step_inputs(m, tokens, seqs, pos, n));
-    DC_TRY(run_forward(m, n, lm_mode, false));
+    DC_TRY(run_forward(m, n, lm_mode, false, true));
     s.len += n;
     return DC_B200_OK;
 }
@@ -396,6 +412,7 @@ extern "C" {
 int dc_b200_model_create(dc_ctx* ctx, const dc_model_config* cfg, dc_model** out) {
     if (!ctx || !cfg || !out) return DC_B200_INVALID_ARGUMENT;
     *out = nullptr;
+    if (!dc_mega_prepare) return dc_fail(ctx, DC_B200_UNSUPPORTED, "model_create: this library was built without the K-quant kernels");
     const dc_model_config& c = *cfg;
     if (c.head_dim != 128 || c.n_layer < 1 || c.hidden % 256 || c.n_head < 2 || c.n_kv_head < 1 || c.n_head % c.n_kv_head ||
         c.n_head / c.n_kv_head > 8 || (c.n_head & 1) || c.vocab < 2 || c.max_seqs < 1 || c.max_seqs > DC_MAX_T || c.max_ctx < 16)
@@ -444,7 +461,6 @@ void dc_b200_model_destroy(dc_model* m) {
     cudaSetDevice(m->ctx->device);
     cudaStreamSynchronize(m->ctx->stream);
     for (auto& kvp : m->graphs) cudaGraphExecDestroy(kvp.second.exec);
-    dc_ep_destroy(m);
     for (dc_weight* w : m->owned) {
         if (w) {
             cudaFree(w->dev);
@@ -458,10 +474,14 @@ void dc_b200_model_destroy(dc_model* m) {
     for (void* p : ptrs)
         if (p) cudaFree(p);
     if (m->dbg_x) cudaFree(m->dbg_x);
-    dc_prefill_release(m);
+    if (m->stack) dc_stack_release(m);
+    else {
+        dc_prefill_release(m);
+        dc_mega_release_xch(m);
+        dc_ep_destroy(m);
+    }
     if (m->mega_layers) cudaFree(m->mega_layers);
     if (m->mega_counter) cudaFree(m->mega_counter);
-    dc_mega_release_xch(m);
     if (m->h_stage) cudaFreeHost(m->h_stage);
     dc_kv_release(&m->kv);
     delete m;
@@ -485,6 +505,7 @@ int dc_b200_model_tensor_names(dc_model* m, const char** names_out, int capacity
 int dc_b200_model_set_tensor(dc_model* m, const char* name, int ggml_type, const int64_t ne[4], const void* data_host) {
     if (!m || !name || !ne || !data_host) return DC_B200_INVALID_ARGUMENT;
     cudaSetDevice(m->ctx->device);
+    if (m->stack) return dc_stack_set_tensor(m, name, ggml_type, ne, data_host);
     TensorSlot s;
     if (!find_slot(m, name, &s)) return dc_fail(m->ctx, DC_B200_MODEL_LOAD_FAILED, "set_tensor: '%s' is not a tensor of this model", name);
     const int64_t E = ne[2] > 0 ? ne[2] : 1, N = ne[1] > 0 ? ne[1] : 1;
@@ -517,6 +538,7 @@ int dc_b200_model_set_tensor(dc_model* m, const char* name, int ggml_type, const
 int dc_b200_model_init_synthetic(dc_model* m, uint64_t seed, float sigma) {
     if (!m) return DC_B200_INVALID_ARGUMENT;
     cudaSetDevice(m->ctx->device);
+    if (m->stack) return dc_stack_init_synthetic(m, seed, sigma);
     for (const std::string& n : tensor_names(m)) {
         TensorSlot s;
         if (!find_slot(m, n, &s)) return dc_fail(m->ctx, DC_B200_INTERNAL_ERROR, "init_synthetic: no slot for %s", n.c_str());
@@ -561,6 +583,12 @@ int dc_b200_model_finalize(dc_model* m) {
     if (!m) return DC_B200_INVALID_ARGUMENT;
     std::string missing;
     if (!model_complete(m, &missing)) return dc_fail(m->ctx, DC_B200_MODEL_LOAD_FAILED, "finalize: tensor '%s' is missing", missing.c_str());
+    if (m->stack) {
+        cudaSetDevice(m->ctx->device);
+        DC_TRY(dc_stack_finalize(m));
+        m->finalized = true;
+        return DC_B200_OK;
+    }
     if (m->cfg.ep_size > 1 && !m->ep_ready) return dc_fail(m->ctx, DC_B200_MODEL_LOAD_FAILED, "finalize: expert-parallel communicator not initialised");
     if (!m->mega_layers) DC_TRY(dc_mega_prepare(m));
     m->finalized = true;
@@ -568,7 +596,7 @@ int dc_b200_model_finalize(dc_model* m) {
 }
 
 size_t dc_b200_model_weight_bytes(dc_model* m) {
-    size_t n = 0;
+    size_t n = m && m->stack ? m->stack->weight_bytes : 0;
     if (m)
         for (dc_weight* w : m->owned) n += w->bytes;
     return n;
@@ -590,16 +618,83 @@ int dc_b200_seq_truncate(dc_model* m, int seq, int new_len) {
     if (!m) return DC_B200_INVALID_ARGUMENT;
     DC_TRY(check_seq(m, seq));
     if (new_len < 0 || new_len > m->kv.seqs[seq].len) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "seq_truncate: bad length %d", new_len);
+    if (m->kv.state_bytes && new_len > 0 && new_len < m->kv.seqs[seq].len)
+        return dc_fail(m->ctx, DC_B200_UNSUPPORTED, "seq_truncate: a recurrent state cannot go back to %d tokens (fork before, or truncate to 0)", new_len);
     m->kv.seqs[seq].len = new_len;  // blocks stay reserved; later positions are simply overwritten
     return DC_B200_OK;
 }
 
 }  // extern "C"
 
+// Room and token ids of the next n tokens of a sequence; reserves their cache blocks.
+int dc_model_check_entry(dc_model* m, int seq, const int32_t* tokens, int n) {
+    DC_TRY(check_seq(m, seq));
+    const dc_kv_seq& s = m->kv.seqs[seq];
+    if (n < 1 || s.len + n > m->cfg.max_ctx) return dc_fail(m->ctx, DC_B200_OUT_OF_MEMORY, "sequence %d would exceed max_ctx %d", seq, m->cfg.max_ctx);
+    for (int i = 0; i < n; ++i)
+        if (tokens[i] < 0 || tokens[i] >= m->cfg.vocab) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "token id %d out of range", tokens[i]);
+    return dc_kv_seq_reserve(&m->kv, seq, s.len + n);
+}
+
+// Next tokens of any number of sequences as one batch (see dc_b200_forward_batch); picks: greedy token per row.
+int dc_model_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, int n_rows, const int32_t* rows,
+                   float* logits_host, int32_t* picks_host) {
+    dc_ctx* ctx = m->ctx;
+    if (E < 1 || E > DC_MAX_T) return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "forward_batch: %d entries", E);
+    long long total = 0;
+    bool single = true;
+    for (int e = 0; e < E; ++e) {
+        for (int j = 0; j < e; ++j)
+            if (seqs[j] == seqs[e]) return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "forward_batch: sequence %d appears twice", seqs[e]);
+        if (counts[e] < 1) return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "forward_batch: entry %d has no tokens", e);
+        total += counts[e];
+        single &= counts[e] == 1;
+    }
+    for (int r = 0; r < n_rows; ++r)
+        if (rows[r] < 0 || rows[r] >= total || (r && rows[r] <= rows[r - 1]))
+            return dc_fail(ctx, DC_B200_INVALID_ARGUMENT, "forward_batch: wanted rows must be ascending and within the batch");
+    for (int e = 0, t = 0; e < E; t += counts[e], ++e) DC_TRY(dc_model_check_entry(m, seqs[e], tokens + t, counts[e]));
+    const size_t V = m->cfg.vocab;
+    if (m->stack && !single) return dc_stack_batch(m, E, seqs, counts, tokens, n_rows, rows, logits_host, picks_host);
+    // one token per sequence: the decode step.  Models without ragged batches also come here, entry by entry.
+    std::vector<float> lg(logits_host ? V * DC_MAX_T : 0);
+    int next_row = 0;
+    auto take = [&](int t0, int n, const int32_t* picks) {
+        for (; next_row < n_rows && rows[next_row] < t0 + n; ++next_row) {
+            if (logits_host) memcpy(logits_host + next_row * V, lg.data() + (rows[next_row] - t0) * V, V * 4);
+            if (picks_host) picks_host[next_row] = picks[rows[next_row] - t0];
+        }
+    };
+    int32_t picks[DC_MAX_T];
+    if (single) {
+        DC_TRY(dc_b200_decode_step(m, seqs, E, tokens, picks, n_rows && logits_host ? lg.data() : nullptr));
+        take(0, E, picks);
+        return DC_B200_OK;
+    }
+    for (int e = 0, t0 = 0; e < E; ++e)
+        for (int i = 0; i < counts[e];) {
+            const int n = counts[e] - i < DC_MAX_T ? counts[e] - i : DC_MAX_T;
+            DC_TRY(forward_chunk(m, seqs[e], tokens + t0, n, 2));
+            DC_TRY(dc_check_cuda(ctx, cudaMemcpyAsync(picks, m->buf.out_tokens, (size_t)n * 4, cudaMemcpyDeviceToHost, ctx->stream), "D2H tokens"));
+            if (logits_host) DC_TRY(dc_check_cuda(ctx, cudaMemcpyAsync(lg.data(), m->buf.logits, n * V * 4, cudaMemcpyDeviceToHost, ctx->stream), "D2H logits"));
+            DC_TRY(dc_b200_synchronize(ctx));
+            take(t0, n, picks);
+            t0 += n;
+            i += n;
+        }
+    return DC_B200_OK;
+}
+
 int dc_model_prefill_range(dc_model* m, int seq, const int32_t* tokens_host, int n, bool final, int32_t* next_token) {
     for (int i0 = 0; i0 < n;) {
         const int left = n - i0;
-        if (dc_prefill_tc_ok(m, left)) {
+        if (m->stack && left > DC_MAX_T) {
+            const int c = left < m->stack->b.cap ? left : m->stack->b.cap, last = c - 1;
+            const bool fin = final && i0 + c >= n;
+            DC_TRY(dc_model_check_entry(m, seq, tokens_host + i0, c));
+            DC_TRY(dc_stack_batch(m, 1, &seq, &c, tokens_host + i0, fin ? 1 : 0, &last, nullptr, nullptr));
+            i0 += c;
+        } else if (!m->stack && dc_prefill_tc_ok(m, left)) {
             // enough tokens for the tensor-core matmuls: one chunk of up to prefill_chunk tokens
             const int c = left < m->prefill_chunk ? left : m->prefill_chunk;
             DC_TRY(dc_prefill_chunk_tc(m, seq, tokens_host + i0, c, final && i0 + c >= n));
@@ -662,6 +757,15 @@ int dc_b200_forward_chunk(dc_model* m, int seq, const int32_t* tokens_host, int 
         return dc_b200_synchronize(m->ctx);
     }
     return DC_B200_OK;
+}
+
+int dc_b200_forward_batch(dc_model* m, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens_host, int n_rows,
+                          const int32_t* rows, float* logits_host, int32_t* picks_host) {
+    if (!m || !seqs || !counts || !tokens_host || n_rows < 0 || (n_rows > 0 && !rows))
+        return m ? dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "forward_batch: bad argument") : DC_B200_INVALID_ARGUMENT;
+    if (!m->finalized) return dc_fail(m->ctx, DC_B200_MODEL_LOAD_FAILED, "forward_batch: model is not finalized");
+    cudaSetDevice(m->ctx->device);
+    return dc_model_batch(m, n_entries, seqs, counts, tokens_host, n_rows, rows, logits_host, picks_host);
 }
 
 void* dc_b200_model_logits_dev(dc_model* m) { return m ? m->buf.logits : nullptr; }
@@ -752,7 +856,8 @@ int dc_b200_decode_run(dc_model* m, const int32_t* seqs, int n_seq, const int32_
 static const char* kClassNames[DC_K_COUNT] = {"embed", "rmsnorm_q8k", "gemv_qkv", "qknorm_rope_kv", "attention",
                                                "gemv_attn_out", "router_topk", "moe_gate_up_swiglu", "quantize_h",
                                                "moe_down", "moe_combine", "ep_allreduce", "ffn_gate_up_swiglu",
-                                               "ffn_down", "lm_head_argmax", "argmax_finish"};
+                                               "ffn_down", "lm_head_argmax", "argmax_finish", "mixer_in", "mixer_out",
+                                               "mixer_delta", "mixer_ssd", "mixer_latent", "post_norm"};
 
 const char* dc_b200_kernel_class_name(int cls) { return (cls >= 0 && cls < DC_K_COUNT) ? kClassNames[cls] : nullptr; }
 
@@ -795,6 +900,8 @@ int dc_b200_model_profile_step(dc_model* m, const int32_t* seqs, int n_seq, cons
 
 int dc_b200_model_set_option(dc_model* m, const char* name, int value) {
     if (!m || !name) return DC_B200_INVALID_ARGUMENT;
+    if (m->stack && strcmp(name, "graphs") && strcmp(name, "capture_layer_inputs") && strcmp(name, "prefill_chunk"))
+        return dc_fail(m->ctx, DC_B200_UNSUPPORTED, "model option '%s' does not apply to this architecture", name);
     if (!strcmp(name, "graphs")) {
         m->use_graphs = value != 0;
         return DC_B200_OK;
@@ -841,6 +948,7 @@ int dc_b200_model_set_option(dc_model* m, const char* name, int value) {
         return DC_B200_OK;
     }
     if (!strcmp(name, "prefill_chunk")) {
+        if (m->finalized && m->stack) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "prefill_chunk is fixed once the model is finalized");
         if (value < 32 || value > 4096) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "prefill_chunk must be 32..4096");
         if (m->prefill) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "prefill_chunk is fixed once a chunk has run");
         m->prefill_chunk = value;
@@ -880,6 +988,7 @@ int dc_b200_model_read_layer_input(dc_model* m, int layer, int n_tokens, float* 
 
 int dc_b200_model_read_kv(dc_model* m, int layer, int seq, int first, int n_tokens, void* k_host, void* v_host) {
     if (!m || !k_host || !v_host) return DC_B200_INVALID_ARGUMENT;
+    if (m->stack) return dc_fail(m->ctx, DC_B200_UNSUPPORTED, "read_kv: this architecture has no K and V arenas");
     DC_TRY(check_seq(m, seq));
     const dc_kv_seq& s = m->kv.seqs[seq];
     if (layer < 0 || layer >= m->cfg.n_layer || first < 0 || n_tokens < 1 || first + n_tokens > (int)s.blocks.size() * DC_KV_BLOCK)
@@ -904,6 +1013,10 @@ int dc_b200_model_step_stats(dc_model* m, int* kernels_per_step, double* weight_
     if (!m) return DC_B200_INVALID_ARGUMENT;
     const dc_model_config& c = m->cfg;
     if (kernels_per_step) *kernels_per_step = m->last_launches;
+    if (m->stack) {
+        dc_stack_stats(m, weight_bytes_per_step, kv_bytes_per_token_ctx);
+        return DC_B200_OK;
+    }
     // bytes one single-token step must read: every dense tensor once, top-k experts per layer, the output matrix
     double wb = 0.0;
     for (int il = 0; il < c.n_layer; ++il) {

@@ -7,6 +7,8 @@
 //     if no prefill is in flight and a sequence slot is free), or
 //   * one decode step for all running sequences together (their tokens form one batch of the decoder),
 // alternating between the two when both are possible, so that a long prompt does not stall running streams.
+// A model with ragged batches (dc_stack.h) does both in one step instead: the prompt chunk and every running
+// sequence's next token form one batch.
 // A newly admitted request first takes over the cached blocks of its longest cached prompt prefix (model
 // option "prefix_cache"); only the rest of the prompt runs.
 #include <deque>
@@ -57,23 +59,58 @@ int finish_reason(const dc_sched* s, const dc_sched_request& r) {
     return r.generated >= r.max_new ? 1 : 0;
 }
 
+// The oldest waiting request becomes the one that is being prefilled.
+int admit(dc_sched* s) {
+    dc_model* m = s->m;
+    dc_sched_request r = std::move(s->waiting.front());
+    s->waiting.pop_front();
+    DC_TRY(dc_b200_seq_alloc(m, &r.seq));
+    if (m->prefix_cache) {
+        int st = dc_kv_prefix_attach(&m->kv, r.seq, r.prompt.data(), (int)r.prompt.size(), &r.cached);
+        if (st != DC_B200_OK) {
+            dc_b200_seq_free(m, r.seq);
+            return st;
+        }
+        s->prompt_tokens_cached += (uint64_t)r.cached;
+    }
+    r.done = r.cached;
+    s->prefilling.push_back(std::move(r));
+    return DC_B200_OK;
+}
+
+// The prefilled request's first token is there: it finishes or joins the running ones.
+void start_running(dc_sched* s, int32_t token, dc_sched_event* ev, int cap, int* n) {
+    dc_sched_request& r = s->prefilling[0];
+    r.last = token;
+    r.generated = 1;
+    const int fin = finish_reason(s, r);
+    emit(ev, cap, n, r.id, token, fin);
+    if (fin) dc_b200_seq_free(s->m, r.seq);
+    else s->running.push_back(std::move(r));
+    s->prefilling.clear();
+}
+
+// next[i]: the running sequences' new tokens, in order.
+void advance_running(dc_sched* s, const int32_t* next, int B, dc_sched_event* ev, int cap, int* n) {
+    ++s->decode_steps;
+    s->decode_tokens += (uint64_t)B;
+    if ((uint64_t)B > s->max_batch) s->max_batch = (uint64_t)B;
+    std::vector<dc_sched_request> keep;
+    for (int i = 0; i < B; ++i) {
+        dc_sched_request& r = s->running[i];
+        r.last = next[i];
+        ++r.generated;
+        const int fin = finish_reason(s, r);
+        emit(ev, cap, n, r.id, next[i], fin);
+        if (fin) dc_b200_seq_free(s->m, r.seq);
+        else keep.push_back(std::move(r));
+    }
+    s->running.swap(keep);
+}
+
 int prefill_step(dc_sched* s, dc_sched_event* ev, int cap, int* n) {
     dc_model* m = s->m;
-    if (s->prefilling.empty()) {
-        dc_sched_request r = std::move(s->waiting.front());
-        s->waiting.pop_front();
-        DC_TRY(dc_b200_seq_alloc(m, &r.seq));
-        if (m->prefix_cache) {
-            int st = dc_kv_prefix_attach(&m->kv, r.seq, r.prompt.data(), (int)r.prompt.size(), &r.cached);
-            if (st != DC_B200_OK) {
-                dc_b200_seq_free(m, r.seq);
-                return st;
-            }
-            s->prompt_tokens_cached += (uint64_t)r.cached;
-        }
-        r.done = r.cached;
-        s->prefilling.push_back(std::move(r));
-    }
+    if (s->prefilling.empty()) DC_TRY(admit(s));
     dc_sched_request& r = s->prefilling[0];
     const int left = (int)r.prompt.size() - r.done;
     const int c = left < s->chunk ? left : s->chunk;
@@ -90,13 +127,7 @@ int prefill_step(dc_sched* s, dc_sched_event* ev, int cap, int* n) {
     ++s->prefill_chunks;
     if (!final) return DC_B200_OK;
     if (m->prefix_cache) dc_kv_prefix_register(&m->kv, r.seq, r.prompt.data(), (int)r.prompt.size());
-    r.last = next;
-    r.generated = 1;
-    const int fin = finish_reason(s, r);
-    emit(ev, cap, n, r.id, next, fin);
-    if (fin) dc_b200_seq_free(m, r.seq);
-    else s->running.push_back(std::move(r));
-    s->prefilling.clear();
+    start_running(s, next, ev, cap, n);
     return DC_B200_OK;
 }
 
@@ -108,20 +139,51 @@ int decode_step(dc_sched* s, dc_sched_event* ev, int cap, int* n) {
         toks[i] = s->running[i].last;
     }
     DC_TRY(dc_b200_decode_step(s->m, seqs, B, toks, next, nullptr));
-    ++s->decode_steps;
-    s->decode_tokens += (uint64_t)B;
-    if ((uint64_t)B > s->max_batch) s->max_batch = (uint64_t)B;
-    std::vector<dc_sched_request> keep;
-    for (int i = 0; i < B; ++i) {
-        dc_sched_request& r = s->running[i];
-        r.last = next[i];
-        ++r.generated;
-        const int fin = finish_reason(s, r);
-        emit(ev, cap, n, r.id, next[i], fin);
-        if (fin) dc_b200_seq_free(s->m, r.seq);
-        else keep.push_back(std::move(r));
+    advance_running(s, next, B, ev, cap, n);
+    return DC_B200_OK;
+}
+
+// One ragged batch: the next token of every running sequence and the next chunk of the prompt being prefilled.
+int mixed_step(dc_sched* s, bool with_prompt, dc_sched_event* ev, int cap, int* n) {
+    dc_model* m = s->m;
+    if (with_prompt && s->prefilling.empty()) DC_TRY(admit(s));
+    const int B = (int)s->running.size();
+    std::vector<int32_t> seqs, counts, tokens, rows;
+    for (auto& r : s->running) {
+        rows.push_back((int32_t)tokens.size());
+        seqs.push_back(r.seq);
+        counts.push_back(1);
+        tokens.push_back(r.last);
     }
-    s->running.swap(keep);
+    int c = 0;
+    bool final = false;
+    if (with_prompt) {
+        dc_sched_request& r = s->prefilling[0];
+        const int left = (int)r.prompt.size() - r.done;
+        c = left < s->chunk ? left : s->chunk;
+        final = c == left;
+        seqs.push_back(r.seq);
+        counts.push_back(c);
+        tokens.insert(tokens.end(), r.prompt.begin() + r.done, r.prompt.begin() + r.done + c);
+        if (final) rows.push_back((int32_t)tokens.size() - 1);
+    }
+    int32_t next[DC_MAX_T + 1];
+    int st = dc_model_batch(m, (int)seqs.size(), seqs.data(), counts.data(), tokens.data(), (int)rows.size(), rows.data(), nullptr, next);
+    if (st != DC_B200_OK) {
+        if (with_prompt) {   // the request being prefilled fails as a whole; its slot returns
+            dc_b200_seq_free(m, s->prefilling[0].seq);
+            emit(ev, cap, n, s->prefilling[0].id, -1, 3);
+            s->prefilling.clear();
+        }
+        return st;
+    }
+    m->prefill_tokens_run += (uint64_t)c;
+    if (B) advance_running(s, next, B, ev, cap, n);
+    if (with_prompt) {
+        ++s->prefill_chunks;
+        s->prefilling[0].done += c;
+        if (final) start_running(s, next[B], ev, cap, n);
+    }
     return DC_B200_OK;
 }
 
@@ -184,6 +246,7 @@ int dc_b200_sched_step(dc_sched* s, dc_sched_event* events, int capacity, int* n
     if (!can_prefill && !can_decode) return DC_B200_OK;
     cudaSetDevice(s->m->ctx->device);
     ++s->steps;
+    if (s->m->stack) return mixed_step(s, can_prefill, events, capacity, n_events);
     const bool do_prefill = can_prefill && (!can_decode || !s->last_was_prefill);
     s->last_was_prefill = do_prefill;
     return do_prefill ? prefill_step(s, events, capacity, n_events) : decode_step(s, events, capacity, n_events);

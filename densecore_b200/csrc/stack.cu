@@ -1,0 +1,547 @@
+// Layer-list decoders: weight upload, step buffers and the forward pass over dc_stack.h's mixers.  Host code plus
+// the small kernels that lay random weights out; arithmetic is in linear*.cu, mix_*.cu, norm_act.cu and the greedy
+// epilogue the other models use.
+#include <math.h>
+#include <string.h>
+
+#include <algorithm>
+
+#include "dc_common.cuh"
+#include "dc_model.h"
+#include "dc_stack.h"
+
+#define DC_TRY(expr)                       \
+    do {                                   \
+        int st_ = (expr);                  \
+        if (st_ != DC_B200_OK) return st_; \
+    } while (0)
+
+namespace {
+
+uint64_t fnv1a64(const char* s) {
+    uint64_t h = 1469598103934665603ull;
+    for (; *s; ++s) {
+        h ^= (uint8_t)*s;
+        h *= 1099511628211ull;
+    }
+    return h;
+}
+
+float bf16_value(uint16_t b) {
+    const uint32_t u = (uint32_t)b << 16;
+    float f;
+    memcpy(&f, &u, 4);
+    return f;
+}
+
+int64_t elems(const dc_stack_tensor& t) {
+    int64_t n = 1;
+    for (int64_t d : t.shape) n *= d;
+    return n;
+}
+
+// Random f32 values rounded to bf16 at the tensor's place in a fused matrix.
+__global__ void k_place_rows(const float* __restrict__ src, int64_t n, int K, __nv_bfloat16* __restrict__ w, int ld, int row0, int step, int head_rows,
+                             int head_pad) {
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+        const int r = (int)(i / K), c = (int)(i % K);
+        const int64_t dst = row0 + (head_rows ? (int64_t)(r / head_rows) * head_pad + r % head_rows : (int64_t)r * step);
+        w[dst * ld + c] = __float2bfloat16_rn(src[i]);
+    }
+}
+
+template <typename T>
+int alloc(dc_model* m, T** p, size_t n, const char* what = "step buffer") {
+    DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)p, n * sizeof(T) + 256), what));
+    m->stack->b.owned.push_back((void*)*p);
+    return dc_check_cuda(m->ctx, cudaMemsetAsync(*p, 0, n * sizeof(T) + 256, m->ctx->stream), what);
+}
+
+}  // namespace
+
+// ---------------------------------------------------------------- weights
+int dc_stack_set_tensor(dc_model* m, const char* name, int type, const int64_t ne[4], const void* data) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    auto it = s->index.find(name);
+    if (it == s->index.end()) return dc_fail(ctx, DC_B200_MODEL_LOAD_FAILED, "set_tensor: '%s' is not a tensor of this model", name);
+    dc_stack_tensor& t = s->tensors[it->second];
+    const bool matrix = t.shape.size() == 2;
+    const int64_t K = matrix ? t.shape[1] : t.shape[0], N = matrix ? t.shape[0] : 1;
+    if (ne[0] != K || (ne[1] > 0 ? ne[1] : 1) != N || (ne[2] > 1))
+        return dc_fail(ctx, DC_B200_MODEL_LOAD_FAILED, "set_tensor: '%s' has shape [%lld, %lld], expected [%lld, %lld]", name, (long long)ne[1],
+                       (long long)ne[0], (long long)N, (long long)K);
+    if (t.loaded) return dc_fail(ctx, DC_B200_MODEL_LOAD_FAILED, "set_tensor: '%s' was already set", name);
+    if (type != DC_TYPE_BF16 && !(type == DC_TYPE_F32 && t.vec))
+        return dc_fail(ctx, DC_B200_UNSUPPORTED, "set_tensor: '%s' has type %d; matrices are bf16, vectors bf16 or f32", name, type);
+    cudaError_t e = cudaSuccess;
+    if (t.vec) {
+        const int64_t n = elems(t);
+        std::vector<float> v((size_t)n);
+        for (int64_t i = 0; i < n; ++i) {
+            v[i] = type == DC_TYPE_F32 ? ((const float*)data)[i] : bf16_value(((const uint16_t*)data)[i]);
+            if (t.neg_exp) v[i] = (float)-exp((double)v[i]);
+        }
+        e = cudaMemcpy(*t.vec + t.vec_off, v.data(), (size_t)n * 4, cudaMemcpyHostToDevice);
+    } else if (!t.lin) {
+        e = cudaMemcpy(s->embed->dev, data, s->embed->bytes, cudaMemcpyHostToDevice);
+    } else {
+        const size_t rb = (size_t)K * 2, pitch = (size_t)t.lin->ld * 2;
+        const int per = t.head_rows ? t.head_rows : (int)N, blocks = (int)N / per;
+        for (int b = 0; b < blocks && e == cudaSuccess; ++b)
+            e = cudaMemcpy2D(t.lin->w + (size_t)(t.row0 + b * t.head_pad) * t.lin->ld, pitch * t.row_step, (const uint8_t*)data + (size_t)b * per * rb, rb, rb,
+                             per, cudaMemcpyHostToDevice);
+    }
+    DC_TRY(dc_check_cuda(ctx, e, "set_tensor"));
+    t.loaded = true;
+    return DC_B200_OK;
+}
+
+int dc_stack_init_synthetic(dc_model* m, uint64_t seed, float sigma) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    if (!dc_launch_synth_f32) return dc_fail(ctx, DC_B200_UNSUPPORTED, "init_synthetic: this library was built without the random-weight kernels");
+    int64_t most = 0;
+    for (auto& t : s->tensors) most = std::max(most, elems(t));
+    float* tmp = nullptr;
+    DC_TRY(dc_check_cuda(ctx, cudaMalloc((void**)&tmp, (size_t)most * 4), "init_synthetic"));
+    int st = DC_B200_OK;
+    for (auto& t : s->tensors) {
+        if (t.loaded || st != DC_B200_OK) continue;
+        const int64_t n = elems(t);
+        // norm weights around 1, decay exponents and step biases in a useful range, convolution taps not tiny
+        const float sg = t.synth == 4 ? 0.4f : t.synth == 2 ? 0.5f : sigma, off = t.synth == 1 ? 1.0f : t.synth == 3 ? -2.0f : 0.0f;
+        float* dst = t.vec ? *t.vec + t.vec_off : tmp;
+        st = dc_launch_synth_f32(ctx, seed + fnv1a64(t.name.c_str()), n, sg, off, dst);
+        if (st != DC_B200_OK) break;
+        if (t.vec && t.neg_exp) {
+            std::vector<float> v((size_t)n);
+            cudaStreamSynchronize(ctx->stream);
+            cudaMemcpy(v.data(), dst, (size_t)n * 4, cudaMemcpyDeviceToHost);
+            for (float& x : v) x = (float)-exp((double)x);
+            st = dc_check_cuda(ctx, cudaMemcpy(dst, v.data(), (size_t)n * 4, cudaMemcpyHostToDevice), "init_synthetic");
+        } else if (!t.vec) {
+            const int K = (int)t.shape[1];
+            __nv_bfloat16* w = t.lin ? t.lin->w : (__nv_bfloat16*)s->embed->dev;
+            k_place_rows<<<1184, 256, 0, ctx->stream>>>(tmp, n, K, w, t.lin ? t.lin->ld : K, t.row0, t.row_step, t.head_rows, t.head_pad);
+            st = dc_check_cuda(ctx, cudaGetLastError(), "k_place_rows");
+        }
+        t.loaded = true;
+    }
+    if (st == DC_B200_OK) st = dc_b200_synchronize(ctx);
+    cudaFree(tmp);
+    return st;
+}
+
+void dc_stack_release(dc_model* m) {
+    dc_stack* s = m->stack;
+    if (!s) return;
+    for (void* p : s->owned) cudaFree(p);
+    for (void* p : s->b.owned) cudaFree(p);
+    for (auto& r : s->rot) cudaFree(r.second);
+    if (s->b.h_meta) cudaFreeHost(s->b.h_meta);
+    if (s->embed) {
+        if (s->embed->dev) cudaFree(s->embed->dev);
+        delete s->embed;
+    }
+    delete s;
+    m->stack = nullptr;
+}
+
+// ---------------------------------------------------------------- cache, state slots, step buffers
+// Cache planes of the layers that write a latent, state slots of the recurrent layers, rotation tables.  The pool
+// holds pool_tokens tokens (0: max_ctx for every sequence).
+int dc_stack_create_cache(dc_model* m, int pool_tokens) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    const dc_model_config& c = m->cfg;
+    const size_t elt = s->dtype == DC_DTYPE_F32 ? 4 : 2;
+    std::vector<size_t> planes;
+    size_t state = 0;
+    auto carve = [&](size_t floats) {
+        const size_t off = state;
+        state += (floats * 4 + 255) & ~(size_t)255;
+        return off;
+    };
+    int span = 1;
+    for (dc_stack_layer& L : s->layers) {
+        if (L.kind == DC_MIX_DELTA) {
+            L.state_off = carve((size_t)L.dl.heads * L.dl.vdim * L.dl.dim);
+            L.ring_off = carve((size_t)L.dl.taps * (L.dl.off_v + L.dl.heads * L.dl.vdim));
+        } else if (L.kind == DC_MIX_SSD) {
+            L.state_off = carve((size_t)L.ssd.heads * L.ssd.vdim * L.ssd.state);
+            L.ring_off = carve((size_t)L.ssd.taps * (L.ssd.heads * L.ssd.vdim + 2 * L.ssd.groups * L.ssd.state));
+        } else {
+            dc_latent_mixer& a = L.la;
+            if (a.kv_from < 0) {
+                a.plane = (int)planes.size();
+                planes.push_back((size_t)a.row * elt);
+            } else {
+                a.plane = s->layers[a.kv_from].la.plane;
+            }
+            auto w = std::find(s->windows.begin(), s->windows.end(), a.window);
+            a.range = (int)(w - s->windows.begin());
+            if (w == s->windows.end()) s->windows.push_back(a.window);
+            span = std::max(span, a.window > 0 ? std::min(a.window, c.max_ctx) : c.max_ctx);
+            float*& table = s->rot[{a.rot_base, a.rot_dim}];
+            if (!table) {
+                std::vector<float> cs((size_t)c.max_ctx * a.rot_dim);
+                for (int p = 0; p < c.max_ctx; ++p)
+                    for (int i = 0; i < a.rot_dim / 2; ++i) {
+                        const double ang = (double)p * pow(a.rot_base, -2.0 * i / a.rot_dim);
+                        cs[(size_t)p * a.rot_dim + 2 * i] = (float)cos(ang);
+                        cs[(size_t)p * a.rot_dim + 2 * i + 1] = (float)sin(ang);
+                    }
+                DC_TRY(dc_check_cuda(ctx, cudaMalloc((void**)&table, cs.size() * 4), "rotation table"));
+                DC_TRY(dc_check_cuda(ctx, cudaMemcpy(table, cs.data(), cs.size() * 4, cudaMemcpyHostToDevice), "rotation table"));
+            }
+            a.cos_sin = table;
+        }
+    }
+    // key splits of a decode step: about 64 keys each at the longest span
+    s->splits = std::max(1, std::min(32, (span + 63) / 64));
+    const int per_seq = (c.max_ctx + DC_KV_BLOCK - 1) / DC_KV_BLOCK;
+    const int blocks = pool_tokens > 0 ? (pool_tokens + DC_KV_BLOCK - 1) / DC_KV_BLOCK : per_seq * c.max_seqs;
+    return dc_kv_init_planes(ctx, &m->kv, planes, state, blocks, c.max_seqs, per_seq);
+}
+
+static constexpr int ENTRY_INTS = DC_MAX_T + 1;
+
+int dc_stack_finalize(dc_model* m) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    if (b.cap) return DC_B200_OK;
+    const size_t H = dc_pad8(s->cfg.width), V = s->cfg.vocab;
+    const bool f32 = s->dtype == DC_DTYPE_F32;
+    const long long all = (long long)m->cfg.max_seqs * m->cfg.max_ctx;
+    const size_t C = std::max<long long>(DC_MAX_T, std::min<long long>(m->prefill_chunk, all));
+    const size_t F = f32 ? C : DC_MAX_T;      // rows of buffers that only the f32 path uses
+    size_t proj = 8, act = 8, low = 8, gate = 8, small = 8, mix = 8, ff = 8, lowb = 8, rank = 8, rot = 8, ukv = 8, qa = 0, part = 0, ml = 0;
+    int span = 1;
+    for (dc_stack_layer& L : s->layers) {
+        auto up = [](size_t& a, long long v) { a = std::max(a, (size_t)dc_pad8((int)v)); };
+        up(ff, L.ff);
+        if (L.kind == DC_MIX_DELTA) {
+            const dc_delta_mixer& d = L.dl;
+            up(proj, d.in.N), up(act, d.off_v + d.heads * d.vdim), up(low, d.a2.N), up(gate, d.g2.N), up(small, d.heads + d.kv_heads);
+            up(mix, d.heads * d.vdim), up(lowb, d.in.N - d.off_a);
+        } else if (L.kind == DC_MIX_SSD) {
+            const dc_ssd_mixer& d = L.ssd;
+            up(proj, d.in.N), up(act, d.heads * d.vdim + 2 * d.groups * d.state), up(small, 2 * d.heads), up(mix, d.heads * d.vdim);
+        } else {
+            const dc_latent_mixer& d = L.la;
+            up(proj, d.in.N), up(mix, d.heads * d.vdim), up(rank, d.kv_rank), up(rot, d.rot_dim), up(ukv, d.ukv.N);
+            const size_t parts = std::max((size_t)DC_MAX_T * s->splits, f32 ? C : 0);
+            qa = std::max(qa, F * d.heads * dc_pad8(d.kv_rank));
+            part = std::max(part, parts * d.heads * d.kv_rank);
+            ml = std::max(ml, parts * d.heads * 2);
+            span = std::max(span, d.window > 0 ? std::min(d.window, m->cfg.max_ctx) : m->cfg.max_ctx);
+        }
+    }
+    b.key_cap = (int)std::min<long long>((long long)C + (long long)m->cfg.max_seqs * (span - 1), all);
+    b.key_cap = std::max(b.key_cap, DC_MAX_T);
+    DC_TRY(alloc(m, &b.x, C * H));
+    DC_TRY(alloc(m, &b.y, C * H));
+    DC_TRY(alloc(m, &b.proj, C * proj));
+    DC_TRY(alloc(m, &b.act, C * act));
+    DC_TRY(alloc(m, &b.scan, C * act));
+    DC_TRY(alloc(m, &b.low, C * low));
+    DC_TRY(alloc(m, &b.gate, C * gate));
+    DC_TRY(alloc(m, &b.small, C * small));
+    DC_TRY(alloc(m, &b.mix, F * mix));
+    DC_TRY(alloc(m, &b.ff, F * ff));
+    DC_TRY(alloc(m, &b.lm_x, DC_MAX_T * H));
+    if (!f32) {
+        DC_TRY(alloc(m, &b.xb, C * H));
+        DC_TRY(alloc(m, &b.mixb, C * mix));
+        DC_TRY(alloc(m, &b.ffb, C * ff));
+        DC_TRY(alloc(m, &b.lowb, C * lowb));
+    }
+    if (!s->windows.empty()) {
+        DC_TRY(alloc(m, &b.qa, qa));
+        DC_TRY(alloc(m, &b.part, part));
+        DC_TRY(alloc(m, &b.part_ml, ml));
+        if (!f32) {
+            DC_TRY(alloc(m, &b.keys_c, b.key_cap * rank));
+            DC_TRY(alloc(m, &b.keys_r, b.key_cap * rot));
+            DC_TRY(alloc(m, &b.keys_kv, b.key_cap * ukv));
+        }
+    }
+    // metadata of a step: tokens, sequences, positions, entry starts, wanted rows, key ranges per window, query tiles
+    b.meta_ints = (int)(4 * C + ENTRY_INTS * (1 + s->windows.size()) + 2 * (C / DC_LATENT_QTILE + DC_MAX_T + 1));
+    DC_TRY(alloc(m, &b.meta, (size_t)b.meta_ints));
+    DC_TRY(dc_check_cuda(ctx, cudaMallocHost((void**)&b.h_meta, (size_t)b.meta_ints * DC_STACK_META_SLOTS * 4), "cudaMallocHost"));
+    DC_TRY(alloc(m, &b.iota, ENTRY_INTS));
+    DC_TRY(alloc(m, &b.chunk, 2 * ENTRY_INTS));
+    int32_t iota[ENTRY_INTS], chunk[2 * ENTRY_INTS];
+    for (int i = 0; i < ENTRY_INTS; ++i) iota[i] = i, chunk[2 * i] = 0, chunk[2 * i + 1] = i;
+    DC_TRY(dc_check_cuda(ctx, cudaStreamSynchronize(ctx->stream), "finalize"));
+    DC_TRY(dc_check_cuda(ctx, cudaMemcpy(b.iota, iota, sizeof(iota), cudaMemcpyHostToDevice), "finalize"));
+    DC_TRY(dc_check_cuda(ctx, cudaMemcpy(b.chunk, chunk, sizeof(chunk), cudaMemcpyHostToDevice), "finalize"));
+    // the step buffers every model has
+    dc_step_buffers& g = m->buf;
+    void** common[] = {(void**)&g.tokens, (void**)&g.seq_ids, (void**)&g.positions, (void**)&g.out_tokens, (void**)&g.argmax_keys,
+                       (void**)&g.logits, (void**)&g.history, (void**)&g.history_len};
+    const size_t bytes[] = {64, 64, 64, 64, 8 * DC_MAX_T, DC_MAX_T * V * 4, (size_t)DC_HISTORY_CAP * DC_MAX_T * 4, 4};
+    for (int i = 0; i < 8; ++i) {
+        DC_TRY(dc_check_cuda(ctx, cudaMalloc(common[i], bytes[i] + 256), "step buffer"));
+        DC_TRY(dc_check_cuda(ctx, cudaMemsetAsync(*common[i], 0, bytes[i] + 256, ctx->stream), "step buffer"));
+    }
+    DC_TRY(dc_check_cuda(ctx, cudaMallocHost((void**)&m->h_stage, 4096), "cudaMallocHost"));
+    b.cap = (int)C;
+    return dc_check_cuda(ctx, cudaStreamSynchronize(ctx->stream), "finalize");
+}
+
+// ---------------------------------------------------------------- one step
+namespace {
+
+struct StepKeys {                       // prompt attention: gathered key ranges per window, query tiles
+    std::vector<const int32_t*> base;   // device, [entries + 1]
+    std::vector<int> count;
+    const int32_t* tiles = nullptr;
+    int n_tiles = 0;
+};
+
+// The tensor map of a step buffer's first K columns, made at its first use.
+int tc_in(dc_model* m, dc_tc_in* out, const __nv_bfloat16* x, int K, int ld, int rows) {
+    auto key = std::make_pair((const void*)x, K);
+    auto it = m->stack->ins.find(key);
+    if (it == m->stack->ins.end() || it->second.ld != ld) {
+        dc_tc_in in;
+        in.x = x, in.K = K, in.ld = ld;
+        DC_TRY(dc_lin_encode(m->ctx, &in.map, x, rows, K, ld));
+        m->stack->ins[key] = in;
+        it = m->stack->ins.find(key);
+    }
+    *out = it->second;
+    return DC_B200_OK;
+}
+
+// y = W x for the step's tokens: xf is the f32 input, xb its bf16 copy (tensor-core steps), same pitch.
+int linear(dc_model* m, const dc_step& st, const dc_lin& w, const float* xf, const __nv_bfloat16* xb, int ldx, int epi, float* out,
+           __nv_bfloat16* outb, int ldo) {
+    if (st.tc) {
+        dc_tc_in in;
+        DC_TRY(tc_in(m, &in, xb, w.K, ldx, m->stack->b.cap));
+        return dc_launch_linear_tc(m->ctx, w, in, st.T, epi, outb ? nullptr : out, outb, ldo);
+    }
+    if (st.T <= DC_MAX_T) return dc_launch_linear_rows(m->ctx, w, xf, ldx, st.T, epi, out, ldo);
+    return dc_launch_linear_f32(m->ctx, w, xf, ldx, st.T, epi, out, ldo);
+}
+
+// cls: kernel class of the per-class timing; bytes: what its launches have to read and write
+#define L(cls, bytes, n, expr)                                           \
+    do {                                                                 \
+        dc_model::ProfRec r_ = {cls, nullptr, nullptr, (double)(bytes)}; \
+        if (m->prof) {                                                   \
+            cudaEventCreate(&r_.e0);                                     \
+            cudaEventCreate(&r_.e1);                                     \
+            cudaEventRecord(r_.e0, ctx->stream);                         \
+        }                                                                \
+        DC_TRY(expr);                                                    \
+        if (m->prof) {                                                   \
+            cudaEventRecord(r_.e1, ctx->stream);                         \
+            m->prof_recs.push_back(r_);                                  \
+        }                                                                \
+        m->last_launches += (n);                                         \
+    } while (0)
+
+double lin_bytes(const dc_lin& w, int T) { return (double)w.N * w.ld * 2 + (double)T * (w.N + w.K) * 4; }
+
+int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
+    const dc_delta_mixer& d = Ly.dl;
+    const dc_stack_buffers& b = m->stack->b;
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
+    const int ldp = d.in.N, lda = dc_pad8(d.off_v + d.heads * d.vdim), ldl = d.in.N - d.off_a, ldm = d.heads * d.vdim;
+    __nv_bfloat16* lowb = st.tc ? b.lowb : nullptr;
+    DC_TRY(dc_launch_delta_prep(m->ctx, d, st, sr, b.proj, ldp, b.act, lda, b.small, lowb, ldl));
+    if (st.tc) {
+        DC_TRY(linear(m, st, d.a2, nullptr, lowb, ldl, DC_LIN_STORE, b.low, nullptr, d.a2.N));
+        DC_TRY(linear(m, st, d.g2, nullptr, lowb + (d.off_g - d.off_a), ldl, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
+    } else {
+        DC_TRY(linear(m, st, d.a2, b.proj + d.off_a, nullptr, ldp, DC_LIN_STORE, b.low, nullptr, d.a2.N));
+        DC_TRY(linear(m, st, d.g2, b.proj + d.off_g, nullptr, ldp, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
+    }
+    return dc_launch_delta_scan(m->ctx, d, st, sr, b.act, lda, b.small, b.low, d.a2.N, b.gate, d.g2.N, m->stack->cfg.eps, b.scan,
+                                st.tc ? nullptr : b.mix, st.tc ? b.mixb : nullptr, dc_pad8(ldm));
+}
+
+int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
+    const dc_ssd_mixer& d = Ly.ssd;
+    const dc_stack_buffers& b = m->stack->b;
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
+    const int inner = d.heads * d.vdim, lda = dc_pad8(inner + 2 * d.groups * d.state);
+    return dc_launch_ssd(m->ctx, d, st, sr, b.proj, d.in.N, b.act, lda, b.small, b.scan, m->stack->cfg.eps, st.tc ? nullptr : b.mix,
+                         st.tc ? b.mixb : nullptr, dc_pad8(inner));
+}
+
+int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
+    const dc_latent_mixer& d = Ly.la;
+    const dc_stack_buffers& b = m->stack->b;
+    dc_latent_cache c;
+    c.arena = m->kv.planes[d.plane].arena;
+    c.f32 = m->stack->dtype == DC_DTYPE_F32;
+    c.tables = m->kv.d_tables;
+    c.max_blocks = m->kv.max_blocks_per_seq;
+    const int ldp = d.in.N, ldm = dc_pad8(d.heads * d.vdim);
+    DC_TRY(dc_launch_latent_prep(m->ctx, d, st, c, b.proj, ldp, m->stack->cfg.eps, m->cfg.max_ctx));
+    if (!st.tc)
+        return dc_launch_latent_absorbed(m->ctx, d, st, c, b.proj, ldp, st.T <= DC_MAX_T ? m->stack->splits : 1, b.qa, b.part, b.part_ml, b.mix, ldm);
+    const int32_t* base = sk.base[d.range];
+    const int nk = sk.count[d.range], ldc = dc_pad8(d.kv_rank), ldr = dc_pad8(d.rot_dim);
+    DC_TRY(dc_launch_latent_gather(m->ctx, d, st, c, base, nk, b.keys_c, ldc, b.keys_r, ldr));
+    dc_tc_in in;
+    DC_TRY(tc_in(m, &in, b.keys_c, d.kv_rank, ldc, b.key_cap));
+    DC_TRY(dc_launch_linear_tc(m->ctx, d.ukv, in, nk, DC_LIN_STORE, nullptr, b.keys_kv, d.ukv.N));
+    return dc_launch_latent_prefill(m->ctx, d, st, base, sk.tiles, sk.n_tiles, b.proj, ldp, b.keys_kv, d.ukv.N, b.keys_r, ldr, b.mixb, ldm);
+}
+
+// Embedding and every layer; the residual ends in b.x.
+int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    const int W = s->cfg.width, H = dc_pad8(W), T = st.T;
+    const float eps = s->cfg.eps;
+    __nv_bfloat16* xb = st.tc ? b.xb : nullptr;
+    auto capture = [&](int il) -> int {     // parity aid: what enters layer il (the last slot: the output norm)
+        if (!m->dbg_x || T > DC_MAX_T) return DC_B200_OK;
+        return dc_check_cuda(ctx, cudaMemcpy2DAsync(m->dbg_x + (size_t)il * DC_MAX_T * W, (size_t)W * 4, b.x, (size_t)H * 4, (size_t)W * 4, T,
+                                                    cudaMemcpyDeviceToDevice, ctx->stream), "capture");
+    };
+    m->last_launches = 0;
+    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, b.x, H, xb));
+    for (size_t il = 0; il < s->layers.size(); ++il) {
+        dc_stack_layer& Ly = s->layers[il];
+        DC_TRY(capture((int)il));
+        const dc_lin& in = Ly.kind == DC_MIX_DELTA ? Ly.dl.in : Ly.kind == DC_MIX_SSD ? Ly.ssd.in : Ly.la.in;
+        const dc_lin& o = Ly.kind == DC_MIX_DELTA ? Ly.dl.o : Ly.kind == DC_MIX_SSD ? Ly.ssd.o : Ly.la.o;
+        L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.x, xb, H, DC_LIN_STORE, b.proj, nullptr, in.N));
+        if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, 7, mix_delta(m, st, Ly));
+        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, 4, mix_ssd(m, st, Ly));
+        else L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, Ly));
+        L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), DC_LIN_STORE, b.y, nullptr, H));
+        L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));
+        if (!Ly.ff) continue;
+        const int F = dc_pad8(Ly.ff);
+        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, DC_LIN_GELU_PAIR, b.ff, st.tc ? b.ffb : nullptr, F));
+        L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, DC_LIN_STORE, b.y, nullptr, H));
+        L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm2, T, W, H, eps, xb));
+    }
+    return capture((int)s->layers.size());
+}
+
+// Logits and greedy picks of R <= DC_MAX_T rows (rows: device list, or first, first + 1, ...).
+int run_head(dc_model* m, const int32_t* rows, int first, int R, bool feedback) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    const int W = s->cfg.width, H = dc_pad8(W);
+    dc_step_buffers& g = m->buf;
+    L(DC_K_POST_NORM, 8.0 * R * W, 1, dc_launch_norm_rows(ctx, s->b.x, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, H));
+    L(DC_K_LM_HEAD, lin_bytes(s->head, R), 1, dc_launch_linear_rows(ctx, s->head, s->b.lm_x, H, R, DC_LIN_STORE, g.logits, s->cfg.vocab, g.argmax_keys));
+    L(DC_K_ARGMAX, 64.0, 1, dc_launch_argmax_finish(ctx, g.argmax_keys, R, g.out_tokens, feedback ? g.tokens : nullptr, feedback ? g.positions : nullptr,
+                                                    feedback ? g.history : nullptr, feedback ? g.history_len : nullptr, DC_HISTORY_CAP));
+    return DC_B200_OK;
+}
+#undef L
+
+}  // namespace
+
+int dc_stack_enqueue_small(dc_model* m, int T, bool chunk, int lm_mode, bool feedback) {
+    dc_step st;
+    st.T = T;
+    st.E = chunk ? 1 : T;
+    st.tokens = m->buf.tokens, st.seq_ids = m->buf.seq_ids, st.positions = m->buf.positions;
+    st.starts = chunk ? m->stack->b.chunk + 2 * T : m->stack->b.iota;
+    st.single = !chunk || T == 1;
+    DC_TRY(run_layers(m, st, StepKeys()));
+    if (lm_mode == 1) return run_head(m, nullptr, T - 1, 1, feedback);
+    return lm_mode ? run_head(m, nullptr, 0, T, feedback) : DC_B200_OK;
+}
+
+int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, int n_rows, const int32_t* rows,
+                   float* logits_host, int32_t* picks_host) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    const int C = b.cap, V = s->cfg.vocab;
+    std::vector<int> done(E, 0), offset(E, 0);
+    int total = 0;
+    for (int e = 0; e < E; ++e) offset[e] = total, total += counts[e];
+    int next_row = 0;                   // rows are ascending; sub-steps take entries front to back
+    std::vector<int> order;             // flat token index of every token of the sub-step
+    for (int left = total; left > 0;) {
+        if (b.meta_slot == 0) DC_TRY(dc_check_cuda(ctx, cudaStreamSynchronize(ctx->stream), "sync"));
+        int32_t* h = b.h_meta + (size_t)b.meta_slot * b.meta_ints;
+        b.meta_slot = (b.meta_slot + 1) % DC_STACK_META_SLOTS;
+        int32_t *h_tok = h, *h_seq = h + C, *h_pos = h + 2 * C, *h_rows = h + 3 * C, *h_start = h + 4 * C;
+        int32_t* h_base = h_start + ENTRY_INTS;
+        int32_t* h_tiles = h_base + ENTRY_INTS * s->windows.size();
+        order.clear();
+        StepKeys sk;
+        sk.count.assign(s->windows.size(), 0);
+        dc_step st;
+        st.single = true;
+        for (int e = 0; e < E && st.T < C; ++e) {
+            const int n = std::min(counts[e] - done[e], C - st.T);
+            if (n <= 0) continue;
+            const int pos0 = m->kv.seqs[seqs[e]].len;
+            h_start[st.E] = st.T;
+            for (size_t w = 0; w < s->windows.size(); ++w) {
+                h_base[w * ENTRY_INTS + st.E] = sk.count[w];
+                sk.count[w] += pos0 + n - (s->windows[w] > 0 ? std::max(0, pos0 - s->windows[w] + 1) : 0);
+            }
+            for (int q = 0; q < n; q += DC_LATENT_QTILE) {
+                h_tiles[2 * sk.n_tiles] = st.E;
+                h_tiles[2 * sk.n_tiles + 1] = q;
+                ++sk.n_tiles;
+            }
+            for (int i = 0; i < n; ++i) {
+                h_tok[st.T + i] = tokens[offset[e] + done[e] + i];
+                h_seq[st.T + i] = seqs[e];
+                h_pos[st.T + i] = pos0 + i;
+                order.push_back(offset[e] + done[e] + i);
+            }
+            st.single &= n == 1;
+            st.T += n;
+            ++st.E;
+            done[e] += n;
+            m->kv.seqs[seqs[e]].len += n;
+        }
+        h_start[st.E] = st.T;
+        for (size_t w = 0; w < s->windows.size(); ++w) h_base[w * ENTRY_INTS + st.E] = sk.count[w];
+        left -= st.T;
+        int R = 0;
+        for (int i = 0; i < st.T && next_row + R < n_rows; ++i)
+            if (order[i] == rows[next_row + R]) h_rows[R++] = i;
+        DC_TRY(dc_check_cuda(ctx, cudaMemcpyAsync(b.meta, h, (size_t)b.meta_ints * 4, cudaMemcpyHostToDevice, ctx->stream), "H2D step"));
+        st.tokens = b.meta, st.seq_ids = b.meta + C, st.positions = b.meta + 2 * C, st.starts = b.meta + (h_start - h);
+        for (size_t w = 0; w < s->windows.size(); ++w) sk.base.push_back(b.meta + (h_base - h) + w * ENTRY_INTS);
+        sk.tiles = b.meta + (h_tiles - h);
+        // more tokens than the row-streaming products take at once: tensor cores (bf16 models)
+        st.tc = s->dtype == DC_DTYPE_BF16 && st.T > DC_MAX_T;
+        DC_TRY(run_layers(m, st, sk));
+        for (int r = 0; r < R; r += DC_MAX_T) {
+            const int n = std::min(DC_MAX_T, R - r);
+            DC_TRY(run_head(m, b.meta + 3 * C + r, 0, n, false));
+            if (logits_host)
+                DC_TRY(dc_check_cuda(ctx, cudaMemcpyAsync(logits_host + (size_t)(next_row + r) * V, m->buf.logits, (size_t)n * V * 4, cudaMemcpyDeviceToHost,
+                                                          ctx->stream), "D2H logits"));
+            if (picks_host)
+                DC_TRY(dc_check_cuda(ctx, cudaMemcpyAsync(picks_host + next_row + r, m->buf.out_tokens, (size_t)n * 4, cudaMemcpyDeviceToHost, ctx->stream),
+                                     "D2H picks"));
+        }
+        next_row += R;
+    }
+    return logits_host || picks_host ? dc_b200_synchronize(ctx) : DC_B200_OK;
+}
+
+void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token) {
+    dc_stack* s = m->stack;
+    if (weight_bytes) *weight_bytes = (double)s->weight_bytes - (double)s->embed->bytes + (double)s->embed->row_bytes;
+    double kv = 0.0;
+    for (dc_stack_layer& L : s->layers)
+        if (L.kind == DC_MIX_LATENT) kv += (double)m->kv.planes[L.la.plane].row_bytes;
+    if (kv_bytes_per_token) *kv_bytes_per_token = kv;
+}

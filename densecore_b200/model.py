@@ -3,6 +3,7 @@ over dc_b200_model_* (the chained ops of one Qwen3-style decoder step)."""
 from __future__ import annotations
 
 import ctypes as C
+import json
 from dataclasses import dataclass, asdict
 
 import numpy as np
@@ -10,6 +11,9 @@ import numpy as np
 from . import _lib
 from .blocks import GGML_TYPE_F32, GGML_TYPE_Q4_K, GGML_TYPE_Q6_K, row_bytes
 from .ops import Context, _vp
+
+
+DTYPES = {"bfloat16": 0, "float32": 1}      # of layer-list decoders
 
 
 @dataclass
@@ -81,6 +85,10 @@ class Model:
         h = C.c_void_p()
         ctx._check(_lib.lib().dc_b200_model_from_gguf(ctx.handle, path.encode(), max_seqs, max_ctx, ep_rank, ep_size,
                                                       C.byref(h)))
+        return cls._wrap(ctx, h)
+
+    @classmethod
+    def _wrap(cls, ctx: Context, h) -> "Model":
         cc = _lib.ModelConfig()
         ctx._check(_lib.lib().dc_b200_model_get_config(h, C.byref(cc)))
         self = cls.__new__(cls)
@@ -89,6 +97,22 @@ class Model:
         kw["tie_embeddings"], kw["qk_norm"] = bool(kw["tie_embeddings"]), bool(kw["qk_norm"])
         self.cfg = Config(**kw)
         return self
+
+    @classmethod
+    def from_dir(cls, ctx: Context, path: str, dtype: str = "bfloat16", max_seqs: int = 4, max_ctx: int = 2560, pool_tokens: int = 0):
+        """Layer-list decoder from a folder with config.json and model.safetensors (not yet finalized)."""
+        h = C.c_void_p()
+        ctx._check(_lib.lib().dc_b200_model_from_dir(ctx.handle, path.encode(), DTYPES[dtype], max_seqs, max_ctx, pool_tokens, C.byref(h)))
+        return cls._wrap(ctx, h)
+
+    @classmethod
+    def from_config(cls, ctx: Context, config: dict, shapes: dict | None = None, dtype: str = "bfloat16", max_seqs: int = 4,
+                    max_ctx: int = 2560, pool_tokens: int = 0):
+        """Layer-list decoder from a config alone (shapes: name -> shape for sizes the config does not give)."""
+        h = C.c_void_p()
+        ctx._check(_lib.lib().dc_b200_model_from_config(ctx.handle, json.dumps(config).encode(), json.dumps(shapes or {}).encode(), DTYPES[dtype],
+                                                        max_seqs, max_ctx, pool_tokens, C.byref(h)))
+        return cls._wrap(ctx, h)
 
     def tensor_names(self):
         n = C.c_int(0)
@@ -208,6 +232,20 @@ class Model:
         self._check(_lib.lib().dc_b200_forward_chunk(self.handle, seq, _vp(tokens), tokens.size, _vp(logits)))
         return logits
 
+    def forward_batch(self, entries, rows=(), want_logits: bool = True, want_picks: bool = False):
+        """One batch of (sequence, next tokens) entries.  rows: ascending places in the concatenated tokens; returns
+        their logits [rows, vocab] (None if not wanted), or (logits, greedy picks) with want_picks."""
+        seqs = np.array([s for s, _ in entries], dtype=np.int32)
+        toks = [np.ascontiguousarray(t, dtype=np.int32).reshape(-1) for _, t in entries]
+        counts = np.array([t.size for t in toks], dtype=np.int32)
+        flat = np.concatenate(toks) if toks else np.zeros(0, np.int32)
+        rows = np.ascontiguousarray(rows, dtype=np.int32)
+        logits = np.empty((rows.size, self.cfg.vocab), dtype=np.float32) if want_logits and rows.size else None
+        picks = np.zeros(rows.size, dtype=np.int32) if want_picks else None
+        self._check(_lib.lib().dc_b200_forward_batch(self.handle, len(toks), _vp(seqs), _vp(counts), _vp(flat), rows.size, _vp(rows),
+                                                     _vp(logits), _vp(picks)))
+        return (logits, picks) if want_picks else logits
+
     def prefix_stats(self) -> dict:
         """Prefix-cache counters: lookups, blocks hit, blocks resident, evictions, prompt tokens run."""
         out = (C.c_uint64 * 5)()
@@ -239,7 +277,7 @@ class Model:
         """One eager decode step timed per kernel class.  Returns {class: (ms, launches, algorithmic bytes)}."""
         seqs = np.ascontiguousarray(seqs, dtype=np.int32)
         tokens = np.ascontiguousarray(tokens, dtype=np.int32)
-        n = 16
+        n = 32
         ms = np.zeros(n, np.float32)
         launches = np.zeros(n, np.int32)
         nbytes = np.zeros(n, np.float64)

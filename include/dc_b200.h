@@ -296,6 +296,16 @@ DC_B200_API int dc_b200_model_tensor_names(dc_model* m, const char** names_out, 
  * dc_b200_model_ep_init (expert-parallel runs) and dc_b200_model_finalize. */
 DC_B200_API int dc_b200_model_from_gguf(dc_ctx* ctx, const char* path, int max_seqs, int max_ctx, int ep_rank,
                                         int ep_size, dc_model** out_model);
+/* Layer-list decoders: config.json names an architecture of the library's table ("Garilix") and, per layer, a mixer
+ * (channel_delta, latent_attention, mamba2) and a feed-forward.  from_dir reads config.json and model.safetensors
+ * (bf16 matrices, bf16 or f32 vectors); from_config takes the config's text and, for sizes that only a tensor's
+ * shape gives, a JSON object name -> shape (dc_b200_model_init_synthetic then fills the weights).  dtype: 0 bf16
+ * products with f32 accumulation, 1 everything in f32.  pool_tokens: tokens the cache pool holds (0: max_ctx for
+ * every sequence).  The model still needs dc_b200_model_finalize. */
+DC_B200_API int dc_b200_model_from_dir(dc_ctx* ctx, const char* dir, int dtype, int max_seqs, int max_ctx, int pool_tokens,
+                                       dc_model** out_model);
+DC_B200_API int dc_b200_model_from_config(dc_ctx* ctx, const char* config_json, const char* shapes_json, int dtype, int max_seqs,
+                                          int max_ctx, int pool_tokens, dc_model** out_model);
 DC_B200_API int dc_b200_model_get_tensor(dc_model* m, const char* name, int* ggml_type, int64_t ne[4], void** dev,
                                          size_t* bytes);
 DC_B200_API int dc_b200_model_finalize(dc_model* m);
@@ -328,6 +338,11 @@ DC_B200_API int dc_b200_decode_run(dc_model* m, const int32_t* seqs, int n_seq, 
  * token ([n, vocab], device-resident; copied to logits_host if not NULL): the
  * batched target forward of a speculative verify step. */
 DC_B200_API int dc_b200_forward_chunk(dc_model* m, int seq, const int32_t* tokens_host, int n, float* logits_host);
+/* The next tokens of up to 16 sequences as one batch: counts[e] tokens of seqs[e], concatenated in tokens_host
+ * (prompt portions of any length beside single decoded tokens).  rows (ascending places in tokens_host) asks for
+ * logits ([n_rows, vocab] to logits_host, may be NULL) and greedy picks ([n_rows] to picks_host, may be NULL). */
+DC_B200_API int dc_b200_forward_batch(dc_model* m, int n_entries, const int32_t* seqs, const int32_t* counts, const int32_t* tokens_host,
+                                      int n_rows, const int32_t* rows, float* logits_host, int32_t* picks_host);
 DC_B200_API void* dc_b200_model_logits_dev(dc_model* m);
 /* With model option "phase_timing" = 1 the persistent decode kernel accumulates, per phase
  * boundary, the nanoseconds CTA 0 spent since the previous boundary (work and barrier waits

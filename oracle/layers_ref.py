@@ -1,0 +1,229 @@
+"""Plain, slow restatement of the layer-list decoders' mechanisms in float64 numpy, one function per mechanism.
+
+TEST INFRASTRUCTURE ONLY: shares no code with the product path.  A model is (config dict, {name: ndarray});
+`forward` runs one whole sequence and returns logits and the residual after every layer; `Stepper` runs the same
+layers with carried state, any number of tokens at a time.
+"""
+from __future__ import annotations
+
+import numpy as np
+
+F = np.float64
+
+
+# ---------------------------------------------------------------- elementwise and norms
+def sigmoid(z):
+    return 1.0 / (1.0 + np.exp(-z))
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def softplus(z):
+    return np.logaddexp(0.0, z)
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (z + 0.044715 * z ** 3)))
+
+
+def rms_norm(x, w, eps):
+    """Over the last axis."""
+    return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * w
+
+
+def unit_vectors(x):
+    return x / np.sqrt(np.sum(x * x, axis=-1, keepdims=True) + 1e-6)
+
+
+def linear(x, w):
+    """x [T, K], w [N, K]."""
+    return x @ w.T
+
+
+# ---------------------------------------------------------------- time mixing pieces
+def short_conv(x, w, bias=None, history=None):
+    """Causal per-channel convolution over time: x [T, C], w [C, taps] (last column: the current token).
+    history [taps - 1, C]: the inputs before x (zeros at the start).  Returns (y, the new history)."""
+    T, taps = x.shape[0], w.shape[1]
+    if history is None:
+        history = np.zeros((taps - 1, x.shape[1]), F)
+    xx = np.concatenate([history, x], axis=0)
+    y = np.zeros_like(x)
+    for j in range(taps):
+        y += xx[j:j + T] * w[:, j]
+    if bias is not None:
+        y = y + bias
+    return y, xx[xx.shape[0] - (taps - 1):]
+
+
+def rotate_interleaved(x, pos, dims, base):
+    """x [T, H, D]: the first `dims` dimensions of every head turned by the position, pairs (2i, 2i + 1)."""
+    out = x.copy()
+    for i in range(dims // 2):
+        a = pos * base ** (-2.0 * i / dims)
+        c, s = np.cos(a)[:, None], np.sin(a)[:, None]
+        u, v = x[:, :, 2 * i], x[:, :, 2 * i + 1]
+        out[:, :, 2 * i] = u * c - v * s
+        out[:, :, 2 * i + 1] = v * c + u * s
+    return out
+
+
+def delta_rule(q, k, v, beta, g, S):
+    """Gated delta rule, token by token.  q, k, g [T, H, d]; v [T, H, e]; beta [T, H]; S [H, d, e] (changed in
+    place).  Returns o [T, H, e]."""
+    T, H = beta.shape
+    o = np.zeros((T, H, v.shape[2]), F)
+    for t in range(T):
+        for h in range(H):
+            S[h] = g[t, h][:, None] * S[h]
+            u = beta[t, h] * (v[t, h] - S[h].T @ k[t, h])
+            S[h] = S[h] + np.outer(k[t, h], u)
+            o[t, h] = S[h].T @ q[t, h]
+    return o
+
+
+def ssd_scan(x, B, C, dt, A_log, D, S):
+    """x [T, H, e]; B, C [T, G, n]; dt [T, H] (after softplus); S [H, n, e] (changed in place).  y [T, H, e]."""
+    T, H, _ = x.shape
+    per = H // B.shape[1]
+    y = np.zeros_like(x)
+    for t in range(T):
+        for h in range(H):
+            b, c = B[t, h // per], C[t, h // per]
+            S[h] = np.exp(-np.exp(A_log[h]) * dt[t, h]) * S[h] + dt[t, h] * np.outer(b, x[t, h])
+            y[t, h] = S[h].T @ c + D[h] * x[t, h]
+    return y
+
+
+def windowed_softmax(scores, i, window):
+    """scores over keys 0 .. i -> weights; keys with i - j >= window are not seen."""
+    n = scores.shape[-1]
+    seen = (i - np.arange(n)) < window if window else np.ones(n, bool)
+    s = np.where(seen, scores, -np.inf)
+    s = np.exp(s - s.max(axis=-1, keepdims=True))
+    return s / s.sum(axis=-1, keepdims=True)
+
+
+# ---------------------------------------------------------------- mixers
+def mix_channel_delta(h, P, m, eps, st):
+    T, H, KH, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    z = {}
+    for n in "qkv":
+        y, st["conv." + n] = short_conv(linear(h, P[n]), P[n + ".conv"], None, st.get("conv." + n))
+        z[n] = silu(y)
+    of = np.arange(H) // (H // KH)
+    q = unit_vectors(z["q"].reshape(T, KH, d))[:, of] * d ** -0.5
+    k = unit_vectors(z["k"].reshape(T, KH, d))[:, of]
+    v = z["v"].reshape(T, H, e)
+    beta = sigmoid(linear(h, P["b"]))
+    raw = linear(linear(h, P["a1"]), P["a2"]) + P["dt_bias"].reshape(-1)
+    g = np.exp(-np.exp(P["A_log"].reshape(-1))[None, :, None] * softplus(raw).reshape(T, H, d))
+    if "S" not in st:
+        st["S"] = np.zeros((H, d, e), F)
+    o = delta_rule(q, k, v, beta, g, st["S"])
+    o = rms_norm(o, P["norm"], eps) * sigmoid(linear(linear(h, P["g1"]), P["g2"])).reshape(T, H, e)
+    return linear(o.reshape(T, H * e), P["o"])
+
+
+def mix_mamba2(h, P, m, eps, st):
+    T, H, e, N, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
+    inner = H * e
+    z, xbc, dt = np.split(linear(h, P["in"]), [inner, 2 * inner + 2 * G * N], axis=1)
+    y, st["conv"] = short_conv(xbc, P["conv"], P["conv.b"], st.get("conv"))
+    x, B, C = np.split(silu(y), [inner, inner + G * N], axis=1)
+    dt = softplus(dt + P["dt_bias"].reshape(-1))
+    if "S" not in st:
+        st["S"] = np.zeros((H, N, e), F)
+    y = ssd_scan(x.reshape(T, H, e), B.reshape(T, G, N), C.reshape(T, G, N), dt, P["A_log"].reshape(-1), P["D"].reshape(-1), st["S"])
+    y = y.reshape(T, inner) * silu(z)
+    ng = m["norm_groups"]
+    y = rms_norm(y.reshape(T, ng, inner // ng), 1.0, eps).reshape(T, inner) * P["norm"]
+    return linear(y, P["o"])
+
+
+def mix_latent_attention(h, P, m, eps, pos, cache):
+    """cache: {"c": [n, kv_rank], "r": [n, rot_dim]} holding every token up to and including these (see
+    latent_append)."""
+    T, H, d, r, e = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
+    q = linear(h, P["q"]).reshape(T, H, d + r)
+    qu, qr = q[:, :, :d], rotate_interleaved(q[:, :, d:], pos, m["rot"]["dims"], m["rot"]["base"])
+    c, kr = cache["c"], cache["r"]
+    ku = linear(c, P["uk"]).reshape(-1, H, d)
+    v = linear(c, P["uv"]).reshape(-1, H, e)
+    window = (m.get("mask") or {}).get("size")
+    out = np.zeros((T, H, e), F)
+    for t in range(T):
+        n = int(pos[t]) + 1
+        s = (np.einsum("hd,nhd->hn", qu[t], ku[:n]) + np.einsum("hr,nr->hn", qr[t], kr[:n])) * m["scale"]
+        out[t] = np.einsum("hn,nhe->he", windowed_softmax(s, n - 1, window), v[:n])
+    return linear(out.reshape(T, H * e), P["o"])
+
+
+def latent_append(h, P, m, eps, pos, cache):
+    kv = linear(h, P["dkv"])
+    c = rms_norm(kv[:, :m["kv_rank"]], P["dkv.norm"], eps)
+    kr = rotate_interleaved(kv[:, None, m["kv_rank"]:], pos, m["rot"]["dims"], m["rot"]["base"])[:, 0]
+    if "c" in cache:
+        c, kr = np.concatenate([cache["c"], c]), np.concatenate([cache["r"], kr])
+    cache["c"], cache["r"] = c, kr
+
+
+def dense_mlp(h, P):
+    return linear(gelu_tanh(linear(h, P["gate"])) * linear(h, P["up"]), P["down"])
+
+
+# ---------------------------------------------------------------- the decoder
+class Stepper:
+    def __init__(self, config: dict, tensors: dict):
+        self.c = config
+        self.w = {k: np.asarray(v, F) for k, v in tensors.items()}
+        self.pos = 0
+        self.state = [dict() for _ in config["layers"]]
+
+    def part(self, prefix):
+        return {k[len(prefix):]: v for k, v in self.w.items() if k.startswith(prefix)}
+
+    def step(self, tokens, trace=None):
+        """Runs the next tokens of the sequence; returns their logits [n, vocab].  trace (a list) receives the
+        residual after every layer."""
+        tokens = np.asarray(tokens)
+        pos = self.pos + np.arange(tokens.size)
+        eps = self.c["norm"]["eps"]
+        x = self.w["embed"][tokens]
+        for i, L in enumerate(self.c["layers"]):
+            P, m, st = self.part(f"l{i}.mix."), L["mixer"], self.state[i]
+            if L["type"] == "channel_delta":
+                y = mix_channel_delta(x, P, m, eps, st)
+            elif L["type"] == "mamba2":
+                y = mix_mamba2(x, P, m, eps, st)
+            elif L["type"] == "latent_attention":
+                src = m.get("kv_from")
+                if src is None:
+                    latent_append(x, P, m, eps, pos, st)
+                y = mix_latent_attention(x, P, m, eps, pos, st if src is None else self.state[src])
+            else:
+                raise ValueError(L["type"])
+            x = x + rms_norm(y, self.w[f"l{i}.norm1"], eps)
+            if L.get("mlp"):
+                x = x + rms_norm(dense_mlp(x, self.part(f"l{i}.mlp.")), self.w[f"l{i}.norm2"], eps)
+            if trace is not None:
+                trace.append(x.copy())
+        self.pos += tokens.size
+        return linear(rms_norm(x, self.w["final.norm"], eps), self.w["head"])
+
+
+def forward(config, tensors, tokens):
+    """(logits [T, vocab], residual after every layer [layers, T, width]) of one whole sequence."""
+    tr = []
+    lg = Stepper(config, tensors).step(tokens, tr)
+    return lg, np.stack(tr)
+
+
+def greedy(config, tensors, prompt, n):
+    s = Stepper(config, tensors)
+    out = [int(np.argmax(s.step(prompt)[-1]))]
+    while len(out) < n:
+        out.append(int(np.argmax(s.step([out[-1]])[-1])))
+    return out
