@@ -351,6 +351,80 @@ def bench_dense_0p8b(ctx, peak_gbs: float, n_decode: int = 256) -> dict:
             "prefill_512_ms": prefill_s * 1e3}
 
 
+def garilix_config(width: int, repeats: int, vocab: int = 32768):
+    """A Garilix decoder whose layers have the sizes of a real model of this width (two delta-rule, two latent
+    attention and two Mamba-2 layers per repeat; the second attention layer reads the first one's cache), and the
+    shapes that its config does not give."""
+    h = width // 128
+    delta = {"type": "channel_delta", "mixer": {"heads": h, "kv_heads": h, "dim": 128, "vdim": 128, "conv": 4}}
+    ssd = {"type": "mamba2", "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}}
+    layers, shapes = [], {}
+    for r in range(repeats):
+        for half in range(2):
+            att = {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "mask": {"size": 1024},
+                   "rot": {"base": 10000.0, "dims": 64}}
+            if half:
+                att["kv_from"] = 6 * r + 1
+            shapes[f"l{len(layers)}.mix.a1"] = shapes[f"l{len(layers)}.mix.g1"] = [128, width]
+            layers += [dict(delta), {"type": "latent_attention", "mixer": att}, dict(ssd)]
+    for ly in layers:
+        ly["mlp"] = {"kind": "dense", "ff": 3 * width}
+    return {"architecture": "Garilix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": layers}, shapes
+
+
+def time_decoder(m, vocab: int, prompt: int, streams, steps: int, reps: int = 5) -> dict:
+    """Prompt throughput (host tokens in, first token out, best of reps on fresh sequences) and greedy decode after
+    that prompt (device time of decode_run) of any decoder of the library."""
+    rng = np.random.default_rng(3)
+    toks = rng.integers(0, vocab, size=prompt)
+    best = 1e9
+    for _ in range(reps + 1):
+        s = m.seq_alloc()
+        t0 = time.perf_counter()
+        m.prefill(s, toks)
+        best = min(best, time.perf_counter() - t0)
+        m.seq_free(s)
+    out = {"prompt_tokens": prompt, "prefill_ms": best * 1e3, "prefill_tok_s": prompt / best, "decode": {}}
+    seqs, first = [], []
+    for _ in range(max(streams)):
+        seqs.append(m.seq_alloc())
+        first.append(m.prefill(seqs[-1], rng.integers(0, vocab, size=prompt)))
+    _, wbytes, kvb = m.step_stats()
+    for n in streams:
+        run, _ = m.decode_run(seqs[:n], first[:n], 8)
+        run, ms = m.decode_run(seqs[:n], run[-1], steps)
+        out["decode"][str(n)] = {"ms_per_step": ms / steps, "tok_s": n * steps / (ms * 1e-3), "kernels_per_step": m.step_stats()[0],
+                                 "weight_bytes": wbytes, "weight_gbs": wbytes / (ms / steps * 1e-3) / 1e9}
+    for s in seqs:
+        m.seq_free(s)
+    return out
+
+
+def bench_garilix(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), repeats: int = 2, prompt: int = 2048) -> dict:
+    """Garilix decoders (bf16, random weights) beside the library's dense K-quant decoder of the same width, depth,
+    feed-forward and vocabulary.  Decode reads more weights than the L2 holds at the larger widths; no flush."""
+    import densecore_b200 as dc
+    out = {"vocab": 32768, "layers": 6 * repeats, "sizes": {}}
+    for w in widths:
+        cfg, shapes = garilix_config(w, repeats)
+        m = dc.Model.from_config(ctx, cfg, shapes, max_seqs=4, max_ctx=prompt + 512)
+        m.init_synthetic(11, 0.02)
+        m.finalize()
+        a = time_decoder(m, cfg["vocab"], prompt, (1, 4), steps)
+        m.close()
+        d = dc.Model(ctx, dc.Config(n_layer=6 * repeats, hidden=w, n_head=w // 128, n_kv_head=max(1, w // 512), vocab=cfg["vocab"], ffn=3 * w,
+                                    max_seqs=4, max_ctx=prompt + 512))
+        d.init_synthetic(11, 0.02)
+        d.finalize()
+        b = time_decoder(d, cfg["vocab"], prompt, (1, 4), steps)
+        d.close()
+        for r in (a, b):
+            for v in r["decode"].values():
+                v["hbm_fraction"] = v["weight_gbs"] / peak_gbs
+        out["sizes"][str(w)] = {"garilix_bf16": a, "dense_kquant": b}
+    return out
+
+
 def spec_sweep(ctx, model, cfg, rng, seqs_to_free) -> dict:
     """Config 5: target = the benchmark model, draft = the dense 0.8B-class model, gamma 4, 1024-token prompt,
     128 output tokens; greedy accept with synthetic drafts at forced 0 / 50 / 100 % acceptance, and the
@@ -424,6 +498,8 @@ def run_single_op(args) -> int:
         out = op_gemm(ctx, B.GGML_TYPE_Q6_K, 2048, 768, 4096, args.steps)
     elif args.op == "moe-layer":
         out = {"T": moe_layer_sweep(ctx, args.steps, peak)}
+    elif args.op == "garilix":
+        out = bench_garilix(ctx, args.steps, peak)
     elif args.op == "dense-0p8b":
         out = bench_dense_0p8b(ctx, peak)
     else:
@@ -456,7 +532,7 @@ def main():
     ap.add_argument("--profiler-range", action="store_true",
                     help="bracket the timed 1-stream decode run with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
     ap.add_argument("--no-extras", action="store_true", help="skip the other workloads (single ops, dense model, speculative sweep)")
-    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b"],
+    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix"],
                     help="time one operator alone and print its own JSON line (not the benchmark line)")
     args = ap.parse_args()
     if args.warmup < 3:
