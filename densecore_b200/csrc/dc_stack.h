@@ -120,7 +120,7 @@ struct dc_stack_buffers {
     int32_t* h_meta = nullptr;  // pinned, DC_STACK_META_SLOTS slots
     int meta_ints = 0, meta_slot = 0;
     int32_t *iota = nullptr, *chunk = nullptr;   // constant entry starts: one token each; one entry of n tokens at chunk + 2 n
-    float *x = nullptr, *y = nullptr, *proj = nullptr, *act = nullptr, *scan = nullptr, *low = nullptr, *gate = nullptr, *small = nullptr;
+    float *x = nullptr, *y = nullptr, *proj = nullptr, *act = nullptr, *scan = nullptr, *low = nullptr, *gate = nullptr, *small = nullptr, *blk = nullptr;
     float *mix = nullptr, *ff = nullptr, *lm_x = nullptr;
     __nv_bfloat16 *xb = nullptr, *mixb = nullptr, *ffb = nullptr, *lowb = nullptr;
     __nv_bfloat16 *keys_c = nullptr, *keys_r = nullptr, *keys_kv = nullptr;
@@ -186,15 +186,19 @@ struct dc_state_ref {           // per-sequence state in the cache manager's slo
     uint8_t* base = nullptr;
     size_t slot_bytes = 0, state_off = 0, ring_off = 0;
 };
+// most blocks that T tokens of E entries make; floats of one block's shared factors, all heads
+int dc_scan_blocks(int T, int E);
+size_t dc_delta_block_floats(const dc_delta_mixer& m);
+size_t dc_ssd_block_floats(const dc_ssd_mixer& m);
 int dc_launch_delta_prep(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp,
                          float* act, int lda, float* small, __nv_bfloat16* lowb, int ldl);
 int dc_launch_delta_scan(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act, int lda,
-                         const float* small, float* decay, int ldd, const float* raw_g, int ldg, float eps, float* o,
+                         const float* small, const float* low, int ldd, float* blk, const float* raw_g, int ldg, float eps, float* o,
                          float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp,
                            float eps, float* mix, int ldm);
 int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* act,
-                  int lda, float* small, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
+                  int lda, float* small, float* blk, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y,
                          float eps, float* mix, int ldm);
 int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps);

@@ -6,9 +6,10 @@
 // from zero whatever its slot holds, so slots need no clearing when they change hands.
 //
 // Value columns of S never mix: a column c obeys S_c <- g S_c; u = beta (v_c - S_c . k); S_c <- S_c + u k;
-// o_c = S_c . q.  k_state_scan gives each column to eight lanes and walks an entry's tokens with the column in
-// registers.  Since o_c = (g S_c) . q + (k . q) u, both dot products of a token share one reduction.  The arithmetic
-// of a token does not depend on where an entry starts, so cutting a prompt changes nothing.
+// o_c = S_c . q.  A single token (decode) is done as written, by one kernel per mixer from projections to normed
+// output.  Longer entries go through blocks of sixteen tokens (see "blocks of sixteen tokens" below): what a head's
+// columns share is computed once per block, and k_state_scan walks the blocks with each column in the registers of
+// eight lanes.  All of it is f32 on the CUDA cores.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -74,7 +75,7 @@ struct DeltaPrep {
     float unit_eps, q_scale;
     float* act;
     int lda;
-    float* small;            // [T][heads + kv_heads]: beta, then k . q
+    float* small;            // [T][heads]: step sizes
     __nv_bfloat16* lowb;     // bf16 copy of the low-rank inputs (columns off_a ..)
     int ldl, T, v_items;
 };
@@ -106,20 +107,16 @@ __global__ void __launch_bounds__(256) k_delta_prep(DeltaPrep p) {
             sk = fmaf(k[j], k[j], sk);
         }
         const float iq = p.q_scale / sqrtf(warp_sum(sq) + p.unit_eps), ik = 1.0f / sqrtf(warp_sum(sk) + p.unit_eps);
-        float kq = 0.0f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int d = lane + 32 * j;
             q[j] *= iq;
             k[j] *= ik;
-            kq = fmaf(q[j], k[j], kq);
             if (d < p.dim) {
                 act[p.off_q + item * p.dim + d] = q[j];
                 act[p.off_k + item * p.dim + d] = k[j];
             }
         }
-        kq = warp_sum(kq);
-        if (lane == 0) p.small[(size_t)t * (p.heads + p.kv_heads) + p.heads + item] = kq;
     } else if (item < p.kv_heads + p.v_items) {
         const int c0 = (item - p.kv_heads) * 128, V = p.heads * p.vdim;
 #pragma unroll
@@ -132,192 +129,459 @@ __global__ void __launch_bounds__(256) k_delta_prep(DeltaPrep p) {
         }
     } else {
         for (int h = lane; h < p.heads; h += 32)
-            p.small[(size_t)t * (p.heads + p.kv_heads) + h] = sigmoid(p.proj[(size_t)t * p.ldp + p.off_b + h]);
+            p.small[(size_t)t * p.heads + h] = sigmoid(p.proj[(size_t)t * p.ldp + p.off_b + h]);
         if (p.lowb)
             for (int c = lane; c < p.n_low; c += 32)
                 p.lowb[(size_t)t * p.ldl + c] = __float2bfloat16_rn(p.proj[(size_t)t * p.ldp + p.off_a + c]);
     }
 }
 
-// decay[t][c] = exp(neg_a[head] * softplus(raw + dt_bias)), in place
-__global__ void __launch_bounds__(256) k_delta_decay(float* __restrict__ raw, int ld, const float* __restrict__ neg_a,
-                                                     const float* __restrict__ dt_bias, int dim, int n) {
-    pdl_launch_dependents();
-    pdl_wait();
-    float* r = raw + (size_t)blockIdx.y * ld;
-    const int c = blockIdx.x * 256 + threadIdx.x;
-    if (c < n) r[c] = expf(neg_a[c / dim] * softplus(r[c] + dt_bias[c]));
+// ---------------------------------------------------------------- blocks of sixteen tokens
+// Within a block that starts from the state S0, with cumulative decays G_t (products of g over the block's tokens up
+// to t) and products P_ti of g over (i, t]:
+//   u_t = beta_t (v_t - S0 . (G_t k_t) - sum_{i<t} A_ti u_i),   A_ti = sum_d P_ti k_i k_t
+//   o_t = S0 . (G_t q_t) + sum_{i<=t} B_ti u_i,                 B_ti = sum_d P_ti k_i q_t
+//   S   = G_15 S0 + sum_i (P_15,i k_i) u_i
+// Everything but S0, v, u and o is shared by a head's value columns and computed once per (block, head): the decayed
+// vectors, B, and W = (I + diag(beta) A)^-1 diag(beta), so that u = W (v - S0 . G k).  Every decay factor is a
+// product of g, at most 1.  The state-space scan is the same with one decay per head, no A, and u_i = dt_i x_i.
+constexpr int BT = 16, BROW = 20;                       // tokens of a block; pitch of a 16 x 16 factor (conflict-free rows)
+
+struct BlockRef {                                       // token range of a block: entries are cut from their own start
+    int e, t0, n;
+};
+__device__ __forceinline__ int block_base(const int32_t* starts, int e) {
+    int b = 0;
+    for (int i = 0; i < e; ++i) b += (starts[i + 1] - starts[i] + BT - 1) / BT;
+    return b;
+}
+__device__ __forceinline__ BlockRef block_at(const int32_t* starts, int E, int blk) {
+    for (int e = 0; e < E; ++e) {
+        const int n = starts[e + 1] - starts[e], nb = (n + BT - 1) / BT;
+        if (blk < nb) return BlockRef{e, starts[e] + blk * BT, min(BT, n - blk * BT)};
+        blk -= nb;
+    }
+    return BlockRef{0, 0, 0};
 }
 
-// ---------------------------------------------------------------- the scan
-constexpr int SC_TOK = 16, SC_COLS = 16, SC_THREADS = 128;   // tokens per staged chunk, columns per CTA
+// Sum of v[i] over the warp lands in lane i (31 shuffles for 32 sums).
+__device__ __forceinline__ float transpose_sum32(float (&v)[32], int lane) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+            if (i < o) {
+                const bool up = lane & o;
+                const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+                v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+    }
+    return v[0];
+}
+
+// Floats of one (block, head) of the delta rule: G k, G q, P k (each [16][dp]), G_15 [dp], W and B [16][20].
+__host__ __device__ constexpr int delta_block_floats(int dp) { return 3 * BT * dp + dp + 2 * BT * BROW; }
+
+struct DeltaBlock {
+    const float* act;
+    int lda, off_q, off_k, heads, per, dim, dp;
+    const float* raw;            // decay projection
+    int ldr;
+    const float *neg_a, *dt_bias, *small;
+    int lds;
+    const int32_t* starts;
+    int E;
+    float* out;
+};
+
+__global__ void __launch_bounds__(128) k_delta_blocks(const DeltaBlock p) {
+    extern __shared__ __align__(16) float sm[];         // k, q, g: [16][dim] each
+    __shared__ float sA[BT][BT + 1], sB[BT][BT], sX[BT][BT + 1], sbeta[BT];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim, dp = p.dp;
+    const BlockRef br = block_at(p.starts, p.E, blockIdx.x);
+    if (br.n <= 0) return;
+    float *sk = sm, *sq = sm + BT * dim, *sg = sm + 2 * BT * dim;
+    float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * delta_block_floats(dp);
+    if (tid < BT) sbeta[tid] = tid < br.n ? p.small[(size_t)(br.t0 + tid) * p.lds + h] : 0.0f;
+    for (int d = tid; d < dp; d += 128) {
+        float k[BT], g[BT], cum = 1.0f;
+        const bool in = d < dim;
+        const float na = p.neg_a[h], bias = in ? p.dt_bias[(size_t)h * dim + d] : 0.0f;
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+            float q = 0.0f;
+            k[t] = 0.0f, g[t] = 1.0f;
+            if (in && t < br.n) {
+                const float* a = p.act + (size_t)(br.t0 + t) * p.lda + (h / p.per) * dim + d;
+                k[t] = a[p.off_k];
+                q = a[p.off_q];
+                g[t] = expf(na * softplus(p.raw[(size_t)(br.t0 + t) * p.ldr + h * dim + d] + bias));
+            }
+            cum *= g[t];
+            out[t * dp + d] = cum * k[t];
+            out[(BT + t) * dp + d] = cum * q;
+            if (in) sk[t * dim + d] = k[t], sq[t * dim + d] = q, sg[t * dim + d] = g[t];
+        }
+        out[3 * BT * dp + d] = cum;
+        float suffix = 1.0f;
+#pragma unroll
+        for (int t = BT - 1; t >= 0; --t) {
+            out[(2 * BT + t) * dp + d] = suffix * k[t];
+            suffix *= g[t];
+        }
+    }
+    __syncthreads();
+    for (int i = warp; i < BT; i += 4) {
+        float v[32];
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] = 0.0f;
+        for (int d = lane; d < dim; d += 32) {
+            float c = sk[i * dim + d];
+#pragma unroll
+            for (int t = 0; t < BT; ++t)
+                if (t >= i) {
+                    if (t > i) {
+                        c *= sg[t * dim + d];
+                        v[t] = fmaf(c, sk[t * dim + d], v[t]);
+                    }
+                    v[BT + t] = fmaf(c, sq[t * dim + d], v[BT + t]);
+                }
+        }
+        const float r = transpose_sum32(v, lane);
+        if (lane < BT) sA[lane][i] = r;
+        else sB[lane - BT][i] = r;
+    }
+    __syncthreads();
+    if (tid < BT) {                                     // column tid of (I + diag(beta) A)^-1 diag(beta)
+        for (int t = 0; t < BT; ++t) {
+            float x = t == tid ? 1.0f : 0.0f;
+            if (t > tid) {
+                float a = 0.0f;
+                for (int i = tid; i < t; ++i) a = fmaf(sA[t][i], sX[i][tid], a);
+                x = -sbeta[t] * a;
+            }
+            sX[t][tid] = x;
+        }
+    }
+    __syncthreads();
+    float* W = out + 3 * BT * dp + dp;
+    for (int i = tid; i < BT * BT; i += 128) {
+        W[i / BT * BROW + i % BT] = sX[i / BT][i % BT] * sbeta[i % BT];
+        W[(BT + i / BT) * BROW + i % BT] = sB[i / BT][i % BT];
+    }
+}
+
+// Floats of one (block, head) of the state-space scan: M [16][20], cumulative decays [16], update factors [16].
+constexpr int SSD_BLOCK = BT * BROW + 2 * BT;
+
+struct SsdBlock {
+    const float* act;
+    int lda, off_b, off_c, heads, per, state;
+    const float* small;          // [T][2 heads]: dt, decay
+    const int32_t* starts;
+    int E;
+    float* out;
+};
+
+// One CTA per (block, group): M_ti = (C_t . B_i) P_ti dt_i for i <= t, for every head of the group.
+__global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
+    extern __shared__ __align__(16) float sm[];         // B, C: [16][state + 1]
+    __shared__ float sa[BT], sd[BT];
+    pdl_launch_dependents();
+    pdl_wait();
+    const BlockRef br = block_at(p.starts, p.E, blockIdx.x);
+    if (br.n <= 0) return;
+    const int g = blockIdx.y, tid = threadIdx.x, ld = p.state + 1, t = tid / BT, i = tid % BT;
+    float *sb = sm, *sc = sm + BT * ld;
+    for (int j = tid; j < BT * p.state; j += 256) {
+        const int tk = j / p.state, d = j - tk * p.state;
+        const float* a = p.act + (size_t)(br.t0 + tk) * p.lda + g * p.state + d;
+        sb[tk * ld + d] = tk < br.n ? a[p.off_b] : 0.0f;
+        sc[tk * ld + d] = tk < br.n ? a[p.off_c] : 0.0f;
+    }
+    __syncthreads();
+    float cb = 0.0f;
+    if (i <= t)
+        for (int d = 0; d < p.state; ++d) cb = fmaf(sc[t * ld + d], sb[i * ld + d], cb);
+    for (int hh = 0; hh < p.per; ++hh) {
+        const int h = g * p.per + hh;
+        __syncthreads();
+        if (tid < BT) {
+            const float* s = p.small + (size_t)(br.t0 + tid) * 2 * p.heads;
+            sd[tid] = tid < br.n ? s[h] : 0.0f;
+            sa[tid] = tid < br.n ? s[p.heads + h] : 1.0f;
+        }
+        __syncthreads();
+        float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * SSD_BLOCK;
+        float m = 0.0f;
+        if (i <= t) {
+            m = cb * sd[i];
+            for (int j = i + 1; j <= t; ++j) m *= sa[j];
+        }
+        out[t * BROW + i] = m;
+        if (tid < BT) {
+            float c = 1.0f, u = sd[tid];
+            for (int j = 0; j <= tid; ++j) c *= sa[j];
+            for (int j = tid + 1; j < BT; ++j) u *= sa[j];
+            out[BT * BROW + tid] = c;
+            out[BT * BROW + BT + tid] = u;
+        }
+    }
+}
+
+// ---------------------------------------------------------------- the scan over blocks
+constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp, eight lanes each
 
 struct ScanParams {
-    const float *k, *q, *v, *g;    // first head's columns; k and q of head h start at (h / per) * dim
-    int ld, ldg;                   // pitch of k, q, v and of g
-    int heads, per, dim, vdim;
-    const float* small;            // delta: beta per head, then k . q per kv head;  ssd: step and decay per head
-    int lds, small2;               // pitch, offset of the second set
+    const float* blocks;           // k_delta_blocks / k_ssd_blocks
+    const float *k, *q;            // ssd: B and C of group 0
+    const float* v;                // values of head 0
+    int ld, heads, per, dim, vdim;
     const float* D;                // ssd: per head
     float* o;
     int ldo;
     uint8_t* base;
     size_t slot_bytes, state_off;
     const int32_t *seq_ids, *positions, *starts;
-    int vec;                       // dim and pitches allow 16-byte copies
+    int vec;                       // ssd: B, C rows allow 16-byte copies
 };
 
-__device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
+__device__ __forceinline__ void cp_async4z(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(ok ? 4 : 0) : "memory");
 }
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// EPL: key channels per lane (the state's key size, padded to 8 EPL).
+// a pair of f32 values in one register pair, two multiply-adds per instruction
+__device__ __forceinline__ uint64_t pair(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(uint64_t v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ ulonglong2 lds_pairs(const float* p) { return *reinterpret_cast<const ulonglong2*>(p); }
+
+// EPL: key channels per lane (the key size, padded to 8 EPL).
 template <int EPL, bool DELTA>
 __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
-    constexpr int DP = 8 * EPL, NV = DELTA ? 3 : 2, BUF = SC_TOK * (NV * DP + SC_COLS + 2);
+    constexpr int DP = 8 * EPL, NR = DELTA ? 2 * BT : BT, BLK = DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK, BUF = BLK + BT * SC_COLS;
     extern __shared__ __align__(16) float sm[];
+    __shared__ float s_r[4][4][NR];                              // a warp's columns: S0 . G k (delta) and S0 . G q
+    __shared__ __align__(16) float s_d[4][4][BT], s_u[4][4][BT];
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, c4 = lane >> 3;
     const int c0 = blockIdx.x * SC_COLS, h = blockIdx.y, e = blockIdx.z, kh = h / p.per;
-    const int col = c0 + warp * 4 + (lane >> 3);
-    for (int i = tid; i < 2 * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels and columns stay zero
-    __syncthreads();
+    const int col = c0 + warp * 4 + c4;
+    if (!DELTA) {
+        for (int i = tid; i < 2 * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels stay zero
+        __syncthreads();
+    }
     pdl_wait();
     const int t0 = p.starts[e], t1 = p.starts[e + 1];
     if (t0 >= t1) return;
-    const int seq = p.seq_ids[t0];
+    const int seq = p.seq_ids[t0], blocks = (t1 - t0 + BT - 1) / BT;
+    const float* bsrc = p.blocks + ((size_t)block_base(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
+    const size_t bstep = (size_t)p.heads * (DELTA ? BLK : SSD_BLOCK);
     float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + col) * p.dim;
-    float s[EPL];
-    const bool fresh = p.positions[t0] == 0;
+    float sf[EPL];
+    const bool fresh = p.positions[t0] == 0, live = col < p.vdim;
 #pragma unroll
     for (int j = 0; j < EPL; ++j) {
         const int d = 4 * (l8 + 8 * (j >> 2)) + (j & 3);
-        s[j] = !fresh && col < p.vdim && d < p.dim ? S[d] : 0.0f;
+        sf[j] = !fresh && live && d < p.dim ? S[d] : 0.0f;
     }
-    auto load = [&](int chunk, int buf) {
-        float* b = sm + buf * BUF;
-        const int tb = t0 + chunk * SC_TOK, n = min(SC_TOK, t1 - tb);
-        const float* src[3] = {p.k + (size_t)kh * p.dim, p.q + (size_t)kh * p.dim, DELTA ? p.g + (size_t)h * p.dim : nullptr};
+    uint64_t s[EPL / 2];
 #pragma unroll
-        for (int a = 0; a < NV; ++a) {
-            const int ld = a == 2 ? p.ldg : p.ld;
-            float* dst = b + a * SC_TOK * DP;
-            if (p.vec) {
-                const int d4 = p.dim >> 2;
-                for (int i = tid; i < n * d4; i += SC_THREADS) {
-                    const int tk = i / d4, d = (i - tk * d4) * 4;
-                    cp_async16(smem_u32(dst + tk * DP + d), src[a] + (size_t)(tb + tk) * ld + d);
-                }
-            } else {
-                for (int i = tid; i < n * p.dim; i += SC_THREADS) {
-                    const int tk = i / p.dim, d = i - tk * p.dim;
-                    cp_async4(smem_u32(dst + tk * DP + d), src[a] + (size_t)(tb + tk) * ld + d);
+    for (int j = 0; j < EPL / 2; ++j) s[j] = pair(sf[2 * j], sf[2 * j + 1]);
+
+    auto load = [&](int b, int buf) {
+        float* dst = sm + buf * BUF;
+        const int tb = t0 + b * BT;
+        const float* src = bsrc + b * bstep;
+        if (DELTA) {
+            for (int i = tid; i < BLK / 4; i += SC_THREADS) cp_async16z(smem_u32(dst + 4 * i), src + 4 * i, true);
+        } else {
+            for (int i = tid; i < SSD_BLOCK / 4; i += SC_THREADS) cp_async16z(smem_u32(dst + 2 * BT * DP + 4 * i), src + 4 * i, true);
+#pragma unroll
+            for (int a = 0; a < 2; ++a) {
+                const float* rows = (a ? p.k : p.q) + (size_t)kh * p.dim;
+                const int w = p.vec ? 4 : 1, n = p.dim / w;
+                for (int i = tid; i < BT * n; i += SC_THREADS) {
+                    const int t = i / n, d = (i - t * n) * w;
+                    const bool ok = tb + t < t1;
+                    const float* from = ok ? rows + (size_t)(tb + t) * p.ld + d : rows;
+                    if (p.vec) cp_async16z(smem_u32(dst + (a * BT + t) * DP + d), from, ok);
+                    else cp_async4z(smem_u32(dst + (a * BT + t) * DP + d), from, ok);
                 }
             }
         }
-        float* bv = b + NV * SC_TOK * DP;
-        for (int i = tid; i < n * SC_COLS; i += SC_THREADS) {
-            const int tk = i / SC_COLS, c = i % SC_COLS;
-            if (c0 + c < p.vdim) cp_async4(smem_u32(bv + i), p.v + (size_t)(tb + tk) * p.ld + (size_t)h * p.vdim + c0 + c);
-        }
-        for (int i = tid; i < n * 2; i += SC_THREADS) {
-            const int tk = i >> 1;
-            const int off = (i & 1) ? p.small2 + (DELTA ? kh : h) : h;
-            cp_async4(smem_u32(bv + SC_TOK * SC_COLS + i), p.small + (size_t)(tb + tk) * p.lds + off);
+        for (int i = tid; i < BT * SC_COLS; i += SC_THREADS) {
+            const int t = i / SC_COLS, c = c0 + i % SC_COLS;
+            const bool ok = tb + t < t1 && c < p.vdim;
+            cp_async4z(smem_u32(dst + BLK + i), ok ? p.v + (size_t)(tb + t) * p.ld + (size_t)h * p.vdim + c : p.v, ok);
         }
         cp_async_commit();
     };
-    const int chunks = (t1 - t0 + SC_TOK - 1) / SC_TOK;
-    const float Dh = !DELTA ? p.D[h] : 0.0f;
+    const float Dh = DELTA ? 0.0f : p.D[h];
     load(0, 0);
-    for (int ch = 0; ch < chunks; ++ch) {
-        if (ch + 1 < chunks) {
-            load(ch + 1, (ch + 1) & 1);
+    for (int b = 0; b < blocks; ++b) {
+        if (b + 1 < blocks) {
+            load(b + 1, (b + 1) & 1);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
         __syncthreads();
-        const float* b = sm + (ch & 1) * BUF;
-        const float* bv = b + NV * SC_TOK * DP + warp * 4 + (lane >> 3);
-        const float* bs = b + NV * SC_TOK * DP + SC_TOK * SC_COLS;
-        const int tb = t0 + ch * SC_TOK, n = min(SC_TOK, t1 - tb);
-#pragma unroll(DELTA ? 1 : 4)
-        for (int tk = 0; tk < n; ++tk) {
-            const float4* kp = reinterpret_cast<const float4*>(b + tk * DP) + l8;
-            const float4* qp = reinterpret_cast<const float4*>(b + (SC_TOK + tk) * DP) + l8;
-            const float v = bv[tk * SC_COLS], s0 = bs[2 * tk], s1 = bs[2 * tk + 1];
-            float pk[4] = {}, pq[4] = {};
-            if (DELTA) {
-                const float4* gp = reinterpret_cast<const float4*>(b + (2 * SC_TOK + tk) * DP) + l8;
-                float kr[EPL];
+        const float* x = sm + (b & 1) * BUF;
+        const float* sv = x + BLK + warp * 4 + c4;
+        // ---- the column against the block's (decayed) keys and queries
+        uint64_t acc[NR];
 #pragma unroll
-                for (int j = 0; j < EPL / 4; ++j) {
-                    const float4 kv = kp[8 * j], qv = qp[8 * j], gv = gp[8 * j];
-                    const float kk[4] = {kv.x, kv.y, kv.z, kv.w}, qq[4] = {qv.x, qv.y, qv.z, qv.w}, gg[4] = {gv.x, gv.y, gv.z, gv.w};
+        for (int i = 0; i < NR; ++i) acc[i] = 0;
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        kr[4 * j + i] = kk[i];
-                        s[4 * j + i] *= gg[i];
-                        pk[i] = fmaf(s[4 * j + i], kk[i], pk[i]);
-                        pq[i] = fmaf(s[4 * j + i], qq[i], pq[i]);
-                    }
-                }
-                float a = (pk[0] + pk[1]) + (pk[2] + pk[3]), c = (pq[0] + pq[1]) + (pq[2] + pq[3]);
+        for (int j = 0; j < EPL / 4; ++j) {
 #pragma unroll
-                for (int o = 4; o > 0; o >>= 1) {
-                    a += __shfl_xor_sync(0xffffffffu, a, o);
-                    c += __shfl_xor_sync(0xffffffffu, c, o);
-                }
-                const float u = s0 * (v - a);
-#pragma unroll
-                for (int j = 0; j < EPL; ++j) s[j] = fmaf(kr[j], u, s[j]);
-                if (l8 == 0 && col < p.vdim) p.o[(size_t)(tb + tk) * p.ldo + (size_t)h * p.vdim + col] = fmaf(s1, u, c);
-            } else {
-                const float u = s0 * v;
-#pragma unroll
-                for (int j = 0; j < EPL / 4; ++j) {
-                    const float4 kv = kp[8 * j], qv = qp[8 * j];
-                    const float kk[4] = {kv.x, kv.y, kv.z, kv.w}, qq[4] = {qv.x, qv.y, qv.z, qv.w};
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        s[4 * j + i] = fmaf(s[4 * j + i], s1, kk[i] * u);
-                        pq[i] = fmaf(s[4 * j + i], qq[i], pq[i]);
-                    }
-                }
-                float c = (pq[0] + pq[1]) + (pq[2] + pq[3]);
-#pragma unroll
-                for (int o = 4; o > 0; o >>= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
-                if (l8 == 0 && col < p.vdim) p.o[(size_t)(tb + tk) * p.ldo + (size_t)h * p.vdim + col] = fmaf(Dh, v, c);
+            for (int i = 0; i < NR; ++i) {
+                const ulonglong2 w = lds_pairs(x + i * DP + 4 * (l8 + 8 * j));
+                acc[i] = fma2(s[2 * j], w.x, acc[i]);
+                acc[i] = fma2(s[2 * j + 1], w.y, acc[i]);
             }
+        }
+        float r[NR];
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const float2 f = unpair(acc[i]);
+            r[i] = f.x + f.y;
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) {                        // sums over the eight lanes: lane l8 keeps NR / 8 of them
+            const bool up = l8 & o;
+            const int half = NR / 8 * o;
+#pragma unroll
+            for (int i = 0; i < NR / 2; ++i)
+                if (i < half) {
+                    const float send = up ? r[i] : r[i + half], keep = up ? r[i + half] : r[i];
+                    r[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+        }
+#pragma unroll
+        for (int i = 0; i < NR / 8; ++i) s_r[warp][c4][l8 * (NR / 8) + i] = r[i];
+        __syncwarp();
+        // ---- u and o: this lane's tokens l8 and l8 + 8
+        const float* scal = x + (DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
+        float v[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int t = l8 + 8 * k;
+            v[k] = sv[t * SC_COLS];
+            s_d[warp][c4][t] = DELTA ? v[k] - s_r[warp][c4][t] : v[k];
+        }
+        __syncwarp();
+        float dv[BT];
+#pragma unroll
+        for (int i = 0; i < BT / 4; ++i) {
+            const float4 f = *reinterpret_cast<const float4*>(&s_d[warp][c4][4 * i]);
+            dv[4 * i] = f.x, dv[4 * i + 1] = f.y, dv[4 * i + 2] = f.z, dv[4 * i + 3] = f.w;
+        }
+        auto row_dot = [&](const float* row) {                   // rows of W, B, M are zero above the diagonal
+            float a[2] = {0.0f, 0.0f};
+#pragma unroll
+            for (int i = 0; i < BT / 4; ++i) {
+                const float4 f = *reinterpret_cast<const float4*>(row + 4 * i);
+                a[0] = fmaf(f.x, dv[4 * i], a[0]);
+                a[1] = fmaf(f.y, dv[4 * i + 1], a[1]);
+                a[0] = fmaf(f.z, dv[4 * i + 2], a[0]);
+                a[1] = fmaf(f.w, dv[4 * i + 3], a[1]);
+            }
+            return a[0] + a[1];
+        };
+        float out[2];
+        if (DELTA) {
+#pragma unroll
+            for (int k = 0; k < 2; ++k) s_u[warp][c4][l8 + 8 * k] = row_dot(scal + (l8 + 8 * k) * BROW);
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < BT / 4; ++i) {
+                const float4 f = *reinterpret_cast<const float4*>(&s_u[warp][c4][4 * i]);
+                dv[4 * i] = f.x, dv[4 * i + 1] = f.y, dv[4 * i + 2] = f.z, dv[4 * i + 3] = f.w;
+            }
+#pragma unroll
+            for (int k = 0; k < 2; ++k) out[k] = s_r[warp][c4][BT + l8 + 8 * k] + row_dot(scal + (BT + l8 + 8 * k) * BROW);
+        } else {
+            const float* cd = scal + BT * BROW;
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int t = l8 + 8 * k;
+                out[k] = fmaf(cd[t], s_r[warp][c4][t], row_dot(scal + t * BROW)) + Dh * v[k];
+            }
+#pragma unroll
+            for (int i = 0; i < BT; ++i) dv[i] *= cd[BT + i];
+        }
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int t = t0 + b * BT + l8 + 8 * k;
+            if (t < t1 && live) p.o[(size_t)t * p.ldo + (size_t)h * p.vdim + col] = out[k];
+        }
+        // ---- the state after the block
+        const float* keys = x + (DELTA ? 2 * BT * DP : BT * DP);
+#pragma unroll
+        for (int j = 0; j < EPL / 4; ++j) {
+            uint64_t a0 = 0, a1 = 0;
+#pragma unroll
+            for (int t = 0; t < BT; ++t) {
+                const ulonglong2 w = lds_pairs(keys + t * DP + 4 * (l8 + 8 * j));
+                const uint64_t u = pair(dv[t], dv[t]);
+                a0 = fma2(w.x, u, a0);
+                a1 = fma2(w.y, u, a1);
+            }
+            ulonglong2 g;
+            if (DELTA) g = lds_pairs(x + 3 * BT * DP + 4 * (l8 + 8 * j));
+            else g.x = g.y = pair(scal[BT * BROW + BT - 1], scal[BT * BROW + BT - 1]);
+            s[2 * j] = fma2(s[2 * j], g.x, a0);
+            s[2 * j + 1] = fma2(s[2 * j + 1], g.y, a1);
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int j = 0; j < EPL; ++j) {
-        const int d = 4 * (l8 + 8 * (j >> 2)) + (j & 3);
-        if (col < p.vdim && d < p.dim) S[d] = s[j];
+    for (int j = 0; j < EPL / 2; ++j) {
+        const float2 f = unpair(s[j]);
+        const int d = 4 * (l8 + 8 * (j >> 1)) + 2 * (j & 1);
+        if (live && d < p.dim) S[d] = f.x;
+        if (live && d + 1 < p.dim) S[d + 1] = f.y;
     }
 }
 
 template <int EPL, bool DELTA>
 int launch_scan_epl(dc_ctx* ctx, const ScanParams& p, int E) {
-    const size_t smem = (size_t)2 * SC_TOK * ((DELTA ? 3 : 2) * 8 * EPL + SC_COLS + 2) * 4;
+    constexpr int DP = 8 * EPL;
+    const size_t smem = (size_t)2 * ((DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK) + BT * SC_COLS) * 4;
     DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, DELTA>, (int)smem, "k_state_scan"));
     return dc_launch(ctx, "k_state_scan", k_state_scan<EPL, DELTA>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_THREADS), smem, p);
 }
+int key_pad(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 template <bool DELTA>
 int launch_scan(dc_ctx* ctx, const ScanParams& p, int E) {
-    if (p.dim <= 32) return launch_scan_epl<4, DELTA>(ctx, p, E);
-    if (p.dim <= 64) return launch_scan_epl<8, DELTA>(ctx, p, E);
-    if (p.dim <= 128) return launch_scan_epl<16, DELTA>(ctx, p, E);
-    return launch_scan_epl<32, DELTA>(ctx, p, E);
+    switch (key_pad(p.dim)) {
+    case 32: return launch_scan_epl<4, DELTA>(ctx, p, E);
+    case 64: return launch_scan_epl<8, DELTA>(ctx, p, E);
+    case 128: return launch_scan_epl<16, DELTA>(ctx, p, E);
+    default: return launch_scan_epl<32, DELTA>(ctx, p, E);
+    }
 }
 
 // ---------------------------------------------------------------- output norms
@@ -394,6 +658,10 @@ ConvRef conv_ref(const dc_step& st, const dc_state_ref& sr, int taps, int C) {
 
 }  // namespace
 
+int dc_scan_blocks(int T, int E) { return T / BT + E; }
+size_t dc_delta_block_floats(const dc_delta_mixer& m) { return (size_t)m.heads * delta_block_floats(key_pad(m.dim)); }
+size_t dc_ssd_block_floats(const dc_ssd_mixer& m) { return (size_t)m.heads * SSD_BLOCK; }
+
 int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps) {
     return dc_launch(ctx, "k_ring_update", k_ring_update, dim3((C + 255) / 256, st.E), dim3(256), 0, conv_ref(st, sr, taps, C), proj, ldp, off);
 }
@@ -415,18 +683,19 @@ int dc_launch_delta_prep(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st
 }
 
 int dc_launch_delta_scan(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act, int lda,
-                         const float* small, float* decay, int ldd, const float* raw_g, int ldg, float eps, float* o,
+                         const float* small, const float* low, int ldd, float* blk, const float* raw_g, int ldg, float eps, float* o,
                          float* mix, __nv_bfloat16* mixb, int ldm) {
-    const int nd = m.heads * m.dim;
-    DC_TRY(dc_launch(ctx, "k_delta_decay", k_delta_decay, dim3((nd + 255) / 256, st.T), dim3(256), 0, decay, ldd, m.neg_a, m.dt_bias, m.dim, nd));
+    const int dp = key_pad(m.dim), nb = dc_scan_blocks(st.T, st.E);
+    DeltaBlock d = {act, lda, m.off_q, m.off_k, m.heads, m.heads / m.kv_heads, m.dim, dp, low, ldd, m.neg_a, m.dt_bias, small, m.heads, st.starts, st.E, blk};
+    const size_t smem = (size_t)3 * BT * m.dim * 4;
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_delta_blocks, (int)smem, "k_delta_blocks"));
+    DC_TRY(dc_launch(ctx, "k_delta_blocks", k_delta_blocks, dim3(nb, m.heads), dim3(128), smem, d));
     ScanParams p = {};
-    p.k = act + m.off_k, p.q = act + m.off_q, p.v = act + m.off_v, p.g = decay;
-    p.ld = lda, p.ldg = ldd, p.heads = m.heads, p.per = m.heads / m.kv_heads, p.dim = m.dim, p.vdim = m.vdim;
-    p.small = small, p.lds = m.heads + m.kv_heads, p.small2 = m.heads;
+    p.blocks = blk, p.v = act + m.off_v;
+    p.ld = lda, p.heads = m.heads, p.per = m.heads / m.kv_heads, p.dim = m.dim, p.vdim = m.vdim;
     p.o = o, p.ldo = lda;
     p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
     p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
-    p.vec = m.dim % 4 == 0 && lda % 4 == 0 && ldd % 4 == 0;
     DC_TRY(launch_scan<true>(ctx, p, st.E));
     const unsigned blocks = (unsigned)(((long long)st.T * m.heads + 7) / 8);
     if (mixb)
@@ -437,16 +706,17 @@ int dc_launch_delta_scan(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st
 }
 
 int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* act,
-                  int lda, float* small, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
+                  int lda, float* small, float* blk, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
     const int inner = m.heads * m.vdim, GN = m.groups * m.state, C = inner + 2 * GN;
     SsdPrep s = {conv_ref(st, sr, m.taps, C), proj, ldp, m.off_x, m.off_dt, m.heads, st.T, m.conv, m.conv_b, m.dt_bias, m.neg_a, act, lda, small};
     DC_TRY(dc_launch(ctx, "k_ssd_prep", k_ssd_prep, dim3((C + 255) / 256, st.T), dim3(256), 0, s));
     DC_TRY(dc_launch_ring_update(ctx, st, sr, proj, ldp, m.off_x, C, m.taps));
+    SsdBlock sb = {act, lda, inner, inner + GN, m.heads, m.heads / m.groups, m.state, small, st.starts, st.E, blk};
+    DC_TRY(dc_launch(ctx, "k_ssd_blocks", k_ssd_blocks, dim3(dc_scan_blocks(st.T, st.E), m.groups), dim3(256), (size_t)2 * BT * (m.state + 1) * 4, sb));
     ScanParams p = {};
-    p.k = act + inner, p.q = act + inner + GN, p.v = act;
+    p.blocks = blk, p.k = act + inner, p.q = act + inner + GN, p.v = act;
     p.ld = lda, p.heads = m.heads, p.per = m.heads / m.groups, p.dim = m.state, p.vdim = m.vdim;
-    p.small = small, p.lds = 2 * m.heads, p.small2 = m.heads, p.D = m.D;
-    p.o = y, p.ldo = lda;
+    p.D = m.D, p.o = y, p.ldo = lda;
     p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
     p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
     p.vec = m.state % 4 == 0 && lda % 4 == 0 && inner % 4 == 0;

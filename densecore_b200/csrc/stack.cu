@@ -217,18 +217,20 @@ int dc_stack_finalize(dc_model* m) {
     const long long all = (long long)m->cfg.max_seqs * m->cfg.max_ctx;
     const size_t C = std::max<long long>(DC_MAX_T, std::min<long long>(m->prefill_chunk, all));
     const size_t F = f32 ? C : DC_MAX_T;      // rows of buffers that only the f32 path uses
-    size_t proj = 8, act = 8, low = 8, gate = 8, small = 8, mix = 8, ff = 8, lowb = 8, rank = 8, rot = 8, ukv = 8, qa = 0, part = 0, ml = 0;
+    size_t proj = 8, act = 8, low = 8, gate = 8, small = 8, mix = 8, ff = 8, lowb = 8, rank = 8, rot = 8, ukv = 8, blk = 8, qa = 0, part = 0, ml = 0;
     int span = 1;
     for (dc_stack_layer& L : s->layers) {
         auto up = [](size_t& a, long long v) { a = std::max(a, (size_t)dc_pad8((int)v)); };
         up(ff, L.ff);
         if (L.kind == DC_MIX_DELTA) {
             const dc_delta_mixer& d = L.dl;
-            up(proj, d.in.N), up(act, d.off_v + d.heads * d.vdim), up(low, d.a2.N), up(gate, d.g2.N), up(small, d.heads + d.kv_heads);
+            up(proj, d.in.N), up(act, d.off_v + d.heads * d.vdim), up(low, d.a2.N), up(gate, d.g2.N), up(small, d.heads);
+            blk = std::max(blk, dc_delta_block_floats(d));
             up(mix, d.heads * d.vdim), up(lowb, d.in.N - d.off_a);
         } else if (L.kind == DC_MIX_SSD) {
             const dc_ssd_mixer& d = L.ssd;
             up(proj, d.in.N), up(act, d.heads * d.vdim + 2 * d.groups * d.state), up(small, 2 * d.heads), up(mix, d.heads * d.vdim);
+            blk = std::max(blk, dc_ssd_block_floats(d));
         } else {
             const dc_latent_mixer& d = L.la;
             up(proj, d.in.N), up(mix, d.heads * d.vdim), up(rank, d.kv_rank), up(rot, d.rot_dim), up(ukv, d.ukv.N);
@@ -249,6 +251,7 @@ int dc_stack_finalize(dc_model* m) {
     DC_TRY(alloc(m, &b.low, C * low));
     DC_TRY(alloc(m, &b.gate, C * gate));
     DC_TRY(alloc(m, &b.small, C * small));
+    DC_TRY(alloc(m, &b.blk, (size_t)dc_scan_blocks((int)C, DC_MAX_T) * blk));
     DC_TRY(alloc(m, &b.mix, F * mix));
     DC_TRY(alloc(m, &b.ff, F * ff));
     DC_TRY(alloc(m, &b.lm_x, DC_MAX_T * H));
@@ -363,7 +366,7 @@ int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
         DC_TRY(linear(m, st, d.a2, b.proj + d.off_a, nullptr, ldp, DC_LIN_STORE, b.low, nullptr, d.a2.N));
         DC_TRY(linear(m, st, d.g2, b.proj + d.off_g, nullptr, ldp, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
     }
-    return dc_launch_delta_scan(m->ctx, d, st, sr, b.act, lda, b.small, b.low, d.a2.N, b.gate, d.g2.N, m->stack->cfg.eps, b.scan,
+    return dc_launch_delta_scan(m->ctx, d, st, sr, b.act, lda, b.small, b.low, d.a2.N, b.blk, b.gate, d.g2.N, m->stack->cfg.eps, b.scan,
                                 st.tc ? nullptr : b.mix, st.tc ? b.mixb : nullptr, dc_pad8(ldm));
 }
 
@@ -372,7 +375,7 @@ int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
     const dc_stack_buffers& b = m->stack->b;
     const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
     const int inner = d.heads * d.vdim, lda = dc_pad8(inner + 2 * d.groups * d.state);
-    return dc_launch_ssd(m->ctx, d, st, sr, b.proj, d.in.N, b.act, lda, b.small, b.scan, m->stack->cfg.eps, st.tc ? nullptr : b.mix,
+    return dc_launch_ssd(m->ctx, d, st, sr, b.proj, d.in.N, b.act, lda, b.small, b.blk, b.scan, m->stack->cfg.eps, st.tc ? nullptr : b.mix,
                          st.tc ? b.mixb : nullptr, dc_pad8(inner));
 }
 
@@ -419,7 +422,7 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
         const dc_lin& o = Ly.kind == DC_MIX_DELTA ? Ly.dl.o : Ly.kind == DC_MIX_SSD ? Ly.ssd.o : Ly.la.o;
         L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.x, xb, H, DC_LIN_STORE, b.proj, nullptr, in.N));
         if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, 7, mix_delta(m, st, Ly));
-        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, 4, mix_ssd(m, st, Ly));
+        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, 5, mix_ssd(m, st, Ly));
         else L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, Ly));
         L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), DC_LIN_STORE, b.y, nullptr, H));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));
