@@ -46,7 +46,7 @@ struct dc_delta_mixer {         // gated delta rule with one decay per key chann
     float unit_eps = 1e-6f, q_scale = 1.0f;
     dc_lin in, a2, g2, o;       // in: q | k | v | b | a1 | g1
     int off_q = 0, off_k = 0, off_v = 0, off_b = 0, off_a = 0, off_g = 0;
-    float *conv = nullptr;      // [C][taps], C = q, k and v channels
+    float *conv = nullptr;      // [taps][C], C = q, k and v projection columns
     float *neg_a = nullptr;     // [heads]: -exp(A_log)
     float *dt_bias = nullptr;   // [heads * dim]
     float *norm = nullptr;      // [vdim]
@@ -94,6 +94,7 @@ struct dc_stack_tensor {
     float** vec = nullptr;
     int64_t vec_off = 0, vec_len = 0;     // destination range and the vector's whole length
     bool neg_exp = false;       // stored as -exp(value)
+    int64_t cols = 0;           // a vector of shape [n, taps] stored transposed: element (c, j) at j * cols + vec_off + c
     bool loaded = false;
     int synth = 0;              // random-weight kind: 0 matrix, 1 norm weight, 2 decay exponent, 3 step bias, 4 small vector
 };
@@ -199,7 +200,7 @@ int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& 
                            float eps, float* mix, int ldm);
 int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* act,
                   int lda, float* small, float* blk, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
-int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y,
+int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y, int ldy,
                          float eps, float* mix, int ldm);
 int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps);
 

@@ -8,8 +8,8 @@
 // Value columns of S never mix: a column c obeys S_c <- g S_c; u = beta (v_c - S_c . k); S_c <- S_c + u k;
 // o_c = S_c . q.  A single token (decode) is done as written, by one kernel per mixer from projections to normed
 // output.  Longer entries go through blocks of sixteen tokens (see "blocks of sixteen tokens" below): what a head's
-// columns share is computed once per block, and k_state_scan walks the blocks with each column in the registers of
-// eight lanes.  All of it is f32 on the CUDA cores.
+// columns share is computed once per block, and k_state_scan walks the blocks with four columns in the registers of
+// each warp.  All of it is f32 on the CUDA cores.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -31,17 +31,24 @@ __device__ __forceinline__ int entry_of(const int32_t* starts, int E, int t) {
     return e;
 }
 
-// Convolution of one channel at token t (local index i in its entry, position pos): weights w[0 .. taps - 1], the last
-// for the token itself.
+// Convolution of one channel at token t (local index i in its entry, position pos): weights w[j * ldw], the last tap for
+// the token itself; inputs before the entry come from the ring, before position 0 they are zero.
 __device__ __forceinline__ float conv_at(const float* __restrict__ proj, int ldp, const float* __restrict__ ring, int C, int rc, int taps,
-                                         const float* __restrict__ w, int col, int t, int i, int pos) {
+                                         const float* __restrict__ w, int ldw, int col, int t, int i, int pos) {
     float s = 0.0f;
+    if (i >= taps - 1) {
+        const float* in = proj + (size_t)(t - taps + 1) * ldp + col;
+#pragma unroll 4
+        for (int j = 0; j < taps; ++j) s = fmaf(w[(size_t)j * ldw], in[(size_t)j * ldp], s);
+        return s;
+    }
+#pragma unroll 4
     for (int j = 0; j < taps; ++j) {
         const int back = taps - 1 - j;
         float in = 0.0f;
         if (back <= i) in = proj[(size_t)(t - back) * ldp + col];
         else if (pos >= back) in = ring[(size_t)((pos - back) % taps) * C + rc];
-        s = fmaf(w[j], in, s);
+        s = fmaf(w[(size_t)j * ldw], in, s);
     }
     return s;
 }
@@ -50,7 +57,7 @@ struct ConvRef {
     uint8_t* base;
     size_t slot_bytes, ring_off;
     const int32_t *seq_ids, *positions, *starts;
-    int E, taps, C;          // C: channels of a ring row
+    int E, taps, C, ldw;     // C: channels of a ring row; ldw: pitch of the convolution weights [taps][ldw]
     __device__ float* ring(int seq) const { return reinterpret_cast<float*>(base + (size_t)seq * slot_bytes + ring_off); }
 };
 
@@ -100,8 +107,8 @@ __global__ void __launch_bounds__(256) k_delta_prep(DeltaPrep p) {
             q[j] = k[j] = 0.0f;
             if (d < p.dim) {
                 const int cq = p.off_q + item * p.dim + d, ck = p.off_k + item * p.dim + d;
-                q[j] = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, cq, taps, p.conv + (size_t)cq * taps, cq, t, i, pos));
-                k[j] = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, ck, taps, p.conv + (size_t)ck * taps, ck, t, i, pos));
+                q[j] = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, cq, taps, p.conv + cq, p.cr.ldw, cq, t, i, pos));
+                k[j] = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, ck, taps, p.conv + ck, p.cr.ldw, ck, t, i, pos));
             }
             sq = fmaf(q[j], q[j], sq);
             sk = fmaf(k[j], k[j], sk);
@@ -124,7 +131,7 @@ __global__ void __launch_bounds__(256) k_delta_prep(DeltaPrep p) {
             const int c = c0 + lane + 32 * j;
             if (c < V) {
                 const int cv = p.off_v + c;
-                act[cv] = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, cv, taps, p.conv + (size_t)cv * taps, cv, t, i, pos));
+                act[cv] = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, cv, taps, p.conv + cv, p.cr.ldw, cv, t, i, pos));
             }
         }
     } else {
@@ -332,7 +339,7 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
 }
 
 // ---------------------------------------------------------------- the scan over blocks
-constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp, eight lanes each
+constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp
 
 struct ScanParams {
     const float* blocks;           // k_delta_blocks / k_ssd_blocks
@@ -374,14 +381,70 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
-__device__ __forceinline__ ulonglong2 lds_pairs(const float* p) { return *reinterpret_cast<const ulonglong2*>(p); }
 
-// EPL: key channels per lane (the key size, padded to 8 EPL).
+// EPL consecutive-chunk channels per lane: lane's channel i is W * lane + 32 W (i / W) + i % W.
+template <int EPL>
+struct Chan {
+    static constexpr int W = EPL < 4 ? EPL : 4;
+    static __device__ __forceinline__ int at(int lane, int i) { return W * lane + 32 * W * (i / W) + i % W; }
+    static __device__ __forceinline__ void load(const float* row, int lane, float (&f)[EPL]) {
+#pragma unroll
+        for (int j = 0; j < EPL / W; ++j) {
+            const float* r = row + W * lane + 32 * W * j;
+            if (W == 4) {
+                const float4 v = *reinterpret_cast<const float4*>(r);
+                f[4 * j] = v.x, f[(4 * j + 1) % EPL] = v.y, f[(4 * j + 2) % EPL] = v.z, f[(4 * j + 3) % EPL] = v.w;
+            } else if (W == 2) {
+                const float2 v = *reinterpret_cast<const float2*>(r);
+                f[2 * j] = v.x, f[(2 * j + 1) % EPL] = v.y;
+            } else {
+                f[j] = *r;
+            }
+        }
+    }
+};
+
+// Dot products of the warp's four columns (s: this lane's channels of each) with sixteen rows of shared memory.  Lane
+// 8 c + j gets column c's products with rows j and j + 8.
+template <int EPL>
+__device__ __forceinline__ void column_dots(const float* rows, int dp, const float (&s)[4][EPL], int lane, float (&out)[2]) {
+    float r[64];
+#pragma unroll
+    for (int t = 0; t < BT; ++t) {
+        float w[EPL];
+        Chan<EPL>::load(rows + t * dp, lane, w);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            if (EPL == 1) {
+                r[16 * c + 2 * (t & 7) + (t >> 3)] = s[c][0] * w[0];
+            } else {
+                uint64_t a = 0;
+#pragma unroll
+                for (int i = 0; i + 1 < EPL; i += 2) a = fma2(pair(s[c][i], s[c][i + 1]), pair(w[i], w[i + 1]), a);
+                const float2 f = unpair(a);
+                r[16 * c + 2 * (t & 7) + (t >> 3)] = f.x + f.y;
+            }
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {                           // each step halves the sums a lane carries
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+            if (i < 2 * o) {
+                const float send = up ? r[i] : r[i + 2 * o], keep = up ? r[i + 2 * o] : r[i];
+                r[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+    }
+    out[0] = r[0];
+    out[1] = r[1];
+}
+
+// EPL: key channels per lane (the key size, padded to 32 EPL).
 template <int EPL, bool DELTA>
 __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
-    constexpr int DP = 8 * EPL, NR = DELTA ? 2 * BT : BT, BLK = DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK, BUF = BLK + BT * SC_COLS;
+    constexpr int DP = 32 * EPL, BLK = DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK, BUF = BLK + BT * SC_COLS;
     extern __shared__ __align__(16) float sm[];
-    __shared__ float s_r[4][4][NR];                              // a warp's columns: S0 . G k (delta) and S0 . G q
     __shared__ __align__(16) float s_d[4][4][BT], s_u[4][4][BT];
     pdl_launch_dependents();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, c4 = lane >> 3;
@@ -397,17 +460,16 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     const int seq = p.seq_ids[t0], blocks = (t1 - t0 + BT - 1) / BT;
     const float* bsrc = p.blocks + ((size_t)block_base(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
     const size_t bstep = (size_t)p.heads * (DELTA ? BLK : SSD_BLOCK);
-    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + col) * p.dim;
-    float sf[EPL];
+    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 4) * p.dim;
+    float s[4][EPL];             // channels Chan::at of the warp's four columns
     const bool fresh = p.positions[t0] == 0, live = col < p.vdim;
 #pragma unroll
-    for (int j = 0; j < EPL; ++j) {
-        const int d = 4 * (l8 + 8 * (j >> 2)) + (j & 3);
-        sf[j] = !fresh && live && d < p.dim ? S[d] : 0.0f;
-    }
-    uint64_t s[EPL / 2];
+    for (int c = 0; c < 4; ++c)
 #pragma unroll
-    for (int j = 0; j < EPL / 2; ++j) s[j] = pair(sf[2 * j], sf[2 * j + 1]);
+        for (int i = 0; i < EPL; ++i) {
+            const int d = Chan<EPL>::at(lane, i);
+            s[c][i] = !fresh && c0 + warp * 4 + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
+        }
 
     auto load = [&](int b, int buf) {
         float* dst = sm + buf * BUF;
@@ -449,39 +511,10 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         __syncthreads();
         const float* x = sm + (b & 1) * BUF;
         const float* sv = x + BLK + warp * 4 + c4;
-        // ---- the column against the block's (decayed) keys and queries
-        uint64_t acc[NR];
-#pragma unroll
-        for (int i = 0; i < NR; ++i) acc[i] = 0;
-#pragma unroll
-        for (int j = 0; j < EPL / 4; ++j) {
-#pragma unroll
-            for (int i = 0; i < NR; ++i) {
-                const ulonglong2 w = lds_pairs(x + i * DP + 4 * (l8 + 8 * j));
-                acc[i] = fma2(s[2 * j], w.x, acc[i]);
-                acc[i] = fma2(s[2 * j + 1], w.y, acc[i]);
-            }
-        }
-        float r[NR];
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const float2 f = unpair(acc[i]);
-            r[i] = f.x + f.y;
-        }
-#pragma unroll
-        for (int o = 4; o > 0; o >>= 1) {                        // sums over the eight lanes: lane l8 keeps NR / 8 of them
-            const bool up = l8 & o;
-            const int half = NR / 8 * o;
-#pragma unroll
-            for (int i = 0; i < NR / 2; ++i)
-                if (i < half) {
-                    const float send = up ? r[i] : r[i + half], keep = up ? r[i + half] : r[i];
-                    r[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                }
-        }
-#pragma unroll
-        for (int i = 0; i < NR / 8; ++i) s_r[warp][c4][l8 * (NR / 8) + i] = r[i];
-        __syncwarp();
+        // ---- the columns against the block's (decayed) keys and queries
+        float rk[2] = {}, rq[2];
+        if (DELTA) column_dots<EPL>(x, DP, s, lane, rk);
+        column_dots<EPL>(x + (DELTA ? BT * DP : 0), DP, s, lane, rq);
         // ---- u and o: this lane's tokens l8 and l8 + 8
         const float* scal = x + (DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
         float v[2];
@@ -489,7 +522,7 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         for (int k = 0; k < 2; ++k) {
             const int t = l8 + 8 * k;
             v[k] = sv[t * SC_COLS];
-            s_d[warp][c4][t] = DELTA ? v[k] - s_r[warp][c4][t] : v[k];
+            s_d[warp][c4][t] = v[k] - rk[k];
         }
         __syncwarp();
         float dv[BT];
@@ -521,16 +554,16 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
                 dv[4 * i] = f.x, dv[4 * i + 1] = f.y, dv[4 * i + 2] = f.z, dv[4 * i + 3] = f.w;
             }
 #pragma unroll
-            for (int k = 0; k < 2; ++k) out[k] = s_r[warp][c4][BT + l8 + 8 * k] + row_dot(scal + (BT + l8 + 8 * k) * BROW);
+            for (int k = 0; k < 2; ++k) out[k] = rq[k] + row_dot(scal + (BT + l8 + 8 * k) * BROW);
         } else {
             const float* cd = scal + BT * BROW;
 #pragma unroll
             for (int k = 0; k < 2; ++k) {
                 const int t = l8 + 8 * k;
-                out[k] = fmaf(cd[t], s_r[warp][c4][t], row_dot(scal + t * BROW)) + Dh * v[k];
+                out[k] = fmaf(cd[t], rq[k], row_dot(scal + t * BROW)) + Dh * v[k];
+                s_u[warp][c4][t] = v[k] * cd[BT + t];
             }
-#pragma unroll
-            for (int i = 0; i < BT; ++i) dv[i] *= cd[BT + i];
+            __syncwarp();
         }
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
@@ -539,36 +572,39 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
         // ---- the state after the block
         const float* keys = x + (DELTA ? 2 * BT * DP : BT * DP);
+        {
+            float g[EPL];
+            if (DELTA) Chan<EPL>::load(x + 3 * BT * DP, lane, g);
 #pragma unroll
-        for (int j = 0; j < EPL / 4; ++j) {
-            uint64_t a0 = 0, a1 = 0;
+            for (int c = 0; c < 4; ++c)
 #pragma unroll
-            for (int t = 0; t < BT; ++t) {
-                const ulonglong2 w = lds_pairs(keys + t * DP + 4 * (l8 + 8 * j));
-                const uint64_t u = pair(dv[t], dv[t]);
-                a0 = fma2(w.x, u, a0);
-                a1 = fma2(w.y, u, a1);
+                for (int i = 0; i < EPL; ++i) s[c][i] *= DELTA ? g[i] : scal[BT * BROW + BT - 1];
+        }
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+            float w[EPL];
+            Chan<EPL>::load(keys + t * DP, lane, w);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const float u = s_u[warp][c][t];
+#pragma unroll
+                for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(w[i], u, s[c][i]);
             }
-            ulonglong2 g;
-            if (DELTA) g = lds_pairs(x + 3 * BT * DP + 4 * (l8 + 8 * j));
-            else g.x = g.y = pair(scal[BT * BROW + BT - 1], scal[BT * BROW + BT - 1]);
-            s[2 * j] = fma2(s[2 * j], g.x, a0);
-            s[2 * j + 1] = fma2(s[2 * j + 1], g.y, a1);
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int j = 0; j < EPL / 2; ++j) {
-        const float2 f = unpair(s[j]);
-        const int d = 4 * (l8 + 8 * (j >> 1)) + 2 * (j & 1);
-        if (live && d < p.dim) S[d] = f.x;
-        if (live && d + 1 < p.dim) S[d + 1] = f.y;
-    }
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int i = 0; i < EPL; ++i) {
+            const int d = Chan<EPL>::at(lane, i);
+            if (c0 + warp * 4 + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
+        }
 }
 
 template <int EPL, bool DELTA>
 int launch_scan_epl(dc_ctx* ctx, const ScanParams& p, int E) {
-    constexpr int DP = 8 * EPL;
+    constexpr int DP = 32 * EPL;
     const size_t smem = (size_t)2 * ((DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK) + BT * SC_COLS) * 4;
     DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, DELTA>, (int)smem, "k_state_scan"));
     return dc_launch(ctx, "k_state_scan", k_state_scan<EPL, DELTA>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_THREADS), smem, p);
@@ -577,10 +613,215 @@ int key_pad(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128
 template <bool DELTA>
 int launch_scan(dc_ctx* ctx, const ScanParams& p, int E) {
     switch (key_pad(p.dim)) {
-    case 32: return launch_scan_epl<4, DELTA>(ctx, p, E);
-    case 64: return launch_scan_epl<8, DELTA>(ctx, p, E);
-    case 128: return launch_scan_epl<16, DELTA>(ctx, p, E);
-    default: return launch_scan_epl<32, DELTA>(ctx, p, E);
+    case 32: return launch_scan_epl<1, DELTA>(ctx, p, E);
+    case 64: return launch_scan_epl<2, DELTA>(ctx, p, E);
+    case 128: return launch_scan_epl<4, DELTA>(ctx, p, E);
+    default: return launch_scan_epl<8, DELTA>(ctx, p, E);
+    }
+}
+
+// ---------------------------------------------------------------- decode: one token per sequence
+struct DeltaDecode {
+    ConvRef cr;
+    const float* proj;
+    int ldp;
+    const float* conv;
+    int heads, per, dim, vdim, off_q, off_k, off_v, off_b, off_a, off_g, a_rank, g_rank;
+    float unit_eps, q_scale, eps;
+    const __nv_bfloat16 *a2, *g2;
+    int lda2, ldg2;
+    const float *neg_a, *dt_bias, *norm;
+    size_t state_off;
+    float* mix;
+    int ldm;
+};
+
+// rows r0 .. of a bf16 matrix (padded with zeros to whole sixteens of eight) times x in shared memory; sixteen lanes a row
+__device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ldw, int n, const float* x, int rank, float* out) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 15;
+#pragma unroll 4
+    for (int r = 2 * warp + (lane >> 4); r < ((n + 1) & ~1); r += 2 * (blockDim.x >> 5)) {
+        float a = 0.0f;
+        if (r < n)
+            for (int k = 8 * sub; k < rank; k += 128) {
+                const uint4 v = *reinterpret_cast<const uint4*>(w + (size_t)r * ldw + k);
+                const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    a = fmaf(__uint_as_float(u[i] << 16), x[k + 2 * i], a);
+                    a = fmaf(__uint_as_float(u[i] & 0xffff0000u), x[k + 2 * i + 1], a);
+                }
+            }
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+        if (sub == 0 && r < n) out[r] = a;
+    }
+}
+
+// One CTA per (head, sequence): convolutions, unit vectors, decays and gates, the state's step, the gated norm.
+template <int EPL>
+__global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
+    constexpr int DP = 32 * EPL;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[33], s_iq, s_ik;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, t = blockIdx.y, kh = h / p.per;
+    const int ra = (p.a_rank + 7) & ~7, rg = (p.g_rank + 7) & ~7;
+    float *sq = sm, *sk = sq + DP, *sg = sk + DP, *sa = sg + DP, *sgl = sa + ra, *sv = sgl + rg, *so = sv + p.vdim, *sgate = so + p.vdim;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int pos = p.cr.positions[t], seq = p.cr.seq_ids[t], taps = p.cr.taps;
+    float* ring = p.cr.ring(seq);
+    const float* row = p.proj + (size_t)t * p.ldp;
+    const bool first = h % p.per == 0;
+    for (int c = tid; c < 2 * DP + p.vdim; c += 256) {
+        const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
+        const int col = c < DP ? p.off_q + kh * p.dim + d : c < 2 * DP ? p.off_k + kh * p.dim + d : p.off_v + h * p.vdim + d;
+        float v = 0.0f;
+        if (c >= 2 * DP || d < p.dim) {
+            v = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, col, taps, p.conv + col, p.cr.ldw, col, t, 0, pos));
+            if (c >= 2 * DP || first) ring[(size_t)(pos % taps) * p.cr.C + col] = row[col];    // a row no tap of this token reads
+        }
+        sm[c < 2 * DP ? c : (int)(sv - sm) + d] = v;
+    }
+    for (int c = tid; c < ra; c += 256) sa[c] = c < p.a_rank ? row[p.off_a + c] : 0.0f;
+    for (int c = tid; c < rg; c += 256) sgl[c] = c < p.g_rank ? row[p.off_g + c] : 0.0f;
+    __syncthreads();
+    if (warp < 2) {
+        float ss = 0.0f;
+        for (int d = lane; d < DP; d += 32) ss = fmaf(sm[warp * DP + d], sm[warp * DP + d], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) (warp ? s_ik : s_iq) = (warp ? 1.0f : p.q_scale) / sqrtf(ss + p.unit_eps);
+    }
+    low_rank_rows(p.a2 + (size_t)h * p.dim * p.lda2, p.lda2, p.dim, sa, ra, sg);
+    low_rank_rows(p.g2 + (size_t)h * p.vdim * p.ldg2, p.ldg2, p.vdim, sgl, rg, sgate);
+    __syncthreads();
+    for (int d = tid; d < DP; d += 256) {
+        sg[d] = d < p.dim ? expf(p.neg_a[h] * softplus(sg[d] + p.dt_bias[(size_t)h * p.dim + d])) : 0.0f;
+        sq[d] *= s_iq;
+        sk[d] *= s_ik;
+    }
+    __syncthreads();
+    float kr[EPL], qr[EPL], gr[EPL], kq = 0.0f;
+    Chan<EPL>::load(sk, lane, kr);
+    Chan<EPL>::load(sq, lane, qr);
+    Chan<EPL>::load(sg, lane, gr);
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) kq = fmaf(kr[i], qr[i], kq);
+    kq = warp_sum(kq);
+    const float beta = sigmoid(row[p.off_b + h]);
+    float* S = reinterpret_cast<float*>(p.cr.base + (size_t)seq * p.cr.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.dim;
+#pragma unroll 2
+    for (int c0 = 4 * warp; c0 < p.vdim; c0 += 32) {
+        float s[4][EPL], a[4], b[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            a[c] = b[c] = 0.0f;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const int d = Chan<EPL>::at(lane, i);
+                s[c][i] = pos > 0 && c0 + c < p.vdim && d < p.dim ? S[(size_t)(c0 + c) * p.dim + d] * gr[i] : 0.0f;
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                a[c] = fmaf(s[c][i], kr[i], a[c]);
+                b[c] = fmaf(s[c][i], qr[i], b[c]);
+            }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            a[c] = warp_sum(a[c]);
+            b[c] = warp_sum(b[c]);
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            if (c0 + c >= p.vdim) continue;
+            const float u = beta * (sv[c0 + c] - a[c]);
+            if (lane == 0) so[c0 + c] = fmaf(kq, u, b[c]);
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const int d = Chan<EPL>::at(lane, i);
+                if (d < p.dim) S[(size_t)(c0 + c) * p.dim + d] = fmaf(kr[i], u, s[c][i]);
+            }
+        }
+    }
+    __syncthreads();
+    float ss = 0.0f;
+    for (int c = tid; c < p.vdim; c += 256) ss = fmaf(so[c], so[c], ss);
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.vdim + p.eps);
+    for (int c = tid; c < p.vdim; c += 256) p.mix[(size_t)t * p.ldm + (size_t)h * p.vdim + c] = so[c] * inv * p.norm[c] * sigmoid(sgate[c]);
+}
+
+struct SsdDecode {
+    ConvRef cr;
+    const float* proj;
+    int ldp;
+    const float *conv, *conv_b, *dt_bias, *neg_a, *D;
+    int heads, per, groups, state, vdim, off_x, off_dt, off_z;
+    size_t state_off;
+    float* y;                    // gated: y silu(z)
+    int ldy;
+};
+
+// One CTA per (head, sequence): convolutions, the state's step, the gate (the group norm spans heads).
+template <int EPL>
+__global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
+    constexpr int DP = 32 * EPL;
+    extern __shared__ __align__(16) float sm[];     // B, C: [DP]; x: [vdim]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, t = blockIdx.y, g = h / p.per;
+    float* sx = sm + 2 * DP;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int pos = p.cr.positions[t], seq = p.cr.seq_ids[t], taps = p.cr.taps, inner = p.heads * p.vdim, GN = p.groups * p.state;
+    float* ring = p.cr.ring(seq);
+    const float* row = p.proj + (size_t)t * p.ldp;
+    const bool first = h % p.per == 0;
+    for (int c = tid; c < 2 * DP + p.vdim; c += 128) {
+        const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
+        const int ch = c < DP ? inner + g * p.state + d : c < 2 * DP ? inner + GN + g * p.state + d : h * p.vdim + d;
+        float v = 0.0f;
+        if (c >= 2 * DP || d < p.state) {
+            v = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, ch, taps, p.conv + ch, p.cr.ldw, p.off_x + ch, t, 0, pos) + p.conv_b[ch]);
+            if (c >= 2 * DP || first) ring[(size_t)(pos % taps) * p.cr.C + ch] = row[p.off_x + ch];
+        }
+        sm[c] = v;
+    }
+    const float dt = softplus(row[p.off_dt + h] + p.dt_bias[h]), decay = expf(p.neg_a[h] * dt), Dh = p.D[h];
+    __syncthreads();
+    float br[EPL], cr[EPL];
+    Chan<EPL>::load(sm, lane, br);
+    Chan<EPL>::load(sm + DP, lane, cr);
+    float* S = reinterpret_cast<float*>(p.cr.base + (size_t)seq * p.cr.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.state;
+#pragma unroll 2
+    for (int c0 = 4 * warp; c0 < p.vdim; c0 += 16) {
+        float s[4][EPL], a[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const int d = Chan<EPL>::at(lane, i);
+                s[c][i] = pos > 0 && c0 + c < p.vdim && d < p.state ? S[(size_t)(c0 + c) * p.state + d] : 0.0f;
+            }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const float u = c0 + c < p.vdim ? dt * sx[c0 + c] : 0.0f;
+            a[c] = 0.0f;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                s[c][i] = fmaf(s[c][i], decay, br[i] * u);
+                a[c] = fmaf(s[c][i], cr[i], a[c]);
+                const int d = Chan<EPL>::at(lane, i);
+                if (c0 + c < p.vdim && d < p.state) S[(size_t)(c0 + c) * p.state + d] = s[c][i];
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) a[c] = warp_sum(a[c]);
+        if (lane < 4 && c0 + lane < p.vdim) {
+            const int c = c0 + lane;
+            const float av = lane == 0 ? a[0] : lane == 1 ? a[1] : lane == 2 ? a[2] : a[3];
+            p.y[(size_t)t * p.ldy + (size_t)h * p.vdim + c] = fmaf(Dh, sx[c], av) * silu(row[p.off_z + (size_t)h * p.vdim + c]);
+        }
     }
 }
 
@@ -614,16 +855,26 @@ __global__ void __launch_bounds__(256) k_gate_group_norm(const float* __restrict
     const int t = blockIdx.y, c0 = blockIdx.x * n;
     const float* yr = y + (size_t)t * ldy + c0;
     const float* zr = z ? z + (size_t)t * ldz + c0 : nullptr;
-    float ss = 0.0f;
-    for (int i = threadIdx.x; i < n; i += 256) {
-        const float v = zr ? yr[i] * silu(zr[i]) : yr[i];
-        ss = fmaf(v, v, ss);
+    constexpr int KEEP = 8;      // values per thread kept between the two passes
+    float v[KEEP], ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        v[j] = i < n ? (zr ? yr[i] * silu(zr[i]) : yr[i]) : 0.0f;
+        ss = fmaf(v[j], v[j], ss);
+    }
+    for (int i = threadIdx.x + 256 * KEEP; i < n; i += 256) {
+        const float x = zr ? yr[i] * silu(zr[i]) : yr[i];
+        ss = fmaf(x, x, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
-    for (int i = threadIdx.x; i < n; i += 256) {
-        const float v = zr ? yr[i] * silu(zr[i]) : yr[i];
-        store_as(out + (size_t)t * ldm + c0 + i, v * inv * w[c0 + i]);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        if (i < n) store_as(out + (size_t)t * ldm + c0 + i, v[j] * inv * w[c0 + i]);
     }
+    for (int i = threadIdx.x + 256 * KEEP; i < n; i += 256)
+        store_as(out + (size_t)t * ldm + c0 + i, (zr ? yr[i] * silu(zr[i]) : yr[i]) * inv * w[c0 + i]);
 }
 
 // ---------------------------------------------------------------- ssd: per-token inputs
@@ -642,7 +893,7 @@ __global__ void __launch_bounds__(256) k_ssd_prep(SsdPrep p) {
     const int t = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
     const int e = entry_of(p.cr.starts, p.cr.E, t), i = t - p.cr.starts[e], pos = p.cr.positions[t];
     if (c < p.cr.C)
-        p.act[(size_t)t * p.lda + c] = silu(conv_at(p.proj, p.ldp, p.cr.ring(p.cr.seq_ids[t]), p.cr.C, c, p.cr.taps, p.conv + (size_t)c * p.cr.taps,
+        p.act[(size_t)t * p.lda + c] = silu(conv_at(p.proj, p.ldp, p.cr.ring(p.cr.seq_ids[t]), p.cr.C, c, p.cr.taps, p.conv + c, p.cr.ldw,
                                                     p.off_x + c, t, i, pos) + p.conv_b[c]);
     if (blockIdx.x == 0)
         for (int h = threadIdx.x; h < p.heads; h += 256) {
@@ -653,7 +904,7 @@ __global__ void __launch_bounds__(256) k_ssd_prep(SsdPrep p) {
 }
 
 ConvRef conv_ref(const dc_step& st, const dc_state_ref& sr, int taps, int C) {
-    return ConvRef{sr.base, sr.slot_bytes, sr.ring_off, st.seq_ids, st.positions, st.starts, st.E, taps, C};
+    return ConvRef{sr.base, sr.slot_bytes, sr.ring_off, st.seq_ids, st.positions, st.starts, st.E, taps, C, C};
 }
 
 }  // namespace
@@ -671,6 +922,7 @@ int dc_launch_delta_prep(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st
     DeltaPrep p;
     const int V = m.heads * m.vdim, C = m.off_v + V;
     p.cr = conv_ref(st, sr, m.taps, C);
+    p.cr.ldw = m.off_v + dc_pad8(V);
     p.proj = proj, p.ldp = ldp, p.conv = m.conv;
     p.heads = m.heads, p.kv_heads = m.kv_heads, p.dim = m.dim, p.vdim = m.vdim;
     p.off_q = m.off_q, p.off_k = m.off_k, p.off_v = m.off_v, p.off_b = m.off_b, p.off_a = m.off_a;
@@ -727,4 +979,37 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
                          m.norm, n, eps, mixb, ldm);
     return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<float>, dim3(m.norm_groups, st.T), dim3(256), 0, y, lda, proj + m.off_z, ldp, m.norm, n,
                      eps, mix, ldm);
+}
+
+int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
+                           float* mix, int ldm) {
+    const int V = m.heads * m.vdim;
+    DeltaDecode p = {conv_ref(st, sr, m.taps, m.off_v + V), proj, ldp, m.conv, m.heads, m.heads / m.kv_heads, m.dim, m.vdim, m.off_q, m.off_k, m.off_v, m.off_b,
+                     m.off_a, m.off_g, m.a_rank, m.g_rank, m.unit_eps, m.q_scale, eps, m.a2.w, m.g2.w, m.a2.ld, m.g2.ld, m.neg_a, m.dt_bias, m.norm,
+                     sr.state_off, mix, ldm};
+    p.cr.ldw = m.off_v + dc_pad8(V);
+    const int dp = key_pad(m.dim);
+    const size_t smem = (size_t)(3 * dp + dc_pad8(m.a_rank) + dc_pad8(m.g_rank) + 3 * m.vdim) * 4;
+    const dim3 grid(m.heads, st.T), block(256);
+    if (smem > 48 * 1024) return dc_fail(ctx, DC_B200_UNSUPPORTED, "delta rule: gate ranks %d and %d are too large", m.a_rank, m.g_rank);
+    if (dp == 32) return dc_launch(ctx, "k_delta_decode", k_delta_decode<1>, grid, block, smem, p);
+    if (dp == 64) return dc_launch(ctx, "k_delta_decode", k_delta_decode<2>, grid, block, smem, p);
+    if (dp == 128) return dc_launch(ctx, "k_delta_decode", k_delta_decode<4>, grid, block, smem, p);
+    return dc_launch(ctx, "k_delta_decode", k_delta_decode<8>, grid, block, smem, p);
+}
+
+int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y, int ldy,
+                         float eps, float* mix, int ldm) {
+    const int inner = m.heads * m.vdim, C = inner + 2 * m.groups * m.state;
+    SsdDecode p = {conv_ref(st, sr, m.taps, C), proj, ldp, m.conv, m.conv_b, m.dt_bias, m.neg_a, m.D, m.heads, m.heads / m.groups, m.groups, m.state, m.vdim,
+                   m.off_x, m.off_dt, m.off_z, sr.state_off, y, ldy};
+    const int dp = key_pad(m.state);
+    const size_t smem = (size_t)(2 * dp + m.vdim) * 4;
+    const dim3 grid(m.heads, st.T), block(128);
+    if (dp == 32) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<1>, grid, block, smem, p));
+    else if (dp == 64) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<2>, grid, block, smem, p));
+    else if (dp == 128) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<4>, grid, block, smem, p));
+    else DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<8>, grid, block, smem, p));
+    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<float>, dim3(m.norm_groups, st.T), dim3(256), 0, y, ldy, nullptr, 0, m.norm,
+                     inner / m.norm_groups, eps, mix, ldm);
 }

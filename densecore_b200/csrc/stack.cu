@@ -50,6 +50,16 @@ __global__ void k_place_rows(const float* __restrict__ src, int64_t n, int K, __
     }
 }
 
+// Values in the tensor's own order to their places in the device vector.
+cudaError_t put_vector(const dc_stack_tensor& t, const std::vector<float>& v) {
+    if (!t.cols) return cudaMemcpy(*t.vec + t.vec_off, v.data(), v.size() * 4, cudaMemcpyHostToDevice);
+    const size_t taps = (size_t)t.shape[1], n = v.size() / taps;
+    std::vector<float> w(v.size());
+    for (size_t c = 0; c < n; ++c)
+        for (size_t j = 0; j < taps; ++j) w[j * n + c] = v[c * taps + j];
+    return cudaMemcpy2D(*t.vec + t.vec_off, (size_t)t.cols * 4, w.data(), n * 4, n * 4, taps, cudaMemcpyHostToDevice);
+}
+
 template <typename T>
 int alloc(dc_model* m, T** p, size_t n, const char* what = "step buffer") {
     DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)p, n * sizeof(T) + 256), what));
@@ -82,7 +92,7 @@ int dc_stack_set_tensor(dc_model* m, const char* name, int type, const int64_t n
             v[i] = type == DC_TYPE_F32 ? ((const float*)data)[i] : bf16_value(((const uint16_t*)data)[i]);
             if (t.neg_exp) v[i] = (float)-exp((double)v[i]);
         }
-        e = cudaMemcpy(*t.vec + t.vec_off, v.data(), (size_t)n * 4, cudaMemcpyHostToDevice);
+        e = put_vector(t, v);
     } else if (!t.lin) {
         e = cudaMemcpy(s->embed->dev, data, s->embed->bytes, cudaMemcpyHostToDevice);
     } else {
@@ -111,16 +121,16 @@ int dc_stack_init_synthetic(dc_model* m, uint64_t seed, float sigma) {
         const int64_t n = elems(t);
         // norm weights around 1, decay exponents and step biases in a useful range, convolution taps not tiny
         const float sg = t.synth == 4 ? 0.4f : t.synth == 2 ? 0.5f : sigma, off = t.synth == 1 ? 1.0f : t.synth == 3 ? -2.0f : 0.0f;
-        float* dst = t.vec ? *t.vec + t.vec_off : tmp;
-        st = dc_launch_synth_f32(ctx, seed + fnv1a64(t.name.c_str()), n, sg, off, dst);
+        st = dc_launch_synth_f32(ctx, seed + fnv1a64(t.name.c_str()), n, sg, off, tmp);
         if (st != DC_B200_OK) break;
-        if (t.vec && t.neg_exp) {
+        if (t.vec) {
             std::vector<float> v((size_t)n);
             cudaStreamSynchronize(ctx->stream);
-            cudaMemcpy(v.data(), dst, (size_t)n * 4, cudaMemcpyDeviceToHost);
-            for (float& x : v) x = (float)-exp((double)x);
-            st = dc_check_cuda(ctx, cudaMemcpy(dst, v.data(), (size_t)n * 4, cudaMemcpyHostToDevice), "init_synthetic");
-        } else if (!t.vec) {
+            cudaMemcpy(v.data(), tmp, (size_t)n * 4, cudaMemcpyDeviceToHost);
+            if (t.neg_exp)
+                for (float& x : v) x = (float)-exp((double)x);
+            st = dc_check_cuda(ctx, put_vector(t, v), "init_synthetic");
+        } else {
             const int K = (int)t.shape[1];
             __nv_bfloat16* w = t.lin ? t.lin->w : (__nv_bfloat16*)s->embed->dev;
             k_place_rows<<<1184, 256, 0, ctx->stream>>>(tmp, n, K, w, t.lin ? t.lin->ld : K, t.row0, t.row_step, t.head_rows, t.head_pad);
@@ -357,6 +367,8 @@ int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
     const dc_stack_buffers& b = m->stack->b;
     const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
     const int ldp = d.in.N, lda = dc_pad8(d.off_v + d.heads * d.vdim), ldl = d.in.N - d.off_a, ldm = d.heads * d.vdim;
+    if (st.single && !st.tc && st.T <= DC_MAX_T)
+        return dc_launch_delta_decode(m->ctx, d, st, sr, b.proj, ldp, m->stack->cfg.eps, b.mix, dc_pad8(ldm));
     __nv_bfloat16* lowb = st.tc ? b.lowb : nullptr;
     DC_TRY(dc_launch_delta_prep(m->ctx, d, st, sr, b.proj, ldp, b.act, lda, b.small, lowb, ldl));
     if (st.tc) {
@@ -375,6 +387,8 @@ int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
     const dc_stack_buffers& b = m->stack->b;
     const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
     const int inner = d.heads * d.vdim, lda = dc_pad8(inner + 2 * d.groups * d.state);
+    if (st.single && !st.tc && st.T <= DC_MAX_T)
+        return dc_launch_ssd_decode(m->ctx, d, st, sr, b.proj, d.in.N, b.scan, lda, m->stack->cfg.eps, b.mix, dc_pad8(inner));
     return dc_launch_ssd(m->ctx, d, st, sr, b.proj, d.in.N, b.act, lda, b.small, b.blk, b.scan, m->stack->cfg.eps, st.tc ? nullptr : b.mix,
                          st.tc ? b.mixb : nullptr, dc_pad8(inner));
 }
@@ -421,8 +435,8 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
         const dc_lin& in = Ly.kind == DC_MIX_DELTA ? Ly.dl.in : Ly.kind == DC_MIX_SSD ? Ly.ssd.in : Ly.la.in;
         const dc_lin& o = Ly.kind == DC_MIX_DELTA ? Ly.dl.o : Ly.kind == DC_MIX_SSD ? Ly.ssd.o : Ly.la.o;
         L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.x, xb, H, DC_LIN_STORE, b.proj, nullptr, in.N));
-        if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, 7, mix_delta(m, st, Ly));
-        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, 5, mix_ssd(m, st, Ly));
+        if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, st.single && !st.tc ? 1 : 7, mix_delta(m, st, Ly));
+        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, st.single && !st.tc ? 2 : 5, mix_ssd(m, st, Ly));
         else L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, Ly));
         L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), DC_LIN_STORE, b.y, nullptr, H));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));

@@ -80,6 +80,11 @@ struct Reader {
         t.synth = synth;
         tensor(t);
     }
+    // convolution weights [n, taps], kept as [taps][cols]
+    void conv(float** p, const std::string& name, int n, int taps, int off, int cols) {
+        vec(p, name, {n, taps}, 4, off, (int64_t)cols * taps);
+        s->tensors.back().cols = cols;
+    }
 };
 
 // ---------------------------------------------------------------- mixers
@@ -107,10 +112,10 @@ void read_delta(Reader& r, const dc_json& j, const std::string& p, const std::st
     r.matrix(&d.g2, p + "g2", V, d.g_rank);
     r.matrix(&d.o, p + "o", H, V);
     // convolution weights sit at the channels' projection columns, so that one index serves both
-    const int64_t C = (int64_t)(d.off_v + dc_pad8(V)) * d.taps;
-    r.vec(&d.conv, p + "q.conv", {Q, d.taps}, 4, (int64_t)d.off_q * d.taps, C);
-    r.vec(&d.conv, p + "k.conv", {Q, d.taps}, 4, (int64_t)d.off_k * d.taps, C);
-    r.vec(&d.conv, p + "v.conv", {V, d.taps}, 4, (int64_t)d.off_v * d.taps, C);
+    const int C = d.off_v + dc_pad8(V);
+    r.conv(&d.conv, p + "q.conv", Q, d.taps, d.off_q, C);
+    r.conv(&d.conv, p + "k.conv", Q, d.taps, d.off_k, C);
+    r.conv(&d.conv, p + "v.conv", V, d.taps, d.off_v, C);
     r.vec(&d.neg_a, p + "A_log", {d.heads}, 2, 0, 0, true);
     r.vec(&d.dt_bias, p + "dt_bias", {(int64_t)d.heads * d.dim}, 3);
     r.vec(&d.norm, p + "norm", {d.vdim}, 1);
@@ -134,7 +139,7 @@ void read_ssd(Reader& r, const dc_json& j, const std::string& p, const std::stri
     d.off_x = inner;
     d.off_dt = inner + C;
     r.matrix(&d.o, p + "o", H, inner);
-    r.vec(&d.conv, p + "conv", {C, d.taps}, 4);
+    r.conv(&d.conv, p + "conv", C, d.taps, 0, C);
     r.vec(&d.conv_b, p + "conv.b", {C}, 4);
     r.vec(&d.dt_bias, p + "dt_bias", {d.heads}, 3);
     r.vec(&d.neg_a, p + "A_log", {d.heads}, 2, 0, 0, true);
