@@ -35,9 +35,27 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     __syncthreads();
     return red[32];
 }
+// a pair of f32 values in one register pair, two multiply-adds per instruction
+__device__ __forceinline__ uint64_t pair(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(uint64_t v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
 __device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 __device__ __forceinline__ float load_as(const float* p) { return *p; }
 __device__ __forceinline__ float load_as(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+// asks for a 128-byte line of global memory to be brought into L2
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 }  // namespace dc

@@ -3,9 +3,8 @@
 // a line in the architecture table (stack_config.cu) and not a forward pass of its own.
 //
 // Numbers: weights are bf16 in HBM; the residual, norms, decays, gates, recurrent state and attention scores are
-// f32.  Steps of up to DC_MAX_T tokens, and every step of an f32 model, keep activations in f32 all the way
-// (row-streaming products); larger steps of a bf16 model round the inputs of matrix products to bf16 and run
-// them on the tensor cores.
+// f32.  A bf16 model rounds the inputs of matrix products to bf16 (accumulation is f32), an f32 model keeps every
+// activation in f32.
 #pragma once
 #include <cuda.h>
 #include <cuda_bf16.h>
@@ -110,7 +109,8 @@ struct dc_stack_config {
 struct dc_step {
     int T = 0, E = 0;
     const int32_t *tokens = nullptr, *seq_ids = nullptr, *positions = nullptr, *starts = nullptr;
-    bool tc = false;            // matrix products on the tensor cores (bf16 inputs)
+    bool b16 = false;           // inputs of matrix products in bf16
+    bool tc = false;            // ... and more than DC_MAX_T tokens: tiled products, prompt attention
     bool single = false;        // every entry is one token
 };
 
@@ -122,8 +122,8 @@ struct dc_stack_buffers {
     int meta_ints = 0, meta_slot = 0;
     int32_t *iota = nullptr, *chunk = nullptr;   // constant entry starts: one token each; one entry of n tokens at chunk + 2 n
     float *x = nullptr, *y = nullptr, *proj = nullptr, *act = nullptr, *scan = nullptr, *low = nullptr, *gate = nullptr, *small = nullptr, *blk = nullptr;
-    float *mix = nullptr, *ff = nullptr, *lm_x = nullptr;
-    __nv_bfloat16 *xb = nullptr, *mixb = nullptr, *ffb = nullptr, *lowb = nullptr;
+    float *mix = nullptr, *ff = nullptr, *lm_x = nullptr;   // mix, ff, lm_x: f32 models
+    __nv_bfloat16 *lm_xb = nullptr, *xb = nullptr, *mixb = nullptr, *ffb = nullptr, *lowb = nullptr;
     __nv_bfloat16 *keys_c = nullptr, *keys_r = nullptr, *keys_kv = nullptr;
     float *qa = nullptr, *part = nullptr, *part_ml = nullptr;
     std::vector<void*> owned;
@@ -166,7 +166,9 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
 void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token);
 
 // ---- linear.cu / linear_tc.cu: y = W x
-// T <= DC_MAX_T tokens, f32 inputs: one pass over the weights.  keys: packed greedy picks per token.
+// T <= DC_MAX_T tokens, bf16 or f32 inputs: one pass over the weights.  keys: packed greedy picks per token.
+int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, int epi, float* out, __nv_bfloat16* outb, int ldo,
+                         unsigned long long* keys = nullptr);
 int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo,
                           unsigned long long* keys = nullptr);
 // any T, f32 inputs (f32 models)
@@ -180,7 +182,7 @@ int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int 
 int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, int T, int H, int ld, float eps, __nv_bfloat16* xb);
 // out[r] = rms(x[rows ? rows[r] : first + r]) * w
 int dc_launch_norm_rows(dc_ctx* ctx, const float* x, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps,
-                        float* out, int ldo);
+                        float* out, __nv_bfloat16* outb, int ldo);
 
 // ---- mix_recur.cu
 struct dc_state_ref {           // per-sequence state in the cache manager's slots
@@ -197,11 +199,11 @@ int dc_launch_delta_scan(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st
                          const float* small, const float* low, int ldd, float* blk, const float* raw_g, int ldg, float eps, float* o,
                          float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp,
-                           float eps, float* mix, int ldm);
+                           float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* act,
                   int lda, float* small, float* blk, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y, int ldy,
-                         float eps, float* mix, int ldm);
+                         float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps);
 
 // ---- mix_latent.cu
@@ -214,7 +216,7 @@ struct dc_latent_cache {
 int dc_launch_latent_prep(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, float* proj, int ldp, float eps,
                           int max_pos);
 int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const float* proj, int ldp,
-                              int splits, float* qa, float* part, float* part_ml, float* mix, int ldm);
+                              int splits, float* qa, float* part, float* part_ml, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const int32_t* key_base,
                             int n_keys, __nv_bfloat16* keys_c, int ldc, __nv_bfloat16* keys_r, int ldr);
 int dc_launch_latent_prefill(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const int32_t* key_base, const int32_t* tiles,

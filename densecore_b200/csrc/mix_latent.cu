@@ -76,41 +76,58 @@ __global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
 }
 
 // ---------------------------------------------------------------- absorbed form
-// qa[t][h][r] = sum_d q[t][h][d] * uk[h][d][r].  CTA: one head, 256 columns, up to NT tokens.
+// qa[t][h][r] = sum_d q[t][h][d] * uk[h][d][r].  CTA: one head, 128 columns, up to NT tokens; warp w takes the rows
+// w, w + 8, ..., a lane four columns.  The first rows are fetched ahead of the dependency wait.
 template <int NT>
-__global__ void __launch_bounds__(128) k_latent_absorb(const float* __restrict__ proj, int ldp, int off_q, int heads, int dim, int rot,
+__global__ void __launch_bounds__(256) k_latent_absorb(const float* __restrict__ proj, int ldp, int off_q, int heads, int dim, int rot,
                                                        const __nv_bfloat16* __restrict__ uk, int ldw, int dim_p, int rank, int T,
                                                        float* __restrict__ qa, int ldq) {
+    constexpr int AHEAD = 16;
     extern __shared__ float sq[];    // [NT][dim]
+    __shared__ float red[8][NT][128];
     pdl_launch_dependents();
+    const int h = blockIdx.x, tb = blockIdx.z * NT, nt = min(NT, T - tb), r0 = blockIdx.y * 128, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r = r0 + 4 * lane;
+    const bool in = r < ldw;         // rows are padded with zeros to ldw columns
+    const __nv_bfloat16* w = uk + (size_t)h * dim_p * ldw + r;
+    uint2 ahead[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+        const int d = warp + 8 * i;
+        ahead[i] = in && d < dim ? __ldg(reinterpret_cast<const uint2*>(w + (size_t)d * ldw)) : make_uint2(0, 0);
+    }
     pdl_wait();
-    const int h = blockIdx.x, tb = blockIdx.z * NT, nt = min(NT, T - tb), r = blockIdx.y * 256 + 2 * threadIdx.x;
-    for (int i = threadIdx.x; i < NT * dim; i += 128) {
+    for (int i = threadIdx.x; i < NT * dim; i += 256) {
         const int t = i / dim, d = i - t * dim;
         sq[i] = t < nt ? proj[(size_t)(tb + t) * ldp + off_q + h * (dim + rot) + d] : 0.0f;
     }
     __syncthreads();
-    if (r >= rank) return;
-    float a[NT][2];
+    float a[NT][4];
 #pragma unroll
-    for (int t = 0; t < NT; ++t) a[t][0] = a[t][1] = 0.0f;
-    const __nv_bfloat16* w = uk + (size_t)h * dim_p * ldw + r;
-#pragma unroll 8
-    for (int d = 0; d < dim; ++d) {
-        const float2 wf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + (size_t)d * ldw));
+    for (int t = 0; t < NT; ++t) a[t][0] = a[t][1] = a[t][2] = a[t][3] = 0.0f;
+    auto add = [&](uint2 v, int d) {
+        const float f[4] = {__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u)};
 #pragma unroll
-        for (int t = 0; t < NT; ++t) {
-            a[t][0] = fmaf(sq[t * dim + d], wf.x, a[t][0]);
-            a[t][1] = fmaf(sq[t * dim + d], wf.y, a[t][1]);
-        }
-    }
+        for (int t = 0; t < NT; ++t)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[t][i] = fmaf(sq[t * dim + d], f[i], a[t][i]);
+    };
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+        if (warp + 8 * i < dim) add(ahead[i], warp + 8 * i);
+    for (int d = warp + 8 * AHEAD; d < dim; d += 8) add(in ? __ldg(reinterpret_cast<const uint2*>(w + (size_t)d * ldw)) : make_uint2(0, 0), d);
 #pragma unroll
     for (int t = 0; t < NT; ++t)
-        if (t < nt) {
-            float* o = qa + ((size_t)(tb + t) * heads + h) * ldq + r;
-            o[0] = a[t][0];
-            if (r + 1 < rank) o[1] = a[t][1];
-        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) red[warp][t][4 * lane + i] = a[t][i];
+    __syncthreads();
+    for (int i = threadIdx.x; i < nt * 128; i += 256) {
+        const int t = i >> 7, c = i & 127;
+        float v = 0.0f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += red[k][t][c];
+        if (r0 + c < rank) qa[((size_t)(tb + t) * heads + h) * ldq + r0 + c] = v;
+    }
 }
 
 __device__ __forceinline__ void unpack16(const uint4& v, float (&f)[8], __nv_bfloat16) {
@@ -170,22 +187,27 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
     const int chunks = row / EPC;
     for (int k0 = kb; k0 < ke; k0 += AB_KEYS) {
         __syncthreads();
-        for (int i = tid; i < AB_KEYS * chunks; i += AB_HEADS * 32) {
-            const int kk = i / chunks, c = i - kk * chunks;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (k0 + kk < ke) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const TC*>(p.c.arena) + p.c.at(seq, k0 + kk) + c * EPC);
-            *reinterpret_cast<uint4*>(sk + kk * ldk + c * EPC) = v;
+#pragma unroll
+        for (int i = 0; i < AB_KEYS / AB_HEADS; ++i) {      // a warp's keys
+            const int kk = warp * (AB_KEYS / AB_HEADS) + i;
+            const bool ok = k0 + kk < ke;
+            const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const TC*>(p.c.arena) + (ok ? p.c.at(seq, k0 + kk) : 0));
+            for (int c = lane; c < chunks; c += 32) *reinterpret_cast<uint4*>(sk + kk * ldk + c * EPC) = ok ? src[c] : make_uint4(0, 0, 0, 0);
         }
         __syncthreads();
         if (!live) continue;
-        float sc = 0.0f;
+        float part[EPC] = {};
         const float* q = sq + warp * row;
+#pragma unroll 4
         for (int c = 0; c < chunks; ++c) {
             float f[EPC];
             unpack16(*reinterpret_cast<const uint4*>(sk + lane * ldk + c * EPC), f, TC());
 #pragma unroll
-            for (int i = 0; i < EPC; ++i) sc = fmaf(f[i], q[c * EPC + i], sc);
+            for (int i = 0; i < EPC; ++i) part[i] = fmaf(f[i], q[c * EPC + i], part[i]);
         }
+        float sc = 0.0f;
+#pragma unroll
+        for (int i = 0; i < EPC; ++i) sc += part[i];
         if (k0 + lane >= ke) sc = -INFINITY;
         float mx = sc;
 #pragma unroll
@@ -198,6 +220,7 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
             acc[j][0] *= corr;
             acc[j][1] *= corr;
         }
+#pragma unroll 4
         for (int kk = 0; kk < AB_KEYS; ++kk) {
             const float w = __shfl_sync(0xffffffffu, pr, kk);
             const TC* kr = sk + kk * ldk;
@@ -225,32 +248,40 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
     }
 }
 
-// Splits of one (head, token) joined, then taken through the head's W_uv.
+// Splits of one (head, token) joined, then taken through OUT_ROWS rows of the head's W_uv.
+constexpr int OUT_ROWS = 64;
 __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits,
                                                     int rank, const __nv_bfloat16* __restrict__ uv, int ldw, int vdim_p, int vdim,
-                                                    float* __restrict__ mix, int ldm) {
+                                                    float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
     extern __shared__ __align__(16) float lat[];      // [rank padded to 8]
+    __shared__ float sw[32];
     pdl_launch_dependents();
+    const int h = blockIdx.x, t = blockIdx.y, e0 = blockIdx.z * OUT_ROWS, e1 = min(vdim, e0 + OUT_ROWS), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const char* rows = reinterpret_cast<const char*>(uv + (size_t)(h * vdim_p + e0) * ldw);
+    for (int i = threadIdx.x * 128; i < (e1 - e0) * ldw * 2; i += 256 * 128) prefetch_l2(rows + i);
     pdl_wait();
-    const int h = blockIdx.x, t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const size_t o = ((size_t)t * heads + h) * splits;
-    float M = -INFINITY;
-    for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[2 * (o + s)]);
-    float L = 0.0f;
-    for (int s = 0; s < splits; ++s) L += part_ml[2 * (o + s) + 1] * expf(part_ml[2 * (o + s)] - M);
-    const float inv = 1.0f / L;
+    if (warp == 0) {             // splits <= 32
+        const float m = lane < splits ? part_ml[2 * (o + lane)] : -INFINITY, l = lane < splits ? part_ml[2 * (o + lane) + 1] : 0.0f;
+        float M = m;
+#pragma unroll
+        for (int k = 16; k > 0; k >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, k));
+        const float w = expf(m - M), L = warp_sum(l * w);
+        sw[lane] = w / L;
+    }
+    __syncthreads();
     const int rank8 = (rank + 7) & ~7;
     for (int r = threadIdx.x; r < rank8; r += 256) {
         float v = 0.0f;
-        if (r < rank)
-            for (int s = 0; s < splits; ++s) {
-                const float w = expf(part_ml[2 * (o + s)] - M);
-                if (w > 0.0f) v = fmaf(part[(o + s) * rank + r], w, v);     // an empty split holds nothing readable
-            }
-        lat[r] = v * inv;
+        if (r < rank) {
+#pragma unroll 8
+            for (int s = 0; s < splits; ++s) v = fmaf(part[(o + s) * rank + r], sw[s], v);
+        }
+        lat[r] = v;
     }
     __syncthreads();
-    for (int e = warp; e < vdim; e += 8) {
+#pragma unroll 4
+    for (int e = e0 + warp; e < e1; e += 8) {
         const uint4* w = reinterpret_cast<const uint4*>(uv + (size_t)(h * vdim_p + e) * ldw);
         float a = 0.0f;
         for (int c = lane; c < rank8 / 8; c += 32) {
@@ -260,7 +291,9 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
             for (int i = 0; i < 8; ++i) a = fmaf(f[i], lat[8 * c + i], a);
         }
         a = warp_sum(a);
-        if (lane == 0) mix[(size_t)t * ldm + (size_t)h * vdim + e] = a;
+        const size_t at = (size_t)t * ldm + (size_t)h * vdim + e;
+        if (lane == 0 && mixb) mixb[at] = __float2bfloat16_rn(a);
+        else if (lane == 0) mix[at] = a;
     }
 }
 
@@ -363,19 +396,27 @@ __global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
     const __nv_bfloat16* kr = p.kr + (size_t)(p.key_base[e] - key0) * p.ldr;
     const int kc = p.dim_p / 8, rc = p.ldr / 8, pad = p.dq / 8, vc = p.vdim_p / 8;
 
+    // eight threads per key row
+    const int lrow = tid >> 3, lc = tid & 7;
     auto load = [&](int tile, int buf) {
-        const int k0 = first + tile * PK;
-        for (int i = tid; i < PK * pad; i += 128) {
-            const int key = i / pad, c = i - key * pad, pos = k0 + key;
-            const bool ok = pos <= last && c < kc + rc;
-            const __nv_bfloat16* src = !ok ? p.kv : c < kc ? kv + (ptrdiff_t)pos * p.ldkv + head * p.dim_p + c * 8 : kr + (ptrdiff_t)pos * p.ldr + (c - kc) * 8;
-            cp_async16z(smem_u32(sK + (buf * PK + key) * ldk + c * 8), src, ok);
-        }
-        for (int i = tid; i < PK * (VD / 8); i += 128) {
-            const int key = i / (VD / 8), c = i - key * (VD / 8), pos = k0 + key;
-            const bool ok = pos <= last && c < vc;
-            const __nv_bfloat16* src = ok ? kv + (ptrdiff_t)pos * p.ldkv + p.uv_row + head * p.vdim_p + c * 8 : p.kv;
-            cp_async16z(smem_u32(sV + (buf * PK + key) * LDV + c * 8), src, ok);
+#pragma unroll
+        for (int i = 0; i < PK / 16; ++i) {
+            const int key = lrow + 16 * i, pos = first + tile * PK + key;
+            const bool ok = pos <= last;
+            const __nv_bfloat16* krow = ok ? kv + (ptrdiff_t)pos * p.ldkv : p.kv;
+            const __nv_bfloat16* rrow = (ok ? kr + (ptrdiff_t)pos * p.ldr : p.kr) - kc * 8;
+            const uint32_t dk = smem_u32(sK + (buf * PK + key) * ldk), dv = smem_u32(sV + (buf * PK + key) * LDV);
+            for (int c = lc; c < pad; c += 8) {
+                const bool in = ok && c < kc + rc;
+                cp_async16z(dk + 16 * c, in ? (c < kc ? krow + head * p.dim_p : rrow) + 8 * c : p.kv, in);
+            }
+#pragma unroll
+            for (int c0 = 0; c0 < VD / 8; c0 += 8) {
+                const int c = c0 + lc;
+                if (VD / 8 < 8 && c >= VD / 8) break;
+                const bool in = ok && c < vc;
+                cp_async16z(dv + 16 * c, in ? krow + p.uv_row + head * p.vdim_p + 8 * c : p.kv, in);
+            }
         }
         cp_async_commit();
     };
@@ -509,20 +550,19 @@ int dc_launch_latent_prep(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& 
 }
 
 int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const float* proj, int ldp,
-                              int splits, float* qa, float* part, float* part_ml, float* mix, int ldm) {
-    const int ldq = dc_pad8(m.kv_rank), rb = (m.kv_rank + 255) / 256;
+                              int splits, float* qa, float* part, float* part_ml, float* mix, __nv_bfloat16* mixb, int ldm) {
+    const int ldq = dc_pad8(m.kv_rank), rb = (m.kv_rank + 127) / 128;
 #define DC_ABSORB(NT)                                                                                                                        \
-    DC_TRY(dc_launch(ctx, "k_latent_absorb", k_latent_absorb<NT>, dim3(m.heads, rb, (st.T + NT - 1) / NT), dim3(128), (size_t)NT * m.dim * 4, \
+    DC_TRY(dc_launch(ctx, "k_latent_absorb", k_latent_absorb<NT>, dim3(m.heads, rb, (st.T + NT - 1) / NT), dim3(256), (size_t)NT * m.dim * 4, \
                      proj, ldp, m.off_q, m.heads, m.dim, m.rot_dim, m.ukv.w, m.ukv.ld, m.dim_p, m.kv_rank, st.T, qa, ldq))
     if (st.T == 1) DC_ABSORB(1);
-    else if (st.T <= 4) DC_ABSORB(4);
-    else DC_ABSORB(16);
+    else DC_ABSORB(4);
 #undef DC_ABSORB
     AbsorbedParams p = {qa, ldq, proj, ldp, m.off_q, m.heads, m.dim, m.rot_dim, m.kv_rank, m.window, splits, m.scale, st.seq_ids, st.positions,
                         cache_ref(c, m.row), part, part_ml};
     DC_TRY(c.f32 ? launch_absorbed<float>(ctx, p, st.T) : launch_absorbed<__nv_bfloat16>(ctx, p, st.T));
-    return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T), dim3(256), (size_t)dc_pad8(m.kv_rank) * 4, part, part_ml, m.heads, splits,
-                     m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim, mix, ldm);
+    return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T, (m.vdim + OUT_ROWS - 1) / OUT_ROWS), dim3(256), (size_t)dc_pad8(m.kv_rank) * 4, part, part_ml, m.heads, splits,
+                     m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim, mix, mixb, ldm);
 }
 
 int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const int32_t* key_base,

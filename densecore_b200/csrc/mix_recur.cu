@@ -365,23 +365,6 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// a pair of f32 values in one register pair, two multiply-adds per instruction
-__device__ __forceinline__ uint64_t pair(float a, float b) {
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ float2 unpair(uint64_t v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-
 // EPL consecutive-chunk channels per lane: lane's channel i is W * lane + 32 W (i / W) + i % W.
 template <int EPL>
 struct Chan {
@@ -633,6 +616,7 @@ struct DeltaDecode {
     const float *neg_a, *dt_bias, *norm;
     size_t state_off;
     float* mix;
+    __nv_bfloat16* mixb;         // instead of mix
     int ldm;
 };
 
@@ -661,15 +645,21 @@ __device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ldw, i
 // One CTA per (head, sequence): convolutions, unit vectors, decays and gates, the state's step, the gated norm.
 template <int EPL>
 __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
-    constexpr int DP = 32 * EPL;
+    constexpr int DP = 32 * EPL, NC = 8;            // columns of a warp at a time
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[33], s_iq, s_ik;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, t = blockIdx.y, kh = h / p.per;
     const int ra = (p.a_rank + 7) & ~7, rg = (p.g_rank + 7) & ~7;
     float *sq = sm, *sk = sq + DP, *sg = sk + DP, *sa = sg + DP, *sgl = sa + ra, *sv = sgl + rg, *so = sv + p.vdim, *sgate = so + p.vdim;
     pdl_launch_dependents();
+    // the gates' weights do not depend on the kernel before: on their way to L2 while this one still waits
+    const char *pa = (const char*)(p.a2 + (size_t)h * p.dim * p.lda2), *pg = (const char*)(p.g2 + (size_t)h * p.vdim * p.ldg2);
+    for (int i = tid * 128; i < p.dim * p.lda2 * 2; i += 256 * 128) prefetch_l2(pa + i);
+    for (int i = tid * 128; i < p.vdim * p.ldg2 * 2; i += 256 * 128) prefetch_l2(pg + i);
     pdl_wait();
     const int pos = p.cr.positions[t], seq = p.cr.seq_ids[t], taps = p.cr.taps;
+    float* S = reinterpret_cast<float*>(p.cr.base + (size_t)seq * p.cr.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.dim;
+    for (int i = tid * 32; i < p.vdim * p.dim; i += 256 * 32) prefetch_l2(S + i);
     float* ring = p.cr.ring(seq);
     const float* row = p.proj + (size_t)t * p.ldp;
     const bool first = h % p.per == 0;
@@ -709,12 +699,10 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
     for (int i = 0; i < EPL; ++i) kq = fmaf(kr[i], qr[i], kq);
     kq = warp_sum(kq);
     const float beta = sigmoid(row[p.off_b + h]);
-    float* S = reinterpret_cast<float*>(p.cr.base + (size_t)seq * p.cr.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.dim;
-#pragma unroll 2
-    for (int c0 = 4 * warp; c0 < p.vdim; c0 += 32) {
-        float s[4][EPL], a[4], b[4];
+    for (int c0 = NC * warp; c0 < p.vdim; c0 += 8 * NC) {
+        float s[NC][EPL], a[NC], b[NC];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < NC; ++c) {
             a[c] = b[c] = 0.0f;
 #pragma unroll
             for (int i = 0; i < EPL; ++i) {
@@ -723,19 +711,19 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
             }
         }
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
+        for (int c = 0; c < NC; ++c)
 #pragma unroll
             for (int i = 0; i < EPL; ++i) {
                 a[c] = fmaf(s[c][i], kr[i], a[c]);
                 b[c] = fmaf(s[c][i], qr[i], b[c]);
             }
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < NC; ++c) {
             a[c] = warp_sum(a[c]);
             b[c] = warp_sum(b[c]);
         }
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < NC; ++c) {
             if (c0 + c >= p.vdim) continue;
             const float u = beta * (sv[c0 + c] - a[c]);
             if (lane == 0) so[c0 + c] = fmaf(kq, u, b[c]);
@@ -750,7 +738,12 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
     float ss = 0.0f;
     for (int c = tid; c < p.vdim; c += 256) ss = fmaf(so[c], so[c], ss);
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.vdim + p.eps);
-    for (int c = tid; c < p.vdim; c += 256) p.mix[(size_t)t * p.ldm + (size_t)h * p.vdim + c] = so[c] * inv * p.norm[c] * sigmoid(sgate[c]);
+    for (int c = tid; c < p.vdim; c += 256) {
+        const float v = so[c] * inv * p.norm[c] * sigmoid(sgate[c]);
+        const size_t o = (size_t)t * p.ldm + (size_t)h * p.vdim + c;
+        if (p.mixb) p.mixb[o] = __float2bfloat16_rn(v);
+        else p.mix[o] = v;
+    }
 }
 
 struct SsdDecode {
@@ -767,13 +760,15 @@ struct SsdDecode {
 // One CTA per (head, sequence): convolutions, the state's step, the gate (the group norm spans heads).
 template <int EPL>
 __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
-    constexpr int DP = 32 * EPL;
+    constexpr int DP = 32 * EPL, NC = 8;            // columns of a warp at a time
     extern __shared__ __align__(16) float sm[];     // B, C: [DP]; x: [vdim]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, t = blockIdx.y, g = h / p.per;
     float* sx = sm + 2 * DP;
     pdl_launch_dependents();
     pdl_wait();
     const int pos = p.cr.positions[t], seq = p.cr.seq_ids[t], taps = p.cr.taps, inner = p.heads * p.vdim, GN = p.groups * p.state;
+    float* S = reinterpret_cast<float*>(p.cr.base + (size_t)seq * p.cr.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.state;
+    for (int i = tid * 32; i < p.vdim * p.state; i += 128 * 32) prefetch_l2(S + i);
     float* ring = p.cr.ring(seq);
     const float* row = p.proj + (size_t)t * p.ldp;
     const bool first = h % p.per == 0;
@@ -792,19 +787,17 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
     float br[EPL], cr[EPL];
     Chan<EPL>::load(sm, lane, br);
     Chan<EPL>::load(sm + DP, lane, cr);
-    float* S = reinterpret_cast<float*>(p.cr.base + (size_t)seq * p.cr.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.state;
-#pragma unroll 2
-    for (int c0 = 4 * warp; c0 < p.vdim; c0 += 16) {
-        float s[4][EPL], a[4];
+    for (int c0 = NC * warp; c0 < p.vdim; c0 += 4 * NC) {
+        float s[NC][EPL], a[NC];
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
+        for (int c = 0; c < NC; ++c)
 #pragma unroll
             for (int i = 0; i < EPL; ++i) {
                 const int d = Chan<EPL>::at(lane, i);
                 s[c][i] = pos > 0 && c0 + c < p.vdim && d < p.state ? S[(size_t)(c0 + c) * p.state + d] : 0.0f;
             }
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < NC; ++c) {
             const float u = c0 + c < p.vdim ? dt * sx[c0 + c] : 0.0f;
             a[c] = 0.0f;
 #pragma unroll
@@ -816,12 +809,11 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
             }
         }
 #pragma unroll
-        for (int c = 0; c < 4; ++c) a[c] = warp_sum(a[c]);
-        if (lane < 4 && c0 + lane < p.vdim) {
-            const int c = c0 + lane;
-            const float av = lane == 0 ? a[0] : lane == 1 ? a[1] : lane == 2 ? a[2] : a[3];
-            p.y[(size_t)t * p.ldy + (size_t)h * p.vdim + c] = fmaf(Dh, sx[c], av) * silu(row[p.off_z + (size_t)h * p.vdim + c]);
-        }
+        for (int c = 0; c < NC; ++c) a[c] = warp_sum(a[c]);
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+            if (lane == c && c0 + c < p.vdim)
+                p.y[(size_t)t * p.ldy + (size_t)h * p.vdim + c0 + c] = fmaf(Dh, sx[c0 + c], a[c]) * silu(row[p.off_z + (size_t)h * p.vdim + c0 + c]);
     }
 }
 
@@ -982,11 +974,11 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
 }
 
 int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
-                           float* mix, int ldm) {
+                           float* mix, __nv_bfloat16* mixb, int ldm) {
     const int V = m.heads * m.vdim;
     DeltaDecode p = {conv_ref(st, sr, m.taps, m.off_v + V), proj, ldp, m.conv, m.heads, m.heads / m.kv_heads, m.dim, m.vdim, m.off_q, m.off_k, m.off_v, m.off_b,
                      m.off_a, m.off_g, m.a_rank, m.g_rank, m.unit_eps, m.q_scale, eps, m.a2.w, m.g2.w, m.a2.ld, m.g2.ld, m.neg_a, m.dt_bias, m.norm,
-                     sr.state_off, mix, ldm};
+                     sr.state_off, mix, mixb, ldm};
     p.cr.ldw = m.off_v + dc_pad8(V);
     const int dp = key_pad(m.dim);
     const size_t smem = (size_t)(3 * dp + dc_pad8(m.a_rank) + dc_pad8(m.g_rank) + 3 * m.vdim) * 4;
@@ -999,7 +991,7 @@ int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& 
 }
 
 int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y, int ldy,
-                         float eps, float* mix, int ldm) {
+                         float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
     const int inner = m.heads * m.vdim, C = inner + 2 * m.groups * m.state;
     SsdDecode p = {conv_ref(st, sr, m.taps, C), proj, ldp, m.conv, m.conv_b, m.dt_bias, m.neg_a, m.D, m.heads, m.heads / m.groups, m.groups, m.state, m.vdim,
                    m.off_x, m.off_dt, m.off_z, sr.state_off, y, ldy};
@@ -1010,6 +1002,9 @@ int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, 
     else if (dp == 64) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<2>, grid, block, smem, p));
     else if (dp == 128) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<4>, grid, block, smem, p));
     else DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<8>, grid, block, smem, p));
+    if (mixb)
+        return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<__nv_bfloat16>, dim3(m.norm_groups, st.T), dim3(256), 0, y, ldy, nullptr, 0, m.norm,
+                         inner / m.norm_groups, eps, mixb, ldm);
     return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<float>, dim3(m.norm_groups, st.T), dim3(256), 0, y, ldy, nullptr, 0, m.norm,
                      inner / m.norm_groups, eps, mix, ldm);
 }

@@ -27,7 +27,8 @@ __global__ void __launch_bounds__(256) k_post_norm(float* __restrict__ x, const 
 }
 
 __global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, const float* __restrict__ w, const int32_t* __restrict__ rows,
-                                                   int first, int H, int ld, float eps, float* __restrict__ out, int ldo) {
+                                                   int first, int H, int ld, float eps, float* __restrict__ out,
+                                                   __nv_bfloat16* __restrict__ outb, int ldo) {
     __shared__ float red[33];
     dc::pdl_launch_dependents();
     dc::pdl_wait();
@@ -36,7 +37,11 @@ __global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, 
     float ss = 0.0f;
     for (int i = threadIdx.x; i < H; i += 256) ss = fmaf(xr[i], xr[i], ss);
     const float inv = 1.0f / sqrtf(dc::block_sum(ss, red) / (float)H + eps);
-    for (int i = threadIdx.x; i < H; i += 256) out[(size_t)blockIdx.x * ldo + i] = xr[i] * inv * w[i];
+    for (int i = threadIdx.x; i < H; i += 256) {
+        const float v = xr[i] * inv * w[i];
+        if (outb) outb[(size_t)blockIdx.x * ldo + i] = __float2bfloat16_rn(v);
+        else out[(size_t)blockIdx.x * ldo + i] = v;
+    }
 }
 
 }  // namespace
@@ -46,6 +51,6 @@ int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, i
 }
 
 int dc_launch_norm_rows(dc_ctx* ctx, const float* x, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps,
-                        float* out, int ldo) {
-    return dc_launch(ctx, "k_norm_rows", k_norm_rows, dim3(R), dim3(256), 0, x, w, rows, first, H, ld, eps, out, ldo);
+                        float* out, __nv_bfloat16* outb, int ldo) {
+    return dc_launch(ctx, "k_norm_rows", k_norm_rows, dim3(R), dim3(256), 0, x, w, rows, first, H, ld, eps, out, outb, ldo);
 }

@@ -208,8 +208,8 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
             a.cos_sin = table;
         }
     }
-    // key splits of a decode step: about 64 keys each at the longest span
-    s->splits = std::max(1, std::min(32, (span + 63) / 64));
+    // key splits of a decode step: about 32 keys each at the longest span
+    s->splits = std::max(1, std::min(32, (span + 31) / 32));
     const int per_seq = (c.max_ctx + DC_KV_BLOCK - 1) / DC_KV_BLOCK;
     const int blocks = pool_tokens > 0 ? (pool_tokens + DC_KV_BLOCK - 1) / DC_KV_BLOCK : per_seq * c.max_seqs;
     return dc_kv_init_planes(ctx, &m->kv, planes, state, blocks, c.max_seqs, per_seq);
@@ -266,6 +266,7 @@ int dc_stack_finalize(dc_model* m) {
     DC_TRY(alloc(m, &b.ff, F * ff));
     DC_TRY(alloc(m, &b.lm_x, DC_MAX_T * H));
     if (!f32) {
+        DC_TRY(alloc(m, &b.lm_xb, DC_MAX_T * H));
         DC_TRY(alloc(m, &b.xb, C * H));
         DC_TRY(alloc(m, &b.mixb, C * mix));
         DC_TRY(alloc(m, &b.ffb, C * ff));
@@ -331,10 +332,11 @@ int tc_in(dc_model* m, dc_tc_in* out, const __nv_bfloat16* x, int K, int ld, int
     return DC_B200_OK;
 }
 
-// y = W x for the step's tokens: xf is the f32 input, xb its bf16 copy (tensor-core steps), same pitch.
+// y = W x for the step's tokens: xf is the input of f32 models, xb that of bf16 models, same pitch.
 int linear(dc_model* m, const dc_step& st, const dc_lin& w, const float* xf, const __nv_bfloat16* xb, int ldx, int epi, float* out,
            __nv_bfloat16* outb, int ldo) {
-    if (st.tc) {
+    if (st.b16 && st.T <= DC_MAX_T) return dc_launch_linear_mma(m->ctx, w, xb, ldx, st.T, epi, outb ? nullptr : out, outb, ldo);
+    if (st.b16) {
         dc_tc_in in;
         DC_TRY(tc_in(m, &in, xb, w.K, ldx, m->stack->b.cap));
         return dc_launch_linear_tc(m->ctx, w, in, st.T, epi, outb ? nullptr : out, outb, ldo);
@@ -367,11 +369,11 @@ int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
     const dc_stack_buffers& b = m->stack->b;
     const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
     const int ldp = d.in.N, lda = dc_pad8(d.off_v + d.heads * d.vdim), ldl = d.in.N - d.off_a, ldm = d.heads * d.vdim;
-    if (st.single && !st.tc && st.T <= DC_MAX_T)
-        return dc_launch_delta_decode(m->ctx, d, st, sr, b.proj, ldp, m->stack->cfg.eps, b.mix, dc_pad8(ldm));
-    __nv_bfloat16* lowb = st.tc ? b.lowb : nullptr;
+    if (st.single && st.T <= DC_MAX_T)
+        return dc_launch_delta_decode(m->ctx, d, st, sr, b.proj, ldp, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(ldm));
+    __nv_bfloat16* lowb = st.b16 ? b.lowb : nullptr;
     DC_TRY(dc_launch_delta_prep(m->ctx, d, st, sr, b.proj, ldp, b.act, lda, b.small, lowb, ldl));
-    if (st.tc) {
+    if (st.b16) {
         DC_TRY(linear(m, st, d.a2, nullptr, lowb, ldl, DC_LIN_STORE, b.low, nullptr, d.a2.N));
         DC_TRY(linear(m, st, d.g2, nullptr, lowb + (d.off_g - d.off_a), ldl, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
     } else {
@@ -379,7 +381,7 @@ int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
         DC_TRY(linear(m, st, d.g2, b.proj + d.off_g, nullptr, ldp, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
     }
     return dc_launch_delta_scan(m->ctx, d, st, sr, b.act, lda, b.small, b.low, d.a2.N, b.blk, b.gate, d.g2.N, m->stack->cfg.eps, b.scan,
-                                st.tc ? nullptr : b.mix, st.tc ? b.mixb : nullptr, dc_pad8(ldm));
+                                st.b16 ? nullptr : b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(ldm));
 }
 
 int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
@@ -387,10 +389,10 @@ int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
     const dc_stack_buffers& b = m->stack->b;
     const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
     const int inner = d.heads * d.vdim, lda = dc_pad8(inner + 2 * d.groups * d.state);
-    if (st.single && !st.tc && st.T <= DC_MAX_T)
-        return dc_launch_ssd_decode(m->ctx, d, st, sr, b.proj, d.in.N, b.scan, lda, m->stack->cfg.eps, b.mix, dc_pad8(inner));
-    return dc_launch_ssd(m->ctx, d, st, sr, b.proj, d.in.N, b.act, lda, b.small, b.blk, b.scan, m->stack->cfg.eps, st.tc ? nullptr : b.mix,
-                         st.tc ? b.mixb : nullptr, dc_pad8(inner));
+    if (st.single && st.T <= DC_MAX_T)
+        return dc_launch_ssd_decode(m->ctx, d, st, sr, b.proj, d.in.N, b.scan, lda, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(inner));
+    return dc_launch_ssd(m->ctx, d, st, sr, b.proj, d.in.N, b.act, lda, b.small, b.blk, b.scan, m->stack->cfg.eps, st.b16 ? nullptr : b.mix,
+                         st.b16 ? b.mixb : nullptr, dc_pad8(inner));
 }
 
 int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
@@ -404,7 +406,8 @@ int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_laye
     const int ldp = d.in.N, ldm = dc_pad8(d.heads * d.vdim);
     DC_TRY(dc_launch_latent_prep(m->ctx, d, st, c, b.proj, ldp, m->stack->cfg.eps, m->cfg.max_ctx));
     if (!st.tc)
-        return dc_launch_latent_absorbed(m->ctx, d, st, c, b.proj, ldp, st.T <= DC_MAX_T ? m->stack->splits : 1, b.qa, b.part, b.part_ml, b.mix, ldm);
+        return dc_launch_latent_absorbed(m->ctx, d, st, c, b.proj, ldp, st.T <= DC_MAX_T ? m->stack->splits : 1, b.qa, b.part, b.part_ml, b.mix,
+                                         st.b16 ? b.mixb : nullptr, ldm);
     const int32_t* base = sk.base[d.range];
     const int nk = sk.count[d.range], ldc = dc_pad8(d.kv_rank), ldr = dc_pad8(d.rot_dim);
     DC_TRY(dc_launch_latent_gather(m->ctx, d, st, c, base, nk, b.keys_c, ldc, b.keys_r, ldr));
@@ -421,7 +424,7 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
     dc_stack_buffers& b = s->b;
     const int W = s->cfg.width, H = dc_pad8(W), T = st.T;
     const float eps = s->cfg.eps;
-    __nv_bfloat16* xb = st.tc ? b.xb : nullptr;
+    __nv_bfloat16* xb = st.b16 ? b.xb : nullptr;
     auto capture = [&](int il) -> int {     // parity aid: what enters layer il (the last slot: the output norm)
         if (!m->dbg_x || T > DC_MAX_T) return DC_B200_OK;
         return dc_check_cuda(ctx, cudaMemcpy2DAsync(m->dbg_x + (size_t)il * DC_MAX_T * W, (size_t)W * 4, b.x, (size_t)H * 4, (size_t)W * 4, T,
@@ -442,7 +445,7 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));
         if (!Ly.ff) continue;
         const int F = dc_pad8(Ly.ff);
-        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, DC_LIN_GELU_PAIR, b.ff, st.tc ? b.ffb : nullptr, F));
+        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, DC_LIN_GELU_PAIR, b.ff, st.b16 ? b.ffb : nullptr, F));
         L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, DC_LIN_STORE, b.y, nullptr, H));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm2, T, W, H, eps, xb));
     }
@@ -455,8 +458,10 @@ int run_head(dc_model* m, const int32_t* rows, int first, int R, bool feedback) 
     dc_ctx* ctx = m->ctx;
     const int W = s->cfg.width, H = dc_pad8(W);
     dc_step_buffers& g = m->buf;
-    L(DC_K_POST_NORM, 8.0 * R * W, 1, dc_launch_norm_rows(ctx, s->b.x, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, H));
-    L(DC_K_LM_HEAD, lin_bytes(s->head, R), 1, dc_launch_linear_rows(ctx, s->head, s->b.lm_x, H, R, DC_LIN_STORE, g.logits, s->cfg.vocab, g.argmax_keys));
+    L(DC_K_POST_NORM, 8.0 * R * W, 1, dc_launch_norm_rows(ctx, s->b.x, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, s->b.lm_xb, H));
+    L(DC_K_LM_HEAD, lin_bytes(s->head, R), 1,
+      s->b.lm_xb ? dc_launch_linear_mma(ctx, s->head, s->b.lm_xb, H, R, DC_LIN_STORE, g.logits, nullptr, s->cfg.vocab, g.argmax_keys)
+                 : dc_launch_linear_rows(ctx, s->head, s->b.lm_x, H, R, DC_LIN_STORE, g.logits, s->cfg.vocab, g.argmax_keys));
     L(DC_K_ARGMAX, 64.0, 1, dc_launch_argmax_finish(ctx, g.argmax_keys, R, g.out_tokens, feedback ? g.tokens : nullptr, feedback ? g.positions : nullptr,
                                                     feedback ? g.history : nullptr, feedback ? g.history_len : nullptr, DC_HISTORY_CAP));
     return DC_B200_OK;
@@ -472,6 +477,7 @@ int dc_stack_enqueue_small(dc_model* m, int T, bool chunk, int lm_mode, bool fee
     st.tokens = m->buf.tokens, st.seq_ids = m->buf.seq_ids, st.positions = m->buf.positions;
     st.starts = chunk ? m->stack->b.chunk + 2 * T : m->stack->b.iota;
     st.single = !chunk || T == 1;
+    st.b16 = m->stack->dtype == DC_DTYPE_BF16;
     DC_TRY(run_layers(m, st, StepKeys()));
     if (lm_mode == 1) return run_head(m, nullptr, T - 1, 1, feedback);
     return lm_mode ? run_head(m, nullptr, 0, T, feedback) : DC_B200_OK;
@@ -536,8 +542,8 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
         st.tokens = b.meta, st.seq_ids = b.meta + C, st.positions = b.meta + 2 * C, st.starts = b.meta + (h_start - h);
         for (size_t w = 0; w < s->windows.size(); ++w) sk.base.push_back(b.meta + (h_base - h) + w * ENTRY_INTS);
         sk.tiles = b.meta + (h_tiles - h);
-        // more tokens than the row-streaming products take at once: tensor cores (bf16 models)
-        st.tc = s->dtype == DC_DTYPE_BF16 && st.T > DC_MAX_T;
+        st.b16 = s->dtype == DC_DTYPE_BF16;
+        st.tc = st.b16 && st.T > DC_MAX_T;
         DC_TRY(run_layers(m, st, sk));
         for (int r = 0; r < R; r += DC_MAX_T) {
             const int n = std::min(DC_MAX_T, R - r);
