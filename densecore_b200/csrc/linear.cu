@@ -1,7 +1,7 @@
 // Products y = W x with bf16 weights and f32 accumulation for up to sixteen tokens, and for f32 activations.
 //
-// k_linear_mma (bf16 activations) streams the weight rows once: a CTA owns sixteen rows, its eight warps take
-// alternate runs of 32 columns and feed them to m16n8k16 products.  A lane loads sixteen bytes of a row at a time;
+// k_linear_mma (bf16 activations) streams the weight rows once: a CTA owns sixteen rows, its sixteen warps
+// take neighbouring runs of 32 columns and feed them to m16n8k16 products.  A lane loads sixteen bytes of a row at a time;
 // both operands use the same order of columns within a run, so the fragments need no shuffling.  k_linear_rows (f32
 // activations, f32 models) does the same on the CUDA cores: a warp owns R rows, a lane takes runs of eight weights, the
 // activations come through L1.  Weights do not depend on the kernel before, so every warp fetches its first ones
@@ -147,7 +147,7 @@ int launch_rows_any(dc_ctx* ctx, const RowsParams& p) {
 }
 
 // ---- sixteen rows per CTA on the tensor cores
-constexpr int LM_WARPS = 8, LM_AHEAD = 4;    // LM_AHEAD: runs of 32 columns a warp keeps in flight
+constexpr int LM_WARPS = 16;
 
 struct MmaParams {
     const __nv_bfloat16* w;
@@ -166,8 +166,8 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-// NT: groups of eight tokens.  Column 8 q + 4 s + e of a run (q: lane % 4) is k-slot 2 q + e % 2 + 8 (e / 2) of product s.
-template <int NT, int EPI>
+// NT: groups of eight tokens; AHEAD: neighbouring runs of 32 columns that a warp keeps in flight.  Column 8 q + 4 s + e of a run (q: lane % 4) is k-slot 2 q + e % 2 + 8 (e / 2) of product s.
+template <int NT, int AHEAD, int EPI>
 __global__ void __launch_bounds__(LM_WARPS * 32) k_linear_mma(const MmaParams p) {
     __shared__ float red[LM_WARPS][16][8 * NT + 1];
     dc::pdl_launch_dependents();
@@ -176,25 +176,25 @@ __global__ void __launch_bounds__(LM_WARPS * 32) k_linear_mma(const MmaParams p)
     // the matrix has a multiple of eight rows
     const uint4* w0 = reinterpret_cast<const uint4*>(p.w + (size_t)(row0 + g) * p.ldw) + q;
     const uint4* w1 = reinterpret_cast<const uint4*>(p.w + (size_t)min(row0 + 8 + g, p.N - 1) * p.ldw) + q;
-    uint4 a[LM_AHEAD][2];
+    uint4 a[AHEAD][2];
     auto fetch = [&](int j, int run) {
         const bool ok = 32 * run + 8 * q < K8;
         a[j][0] = ok ? __ldg(w0 + 4 * run) : make_uint4(0, 0, 0, 0);
         a[j][1] = ok ? __ldg(w1 + 4 * run) : make_uint4(0, 0, 0, 0);
     };
 #pragma unroll
-    for (int j = 0; j < LM_AHEAD; ++j) fetch(j, warp + LM_WARPS * j);
+    for (int j = 0; j < AHEAD; ++j) fetch(j, warp * AHEAD + j);
     dc::pdl_wait();
     float acc[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
-    for (int rb = warp; rb < runs; rb += LM_WARPS * LM_AHEAD) {
+    for (int rb = warp * AHEAD; rb < runs; rb += LM_WARPS * AHEAD) {
 #pragma unroll
-        for (int j = 0; j < LM_AHEAD; ++j) {
-            const int run = rb + LM_WARPS * j, k = 32 * run + 8 * q;
+        for (int j = 0; j < AHEAD; ++j) {
+            const int run = rb + j, k = 32 * run + 8 * q;
             if (run >= runs) break;
             const uint4 a0 = a[j][0], a1 = a[j][1];
-            fetch(j, run + LM_WARPS * LM_AHEAD);
+            fetch(j, run + LM_WARPS * AHEAD);
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
                 uint4 b = make_uint4(0, 0, 0, 0);
@@ -283,6 +283,13 @@ __global__ void __launch_bounds__(256) k_linear_f32(const RowsParams p, int epi)
     }
 }
 
+template <int NT, int AHEAD>
+int launch_mma_any(dc_ctx* ctx, const MmaParams& p, bool gelu) {
+    const dim3 grid((p.N + 15) / 16), block(LM_WARPS * 32);
+    return gelu ? dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD, DC_LIN_GELU_PAIR>, grid, block, 0, p)
+                : dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD, DC_LIN_STORE>, grid, block, 0, p);
+}
+
 }  // namespace
 
 int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, int epi, float* out, __nv_bfloat16* outb, int ldo,
@@ -291,12 +298,10 @@ int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, i
     const bool gelu = epi == DC_LIN_GELU_PAIR;
     MmaParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, out, outb, ldo, gelu ? w.N / 2 : w.N, keys};
     if (p.n_out > ldo) p.n_out = ldo;
-    const dim3 grid((w.N + 15) / 16), block(LM_WARPS * 32);
-    if (T <= 8)
-        return gelu ? dc_launch(ctx, "k_linear_mma", k_linear_mma<1, DC_LIN_GELU_PAIR>, grid, block, 0, p)
-                    : dc_launch(ctx, "k_linear_mma", k_linear_mma<1, DC_LIN_STORE>, grid, block, 0, p);
-    return gelu ? dc_launch(ctx, "k_linear_mma", k_linear_mma<2, DC_LIN_GELU_PAIR>, grid, block, 0, p)
-                : dc_launch(ctx, "k_linear_mma", k_linear_mma<2, DC_LIN_STORE>, grid, block, 0, p);
+    // a small matrix needs more of it in flight per warp, a large one has enough warps
+    const bool small = (w.N + 15) / 16 <= 2 * ctx->num_sms;
+    if (T <= 8) return small ? launch_mma_any<1, 4>(ctx, p, gelu) : launch_mma_any<1, 2>(ctx, p, gelu);
+    return small ? launch_mma_any<2, 4>(ctx, p, gelu) : launch_mma_any<2, 2>(ctx, p, gelu);
 }
 
 int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo, unsigned long long* keys) {

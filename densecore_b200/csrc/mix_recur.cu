@@ -42,13 +42,18 @@ __device__ __forceinline__ float conv_at(const float* __restrict__ proj, int ldp
         for (int j = 0; j < taps; ++j) s = fmaf(w[(size_t)j * ldw], in[(size_t)j * ldp], s);
         return s;
     }
-#pragma unroll 4
-    for (int j = 0; j < taps; ++j) {
-        const int back = taps - 1 - j;
-        float in = 0.0f;
-        if (back <= i) in = proj[(size_t)(t - back) * ldp + col];
-        else if (pos >= back) in = ring[(size_t)((pos - back) % taps) * C + rc];
-        s = fmaf(w[(size_t)j * ldw], in, s);
+    for (int j0 = 0; j0 < taps; j0 += 4) {      // four taps' loads in flight, none behind a branch
+        float in[4], wj[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int j = min(j0 + k, taps - 1), back = taps - 1 - j;
+            const float* src = back <= i ? proj + (size_t)(t - back) * ldp + col : ring + (size_t)(max(pos - back, 0) % taps) * C + rc;
+            in[k] = *src;
+            wj[k] = w[(size_t)j * ldw];
+            if (j0 + k >= taps || pos < back) in[k] = 0.0f;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) s = fmaf(wj[k], in[k], s);
     }
     return s;
 }
@@ -620,26 +625,105 @@ struct DeltaDecode {
     int ldm;
 };
 
-// rows r0 .. of a bf16 matrix (padded with zeros to whole sixteens of eight) times x in shared memory; sixteen lanes a row
+// out[r] = rows r < n of a bf16 matrix (padded with zeros) times x in shared memory (zero up to a multiple of 128); sixteen
+// lanes a row, eight rows of a half-warp in flight
 __device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ldw, int n, const float* x, int rank, float* out) {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 15;
-#pragma unroll 4
-    for (int r = 2 * warp + (lane >> 4); r < ((n + 1) & ~1); r += 2 * (blockDim.x >> 5)) {
-        float a = 0.0f;
-        if (r < n)
-            for (int k = 8 * sub; k < rank; k += 128) {
-                const uint4 v = *reinterpret_cast<const uint4*>(w + (size_t)r * ldw + k);
-                const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+    constexpr int AHEAD = 8;
+    const int lane = threadIdx.x & 31, sub = lane & 15, half = 2 * (threadIdx.x >> 5) + (lane >> 4), halves = blockDim.x >> 4;
+    for (int rb = 0; rb < n; rb += AHEAD * halves) {
+        float a[AHEAD] = {};
+        for (int k = 8 * sub; k < rank; k += 128) {
+            float xr[8];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    a = fmaf(__uint_as_float(u[i] << 16), x[k + 2 * i], a);
-                    a = fmaf(__uint_as_float(u[i] & 0xffff0000u), x[k + 2 * i + 1], a);
-                }
+            for (int i = 0; i < 8; ++i) xr[i] = x[k + i];
+            uint4 v[AHEAD];
+#pragma unroll
+            for (int j = 0; j < AHEAD; ++j) {
+                const int r = rb + j * halves + half;
+                v[j] = r < n && k < ldw ? *reinterpret_cast<const uint4*>(w + (size_t)r * ldw + k) : make_uint4(0, 0, 0, 0);
             }
 #pragma unroll
-        for (int o = 8; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-        if (sub == 0 && r < n) out[r] = a;
+            for (int j = 0; j < AHEAD; ++j) {
+                const uint32_t u[4] = {v[j].x, v[j].y, v[j].z, v[j].w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    a[j] = fmaf(__uint_as_float(u[i] << 16), xr[2 * i], a[j]);
+                    a[j] = fmaf(__uint_as_float(u[i] & 0xffff0000u), xr[2 * i + 1], a[j]);
+                }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) a[j] += __shfl_xor_sync(0xffffffffu, a[j], o);
+            const int r = rb + j * halves + half;
+            if (sub == 0 && r < n) out[r] = a[j];
+        }
     }
+}
+
+// NC columns of a head's state, lane's channels Chan<EPL>::at
+template <int NC, int EPL>
+__device__ __forceinline__ void load_columns(const float* S, int c0, int vdim, int dim, int lane, bool fresh, float (&s)[NC][EPL]) {
+    const bool vec = (dim & 3) == 0 && EPL >= 4;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        const float* col = S + (size_t)min(c0 + c, vdim - 1) * dim;
+        const bool ok = !fresh && c0 + c < vdim;
+        if (vec) {
+#pragma unroll
+            for (int j = 0; j < EPL / 4; ++j) {
+                const int d = Chan<EPL>::at(lane, 4 * j);
+                const float4 v = ok && d < dim ? *reinterpret_cast<const float4*>(col + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                s[c][(4 * j) % EPL] = v.x, s[c][(4 * j + 1) % EPL] = v.y, s[c][(4 * j + 2) % EPL] = v.z, s[c][(4 * j + 3) % EPL] = v.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const int d = Chan<EPL>::at(lane, i);
+                s[c][i] = ok && d < dim ? col[d] : 0.0f;
+            }
+        }
+    }
+}
+template <int NC, int EPL>
+__device__ __forceinline__ void store_columns(float* S, int c0, int vdim, int dim, int lane, const float (&s)[NC][EPL]) {
+    const bool vec = (dim & 3) == 0 && EPL >= 4;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        if (c0 + c >= vdim) continue;
+        float* col = S + (size_t)(c0 + c) * dim;
+        if (vec) {
+#pragma unroll
+            for (int j = 0; j < EPL / 4; ++j) {
+                const int d = Chan<EPL>::at(lane, 4 * j);
+                if (d < dim)
+                    *reinterpret_cast<float4*>(col + d) =
+                        make_float4(s[c][(4 * j) % EPL], s[c][(4 * j + 1) % EPL], s[c][(4 * j + 2) % EPL], s[c][(4 * j + 3) % EPL]);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                const int d = Chan<EPL>::at(lane, i);
+                if (d < dim) col[d] = s[c][i];
+            }
+        }
+    }
+}
+// Sums of v[0 .. 7] over the warp; lane l gets the sum of v[l / 4].
+__device__ __forceinline__ float transpose_sum8(float (&v)[8], int lane) {
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (i < o) {
+                const bool up = lane & (4 * o);
+                const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+                v[i] = keep + __shfl_xor_sync(0xffffffffu, send, 4 * o);
+            }
+    }
+    v[0] += __shfl_xor_sync(0xffffffffu, v[0], 2);
+    return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
 }
 
 // One CTA per (head, sequence): convolutions, unit vectors, decays and gates, the state's step, the gated norm.
@@ -649,7 +733,7 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[33], s_iq, s_ik;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, t = blockIdx.y, kh = h / p.per;
-    const int ra = (p.a_rank + 7) & ~7, rg = (p.g_rank + 7) & ~7;
+    const int ra = (p.a_rank + 127) & ~127, rg = (p.g_rank + 127) & ~127;
     float *sq = sm, *sk = sq + DP, *sg = sk + DP, *sa = sg + DP, *sgl = sa + ra, *sv = sgl + rg, *so = sv + p.vdim, *sgate = so + p.vdim;
     pdl_launch_dependents();
     // the gates' weights do not depend on the kernel before: on their way to L2 while this one still waits
@@ -669,9 +753,13 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
         float v = 0.0f;
         if (c >= 2 * DP || d < p.dim) {
             v = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, col, taps, p.conv + col, p.cr.ldw, col, t, 0, pos));
-            if (c >= 2 * DP || first) ring[(size_t)(pos % taps) * p.cr.C + col] = row[col];    // a row no tap of this token reads
         }
         sm[c < 2 * DP ? c : (int)(sv - sm) + d] = v;
+    }
+    // the token's own inputs into the ring: a row that none of its taps reads
+    for (int c = tid; c < 2 * p.dim + p.vdim; c += 256) {
+        const int col = c < p.dim ? p.off_q + kh * p.dim + c : c < 2 * p.dim ? p.off_k + kh * p.dim + c - p.dim : p.off_v + h * p.vdim + c - 2 * p.dim;
+        if (c >= 2 * p.dim || first) ring[(size_t)(pos % taps) * p.cr.C + col] = row[col];
     }
     for (int c = tid; c < ra; c += 256) sa[c] = c < p.a_rank ? row[p.off_a + c] : 0.0f;
     for (int c = tid; c < rg; c += 256) sgl[c] = c < p.g_rank ? row[p.off_g + c] : 0.0f;
@@ -682,8 +770,8 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
         ss = warp_sum(ss);
         if (lane == 0) (warp ? s_ik : s_iq) = (warp ? 1.0f : p.q_scale) / sqrtf(ss + p.unit_eps);
     }
-    low_rank_rows(p.a2 + (size_t)h * p.dim * p.lda2, p.lda2, p.dim, sa, ra, sg);
-    low_rank_rows(p.g2 + (size_t)h * p.vdim * p.ldg2, p.ldg2, p.vdim, sgl, rg, sgate);
+    low_rank_rows(p.a2 + (size_t)h * p.dim * p.lda2, p.lda2, p.dim, sa, p.a_rank, sg);
+    low_rank_rows(p.g2 + (size_t)h * p.vdim * p.ldg2, p.ldg2, p.vdim, sgl, p.g_rank, sgate);
     __syncthreads();
     for (int d = tid; d < DP; d += 256) {
         sg[d] = d < p.dim ? expf(p.neg_a[h] * softplus(sg[d] + p.dt_bias[(size_t)h * p.dim + d])) : 0.0f;
@@ -701,38 +789,29 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
     const float beta = sigmoid(row[p.off_b + h]);
     for (int c0 = NC * warp; c0 < p.vdim; c0 += 8 * NC) {
         float s[NC][EPL], a[NC], b[NC];
+        load_columns<NC, EPL>(S, c0, p.vdim, p.dim, lane, pos == 0, s);
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
             a[c] = b[c] = 0.0f;
 #pragma unroll
             for (int i = 0; i < EPL; ++i) {
-                const int d = Chan<EPL>::at(lane, i);
-                s[c][i] = pos > 0 && c0 + c < p.vdim && d < p.dim ? S[(size_t)(c0 + c) * p.dim + d] * gr[i] : 0.0f;
-            }
-        }
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-#pragma unroll
-            for (int i = 0; i < EPL; ++i) {
+                s[c][i] *= gr[i];
                 a[c] = fmaf(s[c][i], kr[i], a[c]);
                 b[c] = fmaf(s[c][i], qr[i], b[c]);
             }
+        }
+        // lane l works for column l / 4
+        const float ka = transpose_sum8(a, lane), qb = transpose_sum8(b, lane);
+        const int mine = c0 + (lane >> 2);
+        const float u = mine < p.vdim ? beta * (sv[mine] - ka) : 0.0f;
+        if ((lane & 3) == 0 && mine < p.vdim) so[mine] = fmaf(kq, u, qb);
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-            a[c] = warp_sum(a[c]);
-            b[c] = warp_sum(b[c]);
-        }
+            const float uc = __shfl_sync(0xffffffffu, u, 4 * c);
 #pragma unroll
-        for (int c = 0; c < NC; ++c) {
-            if (c0 + c >= p.vdim) continue;
-            const float u = beta * (sv[c0 + c] - a[c]);
-            if (lane == 0) so[c0 + c] = fmaf(kq, u, b[c]);
-#pragma unroll
-            for (int i = 0; i < EPL; ++i) {
-                const int d = Chan<EPL>::at(lane, i);
-                if (d < p.dim) S[(size_t)(c0 + c) * p.dim + d] = fmaf(kr[i], u, s[c][i]);
-            }
+            for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(kr[i], uc, s[c][i]);
         }
+        store_columns<NC, EPL>(S, c0, p.vdim, p.dim, lane, s);
     }
     __syncthreads();
     float ss = 0.0f;
@@ -778,9 +857,13 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
         float v = 0.0f;
         if (c >= 2 * DP || d < p.state) {
             v = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, ch, taps, p.conv + ch, p.cr.ldw, p.off_x + ch, t, 0, pos) + p.conv_b[ch]);
-            if (c >= 2 * DP || first) ring[(size_t)(pos % taps) * p.cr.C + ch] = row[p.off_x + ch];
         }
         sm[c] = v;
+    }
+    // the token's own inputs into the ring: a row that none of its taps reads
+    for (int c = tid; c < 2 * p.state + p.vdim; c += 128) {
+        const int ch = c < p.state ? inner + g * p.state + c : c < 2 * p.state ? inner + GN + g * p.state + c - p.state : h * p.vdim + c - 2 * p.state;
+        if (c >= 2 * p.state || first) ring[(size_t)(pos % taps) * p.cr.C + ch] = row[p.off_x + ch];
     }
     const float dt = softplus(row[p.off_dt + h] + p.dt_bias[h]), decay = expf(p.neg_a[h] * dt), Dh = p.D[h];
     __syncthreads();
@@ -789,13 +872,7 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
     Chan<EPL>::load(sm + DP, lane, cr);
     for (int c0 = NC * warp; c0 < p.vdim; c0 += 4 * NC) {
         float s[NC][EPL], a[NC];
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-#pragma unroll
-            for (int i = 0; i < EPL; ++i) {
-                const int d = Chan<EPL>::at(lane, i);
-                s[c][i] = pos > 0 && c0 + c < p.vdim && d < p.state ? S[(size_t)(c0 + c) * p.state + d] : 0.0f;
-            }
+        load_columns<NC, EPL>(S, c0, p.vdim, p.state, lane, pos == 0, s);
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
             const float u = c0 + c < p.vdim ? dt * sx[c0 + c] : 0.0f;
@@ -804,16 +881,13 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
             for (int i = 0; i < EPL; ++i) {
                 s[c][i] = fmaf(s[c][i], decay, br[i] * u);
                 a[c] = fmaf(s[c][i], cr[i], a[c]);
-                const int d = Chan<EPL>::at(lane, i);
-                if (c0 + c < p.vdim && d < p.state) S[(size_t)(c0 + c) * p.state + d] = s[c][i];
             }
         }
-#pragma unroll
-        for (int c = 0; c < NC; ++c) a[c] = warp_sum(a[c]);
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-            if (lane == c && c0 + c < p.vdim)
-                p.y[(size_t)t * p.ldy + (size_t)h * p.vdim + c0 + c] = fmaf(Dh, sx[c0 + c], a[c]) * silu(row[p.off_z + (size_t)h * p.vdim + c0 + c]);
+        store_columns<NC, EPL>(S, c0, p.vdim, p.state, lane, s);
+        const float sum = transpose_sum8(a, lane);
+        const int mine = c0 + (lane >> 2);
+        if ((lane & 3) == 0 && mine < p.vdim)
+            p.y[(size_t)t * p.ldy + (size_t)h * p.vdim + mine] = fmaf(Dh, sx[mine], sum) * silu(row[p.off_z + (size_t)h * p.vdim + mine]);
     }
 }
 
@@ -981,7 +1055,7 @@ int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& 
                      sr.state_off, mix, mixb, ldm};
     p.cr.ldw = m.off_v + dc_pad8(V);
     const int dp = key_pad(m.dim);
-    const size_t smem = (size_t)(3 * dp + dc_pad8(m.a_rank) + dc_pad8(m.g_rank) + 3 * m.vdim) * 4;
+    const size_t smem = (size_t)(3 * dp + ((m.a_rank + 127) & ~127) + ((m.g_rank + 127) & ~127) + 3 * m.vdim) * 4;
     const dim3 grid(m.heads, st.T), block(256);
     if (smem > 48 * 1024) return dc_fail(ctx, DC_B200_UNSUPPORTED, "delta rule: gate ranks %d and %d are too large", m.a_rank, m.g_rank);
     if (dp == 32) return dc_launch(ctx, "k_delta_decode", k_delta_decode<1>, grid, block, smem, p);

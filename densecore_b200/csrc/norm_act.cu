@@ -7,22 +7,47 @@
 
 namespace {
 
+// Rows are padded with zeros to ld (a multiple of eight); so are y's rows and the weight's allocation.  KEEP: groups of
+// four values that a thread holds.
+template <int KEEP>
 __global__ void __launch_bounds__(256) k_post_norm(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, int H,
                                                    int ld, float eps, __nv_bfloat16* __restrict__ xb) {
     __shared__ float red[33];
     dc::pdl_launch_dependents();
+    const int n4 = ld / 4;
+    float4 wv[KEEP], xv[KEEP], yv[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        wv[j] = i < n4 ? reinterpret_cast<const float4*>(w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     dc::pdl_wait();
     const size_t off = (size_t)blockIdx.x * ld;
+    const float4 *y4 = reinterpret_cast<const float4*>(y + off), *x4 = reinterpret_cast<const float4*>(x + off);
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < H; i += 256) {
-        const float v = y[off + i];
-        ss = fmaf(v, v, ss);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        yv[j] = i < n4 ? y4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        xv[j] = i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) ss += (yv[j].x * yv[j].x + yv[j].y * yv[j].y) + (yv[j].z * yv[j].z + yv[j].w * yv[j].w);
     const float inv = 1.0f / sqrtf(dc::block_sum(ss, red) / (float)H + eps);
-    for (int i = threadIdx.x; i < H; i += 256) {
-        const float v = x[off + i] + y[off + i] * inv * w[i];
-        x[off + i] = v;
-        if (xb) xb[off + i] = __float2bfloat16_rn(v);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        if (i >= n4) continue;
+        float4 r;
+        r.x = fmaf(yv[j].x * inv, wv[j].x, xv[j].x);
+        r.y = fmaf(yv[j].y * inv, wv[j].y, xv[j].y);
+        r.z = fmaf(yv[j].z * inv, wv[j].z, xv[j].z);
+        r.w = fmaf(yv[j].w * inv, wv[j].w, xv[j].w);
+        reinterpret_cast<float4*>(x + off)[i] = r;
+        if (xb) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+            reinterpret_cast<uint2*>(xb + off)[i] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
     }
 }
 
@@ -47,7 +72,12 @@ __global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, 
 }  // namespace
 
 int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, int T, int H, int ld, float eps, __nv_bfloat16* xb) {
-    return dc_launch(ctx, "k_post_norm", k_post_norm, dim3(T), dim3(256), 0, x, y, w, H, ld, eps, xb);
+    const dim3 grid(T), block(256);
+    if (ld <= 1024) return dc_launch(ctx, "k_post_norm", k_post_norm<1>, grid, block, 0, x, y, w, H, ld, eps, xb);
+    if (ld <= 2048) return dc_launch(ctx, "k_post_norm", k_post_norm<2>, grid, block, 0, x, y, w, H, ld, eps, xb);
+    if (ld <= 4096) return dc_launch(ctx, "k_post_norm", k_post_norm<4>, grid, block, 0, x, y, w, H, ld, eps, xb);
+    if (ld <= 8192) return dc_launch(ctx, "k_post_norm", k_post_norm<8>, grid, block, 0, x, y, w, H, ld, eps, xb);
+    return dc_fail(ctx, DC_B200_UNSUPPORTED, "post_norm: width %d is too large", H);
 }
 
 int dc_launch_norm_rows(dc_ctx* ctx, const float* x, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps,

@@ -257,7 +257,7 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         return dc_fail(m->ctx, DC_B200_UNSUPPORTED, "config: architecture '%s' is not registered", arch ? arch->str.c_str() : "(none)");
     s->cfg.arch = a->name;
     s->cfg.vocab = r.size(cj, "vocab", "config", 2);
-    s->cfg.width = r.size(cj, "width", "config");
+    s->cfg.width = r.size(cj, "width", "config", 1, 8192);
     const dc_json* norm = cj.get("norm");
     if (norm && norm->kind == dc_json::OBJ) s->cfg.eps = (float)r.number(*norm, "eps", "config.norm");
     else r.bad("config: 'norm' is missing");
