@@ -360,6 +360,13 @@ __device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
     return *reinterpret_cast<const uint32_t*>(&h);
 }
 
+// 2^x (the hardware's approximation, relative error about 2^-22)
+__device__ __forceinline__ float ex2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+
 struct PromptParams {
     const float* proj;
     int ldp, off_q, dim, rot, dim_p, vdim, vdim_p, uv_row, window;
@@ -373,21 +380,24 @@ struct PromptParams {
     int ldm;
 };
 
-constexpr int PQ = DC_LATENT_QTILE, PK = 64;
+constexpr int PK = 64;           // keys per tile
 
-// One CTA per (64 queries of one entry, head).  VD: value columns, padded.
-template <int VD>
-__global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
-    constexpr int LDV = VD + 8;
+// One CTA per (PQ queries of one entry, head), sixteen queries a warp; key and value tiles in a ring of ST stages.
+// VD: value columns, padded.
+template <int VD, int PQ, int ST>
+__global__ void __launch_bounds__(2 * PQ) k_latent_prompt(const PromptParams p) {
+    constexpr int LDV = VD + 8, NT = 2 * PQ;
     extern __shared__ __align__(16) uint8_t smem[];
     const int ldk = p.dq + 8;
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);     // [PQ][ldk]
-    __nv_bfloat16* sK = sQ + PQ * ldk;                              // [2][PK][ldk]
-    __nv_bfloat16* sV = sK + 2 * PK * ldk;                          // [2][PK][LDV]
+    __nv_bfloat16* sK = sQ + PQ * ldk;                              // [ST][PK][ldk]
+    __nv_bfloat16* sV = sK + ST * PK * ldk;                         // [ST][PK][LDV]
     pdl_launch_dependents();
     pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, head = blockIdx.y;
-    const int e = p.tiles[2 * blockIdx.x], q0 = p.tiles[2 * blockIdx.x + 1];
+    const int tile0 = (int)(gridDim.x - 1 - blockIdx.x);           // later queries see more keys: they start first
+    const int e = p.tiles[2 * tile0], q0 = p.tiles[2 * tile0 + 1];
+    if (q0 % PQ) return;                                            // tiles are listed per DC_LATENT_QTILE queries
     const int t0 = p.starts[e], n = p.starts[e + 1] - t0, pos0 = p.positions[t0];
     const int key0 = first_key(pos0, p.window);                     // position of the entry's first gathered key
     const int first = first_key(pos0 + q0, p.window), last = pos0 + min(q0 + PQ, n) - 1;
@@ -400,8 +410,8 @@ __global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
     const int lrow = tid >> 3, lc = tid & 7;
     auto load = [&](int tile, int buf) {
 #pragma unroll
-        for (int i = 0; i < PK / 16; ++i) {
-            const int key = lrow + 16 * i, pos = first + tile * PK + key;
+        for (int i = 0; i < PK * 8 / NT; ++i) {
+            const int key = lrow + NT / 8 * i, pos = first + tile * PK + key;
             const bool ok = pos <= last;
             const __nv_bfloat16* krow = ok ? kv + (ptrdiff_t)pos * p.ldkv : p.kv;
             const __nv_bfloat16* rrow = (ok ? kr + (ptrdiff_t)pos * p.ldr : p.kr) - kc * 8;
@@ -420,16 +430,21 @@ __global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
         }
         cp_async_commit();
     };
-    load(0, 0);
-    for (int i = tid; i < PQ * p.dq; i += 128) {
-        const int r = i / p.dq, c = i - r * p.dq;
-        float v = 0.0f;
-        if (q0 + r < n) {
-            const float* q = p.proj + (size_t)(t0 + q0 + r) * p.ldp + p.off_q + head * (p.dim + p.rot);
-            if (c < p.dim) v = q[c];
-            else if (c >= p.dim_p && c < p.dim_p + p.rot) v = q[p.dim + c - p.dim_p];
+#pragma unroll
+    for (int i = 0; i < ST - 1; ++i)
+        if (i < n_tiles) load(i, i);
+        else cp_async_commit();
+    // queries: a warp takes its own sixteen rows, many loads in flight
+    {
+        const float* q0p = p.proj + (size_t)(t0 + q0) * p.ldp + p.off_q + head * (p.dim + p.rot);
+        const int dq = p.dq;
+#pragma unroll 12
+        for (int i = lane; i < 16 * dq; i += 32) {
+            const int r = i / dq, c = i - r * dq, qr = 16 * warp + r;
+            const int from = c < p.dim_p ? (c < p.dim ? c : -1) : c - p.dim_p < p.rot ? p.dim + c - p.dim_p : -1;
+            const float v = q0p[(size_t)min(qr, n - 1 - q0) * p.ldp + max(from, 0)];
+            sQ[qr * ldk + c] = __float2bfloat16_rn(q0 + qr < n && from >= 0 ? v : 0.0f);
         }
-        sQ[r * ldk + c] = __float2bfloat16_rn(v);
     }
     float o[VD / 8][4];
 #pragma unroll
@@ -441,14 +456,11 @@ __global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
     const int window = p.window > 0 ? p.window : 0x7fffffff;
 
     for (int tile = 0; tile < n_tiles; ++tile) {
-        const int buf = tile & 1, k0 = first + tile * PK;
-        if (tile + 1 < n_tiles) {
-            load(tile + 1, buf ^ 1);
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
+        const int buf = tile % ST, k0 = first + tile * PK;
+        cp_async_wait<ST - 2>();
+        __syncthreads();         // the tile has landed; every warp is done with the stage that the next load fills
+        if (tile + ST - 1 < n_tiles) load(tile + ST - 1, (tile + ST - 1) % ST);
+        else cp_async_commit();
         float s[8][4];
 #pragma unroll
         for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
@@ -466,41 +478,51 @@ __global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
                 mma_bf16(s[2 * np + 1], a, b[2], b[3]);
             }
         }
+        // the warp's sixteen queries see the whole tile, or the mask decides key by key
+        const int wq0 = pos0 + q0 + 16 * warp;
+        if (!(k0 + PK - 1 <= wq0 && wq0 + 15 - k0 < window)) {
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int kp = k0 + 8 * nt + 2 * t4 + (j & 1), qp = qpos0 + (j >> 1) * 8;
+                    if (!(kp <= qp && qp - kp < window)) s[nt][j] = -INFINITY;
+                }
+        }
         float mx[2] = {-1e30f, -1e30f};
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int kp = k0 + 8 * nt + 2 * t4 + (j & 1), qp = qpos0 + (j >> 1) * 8;
-                const float v = kp <= qp && qp - kp < window ? s[nt][j] * sl2 : -INFINITY;
-                s[nt][j] = v;
-                mx[j >> 1] = fmaxf(mx[j >> 1], v);
-            }
-        float corr[2];
+        for (int nt = 0; nt < 8; ++nt) {
+            mx[0] = fmaxf(mx[0], fmaxf(s[nt][0], s[nt][1]));
+            mx[1] = fmaxf(mx[1], fmaxf(s[nt][2], s[nt][3]));
+        }
+        float m_new[2];
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
             mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
             mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-            const float m_new = fmaxf(m_run[h], mx[h]);
-            corr[h] = exp2f(m_run[h] - m_new);
-            m_run[h] = m_new;
-            l_run[h] *= corr[h];
+            m_new[h] = fmaxf(m_run[h], mx[h] * sl2);
+        }
+        if (__any_sync(0xffffffffu, m_new[0] > m_run[0] || m_new[1] > m_run[1])) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const float corr = ex2(m_run[h] - m_new[h]);
+                m_run[h] = m_new[h];
+                l_run[h] *= corr;
+#pragma unroll
+                for (int i = 0; i < VD / 8; ++i) {
+                    o[i][2 * h] *= corr;
+                    o[i][2 * h + 1] *= corr;
+                }
+            }
         }
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const float w = exp2f(s[nt][j] - m_run[j >> 1]);
+                const float w = ex2(fmaf(s[nt][j], sl2, -m_run[j >> 1]));
                 s[nt][j] = w;
                 l_run[j >> 1] += w;
             }
-#pragma unroll
-        for (int i = 0; i < VD / 8; ++i) {
-            o[i][0] *= corr[0];
-            o[i][1] *= corr[0];
-            o[i][2] *= corr[1];
-            o[i][3] *= corr[1];
-        }
         const uint32_t va = smem_u32(sV + (buf * PK + (mi & 1) * 8 + r8) * LDV + (mi >> 1) * 8);
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks) {
@@ -517,7 +539,6 @@ __global__ void __launch_bounds__(128) k_latent_prompt(const PromptParams p) {
                 mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
             }
         }
-        __syncthreads();     // every warp is done with this buffer before the next load overwrites it
     }
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -576,12 +597,17 @@ int dc_launch_latent_prefill(dc_ctx* ctx, const dc_latent_mixer& m, const dc_ste
                              int ldr, __nv_bfloat16* mixb, int ldm) {
     PromptParams p = {proj, ldp, m.off_q, m.dim, m.rot_dim, m.dim_p, m.vdim, m.vdim_p, m.uv_row, m.window, m.scale, st.positions, st.starts,
                       key_base, tiles, keys_kv, ldkv, keys_r, ldr, (m.dim_p + ldr + 15) & ~15, mixb, ldm};
-    const dim3 grid(n_tiles, m.heads), block(128);
+    const dim3 grid(n_tiles, m.heads);
+    // 128 queries per CTA and three stages where they fit shared memory
 #define DC_PROMPT(VD)                                                                                                       \
     do {                                                                                                                    \
-        const size_t smem = ((size_t)(PQ + 2 * PK) * (p.dq + 8) + (size_t)2 * PK * (VD + 8)) * 2;                           \
-        DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_prompt<VD>, (int)smem, "k_latent_prompt"));                       \
-        return dc_launch(ctx, "k_latent_prompt", k_latent_prompt<VD>, grid, block, smem, p);                                \
+        auto bytes = [&](int pq, int st) { return ((size_t)(pq + st * PK) * (p.dq + 8) + (size_t)st * PK * (VD + 8)) * 2; }; \
+        if (bytes(128, 3) <= 227 * 1024) {                                                                                  \
+            DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_prompt<VD, 128, 3>, (int)bytes(128, 3), "k_latent_prompt"));  \
+            return dc_launch(ctx, "k_latent_prompt", k_latent_prompt<VD, 128, 3>, grid, dim3(256), bytes(128, 3), p);       \
+        }                                                                                                                   \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_prompt<VD, 64, 2>, (int)bytes(64, 2), "k_latent_prompt"));        \
+        return dc_launch(ctx, "k_latent_prompt", k_latent_prompt<VD, 64, 2>, grid, dim3(128), bytes(64, 2), p);             \
     } while (0)
     if (m.vdim <= 32) DC_PROMPT(32);
     if (m.vdim <= 64) DC_PROMPT(64);

@@ -8,7 +8,7 @@
 // Value columns of S never mix: a column c obeys S_c <- g S_c; u = beta (v_c - S_c . k); S_c <- S_c + u k;
 // o_c = S_c . q.  A single token (decode) is done as written, by one kernel per mixer from projections to normed
 // output.  Longer entries go through blocks of sixteen tokens (see "blocks of sixteen tokens" below): what a head's
-// columns share is computed once per block, and k_state_scan walks the blocks with four columns in the registers of
+// columns share is computed once per block, and k_state_scan walks the blocks with two columns in the registers of
 // each warp.  All of it is f32 on the CUDA cores.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
@@ -65,6 +65,25 @@ struct ConvRef {
     int E, taps, C, ldw;     // C: channels of a ring row; ldw: pitch of the convolution weights [taps][ldw]
     __device__ float* ring(int seq) const { return reinterpret_cast<float*>(base + (size_t)seq * slot_bytes + ring_off); }
 };
+
+constexpr int BT = 16, BROW = 20;                       // tokens of a block; pitch of a 16 x 16 factor (conflict-free rows)
+
+struct BlockRef {                                       // token range of a block: entries are cut from their own start
+    int e, t0, n;
+};
+__device__ __forceinline__ int block_base(const int32_t* starts, int e) {
+    int b = 0;
+    for (int i = 0; i < e; ++i) b += (starts[i + 1] - starts[i] + BT - 1) / BT;
+    return b;
+}
+__device__ __forceinline__ BlockRef block_at(const int32_t* starts, int E, int blk) {
+    for (int e = 0; e < E; ++e) {
+        const int n = starts[e + 1] - starts[e], nb = (n + BT - 1) / BT;
+        if (blk < nb) return BlockRef{e, starts[e] + blk * BT, min(BT, n - blk * BT)};
+        blk -= nb;
+    }
+    return BlockRef{0, 0, 0};
+}
 
 // The entries' last inputs into their rings (after every kernel that read the old ones).
 __global__ void __launch_bounds__(256) k_ring_update(ConvRef cr, const float* __restrict__ proj, int ldp, int off) {
@@ -148,6 +167,106 @@ __global__ void __launch_bounds__(256) k_delta_prep(DeltaPrep p) {
     }
 }
 
+// Four taps: a warp takes an item through a block of up to sixteen tokens with the convolution's window in registers.
+// NJ: groups of 32 key channels.
+template <int NJ>
+__global__ void __launch_bounds__(256) k_delta_prep4(DeltaPrep p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, items = p.kv_heads + p.v_items, item = blockIdx.y * 8 + (threadIdx.x >> 5);
+    const BlockRef br = block_at(p.cr.starts, p.cr.E, blockIdx.x);
+    if (br.n <= 0) return;
+    if (blockIdx.y == gridDim.y - 1) {          // the step sizes and the low-rank columns
+        for (int i = threadIdx.x; i < br.n * p.heads; i += 256) {
+            const int t = br.t0 + i / p.heads, h = i % p.heads;
+            p.small[(size_t)t * p.heads + h] = sigmoid(p.proj[(size_t)t * p.ldp + p.off_b + h]);
+        }
+        if (p.lowb)
+            for (int i = threadIdx.x; i < br.n * p.n_low; i += 256) {
+                const int t = br.t0 + i / p.n_low, c = i % p.n_low;
+                p.lowb[(size_t)t * p.ldl + c] = __float2bfloat16_rn(p.proj[(size_t)t * p.ldp + p.off_a + c]);
+            }
+        return;
+    }
+    if (item >= items) return;
+    const int i0 = br.t0 - p.cr.starts[br.e], pos0 = p.cr.positions[br.t0], ldw = p.cr.ldw;
+    const float* ring = p.cr.ring(p.cr.seq_ids[br.t0]);
+    auto before = [&](int col, int back) {        // the input `back` tokens before the block
+        if (pos0 < back) return 0.0f;
+        return back <= i0 ? p.proj[(size_t)(br.t0 - back) * p.ldp + col] : ring[(size_t)((pos0 - back) % 4) * p.cr.C + col];
+    };
+    if (item < p.kv_heads) {
+        float wq[NJ][4], wk[NJ][4], hq[NJ][3], hk[NJ][3];
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+            const int d = min(lane + 32 * j, p.dim - 1), cq = p.off_q + item * p.dim + d, ck = p.off_k + item * p.dim + d;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) wq[j][k] = p.conv[(size_t)k * ldw + cq], wk[j][k] = p.conv[(size_t)k * ldw + ck];
+#pragma unroll
+            for (int k = 0; k < 3; ++k) hq[j][k] = before(cq, 3 - k), hk[j][k] = before(ck, 3 - k);
+        }
+        constexpr int AHEAD = NJ <= 4 ? 4 : 2;        // tokens whose inputs are in flight
+        for (int ub = 0; ub < br.n; ub += AHEAD) {
+            float xq[AHEAD][NJ], xk[AHEAD][NJ];
+#pragma unroll
+            for (int v = 0; v < AHEAD; ++v) {
+                const float* row = p.proj + (size_t)(br.t0 + min(ub + v, br.n - 1)) * p.ldp + item * p.dim;
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    const int dc = min(lane + 32 * j, p.dim - 1);
+                    xq[v][j] = row[p.off_q + dc], xk[v][j] = row[p.off_k + dc];
+                }
+            }
+#pragma unroll
+            for (int v = 0; v < AHEAD; ++v) {
+                if (ub + v >= br.n) break;
+                float* act = p.act + (size_t)(br.t0 + ub + v) * p.lda;
+                float q[NJ], k[NJ], sq = 0.0f, sk = 0.0f;
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    q[j] = silu(fmaf(wq[j][3], xq[v][j], fmaf(wq[j][2], hq[j][2], fmaf(wq[j][1], hq[j][1], wq[j][0] * hq[j][0]))));
+                    k[j] = silu(fmaf(wk[j][3], xk[v][j], fmaf(wk[j][2], hk[j][2], fmaf(wk[j][1], hk[j][1], wk[j][0] * hk[j][0]))));
+                    hq[j][0] = hq[j][1], hq[j][1] = hq[j][2], hq[j][2] = xq[v][j];
+                    hk[j][0] = hk[j][1], hk[j][1] = hk[j][2], hk[j][2] = xk[v][j];
+                    if (lane + 32 * j >= p.dim) q[j] = k[j] = 0.0f;
+                    sq = fmaf(q[j], q[j], sq);
+                    sk = fmaf(k[j], k[j], sk);
+                }
+                const float iq = p.q_scale / sqrtf(warp_sum(sq) + p.unit_eps), ik = 1.0f / sqrtf(warp_sum(sk) + p.unit_eps);
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    const int d = lane + 32 * j;
+                    if (d < p.dim) {
+                        act[p.off_q + item * p.dim + d] = q[j] * iq;
+                        act[p.off_k + item * p.dim + d] = k[j] * ik;
+                    }
+                }
+            }
+        }
+    } else {
+        const int V = p.heads * p.vdim, c0 = (item - p.kv_heads) * 128 + lane;
+        float w[4][4], h[4][3];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int cv = p.off_v + min(c0 + 32 * j, V - 1);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) w[j][k] = p.conv[(size_t)k * ldw + cv];
+#pragma unroll
+            for (int k = 0; k < 3; ++k) h[j][k] = before(cv, 3 - k);
+        }
+#pragma unroll 4
+        for (int u = 0; u < br.n; ++u) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float x = p.proj[(size_t)(br.t0 + u) * p.ldp + p.off_v + min(c0 + 32 * j, V - 1)];
+                const float y = silu(fmaf(w[j][3], x, fmaf(w[j][2], h[j][2], fmaf(w[j][1], h[j][1], w[j][0] * h[j][0]))));
+                h[j][0] = h[j][1], h[j][1] = h[j][2], h[j][2] = x;
+                if (c0 + 32 * j < V) p.act[(size_t)(br.t0 + u) * p.lda + p.off_v + c0 + 32 * j] = y;
+            }
+        }
+    }
+}
+
 // ---------------------------------------------------------------- blocks of sixteen tokens
 // Within a block that starts from the state S0, with cumulative decays G_t (products of g over the block's tokens up
 // to t) and products P_ti of g over (i, t]:
@@ -157,24 +276,6 @@ __global__ void __launch_bounds__(256) k_delta_prep(DeltaPrep p) {
 // Everything but S0, v, u and o is shared by a head's value columns and computed once per (block, head): the decayed
 // vectors, B, and W = (I + diag(beta) A)^-1 diag(beta), so that u = W (v - S0 . G k).  Every decay factor is a
 // product of g, at most 1.  The state-space scan is the same with one decay per head, no A, and u_i = dt_i x_i.
-constexpr int BT = 16, BROW = 20;                       // tokens of a block; pitch of a 16 x 16 factor (conflict-free rows)
-
-struct BlockRef {                                       // token range of a block: entries are cut from their own start
-    int e, t0, n;
-};
-__device__ __forceinline__ int block_base(const int32_t* starts, int e) {
-    int b = 0;
-    for (int i = 0; i < e; ++i) b += (starts[i + 1] - starts[i] + BT - 1) / BT;
-    return b;
-}
-__device__ __forceinline__ BlockRef block_at(const int32_t* starts, int E, int blk) {
-    for (int e = 0; e < E; ++e) {
-        const int n = starts[e + 1] - starts[e], nb = (n + BT - 1) / BT;
-        if (blk < nb) return BlockRef{e, starts[e] + blk * BT, min(BT, n - blk * BT)};
-        blk -= nb;
-    }
-    return BlockRef{0, 0, 0};
-}
 
 // Sum of v[i] over the warp lands in lane i (31 shuffles for 32 sums).
 __device__ __forceinline__ float transpose_sum32(float (&v)[32], int lane) {
@@ -267,14 +368,14 @@ __global__ void __launch_bounds__(128) k_delta_blocks(const DeltaBlock p) {
     }
     __syncthreads();
     if (tid < BT) {                                     // column tid of (I + diag(beta) A)^-1 diag(beta)
+        float x[BT];
+#pragma unroll
         for (int t = 0; t < BT; ++t) {
-            float x = t == tid ? 1.0f : 0.0f;
-            if (t > tid) {
-                float a = 0.0f;
-                for (int i = tid; i < t; ++i) a = fmaf(sA[t][i], sX[i][tid], a);
-                x = -sbeta[t] * a;
-            }
-            sX[t][tid] = x;
+            float a[2] = {};
+#pragma unroll
+            for (int i = 0; i < t; ++i) a[i & 1] = fmaf(sA[t][i], x[i], a[i & 1]);
+            x[t] = t < tid ? 0.0f : t == tid ? 1.0f : -sbeta[t] * (a[0] + a[1]);
+            sX[t][tid] = x[t];
         }
     }
     __syncthreads();
@@ -344,7 +445,7 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
 }
 
 // ---------------------------------------------------------------- the scan over blocks
-constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp
+constexpr int SC_COLS = 16, SC_THREADS = 256;           // value columns per CTA: two per warp
 
 struct ScanParams {
     const float* blocks;           // k_delta_blocks / k_ssd_blocks
@@ -392,40 +493,29 @@ struct Chan {
     }
 };
 
-// Dot products of the warp's four columns (s: this lane's channels of each) with sixteen rows of shared memory.  Lane
-// 8 c + j gets column c's products with rows j and j + 8.
+// Dot products of the warp's two columns (s: this lane's channels of each) with sixteen rows of shared memory.  Lane
+// 16 c + t gets column c's product with row t.
 template <int EPL>
-__device__ __forceinline__ void column_dots(const float* rows, int dp, const float (&s)[4][EPL], int lane, float (&out)[2]) {
-    float r[64];
+__device__ __forceinline__ float column_dots(const float* rows, int dp, const float (&s)[2][EPL], int lane) {
+    float r[32];
 #pragma unroll
     for (int t = 0; t < BT; ++t) {
         float w[EPL];
         Chan<EPL>::load(rows + t * dp, lane, w);
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < 2; ++c) {
             if (EPL == 1) {
-                r[16 * c + 2 * (t & 7) + (t >> 3)] = s[c][0] * w[0];
+                r[16 * c + t] = s[c][0] * w[0];
             } else {
                 uint64_t a = 0;
 #pragma unroll
                 for (int i = 0; i + 1 < EPL; i += 2) a = fma2(pair(s[c][i], s[c][i + 1]), pair(w[i], w[i + 1]), a);
                 const float2 f = unpair(a);
-                r[16 * c + 2 * (t & 7) + (t >> 3)] = f.x + f.y;
+                r[16 * c + t] = f.x + f.y;
             }
         }
     }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {                           // each step halves the sums a lane carries
-        const bool up = lane & o;
-#pragma unroll
-        for (int i = 0; i < 32; ++i)
-            if (i < 2 * o) {
-                const float send = up ? r[i] : r[i + 2 * o], keep = up ? r[i + 2 * o] : r[i];
-                r[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-            }
-    }
-    out[0] = r[0];
-    out[1] = r[1];
+    return transpose_sum32(r, lane);
 }
 
 // EPL: key channels per lane (the key size, padded to 32 EPL).
@@ -433,11 +523,11 @@ template <int EPL, bool DELTA>
 __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     constexpr int DP = 32 * EPL, BLK = DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK, BUF = BLK + BT * SC_COLS;
     extern __shared__ __align__(16) float sm[];
-    __shared__ __align__(16) float s_d[4][4][BT], s_u[4][4][BT];
+    __shared__ __align__(16) float s_d[8][2][BT], s_u[8][2][BT];
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, c4 = lane >> 3;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lt = lane & 15, lc = lane >> 4;
     const int c0 = blockIdx.x * SC_COLS, h = blockIdx.y, e = blockIdx.z, kh = h / p.per;
-    const int col = c0 + warp * 4 + c4;
+    const int col = c0 + warp * 2 + lc;
     if (!DELTA) {
         for (int i = tid; i < 2 * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels stay zero
         __syncthreads();
@@ -448,15 +538,15 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     const int seq = p.seq_ids[t0], blocks = (t1 - t0 + BT - 1) / BT;
     const float* bsrc = p.blocks + ((size_t)block_base(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
     const size_t bstep = (size_t)p.heads * (DELTA ? BLK : SSD_BLOCK);
-    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 4) * p.dim;
-    float s[4][EPL];             // channels Chan::at of the warp's four columns
+    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 2) * p.dim;
+    float s[2][EPL];             // channels Chan::at of the warp's two columns
     const bool fresh = p.positions[t0] == 0, live = col < p.vdim;
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < 2; ++c)
 #pragma unroll
         for (int i = 0; i < EPL; ++i) {
             const int d = Chan<EPL>::at(lane, i);
-            s[c][i] = !fresh && c0 + warp * 4 + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
+            s[c][i] = !fresh && c0 + warp * 2 + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
         }
 
     auto load = [&](int b, int buf) {
@@ -498,73 +588,45 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
         __syncthreads();
         const float* x = sm + (b & 1) * BUF;
-        const float* sv = x + BLK + warp * 4 + c4;
-        // ---- the columns against the block's (decayed) keys and queries
-        float rk[2] = {}, rq[2];
-        if (DELTA) column_dots<EPL>(x, DP, s, lane, rk);
-        column_dots<EPL>(x + (DELTA ? BT * DP : 0), DP, s, lane, rq);
-        // ---- u and o: this lane's tokens l8 and l8 + 8
-        const float* scal = x + (DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
-        float v[2];
-#pragma unroll
-        for (int k = 0; k < 2; ++k) {
-            const int t = l8 + 8 * k;
-            v[k] = sv[t * SC_COLS];
-            s_d[warp][c4][t] = v[k] - rk[k];
-        }
+        // ---- the columns against the block's (decayed) keys and queries; lane 16 c + t works for column c, token t
+        float rk = 0.0f;
+        if (DELTA) rk = column_dots<EPL>(x, DP, s, lane);
+        const float rq = column_dots<EPL>(x + (DELTA ? BT * DP : 0), DP, s, lane);
+        const float v = x[BLK + lt * SC_COLS + warp * 2 + lc];
+        s_d[warp][lc][lt] = v - rk;
         __syncwarp();
-        float dv[BT];
-#pragma unroll
-        for (int i = 0; i < BT / 4; ++i) {
-            const float4 f = *reinterpret_cast<const float4*>(&s_d[warp][c4][4 * i]);
-            dv[4 * i] = f.x, dv[4 * i + 1] = f.y, dv[4 * i + 2] = f.z, dv[4 * i + 3] = f.w;
-        }
-        auto row_dot = [&](const float* row) {                   // rows of W, B, M are zero above the diagonal
-            float a[2] = {0.0f, 0.0f};
+        auto row_dot = [&](const float* row, const float* vals) {      // rows of W, B, M are zero above the diagonal
+            float a[4] = {};
 #pragma unroll
             for (int i = 0; i < BT / 4; ++i) {
-                const float4 f = *reinterpret_cast<const float4*>(row + 4 * i);
-                a[0] = fmaf(f.x, dv[4 * i], a[0]);
-                a[1] = fmaf(f.y, dv[4 * i + 1], a[1]);
-                a[0] = fmaf(f.z, dv[4 * i + 2], a[0]);
-                a[1] = fmaf(f.w, dv[4 * i + 3], a[1]);
+                const float4 f = *reinterpret_cast<const float4*>(row + 4 * i), d = *reinterpret_cast<const float4*>(vals + 4 * i);
+                a[0] = fmaf(f.x, d.x, a[0]);
+                a[1] = fmaf(f.y, d.y, a[1]);
+                a[2] = fmaf(f.z, d.z, a[2]);
+                a[3] = fmaf(f.w, d.w, a[3]);
             }
-            return a[0] + a[1];
+            return (a[0] + a[1]) + (a[2] + a[3]);
         };
-        float out[2];
+        const float* scal = x + (DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
+        float out;
         if (DELTA) {
-#pragma unroll
-            for (int k = 0; k < 2; ++k) s_u[warp][c4][l8 + 8 * k] = row_dot(scal + (l8 + 8 * k) * BROW);
+            s_u[warp][lc][lt] = row_dot(scal + lt * BROW, s_d[warp][lc]);
             __syncwarp();
-#pragma unroll
-            for (int i = 0; i < BT / 4; ++i) {
-                const float4 f = *reinterpret_cast<const float4*>(&s_u[warp][c4][4 * i]);
-                dv[4 * i] = f.x, dv[4 * i + 1] = f.y, dv[4 * i + 2] = f.z, dv[4 * i + 3] = f.w;
-            }
-#pragma unroll
-            for (int k = 0; k < 2; ++k) out[k] = rq[k] + row_dot(scal + (BT + l8 + 8 * k) * BROW);
+            out = rq + row_dot(scal + (BT + lt) * BROW, s_u[warp][lc]);
         } else {
             const float* cd = scal + BT * BROW;
-#pragma unroll
-            for (int k = 0; k < 2; ++k) {
-                const int t = l8 + 8 * k;
-                out[k] = fmaf(cd[t], rq[k], row_dot(scal + t * BROW)) + Dh * v[k];
-                s_u[warp][c4][t] = v[k] * cd[BT + t];
-            }
+            s_u[warp][lc][lt] = v * cd[BT + lt];
+            out = fmaf(cd[lt], rq, row_dot(scal + lt * BROW, s_d[warp][lc])) + Dh * v;
             __syncwarp();
         }
-#pragma unroll
-        for (int k = 0; k < 2; ++k) {
-            const int t = t0 + b * BT + l8 + 8 * k;
-            if (t < t1 && live) p.o[(size_t)t * p.ldo + (size_t)h * p.vdim + col] = out[k];
-        }
+        if (t0 + b * BT + lt < t1 && live) p.o[(size_t)(t0 + b * BT + lt) * p.ldo + (size_t)h * p.vdim + col] = out;
         // ---- the state after the block
         const float* keys = x + (DELTA ? 2 * BT * DP : BT * DP);
         {
             float g[EPL];
             if (DELTA) Chan<EPL>::load(x + 3 * BT * DP, lane, g);
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
+            for (int c = 0; c < 2; ++c)
 #pragma unroll
                 for (int i = 0; i < EPL; ++i) s[c][i] *= DELTA ? g[i] : scal[BT * BROW + BT - 1];
         }
@@ -573,7 +635,7 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             float w[EPL];
             Chan<EPL>::load(keys + t * DP, lane, w);
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
+            for (int c = 0; c < 2; ++c) {
                 const float u = s_u[warp][c][t];
 #pragma unroll
                 for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(w[i], u, s[c][i]);
@@ -582,11 +644,11 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         __syncthreads();
     }
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < 2; ++c)
 #pragma unroll
         for (int i = 0; i < EPL; ++i) {
             const int d = Chan<EPL>::at(lane, i);
-            if (c0 + warp * 4 + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
+            if (c0 + warp * 2 + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
         }
 }
 
@@ -969,6 +1031,44 @@ __global__ void __launch_bounds__(256) k_ssd_prep(SsdPrep p) {
         }
 }
 
+// Four taps: a thread takes its channel through a block of up to sixteen tokens with the window in registers.
+__global__ void __launch_bounds__(256) k_ssd_prep4(SsdPrep p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = blockIdx.y * 256 + threadIdx.x;
+    const BlockRef br = block_at(p.cr.starts, p.cr.E, blockIdx.x);
+    if (br.n <= 0) return;
+    if (c < p.cr.C) {
+        const int i0 = br.t0 - p.cr.starts[br.e], pos0 = p.cr.positions[br.t0];
+        const float* ring = p.cr.ring(p.cr.seq_ids[br.t0]);
+        const float* in = p.proj + (size_t)br.t0 * p.ldp + p.off_x + c;
+        float w[4], h[3], x[BT];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) w[k] = p.conv[(size_t)k * p.cr.ldw + c];
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            const int back = 3 - k;
+            h[k] = pos0 < back ? 0.0f : back <= i0 ? in[-(ptrdiff_t)back * p.ldp] : ring[(size_t)((pos0 - back) % 4) * p.cr.C + c];
+        }
+#pragma unroll
+        for (int u = 0; u < BT; ++u) x[u] = u < br.n ? in[(size_t)u * p.ldp] : 0.0f;
+        const float bias = p.conv_b[c];
+#pragma unroll
+        for (int u = 0; u < BT; ++u) {
+            const float y = silu(fmaf(w[3], x[u], fmaf(w[2], h[2], fmaf(w[1], h[1], w[0] * h[0]))) + bias);
+            h[0] = h[1], h[1] = h[2], h[2] = x[u];
+            if (u < br.n) p.act[(size_t)(br.t0 + u) * p.lda + c] = y;
+        }
+    }
+    if (blockIdx.y == 0)
+        for (int i = threadIdx.x; i < br.n * p.heads; i += 256) {
+            const int t = br.t0 + i / p.heads, h = i % p.heads;
+            const float dt = softplus(p.proj[(size_t)t * p.ldp + p.off_dt + h] + p.dt_bias[h]);
+            p.small[(size_t)t * 2 * p.heads + h] = dt;
+            p.small[(size_t)t * 2 * p.heads + p.heads + h] = expf(p.neg_a[h] * dt);
+        }
+}
+
 ConvRef conv_ref(const dc_step& st, const dc_state_ref& sr, int taps, int C) {
     return ConvRef{sr.base, sr.slot_bytes, sr.ring_off, st.seq_ids, st.positions, st.starts, st.E, taps, C, C};
 }
@@ -995,8 +1095,18 @@ int dc_launch_delta_prep(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st
     p.n_low = m.off_g + m.g_rank - m.off_a;
     p.unit_eps = m.unit_eps, p.q_scale = m.q_scale;
     p.act = act, p.lda = lda, p.small = small, p.lowb = lowb, p.ldl = ldl, p.T = st.T, p.v_items = (V + 127) / 128;
-    const long long warps = (long long)st.T * (m.kv_heads + p.v_items + 1);
-    DC_TRY(dc_launch(ctx, "k_delta_prep", k_delta_prep, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, p));
+    const int items = m.kv_heads + p.v_items + 1;
+    if (m.taps == 4) {
+        const dim3 grid(dc_scan_blocks(st.T, st.E), (items - 1 + 7) / 8 + 1);
+        switch (key_pad(m.dim)) {
+        case 32: DC_TRY(dc_launch(ctx, "k_delta_prep4", k_delta_prep4<1>, grid, dim3(256), 0, p)); break;
+        case 64: DC_TRY(dc_launch(ctx, "k_delta_prep4", k_delta_prep4<2>, grid, dim3(256), 0, p)); break;
+        case 128: DC_TRY(dc_launch(ctx, "k_delta_prep4", k_delta_prep4<4>, grid, dim3(256), 0, p)); break;
+        default: DC_TRY(dc_launch(ctx, "k_delta_prep4", k_delta_prep4<8>, grid, dim3(256), 0, p));
+        }
+    } else {
+        DC_TRY(dc_launch(ctx, "k_delta_prep", k_delta_prep, dim3((unsigned)(((long long)st.T * items + 7) / 8)), dim3(256), 0, p));
+    }
     return dc_launch_ring_update(ctx, st, sr, proj, ldp, 0, C, m.taps);
 }
 
@@ -1027,7 +1137,8 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
                   int lda, float* small, float* blk, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
     const int inner = m.heads * m.vdim, GN = m.groups * m.state, C = inner + 2 * GN;
     SsdPrep s = {conv_ref(st, sr, m.taps, C), proj, ldp, m.off_x, m.off_dt, m.heads, st.T, m.conv, m.conv_b, m.dt_bias, m.neg_a, act, lda, small};
-    DC_TRY(dc_launch(ctx, "k_ssd_prep", k_ssd_prep, dim3((C + 255) / 256, st.T), dim3(256), 0, s));
+    if (m.taps == 4) DC_TRY(dc_launch(ctx, "k_ssd_prep4", k_ssd_prep4, dim3(dc_scan_blocks(st.T, st.E), (C + 255) / 256), dim3(256), 0, s));
+    else DC_TRY(dc_launch(ctx, "k_ssd_prep", k_ssd_prep, dim3((C + 255) / 256, st.T), dim3(256), 0, s));
     DC_TRY(dc_launch_ring_update(ctx, st, sr, proj, ldp, m.off_x, C, m.taps));
     SsdBlock sb = {act, lda, inner, inner + GN, m.heads, m.heads / m.groups, m.state, small, st.starts, st.E, blk};
     DC_TRY(dc_launch(ctx, "k_ssd_blocks", k_ssd_blocks, dim3(dc_scan_blocks(st.T, st.E), m.groups), dim3(256), (size_t)2 * BT * (m.state + 1) * 4, sb));
