@@ -8,7 +8,7 @@
 // Value columns of S never mix: a column c obeys S_c <- g S_c; u = beta (v_c - S_c . k); S_c <- S_c + u k;
 // o_c = S_c . q.  A single token (decode) is done as written, by one kernel per mixer from projections to normed
 // output.  Longer entries go through blocks of sixteen tokens (see "blocks of sixteen tokens" below): what a head's
-// columns share is computed once per block, and k_state_scan walks the blocks with two columns in the registers of
+// columns share is computed once per block, and k_state_scan walks the blocks with four columns in the registers of
 // each warp.  All of it is f32 on the CUDA cores.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
@@ -254,15 +254,20 @@ __global__ void __launch_bounds__(256) k_delta_prep4(DeltaPrep p) {
 #pragma unroll
             for (int k = 0; k < 3; ++k) h[j][k] = before(cv, 3 - k);
         }
-#pragma unroll 4
-        for (int u = 0; u < br.n; ++u) {
+        for (int ub = 0; ub < br.n; ub += 8) {
+            float x[8][4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const float x = p.proj[(size_t)(br.t0 + u) * p.ldp + p.off_v + min(c0 + 32 * j, V - 1)];
-                const float y = silu(fmaf(w[j][3], x, fmaf(w[j][2], h[j][2], fmaf(w[j][1], h[j][1], w[j][0] * h[j][0]))));
-                h[j][0] = h[j][1], h[j][1] = h[j][2], h[j][2] = x;
-                if (c0 + 32 * j < V) p.act[(size_t)(br.t0 + u) * p.lda + p.off_v + c0 + 32 * j] = y;
-            }
+            for (int v = 0; v < 8; ++v)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) x[v][j] = p.proj[(size_t)(br.t0 + min(ub + v, br.n - 1)) * p.ldp + p.off_v + min(c0 + 32 * j, V - 1)];
+#pragma unroll
+            for (int v = 0; v < 8; ++v)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float y = silu(fmaf(w[j][3], x[v][j], fmaf(w[j][2], h[j][2], fmaf(w[j][1], h[j][1], w[j][0] * h[j][0]))));
+                    h[j][0] = h[j][1], h[j][1] = h[j][2], h[j][2] = x[v][j];
+                    if (ub + v < br.n && c0 + 32 * j < V) p.act[(size_t)(br.t0 + ub + v) * p.lda + p.off_v + c0 + 32 * j] = y;
+                }
         }
     }
 }
@@ -445,7 +450,7 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
 }
 
 // ---------------------------------------------------------------- the scan over blocks
-constexpr int SC_COLS = 16, SC_THREADS = 256;           // value columns per CTA: two per warp
+constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp
 
 struct ScanParams {
     const float* blocks;           // k_delta_blocks / k_ssd_blocks
@@ -493,29 +498,53 @@ struct Chan {
     }
 };
 
-// Dot products of the warp's two columns (s: this lane's channels of each) with sixteen rows of shared memory.  Lane
-// 16 c + t gets column c's product with row t.
-template <int EPL>
-__device__ __forceinline__ float column_dots(const float* rows, int dp, const float (&s)[2][EPL], int lane) {
-    float r[32];
+// Dot products of the warp's four columns (s: this lane's channels of each) with NS sets of sixteen rows of shared
+// memory, eight rows in flight ahead of the arithmetic.  Lane 8 c + j gets column c's products with rows j and j + 8.
+template <int EPL, int NS>
+__device__ __forceinline__ void column_dots(const float* rows, int dp, const float (&s)[4][EPL], int lane, float (&out)[NS][2]) {
+    constexpr int G = EPL <= 4 ? 8 : 4;
+    float r[NS][64], w[2][G][EPL];
 #pragma unroll
-    for (int t = 0; t < BT; ++t) {
-        float w[EPL];
-        Chan<EPL>::load(rows + t * dp, lane, w);
+    for (int t = 0; t < G; ++t) Chan<EPL>::load(rows + t * dp, lane, w[0][t]);
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-            if (EPL == 1) {
-                r[16 * c + t] = s[c][0] * w[0];
-            } else {
-                uint64_t a = 0;
+    for (int g = 0; g < NS * BT / G; ++g) {
+        if (g + 1 < NS * BT / G) {
 #pragma unroll
-                for (int i = 0; i + 1 < EPL; i += 2) a = fma2(pair(s[c][i], s[c][i + 1]), pair(w[i], w[i + 1]), a);
-                const float2 f = unpair(a);
-                r[16 * c + t] = f.x + f.y;
+            for (int t = 0; t < G; ++t) Chan<EPL>::load(rows + (G * (g + 1) + t) * dp, lane, w[(g + 1) & 1][t]);
+        }
+#pragma unroll
+        for (int u = 0; u < G; ++u) {
+            const int row = G * g + u, t = row % BT;
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                float& dst = r[row / BT][16 * c + 2 * (t & 7) + (t >> 3)];
+                if (EPL == 1) {
+                    dst = s[c][0] * w[g & 1][u][0];
+                } else {
+                    uint64_t a = 0;
+#pragma unroll
+                    for (int i = 0; i + 1 < EPL; i += 2) a = fma2(pair(s[c][i], s[c][i + 1]), pair(w[g & 1][u][i], w[g & 1][u][i + 1]), a);
+                    const float2 f = unpair(a);
+                    dst = f.x + f.y;
+                }
             }
         }
     }
-    return transpose_sum32(r, lane);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {                           // each step halves the sums a lane carries
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+            if (i < 2 * o) {
+#pragma unroll
+                for (int k = 0; k < NS; ++k) {
+                    const float send = up ? r[k][i] : r[k][i + 2 * o], keep = up ? r[k][i + 2 * o] : r[k][i];
+                    r[k][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+    }
+#pragma unroll
+    for (int k = 0; k < NS; ++k) out[k][0] = r[k][0], out[k][1] = r[k][1];
 }
 
 // EPL: key channels per lane (the key size, padded to 32 EPL).
@@ -523,11 +552,11 @@ template <int EPL, bool DELTA>
 __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     constexpr int DP = 32 * EPL, BLK = DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK, BUF = BLK + BT * SC_COLS;
     extern __shared__ __align__(16) float sm[];
-    __shared__ __align__(16) float s_d[8][2][BT], s_u[8][2][BT];
+    __shared__ __align__(16) float s_d[4][4][BT], s_u[4][4][BT];
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lt = lane & 15, lc = lane >> 4;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lt = lane & 7, lc = lane >> 3;
     const int c0 = blockIdx.x * SC_COLS, h = blockIdx.y, e = blockIdx.z, kh = h / p.per;
-    const int col = c0 + warp * 2 + lc;
+    const int col = c0 + warp * 4 + lc;
     if (!DELTA) {
         for (int i = tid; i < 2 * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels stay zero
         __syncthreads();
@@ -538,15 +567,15 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     const int seq = p.seq_ids[t0], blocks = (t1 - t0 + BT - 1) / BT;
     const float* bsrc = p.blocks + ((size_t)block_base(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
     const size_t bstep = (size_t)p.heads * (DELTA ? BLK : SSD_BLOCK);
-    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 2) * p.dim;
-    float s[2][EPL];             // channels Chan::at of the warp's two columns
+    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 4) * p.dim;
+    float s[4][EPL];             // channels Chan::at of the warp's four columns
     const bool fresh = p.positions[t0] == 0, live = col < p.vdim;
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+    for (int c = 0; c < 4; ++c)
 #pragma unroll
         for (int i = 0; i < EPL; ++i) {
             const int d = Chan<EPL>::at(lane, i);
-            s[c][i] = !fresh && c0 + warp * 2 + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
+            s[c][i] = !fresh && c0 + warp * 4 + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
         }
 
     auto load = [&](int b, int buf) {
@@ -588,12 +617,16 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
         __syncthreads();
         const float* x = sm + (b & 1) * BUF;
-        // ---- the columns against the block's (decayed) keys and queries; lane 16 c + t works for column c, token t
-        float rk = 0.0f;
-        if (DELTA) rk = column_dots<EPL>(x, DP, s, lane);
-        const float rq = column_dots<EPL>(x + (DELTA ? BT * DP : 0), DP, s, lane);
-        const float v = x[BLK + lt * SC_COLS + warp * 2 + lc];
-        s_d[warp][lc][lt] = v - rk;
+        // ---- the columns against the block's (decayed) keys and queries; lane 8 c + j works for column c, tokens j, j + 8
+        float r[DELTA ? 2 : 1][2];
+        column_dots<EPL, DELTA ? 2 : 1>(x, DP, s, lane, r);
+        const float* rq = r[DELTA ? 1 : 0];
+        float v[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            v[k] = x[BLK + (lt + 8 * k) * SC_COLS + warp * 4 + lc];
+            s_d[warp][lc][lt + 8 * k] = DELTA ? v[k] - r[0][k] : v[k];
+        }
         __syncwarp();
         auto row_dot = [&](const float* row, const float* vals) {      // rows of W, B, M are zero above the diagonal
             float a[4] = {};
@@ -608,47 +641,66 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             return (a[0] + a[1]) + (a[2] + a[3]);
         };
         const float* scal = x + (DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
-        float out;
+        float out[2];
         if (DELTA) {
-            s_u[warp][lc][lt] = row_dot(scal + lt * BROW, s_d[warp][lc]);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) s_u[warp][lc][lt + 8 * k] = row_dot(scal + (lt + 8 * k) * BROW, s_d[warp][lc]);
             __syncwarp();
-            out = rq + row_dot(scal + (BT + lt) * BROW, s_u[warp][lc]);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) out[k] = rq[k] + row_dot(scal + (BT + lt + 8 * k) * BROW, s_u[warp][lc]);
         } else {
             const float* cd = scal + BT * BROW;
-            s_u[warp][lc][lt] = v * cd[BT + lt];
-            out = fmaf(cd[lt], rq, row_dot(scal + lt * BROW, s_d[warp][lc])) + Dh * v;
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int t = lt + 8 * k;
+                s_u[warp][lc][t] = v[k] * cd[BT + t];
+                out[k] = fmaf(cd[t], rq[k], row_dot(scal + t * BROW, s_d[warp][lc])) + Dh * v[k];
+            }
             __syncwarp();
         }
-        if (t0 + b * BT + lt < t1 && live) p.o[(size_t)(t0 + b * BT + lt) * p.ldo + (size_t)h * p.vdim + col] = out;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int t = t0 + b * BT + lt + 8 * k;
+            if (t < t1 && live) p.o[(size_t)t * p.ldo + (size_t)h * p.vdim + col] = out[k];
+        }
         // ---- the state after the block
         const float* keys = x + (DELTA ? 2 * BT * DP : BT * DP);
         {
             float g[EPL];
             if (DELTA) Chan<EPL>::load(x + 3 * BT * DP, lane, g);
 #pragma unroll
-            for (int c = 0; c < 2; ++c)
+            for (int c = 0; c < 4; ++c)
 #pragma unroll
                 for (int i = 0; i < EPL; ++i) s[c][i] *= DELTA ? g[i] : scal[BT * BROW + BT - 1];
         }
+        constexpr int G = EPL <= 4 ? 8 : 4;
 #pragma unroll
-        for (int t = 0; t < BT; ++t) {
-            float w[EPL];
-            Chan<EPL>::load(keys + t * DP, lane, w);
+        for (int t = 0; t < BT; t += G) {
+            float w[G][EPL], u[4][G];
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const float u = s_u[warp][c][t];
+            for (int g = 0; g < G; ++g) Chan<EPL>::load(keys + (t + g) * DP, lane, w[g]);
 #pragma unroll
-                for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(w[i], u, s[c][i]);
-            }
+            for (int c = 0; c < 4; ++c)
+#pragma unroll
+                for (int g = 0; g < G; g += 4) {
+                    const float4 f = *reinterpret_cast<const float4*>(&s_u[warp][c][t + g]);
+                    u[c][g] = f.x, u[c][g + 1] = f.y, u[c][g + 2] = f.z, u[c][g + 3] = f.w;
+                }
+#pragma unroll
+            for (int g = 0; g < G; ++g)
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+#pragma unroll
+                    for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(w[g][i], u[c][g], s[c][i]);
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+    for (int c = 0; c < 4; ++c)
 #pragma unroll
         for (int i = 0; i < EPL; ++i) {
             const int d = Chan<EPL>::at(lane, i);
-            if (c0 + warp * 2 + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
+            if (c0 + warp * 4 + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
         }
 }
 

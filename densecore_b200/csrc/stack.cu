@@ -304,6 +304,7 @@ int dc_stack_finalize(dc_model* m) {
     }
     DC_TRY(dc_check_cuda(ctx, cudaMallocHost((void**)&m->h_stage, 4096), "cudaMallocHost"));
     b.cap = (int)C;
+    DC_TRY(dc_check_cuda(ctx, cudaStreamSynchronize(cudaStreamLegacy), "finalize"));     // the tensors' copies
     return dc_check_cuda(ctx, cudaStreamSynchronize(ctx->stream), "finalize");
 }
 

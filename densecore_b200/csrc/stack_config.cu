@@ -325,5 +325,6 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
             DC_TRY(dc_check_cuda(m->ctx, cudaMemsetAsync(*t.vec, 0, (size_t)t.vec_len * 4 + 64, m->ctx->stream), "weight memory"));
         }
     s->weight_bytes += s->embed->bytes;
-    return DC_B200_OK;
+    // tensors are copied on another stream: the zeros have to be there first
+    return dc_check_cuda(m->ctx, cudaStreamSynchronize(m->ctx->stream), "weight memory");
 }
