@@ -45,26 +45,36 @@ struct PrepParams {
 
 template <typename TC>
 __global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
+    __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x;
     const int pos = min(max(p.positions[t], 0), p.max_pos - 1);
     const float* cs = p.cos_sin + (size_t)pos * p.rot;
     float* row = p.proj + (size_t)t * p.ldp;
     const int half = p.rot / 2;
-    if (p.norm && warp == 0) {
+    if (p.norm) {
         const float* src = row + p.off_kv;
         TC* dst = reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos);
-        float ss = 0.0f;
-        for (int i = lane; i < p.rank; i += 32) ss = fmaf(src[i], src[i], ss);
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.rank + p.eps);
-        for (int i = lane; i < p.rank; i += 32) store_as(dst + i, src[i] * inv * p.norm[i]);
-        for (int i = lane; i < half; i += 32) {
-            const float u = src[p.rank + 2 * i], v = src[p.rank + 2 * i + 1], c = cs[2 * i], s = cs[2 * i + 1];
-            store_as(dst + p.rank + 2 * i, u * c - v * s);
-            store_as(dst + p.rank + 2 * i + 1, v * c + u * s);
+        float v[4], ss = 0.0f;       // kv_rank <= 1024
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            v[j] = i < p.rank ? src[i] : 0.0f;
+            ss = fmaf(v[j], v[j], ss);
         }
-        for (int i = p.rank + p.rot + lane; i < p.c.row; i += 32) store_as(dst + i, 0.0f);
+        const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i < p.rank) store_as(dst + i, v[j] * inv * p.norm[i]);
+        }
+        for (int i = threadIdx.x; i < half; i += 256) {
+            const float u = src[p.rank + 2 * i], w = src[p.rank + 2 * i + 1], c = cs[2 * i], s = cs[2 * i + 1];
+            store_as(dst + p.rank + 2 * i, u * c - w * s);
+            store_as(dst + p.rank + 2 * i + 1, w * c + u * s);
+        }
+        for (int i = p.rank + p.rot + threadIdx.x; i < p.c.row; i += 256) store_as(dst + i, 0.0f);
     }
     for (int i = threadIdx.x; i < p.heads * half; i += 256) {
         const int h = i / half, j = i - h * half;
@@ -156,7 +166,7 @@ struct AbsorbedParams {
 constexpr int AB_KEYS = 32, AB_HEADS = 8;
 
 // One CTA per (key split, group of eight heads, token): a warp is a head.  Scores: a lane is a key; sums: a lane owns
-// column pairs lane, lane + 32, ... of the latent.
+// the 16-byte chunks lane, lane + 32, ... of the latent (RP of them).
 template <typename TC, int RP>
 __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const AbsorbedParams p) {
     constexpr int EPC = 16 / sizeof(TC);      // elements of a 16-byte chunk
@@ -169,21 +179,21 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
     const int s = blockIdx.x, h0 = blockIdx.y * AB_HEADS, t = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = h0 + warp, pos = p.positions[t], seq = p.seq_ids[t];
     const bool live = h < p.heads;
-    for (int i = tid; i < AB_HEADS * row; i += AB_HEADS * 32) {
-        const int hh = i / row, c = i - hh * row;
-        float v = 0.0f;
-        if (h0 + hh < p.heads) {
-            if (c < p.rank) v = p.qa[((size_t)t * p.heads + h0 + hh) * p.ldq + c];
-            else if (c < p.rank + p.rot) v = p.proj[(size_t)t * p.ldp + p.off_q + (h0 + hh) * (p.dim + p.rot) + p.dim + c - p.rank];
-        }
-        sq[i] = v * p.scale;
+    {                            // a warp's own query: the absorbed part, then the rotated part, zeros in the padding
+        const float *qa = p.qa + ((size_t)t * p.heads + min(h, p.heads - 1)) * p.ldq;
+        const float* qr = p.proj + (size_t)t * p.ldp + p.off_q + min(h, p.heads - 1) * (p.dim + p.rot) + p.dim;
+#pragma unroll 8
+        for (int c = lane; c < p.rank; c += 32) sq[warp * row + c] = qa[c] * p.scale;
+        for (int c = p.rank + lane; c < row; c += 32) sq[warp * row + c] = c < p.rank + p.rot ? qr[c - p.rank] * p.scale : 0.0f;
     }
     const int first = first_key(pos, p.window), nk = pos - first + 1;
     const int per = ((nk + p.splits - 1) / p.splits + AB_KEYS - 1) / AB_KEYS * AB_KEYS;
     const int kb = first + s * per, ke = min(first + nk, kb + per);
-    float m = -INFINITY, l = 0.0f, acc[RP][2];
+    float m = -INFINITY, l = 0.0f, acc[RP][EPC];
 #pragma unroll
-    for (int j = 0; j < RP; ++j) acc[j][0] = acc[j][1] = 0.0f;
+    for (int j = 0; j < RP; ++j)
+#pragma unroll
+        for (int i = 0; i < EPC; ++i) acc[j][i] = 0.0f;
     const int chunks = row / EPC;
     for (int k0 = kb; k0 < ke; k0 += AB_KEYS) {
         __syncthreads();
@@ -216,21 +226,20 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
         m = mn;
         l = l * corr + warp_sum(pr);
 #pragma unroll
-        for (int j = 0; j < RP; ++j) {
-            acc[j][0] *= corr;
-            acc[j][1] *= corr;
-        }
+        for (int j = 0; j < RP; ++j)
+#pragma unroll
+            for (int i = 0; i < EPC; ++i) acc[j][i] *= corr;
 #pragma unroll 4
         for (int kk = 0; kk < AB_KEYS; ++kk) {
             const float w = __shfl_sync(0xffffffffu, pr, kk);
-            const TC* kr = sk + kk * ldk;
 #pragma unroll
             for (int j = 0; j < RP; ++j) {
-                const int r = 2 * (lane + 32 * j);
-                if (r < p.rank) {
-                    acc[j][0] = fmaf(w, load_as(kr + r), acc[j][0]);
-                    acc[j][1] = fmaf(w, load_as(kr + r + 1), acc[j][1]);     // rank odd: the neighbour's value, never stored
-                }
+                const int c = lane + 32 * j;
+                if (c >= chunks) continue;       // chunks of the rotated part are summed too and never stored
+                float f[EPC];
+                unpack16(*reinterpret_cast<const uint4*>(sk + kk * ldk + c * EPC), f, TC());
+#pragma unroll
+                for (int i = 0; i < EPC; ++i) acc[j][i] = fmaf(w, f[i], acc[j][i]);
             }
         }
     }
@@ -241,11 +250,12 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
         p.part_ml[2 * o + 1] = l;
     }
 #pragma unroll
-    for (int j = 0; j < RP; ++j) {
-        const int r = 2 * (lane + 32 * j);
-        if (r < p.rank) p.part[o * p.rank + r] = acc[j][0];
-        if (r + 1 < p.rank) p.part[o * p.rank + r + 1] = acc[j][1];
-    }
+    for (int j = 0; j < RP; ++j)
+#pragma unroll
+        for (int i = 0; i < EPC; ++i) {
+            const int r = EPC * (lane + 32 * j) + i;
+            if (r < p.rank) p.part[o * p.rank + r] = acc[j][i];
+        }
 }
 
 // Splits of one (head, token) joined, then taken through OUT_ROWS rows of the head's W_uv.
@@ -274,7 +284,7 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
     for (int r = threadIdx.x; r < rank8; r += 256) {
         float v = 0.0f;
         if (r < rank) {
-#pragma unroll 8
+#pragma unroll 16
             for (int s = 0; s < splits; ++s) v = fmaf(part[(o + s) * rank + r], sw[s], v);
         }
         lat[r] = v;
@@ -306,11 +316,11 @@ int launch_absorbed(dc_ctx* ctx, const AbsorbedParams& p, int T) {
         DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_absorbed<TC, RP>, (int)smem, "k_latent_absorbed"));         \
         return dc_launch(ctx, "k_latent_absorbed", k_latent_absorbed<TC, RP>, grid, block, smem, p);                  \
     } while (0)
-    if (p.rank <= 64) DC_AB(1);
-    if (p.rank <= 128) DC_AB(2);
-    if (p.rank <= 256) DC_AB(4);
-    if (p.rank <= 512) DC_AB(8);
-    DC_AB(16);
+    const int rp = (p.rank * (int)sizeof(TC) + 511) / 512;
+    if (rp <= 1) DC_AB(1);
+    if (rp <= 2) DC_AB(2);
+    if (rp <= 4) DC_AB(4);
+    DC_AB(8);
 #undef DC_AB
 }
 

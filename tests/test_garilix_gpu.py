@@ -60,13 +60,19 @@ ALONE = {
     "delta_grouped_heads": ([delta(heads=6, kv_heads=2, dim=32, vdim=36, conv=3)], {}),
     "delta_one_tap_odd_sizes": ([delta(heads=2, dim=17, vdim=5, conv=1)], dict(a_rank=1, g_rank=7)),
     "delta_wide": ([delta(heads=1, dim=136, vdim=130, conv=5)], dict(a_rank=33, g_rank=64)),
+    "delta_full_heads": ([delta(heads=2, kv_heads=1, dim=128, vdim=128)], {}),
+    "delta_half_heads": ([delta(heads=3, dim=64, vdim=48)], {}),
     "mamba": ([mamba()], {}),
+    "mamba_full_state": ([mamba(heads=4, vdim=64, state=128, groups=2, norm_groups=1)], {}),
+    "mamba_half_state": ([mamba(heads=3, vdim=40, state=64, groups=1, norm_groups=3, conv=5)], {}),
     "mamba_one_group": ([mamba(heads=3, vdim=17, state=10, groups=1, norm_groups=1, conv=3)], {}),
     "mamba_group_per_head": ([mamba(heads=4, vdim=24, state=130, groups=4, norm_groups=3, conv=1)], {}),
     "latent": ([latent()], {}),
     "latent_window_one": ([latent(window=1)], {}),
     "latent_window_two_odd_rank": ([latent(heads=9, dim=20, rot_dim=6, vdim=33, kv_rank=27, window=2, base=300.0, scale=0.31)], {}),
     "latent_wide": ([latent(heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=264, window=70)], {}),
+    "latent_full_rank": ([latent(heads=3, dim=64, rot_dim=32, vdim=64, kv_rank=512, window=40)], {}),
+    "latent_largest": ([latent(heads=2, dim=200, rot_dim=64, vdim=200, kv_rank=768, window=60)], {}),
     "latent_whole_context": ([latent(window=4096)], {}),
     "latent_shared_cache": ([latent(window=9), latent(heads=5, dim=16, vdim=40, window=50, kv_from=0), latent(kv_rank=24, rot_dim=4, window=3)], {}),
 }
