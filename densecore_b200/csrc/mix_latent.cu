@@ -152,6 +152,14 @@ __device__ __forceinline__ void unpack16(const uint4& v, float (&f)[4], float) {
     f[0] = __uint_as_float(v.x), f[1] = __uint_as_float(v.y), f[2] = __uint_as_float(v.z), f[3] = __uint_as_float(v.w);
 }
 
+__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool valid) {
+    const int bytes = valid ? 16 : 0;   // 0: the 16 bytes are zero-filled, the address is not read
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
 struct AbsorbedParams {
     const float* qa;         // [T][heads][ldq]
     int ldq;
@@ -163,9 +171,9 @@ struct AbsorbedParams {
     float *part, *part_ml;   // [T][heads][splits][rank], [T][heads][splits][2]
 };
 
-constexpr int AB_KEYS = 32, AB_HEADS = 8;
+constexpr int AB_KEYS = 32, AB_HEADS = 4;
 
-// One CTA per (key split, group of eight heads, token): a warp is a head.  Scores: a lane is a key; sums: a lane owns
+// One CTA per (key split, group of four heads, token): a warp is a head.  Scores: a lane is a key; sums: a lane owns
 // the 16-byte chunks lane, lane + 32, ... of the latent (RP of them).
 template <typename TC, int RP>
 __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const AbsorbedParams p) {
@@ -197,18 +205,21 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
     const int chunks = row / EPC;
     for (int k0 = kb; k0 < ke; k0 += AB_KEYS) {
         __syncthreads();
+        const TC* src[AB_KEYS / AB_HEADS];                  // a warp's keys: all rows asked for before any arrives
 #pragma unroll
-        for (int i = 0; i < AB_KEYS / AB_HEADS; ++i) {      // a warp's keys
-            const int kk = warp * (AB_KEYS / AB_HEADS) + i;
-            const bool ok = k0 + kk < ke;
-            const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const TC*>(p.c.arena) + (ok ? p.c.at(seq, k0 + kk) : 0));
-            for (int c = lane; c < chunks; c += 32) *reinterpret_cast<uint4*>(sk + kk * ldk + c * EPC) = ok ? src[c] : make_uint4(0, 0, 0, 0);
-        }
+        for (int i = 0; i < AB_KEYS / AB_HEADS; ++i)
+            src[i] = reinterpret_cast<const TC*>(p.c.arena) + p.c.at(seq, min(k0 + warp * (AB_KEYS / AB_HEADS) + i, ke - 1));
+        for (int c = lane; c < chunks; c += 32)
+#pragma unroll
+            for (int i = 0; i < AB_KEYS / AB_HEADS; ++i)
+                cp_async16z(smem_u32(sk + (warp * (AB_KEYS / AB_HEADS) + i) * ldk + c * EPC), src[i] + c * EPC, true);
+        cp_async_commit();
+        cp_async_wait<0>();
         __syncthreads();
         if (!live) continue;
         float part[EPC] = {};
         const float* q = sq + warp * row;
-#pragma unroll 4
+#pragma unroll 8
         for (int c = 0; c < chunks; ++c) {
             float f[EPC];
             unpack16(*reinterpret_cast<const uint4*>(sk + lane * ldk + c * EPC), f, TC());
@@ -229,15 +240,14 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
         for (int j = 0; j < RP; ++j)
 #pragma unroll
             for (int i = 0; i < EPC; ++i) acc[j][i] *= corr;
-#pragma unroll 4
+#pragma unroll 8
         for (int kk = 0; kk < AB_KEYS; ++kk) {
             const float w = __shfl_sync(0xffffffffu, pr, kk);
 #pragma unroll
             for (int j = 0; j < RP; ++j) {
                 const int c = lane + 32 * j;
-                if (c >= chunks) continue;       // chunks of the rotated part are summed too and never stored
                 float f[EPC];
-                unpack16(*reinterpret_cast<const uint4*>(sk + kk * ldk + c * EPC), f, TC());
+                unpack16(*reinterpret_cast<const uint4*>(sk + kk * ldk + min(c, chunks - 1) * EPC), f, TC());   // beyond the latent: never stored
 #pragma unroll
                 for (int i = 0; i < EPC; ++i) acc[j][i] = fmaf(w, f[i], acc[j][i]);
             }
@@ -290,20 +300,29 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
         lat[r] = v;
     }
     __syncthreads();
-#pragma unroll 4
-    for (int e = e0 + warp; e < e1; e += 8) {
-        const uint4* w = reinterpret_cast<const uint4*>(uv + (size_t)(h * vdim_p + e) * ldw);
-        float a = 0.0f;
-        for (int c = lane; c < rank8 / 8; c += 32) {
-            float f[8];
-            unpack16(w[c], f, __nv_bfloat16());
+    constexpr int ROWS = OUT_ROWS / 8;                // of a warp, all in flight
+    float a[ROWS] = {};
+    for (int c = lane; c < rank8 / 8; c += 32) {
+        uint4 v[ROWS];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) a = fmaf(f[i], lat[8 * c + i], a);
+        for (int i = 0; i < ROWS; ++i) v[i] = *reinterpret_cast<const uint4*>(uv + (size_t)(h * vdim_p + min(e0 + warp + 8 * i, e1 - 1)) * ldw + 8 * c);
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) {
+            float f[8];
+            unpack16(v[i], f, __nv_bfloat16());
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a[i] = fmaf(f[j], lat[8 * c + j], a[i]);
         }
-        a = warp_sum(a);
+    }
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        const int e = e0 + warp + 8 * i;
+        const float v = warp_sum(a[i]);
         const size_t at = (size_t)t * ldm + (size_t)h * vdim + e;
-        if (lane == 0 && mixb) mixb[at] = __float2bfloat16_rn(a);
-        else if (lane == 0) mix[at] = a;
+        if (lane == 0 && e < e1) {
+            if (mixb) mixb[at] = __float2bfloat16_rn(v);
+            else mix[at] = v;
+        }
     }
 }
 
@@ -347,13 +366,6 @@ __global__ void __launch_bounds__(256) k_latent_gather(CacheRef c, const int32_t
     for (int j = lane; j < ldr; j += 32) kr[(size_t)i * ldr + j] = j < rot ? src[rank + j] : __float2bfloat16_rn(0.0f);
 }
 
-__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool valid) {
-    const int bytes = valid ? 16 : 0;   // 0: the 16 bytes are zero-filled, the address is not read
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }

@@ -739,6 +739,61 @@ struct DeltaDecode {
     int ldm;
 };
 
+// Decode convolutions of the channels tid, tid + NT, ...: B of them at a time, every load before the arithmetic.  place(c)
+// gives the channel's projection column, ring column and weight column (below zero: none, the result is 0); put(c, y)
+// takes the silu of the convolution.  own(c): this CTA also puts the channel's input into the ring (a row that no tap
+// of this token reads).
+struct ConvPlace {
+    int col, rc, wc;
+};
+template <int NT, int B, typename Place, typename Put, typename Own>
+__device__ __forceinline__ void conv_decode(const float* row, float* ring, int C, int taps, const float* w, int ldw, const float* bias, int pos, int total,
+                                            Place place, Put put, Own own) {
+    for (int c0 = threadIdx.x; c0 < total; c0 += NT * B) {
+        ConvPlace at[B];
+        float s[B] = {}, last[B], add[B];
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+            at[b] = place(min(c0 + NT * b, total - 1));
+            last[b] = row[max(at[b].col, 0)];
+            add[b] = bias ? bias[max(at[b].wc, 0)] : 0.0f;
+        }
+        for (int j0 = 0; j0 < taps - 1; j0 += 3) {
+            float in[B][3], wj[B][3];
+#pragma unroll
+            for (int k = 0; k < 3; ++k) {
+                const int j = min(j0 + k, taps - 2), back = taps - 1 - j;
+                const bool ok = j0 + k < taps - 1 && pos >= back;
+                const size_t r = (size_t)(max(pos - back, 0) % taps) * C;
+#pragma unroll
+                for (int b = 0; b < B; ++b) {
+                    in[b][k] = ring[r + max(at[b].rc, 0)];
+                    wj[b][k] = ok ? w[(size_t)j * ldw + max(at[b].wc, 0)] : 0.0f;
+                }
+                if (!ok) {
+#pragma unroll
+                    for (int b = 0; b < B; ++b) in[b][k] = 0.0f;
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+#pragma unroll
+                for (int b = 0; b < B; ++b) s[b] = fmaf(wj[b][k], in[b][k], s[b]);
+        }
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+            const int c = c0 + NT * b;
+            if (c >= total) continue;
+            if (at[b].col < 0) {
+                put(c, 0.0f);
+                continue;
+            }
+            put(c, silu(fmaf(w[(size_t)(taps - 1) * ldw + at[b].wc], last[b], s[b]) + add[b]));
+            if (own(c)) ring[(size_t)(pos % taps) * C + at[b].rc] = last[b];
+        }
+    }
+}
+
 // out[r] = rows r < n of a bf16 matrix (padded with zeros) times x in shared memory (zero up to a multiple of 128); sixteen
 // lanes a row, eight rows of a half-warp in flight
 __device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ldw, int n, const float* x, int rank, float* out) {
@@ -861,20 +916,15 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
     float* ring = p.cr.ring(seq);
     const float* row = p.proj + (size_t)t * p.ldp;
     const bool first = h % p.per == 0;
-    for (int c = tid; c < 2 * DP + p.vdim; c += 256) {
-        const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
-        const int col = c < DP ? p.off_q + kh * p.dim + d : c < 2 * DP ? p.off_k + kh * p.dim + d : p.off_v + h * p.vdim + d;
-        float v = 0.0f;
-        if (c >= 2 * DP || d < p.dim) {
-            v = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, col, taps, p.conv + col, p.cr.ldw, col, t, 0, pos));
-        }
-        sm[c < 2 * DP ? c : (int)(sv - sm) + d] = v;
-    }
-    // the token's own inputs into the ring: a row that none of its taps reads
-    for (int c = tid; c < 2 * p.dim + p.vdim; c += 256) {
-        const int col = c < p.dim ? p.off_q + kh * p.dim + c : c < 2 * p.dim ? p.off_k + kh * p.dim + c - p.dim : p.off_v + h * p.vdim + c - 2 * p.dim;
-        if (c >= 2 * p.dim || first) ring[(size_t)(pos % taps) * p.cr.C + col] = row[col];
-    }
+    conv_decode<256, 2>(
+        row, ring, p.cr.C, taps, p.conv, p.cr.ldw, nullptr, pos, 2 * DP + p.vdim,
+        [&](int c) {
+            const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
+            if (c < 2 * DP && d >= p.dim) return ConvPlace{-1, -1, -1};
+            const int col = c < DP ? p.off_q + kh * p.dim + d : c < 2 * DP ? p.off_k + kh * p.dim + d : p.off_v + h * p.vdim + d;
+            return ConvPlace{col, col, col};
+        },
+        [&](int c, float v) { sm[c < 2 * DP ? c : (int)(sv - sm) + c - 2 * DP] = v; }, [&](int c) { return c >= 2 * DP || first; });
     for (int c = tid; c < ra; c += 256) sa[c] = c < p.a_rank ? row[p.off_a + c] : 0.0f;
     for (int c = tid; c < rg; c += 256) sgl[c] = c < p.g_rank ? row[p.off_g + c] : 0.0f;
     __syncthreads();
@@ -965,20 +1015,15 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
     float* ring = p.cr.ring(seq);
     const float* row = p.proj + (size_t)t * p.ldp;
     const bool first = h % p.per == 0;
-    for (int c = tid; c < 2 * DP + p.vdim; c += 128) {
-        const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
-        const int ch = c < DP ? inner + g * p.state + d : c < 2 * DP ? inner + GN + g * p.state + d : h * p.vdim + d;
-        float v = 0.0f;
-        if (c >= 2 * DP || d < p.state) {
-            v = silu(conv_at(p.proj, p.ldp, ring, p.cr.C, ch, taps, p.conv + ch, p.cr.ldw, p.off_x + ch, t, 0, pos) + p.conv_b[ch]);
-        }
-        sm[c] = v;
-    }
-    // the token's own inputs into the ring: a row that none of its taps reads
-    for (int c = tid; c < 2 * p.state + p.vdim; c += 128) {
-        const int ch = c < p.state ? inner + g * p.state + c : c < 2 * p.state ? inner + GN + g * p.state + c - p.state : h * p.vdim + c - 2 * p.state;
-        if (c >= 2 * p.state || first) ring[(size_t)(pos % taps) * p.cr.C + ch] = row[p.off_x + ch];
-    }
+    conv_decode<128, 3>(
+        row, ring, p.cr.C, taps, p.conv, p.cr.ldw, p.conv_b, pos, 2 * DP + p.vdim,
+        [&](int c) {
+            const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
+            if (c < 2 * DP && d >= p.state) return ConvPlace{-1, -1, -1};
+            const int ch = c < DP ? inner + g * p.state + d : c < 2 * DP ? inner + GN + g * p.state + d : h * p.vdim + d;
+            return ConvPlace{p.off_x + ch, ch, ch};
+        },
+        [&](int c, float v) { sm[c] = v; }, [&](int c) { return c >= 2 * DP || first; });
     const float dt = softplus(row[p.off_dt + h] + p.dt_bias[h]), decay = expf(p.neg_a[h] * dt), Dh = p.D[h];
     __syncthreads();
     float br[EPL], cr[EPL];
