@@ -217,28 +217,39 @@ __global__ void __launch_bounds__(256) k_delta_prep4(DeltaPrep p) {
                     xq[v][j] = row[p.off_q + dc], xk[v][j] = row[p.off_k + dc];
                 }
             }
+            float sq[AHEAD], sk[AHEAD];
 #pragma unroll
             for (int v = 0; v < AHEAD; ++v) {
-                if (ub + v >= br.n) break;
-                float* act = p.act + (size_t)(br.t0 + ub + v) * p.lda;
-                float q[NJ], k[NJ], sq = 0.0f, sk = 0.0f;
+                sq[v] = sk[v] = 0.0f;
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
-                    q[j] = silu(fmaf(wq[j][3], xq[v][j], fmaf(wq[j][2], hq[j][2], fmaf(wq[j][1], hq[j][1], wq[j][0] * hq[j][0]))));
-                    k[j] = silu(fmaf(wk[j][3], xk[v][j], fmaf(wk[j][2], hk[j][2], fmaf(wk[j][1], hk[j][1], wk[j][0] * hk[j][0]))));
-                    hq[j][0] = hq[j][1], hq[j][1] = hq[j][2], hq[j][2] = xq[v][j];
-                    hk[j][0] = hk[j][1], hk[j][1] = hk[j][2], hk[j][2] = xk[v][j];
-                    if (lane + 32 * j >= p.dim) q[j] = k[j] = 0.0f;
-                    sq = fmaf(q[j], q[j], sq);
-                    sk = fmaf(k[j], k[j], sk);
+                    const float q = xq[v][j], k = xk[v][j];
+                    xq[v][j] = silu(fmaf(wq[j][3], q, fmaf(wq[j][2], hq[j][2], fmaf(wq[j][1], hq[j][1], wq[j][0] * hq[j][0]))));
+                    xk[v][j] = silu(fmaf(wk[j][3], k, fmaf(wk[j][2], hk[j][2], fmaf(wk[j][1], hk[j][1], wk[j][0] * hk[j][0]))));
+                    hq[j][0] = hq[j][1], hq[j][1] = hq[j][2], hq[j][2] = q;
+                    hk[j][0] = hk[j][1], hk[j][1] = hk[j][2], hk[j][2] = k;
+                    if (lane + 32 * j >= p.dim) xq[v][j] = xk[v][j] = 0.0f;
+                    sq[v] = fmaf(xq[v][j], xq[v][j], sq[v]);
+                    sk[v] = fmaf(xk[v][j], xk[v][j], sk[v]);
                 }
-                const float iq = p.q_scale / sqrtf(warp_sum(sq) + p.unit_eps), ik = 1.0f / sqrtf(warp_sum(sk) + p.unit_eps);
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int v = 0; v < AHEAD; ++v) {
+                    sq[v] += __shfl_xor_sync(0xffffffffu, sq[v], o);
+                    sk[v] += __shfl_xor_sync(0xffffffffu, sk[v], o);
+                }
+#pragma unroll
+            for (int v = 0; v < AHEAD; ++v) {
+                const float iq = p.q_scale / sqrtf(sq[v] + p.unit_eps), ik = 1.0f / sqrtf(sk[v] + p.unit_eps);
+                float* act = p.act + (size_t)(br.t0 + ub + v) * p.lda + item * p.dim;
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
                     const int d = lane + 32 * j;
-                    if (d < p.dim) {
-                        act[p.off_q + item * p.dim + d] = q[j] * iq;
-                        act[p.off_k + item * p.dim + d] = k[j] * ik;
+                    if (ub + v < br.n && d < p.dim) {
+                        act[p.off_q + d] = xq[v][j] * iq;
+                        act[p.off_k + d] = xk[v][j] * ik;
                     }
                 }
             }
@@ -324,23 +335,28 @@ __global__ void __launch_bounds__(128) k_delta_blocks(const DeltaBlock p) {
     float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * delta_block_floats(dp);
     if (tid < BT) sbeta[tid] = tid < br.n ? p.small[(size_t)(br.t0 + tid) * p.lds + h] : 0.0f;
     for (int d = tid; d < dp; d += 128) {
-        float k[BT], g[BT], cum = 1.0f;
+        float k[BT], q[BT], g[BT], cum = 1.0f;
         const bool in = d < dim;
-        const float na = p.neg_a[h], bias = in ? p.dt_bias[(size_t)h * dim + d] : 0.0f;
+        const int dc = min(d, dim - 1);
+        const float na = p.neg_a[h], bias = p.dt_bias[(size_t)h * dim + dc];
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {                  // every load before the arithmetic
+            const int tc = br.t0 + min(t, br.n - 1);
+            const float* a = p.act + (size_t)tc * p.lda + (h / p.per) * dim + dc;
+            k[t] = a[p.off_k];
+            q[t] = a[p.off_q];
+            g[t] = p.raw[(size_t)tc * p.ldr + h * dim + dc];
+        }
 #pragma unroll
         for (int t = 0; t < BT; ++t) {
-            float q = 0.0f;
-            k[t] = 0.0f, g[t] = 1.0f;
-            if (in && t < br.n) {
-                const float* a = p.act + (size_t)(br.t0 + t) * p.lda + (h / p.per) * dim + d;
-                k[t] = a[p.off_k];
-                q = a[p.off_q];
-                g[t] = expf(na * softplus(p.raw[(size_t)(br.t0 + t) * p.ldr + h * dim + d] + bias));
-            }
+            const bool ok = in && t < br.n;
+            k[t] = ok ? k[t] : 0.0f;
+            q[t] = ok ? q[t] : 0.0f;
+            g[t] = ok ? expf(na * softplus(g[t] + bias)) : 1.0f;
             cum *= g[t];
             out[t * dp + d] = cum * k[t];
-            out[(BT + t) * dp + d] = cum * q;
-            if (in) sk[t * dim + d] = k[t], sq[t * dim + d] = q, sg[t * dim + d] = g[t];
+            out[(BT + t) * dp + d] = cum * q[t];
+            if (in) sk[t * dim + d] = k[t], sq[t * dim + d] = q[t], sg[t * dim + d] = g[t];
         }
         out[3 * BT * dp + d] = cum;
         float suffix = 1.0f;
@@ -351,25 +367,32 @@ __global__ void __launch_bounds__(128) k_delta_blocks(const DeltaBlock p) {
         }
     }
     __syncthreads();
-    for (int i = warp; i < BT; i += 4) {
-        float v[32];
+    // A and B of the key tokens i = warp, warp + 4, ...: c runs over P_ti k_i (zero before i, k_i at i)
 #pragma unroll
-        for (int j = 0; j < 32; ++j) v[j] = 0.0f;
+    for (int half = 0; half < 2; ++half) {
+        float v[2][32];
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[0][j] = v[1][j] = 0.0f;
         for (int d = lane; d < dim; d += 32) {
-            float c = sk[i * dim + d];
+            float c[2] = {0.0f, 0.0f};
 #pragma unroll
-            for (int t = 0; t < BT; ++t)
-                if (t >= i) {
-                    if (t > i) {
-                        c *= sg[t * dim + d];
-                        v[t] = fmaf(c, sk[t * dim + d], v[t]);
-                    }
-                    v[BT + t] = fmaf(c, sq[t * dim + d], v[BT + t]);
+            for (int t = 0; t < BT; ++t) {
+                const float k = sk[t * dim + d], q = sq[t * dim + d], g = sg[t * dim + d];
+#pragma unroll
+                for (int m = 0; m < 2; ++m) {
+                    c[m] = t == warp + 4 * (2 * half + m) ? k : c[m] * g;
+                    v[m][t] = fmaf(c[m], k, v[m][t]);
+                    v[m][BT + t] = fmaf(c[m], q, v[m][BT + t]);
                 }
+            }
         }
-        const float r = transpose_sum32(v, lane);
-        if (lane < BT) sA[lane][i] = r;
-        else sB[lane - BT][i] = r;
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+            const int i = warp + 4 * (2 * half + m);
+            const float r = transpose_sum32(v[m], lane);
+            if (lane < BT) sA[lane][i] = r;             // read below the diagonal only
+            else sB[lane - BT][i] = r;
+        }
     }
     __syncthreads();
     if (tid < BT) {                                     // column tid of (I + diag(beta) A)^-1 diag(beta)
@@ -586,16 +609,16 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             for (int i = tid; i < BLK / 4; i += SC_THREADS) cp_async16z(smem_u32(dst + 4 * i), src + 4 * i, true);
         } else {
             for (int i = tid; i < SSD_BLOCK / 4; i += SC_THREADS) cp_async16z(smem_u32(dst + 2 * BT * DP + 4 * i), src + 4 * i, true);
+            const int t = tid >> 3;                  // eight threads per token
+            const bool ok = tb + t < t1;
 #pragma unroll
             for (int a = 0; a < 2; ++a) {
-                const float* rows = (a ? p.k : p.q) + (size_t)kh * p.dim;
-                const int w = p.vec ? 4 : 1, n = p.dim / w;
-                for (int i = tid; i < BT * n; i += SC_THREADS) {
-                    const int t = i / n, d = (i - t * n) * w;
-                    const bool ok = tb + t < t1;
-                    const float* from = ok ? rows + (size_t)(tb + t) * p.ld + d : rows;
-                    if (p.vec) cp_async16z(smem_u32(dst + (a * BT + t) * DP + d), from, ok);
-                    else cp_async4z(smem_u32(dst + (a * BT + t) * DP + d), from, ok);
+                const float* row = (a ? p.k : p.q) + (size_t)kh * p.dim + (size_t)(ok ? tb + t : tb) * p.ld;
+                const uint32_t to = smem_u32(dst + (a * BT + t) * DP);
+                if (p.vec) {
+                    for (int d = 4 * (tid & 7); d < p.dim; d += 32) cp_async16z(to + 4 * d, row + d, ok);
+                } else {
+                    for (int d = tid & 7; d < p.dim; d += 8) cp_async4z(to + 4 * d, row + d, ok);
                 }
             }
         }
@@ -1071,8 +1094,8 @@ __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict_
 }
 
 // ssd: one CTA per (token, norm group): y silu(z) (unless gated already), over its root mean square, times w
-template <typename TO>
-__global__ void __launch_bounds__(256) k_gate_group_norm(const float* __restrict__ y, int ldy, const float* __restrict__ z, int ldz,
+template <typename TO, int NT>
+__global__ void __launch_bounds__(NT) k_gate_group_norm(const float* __restrict__ y, int ldy, const float* __restrict__ z, int ldz,
                                                          const float* __restrict__ w, int n, float eps, TO* __restrict__ out, int ldm) {
     __shared__ float red[33];
     pdl_launch_dependents();
@@ -1084,22 +1107,30 @@ __global__ void __launch_bounds__(256) k_gate_group_norm(const float* __restrict
     float v[KEEP], ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-        const int i = threadIdx.x + 256 * j;
+        const int i = threadIdx.x + NT * j;
         v[j] = i < n ? (zr ? yr[i] * silu(zr[i]) : yr[i]) : 0.0f;
         ss = fmaf(v[j], v[j], ss);
     }
-    for (int i = threadIdx.x + 256 * KEEP; i < n; i += 256) {
+    for (int i = threadIdx.x + NT * KEEP; i < n; i += NT) {
         const float x = zr ? yr[i] * silu(zr[i]) : yr[i];
         ss = fmaf(x, x, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-        const int i = threadIdx.x + 256 * j;
+        const int i = threadIdx.x + NT * j;
         if (i < n) store_as(out + (size_t)t * ldm + c0 + i, v[j] * inv * w[c0 + i]);
     }
-    for (int i = threadIdx.x + 256 * KEEP; i < n; i += 256)
+    for (int i = threadIdx.x + NT * KEEP; i < n; i += NT)
         store_as(out + (size_t)t * ldm + c0 + i, (zr ? yr[i] * silu(zr[i]) : yr[i]) * inv * w[c0 + i]);
+}
+
+// small groups get small CTAs: more of them are resident
+template <typename TO>
+int launch_group_norm(dc_ctx* ctx, const float* y, int ldy, const float* z, int ldz, const float* w, int n, int groups, int T, float eps, TO* out, int ldm) {
+    const dim3 grid(groups, T);
+    if (n <= 512) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 64>, grid, dim3(64), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 256>, grid, dim3(256), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
 }
 
 // ---------------------------------------------------------------- ssd: per-token inputs
@@ -1248,11 +1279,9 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
     p.vec = m.state % 4 == 0 && lda % 4 == 0 && inner % 4 == 0;
     DC_TRY(launch_scan<false>(ctx, p, st.E));
     const int n = inner / m.norm_groups;
-    if (mixb)
-        return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<__nv_bfloat16>, dim3(m.norm_groups, st.T), dim3(256), 0, y, lda, proj + m.off_z, ldp,
-                         m.norm, n, eps, mixb, ldm);
-    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<float>, dim3(m.norm_groups, st.T), dim3(256), 0, y, lda, proj + m.off_z, ldp, m.norm, n,
-                     eps, mix, ldm);
+    const float* z = proj + m.off_z;
+    return mixb ? launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
+                : launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
 }
 
 int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
@@ -1284,9 +1313,7 @@ int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, 
     else if (dp == 64) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<2>, grid, block, smem, p));
     else if (dp == 128) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<4>, grid, block, smem, p));
     else DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<8>, grid, block, smem, p));
-    if (mixb)
-        return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<__nv_bfloat16>, dim3(m.norm_groups, st.T), dim3(256), 0, y, ldy, nullptr, 0, m.norm,
-                         inner / m.norm_groups, eps, mixb, ldm);
-    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<float>, dim3(m.norm_groups, st.T), dim3(256), 0, y, ldy, nullptr, 0, m.norm,
-                     inner / m.norm_groups, eps, mix, ldm);
+    const int n = inner / m.norm_groups;
+    return mixb ? launch_group_norm(ctx, y, ldy, nullptr, 0, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
+                : launch_group_norm(ctx, y, ldy, nullptr, 0, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
 }
