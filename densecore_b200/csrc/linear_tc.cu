@@ -4,7 +4,10 @@
 // loads (64 columns of both operands, 128-byte swizzle), one thread issues the UMMAs (128 x 128 x 16, f32
 // accumulators in tensor memory), four warps read the accumulators out.  A weight row is a tensor-memory lane, so
 // a warp's stores of one token are 32 consecutive outputs.  Two CTAs share an SM: one's read-out overlaps the
-// other's products.  Columns beyond K and rows beyond the matrix are the zeros that TMA fills in.  Every wait is
+// other's products.  Large products use tiles of 128 x 256 instead (k_linear_tc_wide): one CTA per SM walks its share
+// of them, with two sets of accumulators, so that the loads and products of a tile run while the tile before is read
+// out; the wider tile reads shared memory less often per product.  Both let the next kernel start only after every
+// CTA has its tensor memory.  Columns beyond K and rows beyond the matrix are the zeros that TMA fills in.  Every wait is
 // bounded; a CTA that gives up drains its copies, frees its tensor memory and leaves.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
@@ -27,13 +30,47 @@ struct LtParams {
     int* err;
 };
 
+// Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.
+template <int COLS>
+__device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int quarter, int lane) {
+    const int row = row0 + 32 * quarter + lane;
+    for (int c0 = 0; c0 < COLS && t0 + c0 < p.T; c0 += 16) {
+        int v[16];
+        tmem_ld16(tmem + ((uint32_t)(32 * quarter) << 16) + c0, v);
+        tmem_ld_wait();
+        if (p.epi == DC_LIN_GELU_PAIR) {
+            // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
+            const bool up = lane & 1;
+            const int o = row >> 1;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
+                const float mine = __int_as_float(up ? v[i + 8] : v[i]);
+                const float h = up ? gelu_tanh(got) * mine : gelu_tanh(mine) * got;
+                const int t = t0 + c0 + i + (up ? 8 : 0);
+                if (t < p.T && o < p.n_out) {
+                    if (p.outb) p.outb[(size_t)t * p.ldo + o] = __float2bfloat16_rn(h);
+                    else p.out[(size_t)t * p.ldo + o] = h;
+                }
+            }
+        } else if (row < p.n_out) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                const int t = t0 + c0 + i;
+                if (t >= p.T) break;
+                if (p.outb) p.outb[(size_t)t * p.ldo + row] = __float2bfloat16_rn(__int_as_float(v[i]));
+                else p.out[(size_t)t * p.ldo + row] = __int_as_float(v[i]);
+            }
+        }
+    }
+}
+
 __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_constant__ CUtensorMap wmap,
                                                              const __grid_constant__ CUtensorMap xmap, const LtParams p) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t s_bar[2 * LT_STAGES + 1];
     __shared__ uint32_t s_tmem;
     __shared__ int s_give_up;
-    pdl_launch_dependents();
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t full = smem_u32(s_bar), empty = full + 8 * LT_STAGES, acc = empty + 8 * LT_STAGES;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -57,6 +94,7 @@ __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_consta
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = s_tmem;
+    pdl_launch_dependents();
     pdl_wait();
     if (warp == 0) {
         if (lane == 0) {
@@ -92,43 +130,120 @@ __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_consta
     } else {
         const bool ok = tc_wait_raw(acc, 0, give_up, p.err) && !*give_up;
         tc_fence_after();
-        if (__all_sync(0xffffffffu, ok)) {
-            const int quarter = warp & 3, row = row0 + 32 * quarter + lane;
-            for (int c0 = 0; c0 < 128 && t0 + c0 < p.T; c0 += 16) {
-                int v[16];
-                tmem_ld16(tmem + ((uint32_t)(32 * quarter) << 16) + c0, v);
-                tmem_ld_wait();
-                if (p.epi == DC_LIN_GELU_PAIR) {
-                    // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
-                    const bool up = lane & 1;
-                    const int o = row >> 1;
-#pragma unroll
-                    for (int i = 0; i < 8; ++i) {
-                        const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
-                        const float mine = __int_as_float(up ? v[i + 8] : v[i]);
-                        const float h = up ? gelu_tanh(got) * mine : gelu_tanh(mine) * got;
-                        const int t = t0 + c0 + i + (up ? 8 : 0);
-                        if (t < p.T && o < p.n_out) {
-                            if (p.outb) p.outb[(size_t)t * p.ldo + o] = __float2bfloat16_rn(h);
-                            else p.out[(size_t)t * p.ldo + o] = h;
-                        }
-                    }
-                } else if (row < p.n_out) {
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) {
-                        const int t = t0 + c0 + i;
-                        if (t >= p.T) break;
-                        if (p.outb) p.outb[(size_t)t * p.ldo + row] = __float2bfloat16_rn(__int_as_float(v[i]));
-                        else p.out[(size_t)t * p.ldo + row] = __int_as_float(v[i]);
-                    }
-                }
-            }
-        }
+        if (__all_sync(0xffffffffu, ok)) read_out<128>(p, tmem, row0, t0, warp & 3, lane);
     }
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
     if (warp == 1) tmem_dealloc(tmem, 128);
+}
+
+// ---- 128 x 256 tiles, one CTA per SM over its share of them
+constexpr int LW_STAGES = 4, LW_STAGE = 3 * LT_TILE;       // 128 weight rows and 256 token rows of 64 columns
+constexpr size_t LW_SMEM = (size_t)LW_STAGES * LW_STAGE + 1024;
+
+__global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_constant__ CUtensorMap wmap,
+                                                                  const __grid_constant__ CUtensorMap xmap, const LtParams p, int row_tiles,
+                                                                  int tok_tiles) {
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t s_bar[2 * LW_STAGES + 4];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_give_up;
+    const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+    const uint32_t full = smem_u32(s_bar), empty = full + 8 * LW_STAGES, acc_full = empty + 8 * LW_STAGES, acc_free = acc_full + 16;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int nk = (p.K + 63) / 64, total = row_tiles * tok_tiles;
+    volatile int* give_up = &s_give_up;
+    if (warp == 1) {
+        tmem_alloc(smem_u32(&s_tmem), 512);
+        tmem_relinquish();
+    }
+    if (tid == 0) {
+        s_give_up = 0;
+        for (int i = 0; i < LW_STAGES; ++i) {
+            mbar_init(full + 8 * i, 1);
+            mbar_init(empty + 8 * i, 1);
+        }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(acc_full + 8 * i, 1);
+            mbar_init(acc_free + 8 * i, 128);
+        }
+        mbar_fence_init();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s_tmem;
+    pdl_launch_dependents();
+    pdl_wait();
+    // Every role walks the same tiles; stages are counted on across tiles.
+    if (warp == 0) {
+        if (lane == 0) {
+            int issued = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
+                const int row0 = tile / tok_tiles * 128, t0 = tile % tok_tiles * 256;
+                for (int k = 0; k < nk; ++k, ++issued) {
+                    const int s = issued % LW_STAGES, use = issued / LW_STAGES;
+                    if (use > 0 && !tc_wait_raw(empty + 8 * s, (use - 1) & 1, give_up, p.err)) {
+                        ok = false;
+                        break;
+                    }
+                    const uint32_t to = base + s * LW_STAGE;
+                    mbar_expect_tx(full + 8 * s, LW_STAGE);
+                    tma_load_2d(to, &wmap, k * 64, row0, full + 8 * s);
+                    tma_load_2d(to + LT_TILE, &xmap, k * 64, t0, full + 8 * s);
+                    tma_load_2d(to + 2 * LT_TILE, &xmap, k * 64, t0 + 128, full + 8 * s);
+                }
+            }
+            // no copy may still be in flight when the CTA leaves (at once unless someone gave up)
+            for (int s = 0; s < LW_STAGES; ++s) {
+                const int uses = (issued - s + LW_STAGES - 1) / LW_STAGES;
+                if (issued > s)
+                    for (uint32_t i = 0; i < DC_WAIT_LIMIT && !mbar_try_wait(full + 8 * s, (uses - 1) & 1); ++i) {}
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc = umma_idesc_bf16(128, 256);
+            int it = 0, j = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x, ++j) {
+                const int set = j & 1;
+                if (j >= 2 && !tc_wait_raw(acc_free + 8 * set, ((j >> 1) - 1) & 1, give_up, p.err)) break;
+                tc_fence_after();
+                for (int k = 0; k < nk; ++k, ++it) {
+                    const int s = it % LW_STAGES;
+                    if (!tc_wait_raw(full + 8 * s, (it / LW_STAGES) & 1, give_up, p.err)) {
+                        ok = false;
+                        break;
+                    }
+                    tc_fence_after();
+                    const uint32_t a = base + s * LW_STAGE, b = a + LT_TILE;
+#pragma unroll
+                    for (int q = 0; q < 4; ++q)
+                        umma_f16(tmem + 256 * set, umma_desc_sw128(a + 32 * q, 1024), umma_desc_sw128(b + 32 * q, 1024), idesc, k > 0 || q > 0);
+                    umma_commit(empty + 8 * s);
+                }
+                umma_commit(acc_full + 8 * set);
+            }
+        }
+    } else {
+        int j = 0;
+        for (int tile = blockIdx.x; tile < total; tile += gridDim.x, ++j) {
+            const int set = j & 1;
+            const bool ok = tc_wait_raw(acc_full + 8 * set, (j >> 1) & 1, give_up, p.err) && !*give_up;
+            tc_fence_after();
+            if (!__all_sync(0xffffffffu, ok)) break;
+            read_out<256>(p, tmem + 256 * set, tile / tok_tiles * 128, tile % tok_tiles * 256, warp & 3, lane);
+            tc_fence_before();
+            mbar_arrive(acc_free + 8 * set);
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 1) tmem_dealloc(tmem, 512);
 }
 
 typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
@@ -159,9 +274,16 @@ int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int 
 
 int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, int epi, float* out, __nv_bfloat16* outb, int ldo) {
     if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: inner sizes %d and %d differ", w.K, x.K);
-    int st = dc_kernel_setup(ctx, (const void*)k_linear_tc, (int)LT_SMEM, "k_linear_tc");
-    if (st != DC_B200_OK) return st;
     LtParams p = {w.K, T, epi == DC_LIN_GELU_PAIR ? w.N / 2 : w.N, ldo, epi, out, outb, ctx->d_err};
     if (p.n_out > ldo) p.n_out = ldo;
+    const int row_tiles = (w.N + 127) / 128, tok_tiles = (T + 255) / 256, tiles = row_tiles * tok_tiles;
+    if (T > 128 && tiles >= ctx->num_sms / 2) {
+        int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide, (int)LW_SMEM, "k_linear_tc_wide");
+        if (st != DC_B200_OK) return st;
+        return dc_launch(ctx, "k_linear_tc_wide", k_linear_tc_wide, dim3(tiles < ctx->num_sms ? tiles : ctx->num_sms), dim3(LT_THREADS), LW_SMEM, w.map,
+                         x.map, p, row_tiles, tok_tiles);
+    }
+    int st = dc_kernel_setup(ctx, (const void*)k_linear_tc, (int)LT_SMEM, "k_linear_tc");
+    if (st != DC_B200_OK) return st;
     return dc_launch(ctx, "k_linear_tc", k_linear_tc, dim3((w.N + 127) / 128, (T + 127) / 128), dim3(LT_THREADS), LT_SMEM, w.map, x.map, p);
 }

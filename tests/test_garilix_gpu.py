@@ -445,3 +445,13 @@ def test_generate_command(stack):
                        input="\n".join(",".join(map(str, p)) for p in ps), capture_output=True, text=True, timeout=300, cwd=root)
     assert r.returncode == 0, r.stderr
     assert [[int(t) for t in ln.split()] for ln in r.stdout.splitlines()] == [R.greedy(stack.cfg, stack.tensors, p, 6) for p in ps]
+
+
+@pytest.mark.parametrize("n", [300, 700])
+def test_large_products(ctx, tmp_path, n):
+    """Enough rows and tokens for the wide tensor-core tiles (more tiles than SMs at the larger size), odd edges included."""
+    c = Case(tmp_path, config([mamba(heads=20, vdim=40, state=16, groups=2, norm_groups=2), delta(heads=8, dim=32, vdim=64)], width=776, vocab=300, ff=[6500, 3000]),
+             n=n, seed=3)
+    m = c.model(ctx, "bfloat16", max_seqs=1, max_ctx=1024)
+    assert close(run(m, c.tokens, [n]), c.want, "bfloat16")
+    m.close()
