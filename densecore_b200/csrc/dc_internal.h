@@ -97,8 +97,8 @@ int dc_launch_gemm_tc_multi(dc_ctx* ctx, const dc_weight* const* ws, const int* 
 
 
 // ---- misc.cu ----
-// ldx (0: the row length) and xb (a bf16 copy) are optional
-int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x, int ldx = 0, __nv_bfloat16* xb = nullptr);
+// rows times scale; ldx (0: the row length) and xb (a bf16 copy) are optional
+int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x, int ldx = 0, __nv_bfloat16* xb = nullptr, float scale = 1.0f);
 // x (+= add) -> RMSNorm * w -> optional f32 copy and Q8_K blocks
 int dc_launch_rmsnorm_q8k(dc_ctx* ctx, float* x, const float* add, const float* w, int T, int H, float eps,
                           float* xn_out, uint8_t* q8_out);

@@ -4,6 +4,9 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "dc_common.cuh"
+#include "dc_stack.h"
+
 namespace dc {
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -55,6 +58,110 @@ __device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 __device__ __forceinline__ float load_as(const float* p) { return *p; }
 __device__ __forceinline__ float load_as(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+// ---- epilogues of the products (dc_lin_epi)
+__device__ __forceinline__ float pair_value(const dc_lin_epi& e, float gate, float up) {
+    if (e.pair_kind == DC_PAIR_GELU) return gelu_tanh(gate) * up;
+    gate = fminf(gate, e.limit);
+    up = fminf(fmaxf(up, -e.limit), e.limit);
+    return gate * sigmoid(1.702f * gate) * (up + 1.0f);
+}
+__device__ __forceinline__ void put_pair(const dc_lin_epi& e, int t, int pair, float v) {
+    const size_t at = (size_t)t * e.ldp + pair;
+    if (e.poutb) e.poutb[at] = __float2bfloat16_rn(v);
+    else e.pout[at] = v;
+}
+// returns the stored value
+__device__ __forceinline__ float put_row(const dc_lin_epi& e, int t, int row, float v) {
+    if (e.bias) v += e.bias[row];
+    if (row < e.silu_rows) v = silu(v);
+    const size_t at = (size_t)t * e.ldo + row;
+    if (e.outb) {
+        e.outb[at] = __float2bfloat16_rn(v);
+    } else {
+        if (e.add) v += e.out[at];
+        e.out[at] = v;
+    }
+    return v;
+}
+
+// ---- blocks of B tokens that entries are cut into from their own start
+struct BlockRef {
+    int e, t0, n;
+};
+template <int B>
+__device__ __forceinline__ int block_base(const int32_t* starts, int e) {
+    int b = 0;
+    for (int i = 0; i < e; ++i) b += (starts[i + 1] - starts[i] + B - 1) / B;
+    return b;
+}
+template <int B>
+__device__ __forceinline__ BlockRef block_at(const int32_t* starts, int E, int blk) {
+    for (int e = 0; e < E; ++e) {
+        const int n = starts[e + 1] - starts[e], nb = (n + B - 1) / B;
+        if (blk < nb) return BlockRef{e, starts[e] + blk * B, min(B, n - blk * B)};
+        blk -= nb;
+    }
+    return BlockRef{0, 0, 0};
+}
+// ---- cached rows of a sequence's tokens
+__device__ __forceinline__ int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
+
+struct CacheRef {
+    void* arena;
+    const int32_t* tables;
+    int max_blocks, row;     // row: elements per cached token
+    __device__ size_t at(int seq, int pos) const {
+        return ((size_t)tables[(size_t)seq * max_blocks + pos / DC_KV_BLOCK] * DC_KV_BLOCK + pos % DC_KV_BLOCK) * row;
+    }
+};
+
+// ---- copies, fragments and products of the attention and chunk kernels
+__device__ __forceinline__ void unpack16(const uint4& v, float (&f)[8], __nv_bfloat16) {
+    const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        f[2 * i] = __uint_as_float(u[i] << 16);
+        f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void unpack16(const uint4& v, float (&f)[4], float) {
+    f[0] = __uint_as_float(v.x), f[1] = __uint_as_float(v.y), f[2] = __uint_as_float(v.z), f[3] = __uint_as_float(v.w);
+}
+
+__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool valid) {
+    const int bytes = valid ? 16 : 0;   // 0: the 16 bytes are zero-filled, the address is not read
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+__device__ __forceinline__ void cp_async4z(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(ok ? 4 : 0) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+
+// 2^x (the hardware's approximation, relative error about 2^-22)
+__device__ __forceinline__ float ex2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+
 // asks for a 128-byte line of global memory to be brought into L2
 __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 

@@ -11,6 +11,7 @@
 
 #include <map>
 #include <string>
+#include <tuple>
 #include <vector>
 
 #include "dc_internal.h"
@@ -19,9 +20,12 @@
 
 struct dc_model;
 
-enum { DC_MIX_DELTA = 0, DC_MIX_LATENT = 1, DC_MIX_SSD = 2 };
+enum { DC_MIX_DELTA = 0, DC_MIX_LATENT = 1, DC_MIX_SSD = 2, DC_MIX_GQA = 3, DC_MIX_LIGHTNING = 4 };
 enum { DC_DTYPE_BF16 = 0, DC_DTYPE_F32 = 1 };
-enum { DC_LIN_STORE = 0, DC_LIN_GELU_PAIR = 1 };
+// How a layer's sublayers meet the residual.  POST_NORM: x += norm1(mixer(x)), then x += norm2(ff(x)).  PARALLEL: with
+// h = norm1(x), x += mixer(h) + ff(h); the input matrices of both are one product, and so are the output matrices.
+enum { DC_BLOCK_POST_NORM = 0, DC_BLOCK_PARALLEL = 1 };
+enum { DC_PAIR_GELU = 0, DC_PAIR_CLAMPED = 1 };
 
 static inline int dc_pad8(int n) { return (n + 7) & ~7; }
 
@@ -31,6 +35,37 @@ struct dc_lin {
     __nv_bfloat16* w = nullptr;
     int N = 0, K = 0, ld = 0;
     CUtensorMap map;            // [N rows][K], box 128 x 64, 128-byte swizzle
+};
+
+// What becomes of a product's rows.  Rows below pair0 are stored (to outb if given, else to out) after the bias and, for
+// the first silu_rows of them, silu; `add` adds to what out holds.  Rows from pair0 on are gate and up rows in turn
+// and each pair is one value of poutb / pout: gelu_tanh(gate) up, or with both clamped (gate from above only)
+// gate sigmoid(1.702 gate) (up + 1).
+#define DC_PAIR_ALIGN 32        // pair0 is a multiple of this
+struct dc_lin_epi {
+    float* out = nullptr;
+    __nv_bfloat16* outb = nullptr;
+    int ldo = 0, n_store = 0;   // rows stored: at most n_store (launchers: also at most the matrix' rows)
+    const float* bias = nullptr;
+    int silu_rows = 0;
+    bool add = false;
+    int pair0 = 1 << 30, pair_kind = DC_PAIR_GELU;
+    float limit = 0.0f;
+    float* pout = nullptr;
+    __nv_bfloat16* poutb = nullptr;
+    int ldp = 0, n_pairs = 0;
+    unsigned long long* keys = nullptr;      // packed greedy picks per token (products of up to DC_MAX_T tokens)
+
+    static dc_lin_epi store(float* out, __nv_bfloat16* outb, int ldo, unsigned long long* keys = nullptr) {
+        dc_lin_epi e;
+        e.out = out, e.outb = outb, e.ldo = e.n_store = ldo, e.keys = keys;
+        return e;
+    }
+    dc_lin_epi& pairs(int row0, int kind, float clamp, float* o, __nv_bfloat16* ob, int ld, int n) {
+        pair0 = row0, pair_kind = kind, limit = clamp, pout = o, poutb = ob, ldp = ld, n_pairs = n;
+        if (n_store > row0) n_store = row0;
+        return *this;
+    }
 };
 
 // Input of a tensor-core product: a bf16 buffer [rows][ld] with the tensor map that reads its first K columns.
@@ -72,11 +107,52 @@ struct dc_latent_mixer {        // attention over a compressed key/value latent 
     int range = 0;              // which of the step's key ranges (distinct windows)
 };
 
+// Rotary angles: pair i of `dims` turns by pos * f_i with f_i = base^(-2i / dims).  YaRN (factor > 0): pairs that turn
+// less than `slow` times over `original` positions turn slower by the factor, those above `fast` turns are left alone,
+// linear in between; cos and sin are multiplied by 0.1 ln(factor) + 1.
+struct dc_rotation {
+    int dims = 0;
+    double base = 10000.0, factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;
+    bool operator<(const dc_rotation& o) const {
+        return std::tie(dims, base, factor, original, fast, slow) < std::tie(o.dims, o.base, o.factor, o.original, o.fast, o.slow);
+    }
+};
+
+struct dc_gqa_mixer {           // grouped-query attention; the values are the key projection before norm and rotation
+    int heads = 0, kv_heads = 0, dim = 0, window = 0;      // window 0: every earlier token
+    float scale = 1.0f;
+    bool sink = false;          // a term of the softmax' denominator with score sink_score and no value
+    float sink_score = 0.0f;
+    dc_rotation rot;
+    int off_q = 0, off_k = 0, dim_p = 0;    // projection rows; dim_p: padded head size of the cached rows
+    float *bias = nullptr;      // of the projection rows
+    float *q_norm = nullptr, *k_norm = nullptr;             // over all heads at once
+    const float* cos_sin = nullptr;
+    int plane = -1, row = 0;    // row: k heads, then v heads, dim_p each
+    int range = 0;
+};
+
+struct dc_lightning_mixer {     // linear attention with one constant decay per head: S <- decay S + k v^T, o = S^T q
+    int heads = 0, dim = 0, vdim = 0;
+    int off_q = 0, off_k = 0, off_v = 0, off_g = 0;         // q, k, v pass through silu
+    std::vector<float> decays;  // one per head, from the configuration
+    float *decay = nullptr;     // their device copy
+    float *norm = nullptr;      // [heads * vdim]: all heads are normed together, then gated by sigmoid(g)
+};
+
 struct dc_stack_layer {
     int kind = DC_MIX_DELTA;
     dc_delta_mixer dl;
     dc_ssd_mixer ssd;
     dc_latent_mixer la;
+    dc_gqa_mixer ga;
+    dc_lightning_mixer li;
+    // parallel blocks: mixer rows, then (from pair0) gate and up rows in turn; mixer columns, then (from out_ff) the
+    // feed-forward's
+    dc_lin in, out;
+    int pair0 = 0, out_ff = 0;
+    float* out_bias = nullptr;
+    float limit = 0.0f;         // of the clamped pairs
     size_t state_off = 0, ring_off = 0;   // byte offsets in a sequence's state slot
     int ff = 0;                 // 0: no feed-forward
     dc_lin gate_up, down;       // gate_up: rows 2i = gate row i, 2i + 1 = up row i
@@ -90,6 +166,7 @@ struct dc_stack_tensor {
     dc_lin* lin = nullptr;
     int row0 = 0, row_step = 1; // destination row of tensor row i: row0 + i * row_step (head_rows 0) ...
     int head_rows = 0, head_pad = 0;      // ... or row0 + (i / head_rows) * head_pad + i % head_rows
+    int col0 = 0;               // destination column
     float** vec = nullptr;
     int64_t vec_off = 0, vec_len = 0;     // destination range and the vector's whole length
     bool neg_exp = false;       // stored as -exp(value)
@@ -100,8 +177,9 @@ struct dc_stack_tensor {
 
 struct dc_stack_config {
     std::string arch;
-    int vocab = 0, width = 0;
-    float eps = 1e-5f;
+    int vocab = 0, width = 0, block = DC_BLOCK_POST_NORM;
+    float eps = 1e-5f, embed_scale = 1.0f;
+    bool tied = false;          // the output matrix is the embedding table
 };
 
 // One step's tokens on the device.  Entry e is tokens starts[e] .. starts[e + 1] - 1, consecutive positions of one
@@ -126,6 +204,9 @@ struct dc_stack_buffers {
     __nv_bfloat16 *lm_xb = nullptr, *xb = nullptr, *mixb = nullptr, *ffb = nullptr, *lowb = nullptr;
     __nv_bfloat16 *keys_c = nullptr, *keys_r = nullptr, *keys_kv = nullptr;
     float *qa = nullptr, *part = nullptr, *part_ml = nullptr;
+    float* q = nullptr;         // grouped-query attention: turned queries (qb: bf16, prompts)
+    __nv_bfloat16 *qb = nullptr, *actb = nullptr;
+    float* chunk_state = nullptr;        // linear attention: the state ahead of every chunk
     std::vector<void*> owned;
 };
 #define DC_STACK_META_SLOTS 4
@@ -141,7 +222,7 @@ struct dc_stack {
     std::map<std::string, int> index;
     std::vector<void*> owned;   // weight memory
     size_t weight_bytes = 0;
-    std::map<std::pair<double, int>, float*> rot;    // (base, dims) -> cos/sin table
+    std::map<dc_rotation, float*> rot;   // cos/sin tables [max_ctx][dims / 2][2]
     std::vector<int> windows;   // distinct windows of the attention layers
     int splits = 1;             // key splits of a decode step's attention
     dc_stack_buffers b;
@@ -166,15 +247,13 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
 void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token);
 
 // ---- linear.cu / linear_tc.cu: y = W x
-// T <= DC_MAX_T tokens, bf16 or f32 inputs: one pass over the weights.  keys: packed greedy picks per token.
-int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, int epi, float* out, __nv_bfloat16* outb, int ldo,
-                         unsigned long long* keys = nullptr);
-int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo,
-                          unsigned long long* keys = nullptr);
+// T <= DC_MAX_T tokens, bf16 or f32 inputs: one pass over the weights
+int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, const dc_lin_epi& epi);
+int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, const dc_lin_epi& epi);
 // any T, f32 inputs (f32 models)
-int dc_launch_linear_f32(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo);
-// any T, bf16 inputs on the tensor cores; exactly one of out / outb is used
-int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, int epi, float* out, __nv_bfloat16* outb, int ldo);
+int dc_launch_linear_f32(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, const dc_lin_epi& epi);
+// any T, bf16 inputs on the tensor cores
+int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, const dc_lin_epi& epi);
 int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int rows, int K, int ld);
 
 // ---- norm_act.cu
@@ -205,6 +284,39 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
 int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y, int ldy,
                          float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps);
+
+// lightning attention.  decode: one token per sequence.  scan: entries of any length in f32 (blocks of sixteen tokens).
+// act: q, k and v after silu and the gate's input, columns off_q ..; y: the states' answers [T][ldy], all heads.
+size_t dc_lightning_block_floats(const dc_lightning_mixer& m);
+int dc_launch_lightning_decode(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act,
+                               const __nv_bfloat16* actb, int lda, float* y, int ldy);
+int dc_launch_lightning_scan(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act, int lda,
+                             float* blk, float* y, int ldy);
+// y / rms(y) * norm * sigmoid(gate) over all heads
+int dc_launch_lightning_norm(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const float* y, int ldy, const float* act,
+                             const __nv_bfloat16* actb, int lda, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
+// ---- mix_lightning.cu: the same for entries of bf16 models on the tensor cores, in chunks of 64 tokens
+int dc_lightning_chunks(int T, int E);       // most chunks that T tokens of E entries make
+int dc_launch_lightning_chunks(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const dc_state_ref& sr, const __nv_bfloat16* act,
+                               int lda, float* chunk_state, float* y, int ldy);
+
+// ---- mix_gqa.cu
+struct dc_gqa_cache {
+    void* arena = nullptr;      // [block][DC_KV_BLOCK][row], bf16 or f32
+    bool f32 = false;
+    const int32_t* tables = nullptr;
+    int max_blocks = 0;
+};
+static inline int dc_gqa_ldq(const dc_gqa_mixer& m) { return (m.dim + 15) & ~15; }      // pitch of a turned query
+// norms, rotation, cache rows of the step's tokens; queries to q or qb [T][heads][dc_gqa_ldq]
+int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
+                       int max_pos, float* q, __nv_bfloat16* qb);
+// every token alone: keys split over CTAs, then joined
+int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
+                         float* part_ml, float* mix, __nv_bfloat16* mixb, int ldm);
+// prompts of bf16 models: tiles of queries over the cached rows
+int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const int32_t* tiles, int n_tiles,
+                         const __nv_bfloat16* qb, __nv_bfloat16* mixb, int ldm);
 
 // ---- mix_latent.cu
 struct dc_latent_cache {

@@ -8,8 +8,10 @@
 // ahead of the dependency wait.  k_linear_f32 (any number of tokens, f32 models) is a 64 x 64 shared-memory tile
 // product.
 //
-// Epilogues: store; or tanh-gelu of the even rows times the odd rows (gate and up rows interleaved), half as many
-// outputs.  The rows kernel can also fold the greedy pick of every token into packed keys.
+// Epilogues (dc_lin_epi): store with bias and silu, add to the residual, one value per gate and up row pair; stored rows
+// can also be folded into packed greedy picks per token.
+#include <algorithm>
+
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -24,14 +26,11 @@ struct RowsParams {
     int N, K, ldw;
     const float* x;
     int ldx, T;
-    float* out;
-    int ldo;
-    int n_out;                     // rows stored (pair epilogue: pairs)
-    unsigned long long* keys;
+    dc_lin_epi e;
 };
 
 // TT: tokens (at most), R: rows of a warp, D: 16-byte loads per row that a lane keeps in flight.
-template <int TT, int R, int D, int EPI>
+template <int TT, int R, int D>
 __global__ void __launch_bounds__(LR_WARPS * 32) k_linear_rows(const RowsParams p) {
     dc::pdl_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -97,23 +96,23 @@ __global__ void __launch_bounds__(LR_WARPS * 32) k_linear_rows(const RowsParams 
             const float2 f = dc::unpair(acc2[t][r]);
             acc[t][r] = dc::warp_sum(f.x + f.y);
         }
-    if (EPI == DC_LIN_GELU_PAIR) {
+    const bool pairs = row0 >= p.e.pair0;
+    if (pairs) {
 #pragma unroll
         for (int t = 0; t < TT; ++t)
 #pragma unroll
             for (int r = 0; r < R; r += 2) {
-                const int o = (row0 + r) >> 1;
-                if (((t * R + r) / 2 & 31) == lane && live && t < p.T && o < p.n_out)
-                    p.out[(size_t)t * p.ldo + o] = dc::gelu_tanh(acc[t][r]) * acc[t][r + 1];
+                const int o = (row0 + r - p.e.pair0) >> 1;
+                if (((t * R + r) / 2 & 31) == lane && live && t < p.T && o < p.e.n_pairs) dc::put_pair(p.e, t, o, dc::pair_value(p.e, acc[t][r], acc[t][r + 1]));
             }
-        return;
+    } else {
+#pragma unroll
+        for (int t = 0; t < TT; ++t)
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+                if (((t * R + r) & 31) == lane && live && t < p.T && row0 + r < p.e.n_store) dc::put_row(p.e, t, row0 + r, acc[t][r]);
     }
-#pragma unroll
-    for (int t = 0; t < TT; ++t)
-#pragma unroll
-        for (int r = 0; r < R; ++r)
-            if (((t * R + r) & 31) == lane && live && t < p.T && row0 + r < p.n_out) p.out[(size_t)t * p.ldo + row0 + r] = acc[t][r];
-    if (!p.keys) return;
+    if (!p.e.keys) return;
     // greedy pick: the first maximum wins (key = order-preserving value bits, then the complement of the row)
     __shared__ unsigned long long best[LR_WARPS][TT];
 #pragma unroll
@@ -121,7 +120,7 @@ __global__ void __launch_bounds__(LR_WARPS * 32) k_linear_rows(const RowsParams 
         unsigned long long k = 0ull;
 #pragma unroll
         for (int r = 0; r < R; ++r)
-            if (live && row0 + r < p.n_out) {
+            if (live && row0 + r < p.e.n_store) {
                 const unsigned long long c = dc::argmax_key(acc[t][r], row0 + r);
                 k = c > k ? c : k;
             }
@@ -131,19 +130,13 @@ __global__ void __launch_bounds__(LR_WARPS * 32) k_linear_rows(const RowsParams 
     if (threadIdx.x < (unsigned)TT && (int)threadIdx.x < p.T) {
         unsigned long long k = 0ull;
         for (int w = 0; w < LR_WARPS; ++w) k = best[w][threadIdx.x] > k ? best[w][threadIdx.x] : k;
-        atomicMax(p.keys + threadIdx.x, k);
+        atomicMax(p.e.keys + threadIdx.x, k);
     }
 }
 
-template <int TT, int R, int D, int EPI>
+template <int TT, int R, int D>
 int launch_rows(dc_ctx* ctx, const RowsParams& p) {
-    return dc_launch(ctx, "k_linear_rows", k_linear_rows<TT, R, D, EPI>, dim3((p.N + LR_WARPS * R - 1) / (LR_WARPS * R)), dim3(LR_WARPS * 32), 0, p);
-}
-template <int EPI>
-int launch_rows_any(dc_ctx* ctx, const RowsParams& p) {
-    if (p.T <= 1) return launch_rows<1, 2, 4, EPI>(ctx, p);
-    if (p.T <= 4) return launch_rows<4, 2, 4, EPI>(ctx, p);
-    return launch_rows<16, 4, 1, EPI>(ctx, p);
+    return dc_launch(ctx, "k_linear_rows", k_linear_rows<TT, R, D>, dim3((p.N + LR_WARPS * R - 1) / (LR_WARPS * R)), dim3(LR_WARPS * 32), 0, p);
 }
 
 // ---- sixteen rows per CTA on the tensor cores
@@ -154,10 +147,7 @@ struct MmaParams {
     int N, K, ldw;
     const __nv_bfloat16* x;
     int ldx, T;
-    float* out;
-    __nv_bfloat16* outb;
-    int ldo, n_out;
-    unsigned long long* keys;
+    dc_lin_epi e;
 };
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -167,7 +157,7 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1
 }
 
 // NT: groups of eight tokens; AHEAD: neighbouring runs of 32 columns that a warp keeps in flight.  Column 8 q + 4 s + e of a run (q: lane % 4) is k-slot 2 q + e % 2 + 8 (e / 2) of product s.
-template <int NT, int AHEAD, int EPI>
+template <int NT, int AHEAD>
 __global__ void __launch_bounds__(LM_WARPS * 32) k_linear_mma(const MmaParams p) {
     __shared__ float red[LM_WARPS][16][8 * NT + 1];
     dc::pdl_launch_dependents();
@@ -214,32 +204,28 @@ __global__ void __launch_bounds__(LM_WARPS * 32) k_linear_mma(const MmaParams p)
         float v = 0.0f;
 #pragma unroll
         for (int w = 0; w < LM_WARPS; ++w) v += red[w][r][t];
-        if (EPI == DC_LIN_GELU_PAIR) {
+        if (row0 >= p.e.pair0) {
             const float up = __shfl_down_sync(0xffffffffu, v, 1);
-            const int o = row >> 1;
-            if (!(r & 1) && t < p.T && o < p.n_out) {
-                const float h = dc::gelu_tanh(v) * up;
-                if (p.outb) p.outb[(size_t)t * p.ldo + o] = __float2bfloat16_rn(h);
-                else p.out[(size_t)t * p.ldo + o] = h;
-            }
+            const int o = (row - p.e.pair0) >> 1;
+            if (!(r & 1) && t < p.T && o < p.e.n_pairs) dc::put_pair(p.e, t, o, dc::pair_value(p.e, v, up));
         } else {
-            const bool ok = t < p.T && row < p.n_out;
-            if (ok) p.out[(size_t)t * p.ldo + row] = v;
-            if (p.keys) {
+            const bool ok = t < p.T && row < p.e.n_store;
+            if (ok) dc::put_row(p.e, t, row, v);
+            if (p.e.keys) {
                 unsigned long long key = ok ? dc::argmax_key(v, row) : 0ull;
 #pragma unroll
                 for (int o = 8; o > 0; o >>= 1) {
                     const unsigned long long other = __shfl_xor_sync(0xffffffffu, key, o);
                     key = other > key ? other : key;
                 }
-                if (r == 0 && t < p.T) atomicMax(p.keys + t, key);
+                if (r == 0 && t < p.T) atomicMax(p.e.keys + t, key);
             }
         }
     }
 }
 
 // ---- f32 tile product: 64 weight rows x 64 tokens per CTA, 4 x 4 outputs per thread
-__global__ void __launch_bounds__(256) k_linear_f32(const RowsParams p, int epi) {
+__global__ void __launch_bounds__(256) k_linear_f32(const RowsParams p) {
     dc::pdl_launch_dependents();
     dc::pdl_wait();
     __shared__ float sw[16][68], sx[16][68];
@@ -268,52 +254,53 @@ __global__ void __launch_bounds__(256) k_linear_f32(const RowsParams p, int epi)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         if (t0 + tt + i >= p.T) continue;
-        float* o = p.out + (size_t)(t0 + tt + i) * p.ldo;
-        if (epi == DC_LIN_GELU_PAIR) {
+        if (n0 + tn >= p.e.pair0) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
-                const int c = (n0 + tn + j) >> 1;
-                if (c < p.n_out) o[c] = dc::gelu_tanh(acc[i][j]) * acc[i][j + 1];
+                const int c = (n0 + tn + j - p.e.pair0) >> 1;
+                if (c < p.e.n_pairs) dc::put_pair(p.e, t0 + tt + i, c, dc::pair_value(p.e, acc[i][j], acc[i][j + 1]));
             }
         } else {
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-                if (n0 + tn + j < p.n_out) o[n0 + tn + j] = acc[i][j];
+                if (n0 + tn + j < p.e.n_store) dc::put_row(p.e, t0 + tt + i, n0 + tn + j, acc[i][j]);
         }
     }
 }
 
 template <int NT, int AHEAD>
-int launch_mma_any(dc_ctx* ctx, const MmaParams& p, bool gelu) {
-    const dim3 grid((p.N + 15) / 16), block(LM_WARPS * 32);
-    return gelu ? dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD, DC_LIN_GELU_PAIR>, grid, block, 0, p)
-                : dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD, DC_LIN_STORE>, grid, block, 0, p);
+int launch_mma(dc_ctx* ctx, const MmaParams& p) {
+    return dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD>, dim3((p.N + 15) / 16), dim3(LM_WARPS * 32), 0, p);
 }
+
+dc_lin_epi clipped(const dc_lin& w, dc_lin_epi e) {
+    e.n_store = std::min(e.n_store, std::min(w.N, e.pair0));
+    e.n_pairs = std::max(0, std::min(e.n_pairs, (w.N - e.pair0) / 2));
+    return e;
+}
+bool epi_ok(const dc_lin_epi& e) { return e.pair0 >= (1 << 30) || e.pair0 % DC_PAIR_ALIGN == 0; }
 
 }  // namespace
 
-int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, int epi, float* out, __nv_bfloat16* outb, int ldo,
-                         unsigned long long* keys) {
-    if (T < 1 || T > DC_MAX_T || ((uintptr_t)x & 15) || (ldx & 7) || (w.N & 7)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_mma: bad operand");
-    const bool gelu = epi == DC_LIN_GELU_PAIR;
-    MmaParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, out, outb, ldo, gelu ? w.N / 2 : w.N, keys};
-    if (p.n_out > ldo) p.n_out = ldo;
+int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, const dc_lin_epi& epi) {
+    if (T < 1 || T > DC_MAX_T || ((uintptr_t)x & 15) || (ldx & 7) || (w.N & 7) || !epi_ok(epi)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_mma: bad operand");
+    MmaParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, clipped(w, epi)};
     // a small matrix needs more of it in flight per warp, a large one has enough warps
     const bool small = (w.N + 15) / 16 <= 2 * ctx->num_sms;
-    if (T <= 8) return small ? launch_mma_any<1, 4>(ctx, p, gelu) : launch_mma_any<1, 2>(ctx, p, gelu);
-    return small ? launch_mma_any<2, 4>(ctx, p, gelu) : launch_mma_any<2, 2>(ctx, p, gelu);
+    if (T <= 8) return small ? launch_mma<1, 4>(ctx, p) : launch_mma<1, 2>(ctx, p);
+    return small ? launch_mma<2, 4>(ctx, p) : launch_mma<2, 2>(ctx, p);
 }
 
-int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo, unsigned long long* keys) {
-    if (T < 1 || T > DC_MAX_T || ((uintptr_t)x & 15) || (ldx & 3)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_rows: bad operand");
-    RowsParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, out, ldo, epi == DC_LIN_GELU_PAIR ? ldo : w.N, keys};
-    if (p.n_out > ldo) p.n_out = ldo;
-    if (epi == DC_LIN_GELU_PAIR) return launch_rows_any<DC_LIN_GELU_PAIR>(ctx, p);
-    return launch_rows_any<DC_LIN_STORE>(ctx, p);
+int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, const dc_lin_epi& epi) {
+    if (T < 1 || T > DC_MAX_T || ((uintptr_t)x & 15) || (ldx & 3) || !epi_ok(epi)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_rows: bad operand");
+    RowsParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, clipped(w, epi)};
+    if (T <= 1) return launch_rows<1, 2, 4>(ctx, p);
+    if (T <= 4) return launch_rows<4, 2, 4>(ctx, p);
+    return launch_rows<16, 4, 1>(ctx, p);
 }
 
-int dc_launch_linear_f32(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, int epi, float* out, int ldo) {
-    RowsParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, out, ldo, epi == DC_LIN_GELU_PAIR ? ldo : w.N, nullptr};
-    if (p.n_out > ldo) p.n_out = ldo;
-    return dc_launch(ctx, "k_linear_f32", k_linear_f32, dim3((w.N + 63) / 64, (T + 63) / 64), dim3(256), 0, p, epi);
+int dc_launch_linear_f32(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, const dc_lin_epi& epi) {
+    if (!epi_ok(epi)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_f32: bad operand");
+    RowsParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, clipped(w, epi)};
+    return dc_launch(ctx, "k_linear_f32", k_linear_f32, dim3((w.N + 63) / 64, (T + 63) / 64), dim3(256), 0, p);
 }

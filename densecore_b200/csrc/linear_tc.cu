@@ -9,6 +9,8 @@
 // out; the wider tile reads shared memory less often per product.  Both let the next kernel start only after every
 // CTA has its tensor memory.  Columns beyond K and rows beyond the matrix are the zeros that TMA fills in.  Every wait is
 // bounded; a CTA that gives up drains its copies, frees its tensor memory and leaves.
+#include <algorithm>
+
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -24,9 +26,8 @@ constexpr int LT_THREADS = 192;
 constexpr size_t LT_SMEM = (size_t)LT_STAGES * 2 * LT_TILE + 1024;
 
 struct LtParams {
-    int K, T, n_out, ldo, epi;
-    float* out;
-    __nv_bfloat16* outb;
+    int K, T;
+    dc_lin_epi e;
     int* err;
 };
 
@@ -38,28 +39,33 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
         int v[16];
         tmem_ld16(tmem + ((uint32_t)(32 * quarter) << 16) + c0, v);
         tmem_ld_wait();
-        if (p.epi == DC_LIN_GELU_PAIR) {
+        if (row0 + 32 * quarter >= p.e.pair0) {
             // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
             const bool up = lane & 1;
-            const int o = row >> 1;
+            const int o = (row - p.e.pair0) >> 1;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
                 const float mine = __int_as_float(up ? v[i + 8] : v[i]);
-                const float h = up ? gelu_tanh(got) * mine : gelu_tanh(mine) * got;
+                const float h = up ? pair_value(p.e, got, mine) : pair_value(p.e, mine, got);
                 const int t = t0 + c0 + i + (up ? 8 : 0);
-                if (t < p.T && o < p.n_out) {
-                    if (p.outb) p.outb[(size_t)t * p.ldo + o] = __float2bfloat16_rn(h);
-                    else p.out[(size_t)t * p.ldo + o] = h;
-                }
+                if (t < p.T && o < p.e.n_pairs) put_pair(p.e, t, o, h);
             }
-        } else if (row < p.n_out) {
+        } else if (row < p.e.n_store) {
+            float old[16];
+            if (p.e.add) {           // every load ahead of the stores
+#pragma unroll
+                for (int i = 0; i < 16; ++i) old[i] = p.e.out[(size_t)min(t0 + c0 + i, p.T - 1) * p.e.ldo + row];
+            }
+            const float bias = p.e.bias ? p.e.bias[row] : 0.0f;
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
                 const int t = t0 + c0 + i;
                 if (t >= p.T) break;
-                if (p.outb) p.outb[(size_t)t * p.ldo + row] = __float2bfloat16_rn(__int_as_float(v[i]));
-                else p.out[(size_t)t * p.ldo + row] = __int_as_float(v[i]);
+                float r = __int_as_float(v[i]) + bias;
+                if (row < p.e.silu_rows) r = silu(r);
+                if (p.e.outb) p.e.outb[(size_t)t * p.e.ldo + row] = __float2bfloat16_rn(r);
+                else p.e.out[(size_t)t * p.e.ldo + row] = p.e.add ? old[i] + r : r;
             }
         }
     }
@@ -272,10 +278,12 @@ int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int 
     return r == CUDA_SUCCESS ? DC_B200_OK : dc_fail(ctx, DC_B200_BACKEND_ERROR, "cuTensorMapEncodeTiled failed (%d) for %d x %d, pitch %d", (int)r, rows, K, ld);
 }
 
-int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, int epi, float* out, __nv_bfloat16* outb, int ldo) {
+int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, const dc_lin_epi& epi) {
     if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: inner sizes %d and %d differ", w.K, x.K);
-    LtParams p = {w.K, T, epi == DC_LIN_GELU_PAIR ? w.N / 2 : w.N, ldo, epi, out, outb, ctx->d_err};
-    if (p.n_out > ldo) p.n_out = ldo;
+    if (epi.keys || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: epilogue not available");
+    LtParams p = {w.K, T, epi, ctx->d_err};
+    p.e.n_store = std::min(epi.n_store, std::min(w.N, epi.pair0));
+    p.e.n_pairs = std::max(0, std::min(epi.n_pairs, (w.N - epi.pair0) / 2));
     const int row_tiles = (w.N + 127) / 128, tok_tiles = (T + 255) / 256, tiles = row_tiles * tok_tiles;
     if (T > 128 && tiles >= ctx->num_sms / 2) {
         int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide, (int)LW_SMEM, "k_linear_tc_wide");

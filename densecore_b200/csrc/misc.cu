@@ -12,7 +12,7 @@ using namespace dc;
 // d*scale*(q-32) with the order of core/src/llm/matmul/q6_small_batch.h:52-74.
 __global__ void __launch_bounds__(256) k_embed(const uint8_t* __restrict__ w, int type, int row_bytes, int H,
                                                const int32_t* __restrict__ tokens, int vocab,
-                                               float* __restrict__ x, int ldx, __nv_bfloat16* __restrict__ xb) {
+                                               float* __restrict__ x, int ldx, __nv_bfloat16* __restrict__ xb, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -56,13 +56,14 @@ __global__ void __launch_bounds__(256) k_embed(const uint8_t* __restrict__ w, in
         } else {
             v = reinterpret_cast<const float*>(row)[e];
         }
+        v *= scale;
         o[e] = v;
         if (xb) xb[(size_t)t * ldx + e] = __float2bfloat16_rn(v);
     }
 }
 
-int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x, int ldx, __nv_bfloat16* xb) {
-    k_embed<<<T, 256, 0, ctx->stream>>>(w->dev, w->type, (int)w->row_bytes, (int)w->K, tokens, (int)w->N, x, ldx ? ldx : (int)w->K, xb);
+int dc_launch_embed(dc_ctx* ctx, const dc_weight* w, const int32_t* tokens, int T, float* x, int ldx, __nv_bfloat16* xb, float scale) {
+    k_embed<<<T, 256, 0, ctx->stream>>>(w->dev, w->type, (int)w->row_bytes, (int)w->K, tokens, (int)w->N, x, ldx ? ldx : (int)w->K, xb, scale);
     return dc_check_cuda(ctx, cudaGetLastError(), "k_embed");
 }
 

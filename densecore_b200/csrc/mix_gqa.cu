@@ -1,0 +1,442 @@
+// Grouped-query attention with a sliding window, norms over the whole query and key projections, partial rotation, an
+// optional sink in the softmax' denominator, and values that are the key projection as it is (before norm and rotation).
+//
+// A cached token is one row: the turned keys of all key heads, then their values.  Steps of up to DC_MAX_T tokens and f32
+// models take every token alone (k_gqa_tokens: keys split over CTAs, k_gqa_join); prompt-sized steps of bf16 models run
+// tiles of queries over the cached rows with bf16 products (k_gqa_prompt).  Scores, weights and their sums are f32.
+#include "dc_common.cuh"
+#include "dc_launch.cuh"
+#include "dc_stack.h"
+#include "dc_stack.cuh"
+
+#define DC_TRY(expr)                       \
+    do {                                   \
+        int st_ = (expr);                  \
+        if (st_ != DC_B200_OK) return st_; \
+    } while (0)
+
+using namespace dc;
+
+namespace {
+
+// ---------------------------------------------------------------- norms, rotation, cache write
+struct PrepParams {
+    const float* proj;
+    int ldp, off_q, off_k, heads, kv_heads, dim, dim_p, ldq, rot, max_pos;
+    const float *q_norm, *k_norm, *cos_sin;
+    float eps;
+    const int32_t *seq_ids, *positions;
+    CacheRef c;
+    float* q;
+    __nv_bfloat16* qb;       // instead of q
+};
+
+// One CTA per token.
+template <typename TC>
+__global__ void __launch_bounds__(256) k_gqa_prep(const PrepParams p) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, pos = min(max(p.positions[t], 0), p.max_pos - 1), Q = p.heads * p.dim, K = p.kv_heads * p.dim;
+    const float *row = p.proj + (size_t)t * p.ldp, *cs = p.cos_sin + (size_t)pos * p.rot;
+    TC* cache = reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos);
+    auto inverse_rms = [&](const float* x, int n) {
+        float ss = 0.0f;
+#pragma unroll 8
+        for (int i = threadIdx.x; i < n; i += 256) ss = fmaf(x[i], x[i], ss);
+        return 1.0f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+    };
+    // dimension pair j of a head: normed, turned within the first `rot` dimensions, zero beyond the head
+    auto turned = [&](const float* x, const float* w, float inv, int head, int j, float (&out)[2]) {
+        const int d = 2 * j, at = head * p.dim + d;
+        float u = d < p.dim ? x[at] * inv * w[at] : 0.0f, v = d + 1 < p.dim ? x[at + 1] * inv * w[at + 1] : 0.0f;
+        if (d < p.rot) {
+            const float c = cs[d], s = cs[d + 1], a = u * c - v * s;
+            v = v * c + u * s;
+            u = a;
+        }
+        out[0] = u, out[1] = v;
+    };
+    const float qi = inverse_rms(row + p.off_q, Q), ki = inverse_rms(row + p.off_k, K);
+    const int qh = p.ldq / 2, kh = p.dim_p / 2;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < p.heads * qh; i += 256) {
+        const int h = i / qh, j = i - h * qh;
+        float o[2];
+        turned(row + p.off_q, p.q_norm, qi, h, j, o);
+        const size_t at = ((size_t)t * p.heads + h) * p.ldq + 2 * j;
+        if (p.qb) *reinterpret_cast<uint32_t*>(p.qb + at) = pack_bf2(o[0], o[1]);
+        else *reinterpret_cast<float2*>(p.q + at) = make_float2(o[0], o[1]);
+    }
+    for (int i = threadIdx.x; i < p.kv_heads * kh; i += 256) {
+        const int h = i / kh, j = i - h * kh, d = 2 * j;
+        const float* v = row + p.off_k + h * p.dim + d;
+        float o[2];
+        turned(row + p.off_k, p.k_norm, ki, h, j, o);
+        TC *kd = cache + h * p.dim_p + d, *vd = kd + p.kv_heads * p.dim_p;
+        store_as(kd, o[0]);
+        store_as(kd + 1, o[1]);
+        store_as(vd, d < p.dim ? v[0] : 0.0f);
+        store_as(vd + 1, d + 1 < p.dim ? v[1] : 0.0f);
+    }
+}
+
+// ---------------------------------------------------------------- every token alone
+struct TokenParams {
+    const float* q;          // [T][heads][ldq]
+    int ldq, heads, per, groups, dim, dim_p, v_off, window, splits;
+    float scale;
+    const int32_t *seq_ids, *positions;
+    CacheRef c;
+    float *part, *part_ml;   // [T][heads][splits][dim], [T][heads][splits][2]
+};
+
+constexpr int TK_KEYS = 32, TK_HEADS = 4;
+
+// One CTA per (key split, four query heads of one key head, token): a warp is a head.  Scores: a lane is a key; sums: a
+// lane owns the value pairs lane, lane + 32, ... (VP of them).
+template <typename TC, int VP>
+__global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams p) {
+    constexpr int EPC = 16 / sizeof(TC);      // elements of a 16-byte chunk
+    extern __shared__ __align__(16) uint8_t sm[];
+    const int ldk = p.dim_p + EPC, chunks = p.dim_p / EPC;
+    float* sq = reinterpret_cast<float*>(sm);                              // [TK_HEADS][dim_p]
+    TC* sk = reinterpret_cast<TC*>(sm + (size_t)TK_HEADS * p.dim_p * 4);   // [TK_KEYS][ldk], then the values
+    TC* sv = sk + TK_KEYS * ldk;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int s = blockIdx.x, g = blockIdx.y / p.groups, t = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int in_group = (blockIdx.y % p.groups) * TK_HEADS + warp, h = g * p.per + in_group, pos = p.positions[t], seq = p.seq_ids[t];
+    const bool live = in_group < p.per;
+    const int first = first_key(pos, p.window), nk = pos - first + 1;
+    const int per = ((nk + p.splits - 1) / p.splits + TK_KEYS - 1) / TK_KEYS * TK_KEYS;
+    const int kb = first + s * per, ke = min(first + nk, kb + per);
+    if (live)
+        for (int c = lane; c < p.dim_p; c += 32) sq[warp * p.dim_p + c] = p.q[((size_t)t * p.heads + h) * p.ldq + c] * p.scale;
+    float m = -INFINITY, l = 0.0f, acc[VP][2];
+#pragma unroll
+    for (int j = 0; j < VP; ++j) acc[j][0] = acc[j][1] = 0.0f;
+    for (int k0 = kb; k0 < ke; k0 += TK_KEYS) {
+        __syncthreads();
+        const TC* src[TK_KEYS / TK_HEADS];                  // a warp's keys: all rows asked for before any arrives
+#pragma unroll
+        for (int i = 0; i < TK_KEYS / TK_HEADS; ++i)
+            src[i] = reinterpret_cast<const TC*>(p.c.arena) + p.c.at(seq, min(k0 + warp * (TK_KEYS / TK_HEADS) + i, ke - 1)) + g * p.dim_p;
+        for (int c = lane; c < 2 * chunks; c += 32) {
+            const bool val = c >= chunks;
+            const int at = (val ? c - chunks : c) * EPC;
+#pragma unroll
+            for (int i = 0; i < TK_KEYS / TK_HEADS; ++i)
+                cp_async16z(smem_u32((val ? sv : sk) + (warp * (TK_KEYS / TK_HEADS) + i) * ldk + at), src[i] + (val ? p.v_off : 0) + at, true);
+        }
+        cp_async_commit();
+        cp_async_wait<0>();
+        __syncthreads();
+        if (!live) continue;
+        float part[EPC] = {};
+        const float* q = sq + warp * p.dim_p;
+#pragma unroll 8
+        for (int c = 0; c < chunks; ++c) {
+            float f[EPC];
+            unpack16(*reinterpret_cast<const uint4*>(sk + lane * ldk + c * EPC), f, TC());
+#pragma unroll
+            for (int i = 0; i < EPC; ++i) part[i] = fmaf(f[i], q[c * EPC + i], part[i]);
+        }
+        float sc = 0.0f;
+#pragma unroll
+        for (int i = 0; i < EPC; ++i) sc += part[i];
+        if (k0 + lane >= ke) sc = -INFINITY;
+        float mx = sc;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float mn = fmaxf(m, mx), corr = expf(m - mn), pr = expf(sc - mn);
+        m = mn;
+        l = l * corr + warp_sum(pr);
+#pragma unroll
+        for (int j = 0; j < VP; ++j) acc[j][0] *= corr, acc[j][1] *= corr;
+#pragma unroll 8
+        for (int kk = 0; kk < TK_KEYS; ++kk) {
+            const float w = __shfl_sync(0xffffffffu, pr, kk);
+#pragma unroll
+            for (int j = 0; j < VP; ++j) {
+                const TC* v = sv + kk * ldk + min(2 * (lane + 32 * j), p.dim_p - 2);     // beyond the head: never stored
+                acc[j][0] = fmaf(w, load_as(v), acc[j][0]);
+                acc[j][1] = fmaf(w, load_as(v + 1), acc[j][1]);
+            }
+        }
+    }
+    if (!live) return;
+    const size_t o = ((size_t)t * p.heads + h) * p.splits + s;
+    if (lane == 0) {
+        p.part_ml[2 * o] = m;
+        p.part_ml[2 * o + 1] = l;
+    }
+#pragma unroll
+    for (int j = 0; j < VP; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int d = 2 * (lane + 32 * j) + i;
+            if (d < p.dim) p.part[o * p.dim + d] = acc[j][i];
+        }
+}
+
+// Splits of one (head, token) and the sink joined.
+__global__ void __launch_bounds__(128) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int dim,
+                                                  float sink, float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
+    __shared__ float sw[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31;
+    const size_t o = ((size_t)t * heads + h) * splits;
+    if (threadIdx.x < 32) {             // splits <= 32
+        const float m = lane < splits ? part_ml[2 * (o + lane)] : -INFINITY, l = lane < splits ? part_ml[2 * (o + lane) + 1] : 0.0f;
+        float M = fmaxf(m, sink);
+#pragma unroll
+        for (int k = 16; k > 0; k >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, k));
+        const float w = expf(m - M), L = warp_sum(l * w) + expf(sink - M);
+        sw[lane] = w / L;
+    }
+    __syncthreads();
+    for (int d = threadIdx.x; d < dim; d += 128) {
+        float v = 0.0f;
+#pragma unroll 16
+        for (int s = 0; s < splits; ++s) v = fmaf(part[(o + s) * dim + d], sw[s], v);
+        const size_t at = (size_t)t * ldm + (size_t)h * dim + d;
+        if (mixb) mixb[at] = __float2bfloat16_rn(v);
+        else mix[at] = v;
+    }
+}
+
+template <typename TC>
+int launch_tokens(dc_ctx* ctx, const TokenParams& p, int kv_heads, int T) {
+    const size_t smem = (size_t)TK_HEADS * p.dim_p * 4 + (size_t)2 * TK_KEYS * (p.dim_p * sizeof(TC) + 16);
+    const dim3 grid(p.splits, kv_heads * p.groups, T), block(TK_HEADS * 32);
+#define DC_TK(VP)                                                                                         \
+    do {                                                                                                  \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_tokens<TC, VP>, (int)smem, "k_gqa_tokens"));       \
+        return dc_launch(ctx, "k_gqa_tokens", k_gqa_tokens<TC, VP>, grid, block, smem, p);                \
+    } while (0)
+    if (p.dim <= 64) DC_TK(1);
+    if (p.dim <= 128) DC_TK(2);
+    DC_TK(4);
+#undef DC_TK
+}
+
+// ---------------------------------------------------------------- prompts
+struct PromptParams {
+    const __nv_bfloat16* q;  // [T][heads][ldq]
+    int ldq, heads, per, dim, dim_p, v_off, window;
+    float scale, sink;
+    const int32_t *seq_ids, *positions, *starts, *tiles;     // tiles: (entry, first query of the entry) pairs
+    CacheRef c;
+    __nv_bfloat16* out;
+    int ldm;
+};
+
+constexpr int PK = 64;           // keys per tile
+
+// One CTA per (PQ queries of one entry, head), sixteen queries a warp; key and value tiles in a ring of ST stages.
+// DP: head size, padded.
+template <int DP, int PQ, int ST>
+__global__ void __launch_bounds__(2 * PQ) k_gqa_prompt(const PromptParams p) {
+    constexpr int LD = DP + 8, NT = 2 * PQ, CH = DP / 8;
+    extern __shared__ __align__(16) uint8_t smem[];
+    __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);     // [PQ][LD]
+    __nv_bfloat16* sK = sQ + PQ * LD;                               // [ST][PK][LD]
+    __nv_bfloat16* sV = sK + ST * PK * LD;                          // [ST][PK][LD]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, head = blockIdx.y;
+    const int tile0 = (int)(gridDim.x - 1 - blockIdx.x);           // later queries see more keys: they start first
+    const int e = p.tiles[2 * tile0], q0 = p.tiles[2 * tile0 + 1];
+    if (q0 % PQ) return;                                            // tiles are listed per DC_LATENT_QTILE queries
+    const int t0 = p.starts[e], n = p.starts[e + 1] - t0, pos0 = p.positions[t0], seq = p.seq_ids[t0];
+    const int first = first_key(pos0 + q0, p.window), last = pos0 + min(q0 + PQ, n) - 1;
+    const int n_tiles = (last - first) / PK + 1, kc = p.dim_p / 8;
+    const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.c.arena) + (head / p.per) * p.dim_p;
+
+    const int lrow = tid >> 3, lc = tid & 7;                        // eight threads per key row
+    auto load = [&](int tile, int buf) {
+#pragma unroll
+        for (int i = 0; i < PK * 8 / NT; ++i) {
+            const int key = lrow + NT / 8 * i, pos = first + tile * PK + key;
+            const bool ok = pos <= last;
+            const __nv_bfloat16* src = cache + p.c.at(seq, ok ? pos : last);
+            const uint32_t dk = smem_u32(sK + (buf * PK + key) * LD), dv = smem_u32(sV + (buf * PK + key) * LD);
+#pragma unroll
+            for (int c0 = 0; c0 < CH; c0 += 8) {
+                const int c = c0 + lc;
+                if (CH % 8 && c >= CH) break;
+                const bool in = ok && c < kc;
+                cp_async16z(dk + 16 * c, in ? src + 8 * c : src, in);
+                cp_async16z(dv + 16 * c, in ? src + p.v_off + 8 * c : src, in);
+            }
+        }
+        cp_async_commit();
+    };
+    for (int i = tid; i < PQ * CH; i += NT) {                       // the queries come with the first tile
+        const int r = i / CH, c = i - r * CH;
+        const bool in = q0 + r < n && 8 * c < p.ldq;
+        cp_async16z(smem_u32(sQ + r * LD + 8 * c), p.q + ((size_t)(t0 + q0 + (in ? r : 0)) * p.heads + head) * p.ldq + (in ? 8 * c : 0), in);
+    }
+#pragma unroll
+    for (int i = 0; i < ST - 1; ++i)
+        if (i < n_tiles) load(i, i);
+        else cp_async_commit();
+    const float sl2 = p.scale * 1.4426950408889634f, sink2 = p.sink * 1.4426950408889634f;
+    const int g = lane >> 2, t4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
+    const int qpos0 = pos0 + q0 + 16 * warp + g;
+    const int window = p.window > 0 ? p.window : 0x7fffffff;
+    float o[CH][4];
+#pragma unroll
+    for (int i = 0; i < CH; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    // the sink is the first term of the sum (one lane of a row's four counts it)
+    const bool sink = p.sink > -INFINITY;
+    float m_run[2], l_run[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) m_run[h] = sink ? sink2 : -1e30f, l_run[h] = sink && t4 == 0 ? 1.0f : 0.0f;
+
+    for (int tile = 0; tile < n_tiles; ++tile) {
+        const int buf = tile % ST, k0 = first + tile * PK;
+        cp_async_wait<ST - 2>();
+        __syncthreads();         // the tile has landed; every warp is done with the stage that the next load fills
+        if (tile + ST - 1 < n_tiles) load(tile + ST - 1, (tile + ST - 1) % ST);
+        else cp_async_commit();
+        const int wq0 = pos0 + q0 + 16 * warp;
+        if (k0 > wq0 + 15 || k0 + PK - 1 <= wq0 - window) continue;          // nothing of the tile is seen by these queries
+        float s[8][4];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+        const uint32_t qa = smem_u32(sQ + (16 * warp + (mi & 1) * 8 + r8) * LD + (mi >> 1) * 8);
+        const uint32_t ka = smem_u32(sK + (buf * PK + (mi >> 1) * 8 + r8) * LD + (mi & 1) * 8);
+#pragma unroll
+        for (int kk = 0; kk < DP; kk += 16) {
+            uint32_t a[4];
+            ldsm_x4(qa + 2 * kk, a);
+#pragma unroll
+            for (int np = 0; np < 4; ++np) {
+                uint32_t b[4];
+                ldsm_x4(ka + 2 * (16 * np * LD + kk), b);
+                mma_bf16(s[2 * np], a, b[0], b[1]);
+                mma_bf16(s[2 * np + 1], a, b[2], b[3]);
+            }
+        }
+        // the warp's sixteen queries see the whole tile, or the mask decides key by key
+        if (!(k0 + PK - 1 <= wq0 && wq0 + 15 - k0 < window)) {
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int kp = k0 + 8 * nt + 2 * t4 + (j & 1), qp = qpos0 + (j >> 1) * 8;
+                    if (!(kp <= qp && qp - kp < window)) s[nt][j] = -INFINITY;
+                }
+        }
+        float mx[2] = {-1e30f, -1e30f};
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt) {
+            mx[0] = fmaxf(mx[0], fmaxf(s[nt][0], s[nt][1]));
+            mx[1] = fmaxf(mx[1], fmaxf(s[nt][2], s[nt][3]));
+        }
+        float m_new[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+            m_new[h] = fmaxf(m_run[h], mx[h] * sl2);
+        }
+        if (__any_sync(0xffffffffu, m_new[0] > m_run[0] || m_new[1] > m_run[1])) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const float corr = ex2(m_run[h] - m_new[h]);
+                m_run[h] = m_new[h];
+                l_run[h] *= corr;
+#pragma unroll
+                for (int i = 0; i < CH; ++i) {
+                    o[i][2 * h] *= corr;
+                    o[i][2 * h + 1] *= corr;
+                }
+            }
+        }
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float w = ex2(fmaf(s[nt][j], sl2, -m_run[j >> 1]));
+                s[nt][j] = w;
+                l_run[j >> 1] += w;
+            }
+        const uint32_t va = smem_u32(sV + (buf * PK + (mi & 1) * 8 + r8) * LD + (mi >> 1) * 8);
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            uint32_t a[4];
+            a[0] = pack_bf2(s[2 * ks][0], s[2 * ks][1]);
+            a[1] = pack_bf2(s[2 * ks][2], s[2 * ks][3]);
+            a[2] = pack_bf2(s[2 * ks + 1][0], s[2 * ks + 1][1]);
+            a[3] = pack_bf2(s[2 * ks + 1][2], s[2 * ks + 1][3]);
+#pragma unroll
+            for (int dp = 0; dp < DP / 16; ++dp) {
+                uint32_t b[4];
+                ldsm_x4_t(va + 2 * (16 * ks * LD + 16 * dp), b);
+                mma_bf16(o[2 * dp], a, b[0], b[1]);
+                mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
+            }
+        }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
+        const int row = q0 + 16 * warp + g + 8 * h;
+        if (row >= n) continue;
+        const float inv = 1.0f / l_run[h];
+        __nv_bfloat16* dst = p.out + (size_t)(t0 + row) * p.ldm + (size_t)head * p.dim;
+#pragma unroll
+        for (int nt = 0; nt < CH; ++nt)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const int c = 8 * nt + 2 * t4 + j;
+                if (c < p.dim) dst[c] = __float2bfloat16_rn(o[nt][2 * h + j] * inv);
+            }
+    }
+}
+
+CacheRef cache_ref(const dc_gqa_cache& c, int row) { return CacheRef{c.arena, c.tables, c.max_blocks, row}; }
+float sink_of(const dc_gqa_mixer& m) { return m.sink ? m.sink_score : -INFINITY; }
+
+}  // namespace
+
+int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
+                       int max_pos, float* q, __nv_bfloat16* qb) {
+    PrepParams p = {proj, ldp, m.off_q, m.off_k, m.heads, m.kv_heads, m.dim, m.dim_p, dc_gqa_ldq(m), m.rot.dims, max_pos, m.q_norm, m.k_norm, m.cos_sin,
+                    eps, st.seq_ids, st.positions, cache_ref(c, m.row), q, qb};
+    if (c.f32) return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<float>, dim3(st.T), dim3(256), 0, p);
+    return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<__nv_bfloat16>, dim3(st.T), dim3(256), 0, p);
+}
+
+int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
+                         float* part_ml, float* mix, __nv_bfloat16* mixb, int ldm) {
+    const int per = m.heads / m.kv_heads;
+    TokenParams p = {q, dc_gqa_ldq(m), m.heads, per, (per + TK_HEADS - 1) / TK_HEADS, m.dim, m.dim_p, m.kv_heads * m.dim_p, m.window, splits, m.scale,
+                     st.seq_ids, st.positions, cache_ref(c, m.row), part, part_ml};
+    DC_TRY(c.f32 ? launch_tokens<float>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16>(ctx, p, m.kv_heads, st.T));
+    return dc_launch(ctx, "k_gqa_join", k_gqa_join, dim3(m.heads, st.T), dim3(128), 0, part, part_ml, m.heads, splits, m.dim, sink_of(m), mix, mixb, ldm);
+}
+
+int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const int32_t* tiles, int n_tiles,
+                         const __nv_bfloat16* qb, __nv_bfloat16* mixb, int ldm) {
+    PromptParams p = {qb, dc_gqa_ldq(m), m.heads, m.heads / m.kv_heads, m.dim, m.dim_p, m.kv_heads * m.dim_p, m.window, m.scale, sink_of(m), st.seq_ids,
+                      st.positions, st.starts, tiles, cache_ref(c, m.row), mixb, ldm};
+    const dim3 grid(n_tiles, m.heads);
+#define DC_PROMPT(DP, PQ, ST)                                                                                      \
+    do {                                                                                                           \
+        const int bytes = (PQ + 2 * ST * PK) * (DP + 8) * 2;                                                       \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_prompt<DP, PQ, ST>, bytes, "k_gqa_prompt"));                \
+        return dc_launch(ctx, "k_gqa_prompt", k_gqa_prompt<DP, PQ, ST>, grid, dim3(2 * PQ), (size_t)bytes, p);     \
+    } while (0)
+    if (m.dim <= 32) DC_PROMPT(32, 128, 3);
+    if (m.dim <= 64) DC_PROMPT(64, 128, 3);
+    if (m.dim <= 96) DC_PROMPT(96, 128, 3);
+    if (m.dim <= 128) DC_PROMPT(128, 128, 3);
+    DC_PROMPT(256, 64, 2);
+#undef DC_PROMPT
+}

@@ -21,17 +21,6 @@ using namespace dc;
 
 namespace {
 
-__device__ __forceinline__ int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
-
-struct CacheRef {
-    void* arena;
-    const int32_t* tables;
-    int max_blocks, row;     // row: elements per cached token
-    __device__ size_t at(int seq, int pos) const {
-        return ((size_t)tables[(size_t)seq * max_blocks + pos / DC_KV_BLOCK] * DC_KV_BLOCK + pos % DC_KV_BLOCK) * row;
-    }
-};
-
 // ---------------------------------------------------------------- rotation, latent norm, cache write
 struct PrepParams {
     float* proj;             // queries are turned in place
@@ -139,26 +128,6 @@ __global__ void __launch_bounds__(256) k_latent_absorb(const float* __restrict__
         if (r0 + c < rank) qa[((size_t)(tb + t) * heads + h) * ldq + r0 + c] = v;
     }
 }
-
-__device__ __forceinline__ void unpack16(const uint4& v, float (&f)[8], __nv_bfloat16) {
-    const uint32_t u[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        f[2 * i] = __uint_as_float(u[i] << 16);
-        f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
-    }
-}
-__device__ __forceinline__ void unpack16(const uint4& v, float (&f)[4], float) {
-    f[0] = __uint_as_float(v.x), f[1] = __uint_as_float(v.y), f[2] = __uint_as_float(v.z), f[3] = __uint_as_float(v.w);
-}
-
-__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool valid) {
-    const int bytes = valid ? 16 : 0;   // 0: the 16 bytes are zero-filled, the address is not read
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 struct AbsorbedParams {
     const float* qa;         // [T][heads][ldq]
@@ -364,29 +333,6 @@ __global__ void __launch_bounds__(256) k_latent_gather(CacheRef c, const int32_t
         for (int j = lane; j < rank; j += 32) kc[(size_t)i * ldc + j] = src[j];
     }
     for (int j = lane; j < ldr; j += 32) kr[(size_t)i * ldr + j] = j < rot ? src[rank + j] : __float2bfloat16_rn(0.0f);
-}
-
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&h);
-}
-
-// 2^x (the hardware's approximation, relative error about 2^-22)
-__device__ __forceinline__ float ex2(float x) {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-    return r;
 }
 
 struct PromptParams {

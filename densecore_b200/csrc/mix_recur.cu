@@ -1,5 +1,5 @@
 // Recurrent mixers: short causal convolution, gated delta rule with one decay per key channel, Mamba-2 state-space
-// scan, and their gated output norms.
+// scan, linear attention with a constant decay per head, and their gated output norms.
 //
 // Per-sequence state (f32) lives in the cache manager's state slots: the matrix S as [head][value column][key
 // channel], and the convolution's last inputs as a ring [position % taps][channel].  A sequence at position 0 starts
@@ -67,23 +67,6 @@ struct ConvRef {
 };
 
 constexpr int BT = 16, BROW = 20;                       // tokens of a block; pitch of a 16 x 16 factor (conflict-free rows)
-
-struct BlockRef {                                       // token range of a block: entries are cut from their own start
-    int e, t0, n;
-};
-__device__ __forceinline__ int block_base(const int32_t* starts, int e) {
-    int b = 0;
-    for (int i = 0; i < e; ++i) b += (starts[i + 1] - starts[i] + BT - 1) / BT;
-    return b;
-}
-__device__ __forceinline__ BlockRef block_at(const int32_t* starts, int E, int blk) {
-    for (int e = 0; e < E; ++e) {
-        const int n = starts[e + 1] - starts[e], nb = (n + BT - 1) / BT;
-        if (blk < nb) return BlockRef{e, starts[e] + blk * BT, min(BT, n - blk * BT)};
-        blk -= nb;
-    }
-    return BlockRef{0, 0, 0};
-}
 
 // The entries' last inputs into their rings (after every kernel that read the old ones).
 __global__ void __launch_bounds__(256) k_ring_update(ConvRef cr, const float* __restrict__ proj, int ldp, int off) {
@@ -174,7 +157,7 @@ __global__ void __launch_bounds__(256) k_delta_prep4(DeltaPrep p) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31, items = p.kv_heads + p.v_items, item = blockIdx.y * 8 + (threadIdx.x >> 5);
-    const BlockRef br = block_at(p.cr.starts, p.cr.E, blockIdx.x);
+    const BlockRef br = block_at<BT>(p.cr.starts, p.cr.E, blockIdx.x);
     if (br.n <= 0) return;
     if (blockIdx.y == gridDim.y - 1) {          // the step sizes and the low-rank columns
         for (int i = threadIdx.x; i < br.n * p.heads; i += 256) {
@@ -291,7 +274,8 @@ __global__ void __launch_bounds__(256) k_delta_prep4(DeltaPrep p) {
 //   S   = G_15 S0 + sum_i (P_15,i k_i) u_i
 // Everything but S0, v, u and o is shared by a head's value columns and computed once per (block, head): the decayed
 // vectors, B, and W = (I + diag(beta) A)^-1 diag(beta), so that u = W (v - S0 . G k).  Every decay factor is a
-// product of g, at most 1.  The state-space scan is the same with one decay per head, no A, and u_i = dt_i x_i.
+// product of g, at most 1.  The state-space scan is the same with one decay per head, no A, and u_i = dt_i x_i; linear
+// attention with a constant decay is that with steps of 1.
 
 // Sum of v[i] over the warp lands in lane i (31 shuffles for 32 sums).
 __device__ __forceinline__ float transpose_sum32(float (&v)[32], int lane) {
@@ -329,7 +313,7 @@ __global__ void __launch_bounds__(128) k_delta_blocks(const DeltaBlock p) {
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim, dp = p.dp;
-    const BlockRef br = block_at(p.starts, p.E, blockIdx.x);
+    const BlockRef br = block_at<BT>(p.starts, p.E, blockIdx.x);
     if (br.n <= 0) return;
     float *sk = sm, *sq = sm + BT * dim, *sg = sm + 2 * BT * dim;
     float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * delta_block_floats(dp);
@@ -420,7 +404,8 @@ constexpr int SSD_BLOCK = BT * BROW + 2 * BT;
 struct SsdBlock {
     const float* act;
     int lda, off_b, off_c, heads, per, state;
-    const float* small;          // [T][2 heads]: dt, decay
+    const float* small;          // [T][2 heads]: dt, decay; or null with
+    const float* decay;          // [heads]: a constant decay and steps of 1
     const int32_t* starts;
     int E;
     float* out;
@@ -432,7 +417,7 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
     __shared__ float sa[BT], sd[BT];
     pdl_launch_dependents();
     pdl_wait();
-    const BlockRef br = block_at(p.starts, p.E, blockIdx.x);
+    const BlockRef br = block_at<BT>(p.starts, p.E, blockIdx.x);
     if (br.n <= 0) return;
     const int g = blockIdx.y, tid = threadIdx.x, ld = p.state + 1, t = tid / BT, i = tid % BT;
     float *sb = sm, *sc = sm + BT * ld;
@@ -450,9 +435,9 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
         const int h = g * p.per + hh;
         __syncthreads();
         if (tid < BT) {
-            const float* s = p.small + (size_t)(br.t0 + tid) * 2 * p.heads;
-            sd[tid] = tid < br.n ? s[h] : 0.0f;
-            sa[tid] = tid < br.n ? s[p.heads + h] : 1.0f;
+            const float* s = p.small ? p.small + (size_t)(br.t0 + tid) * 2 * p.heads : nullptr;
+            sd[tid] = tid < br.n ? (s ? s[h] : 1.0f) : 0.0f;
+            sa[tid] = tid < br.n ? (s ? s[p.heads + h] : p.decay[h]) : 1.0f;
         }
         __syncthreads();
         float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * SSD_BLOCK;
@@ -480,7 +465,7 @@ struct ScanParams {
     const float *k, *q;            // ssd: B and C of group 0
     const float* v;                // values of head 0
     int ld, heads, per, dim, vdim;
-    const float* D;                // ssd: per head
+    const float* D;                // ssd: per head, or null
     float* o;
     int ldo;
     uint8_t* base;
@@ -488,16 +473,6 @@ struct ScanParams {
     const int32_t *seq_ids, *positions, *starts;
     int vec;                       // ssd: B, C rows allow 16-byte copies
 };
-
-__device__ __forceinline__ void cp_async4z(uint32_t dst, const void* src, bool ok) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(ok ? 4 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool ok) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // EPL consecutive-chunk channels per lane: lane's channel i is W * lane + 32 W (i / W) + i % W.
 template <int EPL>
@@ -588,7 +563,7 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     const int t0 = p.starts[e], t1 = p.starts[e + 1];
     if (t0 >= t1) return;
     const int seq = p.seq_ids[t0], blocks = (t1 - t0 + BT - 1) / BT;
-    const float* bsrc = p.blocks + ((size_t)block_base(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
+    const float* bsrc = p.blocks + ((size_t)block_base<BT>(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
     const size_t bstep = (size_t)p.heads * (DELTA ? BLK : SSD_BLOCK);
     float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 4) * p.dim;
     float s[4][EPL];             // channels Chan::at of the warp's four columns
@@ -629,7 +604,7 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
         cp_async_commit();
     };
-    const float Dh = DELTA ? 0.0f : p.D[h];
+    const float Dh = DELTA || !p.D ? 0.0f : p.D[h];
     load(0, 0);
     for (int b = 0; b < blocks; ++b) {
         if (b + 1 < blocks) {
@@ -1093,44 +1068,108 @@ __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict_
         store_as(out + (size_t)t * ldm + (size_t)h * vdim + c, r[c] * inv * w[c] * sigmoid(gate[(size_t)t * ldg + (size_t)h * vdim + c]));
 }
 
-// ssd: one CTA per (token, norm group): y silu(z) (unless gated already), over its root mean square, times w
-template <typename TO, int NT>
-__global__ void __launch_bounds__(NT) k_gate_group_norm(const float* __restrict__ y, int ldy, const float* __restrict__ z, int ldz,
+// One CTA per (token, norm group).  GATE 0: y over its root mean square, times w; 1: y silu(z) first (ssd); 2: times
+// sigmoid(z) afterwards (linear attention).
+template <int GATE, typename TZ, typename TO, int NT>
+__global__ void __launch_bounds__(NT) k_gate_group_norm(const float* __restrict__ y, int ldy, const TZ* __restrict__ z, int ldz,
                                                          const float* __restrict__ w, int n, float eps, TO* __restrict__ out, int ldm) {
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.y, c0 = blockIdx.x * n;
     const float* yr = y + (size_t)t * ldy + c0;
-    const float* zr = z ? z + (size_t)t * ldz + c0 : nullptr;
+    const TZ* zr = GATE ? z + (size_t)t * ldz + c0 : nullptr;
     constexpr int KEEP = 8;      // values per thread kept between the two passes
-    float v[KEEP], ss = 0.0f;
+    auto value = [&](int i) { return GATE == 1 ? yr[i] * silu(load_as(zr + i)) : yr[i]; };
+    float v[KEEP], g[KEEP], wv[KEEP], ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const int i = threadIdx.x + NT * j;
-        v[j] = i < n ? (zr ? yr[i] * silu(zr[i]) : yr[i]) : 0.0f;
+        v[j] = i < n ? value(i) : 0.0f;
+        if (GATE == 2) g[j] = i < n ? load_as(zr + i) : 0.0f;
+        wv[j] = i < n ? w[c0 + i] : 0.0f;
         ss = fmaf(v[j], v[j], ss);
     }
     for (int i = threadIdx.x + NT * KEEP; i < n; i += NT) {
-        const float x = zr ? yr[i] * silu(zr[i]) : yr[i];
+        const float x = value(i);
         ss = fmaf(x, x, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const int i = threadIdx.x + NT * j;
-        if (i < n) store_as(out + (size_t)t * ldm + c0 + i, v[j] * inv * w[c0 + i]);
+        if (i < n) store_as(out + (size_t)t * ldm + c0 + i, v[j] * inv * wv[j] * (GATE == 2 ? sigmoid(g[j]) : 1.0f));
     }
     for (int i = threadIdx.x + NT * KEEP; i < n; i += NT)
-        store_as(out + (size_t)t * ldm + c0 + i, (zr ? yr[i] * silu(zr[i]) : yr[i]) * inv * w[c0 + i]);
+        store_as(out + (size_t)t * ldm + c0 + i, value(i) * inv * w[c0 + i] * (GATE == 2 ? sigmoid(load_as(zr + i)) : 1.0f));
 }
 
 // small groups get small CTAs: more of them are resident
-template <typename TO>
-int launch_group_norm(dc_ctx* ctx, const float* y, int ldy, const float* z, int ldz, const float* w, int n, int groups, int T, float eps, TO* out, int ldm) {
+template <int GATE, typename TZ, typename TO>
+int launch_group_norm(dc_ctx* ctx, const float* y, int ldy, const TZ* z, int ldz, const float* w, int n, int groups, int T, float eps, TO* out, int ldm) {
     const dim3 grid(groups, T);
-    if (n <= 512) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 64>, grid, dim3(64), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
-    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 256>, grid, dim3(256), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+    if (n <= 512) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<GATE, TZ, TO, 64>, grid, dim3(64), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+    if (n <= 2048) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<GATE, TZ, TO, 256>, grid, dim3(256), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<GATE, TZ, TO, 512>, grid, dim3(512), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+}
+
+// ---------------------------------------------------------------- linear attention with a constant decay: decode
+struct LightningDecode {
+    int ld, off_q, off_k, off_v, dim, vdim;
+    const float* decay;
+    uint8_t* base;
+    size_t slot_bytes, state_off;
+    const int32_t *seq_ids, *positions;
+    float* y;
+    int ldy;
+};
+
+// One CTA per (head, 32 value columns, sequence), eight columns a warp.
+template <int EPL, typename TA>
+__global__ void __launch_bounds__(128) k_lightning_decode(const TA* __restrict__ act, const LightningDecode p) {
+    constexpr int NC = 8;
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.x, c0 = blockIdx.y * 32 + NC * warp, t = blockIdx.z;
+    const float decay = p.decay[h];
+    pdl_wait();
+    if (c0 >= p.vdim) return;
+    const int pos = p.positions[t], seq = p.seq_ids[t];
+    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + (size_t)h * p.vdim * p.dim;
+    const TA* row = act + (size_t)t * p.ld;
+    float s[NC][EPL], q[EPL], k[EPL], v[NC], a[NC];
+    load_columns<NC, EPL>(S, c0, p.vdim, p.dim, lane, pos == 0, s);
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+        const int d = Chan<EPL>::at(lane, i);
+        q[i] = d < p.dim ? load_as(row + p.off_q + (size_t)h * p.dim + d) : 0.0f;
+        k[i] = d < p.dim ? load_as(row + p.off_k + (size_t)h * p.dim + d) : 0.0f;
+    }
+#pragma unroll
+    for (int c = 0; c < NC; ++c) v[c] = load_as(row + p.off_v + (size_t)h * p.vdim + min(c0 + c, p.vdim - 1));
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        a[c] = 0.0f;
+#pragma unroll
+        for (int i = 0; i < EPL; ++i) {
+            s[c][i] = fmaf(s[c][i], decay, k[i] * v[c]);
+            a[c] = fmaf(s[c][i], q[i], a[c]);
+        }
+    }
+    store_columns<NC, EPL>(S, c0, p.vdim, p.dim, lane, s);
+    const float sum = transpose_sum8(a, lane);
+    const int mine = c0 + (lane >> 2);
+    if ((lane & 3) == 0 && mine < p.vdim) p.y[(size_t)t * p.ldy + (size_t)h * p.vdim + mine] = sum;
+}
+
+template <typename TA>
+int launch_lightning_decode(dc_ctx* ctx, const TA* act, const LightningDecode& p, int heads, int T) {
+    const dim3 grid(heads, (p.vdim + 31) / 32, T), block(128);
+    switch (key_pad(p.dim)) {
+    case 32: return dc_launch(ctx, "k_lightning_decode", k_lightning_decode<1, TA>, grid, block, 0, act, p);
+    case 64: return dc_launch(ctx, "k_lightning_decode", k_lightning_decode<2, TA>, grid, block, 0, act, p);
+    case 128: return dc_launch(ctx, "k_lightning_decode", k_lightning_decode<4, TA>, grid, block, 0, act, p);
+    default: return dc_launch(ctx, "k_lightning_decode", k_lightning_decode<8, TA>, grid, block, 0, act, p);
+    }
 }
 
 // ---------------------------------------------------------------- ssd: per-token inputs
@@ -1164,7 +1203,7 @@ __global__ void __launch_bounds__(256) k_ssd_prep4(SsdPrep p) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = blockIdx.y * 256 + threadIdx.x;
-    const BlockRef br = block_at(p.cr.starts, p.cr.E, blockIdx.x);
+    const BlockRef br = block_at<BT>(p.cr.starts, p.cr.E, blockIdx.x);
     if (br.n <= 0) return;
     if (c < p.cr.C) {
         const int i0 = br.t0 - p.cr.starts[br.e], pos0 = p.cr.positions[br.t0];
@@ -1268,7 +1307,7 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
     if (m.taps == 4) DC_TRY(dc_launch(ctx, "k_ssd_prep4", k_ssd_prep4, dim3(dc_scan_blocks(st.T, st.E), (C + 255) / 256), dim3(256), 0, s));
     else DC_TRY(dc_launch(ctx, "k_ssd_prep", k_ssd_prep, dim3((C + 255) / 256, st.T), dim3(256), 0, s));
     DC_TRY(dc_launch_ring_update(ctx, st, sr, proj, ldp, m.off_x, C, m.taps));
-    SsdBlock sb = {act, lda, inner, inner + GN, m.heads, m.heads / m.groups, m.state, small, st.starts, st.E, blk};
+    SsdBlock sb = {act, lda, inner, inner + GN, m.heads, m.heads / m.groups, m.state, small, nullptr, st.starts, st.E, blk};
     DC_TRY(dc_launch(ctx, "k_ssd_blocks", k_ssd_blocks, dim3(dc_scan_blocks(st.T, st.E), m.groups), dim3(256), (size_t)2 * BT * (m.state + 1) * 4, sb));
     ScanParams p = {};
     p.blocks = blk, p.k = act + inner, p.q = act + inner + GN, p.v = act;
@@ -1280,8 +1319,8 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
     DC_TRY(launch_scan<false>(ctx, p, st.E));
     const int n = inner / m.norm_groups;
     const float* z = proj + m.off_z;
-    return mixb ? launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
-                : launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
+    return mixb ? launch_group_norm<1>(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
+                : launch_group_norm<1>(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
 }
 
 int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
@@ -1314,6 +1353,36 @@ int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, 
     else if (dp == 128) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<4>, grid, block, smem, p));
     else DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<8>, grid, block, smem, p));
     const int n = inner / m.norm_groups;
-    return mixb ? launch_group_norm(ctx, y, ldy, nullptr, 0, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
-                : launch_group_norm(ctx, y, ldy, nullptr, 0, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
+    const float* no = nullptr;
+    return mixb ? launch_group_norm<0>(ctx, y, ldy, no, 0, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
+                : launch_group_norm<0>(ctx, y, ldy, no, 0, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
+}
+
+size_t dc_lightning_block_floats(const dc_lightning_mixer& m) { return (size_t)m.heads * SSD_BLOCK; }
+
+int dc_launch_lightning_scan(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act, int lda,
+                             float* blk, float* y, int ldy) {
+    SsdBlock sb = {act, lda, m.off_k, m.off_q, m.heads, 1, m.dim, nullptr, m.decay, st.starts, st.E, blk};
+    DC_TRY(dc_launch(ctx, "k_ssd_blocks", k_ssd_blocks, dim3(dc_scan_blocks(st.T, st.E), m.heads), dim3(256), (size_t)2 * BT * (m.dim + 1) * 4, sb));
+    ScanParams p = {};
+    p.blocks = blk, p.k = act + m.off_k, p.q = act + m.off_q, p.v = act + m.off_v;
+    p.ld = lda, p.heads = m.heads, p.per = 1, p.dim = m.dim, p.vdim = m.vdim;
+    p.o = y, p.ldo = ldy;
+    p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
+    p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
+    p.vec = m.dim % 4 == 0 && lda % 4 == 0;
+    return launch_scan<false>(ctx, p, st.E);
+}
+
+int dc_launch_lightning_decode(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act,
+                               const __nv_bfloat16* actb, int lda, float* y, int ldy) {
+    LightningDecode p = {lda, m.off_q, m.off_k, m.off_v, m.dim, m.vdim, m.decay, sr.base, sr.slot_bytes, sr.state_off, st.seq_ids, st.positions, y, ldy};
+    return actb ? launch_lightning_decode(ctx, actb, p, m.heads, st.T) : launch_lightning_decode(ctx, act, p, m.heads, st.T);
+}
+
+int dc_launch_lightning_norm(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const float* y, int ldy, const float* act,
+                             const __nv_bfloat16* actb, int lda, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
+    const int n = m.heads * m.vdim;
+    return mixb ? launch_group_norm<2>(ctx, y, ldy, actb + m.off_g, lda, m.norm, n, 1, st.T, eps, mixb, ldm)
+                : launch_group_norm<2>(ctx, y, ldy, act + m.off_g, lda, m.norm, n, 1, st.T, eps, mix, ldm);
 }

@@ -1,5 +1,5 @@
-// Norms around the sublayers of a layer-list decoder: RMS norm of a sublayer's output added to the f32 residual,
-// and the output norm on the rows whose logits are wanted.
+// Norms around the sublayers of a layer-list decoder: RMS norm of a sublayer's output added to the f32 residual;
+// RMS norm of residual rows (ahead of a layer's products, and the output norm on the rows whose logits are wanted).
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -51,21 +51,43 @@ __global__ void __launch_bounds__(256) k_post_norm(float* __restrict__ x, const 
     }
 }
 
+// Rows as above; KEEP as above.
+template <int KEEP>
 __global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, const float* __restrict__ w, const int32_t* __restrict__ rows,
                                                    int first, int H, int ld, float eps, float* __restrict__ out,
                                                    __nv_bfloat16* __restrict__ outb, int ldo) {
     __shared__ float red[33];
     dc::pdl_launch_dependents();
+    const int n4 = ld / 4;
+    float4 wv[KEEP], xv[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        wv[j] = i < n4 ? reinterpret_cast<const float4*>(w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     dc::pdl_wait();
     const int r = rows ? rows[blockIdx.x] : first + (int)blockIdx.x;
-    const float* xr = x + (size_t)r * ld;
+    const float4* x4 = reinterpret_cast<const float4*>(x + (size_t)r * ld);
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < H; i += 256) ss = fmaf(xr[i], xr[i], ss);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        xv[j] = i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) ss += (xv[j].x * xv[j].x + xv[j].y * xv[j].y) + (xv[j].z * xv[j].z + xv[j].w * xv[j].w);
     const float inv = 1.0f / sqrtf(dc::block_sum(ss, red) / (float)H + eps);
-    for (int i = threadIdx.x; i < H; i += 256) {
-        const float v = xr[i] * inv * w[i];
-        if (outb) outb[(size_t)blockIdx.x * ldo + i] = __float2bfloat16_rn(v);
-        else out[(size_t)blockIdx.x * ldo + i] = v;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        if (i >= n4) continue;
+        const float4 v = make_float4(xv[j].x * inv * wv[j].x, xv[j].y * inv * wv[j].y, xv[j].z * inv * wv[j].z, xv[j].w * inv * wv[j].w);
+        if (outb) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            reinterpret_cast<uint2*>(outb + (size_t)blockIdx.x * ldo)[i] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            reinterpret_cast<float4*>(out + (size_t)blockIdx.x * ldo)[i] = v;
+        }
     }
 }
 
@@ -82,5 +104,11 @@ int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, i
 
 int dc_launch_norm_rows(dc_ctx* ctx, const float* x, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps,
                         float* out, __nv_bfloat16* outb, int ldo) {
-    return dc_launch(ctx, "k_norm_rows", k_norm_rows, dim3(R), dim3(256), 0, x, w, rows, first, H, ld, eps, out, outb, ldo);
+    const dim3 grid(R), block(256);
+    if (ld % 8 || ldo < ld || ldo % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "norm_rows: bad pitch");
+    if (ld <= 1024) return dc_launch(ctx, "k_norm_rows", k_norm_rows<1>, grid, block, 0, x, w, rows, first, H, ld, eps, out, outb, ldo);
+    if (ld <= 2048) return dc_launch(ctx, "k_norm_rows", k_norm_rows<2>, grid, block, 0, x, w, rows, first, H, ld, eps, out, outb, ldo);
+    if (ld <= 4096) return dc_launch(ctx, "k_norm_rows", k_norm_rows<4>, grid, block, 0, x, w, rows, first, H, ld, eps, out, outb, ldo);
+    if (ld <= 8192) return dc_launch(ctx, "k_norm_rows", k_norm_rows<8>, grid, block, 0, x, w, rows, first, H, ld, eps, out, outb, ldo);
+    return dc_fail(ctx, DC_B200_UNSUPPORTED, "norm_rows: width %d is too large", H);
 }

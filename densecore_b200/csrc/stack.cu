@@ -42,11 +42,11 @@ int64_t elems(const dc_stack_tensor& t) {
 
 // Random f32 values rounded to bf16 at the tensor's place in a fused matrix.
 __global__ void k_place_rows(const float* __restrict__ src, int64_t n, int K, __nv_bfloat16* __restrict__ w, int ld, int row0, int step, int head_rows,
-                             int head_pad) {
+                             int head_pad, int col0) {
     for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
         const int r = (int)(i / K), c = (int)(i % K);
         const int64_t dst = row0 + (head_rows ? (int64_t)(r / head_rows) * head_pad + r % head_rows : (int64_t)r * step);
-        w[dst * ld + c] = __float2bfloat16_rn(src[i]);
+        w[dst * ld + col0 + c] = __float2bfloat16_rn(src[i]);
     }
 }
 
@@ -99,7 +99,7 @@ int dc_stack_set_tensor(dc_model* m, const char* name, int type, const int64_t n
         const size_t rb = (size_t)K * 2, pitch = (size_t)t.lin->ld * 2;
         const int per = t.head_rows ? t.head_rows : (int)N, blocks = (int)N / per;
         for (int b = 0; b < blocks && e == cudaSuccess; ++b)
-            e = cudaMemcpy2D(t.lin->w + (size_t)(t.row0 + b * t.head_pad) * t.lin->ld, pitch * t.row_step, (const uint8_t*)data + (size_t)b * per * rb, rb, rb,
+            e = cudaMemcpy2D(t.lin->w + (size_t)(t.row0 + b * t.head_pad) * t.lin->ld + t.col0, pitch * t.row_step, (const uint8_t*)data + (size_t)b * per * rb, rb, rb,
                              per, cudaMemcpyHostToDevice);
     }
     DC_TRY(dc_check_cuda(ctx, e, "set_tensor"));
@@ -133,7 +133,7 @@ int dc_stack_init_synthetic(dc_model* m, uint64_t seed, float sigma) {
         } else {
             const int K = (int)t.shape[1];
             __nv_bfloat16* w = t.lin ? t.lin->w : (__nv_bfloat16*)s->embed->dev;
-            k_place_rows<<<1184, 256, 0, ctx->stream>>>(tmp, n, K, w, t.lin ? t.lin->ld : K, t.row0, t.row_step, t.head_rows, t.head_pad);
+            k_place_rows<<<1184, 256, 0, ctx->stream>>>(tmp, n, K, w, t.lin ? t.lin->ld : K, t.row0, t.row_step, t.head_rows, t.head_pad, t.col0);
             st = dc_check_cuda(ctx, cudaGetLastError(), "k_place_rows");
         }
         t.loaded = true;
@@ -151,7 +151,7 @@ void dc_stack_release(dc_model* m) {
     for (auto& r : s->rot) cudaFree(r.second);
     if (s->b.h_meta) cudaFreeHost(s->b.h_meta);
     if (s->embed) {
-        if (s->embed->dev) cudaFree(s->embed->dev);
+        if (s->embed->dev && !s->cfg.tied) cudaFree(s->embed->dev);
         delete s->embed;
     }
     delete s;
@@ -159,6 +159,44 @@ void dc_stack_release(dc_model* m) {
 }
 
 // ---------------------------------------------------------------- cache, state slots, step buffers
+namespace {
+
+// The cos/sin table of a rotation, made at its first use.
+int rotation_table(dc_model* m, const dc_rotation& r, const float** out) {
+    float*& table = m->stack->rot[r];
+    if (!table) {
+        const int n = m->cfg.max_ctx, half = r.dims / 2;
+        std::vector<double> f(half);
+        double mul = 1.0, lo = 0.0, hi = 0.0;
+        if (r.factor > 0.0) {
+            // the pair that turns t times over the original context
+            auto pair_of = [&](double t) { return r.dims * log(r.original / (2.0 * M_PI * t)) / (2.0 * log(r.base)); };
+            lo = std::max(floor(pair_of(r.fast)), 0.0);
+            hi = std::min(ceil(pair_of(r.slow)), r.dims - 1.0);
+            mul = 0.1 * log(r.factor) + 1.0;
+        }
+        for (int i = 0; i < half; ++i) {
+            f[i] = pow(r.base, -2.0 * i / r.dims);
+            if (r.factor > 0.0) {
+                const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+                f[i] = f[i] / r.factor * ramp + f[i] * (1.0 - ramp);
+            }
+        }
+        std::vector<float> cs((size_t)n * r.dims);
+        for (int p = 0; p < n; ++p)
+            for (int i = 0; i < half; ++i) {
+                cs[(size_t)p * r.dims + 2 * i] = (float)(mul * cos(p * f[i]));
+                cs[(size_t)p * r.dims + 2 * i + 1] = (float)(mul * sin(p * f[i]));
+            }
+        DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)&table, cs.size() * 4), "rotation table"));
+        DC_TRY(dc_check_cuda(m->ctx, cudaMemcpy(table, cs.data(), cs.size() * 4, cudaMemcpyHostToDevice), "rotation table"));
+    }
+    *out = table;
+    return DC_B200_OK;
+}
+
+}  // namespace
+
 // Cache planes of the layers that write a latent, state slots of the recurrent layers, rotation tables.  The pool
 // holds pool_tokens tokens (0: max_ctx for every sequence).
 int dc_stack_create_cache(dc_model* m, int pool_tokens) {
@@ -174,8 +212,22 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
         return off;
     };
     int span = 1;
+    auto key_range = [&](int window) {          // which of the distinct windows
+        span = std::max(span, window > 0 ? std::min(window, c.max_ctx) : c.max_ctx);
+        auto w = std::find(s->windows.begin(), s->windows.end(), window);
+        const int i = (int)(w - s->windows.begin());
+        if (w == s->windows.end()) s->windows.push_back(window);
+        return i;
+    };
     for (dc_stack_layer& L : s->layers) {
-        if (L.kind == DC_MIX_DELTA) {
+        if (L.kind == DC_MIX_LIGHTNING) {
+            L.state_off = carve((size_t)L.li.heads * L.li.vdim * L.li.dim);
+        } else if (L.kind == DC_MIX_GQA) {
+            L.ga.plane = (int)planes.size();
+            planes.push_back((size_t)L.ga.row * elt);
+            L.ga.range = key_range(L.ga.window);
+            DC_TRY(rotation_table(m, L.ga.rot, &L.ga.cos_sin));
+        } else if (L.kind == DC_MIX_DELTA) {
             L.state_off = carve((size_t)L.dl.heads * L.dl.vdim * L.dl.dim);
             L.ring_off = carve((size_t)L.dl.taps * (L.dl.off_v + L.dl.heads * L.dl.vdim));
         } else if (L.kind == DC_MIX_SSD) {
@@ -189,23 +241,10 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
             } else {
                 a.plane = s->layers[a.kv_from].la.plane;
             }
-            auto w = std::find(s->windows.begin(), s->windows.end(), a.window);
-            a.range = (int)(w - s->windows.begin());
-            if (w == s->windows.end()) s->windows.push_back(a.window);
-            span = std::max(span, a.window > 0 ? std::min(a.window, c.max_ctx) : c.max_ctx);
-            float*& table = s->rot[{a.rot_base, a.rot_dim}];
-            if (!table) {
-                std::vector<float> cs((size_t)c.max_ctx * a.rot_dim);
-                for (int p = 0; p < c.max_ctx; ++p)
-                    for (int i = 0; i < a.rot_dim / 2; ++i) {
-                        const double ang = (double)p * pow(a.rot_base, -2.0 * i / a.rot_dim);
-                        cs[(size_t)p * a.rot_dim + 2 * i] = (float)cos(ang);
-                        cs[(size_t)p * a.rot_dim + 2 * i + 1] = (float)sin(ang);
-                    }
-                DC_TRY(dc_check_cuda(ctx, cudaMalloc((void**)&table, cs.size() * 4), "rotation table"));
-                DC_TRY(dc_check_cuda(ctx, cudaMemcpy(table, cs.data(), cs.size() * 4, cudaMemcpyHostToDevice), "rotation table"));
-            }
-            a.cos_sin = table;
+            a.range = key_range(a.window);
+            dc_rotation rot;
+            rot.dims = a.rot_dim, rot.base = a.rot_base;
+            DC_TRY(rotation_table(m, rot, &a.cos_sin));
         }
     }
     // key splits of a decode step: about 32 keys each at the longest span
@@ -227,12 +266,30 @@ int dc_stack_finalize(dc_model* m) {
     const long long all = (long long)m->cfg.max_seqs * m->cfg.max_ctx;
     const size_t C = std::max<long long>(DC_MAX_T, std::min<long long>(m->prefill_chunk, all));
     const size_t F = f32 ? C : DC_MAX_T;      // rows of buffers that only the f32 path uses
+    size_t q = 0, actb = 0, head_state = 0;
+    bool latent = false;
     size_t proj = 8, act = 8, low = 8, gate = 8, small = 8, mix = 8, ff = 8, lowb = 8, rank = 8, rot = 8, ukv = 8, blk = 8, qa = 0, part = 0, ml = 0;
     int span = 1;
     for (dc_stack_layer& L : s->layers) {
         auto up = [](size_t& a, long long v) { a = std::max(a, (size_t)dc_pad8((int)v)); };
         up(ff, L.ff);
-        if (L.kind == DC_MIX_DELTA) {
+        const size_t parts = std::max((size_t)DC_MAX_T * s->splits, f32 ? C : 0);
+        auto attention = [&](int heads, int values, int window) {
+            part = std::max(part, parts * heads * values);
+            ml = std::max(ml, parts * heads * 2);
+            span = std::max(span, window > 0 ? std::min(window, m->cfg.max_ctx) : m->cfg.max_ctx);
+        };
+        if (s->cfg.block == DC_BLOCK_PARALLEL) up(mix, L.out.K);
+        if (L.kind == DC_MIX_GQA) {
+            up(proj, L.ff ? L.pair0 : L.in.N);
+            q = std::max(q, (size_t)L.ga.heads * dc_gqa_ldq(L.ga));
+            attention(L.ga.heads, L.ga.dim, L.ga.window);
+        } else if (L.kind == DC_MIX_LIGHTNING) {
+            up(f32 ? proj : actb, L.ff ? L.pair0 : L.in.N);
+            up(act, L.li.heads * L.li.vdim);
+            if (f32) blk = std::max(blk, dc_lightning_block_floats(L.li));
+            else head_state = std::max(head_state, (size_t)L.li.heads * L.li.dim * L.li.vdim);
+        } else if (L.kind == DC_MIX_DELTA) {
             const dc_delta_mixer& d = L.dl;
             up(proj, d.in.N), up(act, d.off_v + d.heads * d.vdim), up(low, d.a2.N), up(gate, d.g2.N), up(small, d.heads);
             blk = std::max(blk, dc_delta_block_floats(d));
@@ -244,11 +301,9 @@ int dc_stack_finalize(dc_model* m) {
         } else {
             const dc_latent_mixer& d = L.la;
             up(proj, d.in.N), up(mix, d.heads * d.vdim), up(rank, d.kv_rank), up(rot, d.rot_dim), up(ukv, d.ukv.N);
-            const size_t parts = std::max((size_t)DC_MAX_T * s->splits, f32 ? C : 0);
             qa = std::max(qa, F * d.heads * dc_pad8(d.kv_rank));
-            part = std::max(part, parts * d.heads * d.kv_rank);
-            ml = std::max(ml, parts * d.heads * 2);
-            span = std::max(span, d.window > 0 ? std::min(d.window, m->cfg.max_ctx) : m->cfg.max_ctx);
+            attention(d.heads, d.kv_rank, d.window);
+            latent = true;
         }
     }
     b.key_cap = (int)std::min<long long>((long long)C + (long long)m->cfg.max_seqs * (span - 1), all);
@@ -272,10 +327,18 @@ int dc_stack_finalize(dc_model* m) {
         DC_TRY(alloc(m, &b.ffb, C * ff));
         DC_TRY(alloc(m, &b.lowb, C * lowb));
     }
+    if (actb) DC_TRY(alloc(m, &b.actb, C * actb));
+    if (head_state) DC_TRY(alloc(m, &b.chunk_state, (size_t)dc_lightning_chunks((int)C, DC_MAX_T) * head_state));
+    if (q) {
+        DC_TRY(alloc(m, &b.q, F * q));
+        if (!f32) DC_TRY(alloc(m, &b.qb, C * q));
+    }
     if (!s->windows.empty()) {
-        DC_TRY(alloc(m, &b.qa, qa));
         DC_TRY(alloc(m, &b.part, part));
         DC_TRY(alloc(m, &b.part_ml, ml));
+    }
+    if (latent) {
+        DC_TRY(alloc(m, &b.qa, qa));
         if (!f32) {
             DC_TRY(alloc(m, &b.keys_c, b.key_cap * rank));
             DC_TRY(alloc(m, &b.keys_r, b.key_cap * rot));
@@ -334,17 +397,17 @@ int tc_in(dc_model* m, dc_tc_in* out, const __nv_bfloat16* x, int K, int ld, int
 }
 
 // y = W x for the step's tokens: xf is the input of f32 models, xb that of bf16 models, same pitch.
-int linear(dc_model* m, const dc_step& st, const dc_lin& w, const float* xf, const __nv_bfloat16* xb, int ldx, int epi, float* out,
-           __nv_bfloat16* outb, int ldo) {
-    if (st.b16 && st.T <= DC_MAX_T) return dc_launch_linear_mma(m->ctx, w, xb, ldx, st.T, epi, outb ? nullptr : out, outb, ldo);
+int linear(dc_model* m, const dc_step& st, const dc_lin& w, const float* xf, const __nv_bfloat16* xb, int ldx, const dc_lin_epi& epi) {
+    if (st.b16 && st.T <= DC_MAX_T) return dc_launch_linear_mma(m->ctx, w, xb, ldx, st.T, epi);
     if (st.b16) {
         dc_tc_in in;
         DC_TRY(tc_in(m, &in, xb, w.K, ldx, m->stack->b.cap));
-        return dc_launch_linear_tc(m->ctx, w, in, st.T, epi, outb ? nullptr : out, outb, ldo);
+        return dc_launch_linear_tc(m->ctx, w, in, st.T, epi);
     }
-    if (st.T <= DC_MAX_T) return dc_launch_linear_rows(m->ctx, w, xf, ldx, st.T, epi, out, ldo);
-    return dc_launch_linear_f32(m->ctx, w, xf, ldx, st.T, epi, out, ldo);
+    if (st.T <= DC_MAX_T) return dc_launch_linear_rows(m->ctx, w, xf, ldx, st.T, epi);
+    return dc_launch_linear_f32(m->ctx, w, xf, ldx, st.T, epi);
 }
+dc_lin_epi to(float* out, int ld) { return dc_lin_epi::store(out, nullptr, ld); }
 
 // cls: kernel class of the per-class timing; bytes: what its launches have to read and write
 #define L(cls, bytes, n, expr)                                           \
@@ -375,11 +438,11 @@ int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
     __nv_bfloat16* lowb = st.b16 ? b.lowb : nullptr;
     DC_TRY(dc_launch_delta_prep(m->ctx, d, st, sr, b.proj, ldp, b.act, lda, b.small, lowb, ldl));
     if (st.b16) {
-        DC_TRY(linear(m, st, d.a2, nullptr, lowb, ldl, DC_LIN_STORE, b.low, nullptr, d.a2.N));
-        DC_TRY(linear(m, st, d.g2, nullptr, lowb + (d.off_g - d.off_a), ldl, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
+        DC_TRY(linear(m, st, d.a2, nullptr, lowb, ldl, to(b.low, d.a2.N)));
+        DC_TRY(linear(m, st, d.g2, nullptr, lowb + (d.off_g - d.off_a), ldl, to(b.gate, d.g2.N)));
     } else {
-        DC_TRY(linear(m, st, d.a2, b.proj + d.off_a, nullptr, ldp, DC_LIN_STORE, b.low, nullptr, d.a2.N));
-        DC_TRY(linear(m, st, d.g2, b.proj + d.off_g, nullptr, ldp, DC_LIN_STORE, b.gate, nullptr, d.g2.N));
+        DC_TRY(linear(m, st, d.a2, b.proj + d.off_a, nullptr, ldp, to(b.low, d.a2.N)));
+        DC_TRY(linear(m, st, d.g2, b.proj + d.off_g, nullptr, ldp, to(b.gate, d.g2.N)));
     }
     return dc_launch_delta_scan(m->ctx, d, st, sr, b.act, lda, b.small, b.low, d.a2.N, b.blk, b.gate, d.g2.N, m->stack->cfg.eps, b.scan,
                                 st.b16 ? nullptr : b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(ldm));
@@ -414,8 +477,57 @@ int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_laye
     DC_TRY(dc_launch_latent_gather(m->ctx, d, st, c, base, nk, b.keys_c, ldc, b.keys_r, ldr));
     dc_tc_in in;
     DC_TRY(tc_in(m, &in, b.keys_c, d.kv_rank, ldc, b.key_cap));
-    DC_TRY(dc_launch_linear_tc(m->ctx, d.ukv, in, nk, DC_LIN_STORE, nullptr, b.keys_kv, d.ukv.N));
+    DC_TRY(dc_launch_linear_tc(m->ctx, d.ukv, in, nk, dc_lin_epi::store(nullptr, b.keys_kv, d.ukv.N)));
     return dc_launch_latent_prefill(m->ctx, d, st, base, sk.tiles, sk.n_tiles, b.proj, ldp, b.keys_kv, d.ukv.N, b.keys_r, ldr, b.mixb, ldm);
+}
+
+int mix_gqa(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
+    const dc_gqa_mixer& d = Ly.ga;
+    const dc_stack_buffers& b = m->stack->b;
+    dc_gqa_cache c;
+    c.arena = m->kv.planes[d.plane].arena;
+    c.f32 = m->stack->dtype == DC_DTYPE_F32;
+    c.tables = m->kv.d_tables;
+    c.max_blocks = m->kv.max_blocks_per_seq;
+    const int ldp = Ly.ff ? Ly.pair0 : Ly.in.N, ldm = dc_pad8(Ly.out.K);
+    DC_TRY(dc_launch_gqa_prep(m->ctx, d, st, c, b.proj, ldp, m->stack->cfg.eps, m->cfg.max_ctx, b.q, st.tc ? b.qb : nullptr));
+    if (st.tc) return dc_launch_gqa_prompt(m->ctx, d, st, c, sk.tiles, sk.n_tiles, b.qb, b.mixb, ldm);
+    return dc_launch_gqa_tokens(m->ctx, d, st, c, b.q, st.T <= DC_MAX_T ? m->stack->splits : 1, b.part, b.part_ml, b.mix, st.b16 ? b.mixb : nullptr, ldm);
+}
+
+int mix_lightning(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
+    const dc_lightning_mixer& d = Ly.li;
+    const dc_stack_buffers& b = m->stack->b;
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, 0};
+    const int lda = Ly.ff ? Ly.pair0 : Ly.in.N, ldy = dc_pad8(d.heads * d.vdim), ldm = dc_pad8(Ly.out.K);
+    const __nv_bfloat16* actb = st.b16 ? b.actb : nullptr;
+    if (st.single && st.T <= DC_MAX_T) DC_TRY(dc_launch_lightning_decode(m->ctx, d, st, sr, b.proj, actb, lda, b.scan, ldy));
+    else if (st.b16) DC_TRY(dc_launch_lightning_chunks(m->ctx, d, st, sr, b.actb, lda, b.chunk_state, b.scan, ldy));
+    else DC_TRY(dc_launch_lightning_scan(m->ctx, d, st, sr, b.proj, lda, b.blk, b.scan, ldy));
+    return dc_launch_lightning_norm(m->ctx, d, st, b.scan, ldy, b.proj, actb, lda, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, ldm);
+}
+
+// x += mixer(h) + ff(h) with h = norm1(x): one product from h, the mixer, one product back into the residual.  The
+// feed-forward's hidden values lie beside the mixer's output.
+int parallel_layer(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    const int W = s->cfg.width, H = dc_pad8(W), T = st.T, rows = Ly.ff ? Ly.pair0 : Ly.in.N, ldm = dc_pad8(Ly.out.K);
+    L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm1, nullptr, 0, T, W, H, s->cfg.eps, b.y, st.b16 ? b.xb : nullptr, H));
+    const bool light = Ly.kind == DC_MIX_LIGHTNING;
+    dc_lin_epi in = dc_lin_epi::store(b.proj, light && st.b16 ? b.actb : nullptr, rows);
+    if (light) in.silu_rows = Ly.li.off_g;
+    else in.bias = Ly.ga.bias;
+    if (Ly.ff) in.pairs(Ly.pair0, DC_PAIR_CLAMPED, Ly.limit, b.mix + Ly.out_ff, st.b16 ? b.mixb + Ly.out_ff : nullptr, ldm, Ly.ff);
+    L(DC_K_MIX_IN, lin_bytes(Ly.in, T), 1, linear(m, st, Ly.in, b.y, b.xb, H, in));
+    if (light) L(DC_K_MIX_LIGHTNING, 8.0 * st.E * Ly.li.heads * Ly.li.dim * Ly.li.vdim, st.single && !st.tc ? 2 : 4, mix_lightning(m, st, Ly));
+    else L(DC_K_MIX_GQA, 4.0 * T * Ly.in.N, st.tc ? 2 : 3, mix_gqa(m, st, sk, Ly));
+    dc_lin_epi out = to(b.x, H);
+    out.add = true;
+    out.bias = Ly.out_bias;
+    L(DC_K_MIX_OUT, lin_bytes(Ly.out, T), 1, linear(m, st, Ly.out, b.mix, b.mixb, ldm, out));
+    return DC_B200_OK;
 }
 
 // Embedding and every layer; the residual ends in b.x.
@@ -432,22 +544,26 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
                                                     cudaMemcpyDeviceToDevice, ctx->stream), "capture");
     };
     m->last_launches = 0;
-    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, b.x, H, xb));
+    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, b.x, H, s->cfg.block == DC_BLOCK_PARALLEL ? nullptr : xb, s->cfg.embed_scale));
     for (size_t il = 0; il < s->layers.size(); ++il) {
         dc_stack_layer& Ly = s->layers[il];
         DC_TRY(capture((int)il));
+        if (s->cfg.block == DC_BLOCK_PARALLEL) {
+            DC_TRY(parallel_layer(m, st, sk, Ly));
+            continue;
+        }
         const dc_lin& in = Ly.kind == DC_MIX_DELTA ? Ly.dl.in : Ly.kind == DC_MIX_SSD ? Ly.ssd.in : Ly.la.in;
         const dc_lin& o = Ly.kind == DC_MIX_DELTA ? Ly.dl.o : Ly.kind == DC_MIX_SSD ? Ly.ssd.o : Ly.la.o;
-        L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.x, xb, H, DC_LIN_STORE, b.proj, nullptr, in.N));
+        L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.x, xb, H, to(b.proj, in.N)));
         if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, st.single && !st.tc ? 1 : 7, mix_delta(m, st, Ly));
         else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, st.single && !st.tc ? 2 : 5, mix_ssd(m, st, Ly));
         else L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, Ly));
-        L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), DC_LIN_STORE, b.y, nullptr, H));
+        L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), to(b.y, H)));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));
         if (!Ly.ff) continue;
         const int F = dc_pad8(Ly.ff);
-        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, DC_LIN_GELU_PAIR, b.ff, st.b16 ? b.ffb : nullptr, F));
-        L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, DC_LIN_STORE, b.y, nullptr, H));
+        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, dc_lin_epi().pairs(0, DC_PAIR_GELU, 0.0f, b.ff, st.b16 ? b.ffb : nullptr, F, F)));
+        L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, to(b.y, H)));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm2, T, W, H, eps, xb));
     }
     return capture((int)s->layers.size());
@@ -461,8 +577,8 @@ int run_head(dc_model* m, const int32_t* rows, int first, int R, bool feedback) 
     dc_step_buffers& g = m->buf;
     L(DC_K_POST_NORM, 8.0 * R * W, 1, dc_launch_norm_rows(ctx, s->b.x, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, s->b.lm_xb, H));
     L(DC_K_LM_HEAD, lin_bytes(s->head, R), 1,
-      s->b.lm_xb ? dc_launch_linear_mma(ctx, s->head, s->b.lm_xb, H, R, DC_LIN_STORE, g.logits, nullptr, s->cfg.vocab, g.argmax_keys)
-                 : dc_launch_linear_rows(ctx, s->head, s->b.lm_x, H, R, DC_LIN_STORE, g.logits, s->cfg.vocab, g.argmax_keys));
+      s->b.lm_xb ? dc_launch_linear_mma(ctx, s->head, s->b.lm_xb, H, R, dc_lin_epi::store(g.logits, nullptr, s->cfg.vocab, g.argmax_keys))
+                 : dc_launch_linear_rows(ctx, s->head, s->b.lm_x, H, R, dc_lin_epi::store(g.logits, nullptr, s->cfg.vocab, g.argmax_keys)));
     L(DC_K_ARGMAX, 64.0, 1, dc_launch_argmax_finish(ctx, g.argmax_keys, R, g.out_tokens, feedback ? g.tokens : nullptr, feedback ? g.positions : nullptr,
                                                     feedback ? g.history : nullptr, feedback ? g.history_len : nullptr, DC_HISTORY_CAP));
     return DC_B200_OK;
@@ -563,9 +679,10 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
 
 void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token) {
     dc_stack* s = m->stack;
-    if (weight_bytes) *weight_bytes = (double)s->weight_bytes - (double)s->embed->bytes + (double)s->embed->row_bytes;
+    if (weight_bytes) *weight_bytes = (double)s->weight_bytes - (double)s->embed->bytes + (s->cfg.tied ? 0.0 : (double)s->embed->row_bytes);
     double kv = 0.0;
     for (dc_stack_layer& L : s->layers)
-        if (L.kind == DC_MIX_LATENT) kv += (double)m->kv.planes[L.la.plane].row_bytes;
+        if (L.kind == DC_MIX_GQA) kv += (double)m->kv.planes[L.ga.plane].row_bytes;
+        else if (L.kind == DC_MIX_LATENT) kv += (double)m->kv.planes[L.la.plane].row_bytes;
     if (kv_bytes_per_token) *kv_bytes_per_token = kv;
 }

@@ -54,6 +54,24 @@ struct Reader {
         s->index[t.name] = (int)s->tensors.size();
         s->tensors.push_back(std::move(t));
     }
+    const dc_json* object(const dc_json& o, const char* key, const std::string& where) {
+        const dc_json* v = o.get(key);
+        if (v && v->kind == dc_json::OBJ) return v;
+        bad(where + ": '" + key + "' is missing");
+        return nullptr;
+    }
+    // {base, dims, scaling: {factor, original, fast, slow} or null}
+    void rotation(const dc_json& o, const std::string& where, dc_rotation* r) {
+        r->base = number(o, "base", where);
+        r->dims = size(o, "dims", where, 2, 1024);
+        if (r->dims % 2 || !(r->base > 1.0)) bad(where + ": dims must be even and base above 1");
+        const dc_json* s = o.get("scaling");
+        if (!s || s->is_null()) return;
+        const std::string in = where + ".scaling";
+        r->factor = number(*s, "factor", in), r->original = number(*s, "original", in);
+        r->fast = number(*s, "fast", in), r->slow = number(*s, "slow", in);
+        if (!(r->factor > 0.0 && r->original > 0.0 && r->fast > 0.0 && r->slow > 0.0)) bad(in + ": every value must be positive");
+    }
     // rows of a matrix appended to lin (whose K must agree); returns the first row
     int matrix(dc_lin* lin, const std::string& name, int N, int K) {
         const int row0 = lin->N;
@@ -156,10 +174,7 @@ void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::s
     d.vdim = r.size(j, "vdim", where, 1, 256);
     d.kv_rank = r.size(j, "kv_rank", where, 1, 1024);
     d.scale = (float)r.number(j, "scale", where);
-    const dc_json* rot = j.get("rot");
-    if (!rot || rot->kind != dc_json::OBJ) {
-        r.bad(where + ": 'rot' is missing");
-    } else {
+    if (const dc_json* rot = r.object(j, "rot", where)) {
         d.rot_base = r.number(*rot, "base", where + ".rot");
         if (r.size(*rot, "dims", where + ".rot") != d.rot_dim || d.rot_dim % 2) r.bad(where + ": rot.dims must be even and equal rot_dim");
     }
@@ -201,6 +216,89 @@ void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::s
     r.matrix(&d.o, p + "o", H, d.heads * d.vdim);
 }
 
+// Mixers of parallel blocks: their input rows open L->in, their output matrix the columns of L->out.
+void out_columns(Reader& r, const std::string& name, dc_stack_layer* L, int K) {
+    const int H = r.s->cfg.width;
+    dc_stack_tensor t;
+    t.name = name;
+    t.shape = {H, K};
+    t.lin = &L->out;
+    t.col0 = L->out.K;
+    r.tensor(t);
+    L->out.N = dc_pad8(H);
+    L->out.K += K;
+}
+
+void read_gqa(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+    dc_gqa_mixer& d = L->ga;
+    const int H = r.s->cfg.width;
+    d.heads = r.size(j, "heads", where);
+    d.kv_heads = r.size(j, "kv_heads", where);
+    d.dim = r.size(j, "dim", where, 1, 256);
+    if (r.size(j, "vdim", where) != d.dim) r.bad(where + ": the values are the keys, so vdim must equal dim");
+    if (d.heads % d.kv_heads) r.bad(where + ": heads is not a multiple of kv_heads");
+    d.scale = (float)r.number(j, "scale", where);
+    if (const dc_json* rot = r.object(j, "rot", where)) r.rotation(*rot, where + ".rot", &d.rot);
+    if (d.rot.dims > d.dim) r.bad(where + ".rot: dims is larger than the head");
+    const dc_json* mask = j.get("mask");
+    d.window = mask && !mask->is_null() ? r.size(*mask, "size", where + ".mask") : 0;
+    d.sink = true, d.sink_score = 0.0f;
+    d.dim_p = dc_pad8(d.dim);
+    d.row = 2 * d.kv_heads * d.dim_p;
+    const int Q = d.heads * d.dim, K = d.kv_heads * d.dim;
+    d.off_q = r.matrix(&L->in, p + "q", Q, H);
+    d.off_k = r.matrix(&L->in, p + "k", K, H);
+    const int rows = (L->in.N + DC_PAIR_ALIGN - 1) / DC_PAIR_ALIGN * DC_PAIR_ALIGN;     // as many as a product may store
+    r.vec(&d.bias, p + "q.b", {Q}, 4, d.off_q, rows);
+    r.vec(&d.bias, p + "k.b", {K}, 4, d.off_k, rows);
+    r.vec(&d.q_norm, p + "q.norm", {Q}, 1);
+    r.vec(&d.k_norm, p + "k.norm", {K}, 1);
+    out_columns(r, p + "o", L, Q);
+    r.vec(&L->out_bias, p + "o.b", {H}, 4);
+}
+
+void read_lightning(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+    dc_lightning_mixer& d = L->li;
+    const int H = r.s->cfg.width;
+    d.heads = r.size(j, "heads", where);
+    d.dim = r.size(j, "dim", where, 1, 256);
+    d.vdim = r.size(j, "vdim", where, 1, 512);
+    const dc_json* decay = j.get("decay");
+    if (!decay || decay->kind != dc_json::ARR || (int)decay->arr.size() != d.heads) r.bad(where + ": 'decay' must list one number per head");
+    else
+        for (const dc_json& v : decay->arr) {
+            if (v.kind != dc_json::NUM) r.bad(where + ": 'decay' must list one number per head");
+            d.decays.push_back((float)v.num);
+        }
+    const int Q = d.heads * d.dim, V = d.heads * d.vdim;
+    d.off_q = r.matrix(&L->in, p + "q", Q, H);
+    d.off_k = r.matrix(&L->in, p + "k", Q, H);
+    d.off_v = r.matrix(&L->in, p + "v", V, H);
+    d.off_g = r.matrix(&L->in, p + "g", V, H);
+    r.vec(&d.norm, p + "norm", {V}, 1);
+    out_columns(r, p + "o", L, V);
+}
+
+// Gate and up rows in turn from L->pair0 of the input matrix, the down matrix beside the mixer's output matrix.
+void read_dense_clamped(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+    const int H = r.s->cfg.width;
+    L->ff = r.size(j, "ff", where);
+    L->limit = (float)r.number(j, "limit", where);
+    L->pair0 = L->in.N = (L->in.N + DC_PAIR_ALIGN - 1) / DC_PAIR_ALIGN * DC_PAIR_ALIGN;
+    L->in.N += 2 * dc_pad8(L->ff);
+    for (int i = 0; i < 2; ++i) {
+        dc_stack_tensor t;
+        t.name = p + (i ? "up" : "gate");
+        t.shape = {L->ff, H};
+        t.lin = &L->in;
+        t.row0 = L->pair0 + i;
+        t.row_step = 2;
+        r.tensor(t);
+    }
+    L->out_ff = L->out.K = dc_pad8(L->out.K);
+    out_columns(r, p + "down", L, L->ff);
+}
+
 void read_dense_gelu(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
     const int H = r.s->cfg.width;
     L->ff = r.size(j, "ff", where);
@@ -222,16 +320,22 @@ void read_dense_gelu(Reader& r, const dc_json& j, const std::string& p, const st
 struct Arch {
     const char* name;
     unsigned mixers;        // bit per DC_MIX_*
+    int block;              // DC_BLOCK_*; parallel blocks have the clamped feed-forward, the others the tanh-gelu one
+    bool embed_scale;       // config.embedding.scale
+    bool tied;
 };
 const Arch kArchs[] = {
     // Garilix: RMS norms on the sublayers' outputs only (x += norm(f(x))), tanh-gelu gated feed-forward
-    {"Garilix", (1u << DC_MIX_DELTA) | (1u << DC_MIX_LATENT) | (1u << DC_MIX_SSD)},
+    {"Garilix", (1u << DC_MIX_DELTA) | (1u << DC_MIX_LATENT) | (1u << DC_MIX_SSD), DC_BLOCK_POST_NORM, false, false},
+    // Datasun: mixer and clamped feed-forward side by side on one normed input, embedding table as output matrix
+    {"Datasun", (1u << DC_MIX_GQA) | (1u << DC_MIX_LIGHTNING), DC_BLOCK_PARALLEL, true, true},
 };
 struct MixerType {
     const char* name;
     int kind;
 };
-const MixerType kMixers[] = {{"channel_delta", DC_MIX_DELTA}, {"latent_attention", DC_MIX_LATENT}, {"mamba2", DC_MIX_SSD}};
+const MixerType kMixers[] = {{"channel_delta", DC_MIX_DELTA}, {"latent_attention", DC_MIX_LATENT}, {"mamba2", DC_MIX_SSD},
+                              {"attention", DC_MIX_GQA}, {"lightning", DC_MIX_LIGHTNING}};
 
 int alloc_lin(dc_model* m, dc_lin* l) {
     if (!l->N) return DC_B200_OK;
@@ -256,6 +360,10 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
     if (!a)
         return dc_fail(m->ctx, DC_B200_UNSUPPORTED, "config: architecture '%s' is not registered", arch ? arch->str.c_str() : "(none)");
     s->cfg.arch = a->name;
+    s->cfg.block = a->block;
+    s->cfg.tied = a->tied;
+    if (a->embed_scale)
+        if (const dc_json* e = r.object(cj, "embedding", "config")) s->cfg.embed_scale = (float)r.number(*e, "scale", "config.embedding");
     s->cfg.vocab = r.size(cj, "vocab", "config", 2);
     s->cfg.width = r.size(cj, "width", "config", 1, 8192);
     const dc_json* norm = cj.get("norm");
@@ -271,6 +379,11 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         dc_stack_tensor t;
         t.name = "embed";
         t.shape = {s->cfg.vocab, H};
+        if (s->cfg.tied) {
+            t.lin = &s->head;
+            s->head.N = dc_pad8(s->cfg.vocab);
+            s->head.K = H;
+        }
         r.tensor(t);
     }
     for (int i = 0; i < n && r.error.empty(); ++i) {
@@ -287,6 +400,8 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         }
         if (L.kind == DC_MIX_DELTA) read_delta(r, *mixer, p + "mix.", where + ".mixer", &L);
         else if (L.kind == DC_MIX_SSD) read_ssd(r, *mixer, p + "mix.", where + ".mixer", &L);
+        else if (L.kind == DC_MIX_GQA) read_gqa(r, *mixer, p + "mix.", where + ".mixer", &L);
+        else if (L.kind == DC_MIX_LIGHTNING) read_lightning(r, *mixer, p + "mix.", where + ".mixer", &L);
         else read_latent(r, *mixer, p + "mix.", where + ".mixer", &L, i);
         r.vec(&L.norm1, p + "norm1", {H}, 1);
         if (mlp && !mlp->is_null()) {
@@ -295,12 +410,16 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
                 r.bad(where + ".mlp: unknown kind");
                 break;
             }
-            read_dense_gelu(r, *mlp, p + "mlp.", where + ".mlp", &L);
-            r.vec(&L.norm2, p + "norm2", {H}, 1);
+            if (a->block == DC_BLOCK_PARALLEL) {
+                read_dense_clamped(r, *mlp, p + "mlp.", where + ".mlp", &L);
+            } else {
+                read_dense_gelu(r, *mlp, p + "mlp.", where + ".mlp", &L);
+                r.vec(&L.norm2, p + "norm2", {H}, 1);
+            }
         }
     }
     r.vec(&s->final_norm, "final.norm", {H}, 1);
-    r.matrix(&s->head, "head", s->cfg.vocab, H);
+    if (!s->cfg.tied) r.matrix(&s->head, "head", s->cfg.vocab, H);
     if (!r.error.empty()) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "%s", r.error.c_str());
 
     // weight memory
@@ -309,14 +428,26 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
     s->embed->K = H;
     s->embed->N = s->cfg.vocab;
     s->embed->E = 1;
-    s->embed->row_bytes = (size_t)H * 2;
-    s->embed->bytes = s->embed->row_bytes * s->cfg.vocab;
-    DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)&s->embed->dev, s->embed->bytes + 64), "weight memory"));
-    for (dc_stack_layer& L : s->layers) {
-        dc_lin* ls[] = {&L.dl.in, &L.dl.a2, &L.dl.g2, &L.dl.o, &L.ssd.in, &L.ssd.o, &L.la.in, &L.la.ukv, &L.la.o, &L.gate_up, &L.down};
-        for (dc_lin* l : ls) DC_TRY(alloc_lin(m, l));
-    }
     DC_TRY(alloc_lin(m, &s->head));
+    if (s->cfg.tied) {              // rows of the output matrix; bytes 0: the memory is not the embedding's own
+        s->embed->row_bytes = (size_t)s->head.ld * 2;
+        s->embed->bytes = 0;
+        s->embed->dev = (uint8_t*)s->head.w;
+    } else {
+        s->embed->row_bytes = (size_t)H * 2;
+        s->embed->bytes = s->embed->row_bytes * s->cfg.vocab;
+        DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)&s->embed->dev, s->embed->bytes + 64), "weight memory"));
+    }
+    for (dc_stack_layer& L : s->layers) {
+        dc_lin* ls[] = {&L.dl.in, &L.dl.a2, &L.dl.g2, &L.dl.o, &L.ssd.in, &L.ssd.o, &L.la.in, &L.la.ukv, &L.la.o, &L.gate_up, &L.down, &L.in, &L.out};
+        for (dc_lin* l : ls) DC_TRY(alloc_lin(m, l));
+        if (!L.li.decays.empty()) {
+            const size_t bytes = L.li.decays.size() * 4;
+            DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)&L.li.decay, bytes), "weight memory"));
+            s->owned.push_back(L.li.decay);
+            DC_TRY(dc_check_cuda(m->ctx, cudaMemcpy(L.li.decay, L.li.decays.data(), bytes, cudaMemcpyHostToDevice), "weight memory"));
+        }
+    }
     for (dc_stack_tensor& t : s->tensors)
         if (t.vec && !*t.vec) {
             DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)t.vec, (size_t)t.vec_len * 4 + 64), "weight memory"));

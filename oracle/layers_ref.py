@@ -97,13 +97,53 @@ def ssd_scan(x, B, C, dt, A_log, D, S):
     return y
 
 
-def windowed_softmax(scores, i, window):
-    """scores over keys 0 .. i -> weights; keys with i - j >= window are not seen."""
+def windowed_softmax(scores, i, window, sink=None):
+    """scores over keys 0 .. i -> weights; keys with i - j >= window are not seen.  sink: score of one more term of the
+    denominator that has no value."""
     n = scores.shape[-1]
     seen = (i - np.arange(n)) < window if window else np.ones(n, bool)
     s = np.where(seen, scores, -np.inf)
-    s = np.exp(s - s.max(axis=-1, keepdims=True))
-    return s / s.sum(axis=-1, keepdims=True)
+    top = s.max(axis=-1, keepdims=True)
+    if sink is not None:
+        top = np.maximum(top, sink)
+    s = np.exp(s - top)
+    return s / (s.sum(axis=-1, keepdims=True) + (0.0 if sink is None else np.exp(sink - top)))
+
+
+def yarn_frequencies(dims, base, scaling=None):
+    """(angle per position of every pair, factor of cos and sin).  scaling: {factor, original, fast, slow}; pairs that
+    turn less than `slow` times over the original context are slowed down by the factor, those that turn more than
+    `fast` times are left alone, with a linear ramp over the pairs between."""
+    f = np.array([base ** (-2.0 * i / dims) for i in range(dims // 2)], F)
+    if not scaling:
+        return f, 1.0
+    pair_of = lambda turns: dims * np.log(scaling["original"] / (2 * np.pi * turns)) / (2 * np.log(base))
+    lo = max(np.floor(pair_of(scaling["fast"])), 0)
+    hi = min(np.ceil(pair_of(scaling["slow"])), dims - 1)
+    slowed = np.clip((np.arange(dims // 2) - lo) / max(hi - lo, 0.001), 0, 1)
+    return f * (1 - slowed) + f / scaling["factor"] * slowed, 0.1 * np.log(scaling["factor"]) + 1.0
+
+
+def rotate_pairs(x, pos, freq, mul):
+    """x [T, H, D]: pairs (2i, 2i + 1) of the first 2 len(freq) dimensions turned by pos * freq[i] and scaled."""
+    out = x.copy()
+    for i, f in enumerate(freq):
+        c, s = mul * np.cos(pos * f)[:, None], mul * np.sin(pos * f)[:, None]
+        u, v = x[:, :, 2 * i], x[:, :, 2 * i + 1]
+        out[:, :, 2 * i] = u * c - v * s
+        out[:, :, 2 * i + 1] = v * c + u * s
+    return out
+
+
+def decayed_linear_attention(q, k, v, decay, S):
+    """S <- decay S + k v^T, o = S^T q, token by token.  q, k [T, H, d]; v [T, H, e]; decay [H]; S [H, d, e] (changed
+    in place).  Returns o [T, H, e]."""
+    o = np.zeros_like(v)
+    for t in range(q.shape[0]):
+        for h in range(q.shape[1]):
+            S[h] = decay[h] * S[h] + np.outer(k[t, h], v[t, h])
+            o[t, h] = S[h].T @ q[t, h]
+    return o
 
 
 # ---------------------------------------------------------------- mixers
@@ -174,6 +214,43 @@ def dense_mlp(h, P):
     return linear(gelu_tanh(linear(h, P["gate"])) * linear(h, P["up"]), P["down"])
 
 
+def mix_attention(h, P, m, eps, pos, st):
+    """Grouped-query attention whose values are the raw keys; a sink of score 0.  st: {"k", "v"} of earlier tokens."""
+    T, H, G, d = h.shape[0], m["heads"], m["kv_heads"], m["dim"]
+    q = linear(h, P["q"]) + P["q.b"]
+    v = linear(h, P["k"]) + P["k.b"]
+    freq, mul = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+    q = rotate_pairs(rms_norm(q, P["q.norm"], eps).reshape(T, H, d), pos, freq, mul)
+    k = rotate_pairs(rms_norm(v, P["k.norm"], eps).reshape(T, G, d), pos, freq, mul)
+    v = v.reshape(T, G, d)
+    if "k" in st:
+        k, v = np.concatenate([st["k"], k]), np.concatenate([st["v"], v])
+    st["k"], st["v"] = k, v
+    of = np.arange(H) // (H // G)
+    out = np.zeros((T, H, d), F)
+    for t in range(T):
+        n = int(pos[t]) + 1
+        s = np.einsum("hd,nhd->hn", q[t], k[:n, of]) * m["scale"]
+        out[t] = np.einsum("hn,nhd->hd", windowed_softmax(s, n - 1, m["mask"]["size"], sink=0.0), v[:n, of])
+    return linear(out.reshape(T, H * d), P["o"]) + P["o.b"]
+
+
+def mix_lightning(h, P, m, eps, st):
+    T, H, d, e = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q, k = (silu(linear(h, P[n])).reshape(T, H, d) for n in "qk")
+    v = silu(linear(h, P["v"])).reshape(T, H, e)
+    if "S" not in st:
+        st["S"] = np.zeros((H, d, e), F)
+    o = decayed_linear_attention(q, k, v, np.array(m["decay"], F), st["S"]).reshape(T, H * e)
+    return linear(rms_norm(o, P["norm"], eps) * sigmoid(linear(h, P["g"])), P["o"])
+
+
+def clamped_mlp(h, P, limit):
+    g = np.minimum(linear(h, P["gate"]), limit)
+    u = np.clip(linear(h, P["up"]), -limit, limit)
+    return linear(g * sigmoid(1.702 * g) * (u + 1), P["down"])
+
+
 # ---------------------------------------------------------------- the decoder
 class Stepper:
     def __init__(self, config: dict, tensors: dict):
@@ -190,28 +267,46 @@ class Stepper:
         residual after every layer."""
         tokens = np.asarray(tokens)
         pos = self.pos + np.arange(tokens.size)
-        eps = self.c["norm"]["eps"]
-        x = self.w["embed"][tokens]
-        for i, L in enumerate(self.c["layers"]):
-            P, m, st = self.part(f"l{i}.mix."), L["mixer"], self.state[i]
-            if L["type"] == "channel_delta":
-                y = mix_channel_delta(x, P, m, eps, st)
-            elif L["type"] == "mamba2":
-                y = mix_mamba2(x, P, m, eps, st)
-            elif L["type"] == "latent_attention":
-                src = m.get("kv_from")
-                if src is None:
-                    latent_append(x, P, m, eps, pos, st)
-                y = mix_latent_attention(x, P, m, eps, pos, st if src is None else self.state[src])
-            else:
-                raise ValueError(L["type"])
-            x = x + rms_norm(y, self.w[f"l{i}.norm1"], eps)
-            if L.get("mlp"):
-                x = x + rms_norm(dense_mlp(x, self.part(f"l{i}.mlp.")), self.w[f"l{i}.norm2"], eps)
+        run = {"Garilix": self.garilix_layer, "Datasun": self.datasun_layer}[self.c["architecture"]]
+        x = self.w["embed"][tokens] * self.c.get("embedding", {}).get("scale", 1.0)
+        for i in range(len(self.c["layers"])):
+            x = run(i, x, pos)
             if trace is not None:
                 trace.append(x.copy())
         self.pos += tokens.size
-        return linear(rms_norm(x, self.w["final.norm"], eps), self.w["head"])
+        return linear(rms_norm(x, self.w["final.norm"], self.c["norm"]["eps"]), self.w["head" if "head" in self.w else "embed"])
+
+    def garilix_layer(self, i, x, pos):
+        L, P, st, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.state[i], self.c["norm"]["eps"]
+        m = L["mixer"]
+        if L["type"] == "channel_delta":
+            y = mix_channel_delta(x, P, m, eps, st)
+        elif L["type"] == "mamba2":
+            y = mix_mamba2(x, P, m, eps, st)
+        elif L["type"] == "latent_attention":
+            src = m.get("kv_from")
+            if src is None:
+                latent_append(x, P, m, eps, pos, st)
+            y = mix_latent_attention(x, P, m, eps, pos, st if src is None else self.state[src])
+        else:
+            raise ValueError(L["type"])
+        x = x + rms_norm(y, self.w[f"l{i}.norm1"], eps)
+        if L.get("mlp"):
+            x = x + rms_norm(dense_mlp(x, self.part(f"l{i}.mlp.")), self.w[f"l{i}.norm2"], eps)
+        return x
+
+    def datasun_layer(self, i, x, pos):
+        L, P, st, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.state[i], self.c["norm"]["eps"]
+        h = rms_norm(x, self.w[f"l{i}.norm1"], eps)
+        if L["type"] == "attention":
+            y = mix_attention(h, P, L["mixer"], eps, pos, st)
+        elif L["type"] == "lightning":
+            y = mix_lightning(h, P, L["mixer"], eps, st)
+        else:
+            raise ValueError(L["type"])
+        if L.get("mlp"):
+            y = y + clamped_mlp(h, self.part(f"l{i}.mlp."), L["mlp"]["limit"])
+        return x + y
 
 
 def forward(config, tensors, tokens):
