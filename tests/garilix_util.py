@@ -1,16 +1,9 @@
-"""Small Garilix decoders with random weights for the tests: configs, tensors, safetensors files."""
+"""Small Garilix decoders with random weights for the tests: configs and tensors."""
 from __future__ import annotations
-
-import json
-import os
-import struct
 
 import numpy as np
 
-
-def bf16_round(x):
-    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) & 0xFFFF0000).astype(np.uint32).view(np.float32)
+from stack_util import bf16_round
 
 
 def delta(heads=3, kv_heads=None, dim=24, vdim=20, conv=4):
@@ -96,29 +89,3 @@ def make_tensors(cfg, seed=0, a_rank=12, g_rank=20):
     vec("final.norm", W)
     mat("head", V, W)
     return t
-
-
-def write_model(path, cfg, tensors, f32=()):
-    """config.json and model.safetensors; tensors named in f32 are stored as F32, the others as BF16."""
-    os.makedirs(path, exist_ok=True)
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg, f)
-    header, blobs, off = {"__metadata__": {"note": "test"}}, [], 0
-    for n, a in tensors.items():
-        a = np.ascontiguousarray(a, dtype=np.float32)
-        b = a.tobytes() if n in f32 else (a.view(np.uint32) >> 16).astype(np.uint16).tobytes()
-        header[n] = {"dtype": "F32" if n in f32 else "BF16", "shape": list(a.shape), "data_offsets": [off, off + len(b)]}
-        blobs.append(b)
-        off += len(b)
-    h = json.dumps(header).encode()
-    with open(os.path.join(path, "model.safetensors"), "wb") as f:
-        f.write(struct.pack("<Q", len(h)) + h + b"".join(blobs))
-    return str(path)
-
-
-def rel(got, want):
-    """Root mean square of the difference of each row over that of the wanted rows (means taken off)."""
-    d = got - want
-    d = d - d.mean(axis=-1, keepdims=True)
-    w = want - want.mean(axis=-1, keepdims=True)
-    return np.sqrt((d ** 2).mean(axis=-1)) / np.sqrt((w ** 2).mean())

@@ -5,8 +5,9 @@ import json
 import numpy as np
 import pytest
 
-from garilix_util import bf16_round, config, delta, latent, make_tensors, mamba, rel
+from garilix_util import config, delta, latent, make_tensors, mamba
 from oracle import layers_ref as R
+from stack_util import bf16_round, rel
 
 LAYERS = [delta(heads=2, kv_heads=1, dim=6, vdim=5), latent(heads=2, dim=6, rot_dim=4, vdim=5, kv_rank=8, window=7), mamba(heads=2, vdim=4, state=3),
           latent(heads=1, dim=5, rot_dim=4, vdim=3, kv_rank=8, window=4, kv_from=1)]

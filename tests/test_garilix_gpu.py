@@ -4,50 +4,19 @@ import numpy as np
 import pytest
 
 import densecore_b200 as dc
-from garilix_util import bf16_round, config, delta, latent, make_tensors, mamba, rel, write_model
+from garilix_util import config, delta, latent, make_tensors, mamba
 from oracle import layers_ref as R
+from stack_util import TOL, ModelCase, bf16_round, close, rel, run, write_model
 
 pytestmark = pytest.mark.gpu
-
-TOL = {"float32": (2e-5, 5e-5), "bfloat16": (2.5e-2, 0.12)}      # median and largest relative error of a position
-
-
-def close(got, want, dtype):
-    e = rel(got, want)
-    return np.median(e) < TOL[dtype][0] and e.max() < TOL[dtype][1]
-
 
 STACK = [delta(heads=4, kv_heads=2), latent(window=21), mamba(), latent(window=37, kv_from=1), delta(heads=2, dim=40, vdim=12, conv=3),
          mamba(heads=6, vdim=12, state=12, groups=3, norm_groups=4, conv=2)]
 
 
-class Case:
-    """A model on disk, random tokens and their reference logits (of every position)."""
-
+class Case(ModelCase):
     def __init__(self, path, cfg, n=150, seed=0, **kw):
-        self.cfg, self.tensors = cfg, make_tensors(cfg, seed, **kw)
-        self.path = write_model(path, cfg, self.tensors)
-        rng = np.random.default_rng(seed + 1)
-        self.tokens = rng.integers(0, cfg["vocab"], size=n)
-        self.want = R.Stepper(cfg, self.tensors).step(self.tokens)
-
-    def model(self, ctx, dtype, max_seqs=4, max_ctx=512, pool_tokens=0, chunk=None):
-        m = dc.Model.from_dir(ctx, self.path, dtype, max_seqs, max_ctx, pool_tokens)
-        if chunk:
-            m.set_option("prefill_chunk", chunk)
-        m.finalize()
-        return m
-
-
-def run(m, tokens, cuts):
-    """One sequence in portions (cuts: their lengths, repeated as needed); logits of every position."""
-    s, out, i, j = m.seq_alloc(), [], 0, 0
-    while i < len(tokens):
-        n = min(cuts[j % len(cuts)], len(tokens) - i)
-        out.append(m.forward_batch([(s, tokens[i:i + n])], np.arange(n)))
-        i, j = i + n, j + 1
-    m.seq_free(s)
-    return np.concatenate(out)
+        super().__init__(path, cfg, make_tensors(cfg, seed, **kw), n, seed)
 
 
 @pytest.fixture(scope="module")
