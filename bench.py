@@ -27,6 +27,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import subprocess
 import sys
@@ -372,6 +373,17 @@ def garilix_config(width: int, repeats: int, vocab: int = 32768):
     return {"architecture": "Garilix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": layers}, shapes
 
 
+def datasun_config(width: int, repeats: int, vocab: int = 32768):
+    """A Datasun decoder whose layers have the sizes of a real model of this width (four lightning and two windowed
+    attention layers per repeat)."""
+    h = width // 128
+    light = {"type": "lightning", "mixer": {"heads": h, "dim": 128, "vdim": 128, "decay": [math.exp(-8.0 * 0.5 ** (i * 10.0 / h)) for i in range(h)]}}
+    att = {"type": "attention", "mixer": {"heads": h, "kv_heads": max(1, width // 512), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+                                          "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}}
+    layers = [dict(ly, mlp={"kind": "dense", "ff": 3 * width, "limit": 7.0}) for ly in (light, light, att) * 2 * repeats]
+    return {"architecture": "Datasun", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def time_decoder(m, vocab: int, prompt: int, streams, steps: int, reps: int = 5) -> dict:
     """Prompt throughput (host tokens in, first token out, best of reps on fresh sequences) and greedy decode after
     that prompt (device time of decode_run) of any decoder of the library."""
@@ -422,6 +434,25 @@ def bench_garilix(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), r
             for v in r["decode"].values():
                 v["hbm_fraction"] = v["weight_gbs"] / peak_gbs
         out["sizes"][str(w)] = {"garilix_bf16": a, "dense_kquant": b}
+    return out
+
+
+def bench_datasun(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), repeats: int = 2, prompt: int = 2048) -> dict:
+    """Datasun decoders (bf16, random weights) beside Garilix decoders of the same width, depth, feed-forward and
+    vocabulary.  Decode reads more weights than the L2 holds at the larger widths; no flush."""
+    import densecore_b200 as dc
+    out = {"vocab": 32768, "layers": 6 * repeats, "sizes": {}}
+    for w in widths:
+        r = {}
+        for name, (cfg, shapes) in (("datasun_bf16", (datasun_config(w, repeats), {})), ("garilix_bf16", garilix_config(w, repeats))):
+            m = dc.Model.from_config(ctx, cfg, shapes, max_seqs=4, max_ctx=prompt + 512)
+            m.init_synthetic(11, 0.02)
+            m.finalize()
+            r[name] = time_decoder(m, cfg["vocab"], prompt, (1, 4), steps)
+            m.close()
+            for v in r[name]["decode"].values():
+                v["hbm_fraction"] = v["weight_gbs"] / peak_gbs
+        out["sizes"][str(w)] = r
     return out
 
 
@@ -500,6 +531,8 @@ def run_single_op(args) -> int:
         out = {"T": moe_layer_sweep(ctx, args.steps, peak)}
     elif args.op == "garilix":
         out = bench_garilix(ctx, args.steps, peak)
+    elif args.op == "datasun":
+        out = bench_datasun(ctx, args.steps, peak)
     elif args.op == "dense-0p8b":
         out = bench_dense_0p8b(ctx, peak)
     else:
@@ -532,7 +565,7 @@ def main():
     ap.add_argument("--profiler-range", action="store_true",
                     help="bracket the timed 1-stream decode run with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
     ap.add_argument("--no-extras", action="store_true", help="skip the other workloads (single ops, dense model, speculative sweep)")
-    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix"],
+    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix", "datasun"],
                     help="time one operator alone and print its own JSON line (not the benchmark line)")
     args = ap.parse_args()
     if args.warmup < 3:

@@ -31,6 +31,14 @@ struct LtParams {
     int* err;
 };
 
+// activations whose results are rounded to bf16: z / (1 + e^-z) with the hardware's exponential and division
+__device__ __forceinline__ float quick_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float quick_clamped(float limit, float gate, float up) {
+    gate = fminf(gate, limit);
+    up = fminf(fmaxf(up, -limit), limit);
+    return __fdividef(gate, 1.0f + __expf(-1.702f * gate)) * (up + 1.0f);
+}
+
 // Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.
 template <int COLS>
 __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int quarter, int lane) {
@@ -47,25 +55,39 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
             for (int i = 0; i < 8; ++i) {
                 const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
                 const float mine = __int_as_float(up ? v[i + 8] : v[i]);
-                const float h = up ? pair_value(p.e, got, mine) : pair_value(p.e, mine, got);
+                const float gate = up ? got : mine, val = up ? mine : got;
+                const float h = p.e.pair_kind == DC_PAIR_GELU ? gelu_tanh(gate) * val : quick_clamped(p.e.limit, gate, val);
                 const int t = t0 + c0 + i + (up ? 8 : 0);
                 if (t < p.T && o < p.e.n_pairs) put_pair(p.e, t, o, h);
             }
         } else if (row < p.e.n_store) {
-            float old[16];
-            if (p.e.add) {           // every load ahead of the stores
-#pragma unroll
-                for (int i = 0; i < 16; ++i) old[i] = p.e.out[(size_t)min(t0 + c0 + i, p.T - 1) * p.e.ldo + row];
-            }
+            const int n = min(16, p.T - t0 - c0);
             const float bias = p.e.bias ? p.e.bias[row] : 0.0f;
+            const size_t at = (size_t)(t0 + c0) * p.e.ldo + row;
+            if (p.e.outb) {
+                __nv_bfloat16* o = p.e.outb + at;
+                if (row < p.e.silu_rows) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                const int t = t0 + c0 + i;
-                if (t >= p.T) break;
-                float r = __int_as_float(v[i]) + bias;
-                if (row < p.e.silu_rows) r = silu(r);
-                if (p.e.outb) p.e.outb[(size_t)t * p.e.ldo + row] = __float2bfloat16_rn(r);
-                else p.e.out[(size_t)t * p.e.ldo + row] = p.e.add ? old[i] + r : r;
+                    for (int i = 0; i < 16; ++i) v[i] = __float_as_int(quick_silu(__int_as_float(v[i]) + bias));
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) v[i] = __float_as_int(__int_as_float(v[i]) + bias);
+                }
+#pragma unroll
+                for (int i = 0; i < 16; ++i, o += p.e.ldo)
+                    if (i < n) *o = __float2bfloat16_rn(__int_as_float(v[i]));
+            } else if (p.e.add) {
+                float old[16], *o = p.e.out + at;
+#pragma unroll
+                for (int i = 0; i < 16; ++i) old[i] = o[(size_t)min(i, n - 1) * p.e.ldo];        // every load ahead of the stores
+#pragma unroll
+                for (int i = 0; i < 16; ++i, o += p.e.ldo)
+                    if (i < n) *o = old[i] + (__int_as_float(v[i]) + bias);
+            } else {
+                float* o = p.e.out + at;
+#pragma unroll
+                for (int i = 0; i < 16; ++i, o += p.e.ldo)
+                    if (i < n) *o = __int_as_float(v[i]) + bias;
             }
         }
     }
