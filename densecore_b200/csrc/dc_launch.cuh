@@ -4,6 +4,26 @@
 #pragma once
 #include "dc_internal.h"
 
+// The same for a kernel whose CTAs form clusters of `cluster` neighbours.
+template <typename... KArgs, typename... Args>
+static inline int dc_launch_cluster(dc_ctx* ctx, const char* name, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, int cluster,
+                                    Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = cluster;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = ctx->use_pdl ? 2 : 1;
+    return dc_check_cuda(ctx, cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...), name);
+}
+
 template <typename... KArgs, typename... Args>
 static inline int dc_launch(dc_ctx* ctx, const char* name, void (*kernel)(KArgs...), dim3 grid, dim3 block,
                             size_t smem, Args... args) {

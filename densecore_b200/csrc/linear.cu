@@ -1,6 +1,6 @@
 // Products y = W x with bf16 weights and f32 accumulation for up to sixteen tokens, and for f32 activations.
 //
-// k_linear_mma (bf16 activations) streams the weight rows once: a CTA owns sixteen rows, its sixteen warps
+// k_linear_mma (bf16 activations) streams the weight rows once: a CTA takes sixteen rows at a time, its sixteen warps
 // take neighbouring runs of 32 columns and feed them to m16n8k16 products.  A lane loads sixteen bytes of a row at a time;
 // both operands use the same order of columns within a run, so the fragments need no shuffling.  k_linear_rows (f32
 // activations, f32 models) does the same on the CUDA cores: a warp owns R rows, a lane takes runs of eight weights, the
@@ -140,7 +140,7 @@ int launch_rows(dc_ctx* ctx, const RowsParams& p) {
 }
 
 // ---- sixteen rows per CTA on the tensor cores
-constexpr int LM_WARPS = 16;
+constexpr int LM_WARPS = 16, LM_CTAS = 2;       // warps of a CTA, resident CTAs per SM
 
 struct MmaParams {
     const __nv_bfloat16* w;
@@ -157,53 +157,80 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1
 }
 
 // NT: groups of eight tokens; AHEAD: neighbouring runs of 32 columns that a warp keeps in flight.  Column 8 q + 4 s + e of a run (q: lane % 4) is k-slot 2 q + e % 2 + 8 (e / 2) of product s.
-template <int NT, int AHEAD>
+// KS: CTAs of a cluster that share sixteen rows, each with its part of the columns; the first adds the parts up.
+// With KS 1 a CTA walks over its tiles of sixteen rows and fetches the next tile's first runs ahead of a tile's sum.
+template <int NT, int AHEAD, int KS>
 __global__ void __launch_bounds__(LM_WARPS * 32) k_linear_mma(const MmaParams p) {
-    __shared__ float red[LM_WARPS][16][8 * NT + 1];
+    __shared__ float red[2][LM_WARPS][16][8 * NT + 1];
+    __shared__ float other[KS > 1 ? KS - 1 : 1][KS > 1 ? 128 * NT : 1];
+    if (KS > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");       // waited for ahead of the first remote store
     dc::pdl_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
-    const int row0 = blockIdx.x * 16, runs = (p.K + 31) / 32, K8 = (p.K + 7) & ~7;
-    // the matrix has a multiple of eight rows
-    const uint4* w0 = reinterpret_cast<const uint4*>(p.w + (size_t)(row0 + g) * p.ldw) + q;
-    const uint4* w1 = reinterpret_cast<const uint4*>(p.w + (size_t)min(row0 + 8 + g, p.N - 1) * p.ldw) + q;
+    const int part = blockIdx.x % KS, tiles = (p.N + 15) / 16, K8 = (p.K + 7) & ~7;
+    const int all = (p.K + 31) / 32, per = (all + KS - 1) / KS, first = part * per, runs = min(all, first + per);
     uint4 a[AHEAD][2];
-    auto fetch = [&](int j, int run) {
-        const bool ok = 32 * run + 8 * q < K8;
+    // the matrix has a multiple of eight rows
+    auto fetch = [&](int j, int tile, int run) {
+        const bool ok = tile < tiles && run < runs && 32 * run + 8 * q < K8;
+        const uint4* w0 = reinterpret_cast<const uint4*>(p.w + (size_t)(16 * tile + g) * p.ldw) + q;
+        const uint4* w1 = reinterpret_cast<const uint4*>(p.w + (size_t)min(16 * tile + 8 + g, p.N - 1) * p.ldw) + q;
         a[j][0] = ok ? __ldg(w0 + 4 * run) : make_uint4(0, 0, 0, 0);
         a[j][1] = ok ? __ldg(w1 + 4 * run) : make_uint4(0, 0, 0, 0);
     };
+    int tile = blockIdx.x / KS;
+    const int step = gridDim.x / KS;
 #pragma unroll
-    for (int j = 0; j < AHEAD; ++j) fetch(j, warp * AHEAD + j);
+    for (int j = 0; j < AHEAD; ++j) fetch(j, tile, first + warp * AHEAD + j);
     dc::pdl_wait();
-    float acc[NT][4];
+    for (int buf = 0; tile < tiles; tile += step, buf ^= 1) {
+        const int row0 = 16 * tile;
+        float acc[NT][4];
 #pragma unroll
-    for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
-    for (int rb = warp * AHEAD; rb < runs; rb += LM_WARPS * AHEAD) {
+        for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
+        for (int rb = first + warp * AHEAD; rb < runs; rb += LM_WARPS * AHEAD) {
+            const bool last = KS == 1 && rb + LM_WARPS * AHEAD >= runs;
 #pragma unroll
-        for (int j = 0; j < AHEAD; ++j) {
-            const int run = rb + j, k = 32 * run + 8 * q;
-            if (run >= runs) break;
-            const uint4 a0 = a[j][0], a1 = a[j][1];
-            fetch(j, run + LM_WARPS * AHEAD);
+            for (int j = 0; j < AHEAD; ++j) {
+                const int run = rb + j, k = 32 * run + 8 * q;
+                const uint4 a0 = a[j][0], a1 = a[j][1];
+                if (last) fetch(j, tile + step, first + warp * AHEAD + j);
+                else fetch(j, tile, run + LM_WARPS * AHEAD);
+                if (run >= runs) continue;
 #pragma unroll
-            for (int n = 0; n < NT; ++n) {
-                uint4 b = make_uint4(0, 0, 0, 0);
-                if (8 * n + g < p.T && k < K8) b = *reinterpret_cast<const uint4*>(p.x + (size_t)(8 * n + g) * p.ldx + k);
-                mma_bf16(acc[n], a0.x, a1.x, a0.y, a1.y, b.x, b.y);
-                mma_bf16(acc[n], a0.z, a1.z, a0.w, a1.w, b.z, b.w);
+                for (int n = 0; n < NT; ++n) {
+                    uint4 b = make_uint4(0, 0, 0, 0);
+                    if (8 * n + g < p.T && k < K8) b = *reinterpret_cast<const uint4*>(p.x + (size_t)(8 * n + g) * p.ldx + k);
+                    mma_bf16(acc[n], a0.x, a1.x, a0.y, a1.y, b.x, b.y);
+                    mma_bf16(acc[n], a0.z, a1.z, a0.w, a1.w, b.z, b.w);
+                }
             }
         }
-    }
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+        for (int n = 0; n < NT; ++n)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) red[warp][g + 8 * (i >> 1)][8 * n + 2 * q + (i & 1)] = acc[n][i];
-    __syncthreads();
-    if (threadIdx.x < 128 * NT) {               // one thread per (row, token), rows fastest
-        const int r = threadIdx.x & 15, t = threadIdx.x >> 4, row = row0 + r;
+            for (int i = 0; i < 4; ++i) red[buf][warp][g + 8 * (i >> 1)][8 * n + 2 * q + (i & 1)] = acc[n][i];
+        __syncthreads();
+        const int r = threadIdx.x & 15, t = threadIdx.x >> 4, row = row0 + r;      // one thread per (row, token), rows fastest
+        const bool mine = threadIdx.x < 128 * NT;
         float v = 0.0f;
+        if (mine)
 #pragma unroll
-        for (int w = 0; w < LM_WARPS; ++w) v += red[w][r][t];
+            for (int w = 0; w < LM_WARPS; ++w) v += red[buf][w][r][t];
+        if (KS > 1) {                // one tile a cluster
+            asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+            if (part > 0 && mine) {
+                uint32_t to;
+                asm("mapa.shared::cluster.u32 %0, %1, 0;" : "=r"(to) : "r"(dc::smem_u32(&other[part - 1][threadIdx.x])));
+                asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(to), "f"(v) : "memory");
+            }
+            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+            asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+            if (part > 0) return;
+            if (mine)
+#pragma unroll
+                for (int k = 0; k < KS - 1; ++k) v += other[k][threadIdx.x];
+        }
+        if (!mine) continue;
         if (row0 >= p.e.pair0) {
             const float up = __shfl_down_sync(0xffffffffu, v, 1);
             const int o = (row - p.e.pair0) >> 1;
@@ -215,8 +242,8 @@ __global__ void __launch_bounds__(LM_WARPS * 32) k_linear_mma(const MmaParams p)
                 unsigned long long key = ok ? dc::argmax_key(v, row) : 0ull;
 #pragma unroll
                 for (int o = 8; o > 0; o >>= 1) {
-                    const unsigned long long other = __shfl_xor_sync(0xffffffffu, key, o);
-                    key = other > key ? other : key;
+                    const unsigned long long best = __shfl_xor_sync(0xffffffffu, key, o);
+                    key = best > key ? best : key;
                 }
                 if (r == 0 && t < p.T) atomicMax(p.e.keys + t, key);
             }
@@ -268,9 +295,13 @@ __global__ void __launch_bounds__(256) k_linear_f32(const RowsParams p) {
     }
 }
 
-template <int NT, int AHEAD>
+template <int NT, int AHEAD, int KS>
 int launch_mma(dc_ctx* ctx, const MmaParams& p) {
-    return dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD>, dim3((p.N + 15) / 16), dim3(LM_WARPS * 32), 0, p);
+    const int tiles = (p.N + 15) / 16;
+    const dim3 block(LM_WARPS * 32);
+    if (KS > 1) return dc_launch_cluster(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD, KS>, dim3(tiles * KS), block, 0, KS, p);
+    const int room = LM_CTAS * ctx->num_sms, rounds = (tiles + room - 1) / room;
+    return dc_launch(ctx, "k_linear_mma", k_linear_mma<NT, AHEAD, 1>, dim3((tiles + rounds - 1) / rounds), block, 0, p);
 }
 
 dc_lin_epi clipped(const dc_lin& w, dc_lin_epi e) {
@@ -285,10 +316,12 @@ bool epi_ok(const dc_lin_epi& e) { return e.pair0 >= (1 << 30) || e.pair0 % DC_P
 int dc_launch_linear_mma(dc_ctx* ctx, const dc_lin& w, const __nv_bfloat16* x, int ldx, int T, const dc_lin_epi& epi) {
     if (T < 1 || T > DC_MAX_T || ((uintptr_t)x & 15) || (ldx & 7) || (w.N & 7) || !epi_ok(epi)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_mma: bad operand");
     MmaParams p = {w.w, w.N, w.K, w.ld, x, ldx, T, clipped(w, epi)};
-    // a small matrix needs more of it in flight per warp, a large one has enough warps
-    const bool small = (w.N + 15) / 16 <= 2 * ctx->num_sms;
-    if (T <= 8) return small ? launch_mma<1, 4>(ctx, p) : launch_mma<1, 2>(ctx, p);
-    return small ? launch_mma<2, 4>(ctx, p) : launch_mma<2, 2>(ctx, p);
+    // fewer tiles than SMs: long rows are shared by a cluster, short ones need more in flight per warp
+    const int tiles = (w.N + 15) / 16;
+    if (2 * tiles <= ctx->num_sms && w.K >= 2048) return T <= 8 ? launch_mma<1, 2, 4>(ctx, p) : launch_mma<2, 2, 4>(ctx, p);
+    if (tiles <= ctx->num_sms && w.K >= 4096) return T <= 8 ? launch_mma<1, 2, 2>(ctx, p) : launch_mma<2, 2, 2>(ctx, p);
+    if (tiles <= ctx->num_sms) return T <= 8 ? launch_mma<1, 4, 1>(ctx, p) : launch_mma<2, 4, 1>(ctx, p);
+    return T <= 8 ? launch_mma<1, 2, 1>(ctx, p) : launch_mma<2, 2, 1>(ctx, p);
 }
 
 int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, const dc_lin_epi& epi) {

@@ -4,6 +4,8 @@
 // A cached token is one row: the turned keys of all key heads, then their values.  Steps of up to DC_MAX_T tokens and f32
 // models take every token alone (k_gqa_tokens: keys split over CTAs, k_gqa_join); prompt-sized steps of bf16 models run
 // tiles of queries over the cached rows with bf16 products (k_gqa_prompt).  Scores, weights and their sums are f32.
+#include <algorithm>
+
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -19,6 +21,9 @@ using namespace dc;
 
 namespace {
 
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf2(a, b); }
+
 // ---------------------------------------------------------------- norms, rotation, cache write
 struct PrepParams {
     const float* proj;
@@ -31,53 +36,67 @@ struct PrepParams {
     __nv_bfloat16* qb;       // instead of q
 };
 
-// One CTA per token.
+// One CTA per token and part: the last part is the keys and values, the others share the query heads (every one sums up
+// the whole projection's squares).
 template <typename TC>
 __global__ void __launch_bounds__(256) k_gqa_prep(const PrepParams p) {
     __shared__ float red[33];
     pdl_launch_dependents();
+    const bool keys = blockIdx.y == gridDim.y - 1;
+    const int parts = gridDim.y - 1, share = (p.heads + parts - 1) / parts;
+    const int h0 = keys ? 0 : blockIdx.y * share, h1 = keys ? p.kv_heads : min(p.heads, h0 + share), n = (keys ? p.kv_heads : p.heads) * p.dim;
+    const int pitch = keys ? p.dim_p : p.ldq, half = pitch / 2;
+    const float* w = keys ? p.k_norm : p.q_norm;
     pdl_wait();
-    const int t = blockIdx.x, pos = min(max(p.positions[t], 0), p.max_pos - 1), Q = p.heads * p.dim, K = p.kv_heads * p.dim;
-    const float *row = p.proj + (size_t)t * p.ldp, *cs = p.cos_sin + (size_t)pos * p.rot;
+    const int t = blockIdx.x, pos = min(max(p.positions[t], 0), p.max_pos - 1);
+    const float *x = p.proj + (size_t)t * p.ldp + (keys ? p.off_k : p.off_q), *cs = p.cos_sin + (size_t)pos * p.rot;
     TC* cache = reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos);
-    auto inverse_rms = [&](const float* x, int n) {
-        float ss = 0.0f;
-#pragma unroll 8
-        for (int i = threadIdx.x; i < n; i += 256) ss = fmaf(x[i], x[i], ss);
-        return 1.0f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
-    };
-    // dimension pair j of a head: normed, turned within the first `rot` dimensions, zero beyond the head
-    auto turned = [&](const float* x, const float* w, float inv, int head, int j, float (&out)[2]) {
-        const int d = 2 * j, at = head * p.dim + d;
-        float u = d < p.dim ? x[at] * inv * w[at] : 0.0f, v = d + 1 < p.dim ? x[at + 1] * inv * w[at + 1] : 0.0f;
-        if (d < p.rot) {
-            const float c = cs[d], s = cs[d + 1], a = u * c - v * s;
-            v = v * c + u * s;
-            u = a;
-        }
-        out[0] = u, out[1] = v;
-    };
-    const float qi = inverse_rms(row + p.off_q, Q), ki = inverse_rms(row + p.off_k, K);
-    const int qh = p.ldq / 2, kh = p.dim_p / 2;
-#pragma unroll 4
-    for (int i = threadIdx.x; i < p.heads * qh; i += 256) {
-        const int h = i / qh, j = i - h * qh;
-        float o[2];
-        turned(row + p.off_q, p.q_norm, qi, h, j, o);
-        const size_t at = ((size_t)t * p.heads + h) * p.ldq + 2 * j;
-        if (p.qb) *reinterpret_cast<uint32_t*>(p.qb + at) = pack_bf2(o[0], o[1]);
-        else *reinterpret_cast<float2*>(p.q + at) = make_float2(o[0], o[1]);
+    float ss = 0.0f;
+    constexpr int B = 8;
+    for (int i0 = threadIdx.x; i0 < n; i0 += 256 * B) {
+        float v[B];
+#pragma unroll
+        for (int j = 0; j < B; ++j) v[j] = i0 + 256 * j < n ? x[i0 + 256 * j] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < B; ++j) ss = fmaf(v[j], v[j], ss);
     }
-    for (int i = threadIdx.x; i < p.kv_heads * kh; i += 256) {
-        const int h = i / kh, j = i - h * kh, d = 2 * j;
-        const float* v = row + p.off_k + h * p.dim + d;
-        float o[2];
-        turned(row + p.off_k, p.k_norm, ki, h, j, o);
-        TC *kd = cache + h * p.dim_p + d, *vd = kd + p.kv_heads * p.dim_p;
-        store_as(kd, o[0]);
-        store_as(kd + 1, o[1]);
-        store_as(vd, d < p.dim ? v[0] : 0.0f);
-        store_as(vd + 1, d + 1 < p.dim ? v[1] : 0.0f);
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+    const bool even = !(p.dim & 1);
+    // a thread takes a pair of dimensions: normed, turned within the first `rot` of a head, zero beyond the head
+    constexpr int U = 4;
+    for (int i0 = threadIdx.x; i0 < (h1 - h0) * half; i0 += 256 * U) {
+        float2 raw[U], nw[U], turn[U];
+        int head[U], dim[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int i = min(i0 + 256 * u, (h1 - h0) * half - 1);
+            head[u] = h0 + i / half, dim[u] = 2 * (i % half);
+            const int at = head[u] * p.dim + dim[u];
+            raw[u] = nw[u] = make_float2(0.0f, 0.0f);
+            turn[u] = make_float2(1.0f, 0.0f);
+            if (dim[u] + 1 < p.dim && even) {
+                raw[u] = *reinterpret_cast<const float2*>(x + at), nw[u] = *reinterpret_cast<const float2*>(w + at);
+            } else {
+                if (dim[u] < p.dim) raw[u].x = x[at], nw[u].x = w[at];
+                if (dim[u] + 1 < p.dim) raw[u].y = x[at + 1], nw[u].y = w[at + 1];
+            }
+            if (dim[u] < p.rot) turn[u] = *reinterpret_cast<const float2*>(cs + dim[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            if (i0 + 256 * u >= (h1 - h0) * half) break;
+            const float a = raw[u].x * inv * nw[u].x, b = raw[u].y * inv * nw[u].y;
+            const float c = a * turn[u].x - b * turn[u].y, d = b * turn[u].x + a * turn[u].y;
+            if (keys) {
+                TC *kd = cache + head[u] * pitch + dim[u], *vd = kd + p.kv_heads * pitch;
+                store_pair(kd, c, d);
+                store_pair(vd, raw[u].x, raw[u].y);
+            } else {
+                const size_t at = ((size_t)t * p.heads + head[u]) * pitch + dim[u];
+                if (p.qb) store_pair(p.qb + at, c, d);
+                else store_pair(p.q + at, c, d);
+            }
+        }
     }
 }
 
@@ -409,8 +428,10 @@ int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, co
                        int max_pos, float* q, __nv_bfloat16* qb) {
     PrepParams p = {proj, ldp, m.off_q, m.off_k, m.heads, m.kv_heads, m.dim, m.dim_p, dc_gqa_ldq(m), m.rot.dims, max_pos, m.q_norm, m.k_norm, m.cos_sin,
                     eps, st.seq_ids, st.positions, cache_ref(c, m.row), q, qb};
-    if (c.f32) return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<float>, dim3(st.T), dim3(256), 0, p);
-    return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<__nv_bfloat16>, dim3(st.T), dim3(256), 0, p);
+    const int parts = st.T > DC_MAX_T ? 1 : std::min(m.heads, (m.heads * m.dim + 511) / 512);      // few tokens: more CTAs each
+    const dim3 grid(st.T, parts + 1), block(256);
+    if (c.f32) return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<float>, grid, block, 0, p);
+    return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<__nv_bfloat16>, grid, block, 0, p);
 }
 
 int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
