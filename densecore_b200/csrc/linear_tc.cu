@@ -39,57 +39,93 @@ __device__ __forceinline__ float quick_clamped(float limit, float gate, float up
     return __fdividef(gate, 1.0f + __expf(-1.702f * gate)) * (up + 1.0f);
 }
 
+// f(v, c0) for every sixteen columns of the warp's tensor-memory lanes that belong to the step; the next ones are on their way
+// meanwhile.
+template <int COLS, typename F>
+__device__ __forceinline__ void each16(uint32_t tmem, int n, F f) {
+    int v[2][16];
+    tmem_ld16(tmem, v[0]);
+    for (int c0 = 0; c0 < COLS && c0 < n; c0 += 32) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int c = c0 + 16 * i;
+            if (c >= n) break;
+            tmem_ld_wait(v[i]);
+            if (c + 16 < COLS && c + 16 < n) tmem_ld16(tmem + c + 16, v[i ^ 1]);
+            f(v[i], c);
+        }
+    }
+}
+
 // Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.
 template <int COLS>
 __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int quarter, int lane) {
-    const int row = row0 + 32 * quarter + lane;
-    for (int c0 = 0; c0 < COLS && t0 + c0 < p.T; c0 += 16) {
-        int v[16];
-        tmem_ld16(tmem + ((uint32_t)(32 * quarter) << 16) + c0, v);
-        tmem_ld_wait();
-        if (row0 + 32 * quarter >= p.e.pair0) {
-            // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
-            const bool up = lane & 1;
-            const int o = (row - p.e.pair0) >> 1;
+    const int row = row0 + 32 * quarter + lane, n = p.T - t0;
+    const dc_lin_epi& e = p.e;
+    tmem += (uint32_t)(32 * quarter) << 16;
+    if (row0 + 32 * quarter >= e.pair0) {
+        // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
+        const bool up = lane & 1, gelu = e.pair_kind == DC_PAIR_GELU;
+        const int o = (row - e.pair0) >> 1, first = up ? 8 : 0;
+        const bool in = o < e.n_pairs;
+        const size_t at = (size_t)(t0 + first) * e.ldp + o;
+        each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
+            float h[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
                 const float mine = __int_as_float(up ? v[i + 8] : v[i]);
                 const float gate = up ? got : mine, val = up ? mine : got;
-                const float h = p.e.pair_kind == DC_PAIR_GELU ? gelu_tanh(gate) * val : quick_clamped(p.e.limit, gate, val);
-                const int t = t0 + c0 + i + (up ? 8 : 0);
-                if (t < p.T && o < p.e.n_pairs) put_pair(p.e, t, o, h);
+                h[i] = gelu ? gelu_tanh(gate) * val : quick_clamped(e.limit, gate, val);
             }
-        } else if (row < p.e.n_store) {
-            const int n = min(16, p.T - t0 - c0);
-            const float bias = p.e.bias ? p.e.bias[row] : 0.0f;
-            const size_t at = (size_t)(t0 + c0) * p.e.ldo + row;
-            if (p.e.outb) {
-                __nv_bfloat16* o = p.e.outb + at;
-                if (row < p.e.silu_rows) {
+            const int m = in ? n - c0 - first : 0;
+            if (e.poutb) {
+                __nv_bfloat16* to = e.poutb + at + (size_t)c0 * e.ldp;
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) v[i] = __float_as_int(quick_silu(__int_as_float(v[i]) + bias));
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) v[i] = __float_as_int(__int_as_float(v[i]) + bias);
-                }
-#pragma unroll
-                for (int i = 0; i < 16; ++i, o += p.e.ldo)
-                    if (i < n) *o = __float2bfloat16_rn(__int_as_float(v[i]));
-            } else if (p.e.add) {
-                float old[16], *o = p.e.out + at;
-#pragma unroll
-                for (int i = 0; i < 16; ++i) old[i] = o[(size_t)min(i, n - 1) * p.e.ldo];        // every load ahead of the stores
-#pragma unroll
-                for (int i = 0; i < 16; ++i, o += p.e.ldo)
-                    if (i < n) *o = old[i] + (__int_as_float(v[i]) + bias);
+                for (int i = 0; i < 8; ++i, to += e.ldp)
+                    if (i < m) *to = __float2bfloat16_rn(h[i]);
             } else {
-                float* o = p.e.out + at;
+                float* to = e.pout + at + (size_t)c0 * e.ldp;
 #pragma unroll
-                for (int i = 0; i < 16; ++i, o += p.e.ldo)
-                    if (i < n) *o = __int_as_float(v[i]) + bias;
+                for (int i = 0; i < 8; ++i, to += e.ldp)
+                    if (i < m) *to = h[i];
             }
-        }
+        });
+        return;
+    }
+    const bool in = row < e.n_store;
+    const float bias = in && e.bias ? e.bias[row] : 0.0f;
+    const size_t at = (size_t)t0 * e.ldo + row;
+    if (e.outb) {
+        const bool act = row < e.silu_rows;
+        each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
+            const int m = in ? n - c0 : 0;
+            __nv_bfloat16* to = e.outb + at + (size_t)c0 * e.ldo;
+#pragma unroll
+            for (int i = 0; i < 16; ++i, to += e.ldo) {
+                const float r = __int_as_float(v[i]) + bias;
+                if (i < m) *to = __float2bfloat16_rn(act ? quick_silu(r) : r);
+            }
+        });
+    } else if (e.add) {
+        each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
+            const int m = in ? n - c0 : 0;
+            float* to = e.out + at + (size_t)c0 * e.ldo;
+            float old[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) old[i] = i < m ? to[(size_t)i * e.ldo] : 0.0f;         // every load ahead of the stores
+#pragma unroll
+            for (int i = 0; i < 16; ++i, to += e.ldo)
+                if (i < m) *to = old[i] + (__int_as_float(v[i]) + bias);
+        });
+    } else {
+        each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
+            const int m = in ? n - c0 : 0;
+            float* to = e.out + at + (size_t)c0 * e.ldo;
+#pragma unroll
+            for (int i = 0; i < 16; ++i, to += e.ldo)
+                if (i < m) *to = __int_as_float(v[i]) + bias;
+        });
     }
 }
 

@@ -27,7 +27,7 @@ __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
 // ---------------------------------------------------------------- norms, rotation, cache write
 struct PrepParams {
     const float* proj;
-    int ldp, off_q, off_k, heads, kv_heads, dim, dim_p, ldq, rot, max_pos;
+    int ldp, off_q, off_k, heads, kv_heads, dim, dim_p, ldq, rot, max_pos, lanes;
     const float *q_norm, *k_norm, *cos_sin;
     float eps;
     const int32_t *seq_ids, *positions;
@@ -37,64 +37,73 @@ struct PrepParams {
 };
 
 // One CTA per token and part: the last part is the keys and values, the others share the query heads (every one sums up
-// the whole projection's squares).
+// the whole projection's squares).  A thread has one pair of dimensions (2^lanes threads a head) of several heads.
 template <typename TC>
 __global__ void __launch_bounds__(256) k_gqa_prep(const PrepParams p) {
+    constexpr int U = 4, B = 8;
     __shared__ float red[33];
     pdl_launch_dependents();
     const bool keys = blockIdx.y == gridDim.y - 1;
     const int parts = gridDim.y - 1, share = (p.heads + parts - 1) / parts;
     const int h0 = keys ? 0 : blockIdx.y * share, h1 = keys ? p.kv_heads : min(p.heads, h0 + share), n = (keys ? p.kv_heads : p.heads) * p.dim;
-    const int pitch = keys ? p.dim_p : p.ldq, half = pitch / 2;
-    const float* w = keys ? p.k_norm : p.q_norm;
+    const int pitch = keys ? p.dim_p : p.ldq, step = 256 >> p.lanes;
+    const int first = h0 + (threadIdx.x >> p.lanes), d = 2 * (threadIdx.x & ((1 << p.lanes) - 1));
+    const float* w = (keys ? p.k_norm : p.q_norm) + d;
+    const bool whole = d + 1 < p.dim && !(p.dim & 1), one = d < p.dim, two = d + 1 < p.dim;
     pdl_wait();
-    const int t = blockIdx.x, pos = min(max(p.positions[t], 0), p.max_pos - 1);
-    const float *x = p.proj + (size_t)t * p.ldp + (keys ? p.off_k : p.off_q), *cs = p.cos_sin + (size_t)pos * p.rot;
-    TC* cache = reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos);
-    float ss = 0.0f;
-    constexpr int B = 8;
-    for (int i0 = threadIdx.x; i0 < n; i0 += 256 * B) {
-        float v[B];
-#pragma unroll
-        for (int j = 0; j < B; ++j) v[j] = i0 + 256 * j < n ? x[i0 + 256 * j] : 0.0f;
-#pragma unroll
-        for (int j = 0; j < B; ++j) ss = fmaf(v[j], v[j], ss);
-    }
-    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
-    const bool even = !(p.dim & 1);
-    // a thread takes a pair of dimensions: normed, turned within the first `rot` of a head, zero beyond the head
-    constexpr int U = 4;
-    for (int i0 = threadIdx.x; i0 < (h1 - h0) * half; i0 += 256 * U) {
-        float2 raw[U], nw[U], turn[U];
-        int head[U], dim[U];
+    const int t = blockIdx.x, at_pos = p.positions[t], seq = p.seq_ids[t];
+    const float* x = p.proj + (size_t)t * p.ldp + (keys ? p.off_k : p.off_q);
+    float2 raw[U], nw[U];
+    auto fetch = [&](int head0) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
-            const int i = min(i0 + 256 * u, (h1 - h0) * half - 1);
-            head[u] = h0 + i / half, dim[u] = 2 * (i % half);
-            const int at = head[u] * p.dim + dim[u];
+            const int head = head0 + step * u;
+            const float *xs = x + head * p.dim + d, *ws = w + head * p.dim;
             raw[u] = nw[u] = make_float2(0.0f, 0.0f);
-            turn[u] = make_float2(1.0f, 0.0f);
-            if (dim[u] + 1 < p.dim && even) {
-                raw[u] = *reinterpret_cast<const float2*>(x + at), nw[u] = *reinterpret_cast<const float2*>(w + at);
+            if (head >= h1) continue;
+            if (whole) {
+                raw[u] = *reinterpret_cast<const float2*>(xs), nw[u] = *reinterpret_cast<const float2*>(ws);
             } else {
-                if (dim[u] < p.dim) raw[u].x = x[at], nw[u].x = w[at];
-                if (dim[u] + 1 < p.dim) raw[u].y = x[at + 1], nw[u].y = w[at + 1];
+                if (one) raw[u].x = xs[0], nw[u].x = ws[0];
+                if (two) raw[u].y = xs[1], nw[u].y = ws[1];
             }
-            if (dim[u] < p.rot) turn[u] = *reinterpret_cast<const float2*>(cs + dim[u]);
         }
+    };
+    fetch(first);                                        // on its way while the squares are summed up
+    const int pos = min(max(at_pos, 0), p.max_pos - 1);
+    const float2 turn = d < p.rot ? *reinterpret_cast<const float2*>(p.cos_sin + (size_t)pos * p.rot + d) : make_float2(1.0f, 0.0f);
+    float ss = 0.0f;
+    if ((keys || parts == 1) && h1 - h0 <= U * step) {   // ... from the same values
+#pragma unroll
+        for (int u = 0; u < U; ++u) ss = fmaf(raw[u].x, raw[u].x, fmaf(raw[u].y, raw[u].y, ss));
+    } else {
+        for (int i0 = threadIdx.x; i0 < n; i0 += 256 * B) {
+            float v[B];
+#pragma unroll
+            for (int j = 0; j < B; ++j) v[j] = i0 + 256 * j < n ? x[i0 + 256 * j] : 0.0f;
+#pragma unroll
+            for (int j = 0; j < B; ++j) ss = fmaf(v[j], v[j], ss);
+        }
+    }
+    TC* cache = keys ? reinterpret_cast<TC*>(p.c.arena) + p.c.at(seq, pos) + d : nullptr;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+    if (d >= pitch) return;
+    for (int head0 = first; head0 < h1; head0 += U * step) {
+        if (head0 > first) fetch(head0);
 #pragma unroll
         for (int u = 0; u < U; ++u) {
-            if (i0 + 256 * u >= (h1 - h0) * half) break;
+            const int head = head0 + step * u;
+            if (head >= h1) break;
             const float a = raw[u].x * inv * nw[u].x, b = raw[u].y * inv * nw[u].y;
-            const float c = a * turn[u].x - b * turn[u].y, d = b * turn[u].x + a * turn[u].y;
+            const float c = a * turn.x - b * turn.y, e = b * turn.x + a * turn.y;
             if (keys) {
-                TC *kd = cache + head[u] * pitch + dim[u], *vd = kd + p.kv_heads * pitch;
-                store_pair(kd, c, d);
-                store_pair(vd, raw[u].x, raw[u].y);
+                TC* kd = cache + head * pitch;
+                store_pair(kd, c, e);
+                store_pair(kd + p.kv_heads * pitch, raw[u].x, raw[u].y);
             } else {
-                const size_t at = ((size_t)t * p.heads + head[u]) * pitch + dim[u];
-                if (p.qb) store_pair(p.qb + at, c, d);
-                else store_pair(p.q + at, c, d);
+                const size_t at = ((size_t)t * p.heads + head) * pitch + d;
+                if (p.qb) store_pair(p.qb + at, c, e);
+                else store_pair(p.q + at, c, e);
             }
         }
     }
@@ -254,10 +263,10 @@ struct PromptParams {
 
 constexpr int PK = 64;           // keys per tile
 
-// One CTA per (PQ queries of one entry, head), sixteen queries a warp; key and value tiles in a ring of ST stages.
-// DP: head size, padded.
+// One CTA per (PQ queries of one entry, head), sixteen queries a warp; key and value tiles in a ring of ST stages, two
+// CTAs an SM.  DP: head size, padded.
 template <int DP, int PQ, int ST>
-__global__ void __launch_bounds__(2 * PQ) k_gqa_prompt(const PromptParams p) {
+__global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const PromptParams p) {
     constexpr int LD = DP + 8, NT = 2 * PQ, CH = DP / 8;
     extern __shared__ __align__(16) uint8_t smem[];
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);     // [PQ][LD]
@@ -426,7 +435,9 @@ float sink_of(const dc_gqa_mixer& m) { return m.sink ? m.sink_score : -INFINITY;
 
 int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
                        int max_pos, float* q, __nv_bfloat16* qb) {
-    PrepParams p = {proj, ldp, m.off_q, m.off_k, m.heads, m.kv_heads, m.dim, m.dim_p, dc_gqa_ldq(m), m.rot.dims, max_pos, m.q_norm, m.k_norm, m.cos_sin,
+    int lanes = 3;               // a head's pairs, padding included, up to a power of two
+    while (2 << lanes < dc_gqa_ldq(m)) ++lanes;
+    PrepParams p = {proj, ldp, m.off_q, m.off_k, m.heads, m.kv_heads, m.dim, m.dim_p, dc_gqa_ldq(m), m.rot.dims, max_pos, lanes, m.q_norm, m.k_norm, m.cos_sin,
                     eps, st.seq_ids, st.positions, cache_ref(c, m.row), q, qb};
     const int parts = st.T > DC_MAX_T ? 1 : std::min(m.heads, (m.heads * m.dim + 511) / 512);      // few tokens: more CTAs each
     const dim3 grid(st.T, parts + 1), block(256);
@@ -456,8 +467,8 @@ int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, 
     } while (0)
     if (m.dim <= 32) DC_PROMPT(32, 128, 3);
     if (m.dim <= 64) DC_PROMPT(64, 128, 3);
-    if (m.dim <= 96) DC_PROMPT(96, 128, 3);
-    if (m.dim <= 128) DC_PROMPT(128, 128, 3);
+    if (m.dim <= 96) DC_PROMPT(96, 128, 2);
+    if (m.dim <= 128) DC_PROMPT(128, 128, 2);
     DC_PROMPT(256, 64, 2);
 #undef DC_PROMPT
 }

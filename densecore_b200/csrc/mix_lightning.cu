@@ -38,15 +38,19 @@ struct ChunkParams {
     int ldy;
 };
 
-// rows x cols (a multiple of eight) of a bf16 matrix into shared memory; what lies beyond n rows or `valid` columns is zero
+// CT rows x cols (a multiple of eight) of a bf16 matrix into shared memory by 128 threads, eight a row; what lies beyond n
+// rows or `valid` columns is zero
 __device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int ldd, const __nv_bfloat16* src, int lds, int n, int valid, int cols, bool vec) {
     if (vec) {
-        const int ch = cols / 8;
-        for (int i = threadIdx.x; i < CT * ch; i += blockDim.x) {
-            const int r = i / ch, c = 8 * (i - r * ch);
-            const bool ok = r < n && c < valid;
-            cp_async16z(smem_u32(dst + r * ldd + c), ok ? src + (size_t)r * lds + c : src, ok);
-        }
+        const int r0 = threadIdx.x >> 3, c0 = 8 * (threadIdx.x & 7);
+        const uint32_t to = smem_u32(dst + r0 * ldd + c0);
+        const __nv_bfloat16* from = src + (size_t)r0 * lds + c0;
+        for (int c = 0; c0 + c < cols; c += 64)
+#pragma unroll
+            for (int i = 0; i < CT / 16; ++i) {
+                const bool ok = r0 + 16 * i < n && c0 + c < valid;
+                cp_async16z(to + 2 * (16 * i * ldd + c), ok ? from + (size_t)(16 * i) * lds + c : src, ok);
+            }
     } else {
         for (int i = threadIdx.x; i < CT * cols; i += blockDim.x) {
             const int r = i / cols, c = i - r * cols;
@@ -99,16 +103,16 @@ __global__ void __launch_bounds__(128) k_lightning_sums(const ChunkParams p) {
             split3(bf_lo(v[i]) * w.x, bf_hi(v[i]) * w.y, t);
             a[0][i] = t[0], a[1][i] = t[1], a[2][i] = t[2];
         }
+        uint32_t b[4][4];
 #pragma unroll
-        for (int np = 0; np < 4; ++np) {
-            uint32_t b[4];
-            ldsm_x4_t(smem_u32(sK + (16 * ks + (mi & 1) * 8 + r8) * LDT + 16 * np + (mi >> 1) * 8), b);
+        for (int np = 0; np < 4; ++np) ldsm_x4_t(smem_u32(sK + (16 * ks + (mi & 1) * 8 + r8) * LDT + 16 * np + (mi >> 1) * 8), b[np]);
 #pragma unroll
-            for (int i = 2; i >= 0; --i) {
-                mma_bf16(acc[2 * np], a[i], b[0], b[1]);
-                mma_bf16(acc[2 * np + 1], a[i], b[2], b[3]);
+        for (int i = 2; i >= 0; --i)             // products of one term are independent of each other
+#pragma unroll
+            for (int np = 0; np < 4; ++np) {
+                mma_bf16(acc[2 * np], a[i], b[np][0], b[np][1]);
+                mma_bf16(acc[2 * np + 1], a[i], b[np][2], b[np][3]);
             }
-        }
     }
     float* out = p.state + ((size_t)blockIdx.x * p.heads + h) * p.vdim * p.dim;
 #pragma unroll
@@ -175,158 +179,165 @@ __global__ void __launch_bounds__(256) k_lightning_carry(const ChunkParams p) {
     put(slot, s);
 }
 
-// One CTA per (chunk, head).  Inside the chunk a warp has sixteen queries; against the state it has sixteen value columns
-// of the tile, so that a column of the state is taken apart once.
-__global__ void __launch_bounds__(128) k_lightning_out(const ChunkParams p) {
+// One CTA per (chunk, head, tile of 64 value columns).  Against the state a warp has sixteen value columns and all queries,
+// so that a column of the state is taken apart once; inside the chunk it has sixteen queries.  Shared memory is used twice:
+// keys and values take the place of the state's columns, the answers from the state that of the queries.
+struct OutSmem {
+    int ldq, lds, first, second;                        // pitches; bytes of the two regions
+    __host__ __device__ explicit OutSmem(int dim) {
+        const int dp = (dim + 15) & ~15;
+        ldq = dp + 8, lds = dp + 8;
+        const int queries = CT * ldq * 2, answers = CT * (TE + 4) * 4, state = TE * lds * 4, tokens = CT * (ldq + LDT) * 2;
+        first = queries > answers ? queries : answers;
+        second = state > tokens ? state : tokens;
+    }
+};
+
+__global__ void __launch_bounds__(128, 4) k_lightning_out(const ChunkParams p) {
     extern __shared__ __align__(16) uint8_t smem[];
     __shared__ float spow[CT + 1];
-    const int dp = (p.dim + 15) & ~15, LDQ = dp + 8;
+    const OutSmem L(p.dim);
+    const int dp = (p.dim + 15) & ~15, LDQ = L.ldq, LDS = L.lds;
     constexpr int LDO = TE + 4;
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);     // [CT][LDQ]
-    __nv_bfloat16* sK = sQ + CT * LDQ;                              // [CT][LDQ]
+    float* sO = reinterpret_cast<float*>(smem);                     // [CT][LDO]
+    float* sS = reinterpret_cast<float*>(smem + L.first);           // [TE][LDS]: columns of the state
+    __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(smem + L.first);    // [CT][LDQ]
     __nv_bfloat16* sV = sK + CT * LDQ;                              // [CT][LDT]
-    float* sO = reinterpret_cast<float*>(sV + CT * LDT);            // [CT][LDO]
     pdl_launch_dependents();
     pdl_wait();
     const BlockRef br = block_at<CT>(p.starts, p.E, blockIdx.x);
     if (br.n <= 0) return;
-    const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, mi = lane >> 3, r8 = lane & 7;
+    const int h = blockIdx.y, e0 = blockIdx.z * TE, ne = min(TE, p.vdim - e0);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, mi = lane >> 3, r8 = lane & 7;
     const __nv_bfloat16* row = p.act + (size_t)br.t0 * p.ld;
+    const float* S = p.state + (((size_t)blockIdx.x * p.heads + h) * p.vdim + e0) * p.dim;
     load_tile(sQ, LDQ, row + p.off_q + h * p.dim, p.ld, br.n, p.dim, dp, p.vec);
-    load_tile(sK, LDQ, row + p.off_k + h * p.dim, p.ld, br.n, p.dim, dp, p.vec);
-    load_tile(sV, LDT, row + p.off_v + h * p.vdim, p.ld, br.n, p.vdim, TE, p.vec);
+    if (p.dim % 4 == 0) {
+        const int r0 = tid >> 3, c0 = 4 * (tid & 7);
+        for (int c = c0; c < dp; c += 32)
+#pragma unroll
+            for (int i = 0; i < TE / 16; ++i) {
+                const int r = r0 + 16 * i;
+                const bool ok = r < ne && c < p.dim;
+                cp_async16z(smem_u32(sS + r * LDS + c), ok ? S + r * p.dim + c : S, ok);
+            }
+    } else {
+        for (int i = tid; i < TE * dp; i += 128) {
+            const int r = i / dp, c = i - r * dp;
+            sS[r * LDS + c] = r < ne && c < p.dim ? S[(size_t)r * p.dim + c] : 0.0f;
+        }
+    }
     cp_async_commit();
     if (tid <= CT) spow[tid] = powf(p.decay[h], (float)tid);
     cp_async_wait<0>();
     __syncthreads();
-    // weights a^(t - i) (q_t . k_i) of the warp's queries, as operands of three bf16 terms
-    uint32_t pa[3][CT / 16][4];
-    {
-        float s[8][4];
+    // ---- S0^T q for the columns 16 warp .. + 15, all queries
+    float acc[4][2][4];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
-        const uint32_t qa = smem_u32(sQ + (16 * warp + (mi & 1) * 8 + r8) * LDQ + (mi >> 1) * 8);
-        const uint32_t ka = smem_u32(sK + ((mi >> 1) * 8 + r8) * LDQ + (mi & 1) * 8);
-        for (int kk = 0; kk < dp; kk += 16) {
-            uint32_t a[4];
-            ldsm_x4(qa + 2 * kk, a);
+    for (int m = 0; m < 4; ++m)
 #pragma unroll
-            for (int np = 0; np < 4; ++np) {
-                if (np > warp) break;                               // keys after every query of the warp
-                uint32_t b[4];
-                ldsm_x4(ka + 2 * (16 * np * LDQ + kk), b);
-                mma_bf16(s[2 * np], a, b[0], b[1]);
-                mma_bf16(s[2 * np + 1], a, b[2], b[3]);
-            }
-        }
+        for (int j = 0; j < 2; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.0f;
+    for (int kk = 0; kk < dp; kk += 16) {
+        uint32_t b[2][2][3], a[4][4];
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
+        for (int m = 0; m < 4; ++m) ldsm_x4(smem_u32(sQ + (16 * m + (mi & 1) * 8 + r8) * LDQ + (mi >> 1) * 8 + kk), a[m]);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int back = 16 * warp + g + (j >> 1) * 8 - (8 * nt + 2 * q + (j & 1));
-                s[nt][j] = back >= 0 ? s[nt][j] * spow[back] : 0.0f;
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const float2 f = *reinterpret_cast<const float2*>(sS + (16 * warp + 8 * j + g) * LDS + kk + 8 * i + 2 * q);
+                split3(f.x, f.y, b[j][i]);
             }
 #pragma unroll
-        for (int ks = 0; ks < CT / 16; ++ks)
+        for (int i = 2; i >= 0; --i)             // products of one term are independent of each other
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                uint32_t t[3];
-                split3(s[2 * ks + (i >> 1)][2 * (i & 1)], s[2 * ks + (i >> 1)][2 * (i & 1) + 1], t);
-                pa[0][ks][i] = t[0], pa[1][ks][i] = t[1], pa[2][ks][i] = t[2];
+            for (int m = 0; m < 4; ++m) {
+                mma_bf16(acc[m][0], a[m], b[0][0][i], b[0][1][i]);
+                mma_bf16(acc[m][1], a[m], b[1][0][i], b[1][1][i]);
             }
     }
-    const float* S = p.state + ((size_t)blockIdx.x * p.heads + h) * p.vdim * p.dim;
-    const bool even = !(p.dim & 1);
-    for (int e0 = 0; e0 < p.vdim; e0 += TE) {
-        // ---- S0^T q for the tile's columns 16 warp .. + 15, all queries
-        {
-            float acc[4][2][4];
+    __syncthreads();
+    load_tile(sK, LDQ, row + p.off_k + h * p.dim, p.ld, br.n, p.dim, dp, p.vec);
+    load_tile(sV, LDT, row + p.off_v + h * p.vdim + e0, p.ld, br.n, ne, TE, p.vec);
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    // ---- the chunk's own tokens: weights a^(t - i) (q_t . k_i) of the warp's queries, then the values
+    float s[8][4];
 #pragma unroll
-            for (int m = 0; m < 4; ++m)
+    for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+    const uint32_t qa = smem_u32(sQ + (16 * warp + (mi & 1) * 8 + r8) * LDQ + (mi >> 1) * 8);
+    const uint32_t ka = smem_u32(sK + ((mi >> 1) * 8 + r8) * LDQ + (mi & 1) * 8);
+    for (int kk = 0; kk < dp; kk += 16) {
+        uint32_t a[4];
+        ldsm_x4(qa + 2 * kk, a);
 #pragma unroll
-                for (int j = 0; j < 2; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.0f;
-            auto fetch = [&](int kk, float2 (&f)[2][2]) {
-#pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) {
-                        const int e = e0 + 16 * warp + 8 * j + g, d = kk + 8 * i + 2 * q;
-                        const float* at = S + (size_t)e * p.dim + d;
-                        f[j][i] = make_float2(0.0f, 0.0f);
-                        if (e < p.vdim && d + 1 < p.dim && even) f[j][i] = *reinterpret_cast<const float2*>(at);
-                        else if (e < p.vdim) {
-                            if (d < p.dim) f[j][i].x = at[0];
-                            if (d + 1 < p.dim) f[j][i].y = at[1];
-                        }
-                    }
-            };
-            float2 next[2][2];
-            fetch(0, next);
-            for (int kk = 0; kk < dp; kk += 16) {
-                float2 f[2][2];
-#pragma unroll
-                for (int j = 0; j < 2; ++j) f[j][0] = next[j][0], f[j][1] = next[j][1];
-                if (kk + 16 < dp) fetch(kk + 16, next);
-                uint32_t b[2][2][3];
-#pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) split3(f[j][i].x, f[j][i].y, b[j][i]);
-#pragma unroll
-                for (int m = 0; m < 4; ++m) {
-                    uint32_t a[4];
-                    ldsm_x4(smem_u32(sQ + (16 * m + (mi & 1) * 8 + r8) * LDQ + (mi >> 1) * 8 + kk), a);
-#pragma unroll
-                    for (int i = 2; i >= 0; --i) {
-                        mma_bf16(acc[m][0], a, b[0][0][i], b[0][1][i]);
-                        mma_bf16(acc[m][1], a, b[1][0][i], b[1][1][i]);
-                    }
-                }
-            }
-#pragma unroll
-            for (int m = 0; m < 4; ++m)
-#pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const int t = 16 * m + g + 8 * (i >> 1);
-                        sO[t * LDO + 16 * warp + 8 * j + 2 * q + (i & 1)] = acc[m][j][i] * spow[t + 1];
-                    }
-        }
-        cp_async_wait<0>();
-        __syncthreads();
-        // ---- the chunk's own tokens
-        float o[8][4];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
-#pragma unroll
-        for (int ks = 0; ks < CT / 16; ++ks) {
-            if (ks > warp) break;
-#pragma unroll
-            for (int np = 0; np < 4; ++np) {
-                uint32_t b[4];
-                ldsm_x4_t(smem_u32(sV + (16 * ks + (mi & 1) * 8 + r8) * LDT + 16 * np + (mi >> 1) * 8), b);
-#pragma unroll
-                for (int i = 2; i >= 0; --i) {
-                    mma_bf16(o[2 * np], pa[i][ks], b[0], b[1]);
-                    mma_bf16(o[2 * np + 1], pa[i][ks], b[2], b[3]);
-                }
-            }
-        }
-#pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int t = 16 * warp + g + 8 * (i >> 1), c = 8 * nt + 2 * q + (i & 1);
-                if (t < br.n && e0 + c < p.vdim)
-                    p.y[(size_t)(br.t0 + t) * p.ldy + (size_t)h * p.vdim + e0 + c] = o[nt][i] + sO[t * LDO + c];
-            }
-        if (e0 + TE < p.vdim) {
-            __syncthreads();
-            load_tile(sV, LDT, row + p.off_v + h * p.vdim + e0 + TE, p.ld, br.n, p.vdim - e0 - TE, TE, p.vec);
-            cp_async_commit();
+        for (int np = 0; np < 4; ++np) {
+            if (np > warp) break;                                   // keys after every query of the warp
+            uint32_t b[4];
+            ldsm_x4(ka + 2 * (16 * np * LDQ + kk), b);
+            mma_bf16(s[2 * np], a, b[0], b[1]);
+            mma_bf16(s[2 * np + 1], a, b[2], b[3]);
         }
     }
+    __syncthreads();             // every warp is done with the queries
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int t = 16 * m + g + 8 * i;
+                *reinterpret_cast<float2*>(sO + t * LDO + 16 * warp + 8 * j + 2 * q) = make_float2(acc[m][j][2 * i] * spow[t + 1], acc[m][j][2 * i + 1] * spow[t + 1]);
+            }
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int back = 16 * warp + g + (j >> 1) * 8 - (8 * nt + 2 * q + (j & 1));
+            s[nt][j] = back >= 0 ? s[nt][j] * spow[back] : 0.0f;
+        }
+    float o[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+#pragma unroll
+    for (int ks = 0; ks < CT / 16; ++ks) {
+        if (ks > warp) break;
+        uint32_t pa[3][4], b[4][4];
+#pragma unroll
+        for (int np = 0; np < 4; ++np) ldsm_x4_t(smem_u32(sV + (16 * ks + (mi & 1) * 8 + r8) * LDT + 16 * np + (mi >> 1) * 8), b[np]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            uint32_t t[3];
+            split3(s[2 * ks + (i >> 1)][2 * (i & 1)], s[2 * ks + (i >> 1)][2 * (i & 1) + 1], t);
+            pa[0][i] = t[0], pa[1][i] = t[1], pa[2][i] = t[2];
+        }
+#pragma unroll
+        for (int i = 2; i >= 0; --i)
+#pragma unroll
+            for (int np = 0; np < 4; ++np) {
+                mma_bf16(o[2 * np], pa[i], b[np][0], b[np][1]);
+                mma_bf16(o[2 * np + 1], pa[i], b[np][2], b[np][3]);
+            }
+    }
+    __syncthreads();
+    const bool even = !(p.vdim & 1);
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int t = 16 * warp + g + 8 * i, c = 8 * nt + 2 * q;
+            if (t >= br.n || c >= ne) continue;
+            const float2 f = *reinterpret_cast<const float2*>(sO + t * LDO + c);
+            float* y = p.y + (size_t)(br.t0 + t) * p.ldy + (size_t)h * p.vdim + e0 + c;
+            if (even) {
+                *reinterpret_cast<float2*>(y) = make_float2(o[nt][2 * i] + f.x, o[nt][2 * i + 1] + f.y);
+            } else {
+                y[0] = o[nt][2 * i] + f.x;
+                if (c + 1 < ne) y[1] = o[nt][2 * i + 1] + f.y;
+            }
+        }
 }
 
 }  // namespace
@@ -337,11 +348,12 @@ int dc_launch_lightning_chunks(dc_ctx* ctx, const dc_lightning_mixer& m, const d
                                int lda, float* chunk_state, float* y, int ldy) {
     ChunkParams p = {act, lda, m.off_q, m.off_k, m.off_v, m.heads, m.dim, m.vdim, m.decay, chunk_state, sr.base, sr.slot_bytes, sr.state_off, st.seq_ids,
                      st.positions, st.starts, st.E, m.dim % 8 == 0 && m.vdim % 8 == 0 && lda % 8 == 0, y, ldy};
-    const int nc = dc_lightning_chunks(st.T, st.E), size = m.dim * m.vdim, dp = (m.dim + 15) & ~15;
+    const int nc = dc_lightning_chunks(st.T, st.E), size = m.dim * m.vdim;
     DC_TRY(dc_launch(ctx, "k_lightning_sums", k_lightning_sums, dim3(nc, m.heads, ((m.dim + 63) / 64) * ((m.vdim + TE - 1) / TE)), dim3(128), 0, p));
     if (size % 4 == 0) DC_TRY(dc_launch(ctx, "k_lightning_carry", k_lightning_carry<4>, dim3((size / 4 + 255) / 256, m.heads, st.E), dim3(256), 0, p));
     else DC_TRY(dc_launch(ctx, "k_lightning_carry", k_lightning_carry<1>, dim3((size + 255) / 256, m.heads, st.E), dim3(256), 0, p));
-    const int bytes = (2 * CT * (dp + 8) + CT * LDT) * 2 + CT * (TE + 4) * 4;
+    const OutSmem L(m.dim);
+    const int bytes = L.first + L.second;
     DC_TRY(dc_kernel_setup(ctx, (const void*)k_lightning_out, bytes, "k_lightning_out"));
-    return dc_launch(ctx, "k_lightning_out", k_lightning_out, dim3(nc, m.heads), dim3(128), (size_t)bytes, p);
+    return dc_launch(ctx, "k_lightning_out", k_lightning_out, dim3(nc, m.heads, (m.vdim + TE - 1) / TE), dim3(128), (size_t)bytes, p);
 }

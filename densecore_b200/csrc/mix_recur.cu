@@ -1068,49 +1068,99 @@ __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict_
         store_as(out + (size_t)t * ldm + (size_t)h * vdim + c, r[c] * inv * w[c] * sigmoid(gate[(size_t)t * ldg + (size_t)h * vdim + c]));
 }
 
-// One CTA per (token, norm group).  GATE 0: y over its root mean square, times w; 1: y silu(z) first (ssd); 2: times
-// sigmoid(z) afterwards (linear attention).
-template <int GATE, typename TZ, typename TO, int NT>
-__global__ void __launch_bounds__(NT) k_gate_group_norm(const float* __restrict__ y, int ldy, const TZ* __restrict__ z, int ldz,
+// ssd: one CTA per (token, norm group): y silu(z) (unless gated already), over its root mean square, times w
+template <typename TO, int NT>
+__global__ void __launch_bounds__(NT) k_gate_group_norm(const float* __restrict__ y, int ldy, const float* __restrict__ z, int ldz,
                                                          const float* __restrict__ w, int n, float eps, TO* __restrict__ out, int ldm) {
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.y, c0 = blockIdx.x * n;
     const float* yr = y + (size_t)t * ldy + c0;
-    const TZ* zr = GATE ? z + (size_t)t * ldz + c0 : nullptr;
+    const float* zr = z ? z + (size_t)t * ldz + c0 : nullptr;
     constexpr int KEEP = 8;      // values per thread kept between the two passes
-    auto value = [&](int i) { return GATE == 1 ? yr[i] * silu(load_as(zr + i)) : yr[i]; };
-    float v[KEEP], g[KEEP], wv[KEEP], ss = 0.0f;
+    float v[KEEP], ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const int i = threadIdx.x + NT * j;
-        v[j] = i < n ? value(i) : 0.0f;
-        if (GATE == 2) g[j] = i < n ? load_as(zr + i) : 0.0f;
-        wv[j] = i < n ? w[c0 + i] : 0.0f;
+        v[j] = i < n ? (zr ? yr[i] * silu(zr[i]) : yr[i]) : 0.0f;
         ss = fmaf(v[j], v[j], ss);
     }
     for (int i = threadIdx.x + NT * KEEP; i < n; i += NT) {
-        const float x = value(i);
+        const float x = zr ? yr[i] * silu(zr[i]) : yr[i];
         ss = fmaf(x, x, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const int i = threadIdx.x + NT * j;
-        if (i < n) store_as(out + (size_t)t * ldm + c0 + i, v[j] * inv * wv[j] * (GATE == 2 ? sigmoid(g[j]) : 1.0f));
+        if (i < n) store_as(out + (size_t)t * ldm + c0 + i, v[j] * inv * w[c0 + i]);
     }
     for (int i = threadIdx.x + NT * KEEP; i < n; i += NT)
-        store_as(out + (size_t)t * ldm + c0 + i, value(i) * inv * w[c0 + i] * (GATE == 2 ? sigmoid(load_as(zr + i)) : 1.0f));
+        store_as(out + (size_t)t * ldm + c0 + i, (zr ? yr[i] * silu(zr[i]) : yr[i]) * inv * w[c0 + i]);
 }
 
 // small groups get small CTAs: more of them are resident
-template <int GATE, typename TZ, typename TO>
-int launch_group_norm(dc_ctx* ctx, const float* y, int ldy, const TZ* z, int ldz, const float* w, int n, int groups, int T, float eps, TO* out, int ldm) {
+template <typename TO>
+int launch_group_norm(dc_ctx* ctx, const float* y, int ldy, const float* z, int ldz, const float* w, int n, int groups, int T, float eps, TO* out, int ldm) {
     const dim3 grid(groups, T);
-    if (n <= 512) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<GATE, TZ, TO, 64>, grid, dim3(64), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
-    if (n <= 2048) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<GATE, TZ, TO, 256>, grid, dim3(256), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
-    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<GATE, TZ, TO, 512>, grid, dim3(512), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+    if (n <= 512) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 64>, grid, dim3(64), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+    return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 256>, grid, dim3(256), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
+}
+
+// Four neighbouring values as f32.
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w)); }
+
+// lightning: one CTA per token: y over its root mean square, times w, times sigmoid(gate).  Rows are padded to multiples of
+// eight (what the padding holds does not matter); KEEP: groups of four values of a thread.
+template <int KEEP, typename TZ, typename TO>
+__global__ void __launch_bounds__(256) k_norm_gate(const float* __restrict__ y, int ldy, const TZ* __restrict__ gate, int ldz, const float* __restrict__ w,
+                                                   int n, float eps, TO* __restrict__ out, int ldm) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    float4 v[KEEP], g[KEEP], wv[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = 4 * (threadIdx.x + 256 * j);
+        wv[j] = i < n ? load4(w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    pdl_wait();
+    const int t = blockIdx.x;
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = 4 * (threadIdx.x + 256 * j);
+        v[j] = g[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n) v[j] = load4(y + (size_t)t * ldy + i), g[j] = load4(gate + (size_t)t * ldz + i);
+        if (i + 1 >= n) v[j].y = 0.0f;
+        if (i + 2 >= n) v[j].z = 0.0f;
+        if (i + 3 >= n) v[j].w = 0.0f;
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = 4 * (threadIdx.x + 256 * j);
+        if (i < n)
+            store4(out + (size_t)t * ldm + i, make_float4(v[j].x * inv * wv[j].x * sigmoid(g[j].x), v[j].y * inv * wv[j].y * sigmoid(g[j].y),
+                                                          v[j].z * inv * wv[j].z * sigmoid(g[j].z), v[j].w * inv * wv[j].w * sigmoid(g[j].w)));
+    }
+}
+template <typename TZ, typename TO>
+int launch_norm_gate(dc_ctx* ctx, const float* y, int ldy, const TZ* gate, int ldz, const float* w, int n, int T, float eps, TO* out, int ldm) {
+    const dim3 grid(T), block(256);
+    if (n <= 1024) return dc_launch(ctx, "k_norm_gate", k_norm_gate<1, TZ, TO>, grid, block, 0, y, ldy, gate, ldz, w, n, eps, out, ldm);
+    if (n <= 2048) return dc_launch(ctx, "k_norm_gate", k_norm_gate<2, TZ, TO>, grid, block, 0, y, ldy, gate, ldz, w, n, eps, out, ldm);
+    if (n <= 4096) return dc_launch(ctx, "k_norm_gate", k_norm_gate<4, TZ, TO>, grid, block, 0, y, ldy, gate, ldz, w, n, eps, out, ldm);
+    if (n <= 8192) return dc_launch(ctx, "k_norm_gate", k_norm_gate<8, TZ, TO>, grid, block, 0, y, ldy, gate, ldz, w, n, eps, out, ldm);
+    return dc_launch(ctx, "k_norm_gate", k_norm_gate<16, TZ, TO>, grid, block, 0, y, ldy, gate, ldz, w, n, eps, out, ldm);
 }
 
 // ---------------------------------------------------------------- linear attention with a constant decay: decode
@@ -1319,8 +1369,8 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
     DC_TRY(launch_scan<false>(ctx, p, st.E));
     const int n = inner / m.norm_groups;
     const float* z = proj + m.off_z;
-    return mixb ? launch_group_norm<1>(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
-                : launch_group_norm<1>(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
+    return mixb ? launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
+                : launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
 }
 
 int dc_launch_delta_decode(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
@@ -1353,9 +1403,8 @@ int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, 
     else if (dp == 128) DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<4>, grid, block, smem, p));
     else DC_TRY(dc_launch(ctx, "k_ssd_decode", k_ssd_decode<8>, grid, block, smem, p));
     const int n = inner / m.norm_groups;
-    const float* no = nullptr;
-    return mixb ? launch_group_norm<0>(ctx, y, ldy, no, 0, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
-                : launch_group_norm<0>(ctx, y, ldy, no, 0, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
+    return mixb ? launch_group_norm(ctx, y, ldy, nullptr, 0, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
+                : launch_group_norm(ctx, y, ldy, nullptr, 0, m.norm, n, m.norm_groups, st.T, eps, mix, ldm);
 }
 
 size_t dc_lightning_block_floats(const dc_lightning_mixer& m) { return (size_t)m.heads * SSD_BLOCK; }
@@ -1383,6 +1432,6 @@ int dc_launch_lightning_decode(dc_ctx* ctx, const dc_lightning_mixer& m, const d
 int dc_launch_lightning_norm(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const float* y, int ldy, const float* act,
                              const __nv_bfloat16* actb, int lda, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
     const int n = m.heads * m.vdim;
-    return mixb ? launch_group_norm<2>(ctx, y, ldy, actb + m.off_g, lda, m.norm, n, 1, st.T, eps, mixb, ldm)
-                : launch_group_norm<2>(ctx, y, ldy, act + m.off_g, lda, m.norm, n, 1, st.T, eps, mix, ldm);
+    return mixb ? launch_norm_gate(ctx, y, ldy, actb + m.off_g, lda, m.norm, n, st.T, eps, mixb, ldm)
+                : launch_norm_gate(ctx, y, ldy, act + m.off_g, lda, m.norm, n, st.T, eps, mix, ldm);
 }

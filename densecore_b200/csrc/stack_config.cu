@@ -271,6 +271,7 @@ void read_lightning(Reader& r, const dc_json& j, const std::string& p, const std
             d.decays.push_back((float)v.num);
         }
     const int Q = d.heads * d.dim, V = d.heads * d.vdim;
+    if (V > 16384) r.bad(where + ": heads * vdim is above 16384");
     d.off_q = r.matrix(&L->in, p + "q", Q, H);
     d.off_k = r.matrix(&L->in, p + "k", Q, H);
     d.off_v = r.matrix(&L->in, p + "v", V, H);
