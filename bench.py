@@ -379,7 +379,7 @@ def datasun_config(width: int, repeats: int, vocab: int = 32768):
     h = width // 128
     light = {"type": "lightning", "mixer": {"heads": h, "dim": 128, "vdim": 128, "decay": [math.exp(-8.0 * 0.5 ** (i * 10.0 / h)) for i in range(h)]}}
     att = {"type": "attention", "mixer": {"heads": h, "kv_heads": max(1, width // 512), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
-                                          "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}}
+                                          "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 2.0, "original": 2048, "fast": 24.0, "slow": 2.0}}}}
     layers = [dict(ly, mlp={"kind": "dense", "ff": 3 * width, "limit": 7.0}) for ly in (light, light, att) * 2 * repeats]
     return {"architecture": "Datasun", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "layers": layers}
 

@@ -296,8 +296,8 @@ DC_B200_API int dc_b200_model_tensor_names(dc_model* m, const char** names_out, 
  * dc_b200_model_ep_init (expert-parallel runs) and dc_b200_model_finalize. */
 DC_B200_API int dc_b200_model_from_gguf(dc_ctx* ctx, const char* path, int max_seqs, int max_ctx, int ep_rank,
                                         int ep_size, dc_model** out_model);
-/* Layer-list decoders: config.json names an architecture of the library's table ("Garilix") and, per layer, a mixer
- * (channel_delta, latent_attention, mamba2) and a feed-forward.  from_dir reads config.json and model.safetensors
+/* Layer-list decoders: config.json names an architecture of the library's table ("Garilix", "Datasun") and, per layer, a
+ * mixer (channel_delta, latent_attention, mamba2; attention, lightning) and a feed-forward.  from_dir reads config.json and model.safetensors
  * (bf16 matrices, bf16 or f32 vectors); from_config takes the config's text and, for sizes that only a tensor's
  * shape gives, a JSON object name -> shape (dc_b200_model_init_synthetic then fills the weights).  dtype: 0 bf16
  * products with f32 accumulation, 1 everything in f32.  pool_tokens: tokens the cache pool holds (0: max_ctx for
