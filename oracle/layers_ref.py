@@ -97,11 +97,11 @@ def ssd_scan(x, B, C, dt, A_log, D, S):
     return y
 
 
-def windowed_softmax(scores, i, window, sink=None):
-    """scores over keys 0 .. i -> weights; keys with i - j >= window are not seen.  sink: score of one more term of the
-    denominator that has no value."""
+def windowed_softmax(scores, i, window, sink=None, keep=0):
+    """scores over keys 0 .. i -> weights; keys with i - j >= window are not seen, except the first `keep` of the
+    sequence.  sink: score of one more term of the denominator that has no value."""
     n = scores.shape[-1]
-    seen = (i - np.arange(n)) < window if window else np.ones(n, bool)
+    seen = ((i - np.arange(n)) < window) | (np.arange(n) < keep) if window else np.ones(n, bool)
     s = np.where(seen, scores, -np.inf)
     top = s.max(axis=-1, keepdims=True)
     if sink is not None:
@@ -133,6 +133,42 @@ def rotate_pairs(x, pos, freq, mul):
         out[:, :, 2 * i] = u * c - v * s
         out[:, :, 2 * i + 1] = v * c + u * s
     return out
+
+
+def rotate_halves(x, pos, freq, mul):
+    """x [T, H, D]: pairs (i, i + n) of the first 2 n dimensions (n frequencies) turned by pos * freq[i] and scaled."""
+    out, n = x.copy(), len(freq)
+    for i, f in enumerate(freq):
+        c, s = mul * np.cos(pos * f)[:, None], mul * np.sin(pos * f)[:, None]
+        u, v = x[:, :, i], x[:, :, i + n]
+        out[:, :, i] = u * c - v * s
+        out[:, :, i + n] = v * c + u * s
+    return out
+
+
+def soft_cap(scores, cap):
+    return cap * np.tanh(scores / cap)
+
+
+def paged_attention(q, k, v, pos, scale, cap=None, window=None, keep=0):
+    """q [T, H, d] over every earlier key k [n, G, d] and value v [n, G, e]; query head h reads key head h // (H / G)."""
+    T, H, _ = q.shape
+    of = np.arange(H) // (H // k.shape[1])
+    out = np.zeros((T, H, v.shape[2]), F)
+    for t in range(T):
+        n = int(pos[t]) + 1
+        s = np.einsum("hd,nhd->hn", q[t], k[:n, of]) * scale
+        if cap:
+            s = soft_cap(s, cap)
+        out[t] = np.einsum("hn,nhe->he", windowed_softmax(s, n - 1, window, keep=keep), v[:n, of])
+    return out
+
+
+def grow(st, **new):
+    """Appends rows to the cached arrays and returns them whole."""
+    for n, a in new.items():
+        st[n] = np.concatenate([st[n], a]) if n in st else a
+    return [st[n] for n in new]
 
 
 def decayed_linear_attention(q, k, v, decay, S):
@@ -198,6 +234,8 @@ def mix_latent_attention(h, P, m, eps, pos, cache):
         n = int(pos[t]) + 1
         s = (np.einsum("hd,nhd->hn", qu[t], ku[:n]) + np.einsum("hr,nr->hn", qr[t], kr[:n])) * m["scale"]
         out[t] = np.einsum("hn,nhe->he", windowed_softmax(s, n - 1, window), v[:n])
+    if "g" in P:                # one gate per head
+        out = out * sigmoid(linear(h, P["g"]))[:, :, None]
     return linear(out.reshape(T, H * e), P["o"])
 
 
@@ -251,13 +289,72 @@ def clamped_mlp(h, P, limit):
     return linear(g * sigmoid(1.702 * g) * (u + 1), P["down"])
 
 
+def mix_differential(h, P, m, eps, pos, st):
+    """Two attention maps per head over the same values; the second is taken off, weighted by one learned number."""
+    T, H, G, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    freq, mul = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+    q = rotate_halves(rms_norm(linear(h, P["q"]).reshape(T, H * 2, d), P["q.norm"], eps), pos, freq, mul).reshape(T, H, 2, d)
+    k = rotate_halves(rms_norm(linear(h, P["k"]).reshape(T, G * 2, d), P["k.norm"], eps), pos, freq, mul).reshape(T, G, 2, d)
+    k, v = grow(st, k=k, v=linear(h, P["v"]).reshape(T, G, e))
+    a1, a2 = (paged_attention(q[:, :, i], k[:, :, i], v, pos, m["scale"], m.get("softcap")) for i in range(2))
+    lam = np.exp(np.sum(P["lq1"] * P["lk1"])) - np.exp(np.sum(P["lq2"] * P["lk2"])) + m["diff"]
+    o = rms_norm(a1 - lam * a2, 1.0, eps) * (1.0 - m["diff"])
+    return linear(o.reshape(T, H * e), P["o"])
+
+
+def mix_kept_window(h, P, m, eps, pos, st):
+    """Grouped-query attention with biased projections over a sliding window and the first tokens of the sequence."""
+    T, H, G, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q, k, v = (linear(h, P[n]) + P[n + ".b"] for n in "qkv")
+    freq, mul = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+    q = rotate_halves(q.reshape(T, H, d), pos, freq, mul)
+    k, v = grow(st, k=rotate_halves(k.reshape(T, G, d), pos, freq, mul), v=v.reshape(T, G, e))
+    mask = m.get("mask") or {}
+    o = paged_attention(q, k, v, pos, m["scale"], m.get("softcap"), mask.get("size"), mask.get("keep_first", 0))
+    return linear(o.reshape(T, H * e), P["o"])
+
+
+def route(z, correction, groups, keep, top, scale):
+    """Router logits of one token -> (chosen experts, their weights).  Choices are made on sigmoid + correction, among the
+    experts of the groups whose two best choice scores sum up highest; weights are the plain sigmoids times scale."""
+    s = sigmoid(z)
+    choice = s + correction
+    per = len(z) // groups
+    score = [np.sort(choice[g * per:(g + 1) * per])[-2:].sum() for g in range(groups)]
+    allowed = np.repeat(np.isin(np.arange(groups), np.argsort(-np.array(score), kind="stable")[:keep]), per)
+    ids = np.argsort(-np.where(allowed, choice, -np.inf), kind="stable")[:top]
+    return ids, s[ids] * scale
+
+
+def moe_mlp(h, P, mlp):
+    r, e, out = mlp["router"], mlp["expert"], np.zeros_like(h)
+    groups = r.get("groups") or {"count": 1, "keep": 1}
+    z = linear(h, P["router"])
+    for t in range(h.shape[0]):
+        ids, w = route(z[t], P["correction"].reshape(-1), groups["count"], groups["keep"], r["top"], r["scale"])
+        for i, wi in zip(ids, w):
+            out[t] += wi * clamped_mlp(h[t:t + 1], {n: P[f"e{i}.{n}"] for n in ("gate", "up", "down")}, e["limit"])[0]
+    return out
+
+
 # ---------------------------------------------------------------- the decoder
+def layer_runs(config):
+    """(layer, pass that starts here or None) in the order in which layers run."""
+    n, loop = len(config["layers"]), config.get("loop")
+    if not loop:
+        return [(i, None) for i in range(n)]
+    a, b = loop["start"], loop["stop"]
+    again = [(i, t if i == a else None) for t in range(loop["times"]) for i in range(a, b)]
+    return [(i, None) for i in range(a)] + again + [(i, None) for i in range(b, n)]
+
+
 class Stepper:
     def __init__(self, config: dict, tensors: dict):
         self.c = config
         self.w = {k: np.asarray(v, F) for k, v in tensors.items()}
         self.pos = 0
-        self.state = [dict() for _ in config["layers"]]
+        self.runs = layer_runs(config)
+        self.state = [dict() for _ in self.runs]
 
     def part(self, prefix):
         return {k[len(prefix):]: v for k, v in self.w.items() if k.startswith(prefix)}
@@ -267,17 +364,19 @@ class Stepper:
         residual after every layer."""
         tokens = np.asarray(tokens)
         pos = self.pos + np.arange(tokens.size)
-        run = {"Garilix": self.garilix_layer, "Datasun": self.datasun_layer}[self.c["architecture"]]
+        layer = {"Garilix": self.garilix_layer, "Datasun": self.datasun_layer, "Gomuzen": self.gomuzen_layer}[self.c["architecture"]]
         x = self.w["embed"][tokens] * self.c.get("embedding", {}).get("scale", 1.0)
-        for i in range(len(self.c["layers"])):
-            x = run(i, x, pos)
+        for st, (i, t) in zip(self.state, self.runs):
+            if t is not None:
+                x = x + self.w["loop.step"][t]
+            x = layer(i, x, pos, st)
             if trace is not None:
                 trace.append(x.copy())
         self.pos += tokens.size
         return linear(rms_norm(x, self.w["final.norm"], self.c["norm"]["eps"]), self.w["head" if "head" in self.w else "embed"])
 
-    def garilix_layer(self, i, x, pos):
-        L, P, st, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.state[i], self.c["norm"]["eps"]
+    def garilix_layer(self, i, x, pos, st):
+        L, P, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.c["norm"]["eps"]
         m = L["mixer"]
         if L["type"] == "channel_delta":
             y = mix_channel_delta(x, P, m, eps, st)
@@ -295,8 +394,8 @@ class Stepper:
             x = x + rms_norm(dense_mlp(x, self.part(f"l{i}.mlp.")), self.w[f"l{i}.norm2"], eps)
         return x
 
-    def datasun_layer(self, i, x, pos):
-        L, P, st, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.state[i], self.c["norm"]["eps"]
+    def datasun_layer(self, i, x, pos, st):
+        L, P, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.c["norm"]["eps"]
         h = rms_norm(x, self.w[f"l{i}.norm1"], eps)
         if L["type"] == "attention":
             y = mix_attention(h, P, L["mixer"], eps, pos, st)
@@ -308,9 +407,25 @@ class Stepper:
             y = y + clamped_mlp(h, self.part(f"l{i}.mlp."), L["mlp"]["limit"])
         return x + y
 
+    def gomuzen_layer(self, i, x, pos, st):
+        L, P, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.c["norm"]["eps"]
+        h = rms_norm(x, self.w[f"l{i}.norm1"], eps)
+        if L["type"] == "latent_attention":
+            latent_append(h, P, L["mixer"], eps, pos, st)
+            x = x + mix_latent_attention(h, P, L["mixer"], eps, pos, st)
+        elif L["type"] == "attention":
+            x = x + mix_differential(h, P, L["mixer"], eps, pos, st)
+        elif L["type"] == "attention_2":
+            x = x + mix_kept_window(h, P, L["mixer"], eps, pos, st)
+        else:
+            raise ValueError(L["type"])
+        if L.get("mlp"):
+            x = x + moe_mlp(rms_norm(x, self.w[f"l{i}.norm2"], eps), self.part(f"l{i}.mlp."), L["mlp"])
+        return x
+
 
 def forward(config, tensors, tokens):
-    """(logits [T, vocab], residual after every layer [layers, T, width]) of one whole sequence."""
+    """(logits [T, vocab], residual after every layer run [runs, T, width]) of one whole sequence."""
     tr = []
     lg = Stepper(config, tensors).step(tokens, tr)
     return lg, np.stack(tr)

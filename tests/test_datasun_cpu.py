@@ -161,8 +161,8 @@ def test_the_test_weights_show_each_mechanism(spoil, monkeypatch):
     assert rel(R.forward(bad, u, tokens)[0], want).max() > 0.05
 
 
-def _one_after_the_other(self, i, x, pos):
-    L, P, st, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.state[i], self.c["norm"]["eps"]
+def _one_after_the_other(self, i, x, pos, st):
+    L, P, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.c["norm"]["eps"]
     w = self.w[f"l{i}.norm1"]
     h = R.rms_norm(x, w, eps)
     x = x + (R.mix_attention(h, P, L["mixer"], eps, pos, st) if L["type"] == "attention" else R.mix_lightning(h, P, L["mixer"], eps, st))
