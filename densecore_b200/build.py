@@ -26,7 +26,7 @@ NVCC_FLAGS = [
 
 
 # Sources of the layer-list decoders alone (no K-quant kernels): what a process that serves only such a model compiles.
-PARTS = {"layers": ["api", "kv", "linear", "linear_tc", "misc", "mix_gqa", "mix_latent", "mix_lightning", "mix_recur", "model", "norm_act", "stack", "stack_config",
+PARTS = {"layers": ["api", "ffn_moe", "kv", "linear", "linear_tc", "misc", "mix_gqa", "mix_latent", "mix_lightning", "mix_recur", "model", "norm_act", "stack", "stack_config",
                     "stack_load"]}
 
 

@@ -24,7 +24,8 @@ enum { DC_MIX_DELTA = 0, DC_MIX_LATENT = 1, DC_MIX_SSD = 2, DC_MIX_GQA = 3, DC_M
 enum { DC_DTYPE_BF16 = 0, DC_DTYPE_F32 = 1 };
 // How a layer's sublayers meet the residual.  POST_NORM: x += norm1(mixer(x)), then x += norm2(ff(x)).  PARALLEL: with
 // h = norm1(x), x += mixer(h) + ff(h); the input matrices of both are one product, and so are the output matrices.
-enum { DC_BLOCK_POST_NORM = 0, DC_BLOCK_PARALLEL = 1 };
+// PRE_NORM: x += mixer(norm1(x)), then x += ff(norm2(x)).
+enum { DC_BLOCK_POST_NORM = 0, DC_BLOCK_PARALLEL = 1, DC_BLOCK_PRE_NORM = 2 };
 enum { DC_PAIR_GELU = 0, DC_PAIR_CLAMPED = 1 };
 
 static inline int dc_pad8(int n) { return (n + 7) & ~7; }
@@ -54,6 +55,7 @@ struct dc_lin_epi {
     float* pout = nullptr;
     __nv_bfloat16* poutb = nullptr;
     int ldp = 0, n_pairs = 0;
+    const float* tok_scale = nullptr;        // factor of every pair value of a token (grouped products)
     unsigned long long* keys = nullptr;      // packed greedy picks per token (products of up to DC_MAX_T tokens)
 
     static dc_lin_epi store(float* out, __nv_bfloat16* outb, int ldo, unsigned long long* keys = nullptr) {
@@ -100,9 +102,9 @@ struct dc_latent_mixer {        // attention over a compressed key/value latent 
     double rot_base = 10000.0;
     dc_lin in, ukv, o;          // in: q | c and rotated key part;  ukv: per head uk, then per head uv (rows padded to 8)
     int off_q = 0, off_kv = 0, dim_p = 0, vdim_p = 0, uv_row = 0;
+    int off_g = -1;             // one gate per head: the head's output is multiplied by sigmoid of this row (-1: none)
     float* kv_norm = nullptr;   // [kv_rank]
     const float* cos_sin = nullptr;   // [max_ctx][rot_dim / 2][2]
-    int plane = -1;             // cache plane read (and, without kv_from, written)
     int row = 0;                // elements per cached token
     int range = 0;              // which of the step's key ranges (distinct windows)
 };
@@ -118,17 +120,27 @@ struct dc_rotation {
     }
 };
 
-struct dc_gqa_mixer {           // grouped-query attention; the values are the key projection before norm and rotation
-    int heads = 0, kv_heads = 0, dim = 0, window = 0;      // window 0: every earlier token
-    float scale = 1.0f;
+enum { DC_QK_PLAIN = 0, DC_QK_NORM_ALL = 1, DC_QK_NORM_HEAD = 2 };
+
+// Grouped-query attention.  maps 2: every head has two queries and keys over the same values; the second map's output is
+// taken off the first's, weighted by lambda, and the difference is normed per head and multiplied by 1 - diff.
+struct dc_gqa_mixer {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0, maps = 1;
+    int window = 0, keep = 0;   // window 0: every earlier token; else the last `window` and the sequence's first `keep`
+    float scale = 1.0f, softcap = 0.0f;     // softcap c > 0: scores become c tanh(score / c)
     bool sink = false;          // a term of the softmax' denominator with score sink_score and no value
     float sink_score = 0.0f;
     dc_rotation rot;
-    int off_q = 0, off_k = 0, dim_p = 0;    // projection rows; dim_p: padded head size of the cached rows
+    bool halves = false;        // pairs (i, i + dims / 2) instead of (2i, 2i + 1)
+    int qk_norm = DC_QK_PLAIN;  // RMS norm of queries and keys ahead of the rotation: none, over all heads, per head and map
+    int off_q = 0, off_k = 0, off_v = 0;    // projection rows; off_v = off_k: the values are the keys before norm and rotation
+    int dim_p = 0, vdim_p = 0;  // padded sizes in the cached rows
     float *bias = nullptr;      // of the projection rows
-    float *q_norm = nullptr, *k_norm = nullptr;             // over all heads at once
+    float *q_norm = nullptr, *k_norm = nullptr;             // [heads * dim] and [kv_heads * dim], or [dim]
+    float diff = 0.0f, lambda = 0.0f;       // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
+    float* lam[4] = {};         // lq1, lk1, lq2, lk2 [dim]
     const float* cos_sin = nullptr;
-    int plane = -1, row = 0;    // row: k heads, then v heads, dim_p each
+    int row = 0, v_at = 0;      // row: kv_heads * maps keys of dim_p, from v_at kv_heads values of vdim_p
     int range = 0;
 };
 
@@ -138,6 +150,19 @@ struct dc_lightning_mixer {     // linear attention with one constant decay per 
     std::vector<float> decays;  // one per head, from the configuration
     float *decay = nullptr;     // their device copy
     float *norm = nullptr;      // [heads * vdim]: all heads are normed together, then gated by sigmoid(g)
+};
+
+// Mixture of clamped gated experts.  Scores are sigmoid(router); choices are made on score + correction, among the
+// experts of the `keep` groups whose two best choice scores sum up highest; an expert's weight is its score times scale.
+#define DC_MOE_MAX_EXPERTS 512
+#define DC_MOE_MAX_TOP 32
+#define DC_MOE_MAX_GROUPS 32
+struct dc_moe_ffn {
+    int experts = 0, top = 0, groups = 1, keep = 1, ff = 0;
+    float scale = 1.0f, limit = 0.0f;
+    dc_lin router, up, down;    // up: per expert up_rows rows (gate and up in turn), down: per expert down_rows
+    int up_rows = 0, down_rows = 0;
+    float* correction = nullptr;
 };
 
 struct dc_stack_layer {
@@ -153,10 +178,18 @@ struct dc_stack_layer {
     int pair0 = 0, out_ff = 0;
     float* out_bias = nullptr;
     float limit = 0.0f;         // of the clamped pairs
-    size_t state_off = 0, ring_off = 0;   // byte offsets in a sequence's state slot
-    int ff = 0;                 // 0: no feed-forward
+    int ff = 0;                 // 0: no dense feed-forward
+    dc_moe_ffn moe;             // experts 0: none
     dc_lin gate_up, down;       // gate_up: rows 2i = gate row i, 2i + 1 = up row i
     float *norm1 = nullptr, *norm2 = nullptr;
+};
+
+// One run of a layer: a looped layer has several, each with a cache or state of its own.
+struct dc_stack_run {
+    int layer = 0;
+    int step = -1;              // row of the loop's vectors that is added to the residual ahead of this run
+    int plane = -1;             // cache plane of an attention layer
+    size_t state_off = 0, ring_off = 0;     // byte offsets in a sequence's state slot
 };
 
 // Where a named tensor goes: rows of a dc_lin, or a vector of floats.
@@ -170,6 +203,7 @@ struct dc_stack_tensor {
     float** vec = nullptr;
     int64_t vec_off = 0, vec_len = 0;     // destination range and the vector's whole length
     bool neg_exp = false;       // stored as -exp(value)
+    int64_t pitch = 0;          // a vector of shape [n, k] stored with rows of this many floats
     int64_t cols = 0;           // a vector of shape [n, taps] stored transposed: element (c, j) at j * cols + vec_off + c
     bool loaded = false;
     int synth = 0;              // random-weight kind: 0 matrix, 1 norm weight, 2 decay exponent, 3 step bias, 4 small vector
@@ -178,6 +212,7 @@ struct dc_stack_tensor {
 struct dc_stack_config {
     std::string arch;
     int vocab = 0, width = 0, block = DC_BLOCK_POST_NORM;
+    int loop_start = 0, loop_stop = 0, loop_times = 0;      // layers start .. stop - 1 run `times` times in a row (0: no loop)
     float eps = 1e-5f, embed_scale = 1.0f;
     bool tied = false;          // the output matrix is the embedding table
 };
@@ -207,6 +242,11 @@ struct dc_stack_buffers {
     float* q = nullptr;         // grouped-query attention: turned queries (qb: bf16, prompts)
     __nv_bfloat16 *qb = nullptr, *actb = nullptr;
     float* chunk_state = nullptr;        // linear attention: the state ahead of every chunk
+    // mixture of experts: an assignment is a (token, choice); rows are assignments sorted by expert
+    int32_t *moe_ids = nullptr, *moe_row = nullptr, *moe_src = nullptr, *moe_off = nullptr;
+    float *moe_w = nullptr, *moe_row_w = nullptr, *moe_logits = nullptr, *moe_hid = nullptr, *moe_y = nullptr;
+    __nv_bfloat16 *moe_x = nullptr, *moe_hidb = nullptr, *moe_yb = nullptr;
+    int moe_rows = 0;
     std::vector<void*> owned;
 };
 #define DC_STACK_META_SLOTS 4
@@ -215,6 +255,8 @@ struct dc_stack {
     dc_stack_config cfg;
     int dtype = DC_DTYPE_BF16;
     std::vector<dc_stack_layer> layers;
+    std::vector<dc_stack_run> runs;
+    float* loop_step = nullptr; // [loop_times][width padded to 8]
     dc_weight* embed = nullptr;
     dc_lin head;
     float* final_norm = nullptr;
@@ -254,6 +296,9 @@ int dc_launch_linear_rows(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx,
 int dc_launch_linear_f32(dc_ctx* ctx, const dc_lin& w, const float* x, int ldx, int T, const dc_lin_epi& epi);
 // any T, bf16 inputs on the tensor cores
 int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, const dc_lin_epi& epi);
+// the same per expert: rows group_off[e] .. group_off[e + 1] - 1 of x (of max_rows) with rows e * group_rows .. of w
+int dc_launch_linear_grouped_tc(dc_ctx* ctx, const dc_lin& w, int groups, int group_rows, const int32_t* group_off, const dc_tc_in& x, int max_rows,
+                                const dc_lin_epi& epi);
 int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int rows, int K, int ld);
 
 // ---- norm_act.cu
@@ -262,6 +307,35 @@ int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, i
 // out[r] = rms(x[rows ? rows[r] : first + r]) * w
 int dc_launch_norm_rows(dc_ctx* ctx, const float* x, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps,
                         float* out, __nv_bfloat16* outb, int ldo);
+
+// x += step (one row, optional) + for every token the sum of its k rows y[rows[t * k + i]] (optional, yb: bf16); then, with
+// w, out = rms(x) * w as above.  x is rewritten where something was added.
+struct dc_row_sum {
+    const float* y = nullptr;
+    const __nv_bfloat16* yb = nullptr;
+    const int32_t* rows = nullptr;
+    int k = 0, ld = 0;
+};
+int dc_launch_pre_norm(dc_ctx* ctx, float* x, const float* step, const dc_row_sum& sum, const float* w, int T, int H, int ld, float eps, float* out,
+                       __nv_bfloat16* outb);
+
+// ---- ffn_moe.cu
+// up to DC_MAX_T tokens: norm of the residual (out / outb), router logits, choices (ids and weights [T][top])
+int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const float* w, int T, int H, int ld, float eps, float* out,
+                             __nv_bfloat16* outb, int32_t* ids, float* weights);
+// choices from logits [T][ldl]
+int dc_launch_moe_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* logits, int ldl, int T, int32_t* ids, float* weights);
+// assignments sorted by expert: off [experts + 1]; src, row_w [rows]: token and weight of a row; row [T][top]: an assignment's row
+int dc_launch_moe_order(dc_ctx* ctx, const dc_moe_ffn& f, const int32_t* ids, const float* weights, int T, int32_t* off, int32_t* src, float* row_w,
+                        int32_t* row);
+int dc_launch_moe_gather(dc_ctx* ctx, const __nv_bfloat16* x, int ldx, const int32_t* src, int rows, __nv_bfloat16* out);
+// up to DC_MAX_T tokens of bf16 models: hidden values of every assignment times its weight, then x += their products
+int dc_launch_moe_up_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* xb, int ldx, int T, const int32_t* ids, const float* weights,
+                         __nv_bfloat16* hid, int ldh);
+int dc_launch_moe_down_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* hid, int ldh, int T, const int32_t* ids, int H, float* x, int ldx);
+// f32 models: sorted rows; src: input row of a row (null: itself)
+int dc_launch_moe_f32(dc_ctx* ctx, const dc_lin& w, int experts, int group_rows, const int32_t* off, int rows, const float* x, int ldx,
+                      const int32_t* src, const dc_lin_epi& epi);
 
 // ---- mix_recur.cu
 struct dc_state_ref {           // per-sequence state in the cache manager's slots
@@ -308,15 +382,15 @@ struct dc_gqa_cache {
     int max_blocks = 0;
 };
 static inline int dc_gqa_ldq(const dc_gqa_mixer& m) { return (m.dim + 15) & ~15; }      // pitch of a turned query
-// norms, rotation, cache rows of the step's tokens; queries to q or qb [T][heads][dc_gqa_ldq]
+// norms, rotation, cache rows of the step's tokens; queries to q or qb [T][heads * maps][dc_gqa_ldq]
 int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
                        int max_pos, float* q, __nv_bfloat16* qb);
 // every token alone: keys split over CTAs, then joined
 int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
-                         float* part_ml, float* mix, __nv_bfloat16* mixb, int ldm);
+                         float* part_ml, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 // prompts of bf16 models: tiles of queries over the cached rows
 int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const int32_t* tiles, int n_tiles,
-                         const __nv_bfloat16* qb, __nv_bfloat16* mixb, int ldm);
+                         const __nv_bfloat16* qb, float eps, __nv_bfloat16* mixb, int ldm);
 
 // ---- mix_latent.cu
 struct dc_latent_cache {

@@ -1,0 +1,588 @@
+// Mixture of clamped gated experts with a sigmoid router whose choices are limited to groups of experts (dc_moe_ffn).
+//
+// Steps of up to DC_MAX_T tokens: k_moe_norm_route norms the residual and routes it (one cluster per token), k_moe_up_mma
+// streams the gate and up rows of the chosen experts, k_moe_down_mma streams their down rows, every distinct expert once,
+// and adds the sum over experts to the residual.  Hidden values carry the routing weight already, so the down products
+// of a token are one long sum.  Larger steps sort the assignments by expert (k_moe_order), gather the input rows and run
+// grouped tensor-core products (linear_tc.cu); f32 models use k_moe_f32 instead.  The rows of a token are then added up
+// by the norm that follows (norm_act.cu).
+#include <algorithm>
+
+#include "dc_common.cuh"
+#include "dc_launch.cuh"
+#include "dc_stack.h"
+#include "dc_stack.cuh"
+
+using namespace dc;
+
+namespace {
+
+// ---------------------------------------------------------------- choices
+struct RouteParams {
+    int experts, top, groups, keep;
+    float scale;
+    const float* correction;
+    int32_t* ids;
+    float* weights;
+};
+
+__device__ __forceinline__ uint32_t ordered(float f) {      // order-preserving, never 0 for a number
+    const uint32_t u = __float_as_uint(f);
+    return f != f ? 1u : (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+}
+
+// One warp: the choices of a token whose scores are in shared memory.  Equal scores: the lower index first.
+__device__ __forceinline__ void choose(const RouteParams& p, const float* score, int t, int lane) {
+    constexpr int PER = DC_MOE_MAX_EXPERTS / 32;
+    uint32_t c[PER];             // choice of expert lane + 32 j; 0: not available
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int e = lane + 32 * j;
+        c[j] = e < p.experts ? ordered(score[e] + p.correction[e]) : 0u;
+    }
+    if (p.keep < p.groups) {
+        const int n = p.experts / p.groups;
+        float mine = -INFINITY;  // lane g: score of group g
+        for (int g = 0; g < p.groups; ++g) {
+            float a = -INFINITY, b = -INFINITY;             // the two best
+            for (int i = lane; i < n; i += 32) {
+                const float v = score[g * n + i] + p.correction[g * n + i];
+                b = fmaxf(b, fminf(a, v)), a = fmaxf(a, v);
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+                b = fmaxf(fmaxf(b, ob), fminf(a, oa)), a = fmaxf(a, oa);
+            }
+            if (lane == g) mine = n > 1 ? a + b : a;
+        }
+        uint32_t key = lane < p.groups ? ordered(mine) : 0u, kept = 0u;
+        for (int k = 0; k < p.keep; ++k) {
+            const uint32_t best = __reduce_max_sync(0xffffffffu, key);
+            const int g = __ffs(__ballot_sync(0xffffffffu, key == best)) - 1;
+            kept |= 1u << g;
+            if (lane == g) key = 0u;
+        }
+#pragma unroll
+        for (int j = 0; j < PER; ++j)
+            if (lane + 32 * j < p.experts && !(kept >> ((lane + 32 * j) / n) & 1)) c[j] = 0u;
+    }
+    for (int k = 0; k < p.top; ++k) {
+        uint32_t best = 0u;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) best = max(best, c[j]);
+        best = __reduce_max_sync(0xffffffffu, best);
+        int e = DC_MOE_MAX_EXPERTS;
+#pragma unroll
+        for (int j = PER - 1; j >= 0; --j)
+            if (c[j] == best && lane + 32 * j < p.experts) e = lane + 32 * j;
+        e = __reduce_min_sync(0xffffffffu, e);
+#pragma unroll
+        for (int j = 0; j < PER; ++j)
+            if (lane + 32 * j == e) c[j] = 0u;
+        if (lane == 0) {
+            p.ids[(size_t)t * p.top + k] = e;
+            p.weights[(size_t)t * p.top + k] = score[e] * p.scale;
+        }
+    }
+}
+
+// A warp per token.
+__global__ void __launch_bounds__(128) k_moe_route(const RouteParams p, const float* __restrict__ logits, int ldl, int T) {
+    __shared__ float score[4][DC_MOE_MAX_EXPERTS];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp;
+    if (t >= T) return;
+    for (int e = lane; e < p.experts; e += 32) score[warp][e] = sigmoid(logits[(size_t)t * ldl + e]);
+    __syncwarp();
+    choose(p, score[warp], t, lane);
+}
+
+// ---------------------------------------------------------------- norm and choices of few tokens
+struct NormRouteParams {
+    RouteParams r;
+    const float *x, *w;
+    const __nv_bfloat16* router;
+    int ldw, H, ld;
+    float eps;
+    float* out;
+    __nv_bfloat16* outb;
+};
+
+constexpr int NR_CTAS = 8, NR_WARPS = 8, NR_AHEAD = 4;
+
+// A cluster per token: every CTA norms the row and takes its share of the experts, the first one chooses.
+__global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRouteParams p) {
+    extern __shared__ __align__(16) float h[];              // the normed row, padded with zeros to a multiple of 256
+    __shared__ float red[33], score[DC_MOE_MAX_EXPERTS];
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");       // waited for ahead of the first remote store
+    pdl_launch_dependents();
+    const int rank = blockIdx.x % NR_CTAS, t = blockIdx.x / NR_CTAS, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int per = (p.r.experts + NR_CTAS - 1) / NR_CTAS, e0 = rank * per, e1 = min(p.r.experts, e0 + per);
+    const int K8 = p.ld;         // rows of the matrix are padded with zeros beyond the width
+    auto fetch = [&](int e, int i) {
+        const int k = 8 * lane + 256 * i;
+        return e < e1 && k < K8 ? __ldg(reinterpret_cast<const uint4*>(p.router + (size_t)e * p.ldw + k)) : make_uint4(0, 0, 0, 0);
+    };
+    uint4 ahead[NR_AHEAD];
+#pragma unroll
+    for (int i = 0; i < NR_AHEAD; ++i) ahead[i] = fetch(e0 + warp, i);
+    for (int e = e0 + warp; e < e1; e += NR_WARPS)          // the rest comes from L2
+        for (int k = 64 * lane; k < K8; k += 64 * 32) prefetch_l2(p.router + (size_t)e * p.ldw + k);
+    pdl_wait();
+    const int n4 = p.ld / 4;
+    const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)t * p.ld);
+    float ss = 0.0f;
+    for (int i = tid; i < n4; i += NR_WARPS * 32) {
+        const float4 v = x4[i];
+        reinterpret_cast<float4*>(h)[i] = v;
+        ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)p.H + p.eps);
+    for (int i = tid; i < (p.ld + 255) / 256 * 64; i += NR_WARPS * 32) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n4) {
+            const float4 a = reinterpret_cast<float4*>(h)[i], w = reinterpret_cast<const float4*>(p.w)[i];
+            v = make_float4(a.x * inv * w.x, a.y * inv * w.y, a.z * inv * w.z, a.w * inv * w.w);
+            if (i % NR_CTAS == rank) {
+                const size_t at = (size_t)t * p.ld / 4 + i;
+                if (p.outb) reinterpret_cast<uint2*>(p.outb)[at] = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
+                else reinterpret_cast<float4*>(p.out)[at] = v;
+            }
+        }
+        reinterpret_cast<float4*>(h)[i] = v;
+    }
+    __syncthreads();
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    for (int e = e0 + warp; e < e1; e += NR_WARPS) {
+        float a = 0.0f;
+        for (int i0 = 0; 256 * i0 < K8; i0 += NR_AHEAD) {
+            uint4 c[NR_AHEAD];
+#pragma unroll
+            for (int i = 0; i < NR_AHEAD; ++i) {
+                c[i] = ahead[i];
+                const bool more = 256 * (i0 + NR_AHEAD) < K8;
+                ahead[i] = more ? fetch(e, i0 + NR_AHEAD + i) : fetch(e + NR_WARPS, i);
+            }
+#pragma unroll
+            for (int i = 0; i < NR_AHEAD; ++i) {
+                const int k = 8 * lane + 256 * (i0 + i);
+                if (256 * (i0 + i) >= K8) break;
+                float f[8];
+                unpack16(c[i], f, __nv_bfloat16());
+                const float4 u = *reinterpret_cast<const float4*>(h + k), v = *reinterpret_cast<const float4*>(h + k + 4);
+                a = fmaf(f[0], u.x, fmaf(f[1], u.y, fmaf(f[2], u.z, fmaf(f[3], u.w, a))));
+                a = fmaf(f[4], v.x, fmaf(f[5], v.y, fmaf(f[6], v.z, fmaf(f[7], v.w, a))));
+            }
+        }
+        a = sigmoid(warp_sum(a));
+        if (lane == 0) {
+            uint32_t to;
+            asm("mapa.shared::cluster.u32 %0, %1, 0;" : "=r"(to) : "r"(smem_u32(score + e)));
+            asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(to), "f"(a) : "memory");
+        }
+    }
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    if (rank == 0 && warp == 0) choose(p.r, score, t, lane);
+}
+
+// ---------------------------------------------------------------- few tokens: weights streamed once
+constexpr int ME_WARPS = 16;     // warps of a CTA; a CTA takes sixteen rows at a time
+
+// Gate and up rows of one assignment's expert for all its tokens: hidden value times routing weight.  Grid: row tiles x
+// assignments; only an expert's first assignment works.  Column order within a run of 32 as in linear.cu.
+struct UpParams {
+    const __nv_bfloat16* w;
+    int K, ldw, rows, top, T, ff;
+    float limit;
+    const __nv_bfloat16* x;
+    int ldx;
+    const int32_t* ids;
+    const float* weights;
+    __nv_bfloat16* hid;
+    int ldh;
+};
+
+template <int NT>
+__global__ void __launch_bounds__(ME_WARPS * 32) k_moe_up_mma(const UpParams p) {
+    constexpr int AHEAD = 4;
+    __shared__ float red[ME_WARPS][16][8 * NT + 1];
+    __shared__ int s_asg[8 * NT], s_n;
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, first = blockIdx.y, A = p.T * p.top;
+    const int K8 = (p.K + 7) & ~7, runs = (p.K + 31) / 32;
+    pdl_wait();
+    const int e = p.ids[first];
+    const __nv_bfloat16* w0 = p.w + ((size_t)e * p.rows + 16 * blockIdx.x + g) * p.ldw + 8 * q;
+    uint4 a[AHEAD][2];
+    auto fetch = [&](int j, int run) {
+        const bool ok = run < runs && 32 * run + 8 * q < K8;
+        a[j][0] = ok ? __ldg(reinterpret_cast<const uint4*>(w0 + 32 * run)) : make_uint4(0, 0, 0, 0);
+        a[j][1] = ok ? __ldg(reinterpret_cast<const uint4*>(w0 + (size_t)8 * p.ldw + 32 * run)) : make_uint4(0, 0, 0, 0);
+    };
+    if (p.T > 1) {               // the expert's assignments (at most one a token), or nothing if an earlier one has it
+        if (warp == 0) {
+            int n = 0;
+            bool mine = true;
+            for (int i0 = 0; i0 < A && mine; i0 += 32) {
+                const int i = i0 + lane;
+                const unsigned hit = __ballot_sync(0xffffffffu, i < A && p.ids[min(i, A - 1)] == e);
+                if (hit && n == 0) mine = i0 + __ffs(hit) - 1 == first;
+                if (hit >> lane & 1) s_asg[n + __popc(hit & ((1u << lane) - 1))] = i;
+                n += __popc(hit);
+            }
+            if (lane == 0) s_n = mine ? n : 0;
+        }
+        __syncthreads();
+        if (!s_n) return;
+    } else if (tid == 0) {
+        s_asg[0] = first, s_n = 1;
+    }
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j) fetch(j, warp * AHEAD + j);
+    if (p.T == 1) __syncthreads();
+    const int n = s_n;
+    const __nv_bfloat16* x[NT];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) x[i] = 8 * i + g < n ? p.x + (size_t)(s_asg[8 * i + g] / p.top) * p.ldx : nullptr;
+    float acc[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    for (int rb = warp * AHEAD; rb < runs; rb += ME_WARPS * AHEAD) {
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int run = rb + j, k = 32 * run + 8 * q;
+            const uint4 a0 = a[j][0], a1 = a[j][1];
+            fetch(j, run + ME_WARPS * AHEAD);
+            if (run >= runs) continue;
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                const uint4 b = x[i] && k < K8 ? *reinterpret_cast<const uint4*>(x[i] + k) : make_uint4(0, 0, 0, 0);
+                const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
+                mma_bf16(acc[i], lo, b.x, b.y);
+                mma_bf16(acc[i], hi, b.z, b.w);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) red[warp][g + 8 * (j >> 1)][8 * i + 2 * q + (j & 1)] = acc[i][j];
+    __syncthreads();
+    const int r = tid & 15, t = tid >> 4, o = 8 * blockIdx.x + (r >> 1);
+    if (t >= 8 * NT) return;
+    float v = 0.0f;
+#pragma unroll
+    for (int i = 0; i < ME_WARPS; ++i) v += red[i][r][t];
+    const float up = __shfl_down_sync(0xffffffffu, v, 1);
+    if (!(r & 1) && t < n && o < p.ff) {
+        const int as = s_asg[t];
+        dc_lin_epi epi;
+        epi.pair_kind = DC_PAIR_CLAMPED, epi.limit = p.limit;
+        p.hid[(size_t)as * p.ldh + o] = __float2bfloat16_rn(pair_value(epi, v, up) * p.weights[as]);
+    }
+}
+
+struct DownParams {
+    const __nv_bfloat16* w;
+    int K, ldw, rows, top, T, H, experts;
+    const __nv_bfloat16* hid;
+    int ldh;
+    const int32_t* ids;
+    float* x;
+    int ldx;
+};
+
+// x[t] += sum over the token's assignments of W_down hid.  The distinct experts' columns are one long row: a token has
+// zeros where an expert is not its own.  KS: CTAs of a cluster that share sixteen rows, each with its part of that row.
+template <int NT, int KS>
+__global__ void __launch_bounds__(ME_WARPS * 32) k_moe_down_mma(const DownParams p) {
+    constexpr int AHEAD = 2, CAP = 8 * NT * DC_MOE_MAX_TOP;
+    __shared__ float red[ME_WARPS][16][8 * NT + 1];
+    __shared__ float other[KS > 1 ? KS - 1 : 1][KS > 1 ? 128 * NT : 1];
+    __shared__ int16_t s_expert[CAP], s_asg[CAP][8 * NT];       // distinct experts; their assignment of every token, -1: none
+    __shared__ int s_first[DC_MOE_MAX_EXPERTS], s_n;
+    if (KS > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, part = blockIdx.x % KS, row0 = blockIdx.x / KS * 16;
+    const int A = p.T * p.top, K8 = (p.K + 7) & ~7, per_expert = (p.K + 31) / 32;
+    if (p.T > 1) {
+        for (int i = tid; i < p.experts; i += ME_WARPS * 32) s_first[i] = 1 << 30;
+        for (int i = tid; i < CAP * 8 * NT / 2; i += ME_WARPS * 32) reinterpret_cast<uint32_t*>(&s_asg[0][0])[i] = 0xffffffffu;
+        __syncthreads();
+    }
+    pdl_wait();
+    if (p.T > 1) {
+        for (int i = tid; i < A; i += ME_WARPS * 32) atomicMin(&s_first[p.ids[i]], i);
+        __syncthreads();
+        if (warp == 0) {
+            int n = 0;
+            for (int i0 = 0; i0 < A; i0 += 32) {
+                const int i = i0 + lane, e = i < A ? p.ids[i] : 0;
+                const bool is = i < A && s_first[e] == i;
+                const unsigned hit = __ballot_sync(0xffffffffu, is);
+                const int u = n + __popc(hit & ((1u << lane) - 1));
+                if (is) s_expert[u] = (int16_t)e;
+                __syncwarp();
+                if (is) s_first[e] = -1 - u;
+                __syncwarp();
+                n += __popc(hit);
+            }
+            if (lane == 0) s_n = n;
+        }
+        __syncthreads();
+        for (int i = tid; i < A; i += ME_WARPS * 32) s_asg[-1 - s_first[p.ids[i]]][i / p.top] = (int16_t)i;
+    } else {
+        if (tid < A) s_expert[tid] = (int16_t)p.ids[tid], s_asg[tid][0] = (int16_t)tid;
+        if (tid == 0) s_n = A;
+    }
+    __syncthreads();
+    const int all = s_n * per_expert, share = (all + KS - 1) / KS, begin = part * share, end = min(all, begin + share);
+    uint4 a[AHEAD][2];
+    auto fetch = [&](int j, int run) {
+        const int u = run / per_expert, k = 32 * (run - u * per_expert) + 8 * q;
+        const bool ok = run < end && k < K8;
+        const __nv_bfloat16* w = p.w + ((size_t)s_expert[ok ? u : 0] * p.rows + row0 + g) * p.ldw + (ok ? k : 0);
+        a[j][0] = ok ? __ldg(reinterpret_cast<const uint4*>(w)) : make_uint4(0, 0, 0, 0);
+        a[j][1] = ok ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)8 * p.ldw)) : make_uint4(0, 0, 0, 0);
+    };
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j) fetch(j, begin + warp * AHEAD + j);
+    float acc[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    for (int rb = begin + warp * AHEAD; rb < end; rb += ME_WARPS * AHEAD) {
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int run = rb + j;
+            const uint4 a0 = a[j][0], a1 = a[j][1];
+            fetch(j, run + ME_WARPS * AHEAD);
+            if (run >= end) continue;
+            const int u = run / per_expert, k = 32 * (run - u * per_expert) + 8 * q;
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                const int t = 8 * i + g, as = t < p.T ? s_asg[u][t] : -1;
+                const uint4 b = as >= 0 && k < K8 ? *reinterpret_cast<const uint4*>(p.hid + (size_t)as * p.ldh + k) : make_uint4(0, 0, 0, 0);
+                const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
+                mma_bf16(acc[i], lo, b.x, b.y);
+                mma_bf16(acc[i], hi, b.z, b.w);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) red[warp][g + 8 * (j >> 1)][8 * i + 2 * q + (j & 1)] = acc[i][j];
+    __syncthreads();
+    const int r = tid & 15, t = tid >> 4, row = row0 + r;
+    const bool mine = tid < 128 * NT;
+    float v = 0.0f;
+    if (mine)
+#pragma unroll
+        for (int i = 0; i < ME_WARPS; ++i) v += red[i][r][t];
+    if (KS > 1) {
+        asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+        if (part > 0 && mine) {
+            uint32_t to;
+            asm("mapa.shared::cluster.u32 %0, %1, 0;" : "=r"(to) : "r"(smem_u32(&other[part - 1][tid])));
+            asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(to), "f"(v) : "memory");
+        }
+        asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+        asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        if (part > 0) return;
+        if (mine)
+#pragma unroll
+            for (int k = 0; k < KS - 1; ++k) v += other[k][tid];
+    }
+    if (mine && t < p.T && row < p.H) p.x[(size_t)t * p.ldx + row] += v;
+}
+
+// ---------------------------------------------------------------- many tokens: assignments sorted by expert
+// A CTA per expert: how many assignments go to lower experts, then its own in order.
+__global__ void __launch_bounds__(256) k_moe_order(const int32_t* __restrict__ ids, const float* __restrict__ weights, int A, int top, int experts,
+                                                   int32_t* __restrict__ off, int32_t* __restrict__ src, float* __restrict__ row_w,
+                                                   int32_t* __restrict__ row) {
+    __shared__ int s_mine[8], s_below[8];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int e = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    // a thread's run of assignments
+    const int per = ((A + 255) / 256 + 3) & ~3, i0 = min(A, tid * per), i1 = min(A, i0 + per);
+    int mine = 0, below = 0;
+#pragma unroll 8
+    for (int i = i0; i < i1; ++i) {
+        const int v = ids[i];
+        mine += v == e;
+        below += v < e;
+    }
+    int before = mine;           // inclusive sum over the warp
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, before, o);
+        if (lane >= o) before += v;
+    }
+    below = __reduce_add_sync(0xffffffffu, below);
+    if (lane == 31) s_mine[warp] = before, s_below[warp] = below;
+    __syncthreads();
+    int at = before - mine, total = 0;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+        at += s_below[w] + (w < warp ? s_mine[w] : 0);
+        total += s_below[w];
+    }
+    if (tid == 0) {
+        off[e] = total;
+        if (e == experts - 1) off[experts] = A;
+    }
+    for (int i = i0; i < i1 && mine; ++i)
+        if (ids[i] == e) {
+            src[at] = i / top;
+            row_w[at] = weights[i];
+            row[i] = at;
+            ++at, --mine;
+        }
+}
+
+// out[r] = x[src[r]], rows of ld elements (a multiple of eight); a warp per row
+__global__ void __launch_bounds__(256) k_moe_gather(const __nv_bfloat16* __restrict__ x, int ld, const int32_t* __restrict__ src, int rows,
+                                                    __nv_bfloat16* __restrict__ out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (r >= rows) return;
+    const uint4* from = reinterpret_cast<const uint4*>(x + (size_t)src[r] * ld);
+    uint4* to = reinterpret_cast<uint4*>(out + (size_t)r * ld);
+#pragma unroll 8
+    for (int i = lane; i < ld / 8; i += 32) to[i] = from[i];
+}
+
+// f32 tile product of an expert's rows: 64 weight rows x 64 sorted rows per CTA, 4 x 4 outputs per thread.
+struct F32Params {
+    const __nv_bfloat16* w;
+    int K, ldw, experts, group_rows;
+    const int32_t* off;
+    const float* x;
+    int ldx;
+    const int32_t* src;
+    dc_lin_epi e;
+};
+
+__global__ void __launch_bounds__(256) k_moe_f32(const F32Params p) {
+    __shared__ float sw[16][68], sx[16][68];
+    pdl_launch_dependents();
+    pdl_wait();
+    int tile = blockIdx.y, ex = 0, r0 = 0, r1 = 0;
+    for (; ex < p.experts; ++ex) {
+        r0 = p.off[ex], r1 = p.off[ex + 1];
+        const int tiles = (r1 - r0 + 63) / 64;
+        if (tile < tiles) break;
+        tile -= tiles;
+    }
+    if (ex == p.experts) return;
+    r0 += 64 * tile;
+    const __nv_bfloat16* w = p.w + (size_t)ex * p.group_rows * p.ldw;
+    const int tid = threadIdx.x, n0 = blockIdx.x * 64, tn = (tid & 15) * 4, tt = (tid >> 4) * 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < p.K; k0 += 16) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int at = tid + i * 256, r = at >> 4, k = at & 15;
+            sw[k][r] = n0 + r < p.group_rows && k0 + k < p.K ? __bfloat162float(w[(size_t)(n0 + r) * p.ldw + k0 + k]) : 0.0f;
+            const int in = r0 + r < r1 ? p.src ? p.src[r0 + r] : r0 + r : -1;
+            sx[k][r] = in >= 0 && k0 + k < p.K ? p.x[(size_t)in * p.ldx + k0 + k] : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+            const float4 a = *reinterpret_cast<const float4*>(&sw[k][tn]), b = *reinterpret_cast<const float4*>(&sx[k][tt]);
+            const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(bv[i], av[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = r0 + tt + i;
+        if (t >= r1) continue;
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {
+            const int n = n0 + tn + j;
+            if (n >= p.e.pair0) {
+                const int c = (n - p.e.pair0) >> 1;
+                if (c < p.e.n_pairs) put_pair(p.e, t, c, pair_value(p.e, acc[i][j], acc[i][j + 1]) * (p.e.tok_scale ? p.e.tok_scale[t] : 1.0f));
+            } else {
+                if (n < p.e.n_store) put_row(p.e, t, n, acc[i][j]);
+                if (n + 1 < p.e.n_store) put_row(p.e, t, n + 1, acc[i][j + 1]);
+            }
+        }
+    }
+}
+
+RouteParams route_params(const dc_moe_ffn& f, int32_t* ids, float* weights) {
+    return RouteParams{f.experts, f.top, f.groups, f.keep, f.scale, f.correction, ids, weights};
+}
+
+template <int NT, int KS>
+int launch_down(dc_ctx* ctx, const DownParams& p) {
+    const int tiles = p.rows / 16;
+    const dim3 block(ME_WARPS * 32);
+    if (KS > 1) return dc_launch_cluster(ctx, "k_moe_down_mma", k_moe_down_mma<NT, KS>, dim3(tiles * KS), block, 0, KS, p);
+    return dc_launch(ctx, "k_moe_down_mma", k_moe_down_mma<NT, 1>, dim3(tiles), block, 0, p);
+}
+
+}  // namespace
+
+int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const float* w, int T, int H, int ld, float eps, float* out,
+                             __nv_bfloat16* outb, int32_t* ids, float* weights) {
+    if (f.experts > DC_MOE_MAX_EXPERTS || f.groups > DC_MOE_MAX_GROUPS || ld % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad operand");
+    const NormRouteParams p = {route_params(f, ids, weights), x, w, f.router.w, f.router.ld, H, ld, eps, out, outb};
+    const size_t smem = (size_t)(ld + 255) / 256 * 256 * 4;
+    const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route, (int)smem, "k_moe_norm_route");
+    if (st != DC_B200_OK) return st;
+    return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);
+}
+
+int dc_launch_moe_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* logits, int ldl, int T, int32_t* ids, float* weights) {
+    if (f.experts > DC_MOE_MAX_EXPERTS || f.groups > DC_MOE_MAX_GROUPS) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_route: bad operand");
+    return dc_launch(ctx, "k_moe_route", k_moe_route, dim3((T + 3) / 4), dim3(128), 0, route_params(f, ids, weights), logits, ldl, T);
+}
+
+int dc_launch_moe_order(dc_ctx* ctx, const dc_moe_ffn& f, const int32_t* ids, const float* weights, int T, int32_t* off, int32_t* src, float* row_w,
+                        int32_t* row) {
+    return dc_launch(ctx, "k_moe_order", k_moe_order, dim3(f.experts), dim3(256), 0, ids, weights, T * f.top, f.top, f.experts, off, src, row_w, row);
+}
+
+int dc_launch_moe_gather(dc_ctx* ctx, const __nv_bfloat16* x, int ldx, const int32_t* src, int rows, __nv_bfloat16* out) {
+    return dc_launch(ctx, "k_moe_gather", k_moe_gather, dim3((rows + 7) / 8), dim3(256), 0, x, ldx, src, rows, out);
+}
+
+int dc_launch_moe_up_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* xb, int ldx, int T, const int32_t* ids, const float* weights,
+                         __nv_bfloat16* hid, int ldh) {
+    if (T < 1 || T > DC_MAX_T || ldx % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_up: bad operand");
+    const UpParams p = {f.up.w, f.up.K, f.up.ld, f.up_rows, f.top, T, f.ff, f.limit, xb, ldx, ids, weights, hid, ldh};
+    const dim3 grid(f.up_rows / 16, T * f.top), block(ME_WARPS * 32);
+    if (T <= 8) return dc_launch(ctx, "k_moe_up_mma", k_moe_up_mma<1>, grid, block, 0, p);
+    return dc_launch(ctx, "k_moe_up_mma", k_moe_up_mma<2>, grid, block, 0, p);
+}
+
+int dc_launch_moe_down_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* hid, int ldh, int T, const int32_t* ids, int H, float* x, int ldx) {
+    if (T < 1 || T > DC_MAX_T || ldh % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_down: bad operand");
+    const DownParams p = {f.down.w, f.down.K, f.down.ld, f.down_rows, f.top, T, H, f.experts, hid, ldh, ids, x, ldx};
+    // fewer row tiles than SMs: the long rows are shared by a cluster
+    const int tiles = f.down_rows / 16;
+    if (2 * tiles <= ctx->num_sms) return T <= 8 ? launch_down<1, 4>(ctx, p) : launch_down<2, 4>(ctx, p);
+    if (tiles <= ctx->num_sms) return T <= 8 ? launch_down<1, 2>(ctx, p) : launch_down<2, 2>(ctx, p);
+    return T <= 8 ? launch_down<1, 1>(ctx, p) : launch_down<2, 1>(ctx, p);
+}
+
+int dc_launch_moe_f32(dc_ctx* ctx, const dc_lin& w, int experts, int group_rows, const int32_t* off, int rows, const float* x, int ldx,
+                      const int32_t* src, const dc_lin_epi& epi) {
+    F32Params p = {w.w, w.K, w.ld, experts, group_rows, off, x, ldx, src, epi};
+    p.e.n_store = std::min(epi.n_store, std::min(group_rows, epi.pair0));
+    return dc_launch(ctx, "k_moe_f32", k_moe_f32, dim3((group_rows + 63) / 64, rows / 64 + std::min(experts, rows)), dim3(256), 0, p);
+}

@@ -6,7 +6,9 @@
 // a warp's stores of one token are 32 consecutive outputs.  Two CTAs share an SM: one's read-out overlaps the
 // other's products.  Large products use tiles of 128 x 256 instead (k_linear_tc_wide): one CTA per SM walks its share
 // of them, with two sets of accumulators, so that the loads and products of a tile run while the tile before is read
-// out; the wider tile reads shared memory less often per product.  Both let the next kernel start only after every
+// out; the wider tile reads shared memory less often per product.  Its grouped form multiplies runs of sorted tokens with
+// a matrix of their own each (experts); the runs' ends are device data, so every CTA lists the tiles itself, and a tile
+// of few tokens takes narrower products.  All let the next kernel start only after every
 // CTA has its tensor memory.  Columns beyond K and rows beyond the matrix are the zeros that TMA fills in.  Every wait is
 // bounded; a CTA that gives up drains its copies, frees its tensor memory and leaves.
 #include <algorithm>
@@ -59,8 +61,8 @@ __device__ __forceinline__ void each16(uint32_t tmem, int n, F f) {
 
 // Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.
 template <int COLS>
-__device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int quarter, int lane) {
-    const int row = row0 + 32 * quarter + lane, n = p.T - t0;
+__device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int t1, int quarter, int lane) {
+    const int row = row0 + 32 * quarter + lane, n = t1 - t0;
     const dc_lin_epi& e = p.e;
     tmem += (uint32_t)(32 * quarter) << 16;
     if (row0 + 32 * quarter >= e.pair0) {
@@ -79,6 +81,12 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
                 h[i] = gelu ? gelu_tanh(gate) * val : quick_clamped(e.limit, gate, val);
             }
             const int m = in ? n - c0 - first : 0;
+            if (e.tok_scale) {
+                const float* f = e.tok_scale + t0 + c0 + first;
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                    if (i < m) h[i] *= f[i];
+            }
             if (e.poutb) {
                 __nv_bfloat16* to = e.poutb + at + (size_t)c0 * e.ldp;
 #pragma unroll
@@ -194,7 +202,7 @@ __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_consta
     } else {
         const bool ok = tc_wait_raw(acc, 0, give_up, p.err) && !*give_up;
         tc_fence_after();
-        if (__all_sync(0xffffffffu, ok)) read_out<128>(p, tmem, row0, t0, warp & 3, lane);
+        if (__all_sync(0xffffffffu, ok)) read_out<128>(p, tmem, row0, t0, p.T, warp & 3, lane);
     }
     tc_fence_before();
     __syncthreads();
@@ -206,17 +214,24 @@ __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_consta
 constexpr int LW_STAGES = 4, LW_STAGE = 3 * LT_TILE;       // 128 weight rows and 256 token rows of 64 columns
 constexpr size_t LW_SMEM = (size_t)LW_STAGES * LW_STAGE + 1024;
 
+struct LwTiles {
+    int row_tiles, tok_tiles;        // one matrix
+    int groups, group_rows;          // grouped: matrix g is rows g * group_rows .., its tokens are off[g] .. off[g + 1] - 1
+    const int32_t* off;
+};
+
+template <bool GROUPED>
 __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_constant__ CUtensorMap wmap,
-                                                                  const __grid_constant__ CUtensorMap xmap, const LtParams p, int row_tiles,
-                                                                  int tok_tiles) {
+                                                                  const __grid_constant__ CUtensorMap xmap, const LtParams p, const LwTiles tl) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t s_bar[2 * LW_STAGES + 4];
     __shared__ uint32_t s_tmem;
     __shared__ int s_give_up;
+    __shared__ int s_off[GROUPED ? DC_MOE_MAX_EXPERTS + 1 : 1], s_first[GROUPED ? DC_MOE_MAX_EXPERTS + 1 : 1];
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t full = smem_u32(s_bar), empty = full + 8 * LW_STAGES, acc_full = empty + 8 * LW_STAGES, acc_free = acc_full + 16;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int nk = (p.K + 63) / 64, total = row_tiles * tok_tiles;
+    const int nk = (p.K + 63) / 64;
     volatile int* give_up = &s_give_up;
     if (warp == 1) {
         tmem_alloc(smem_u32(&s_tmem), 512);
@@ -240,13 +255,49 @@ __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_c
     const uint32_t tmem = s_tmem;
     pdl_launch_dependents();
     pdl_wait();
+    if (GROUPED) {               // the tiles of every group
+        if (warp == 2) {
+            int before = 0;
+            for (int g0 = 0; g0 < tl.groups; g0 += 32) {
+                const int g = g0 + lane, a = tl.off[min(g, tl.groups)], b = tl.off[min(g + 1, tl.groups)];
+                int n = (b - a + 255) / 256 * tl.row_tiles;
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    const int v = __shfl_up_sync(0xffffffffu, n, o);
+                    if (lane >= o) n += v;
+                }
+                if (g < tl.groups) s_off[g + 1] = b, s_first[g + 1] = before + n;
+                before += __shfl_sync(0xffffffffu, n, 31);
+            }
+            if (lane == 0) s_off[0] = s_first[0] = 0;
+        }
+        __syncthreads();
+    }
+    const int total = GROUPED ? s_first[tl.groups] : tl.row_tiles * tl.tok_tiles;
+    struct Place {
+        int wrow, row0, t0, t1;      // row of the map, row of the matrix, tokens
+        __device__ int cols() const { return min(256, t1 - t0); }
+    };
+    auto place = [&](int tile, int& group) {
+        Place at;
+        if (GROUPED) {
+            while (tile >= s_first[group + 1]) ++group;
+            const int a = s_off[group], b = s_off[group + 1], tok_tiles = (b - a + 255) / 256, i = tile - s_first[group];
+            at.row0 = i / tok_tiles * 128, at.t0 = a + i % tok_tiles * 256, at.t1 = b;
+            at.wrow = group * tl.group_rows + at.row0;
+        } else {
+            at.row0 = at.wrow = tile / tl.tok_tiles * 128, at.t0 = tile % tl.tok_tiles * 256, at.t1 = p.T;
+        }
+        return at;
+    };
     // Every role walks the same tiles; stages are counted on across tiles.
     if (warp == 0) {
         if (lane == 0) {
-            int issued = 0;
+            int issued = 0, group = 0;
             bool ok = true;
             for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
-                const int row0 = tile / tok_tiles * 128, t0 = tile % tok_tiles * 256;
+                const Place at = place(tile, group);
+                const bool both = !GROUPED || at.cols() > 128;
                 for (int k = 0; k < nk; ++k, ++issued) {
                     const int s = issued % LW_STAGES, use = issued / LW_STAGES;
                     if (use > 0 && !tc_wait_raw(empty + 8 * s, (use - 1) & 1, give_up, p.err)) {
@@ -254,10 +305,10 @@ __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_c
                         break;
                     }
                     const uint32_t to = base + s * LW_STAGE;
-                    mbar_expect_tx(full + 8 * s, LW_STAGE);
-                    tma_load_2d(to, &wmap, k * 64, row0, full + 8 * s);
-                    tma_load_2d(to + LT_TILE, &xmap, k * 64, t0, full + 8 * s);
-                    tma_load_2d(to + 2 * LT_TILE, &xmap, k * 64, t0 + 128, full + 8 * s);
+                    mbar_expect_tx(full + 8 * s, both ? LW_STAGE : 2 * LT_TILE);
+                    tma_load_2d(to, &wmap, k * 64, at.wrow, full + 8 * s);
+                    tma_load_2d(to + LT_TILE, &xmap, k * 64, at.t0, full + 8 * s);
+                    if (both) tma_load_2d(to + 2 * LT_TILE, &xmap, k * 64, at.t0 + 128, full + 8 * s);
                 }
             }
             // no copy may still be in flight when the CTA leaves (at once unless someone gave up)
@@ -269,11 +320,11 @@ __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_c
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            const uint32_t idesc = umma_idesc_bf16(128, 256);
-            int it = 0, j = 0;
+            int it = 0, j = 0, group = 0;
             bool ok = true;
             for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x, ++j) {
                 const int set = j & 1;
+                const uint32_t idesc = umma_idesc_bf16(128, GROUPED ? (place(tile, group).cols() + 15) & ~15 : 256);
                 if (j >= 2 && !tc_wait_raw(acc_free + 8 * set, ((j >> 1) - 1) & 1, give_up, p.err)) break;
                 tc_fence_after();
                 for (int k = 0; k < nk; ++k, ++it) {
@@ -293,13 +344,14 @@ __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_c
             }
         }
     } else {
-        int j = 0;
+        int j = 0, group = 0;
         for (int tile = blockIdx.x; tile < total; tile += gridDim.x, ++j) {
             const int set = j & 1;
             const bool ok = tc_wait_raw(acc_full + 8 * set, (j >> 1) & 1, give_up, p.err) && !*give_up;
             tc_fence_after();
             if (!__all_sync(0xffffffffu, ok)) break;
-            read_out<256>(p, tmem + 256 * set, tile / tok_tiles * 128, tile % tok_tiles * 256, warp & 3, lane);
+            const Place at = place(tile, group);
+            read_out<256>(p, tmem + 256 * set, at.row0, at.t0, at.t1, warp & 3, lane);
             tc_fence_before();
             mbar_arrive(acc_free + 8 * set);
         }
@@ -344,12 +396,29 @@ int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, 
     p.e.n_pairs = std::max(0, std::min(epi.n_pairs, (w.N - epi.pair0) / 2));
     const int row_tiles = (w.N + 127) / 128, tok_tiles = (T + 255) / 256, tiles = row_tiles * tok_tiles;
     if (T > 128 && tiles >= ctx->num_sms / 2) {
-        int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide, (int)LW_SMEM, "k_linear_tc_wide");
+        int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide<false>, (int)LW_SMEM, "k_linear_tc_wide");
         if (st != DC_B200_OK) return st;
-        return dc_launch(ctx, "k_linear_tc_wide", k_linear_tc_wide, dim3(tiles < ctx->num_sms ? tiles : ctx->num_sms), dim3(LT_THREADS), LW_SMEM, w.map,
-                         x.map, p, row_tiles, tok_tiles);
+        const LwTiles tl = {row_tiles, tok_tiles, 0, 0, nullptr};
+        return dc_launch(ctx, "k_linear_tc_wide", k_linear_tc_wide<false>, dim3(tiles < ctx->num_sms ? tiles : ctx->num_sms), dim3(LT_THREADS), LW_SMEM,
+                         w.map, x.map, p, tl);
     }
     int st = dc_kernel_setup(ctx, (const void*)k_linear_tc, (int)LT_SMEM, "k_linear_tc");
     if (st != DC_B200_OK) return st;
     return dc_launch(ctx, "k_linear_tc", k_linear_tc, dim3((w.N + 127) / 128, (T + 127) / 128), dim3(LT_THREADS), LT_SMEM, w.map, x.map, p);
+}
+
+int dc_launch_linear_grouped_tc(dc_ctx* ctx, const dc_lin& w, int groups, int group_rows, const int32_t* group_off, const dc_tc_in& x, int max_rows,
+                                const dc_lin_epi& epi) {
+    if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: inner sizes %d and %d differ", w.K, x.K);
+    if (groups < 1 || groups > DC_MOE_MAX_EXPERTS || groups * group_rows != w.N || max_rows < 1) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: bad groups");
+    if (epi.keys || epi.add || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: epilogue not available");
+    LtParams p = {w.K, max_rows, epi, ctx->d_err};
+    p.e.n_store = std::min(epi.n_store, std::min(group_rows, epi.pair0));
+    p.e.n_pairs = std::max(0, std::min(epi.n_pairs, (group_rows - epi.pair0) / 2));
+    const LwTiles tl = {(group_rows + 127) / 128, 0, groups, group_rows, group_off};
+    const int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide<true>, (int)LW_SMEM, "k_linear_tc_grouped");
+    if (st != DC_B200_OK) return st;
+    const long long most = (long long)tl.row_tiles * (max_rows / 256 + std::min(groups, max_rows));
+    return dc_launch(ctx, "k_linear_tc_grouped", k_linear_tc_wide<true>, dim3((int)std::min<long long>(most, ctx->num_sms)), dim3(LT_THREADS), LW_SMEM, w.map, x.map,
+                     p, tl);
 }

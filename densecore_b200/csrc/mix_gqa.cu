@@ -1,9 +1,12 @@
-// Grouped-query attention with a sliding window, norms over the whole query and key projections, partial rotation, an
-// optional sink in the softmax' denominator, and values that are the key projection as it is (before norm and rotation).
+// Grouped-query attention with its variants: a sliding window with or without the sequence's first tokens kept in sight, a
+// soft cap on the scores, a sink in the softmax' denominator, norms of queries and keys over the whole projection or per
+// head, rotation of neighbouring or of half-distant pairs, values of their own or the key projection before norm and
+// rotation, and two maps per head whose outputs are subtracted.
 //
-// A cached token is one row: the turned keys of all key heads, then their values.  Steps of up to DC_MAX_T tokens and f32
-// models take every token alone (k_gqa_tokens: keys split over CTAs, k_gqa_join); prompt-sized steps of bf16 models run
-// tiles of queries over the cached rows with bf16 products (k_gqa_prompt).  Scores, weights and their sums are f32.
+// A cached token is one row: the turned keys of all key heads (and maps), then the values.  Steps of up to DC_MAX_T tokens
+// and f32 models take every token alone (k_gqa_tokens: keys split over CTAs, k_gqa_join); prompt-sized steps of bf16
+// models run tiles of queries over the cached rows with bf16 products (k_gqa_prompt).  Scores, weights and their sums are
+// f32.
 #include <algorithm>
 
 #include "dc_common.cuh"
@@ -109,38 +112,110 @@ __global__ void __launch_bounds__(256) k_gqa_prep(const PrepParams p) {
     }
 }
 
-// ---------------------------------------------------------------- every token alone
-struct TokenParams {
-    const float* q;          // [T][heads][ldq]
-    int ldq, heads, per, groups, dim, dim_p, v_off, window, splits;
-    float scale;
+// The same with a norm per head or none: a warp per head of a token, a lane has the dimensions lane, lane + 32, ...
+struct HeadsParams {
+    const float* proj;
+    int ldp, off_q, off_k, off_v, nq, nk, nv, dim, vdim, dim_p, vdim_p, v_at, ldq, rot, halves, max_pos;
+    const float *q_norm, *k_norm, *cos_sin;
+    float eps;
     const int32_t *seq_ids, *positions;
     CacheRef c;
-    float *part, *part_ml;   // [T][heads][splits][dim], [T][heads][splits][2]
+    float* q;
+    __nv_bfloat16* qb;       // instead of q
+};
+
+template <typename TC, int VP>      // VP: dimensions of a lane
+__global__ void __launch_bounds__(256) k_gqa_prep_heads(const HeadsParams p) {
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5);
+    if (u >= p.nq + p.nk + p.nv) return;
+    const bool query = u < p.nq, value = u >= p.nq + p.nk;
+    const int head = query ? u : value ? u - p.nq - p.nk : u - p.nq, n = value ? p.vdim : p.dim;
+    const float* w = value ? nullptr : query ? p.q_norm : p.k_norm;
+    float nw[VP];
+#pragma unroll
+    for (int j = 0; j < VP; ++j) nw[j] = w && lane + 32 * j < n ? w[lane + 32 * j] : 1.0f;
+    pdl_wait();
+    const int t = blockIdx.x, pos = min(max(p.positions[t], 0), p.max_pos - 1);
+    const float* x = p.proj + (size_t)t * p.ldp + (query ? p.off_q : value ? p.off_v : p.off_k) + head * n;
+    const float* cs = p.cos_sin + (size_t)pos * p.rot;
+    const int half = p.rot / 2;
+    float v[VP], other[VP], ss = 0.0f;
+    float2 turn[VP];
+#pragma unroll
+    for (int j = 0; j < VP; ++j) {
+        const int d = lane + 32 * j;
+        const bool first = p.halves ? d < half : !(d & 1), turned = !value && d < p.rot;
+        const int mate = p.halves ? (first ? d + half : d - half) : d ^ 1;
+        v[j] = d < n ? x[d] : 0.0f;
+        other[j] = 0.0f, turn[j] = make_float2(1.0f, 0.0f);
+        if (turned) {
+            other[j] = x[mate] * (w ? w[mate] : 1.0f);
+            turn[j] = *reinterpret_cast<const float2*>(cs + 2 * (p.halves ? min(d, mate) : d / 2));
+            if (first) turn[j].y = -turn[j].y;
+        }
+        ss = fmaf(v[j], v[j], ss);
+    }
+    const float inv = w ? 1.0f / sqrtf(warp_sum(ss) / (float)n + p.eps) : 1.0f;
+    TC* cache = query ? nullptr : reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos) + (value ? p.v_at + head * p.vdim_p : head * p.dim_p);
+    const int pitch = query ? p.ldq : value ? p.vdim_p : p.dim_p;
+#pragma unroll
+    for (int j = 0; j < VP; ++j) {
+        const int d = lane + 32 * j;
+        if (d >= pitch) break;
+        const float r = (v[j] * nw[j] * turn[j].x + other[j] * turn[j].y) * inv;       // zero in the padding
+        const size_t at = ((size_t)t * p.nq + head) * pitch + d;
+        if (!query) store_as(cache + d, r);
+        else if (p.qb) store_as(p.qb + at, r);
+        else p.q[at] = r;
+    }
+}
+
+// ---------------------------------------------------------------- every token alone
+// The keys that a token sees, in order: the kept first ones that its window has left behind, then the window.
+struct Keys {
+    int first, kept, n;
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + i - kept; }
+};
+__device__ __forceinline__ Keys keys_of(int pos, int last, int window, int keep) {
+    Keys k;
+    k.first = first_key(pos, window);
+    k.kept = min(keep, k.first);
+    k.n = k.kept + last - k.first + 1;
+    return k;
+}
+
+struct TokenParams {
+    const float* q;          // [T][heads * MAPS][ldq]
+    int ldq, heads, per, groups, dim, vdim, dim_p, vdim_p, v_at, window, keep, splits;
+    float scale, softcap;
+    const int32_t *seq_ids, *positions;
+    CacheRef c;
+    float *part, *part_ml;   // [T][heads * MAPS][splits][vdim], [T][heads * MAPS][splits][2]
 };
 
 constexpr int TK_KEYS = 32, TK_HEADS = 4;
 
-// One CTA per (key split, four query heads of one key head, token): a warp is a head.  Scores: a lane is a key; sums: a
-// lane owns the value pairs lane, lane + 32, ... (VP of them).
-template <typename TC, int VP>
+// One CTA per (key split, four query heads of one key head, token); with two maps per head two heads and their maps.  A
+// warp is a head and map.  Scores: a lane is a key; sums: a lane owns the value pairs lane, lane + 32, ... (VP of them).
+template <typename TC, int VP, int MAPS>
 __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams p) {
     constexpr int EPC = 16 / sizeof(TC);      // elements of a 16-byte chunk
     extern __shared__ __align__(16) uint8_t sm[];
-    const int ldk = p.dim_p + EPC, chunks = p.dim_p / EPC;
+    const int ldk = MAPS * p.dim_p + EPC, ldv = p.vdim_p + EPC, chunks = p.dim_p / EPC, vchunks = p.vdim_p / EPC;
     float* sq = reinterpret_cast<float*>(sm);                              // [TK_HEADS][dim_p]
-    TC* sk = reinterpret_cast<TC*>(sm + (size_t)TK_HEADS * p.dim_p * 4);   // [TK_KEYS][ldk], then the values
+    TC* sk = reinterpret_cast<TC*>(sm + (size_t)TK_HEADS * p.dim_p * 4);   // [TK_KEYS][ldk], then the values [TK_KEYS][ldv]
     TC* sv = sk + TK_KEYS * ldk;
     pdl_launch_dependents();
     pdl_wait();
     const int s = blockIdx.x, g = blockIdx.y / p.groups, t = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int in_group = (blockIdx.y % p.groups) * TK_HEADS + warp, h = g * p.per + in_group, pos = p.positions[t], seq = p.seq_ids[t];
-    const bool live = in_group < p.per;
-    const int first = first_key(pos, p.window), nk = pos - first + 1;
-    const int per = ((nk + p.splits - 1) / p.splits + TK_KEYS - 1) / TK_KEYS * TK_KEYS;
-    const int kb = first + s * per, ke = min(first + nk, kb + per);
+    const int unit = (blockIdx.y % p.groups) * TK_HEADS + warp, map = unit % MAPS, h = g * p.per * MAPS + unit, pos = p.positions[t], seq = p.seq_ids[t];
+    const bool live = unit < p.per * MAPS;
+    const Keys keys = keys_of(pos, pos, p.window, p.keep);
+    const int per = ((keys.n + p.splits - 1) / p.splits + TK_KEYS - 1) / TK_KEYS * TK_KEYS;
+    const int kb = s * per, ke = min(keys.n, kb + per);
     if (live)
-        for (int c = lane; c < p.dim_p; c += 32) sq[warp * p.dim_p + c] = p.q[((size_t)t * p.heads + h) * p.ldq + c] * p.scale;
+        for (int c = lane; c < p.dim_p; c += 32) sq[warp * p.dim_p + c] = p.q[((size_t)t * p.heads * MAPS + h) * p.ldq + c] * p.scale;
     float m = -INFINITY, l = 0.0f, acc[VP][2];
 #pragma unroll
     for (int j = 0; j < VP; ++j) acc[j][0] = acc[j][1] = 0.0f;
@@ -149,13 +224,14 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
         const TC* src[TK_KEYS / TK_HEADS];                  // a warp's keys: all rows asked for before any arrives
 #pragma unroll
         for (int i = 0; i < TK_KEYS / TK_HEADS; ++i)
-            src[i] = reinterpret_cast<const TC*>(p.c.arena) + p.c.at(seq, min(k0 + warp * (TK_KEYS / TK_HEADS) + i, ke - 1)) + g * p.dim_p;
-        for (int c = lane; c < 2 * chunks; c += 32) {
-            const bool val = c >= chunks;
-            const int at = (val ? c - chunks : c) * EPC;
+            src[i] = reinterpret_cast<const TC*>(p.c.arena) + p.c.at(seq, keys.at(min(k0 + warp * (TK_KEYS / TK_HEADS) + i, ke - 1)));
+        for (int c = lane; c < MAPS * chunks + vchunks; c += 32) {
+            const bool val = c >= MAPS * chunks;
+            const int at = (val ? c - MAPS * chunks : c) * EPC, from = val ? p.v_at + g * p.vdim_p + at : g * MAPS * p.dim_p + at;
+            TC* to = (val ? sv : sk) + at;
 #pragma unroll
             for (int i = 0; i < TK_KEYS / TK_HEADS; ++i)
-                cp_async16z(smem_u32((val ? sv : sk) + (warp * (TK_KEYS / TK_HEADS) + i) * ldk + at), src[i] + (val ? p.v_off : 0) + at, true);
+                cp_async16z(smem_u32(to + (warp * (TK_KEYS / TK_HEADS) + i) * (val ? ldv : ldk)), src[i] + from, true);
         }
         cp_async_commit();
         cp_async_wait<0>();
@@ -166,13 +242,14 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
 #pragma unroll 8
         for (int c = 0; c < chunks; ++c) {
             float f[EPC];
-            unpack16(*reinterpret_cast<const uint4*>(sk + lane * ldk + c * EPC), f, TC());
+            unpack16(*reinterpret_cast<const uint4*>(sk + lane * ldk + map * p.dim_p + c * EPC), f, TC());
 #pragma unroll
             for (int i = 0; i < EPC; ++i) part[i] = fmaf(f[i], q[c * EPC + i], part[i]);
         }
         float sc = 0.0f;
 #pragma unroll
         for (int i = 0; i < EPC; ++i) sc += part[i];
+        if (p.softcap > 0.0f) sc = p.softcap * tanhf(sc / p.softcap);
         if (k0 + lane >= ke) sc = -INFINITY;
         float mx = sc;
 #pragma unroll
@@ -187,14 +264,14 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
             const float w = __shfl_sync(0xffffffffu, pr, kk);
 #pragma unroll
             for (int j = 0; j < VP; ++j) {
-                const TC* v = sv + kk * ldk + min(2 * (lane + 32 * j), p.dim_p - 2);     // beyond the head: never stored
+                const TC* v = sv + kk * ldv + min(2 * (lane + 32 * j), p.vdim_p - 2);     // beyond the head: never stored
                 acc[j][0] = fmaf(w, load_as(v), acc[j][0]);
                 acc[j][1] = fmaf(w, load_as(v + 1), acc[j][1]);
             }
         }
     }
     if (!live) return;
-    const size_t o = ((size_t)t * p.heads + h) * p.splits + s;
+    const size_t o = ((size_t)t * p.heads * MAPS + h) * p.splits + s;
     if (lane == 0) {
         p.part_ml[2 * o] = m;
         p.part_ml[2 * o + 1] = l;
@@ -204,57 +281,74 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int d = 2 * (lane + 32 * j) + i;
-            if (d < p.dim) p.part[o * p.dim + d] = acc[j][i];
+            if (d < p.vdim) p.part[o * p.vdim + d] = acc[j][i];
         }
 }
 
-// Splits of one (head, token) and the sink joined.
-__global__ void __launch_bounds__(128) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int dim,
-                                                  float sink, float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
-    __shared__ float sw[32];
+// Splits of one (head, token) and the sink joined; with two maps the second is taken off the first and the rest normed.
+template <int MAPS>
+__global__ void __launch_bounds__(128) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int vdim,
+                                                  float sink, float lambda, float mul, float eps, float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb,
+                                                  int ldm) {
+    __shared__ float sw[MAPS][32], red[33];
     pdl_launch_dependents();
     pdl_wait();
-    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31;
-    const size_t o = ((size_t)t * heads + h) * splits;
-    if (threadIdx.x < 32) {             // splits <= 32
-        const float m = lane < splits ? part_ml[2 * (o + lane)] : -INFINITY, l = lane < splits ? part_ml[2 * (o + lane) + 1] : 0.0f;
+    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const size_t o = ((size_t)t * heads + h) * MAPS * splits;
+    if (warp < MAPS) {                  // splits <= 32
+        const size_t at = o + warp * splits + lane;
+        const float m = lane < splits ? part_ml[2 * at] : -INFINITY, l = lane < splits ? part_ml[2 * at + 1] : 0.0f;
         float M = fmaxf(m, sink);
 #pragma unroll
         for (int k = 16; k > 0; k >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, k));
         const float w = expf(m - M), L = warp_sum(l * w) + expf(sink - M);
-        sw[lane] = w / L;
+        sw[warp][lane] = w / L * (warp ? -lambda : 1.0f);
     }
     __syncthreads();
-    for (int d = threadIdx.x; d < dim; d += 128) {
-        float v = 0.0f;
+    float v[2] = {0.0f, 0.0f}, ss = 0.0f;         // vdim <= 256
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int d = threadIdx.x + 128 * j;
+        if (d < vdim) {
+#pragma unroll
+            for (int i = 0; i < MAPS; ++i)
 #pragma unroll 16
-        for (int s = 0; s < splits; ++s) v = fmaf(part[(o + s) * dim + d], sw[s], v);
-        const size_t at = (size_t)t * ldm + (size_t)h * dim + d;
-        if (mixb) mixb[at] = __float2bfloat16_rn(v);
-        else mix[at] = v;
+                for (int s = 0; s < splits; ++s) v[j] = fmaf(part[(o + i * splits + s) * vdim + d], sw[i][s], v[j]);
+        }
+        ss = fmaf(v[j], v[j], ss);
+    }
+    const float f = MAPS > 1 ? mul / sqrtf(block_sum(ss, red) / (float)vdim + eps) : 1.0f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int d = threadIdx.x + 128 * j;
+        if (d >= vdim) break;
+        const size_t at = (size_t)t * ldm + (size_t)h * vdim + d;
+        if (mixb) mixb[at] = __float2bfloat16_rn(v[j] * f);
+        else mix[at] = v[j] * f;
     }
 }
 
-template <typename TC>
+template <typename TC, int MAPS>
 int launch_tokens(dc_ctx* ctx, const TokenParams& p, int kv_heads, int T) {
-    const size_t smem = (size_t)TK_HEADS * p.dim_p * 4 + (size_t)2 * TK_KEYS * (p.dim_p * sizeof(TC) + 16);
+    const size_t smem = (size_t)TK_HEADS * p.dim_p * 4 + (size_t)TK_KEYS * ((MAPS * p.dim_p + p.vdim_p) * sizeof(TC) + 32);
     const dim3 grid(p.splits, kv_heads * p.groups, T), block(TK_HEADS * 32);
-#define DC_TK(VP)                                                                                         \
-    do {                                                                                                  \
-        DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_tokens<TC, VP>, (int)smem, "k_gqa_tokens"));       \
-        return dc_launch(ctx, "k_gqa_tokens", k_gqa_tokens<TC, VP>, grid, block, smem, p);                \
+#define DC_TK(VP)                                                                                               \
+    do {                                                                                                        \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_tokens<TC, VP, MAPS>, (int)smem, "k_gqa_tokens"));       \
+        return dc_launch(ctx, "k_gqa_tokens", k_gqa_tokens<TC, VP, MAPS>, grid, block, smem, p);                \
     } while (0)
-    if (p.dim <= 64) DC_TK(1);
-    if (p.dim <= 128) DC_TK(2);
+    if (p.vdim <= 64) DC_TK(1);
+    if (p.vdim <= 128) DC_TK(2);
     DC_TK(4);
 #undef DC_TK
 }
 
 // ---------------------------------------------------------------- prompts
 struct PromptParams {
-    const __nv_bfloat16* q;  // [T][heads][ldq]
-    int ldq, heads, per, dim, dim_p, v_off, window;
-    float scale, sink;
+    const __nv_bfloat16* q;  // [T][heads * MAPS][ldq]
+    int ldq, heads, per, dim, vdim, dim_p, vdim_p, v_at, window, keep;
+    float scale, softcap, sink;
+    float lambda, mul, eps;  // two maps
     const int32_t *seq_ids, *positions, *starts, *tiles;     // tiles: (entry, first query of the entry) pairs
     CacheRef c;
     __nv_bfloat16* out;
@@ -263,61 +357,79 @@ struct PromptParams {
 
 constexpr int PK = 64;           // keys per tile
 
-// One CTA per (PQ queries of one entry, head), sixteen queries a warp; key and value tiles in a ring of ST stages, two
-// CTAs an SM.  DP: head size, padded.
-template <int DP, int PQ, int ST>
+// cap tanh(s / cap), s in units of cap: to about 2e-7 of the cap
+__device__ __forceinline__ float soft_cap(float z, float cap) {
+    return cap - __fdividef(2.0f * cap, 1.0f + ex2(2.8853900817779268f * z));
+}
+
+// One CTA per (QT = PQ / MAPS queries of one entry, head), sixteen rows (queries of one map) a warp; key and value tiles in
+// a ring of ST stages, two CTAs an SM.  DP, VP: key and value size, padded.
+template <int DP, int VP, int PQ, int ST, int MAPS>
 __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const PromptParams p) {
-    constexpr int LD = DP + 8, NT = 2 * PQ, CH = DP / 8;
+    constexpr int LD = DP + 8, LDK = MAPS * DP + 8, LDV = VP + 8, NT = 2 * PQ, CH = DP / 8, VCH = VP / 8, QT = PQ / MAPS;
     extern __shared__ __align__(16) uint8_t smem[];
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);     // [PQ][LD]
-    __nv_bfloat16* sK = sQ + PQ * LD;                               // [ST][PK][LD]
-    __nv_bfloat16* sV = sK + ST * PK * LD;                          // [ST][PK][LD]
+    __nv_bfloat16* sK = sQ + PQ * LD;                               // [ST][PK][LDK]
+    __nv_bfloat16* sV = sK + ST * PK * LDK;                         // [ST][PK][LDV]
     pdl_launch_dependents();
     pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, head = blockIdx.y;
     const int tile0 = (int)(gridDim.x - 1 - blockIdx.x);           // later queries see more keys: they start first
-    const int e = p.tiles[2 * tile0], q0 = p.tiles[2 * tile0 + 1];
-    if (q0 % PQ) return;                                            // tiles are listed per DC_LATENT_QTILE queries
+    const int e = p.tiles[2 * tile0], q0 = p.tiles[2 * tile0 + 1] + QT * blockIdx.z;
     const int t0 = p.starts[e], n = p.starts[e + 1] - t0, pos0 = p.positions[t0], seq = p.seq_ids[t0];
-    const int first = first_key(pos0 + q0, p.window), last = pos0 + min(q0 + PQ, n) - 1;
-    const int n_tiles = (last - first) / PK + 1, kc = p.dim_p / 8;
-    const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.c.arena) + (head / p.per) * p.dim_p;
+    if (q0 % QT || q0 >= n) return;                                 // tiles are listed per DC_LATENT_QTILE queries
+    const int last = pos0 + min(q0 + QT, n) - 1;
+    const Keys keys = keys_of(pos0 + q0, last, p.window, p.keep);
+    const int n_tiles = (keys.n + PK - 1) / PK, kc = p.dim_p / 8, vc = p.vdim_p / 8;
+    const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.c.arena);
+    const int k_at = (head / p.per) * MAPS * p.dim_p, v_at = p.v_at + (head / p.per) * p.vdim_p;
 
     const int lrow = tid >> 3, lc = tid & 7;                        // eight threads per key row
     auto load = [&](int tile, int buf) {
 #pragma unroll
         for (int i = 0; i < PK * 8 / NT; ++i) {
-            const int key = lrow + NT / 8 * i, pos = first + tile * PK + key;
-            const bool ok = pos <= last;
-            const __nv_bfloat16* src = cache + p.c.at(seq, ok ? pos : last);
-            const uint32_t dk = smem_u32(sK + (buf * PK + key) * LD), dv = smem_u32(sV + (buf * PK + key) * LD);
+            const int key = lrow + NT / 8 * i, at = tile * PK + key;
+            const bool ok = at < keys.n;
+            const __nv_bfloat16* src = cache + p.c.at(seq, ok ? keys.at(at) : last);
+            const uint32_t dk = smem_u32(sK + (buf * PK + key) * LDK), dv = smem_u32(sV + (buf * PK + key) * LDV);
 #pragma unroll
-            for (int c0 = 0; c0 < CH; c0 += 8) {
+            for (int c0 = 0; c0 < MAPS * CH; c0 += 8) {
+                const int c = c0 + lc, of = MAPS > 1 ? c % CH : c;
+                if (MAPS * CH % 8 && c >= MAPS * CH) break;
+                const bool in = ok && of < kc;
+                cp_async16z(dk + 16 * c, in ? src + k_at + (MAPS > 1 ? c / CH * p.dim_p : 0) + 8 * of : src, in);
+            }
+#pragma unroll
+            for (int c0 = 0; c0 < VCH; c0 += 8) {
                 const int c = c0 + lc;
-                if (CH % 8 && c >= CH) break;
-                const bool in = ok && c < kc;
-                cp_async16z(dk + 16 * c, in ? src + 8 * c : src, in);
-                cp_async16z(dv + 16 * c, in ? src + p.v_off + 8 * c : src, in);
+                if (VCH % 8 && c >= VCH) break;
+                const bool in = ok && c < vc;
+                cp_async16z(dv + 16 * c, in ? src + v_at + 8 * c : src, in);
             }
         }
         cp_async_commit();
     };
     for (int i = tid; i < PQ * CH; i += NT) {                       // the queries come with the first tile
-        const int r = i / CH, c = i - r * CH;
-        const bool in = q0 + r < n && 8 * c < p.ldq;
-        cp_async16z(smem_u32(sQ + r * LD + 8 * c), p.q + ((size_t)(t0 + q0 + (in ? r : 0)) * p.heads + head) * p.ldq + (in ? 8 * c : 0), in);
+        const int r = i / CH, c = i - r * CH, qr = r % QT;
+        const bool in = q0 + qr < n && 8 * c < p.ldq;
+        cp_async16z(smem_u32(sQ + r * LD + 8 * c),
+                    p.q + ((size_t)(t0 + q0 + (in ? qr : 0)) * p.heads * MAPS + head * MAPS + r / QT) * p.ldq + (in ? 8 * c : 0), in);
     }
 #pragma unroll
     for (int i = 0; i < ST - 1; ++i)
         if (i < n_tiles) load(i, i);
         else cp_async_commit();
-    const float sl2 = p.scale * 1.4426950408889634f, sink2 = p.sink * 1.4426950408889634f;
+    // capped scores are in units of log2 e already, others are multiplied on the way into the exponential
+    const bool capped = p.softcap > 0.0f;
+    const float cap = p.softcap * 1.4426950408889634f, to_cap = capped ? p.scale / p.softcap : 0.0f;
+    const float sl2 = capped ? 1.0f : p.scale * 1.4426950408889634f, sink2 = p.sink * 1.4426950408889634f;
     const int g = lane >> 2, t4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
-    const int qpos0 = pos0 + q0 + 16 * warp + g;
+    const int map = MAPS > 1 ? 16 * warp / QT : 0, qrow = 16 * warp - map * QT;       // first query of the warp
+    const int qpos0 = pos0 + q0 + qrow + g;
     const int window = p.window > 0 ? p.window : 0x7fffffff;
-    float o[CH][4];
+    float o[VCH][4];
 #pragma unroll
-    for (int i = 0; i < CH; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    for (int i = 0; i < VCH; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     // the sink is the first term of the sum (one lane of a row's four counts it)
     const bool sink = p.sink > -INFINITY;
     float m_run[2], l_run[2];
@@ -325,18 +437,18 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
     for (int h = 0; h < 2; ++h) m_run[h] = sink ? sink2 : -1e30f, l_run[h] = sink && t4 == 0 ? 1.0f : 0.0f;
 
     for (int tile = 0; tile < n_tiles; ++tile) {
-        const int buf = tile % ST, k0 = first + tile * PK;
+        const int buf = tile % ST, k0 = keys.at(tile * PK), k1 = keys.at(tile * PK + PK - 1);
         cp_async_wait<ST - 2>();
         __syncthreads();         // the tile has landed; every warp is done with the stage that the next load fills
         if (tile + ST - 1 < n_tiles) load(tile + ST - 1, (tile + ST - 1) % ST);
         else cp_async_commit();
-        const int wq0 = pos0 + q0 + 16 * warp;
-        if (k0 > wq0 + 15 || k0 + PK - 1 <= wq0 - window) continue;          // nothing of the tile is seen by these queries
+        const int wq0 = pos0 + q0 + qrow;
+        if (k0 > wq0 + 15 || (k1 <= wq0 - window && k0 >= p.keep)) continue;         // nothing of the tile is seen by these queries
         float s[8][4];
 #pragma unroll
         for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
         const uint32_t qa = smem_u32(sQ + (16 * warp + (mi & 1) * 8 + r8) * LD + (mi >> 1) * 8);
-        const uint32_t ka = smem_u32(sK + (buf * PK + (mi >> 1) * 8 + r8) * LD + (mi & 1) * 8);
+        const uint32_t ka = smem_u32(sK + (buf * PK + (mi >> 1) * 8 + r8) * LDK + map * DP + (mi & 1) * 8);
 #pragma unroll
         for (int kk = 0; kk < DP; kk += 16) {
             uint32_t a[4];
@@ -344,19 +456,25 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
 #pragma unroll
             for (int np = 0; np < 4; ++np) {
                 uint32_t b[4];
-                ldsm_x4(ka + 2 * (16 * np * LD + kk), b);
+                ldsm_x4(ka + 2 * (16 * np * LDK + kk), b);
                 mma_bf16(s[2 * np], a, b[0], b[1]);
                 mma_bf16(s[2 * np + 1], a, b[2], b[3]);
             }
         }
+        if (capped) {
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) s[nt][j] = soft_cap(s[nt][j] * to_cap, cap);
+        }
         // the warp's sixteen queries see the whole tile, or the mask decides key by key
-        if (!(k0 + PK - 1 <= wq0 && wq0 + 15 - k0 < window)) {
+        if (!(k1 <= wq0 && wq0 + 15 - k0 < window)) {
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
-                    const int kp = k0 + 8 * nt + 2 * t4 + (j & 1), qp = qpos0 + (j >> 1) * 8;
-                    if (!(kp <= qp && qp - kp < window)) s[nt][j] = -INFINITY;
+                    const int kp = keys.at(tile * PK + 8 * nt + 2 * t4 + (j & 1)), qp = qpos0 + (j >> 1) * 8;
+                    if (!(kp <= qp && (qp - kp < window || kp < p.keep))) s[nt][j] = -INFINITY;
                 }
         }
         float mx[2] = {-1e30f, -1e30f};
@@ -379,7 +497,7 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
                 m_run[h] = m_new[h];
                 l_run[h] *= corr;
 #pragma unroll
-                for (int i = 0; i < CH; ++i) {
+                for (int i = 0; i < VCH; ++i) {
                     o[i][2 * h] *= corr;
                     o[i][2 * h + 1] *= corr;
                 }
@@ -393,7 +511,7 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
                 s[nt][j] = w;
                 l_run[j >> 1] += w;
             }
-        const uint32_t va = smem_u32(sV + (buf * PK + (mi & 1) * 8 + r8) * LD + (mi >> 1) * 8);
+        const uint32_t va = smem_u32(sV + (buf * PK + (mi & 1) * 8 + r8) * LDV + (mi >> 1) * 8);
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks) {
             uint32_t a[4];
@@ -402,9 +520,9 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
             a[2] = pack_bf2(s[2 * ks + 1][0], s[2 * ks + 1][1]);
             a[3] = pack_bf2(s[2 * ks + 1][2], s[2 * ks + 1][3]);
 #pragma unroll
-            for (int dp = 0; dp < DP / 16; ++dp) {
+            for (int dp = 0; dp < VP / 16; ++dp) {
                 uint32_t b[4];
-                ldsm_x4_t(va + 2 * (16 * ks * LD + 16 * dp), b);
+                ldsm_x4_t(va + 2 * (16 * ks * LDV + 16 * dp), b);
                 mma_bf16(o[2 * dp], a, b[0], b[1]);
                 mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
             }
@@ -414,18 +532,59 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
     for (int h = 0; h < 2; ++h) {
         l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
         l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
-        const int row = q0 + 16 * warp + g + 8 * h;
-        if (row >= n) continue;
-        const float inv = 1.0f / l_run[h];
-        __nv_bfloat16* dst = p.out + (size_t)(t0 + row) * p.ldm + (size_t)head * p.dim;
+    }
+    float mul[2] = {1.0f / l_run[0], 1.0f / l_run[1]};
+    if (MAPS > 1) {
+        constexpr int LDX = VP + 4;
+        float* other = reinterpret_cast<float*>(smem);              // [QT][LDX]: the second map's answers
+        __syncthreads();                                            // every warp is done with queries, keys and values
 #pragma unroll
-        for (int nt = 0; nt < CH; ++nt)
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+            for (int nt = 0; nt < VCH; ++nt)
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+                    if (map) other[(qrow + g + 8 * h) * LDX + 8 * nt + 2 * t4 + j] = o[nt][2 * h + j] * mul[h];
+        __syncthreads();
+        if (map) return;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int nt = 0; nt < VCH; ++nt)
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {                       // zero beyond the head
+                    float& v = o[nt][2 * h + j];
+                    v = v * mul[h] - p.lambda * other[(qrow + g + 8 * h) * LDX + 8 * nt + 2 * t4 + j];
+                    ss = fmaf(v, v, ss);
+                }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            mul[h] = p.mul / sqrtf(ss / (float)p.vdim + p.eps);
+        }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        const int row = q0 + qrow + g + 8 * h;
+        if (row >= n) continue;
+        __nv_bfloat16* dst = p.out + (size_t)(t0 + row) * p.ldm + (size_t)head * p.vdim;
+#pragma unroll
+        for (int nt = 0; nt < VCH; ++nt)
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
                 const int c = 8 * nt + 2 * t4 + j;
-                if (c < p.dim) dst[c] = __float2bfloat16_rn(o[nt][2 * h + j] * inv);
+                if (c < p.vdim) dst[c] = __float2bfloat16_rn(o[nt][2 * h + j] * mul[h]);
             }
     }
+}
+
+template <int DP, int VP, int PQ, int ST, int MAPS>
+int launch_prompt(dc_ctx* ctx, const PromptParams& p, int n_tiles) {
+    constexpr int QT = PQ / MAPS, bytes = (PQ * (DP + 8) + ST * PK * (MAPS * DP + VP + 16)) * 2;
+    static_assert(bytes <= 227 * 1024 && (MAPS == 1 || QT * (VP + 4) * 4 <= bytes), "shared memory");
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_prompt<DP, VP, PQ, ST, MAPS>, bytes, "k_gqa_prompt"));
+    const dim3 grid(n_tiles, p.heads, QT < DC_LATENT_QTILE ? DC_LATENT_QTILE / QT : 1);
+    return dc_launch(ctx, "k_gqa_prompt", k_gqa_prompt<DP, VP, PQ, ST, MAPS>, grid, dim3(2 * PQ), (size_t)bytes, p);
 }
 
 CacheRef cache_ref(const dc_gqa_cache& c, int row) { return CacheRef{c.arena, c.tables, c.max_blocks, row}; }
@@ -435,6 +594,21 @@ float sink_of(const dc_gqa_mixer& m) { return m.sink ? m.sink_score : -INFINITY;
 
 int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
                        int max_pos, float* q, __nv_bfloat16* qb) {
+    if (m.qk_norm != DC_QK_NORM_ALL) {
+        if (m.off_v == m.off_k) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prep: values from the keys need the norm over all heads");
+        HeadsParams p = {proj, ldp, m.off_q, m.off_k, m.off_v, m.heads * m.maps, m.kv_heads * m.maps, m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at,
+                         dc_gqa_ldq(m), m.rot.dims, m.halves, max_pos, m.q_norm, m.k_norm, m.cos_sin, eps, st.seq_ids, st.positions, cache_ref(c, m.row), q, qb};
+        const dim3 grid(st.T, (p.nq + p.nk + p.nv + 7) / 8), block(256);
+#define DC_HEADS(VP)                                                                                                          \
+    return c.f32 ? dc_launch(ctx, "k_gqa_prep_heads", k_gqa_prep_heads<float, VP>, grid, block, 0, p)                          \
+                 : dc_launch(ctx, "k_gqa_prep_heads", k_gqa_prep_heads<__nv_bfloat16, VP>, grid, block, 0, p)
+        const int most = std::max(std::max(p.ldq, p.dim_p), p.vdim_p);
+        if (most <= 64) DC_HEADS(2);
+        if (most <= 128) DC_HEADS(4);
+        DC_HEADS(8);
+#undef DC_HEADS
+    }
+    if (m.halves || m.maps > 1 || m.off_v != m.off_k) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prep: form not available with the norm over all heads");
     int lanes = 3;               // a head's pairs, padding included, up to a power of two
     while (2 << lanes < dc_gqa_ldq(m)) ++lanes;
     PrepParams p = {proj, ldp, m.off_q, m.off_k, m.heads, m.kv_heads, m.dim, m.dim_p, dc_gqa_ldq(m), m.rot.dims, max_pos, lanes, m.q_norm, m.k_norm, m.cos_sin,
@@ -446,29 +620,40 @@ int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, co
 }
 
 int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
-                         float* part_ml, float* mix, __nv_bfloat16* mixb, int ldm) {
+                         float* part_ml, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
     const int per = m.heads / m.kv_heads;
-    TokenParams p = {q, dc_gqa_ldq(m), m.heads, per, (per + TK_HEADS - 1) / TK_HEADS, m.dim, m.dim_p, m.kv_heads * m.dim_p, m.window, splits, m.scale,
-                     st.seq_ids, st.positions, cache_ref(c, m.row), part, part_ml};
-    DC_TRY(c.f32 ? launch_tokens<float>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16>(ctx, p, m.kv_heads, st.T));
-    return dc_launch(ctx, "k_gqa_join", k_gqa_join, dim3(m.heads, st.T), dim3(128), 0, part, part_ml, m.heads, splits, m.dim, sink_of(m), mix, mixb, ldm);
+    TokenParams p = {q, dc_gqa_ldq(m), m.heads, per, (per * m.maps + TK_HEADS - 1) / TK_HEADS, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at, m.window, m.keep, splits,
+                     m.scale, m.softcap, st.seq_ids, st.positions, cache_ref(c, m.row), part, part_ml};
+    if (m.maps > 1) {
+        DC_TRY((c.f32 ? launch_tokens<float, 2>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16, 2>(ctx, p, m.kv_heads, st.T)));
+        return dc_launch(ctx, "k_gqa_join", k_gqa_join<2>, dim3(m.heads, st.T), dim3(128), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), m.lambda,
+                         1.0f - m.diff, eps, mix, mixb, ldm);
+    }
+    DC_TRY((c.f32 ? launch_tokens<float, 1>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16, 1>(ctx, p, m.kv_heads, st.T)));
+    return dc_launch(ctx, "k_gqa_join", k_gqa_join<1>, dim3(m.heads, st.T), dim3(128), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), 0.0f, 1.0f, eps, mix,
+                     mixb, ldm);
 }
 
 int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const int32_t* tiles, int n_tiles,
-                         const __nv_bfloat16* qb, __nv_bfloat16* mixb, int ldm) {
-    PromptParams p = {qb, dc_gqa_ldq(m), m.heads, m.heads / m.kv_heads, m.dim, m.dim_p, m.kv_heads * m.dim_p, m.window, m.scale, sink_of(m), st.seq_ids,
-                      st.positions, st.starts, tiles, cache_ref(c, m.row), mixb, ldm};
-    const dim3 grid(n_tiles, m.heads);
-#define DC_PROMPT(DP, PQ, ST)                                                                                      \
-    do {                                                                                                           \
-        const int bytes = (PQ + 2 * ST * PK) * (DP + 8) * 2;                                                       \
-        DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_prompt<DP, PQ, ST>, bytes, "k_gqa_prompt"));                \
-        return dc_launch(ctx, "k_gqa_prompt", k_gqa_prompt<DP, PQ, ST>, grid, dim3(2 * PQ), (size_t)bytes, p);     \
-    } while (0)
-    if (m.dim <= 32) DC_PROMPT(32, 128, 3);
-    if (m.dim <= 64) DC_PROMPT(64, 128, 3);
-    if (m.dim <= 96) DC_PROMPT(96, 128, 2);
-    if (m.dim <= 128) DC_PROMPT(128, 128, 2);
-    DC_PROMPT(256, 64, 2);
+                         const __nv_bfloat16* qb, float eps, __nv_bfloat16* mixb, int ldm) {
+    PromptParams p = {qb, dc_gqa_ldq(m), m.heads, m.heads / m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at, m.window, m.keep, m.scale, m.softcap, sink_of(m),
+                      m.lambda, 1.0f - m.diff, eps, st.seq_ids, st.positions, st.starts, tiles, cache_ref(c, m.row), mixb, ldm};
+    // the smallest pair of padded key and value sizes that holds the head
+#define DC_PROMPT(DP, VP, PQ, ST, MAPS)                                                                  \
+    if (m.maps == MAPS && m.dim <= DP && m.vdim <= VP) return launch_prompt<DP, VP, PQ, ST, MAPS>(ctx, p, n_tiles)
+    DC_PROMPT(32, 32, 128, 3, 1);
+    DC_PROMPT(32, 64, 128, 3, 1);
+    DC_PROMPT(64, 64, 128, 3, 1);
+    DC_PROMPT(96, 96, 128, 2, 1);
+    DC_PROMPT(64, 128, 128, 2, 1);
+    DC_PROMPT(128, 128, 128, 2, 1);
+    DC_PROMPT(256, 256, 64, 2, 1);
+    DC_PROMPT(32, 32, 128, 3, 2);
+    DC_PROMPT(32, 64, 128, 3, 2);
+    DC_PROMPT(64, 64, 128, 3, 2);
+    DC_PROMPT(64, 128, 128, 2, 2);
+    DC_PROMPT(128, 128, 128, 2, 2);
+    DC_PROMPT(128, 256, 64, 2, 2);
 #undef DC_PROMPT
+    return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prompt: head sizes %d and %d", m.dim, m.vdim);
 }

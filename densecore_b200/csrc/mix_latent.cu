@@ -1,5 +1,5 @@
 // Attention over a compressed key/value latent (one row per token: the normed latent c and a rotated key part that
-// all heads share), with an optional sliding window.
+// all heads share), with an optional sliding window and an optional gate per head on the output.
 //
 // Decode-sized steps and f32 models use the absorbed form: a head's unrotated query is taken through its W_uk once
 // (q' = W_uk^T q), scores are q' . c + q_rot . k_rot, the softmax-weighted sum of latents goes through W_uv at the
@@ -237,10 +237,11 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
         }
 }
 
-// Splits of one (head, token) joined, then taken through OUT_ROWS rows of the head's W_uv.
+// Splits of one (head, token) joined, then taken through OUT_ROWS rows of the head's W_uv and multiplied by the head's gate.
 constexpr int OUT_ROWS = 64;
 __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits,
                                                     int rank, const __nv_bfloat16* __restrict__ uv, int ldw, int vdim_p, int vdim,
+                                                    const float* __restrict__ gate, int ldg,
                                                     float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
     extern __shared__ __align__(16) float lat[];      // [rank padded to 8]
     __shared__ float sw[32];
@@ -250,6 +251,7 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
     for (int i = threadIdx.x * 128; i < (e1 - e0) * ldw * 2; i += 256 * 128) prefetch_l2(rows + i);
     pdl_wait();
     const size_t o = ((size_t)t * heads + h) * splits;
+    const float mul = gate ? sigmoid(gate[(size_t)t * ldg + h]) : 1.0f;
     if (warp == 0) {             // splits <= 32
         const float m = lane < splits ? part_ml[2 * (o + lane)] : -INFINITY, l = lane < splits ? part_ml[2 * (o + lane) + 1] : 0.0f;
         float M = m;
@@ -286,7 +288,7 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
         const int e = e0 + warp + 8 * i;
-        const float v = warp_sum(a[i]);
+        const float v = warp_sum(a[i]) * mul;
         const size_t at = (size_t)t * ldm + (size_t)h * vdim + e;
         if (lane == 0 && e < e1) {
             if (mixb) mixb[at] = __float2bfloat16_rn(v);
@@ -337,7 +339,7 @@ __global__ void __launch_bounds__(256) k_latent_gather(CacheRef c, const int32_t
 
 struct PromptParams {
     const float* proj;
-    int ldp, off_q, dim, rot, dim_p, vdim, vdim_p, uv_row, window;
+    int ldp, off_q, off_g, dim, rot, dim_p, vdim, vdim_p, uv_row, window;
     float scale;
     const int32_t *positions, *starts, *key_base, *tiles;    // tiles: (entry, first query of the entry) pairs
     const __nv_bfloat16* kv;
@@ -514,7 +516,7 @@ __global__ void __launch_bounds__(2 * PQ) k_latent_prompt(const PromptParams p) 
         l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
         const int row = q0 + 16 * warp + g + 8 * h;
         if (row >= n) continue;
-        const float inv = 1.0f / l_run[h];
+        const float inv = (p.off_g < 0 ? 1.0f : sigmoid(p.proj[(size_t)(t0 + row) * p.ldp + p.off_g + head])) / l_run[h];
         __nv_bfloat16* dst = p.out + (size_t)(t0 + row) * p.ldm + (size_t)head * p.vdim;
 #pragma unroll
         for (int nt = 0; nt < VD / 8; ++nt)
@@ -551,7 +553,8 @@ int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_st
                         cache_ref(c, m.row), part, part_ml};
     DC_TRY(c.f32 ? launch_absorbed<float>(ctx, p, st.T) : launch_absorbed<__nv_bfloat16>(ctx, p, st.T));
     return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T, (m.vdim + OUT_ROWS - 1) / OUT_ROWS), dim3(256), (size_t)dc_pad8(m.kv_rank) * 4, part, part_ml, m.heads, splits,
-                     m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim, mix, mixb, ldm);
+                     m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim,
+                     m.off_g < 0 ? nullptr : proj + m.off_g, ldp, mix, mixb, ldm);
 }
 
 int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const int32_t* key_base,
@@ -563,7 +566,7 @@ int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step
 int dc_launch_latent_prefill(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const int32_t* key_base, const int32_t* tiles,
                              int n_tiles, const float* proj, int ldp, const __nv_bfloat16* keys_kv, int ldkv, const __nv_bfloat16* keys_r,
                              int ldr, __nv_bfloat16* mixb, int ldm) {
-    PromptParams p = {proj, ldp, m.off_q, m.dim, m.rot_dim, m.dim_p, m.vdim, m.vdim_p, m.uv_row, m.window, m.scale, st.positions, st.starts,
+    PromptParams p = {proj, ldp, m.off_q, m.off_g, m.dim, m.rot_dim, m.dim_p, m.vdim, m.vdim_p, m.uv_row, m.window, m.scale, st.positions, st.starts,
                       key_base, tiles, keys_kv, ldkv, keys_r, ldr, (m.dim_p + ldr + 15) & ~15, mixb, ldm};
     const dim3 grid(n_tiles, m.heads);
     // 128 queries per CTA and three stages where they fit shared memory

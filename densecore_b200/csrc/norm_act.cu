@@ -1,5 +1,6 @@
 // Norms around the sublayers of a layer-list decoder: RMS norm of a sublayer's output added to the f32 residual;
-// RMS norm of residual rows (ahead of a layer's products, and the output norm on the rows whose logits are wanted).
+// RMS norm of residual rows (ahead of a layer's products, and the output norm on the rows whose logits are wanted), with
+// what a step still owes the residual added on the way.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -91,7 +92,95 @@ __global__ void __launch_bounds__(256) k_norm_rows(const float* __restrict__ x, 
     }
 }
 
+// Rows as above.  The step's row and the gathered rows (bf16 or f32, pitch sum.ld, a multiple of eight) are added first.
+template <int KEEP>
+__global__ void __launch_bounds__(256) k_pre_norm(float* __restrict__ x, const float* __restrict__ step, const dc_row_sum sum,
+                                                  const float* __restrict__ w, int H, int ld, float eps, float* __restrict__ out,
+                                                  __nv_bfloat16* __restrict__ outb) {
+    __shared__ float red[33];
+    __shared__ int32_t s_rows[DC_MOE_MAX_TOP];
+    dc::pdl_launch_dependents();
+    const int n4 = ld / 4;
+    float4 wv[KEEP], xv[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        wv[j] = w && i < n4 ? reinterpret_cast<const float4*>(w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    dc::pdl_wait();
+    const size_t off = (size_t)blockIdx.x * ld;
+    float4* x4 = reinterpret_cast<float4*>(x + off);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        xv[j] = i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    auto add = [&](float4& a, float4 b) { a.x += b.x, a.y += b.y, a.z += b.z, a.w += b.w; };
+    if (sum.k) {
+        if (threadIdx.x < (unsigned)sum.k) s_rows[threadIdx.x] = sum.rows[blockIdx.x * sum.k + threadIdx.x];
+        __syncthreads();
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i >= n4) continue;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+            for (int k = 0; k < sum.k; ++k) {
+                const size_t at = (size_t)s_rows[k] * sum.ld + 4 * i;
+                if (sum.yb) {
+                    const uint2 u = *reinterpret_cast<const uint2*>(sum.yb + at);
+                    add(v, make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                                       __uint_as_float(u.y & 0xffff0000u)));
+                } else {
+                    add(v, *reinterpret_cast<const float4*>(sum.y + at));
+                }
+            }
+            add(xv[j], v);
+        }
+    }
+    if (step)
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i < n4) add(xv[j], reinterpret_cast<const float4*>(step)[i]);
+        }
+    if (sum.k || step)
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i < n4) x4[i] = xv[j];
+        }
+    if (!w) return;
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) ss += (xv[j].x * xv[j].x + xv[j].y * xv[j].y) + (xv[j].z * xv[j].z + xv[j].w * xv[j].w);
+    const float inv = 1.0f / sqrtf(dc::block_sum(ss, red) / (float)H + eps);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        if (i >= n4) continue;
+        const float4 v = make_float4(xv[j].x * inv * wv[j].x, xv[j].y * inv * wv[j].y, xv[j].z * inv * wv[j].z, xv[j].w * inv * wv[j].w);
+        if (outb) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            reinterpret_cast<uint2*>(outb + off)[i] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            reinterpret_cast<float4*>(out + off)[i] = v;
+        }
+    }
+}
+
 }  // namespace
+
+int dc_launch_pre_norm(dc_ctx* ctx, float* x, const float* step, const dc_row_sum& sum, const float* w, int T, int H, int ld, float eps, float* out,
+                       __nv_bfloat16* outb) {
+    const dim3 grid(T), block(256);
+    if (ld % 8 || sum.k > DC_MOE_MAX_TOP || (sum.k && (sum.ld < ld || sum.ld % 8))) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "pre_norm: bad operand");
+    if (ld <= 1024) return dc_launch(ctx, "k_pre_norm", k_pre_norm<1>, grid, block, 0, x, step, sum, w, H, ld, eps, out, outb);
+    if (ld <= 2048) return dc_launch(ctx, "k_pre_norm", k_pre_norm<2>, grid, block, 0, x, step, sum, w, H, ld, eps, out, outb);
+    if (ld <= 4096) return dc_launch(ctx, "k_pre_norm", k_pre_norm<4>, grid, block, 0, x, step, sum, w, H, ld, eps, out, outb);
+    if (ld <= 8192) return dc_launch(ctx, "k_pre_norm", k_pre_norm<8>, grid, block, 0, x, step, sum, w, H, ld, eps, out, outb);
+    return dc_fail(ctx, DC_B200_UNSUPPORTED, "pre_norm: width %d is too large", H);
+}
 
 int dc_launch_post_norm(dc_ctx* ctx, float* x, const float* y, const float* w, int T, int H, int ld, float eps, __nv_bfloat16* xb) {
     const dim3 grid(T), block(256);

@@ -52,6 +52,7 @@ __global__ void k_place_rows(const float* __restrict__ src, int64_t n, int K, __
 
 // Values in the tensor's own order to their places in the device vector.
 cudaError_t put_vector(const dc_stack_tensor& t, const std::vector<float>& v) {
+    if (t.pitch) return cudaMemcpy2D(*t.vec + t.vec_off, (size_t)t.pitch * 4, v.data(), (size_t)t.shape[1] * 4, (size_t)t.shape[1] * 4, (size_t)t.shape[0], cudaMemcpyHostToDevice);
     if (!t.cols) return cudaMemcpy(*t.vec + t.vec_off, v.data(), v.size() * 4, cudaMemcpyHostToDevice);
     const size_t taps = (size_t)t.shape[1], n = v.size() / taps;
     std::vector<float> w(v.size());
@@ -212,36 +213,36 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
         return off;
     };
     int span = 1;
-    auto key_range = [&](int window) {          // which of the distinct windows
-        span = std::max(span, window > 0 ? std::min(window, c.max_ctx) : c.max_ctx);
+    auto key_range = [&](int window, int keep) {        // which of the distinct windows
+        span = std::max(span, window > 0 ? std::min(window + keep, c.max_ctx) : c.max_ctx);
         auto w = std::find(s->windows.begin(), s->windows.end(), window);
         const int i = (int)(w - s->windows.begin());
         if (w == s->windows.end()) s->windows.push_back(window);
         return i;
     };
-    for (dc_stack_layer& L : s->layers) {
+    auto plane = [&](int row) {
+        planes.push_back((size_t)row * elt);
+        return (int)planes.size() - 1;
+    };
+    std::vector<int> written(s->layers.size(), -1);     // plane of a layer's last run
+    for (dc_stack_run& r : s->runs) {
+        dc_stack_layer& L = s->layers[r.layer];
         if (L.kind == DC_MIX_LIGHTNING) {
-            L.state_off = carve((size_t)L.li.heads * L.li.vdim * L.li.dim);
+            r.state_off = carve((size_t)L.li.heads * L.li.vdim * L.li.dim);
         } else if (L.kind == DC_MIX_GQA) {
-            L.ga.plane = (int)planes.size();
-            planes.push_back((size_t)L.ga.row * elt);
-            L.ga.range = key_range(L.ga.window);
+            r.plane = plane(L.ga.row);
+            L.ga.range = key_range(L.ga.window, L.ga.keep);
             DC_TRY(rotation_table(m, L.ga.rot, &L.ga.cos_sin));
         } else if (L.kind == DC_MIX_DELTA) {
-            L.state_off = carve((size_t)L.dl.heads * L.dl.vdim * L.dl.dim);
-            L.ring_off = carve((size_t)L.dl.taps * (L.dl.off_v + L.dl.heads * L.dl.vdim));
+            r.state_off = carve((size_t)L.dl.heads * L.dl.vdim * L.dl.dim);
+            r.ring_off = carve((size_t)L.dl.taps * (L.dl.off_v + L.dl.heads * L.dl.vdim));
         } else if (L.kind == DC_MIX_SSD) {
-            L.state_off = carve((size_t)L.ssd.heads * L.ssd.vdim * L.ssd.state);
-            L.ring_off = carve((size_t)L.ssd.taps * (L.ssd.heads * L.ssd.vdim + 2 * L.ssd.groups * L.ssd.state));
+            r.state_off = carve((size_t)L.ssd.heads * L.ssd.vdim * L.ssd.state);
+            r.ring_off = carve((size_t)L.ssd.taps * (L.ssd.heads * L.ssd.vdim + 2 * L.ssd.groups * L.ssd.state));
         } else {
             dc_latent_mixer& a = L.la;
-            if (a.kv_from < 0) {
-                a.plane = (int)planes.size();
-                planes.push_back((size_t)a.row * elt);
-            } else {
-                a.plane = s->layers[a.kv_from].la.plane;
-            }
-            a.range = key_range(a.window);
+            r.plane = written[r.layer] = a.kv_from < 0 ? plane(a.row) : written[a.kv_from];
+            a.range = key_range(a.window, 0);
             dc_rotation rot;
             rot.dims = a.rot_dim, rot.base = a.rot_base;
             DC_TRY(rotation_table(m, rot, &a.cos_sin));
@@ -252,6 +253,20 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
     const int per_seq = (c.max_ctx + DC_KV_BLOCK - 1) / DC_KV_BLOCK;
     const int blocks = pool_tokens > 0 ? (pool_tokens + DC_KV_BLOCK - 1) / DC_KV_BLOCK : per_seq * c.max_seqs;
     return dc_kv_init_planes(ctx, &m->kv, planes, state, blocks, c.max_seqs, per_seq);
+}
+
+// lambda of a differential attention layer, from its loaded vectors
+static int map_weight(dc_model* m, dc_gqa_mixer* d) {
+    std::vector<float> v[4];
+    for (int i = 0; i < 4; ++i) {
+        v[i].resize(d->dim);
+        DC_TRY(dc_check_cuda(m->ctx, cudaMemcpy(v[i].data(), d->lam[i], (size_t)d->dim * 4, cudaMemcpyDeviceToHost), "finalize"));
+    }
+    double dot[2] = {0.0, 0.0};
+    for (int i = 0; i < d->dim; ++i)
+        for (int j = 0; j < 2; ++j) dot[j] += (double)v[2 * j][i] * v[2 * j + 1][i];
+    d->lambda = (float)(exp(dot[0]) - exp(dot[1]) + (double)d->diff);
+    return DC_B200_OK;
 }
 
 static constexpr int ENTRY_INTS = DC_MAX_T + 1;
@@ -269,10 +284,15 @@ int dc_stack_finalize(dc_model* m) {
     size_t q = 0, actb = 0, head_state = 0;
     bool latent = false;
     size_t proj = 8, act = 8, low = 8, gate = 8, small = 8, mix = 8, ff = 8, lowb = 8, rank = 8, rot = 8, ukv = 8, blk = 8, qa = 0, part = 0, ml = 0;
+    size_t top = 0, experts = 8, hid = 8;
     int span = 1;
     for (dc_stack_layer& L : s->layers) {
         auto up = [](size_t& a, long long v) { a = std::max(a, (size_t)dc_pad8((int)v)); };
         up(ff, L.ff);
+        if (L.moe.experts) {
+            top = std::max(top, (size_t)L.moe.top);
+            up(experts, L.moe.experts), up(hid, L.moe.ff);
+        }
         const size_t parts = std::max((size_t)DC_MAX_T * s->splits, f32 ? C : 0);
         auto attention = [&](int heads, int values, int window) {
             part = std::max(part, parts * heads * values);
@@ -282,8 +302,10 @@ int dc_stack_finalize(dc_model* m) {
         if (s->cfg.block == DC_BLOCK_PARALLEL) up(mix, L.out.K);
         if (L.kind == DC_MIX_GQA) {
             up(proj, L.ff ? L.pair0 : L.in.N);
-            q = std::max(q, (size_t)L.ga.heads * dc_gqa_ldq(L.ga));
-            attention(L.ga.heads, L.ga.dim, L.ga.window);
+            up(mix, L.out.K);
+            q = std::max(q, (size_t)L.ga.heads * L.ga.maps * dc_gqa_ldq(L.ga));
+            attention(L.ga.heads * L.ga.maps, L.ga.vdim, L.ga.window);
+            if (L.ga.maps > 1) DC_TRY(map_weight(m, &L.ga));
         } else if (L.kind == DC_MIX_LIGHTNING) {
             up(f32 ? proj : actb, L.ff ? L.pair0 : L.in.N);
             up(act, L.li.heads * L.li.vdim);
@@ -332,6 +354,25 @@ int dc_stack_finalize(dc_model* m) {
     if (q) {
         DC_TRY(alloc(m, &b.q, F * q));
         if (!f32) DC_TRY(alloc(m, &b.qb, C * q));
+    }
+    if (top) {
+        const size_t rows = C * top;
+        b.moe_rows = (int)rows;
+        DC_TRY(alloc(m, &b.moe_ids, rows));
+        DC_TRY(alloc(m, &b.moe_row, rows));
+        DC_TRY(alloc(m, &b.moe_src, rows));
+        DC_TRY(alloc(m, &b.moe_w, rows));
+        DC_TRY(alloc(m, &b.moe_row_w, rows));
+        DC_TRY(alloc(m, &b.moe_off, experts + 1));
+        DC_TRY(alloc(m, &b.moe_logits, C * experts));
+        if (f32) {
+            DC_TRY(alloc(m, &b.moe_hid, rows * hid));
+            DC_TRY(alloc(m, &b.moe_y, rows * H));
+        } else {
+            DC_TRY(alloc(m, &b.moe_x, rows * H));
+            DC_TRY(alloc(m, &b.moe_hidb, rows * hid));
+            DC_TRY(alloc(m, &b.moe_yb, rows * H));
+        }
     }
     if (!s->windows.empty()) {
         DC_TRY(alloc(m, &b.part, part));
@@ -428,10 +469,10 @@ dc_lin_epi to(float* out, int ld) { return dc_lin_epi::store(out, nullptr, ld); 
 
 double lin_bytes(const dc_lin& w, int T) { return (double)w.N * w.ld * 2 + (double)T * (w.N + w.K) * 4; }
 
-int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
+int mix_delta(dc_model* m, const dc_step& st, const dc_stack_run& run, dc_stack_layer& Ly) {
     const dc_delta_mixer& d = Ly.dl;
     const dc_stack_buffers& b = m->stack->b;
-    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, run.state_off, run.ring_off};
     const int ldp = d.in.N, lda = dc_pad8(d.off_v + d.heads * d.vdim), ldl = d.in.N - d.off_a, ldm = d.heads * d.vdim;
     if (st.single && st.T <= DC_MAX_T)
         return dc_launch_delta_decode(m->ctx, d, st, sr, b.proj, ldp, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(ldm));
@@ -448,10 +489,10 @@ int mix_delta(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
                                 st.b16 ? nullptr : b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(ldm));
 }
 
-int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
+int mix_ssd(dc_model* m, const dc_step& st, const dc_stack_run& run, dc_stack_layer& Ly) {
     const dc_ssd_mixer& d = Ly.ssd;
     const dc_stack_buffers& b = m->stack->b;
-    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, Ly.ring_off};
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, run.state_off, run.ring_off};
     const int inner = d.heads * d.vdim, lda = dc_pad8(inner + 2 * d.groups * d.state);
     if (st.single && st.T <= DC_MAX_T)
         return dc_launch_ssd_decode(m->ctx, d, st, sr, b.proj, d.in.N, b.scan, lda, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, dc_pad8(inner));
@@ -459,11 +500,11 @@ int mix_ssd(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
                          st.b16 ? b.mixb : nullptr, dc_pad8(inner));
 }
 
-int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
+int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_stack_run& run, dc_stack_layer& Ly) {
     const dc_latent_mixer& d = Ly.la;
     const dc_stack_buffers& b = m->stack->b;
     dc_latent_cache c;
-    c.arena = m->kv.planes[d.plane].arena;
+    c.arena = m->kv.planes[run.plane].arena;
     c.f32 = m->stack->dtype == DC_DTYPE_F32;
     c.tables = m->kv.d_tables;
     c.max_blocks = m->kv.max_blocks_per_seq;
@@ -481,24 +522,24 @@ int mix_latent(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_laye
     return dc_launch_latent_prefill(m->ctx, d, st, base, sk.tiles, sk.n_tiles, b.proj, ldp, b.keys_kv, d.ukv.N, b.keys_r, ldr, b.mixb, ldm);
 }
 
-int mix_gqa(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
+int mix_gqa(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_stack_run& run, dc_stack_layer& Ly) {
     const dc_gqa_mixer& d = Ly.ga;
     const dc_stack_buffers& b = m->stack->b;
     dc_gqa_cache c;
-    c.arena = m->kv.planes[d.plane].arena;
+    c.arena = m->kv.planes[run.plane].arena;
     c.f32 = m->stack->dtype == DC_DTYPE_F32;
     c.tables = m->kv.d_tables;
     c.max_blocks = m->kv.max_blocks_per_seq;
     const int ldp = Ly.ff ? Ly.pair0 : Ly.in.N, ldm = dc_pad8(Ly.out.K);
     DC_TRY(dc_launch_gqa_prep(m->ctx, d, st, c, b.proj, ldp, m->stack->cfg.eps, m->cfg.max_ctx, b.q, st.tc ? b.qb : nullptr));
-    if (st.tc) return dc_launch_gqa_prompt(m->ctx, d, st, c, sk.tiles, sk.n_tiles, b.qb, b.mixb, ldm);
-    return dc_launch_gqa_tokens(m->ctx, d, st, c, b.q, st.T <= DC_MAX_T ? m->stack->splits : 1, b.part, b.part_ml, b.mix, st.b16 ? b.mixb : nullptr, ldm);
+    if (st.tc) return dc_launch_gqa_prompt(m->ctx, d, st, c, sk.tiles, sk.n_tiles, b.qb, m->stack->cfg.eps, b.mixb, ldm);
+    return dc_launch_gqa_tokens(m->ctx, d, st, c, b.q, st.T <= DC_MAX_T ? m->stack->splits : 1, b.part, b.part_ml, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, ldm);
 }
 
-int mix_lightning(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
+int mix_lightning(dc_model* m, const dc_step& st, const dc_stack_run& run, dc_stack_layer& Ly) {
     const dc_lightning_mixer& d = Ly.li;
     const dc_stack_buffers& b = m->stack->b;
-    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, Ly.state_off, 0};
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, run.state_off, 0};
     const int lda = Ly.ff ? Ly.pair0 : Ly.in.N, ldy = dc_pad8(d.heads * d.vdim), ldm = dc_pad8(Ly.out.K);
     const __nv_bfloat16* actb = st.b16 ? b.actb : nullptr;
     if (st.single && st.T <= DC_MAX_T) DC_TRY(dc_launch_lightning_decode(m->ctx, d, st, sr, b.proj, actb, lda, b.scan, ldy));
@@ -509,7 +550,7 @@ int mix_lightning(dc_model* m, const dc_step& st, dc_stack_layer& Ly) {
 
 // x += mixer(h) + ff(h) with h = norm1(x): one product from h, the mixer, one product back into the residual.  The
 // feed-forward's hidden values lie beside the mixer's output.
-int parallel_layer(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_layer& Ly) {
+int parallel_layer(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_stack_run& run, dc_stack_layer& Ly) {
     dc_stack* s = m->stack;
     dc_ctx* ctx = m->ctx;
     dc_stack_buffers& b = s->b;
@@ -521,13 +562,77 @@ int parallel_layer(dc_model* m, const dc_step& st, const StepKeys& sk, dc_stack_
     else in.bias = Ly.ga.bias;
     if (Ly.ff) in.pairs(Ly.pair0, DC_PAIR_CLAMPED, Ly.limit, b.mix + Ly.out_ff, st.b16 ? b.mixb + Ly.out_ff : nullptr, ldm, Ly.ff);
     L(DC_K_MIX_IN, lin_bytes(Ly.in, T), 1, linear(m, st, Ly.in, b.y, b.xb, H, in));
-    if (light) L(DC_K_MIX_LIGHTNING, 8.0 * st.E * Ly.li.heads * Ly.li.dim * Ly.li.vdim, st.single && !st.tc ? 2 : 4, mix_lightning(m, st, Ly));
-    else L(DC_K_MIX_GQA, 4.0 * T * Ly.in.N, st.tc ? 2 : 3, mix_gqa(m, st, sk, Ly));
+    if (light) L(DC_K_MIX_LIGHTNING, 8.0 * st.E * Ly.li.heads * Ly.li.dim * Ly.li.vdim, st.single && !st.tc ? 2 : 4, mix_lightning(m, st, run, Ly));
+    else L(DC_K_MIX_GQA, 4.0 * T * Ly.in.N, st.tc ? 2 : 3, mix_gqa(m, st, sk, run, Ly));
     dc_lin_epi out = to(b.x, H);
     out.add = true;
     out.bias = Ly.out_bias;
     L(DC_K_MIX_OUT, lin_bytes(Ly.out, T), 1, linear(m, st, Ly.out, b.mix, b.mixb, ldm, out));
     return DC_B200_OK;
+}
+
+// x += the layer's experts on norm2(x).  Steps of up to DC_MAX_T tokens of bf16 models add to x at once; the others leave
+// a row of every chosen expert behind, which *owed names.
+int moe_layer(dc_model* m, const dc_step& st, dc_stack_layer& Ly, dc_row_sum* owed) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    const dc_moe_ffn& f = Ly.moe;
+    const int W = s->cfg.width, H = dc_pad8(W), T = st.T, rows = T * f.top, F = dc_pad8(f.ff);
+    __nv_bfloat16* xb = st.b16 ? b.xb : nullptr;
+    const double up_bytes = (double)f.up_rows * f.up.ld * 2, down_bytes = (double)f.down_rows * f.down.ld * 2;
+    const double touched = std::min<double>(f.experts, rows);
+    if (T <= DC_MAX_T) {
+        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, dc_launch_moe_norm_route(ctx, f, b.x, Ly.norm2, T, W, H, s->cfg.eps, b.y, xb, b.moe_ids, b.moe_w));
+    } else {
+        L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, b.y, xb, H));
+        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, linear(m, st, f.router, b.y, b.xb, H, to(b.moe_logits, f.router.N)));
+        L(DC_K_ROUTER, 4.0 * T * f.experts, 1, dc_launch_moe_route(ctx, f, b.moe_logits, f.router.N, T, b.moe_ids, b.moe_w));
+    }
+    if (st.b16 && T <= DC_MAX_T) {
+        L(DC_K_MOE_GATEUP, touched * up_bytes, 1, dc_launch_moe_up_mma(ctx, f, b.xb, H, T, b.moe_ids, b.moe_w, b.moe_hidb, F));
+        L(DC_K_MOE_DOWN, touched * down_bytes, 1, dc_launch_moe_down_mma(ctx, f, b.moe_hidb, F, T, b.moe_ids, W, b.x, H));
+        return DC_B200_OK;
+    }
+    L(DC_K_ROUTER, 16.0 * rows, 1, dc_launch_moe_order(ctx, f, b.moe_ids, b.moe_w, T, b.moe_off, b.moe_src, b.moe_row_w, b.moe_row));
+    dc_lin_epi hid = dc_lin_epi().pairs(0, DC_PAIR_CLAMPED, f.limit, b.moe_hid, b.moe_hidb, F, f.ff);
+    hid.tok_scale = b.moe_row_w;
+    const dc_lin_epi y = dc_lin_epi::store(b.moe_y, b.moe_yb, H);
+    if (st.b16) {
+        dc_tc_in in;
+        L(DC_K_MOE_GATEUP, 4.0 * rows * W, 1, dc_launch_moe_gather(ctx, b.xb, H, b.moe_src, rows, b.moe_x));
+        DC_TRY(tc_in(m, &in, b.moe_x, W, H, b.moe_rows));
+        L(DC_K_MOE_GATEUP, touched * up_bytes + 2.0 * rows * (W + f.ff), 1, dc_launch_linear_grouped_tc(ctx, f.up, f.experts, f.up_rows, b.moe_off, in, rows, hid));
+        DC_TRY(tc_in(m, &in, b.moe_hidb, f.ff, F, b.moe_rows));
+        L(DC_K_MOE_DOWN, touched * down_bytes + 2.0 * rows * (W + f.ff), 1, dc_launch_linear_grouped_tc(ctx, f.down, f.experts, f.down_rows, b.moe_off, in, rows, y));
+    } else {
+        L(DC_K_MOE_GATEUP, touched * up_bytes, 1, dc_launch_moe_f32(ctx, f.up, f.experts, f.up_rows, b.moe_off, rows, b.y, H, b.moe_src, hid));
+        L(DC_K_MOE_DOWN, touched * down_bytes, 1, dc_launch_moe_f32(ctx, f.down, f.experts, f.down_rows, b.moe_off, rows, b.moe_hid, F, nullptr, y));
+    }
+    owed->y = b.moe_y, owed->yb = b.moe_yb, owed->rows = b.moe_row, owed->k = f.top, owed->ld = H;
+    return DC_B200_OK;
+}
+
+// x += mixer(norm1(x)), then x += experts(norm2(x)).  *owed: rows that the feed-forward before has not added yet.
+int pre_norm_layer(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_stack_run& run, dc_stack_layer& Ly, dc_row_sum* owed) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    const int W = s->cfg.width, H = dc_pad8(W), T = st.T;
+    const bool latent = Ly.kind == DC_MIX_LATENT;
+    const dc_lin &in = latent ? Ly.la.in : Ly.in, &o = latent ? Ly.la.o : Ly.out;
+    const float* step = run.step < 0 ? nullptr : s->loop_step + (size_t)run.step * H;
+    L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_pre_norm(ctx, b.x, step, *owed, Ly.norm1, T, W, H, s->cfg.eps, b.y, st.b16 ? b.xb : nullptr));
+    *owed = dc_row_sum();
+    dc_lin_epi proj = to(b.proj, in.N);
+    if (!latent) proj.bias = Ly.ga.bias;
+    L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.y, b.xb, H, proj));
+    if (latent) L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, run, Ly));
+    else L(DC_K_MIX_GQA, 4.0 * T * in.N, st.tc ? 2 : 3, mix_gqa(m, st, sk, run, Ly));
+    dc_lin_epi out = to(b.x, H);
+    out.add = true;
+    L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), out));
+    return Ly.moe.experts ? moe_layer(m, st, Ly, owed) : DC_B200_OK;
 }
 
 // Embedding and every layer; the residual ends in b.x.
@@ -544,20 +649,33 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
                                                     cudaMemcpyDeviceToDevice, ctx->stream), "capture");
     };
     m->last_launches = 0;
-    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, b.x, H, s->cfg.block == DC_BLOCK_PARALLEL ? nullptr : xb, s->cfg.embed_scale));
-    for (size_t il = 0; il < s->layers.size(); ++il) {
-        dc_stack_layer& Ly = s->layers[il];
+    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, b.x, H, s->cfg.block == DC_BLOCK_POST_NORM ? xb : nullptr, s->cfg.embed_scale));
+    dc_row_sum owed;
+    auto settle = [&]() -> int {
+        if (!owed.k) return DC_B200_OK;
+        L(DC_K_COMBINE, 4.0 * T * W * owed.k, 1, dc_launch_pre_norm(ctx, b.x, nullptr, owed, nullptr, T, W, H, eps, nullptr, nullptr));
+        owed = dc_row_sum();
+        return DC_B200_OK;
+    };
+    for (size_t il = 0; il < s->runs.size(); ++il) {
+        const dc_stack_run& run = s->runs[il];
+        dc_stack_layer& Ly = s->layers[run.layer];
+        if (m->dbg_x) DC_TRY(settle());
         DC_TRY(capture((int)il));
         if (s->cfg.block == DC_BLOCK_PARALLEL) {
-            DC_TRY(parallel_layer(m, st, sk, Ly));
+            DC_TRY(parallel_layer(m, st, sk, run, Ly));
+            continue;
+        }
+        if (s->cfg.block == DC_BLOCK_PRE_NORM) {
+            DC_TRY(pre_norm_layer(m, st, sk, run, Ly, &owed));
             continue;
         }
         const dc_lin& in = Ly.kind == DC_MIX_DELTA ? Ly.dl.in : Ly.kind == DC_MIX_SSD ? Ly.ssd.in : Ly.la.in;
         const dc_lin& o = Ly.kind == DC_MIX_DELTA ? Ly.dl.o : Ly.kind == DC_MIX_SSD ? Ly.ssd.o : Ly.la.o;
         L(DC_K_MIX_IN, lin_bytes(in, T), 1, linear(m, st, in, b.x, xb, H, to(b.proj, in.N)));
-        if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, st.single && !st.tc ? 1 : 7, mix_delta(m, st, Ly));
-        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, st.single && !st.tc ? 2 : 5, mix_ssd(m, st, Ly));
-        else L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, Ly));
+        if (Ly.kind == DC_MIX_DELTA) L(DC_K_MIX_DELTA, 8.0 * st.E * Ly.dl.heads * Ly.dl.dim * Ly.dl.vdim, st.single && !st.tc ? 1 : 7, mix_delta(m, st, run, Ly));
+        else if (Ly.kind == DC_MIX_SSD) L(DC_K_MIX_SSD, 8.0 * st.E * Ly.ssd.heads * Ly.ssd.state * Ly.ssd.vdim, st.single && !st.tc ? 2 : 5, mix_ssd(m, st, run, Ly));
+        else L(DC_K_MIX_LATENT, (double)Ly.la.ukv.N * Ly.la.ukv.ld * 2, 4, mix_latent(m, st, sk, run, Ly));
         L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), to(b.y, H)));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));
         if (!Ly.ff) continue;
@@ -566,7 +684,8 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
         L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, to(b.y, H)));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm2, T, W, H, eps, xb));
     }
-    return capture((int)s->layers.size());
+    DC_TRY(settle());
+    return capture((int)s->runs.size());
 }
 
 // Logits and greedy picks of R <= DC_MAX_T rows (rows: device list, or first, first + 1, ...).
@@ -679,10 +798,19 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
 
 void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token) {
     dc_stack* s = m->stack;
-    if (weight_bytes) *weight_bytes = (double)s->weight_bytes - (double)s->embed->bytes + (s->cfg.tied ? 0.0 : (double)s->embed->row_bytes);
-    double kv = 0.0;
-    for (dc_stack_layer& L : s->layers)
-        if (L.kind == DC_MIX_GQA) kv += (double)m->kv.planes[L.ga.plane].row_bytes;
-        else if (L.kind == DC_MIX_LATENT) kv += (double)m->kv.planes[L.la.plane].row_bytes;
+    double w = (double)s->head.N * s->head.ld * 2 + (s->cfg.tied ? 0.0 : (double)s->embed->row_bytes), kv = 0.0;
+    if (s->cfg.block != DC_BLOCK_PRE_NORM) {
+        w = (double)s->weight_bytes - (double)s->embed->bytes + (s->cfg.tied ? 0.0 : (double)s->embed->row_bytes);
+    } else {
+        for (const dc_stack_run& r : s->runs) {         // every run reads its layer; of the experts, those that a token chooses
+            const dc_stack_layer& L = s->layers[r.layer];
+            const dc_moe_ffn& f = L.moe;
+            for (const dc_lin* l : {&L.la.in, &L.la.ukv, &L.la.o, &L.in, &L.out, &f.router}) w += (double)l->N * l->ld * 2;
+            if (f.experts) w += ((double)f.up.N * f.up.ld + (double)f.down.N * f.down.ld) * 2 * f.top / f.experts;
+        }
+    }
+    for (const dc_stack_run& r : s->runs)
+        if (r.plane >= 0) kv += (double)m->kv.planes[r.plane].row_bytes;
+    if (weight_bytes) *weight_bytes = w;
     if (kv_bytes_per_token) *kv_bytes_per_token = kv;
 }

@@ -72,6 +72,17 @@ struct Reader {
         r->fast = number(*s, "fast", in), r->slow = number(*s, "slow", in);
         if (!(r->factor > 0.0 && r->original > 0.0 && r->fast > 0.0 && r->slow > 0.0)) bad(in + ": every value must be positive");
     }
+    // a sliding window, with the first tokens of the sequence kept in sight or not; no mask: every earlier token
+    void mask(const dc_json& o, const std::string& where, int* window, int* keep) {
+        const dc_json* v = o.get("mask");
+        if (!v || v->is_null()) return;
+        *window = size(*v, "size", where + ".mask");
+        const dc_json* k = v->get("keep_first");
+        if (k && !k->is_null()) {
+            if (keep) *keep = size(*v, "keep_first", where + ".mask", 0);
+            else bad(where + ".mask: 'keep_first' is not available here");
+        }
+    }
     // rows of a matrix appended to lin (whose K must agree); returns the first row
     int matrix(dc_lin* lin, const std::string& name, int N, int K) {
         const int row0 = lin->N;
@@ -165,7 +176,7 @@ void read_ssd(Reader& r, const dc_json& j, const std::string& p, const std::stri
     r.vec(&d.norm, p + "norm", {inner}, 1);
 }
 
-void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L, int il) {
+void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L, int il, bool gate) {
     dc_latent_mixer& d = L->la;
     const int H = r.s->cfg.width;
     d.heads = r.size(j, "heads", where);
@@ -178,8 +189,7 @@ void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::s
         d.rot_base = r.number(*rot, "base", where + ".rot");
         if (r.size(*rot, "dims", where + ".rot") != d.rot_dim || d.rot_dim % 2) r.bad(where + ": rot.dims must be even and equal rot_dim");
     }
-    const dc_json* mask = j.get("mask");
-    d.window = mask && !mask->is_null() ? r.size(*mask, "size", where + ".mask") : 0;
+    r.mask(j, where, &d.window, nullptr);
     const dc_json* from = j.get("kv_from");
     d.kv_from = from && !from->is_null() ? r.size(j, "kv_from", where, 0) : -1;
     d.row = dc_pad8(d.kv_rank + d.rot_dim);
@@ -197,6 +207,7 @@ void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::s
             return;
         }
     }
+    if (gate) d.off_g = r.matrix(&d.in, p + "g", d.heads, H);
     // every head's rows start at a multiple of eight in the expanded keys and values
     auto heads_of = [&](const char* n, int rows, int pad) {
         dc_stack_tensor t;
@@ -216,7 +227,8 @@ void read_latent(Reader& r, const dc_json& j, const std::string& p, const std::s
     r.matrix(&d.o, p + "o", H, d.heads * d.vdim);
 }
 
-// Mixers of parallel blocks: their input rows open L->in, their output matrix the columns of L->out.
+// The projections of these mixers open L->in, their output matrix the columns of L->out: a parallel block's feed-forward
+// goes beside both.
 void out_columns(Reader& r, const std::string& name, dc_stack_layer* L, int K) {
     const int H = r.s->cfg.width;
     dc_stack_tensor t;
@@ -229,32 +241,64 @@ void out_columns(Reader& r, const std::string& name, dc_stack_layer* L, int K) {
     L->out.K += K;
 }
 
-void read_gqa(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+// What a design fixes of its grouped-query attention
+enum {
+    GQA_KEY_VALUES = 1,     // the values are the key projection before norm and rotation
+    GQA_BIAS = 2,           // of the projections
+    GQA_OUT_BIAS = 4,
+    GQA_NORM_ALL = 8,       // queries and keys normed over all heads
+    GQA_NORM_HEAD = 16,     // ... per head and map
+    GQA_HALVES = 32,        // rotated pairs (i, i + dims / 2)
+    GQA_SINK = 64,          // a sink of score 0
+    GQA_TWO_MAPS = 128,     // differential attention
+};
+
+void read_gqa(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L, unsigned form) {
     dc_gqa_mixer& d = L->ga;
     const int H = r.s->cfg.width;
+    d.maps = form & GQA_TWO_MAPS ? 2 : 1;
     d.heads = r.size(j, "heads", where);
     d.kv_heads = r.size(j, "kv_heads", where);
-    d.dim = r.size(j, "dim", where, 1, 256);
-    if (r.size(j, "vdim", where) != d.dim) r.bad(where + ": the values are the keys, so vdim must equal dim");
+    d.dim = r.size(j, "dim", where, 1, d.maps > 1 ? 128 : 256);
+    d.vdim = r.size(j, "vdim", where, 1, 256);
+    if (form & GQA_KEY_VALUES && d.vdim != d.dim) r.bad(where + ": the values are the keys, so vdim must equal dim");
     if (d.heads % d.kv_heads) r.bad(where + ": heads is not a multiple of kv_heads");
     d.scale = (float)r.number(j, "scale", where);
     if (const dc_json* rot = r.object(j, "rot", where)) r.rotation(*rot, where + ".rot", &d.rot);
     if (d.rot.dims > d.dim) r.bad(where + ".rot: dims is larger than the head");
-    const dc_json* mask = j.get("mask");
-    d.window = mask && !mask->is_null() ? r.size(*mask, "size", where + ".mask") : 0;
-    d.sink = true, d.sink_score = 0.0f;
+    d.halves = form & GQA_HALVES;
+    r.mask(j, where, &d.window, &d.keep);
+    const dc_json* cap = j.get("softcap");
+    if (cap && !cap->is_null() && !((d.softcap = (float)r.number(j, "softcap", where)) > 0.0f)) r.bad(where + ": 'softcap' must be positive");
+    d.sink = form & GQA_SINK, d.sink_score = 0.0f;
+    d.qk_norm = form & GQA_NORM_ALL ? DC_QK_NORM_ALL : form & GQA_NORM_HEAD ? DC_QK_NORM_HEAD : DC_QK_PLAIN;
     d.dim_p = dc_pad8(d.dim);
-    d.row = 2 * d.kv_heads * d.dim_p;
-    const int Q = d.heads * d.dim, K = d.kv_heads * d.dim;
+    d.vdim_p = dc_pad8(d.vdim);
+    d.v_at = d.kv_heads * d.maps * d.dim_p;
+    d.row = d.v_at + d.kv_heads * d.vdim_p;
+    const int Q = d.heads * d.maps * d.dim, K = d.kv_heads * d.maps * d.dim, V = d.kv_heads * d.vdim;
+    const bool own_values = !(form & GQA_KEY_VALUES);
     d.off_q = r.matrix(&L->in, p + "q", Q, H);
     d.off_k = r.matrix(&L->in, p + "k", K, H);
-    const int rows = (L->in.N + DC_PAIR_ALIGN - 1) / DC_PAIR_ALIGN * DC_PAIR_ALIGN;     // as many as a product may store
-    r.vec(&d.bias, p + "q.b", {Q}, 4, d.off_q, rows);
-    r.vec(&d.bias, p + "k.b", {K}, 4, d.off_k, rows);
-    r.vec(&d.q_norm, p + "q.norm", {Q}, 1);
-    r.vec(&d.k_norm, p + "k.norm", {K}, 1);
-    out_columns(r, p + "o", L, Q);
-    r.vec(&L->out_bias, p + "o.b", {H}, 4);
+    d.off_v = own_values ? r.matrix(&L->in, p + "v", V, H) : d.off_k;
+    if (form & GQA_BIAS) {
+        const int rows = (L->in.N + DC_PAIR_ALIGN - 1) / DC_PAIR_ALIGN * DC_PAIR_ALIGN;     // as many as a product may store
+        r.vec(&d.bias, p + "q.b", {Q}, 4, d.off_q, rows);
+        r.vec(&d.bias, p + "k.b", {K}, 4, d.off_k, rows);
+        if (own_values) r.vec(&d.bias, p + "v.b", {V}, 4, d.off_v, rows);
+    }
+    if (d.qk_norm != DC_QK_PLAIN) {
+        const bool all = d.qk_norm == DC_QK_NORM_ALL;
+        r.vec(&d.q_norm, p + "q.norm", {all ? Q : d.dim}, 1);
+        r.vec(&d.k_norm, p + "k.norm", {all ? K : d.dim}, 1);
+    }
+    if (d.maps > 1) {
+        const char* names[] = {"lq1", "lk1", "lq2", "lk2"};
+        for (int i = 0; i < 4; ++i) r.vec(&d.lam[i], p + names[i], {d.dim}, 0);
+        d.diff = (float)r.number(j, "diff", where);
+    }
+    out_columns(r, p + "o", L, d.heads * d.vdim);
+    if (form & GQA_OUT_BIAS) r.vec(&L->out_bias, p + "o.b", {H}, 4);
 }
 
 void read_lightning(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
@@ -317,26 +361,83 @@ void read_dense_gelu(Reader& r, const dc_json& j, const std::string& p, const st
     r.matrix(&L->down, p + "down", H, L->ff);
 }
 
+void read_moe(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+    dc_moe_ffn& f = L->moe;
+    const int H = r.s->cfg.width;
+    const dc_json *router = r.object(j, "router", where), *expert = r.object(j, "expert", where);
+    if (!router || !expert) return;
+    f.experts = r.size(*router, "experts", where + ".router", 1, DC_MOE_MAX_EXPERTS);
+    f.top = r.size(*router, "top", where + ".router", 1, DC_MOE_MAX_TOP);
+    f.scale = (float)r.number(*router, "scale", where + ".router");
+    const dc_json* groups = router->get("groups");
+    if (groups && !groups->is_null()) {
+        f.groups = r.size(*groups, "count", where + ".router.groups", 1, DC_MOE_MAX_GROUPS);
+        f.keep = r.size(*groups, "keep", where + ".router.groups");
+    }
+    if (f.experts % f.groups) r.bad(where + ".router: experts is not a multiple of groups.count");
+    else if (f.keep > f.groups || f.top > f.experts / f.groups * f.keep) r.bad(where + ".router: fewer experts than 'top' in the kept groups");
+    f.ff = r.size(*expert, "ff", where + ".expert");
+    f.limit = (float)r.number(*expert, "limit", where + ".expert");
+    if (!r.error.empty()) return;
+    f.up_rows = 2 * dc_pad8(f.ff);
+    f.down_rows = (H + 15) & ~15;
+    r.matrix(&f.router, p + "router", f.experts, H);
+    r.vec(&f.correction, p + "correction", {f.experts}, 4);
+    f.up.N = f.experts * f.up_rows, f.up.K = H;
+    f.down.N = f.experts * f.down_rows, f.down.K = f.ff;
+    for (int e = 0; e < f.experts; ++e) {
+        const std::string in = p + "e" + std::to_string(e) + ".";
+        for (int i = 0; i < 3; ++i) {
+            const bool down = i == 2;
+            dc_stack_tensor t;
+            t.name = in + (down ? "down" : i ? "up" : "gate");
+            t.shape = {down ? H : f.ff, down ? f.ff : H};
+            t.lin = down ? &f.down : &f.up;
+            t.row0 = down ? e * f.down_rows : e * f.up_rows + i;
+            t.row_step = down ? 1 : 2;
+            r.tensor(t);
+        }
+    }
+}
+
+// {start, stop, times}: layers start .. stop - 1 run `times` times in a row
+void read_loop(Reader& r, const dc_json& j, int layers) {
+    dc_stack_config& c = r.s->cfg;
+    c.loop_start = r.size(j, "start", "config.loop", 0, layers - 1);
+    c.loop_stop = r.size(j, "stop", "config.loop", c.loop_start + 1, layers);
+    c.loop_times = r.size(j, "times", "config.loop", 1, 1024);
+    if (!r.error.empty()) return;
+    const int ld = dc_pad8(c.width);
+    r.vec(&r.s->loop_step, "loop.step", {c.loop_times, c.width}, 0, 0, (int64_t)c.loop_times * ld);
+    r.s->tensors.back().pitch = ld;
+}
+
 // ---------------------------------------------------------------- designs
-struct Arch {
-    const char* name;
-    unsigned mixers;        // bit per DC_MIX_*
-    int block;              // DC_BLOCK_*; parallel blocks have the clamped feed-forward, the others the tanh-gelu one
-    bool embed_scale;       // config.embedding.scale
-    bool tied;
-};
-const Arch kArchs[] = {
-    // Garilix: RMS norms on the sublayers' outputs only (x += norm(f(x))), tanh-gelu gated feed-forward
-    {"Garilix", (1u << DC_MIX_DELTA) | (1u << DC_MIX_LATENT) | (1u << DC_MIX_SSD), DC_BLOCK_POST_NORM, false, false},
-    // Datasun: mixer and clamped feed-forward side by side on one normed input, embedding table as output matrix
-    {"Datasun", (1u << DC_MIX_GQA) | (1u << DC_MIX_LIGHTNING), DC_BLOCK_PARALLEL, true, true},
-};
 struct MixerType {
     const char* name;
     int kind;
+    unsigned form;          // GQA_* of grouped-query attention; latent attention: 1 if its heads are gated
 };
-const MixerType kMixers[] = {{"channel_delta", DC_MIX_DELTA}, {"latent_attention", DC_MIX_LATENT}, {"mamba2", DC_MIX_SSD},
-                              {"attention", DC_MIX_GQA}, {"lightning", DC_MIX_LIGHTNING}};
+struct Arch {
+    const char* name;
+    int block;              // DC_BLOCK_*: post-norm blocks have the tanh-gelu feed-forward, parallel ones the clamped one, pre-norm ones experts
+    bool embed_scale;       // config.embedding.scale
+    bool tied;
+    bool loops;             // config.loop
+    std::vector<MixerType> mixers;
+};
+const Arch kArchs[] = {
+    // Garilix: RMS norms on the sublayers' outputs only (x += norm(f(x))), tanh-gelu gated feed-forward
+    {"Garilix", DC_BLOCK_POST_NORM, false, false, false,
+     {{"channel_delta", DC_MIX_DELTA, 0}, {"latent_attention", DC_MIX_LATENT, 0}, {"mamba2", DC_MIX_SSD, 0}}},
+    // Datasun: mixer and clamped feed-forward side by side on one normed input, embedding table as output matrix
+    {"Datasun", DC_BLOCK_PARALLEL, true, true, false,
+     {{"attention", DC_MIX_GQA, GQA_KEY_VALUES | GQA_BIAS | GQA_OUT_BIAS | GQA_NORM_ALL | GQA_SINK}, {"lightning", DC_MIX_LIGHTNING, 0}}},
+    // Gomuzen: norms ahead of the sublayers, looped layers, gated latent attention, differential attention, biased attention over
+    // a window and the first tokens, experts in groups
+    {"Gomuzen", DC_BLOCK_PRE_NORM, false, false, true,
+     {{"latent_attention", DC_MIX_LATENT, 1}, {"attention", DC_MIX_GQA, GQA_NORM_HEAD | GQA_HALVES | GQA_TWO_MAPS}, {"attention_2", DC_MIX_GQA, GQA_BIAS | GQA_HALVES}}},
+};
 
 int alloc_lin(dc_model* m, dc_lin* l) {
     if (!l->N) return DC_B200_OK;
@@ -376,6 +477,10 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
 
     const int H = s->cfg.width, n = (int)layers->arr.size();
     s->layers.resize(n);
+    if (const dc_json* loop = cj.get("loop"); loop && !loop->is_null()) {
+        if (!a->loops) r.bad("config: 'loop' is not available in this architecture");
+        else read_loop(r, *loop, n);
+    }
     {
         dc_stack_tensor t;
         t.name = "embed";
@@ -393,32 +498,49 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         dc_stack_layer& L = s->layers[i];
         const dc_json *type = lj.get("type"), *mixer = lj.get("mixer"), *mlp = lj.get("mlp");
         L.kind = -1;
-        for (const MixerType& t : kMixers)
-            if (type && type->kind == dc_json::STR && type->str == t.name && (a->mixers >> t.kind & 1)) L.kind = t.kind;
+        unsigned form = 0;
+        for (const MixerType& t : a->mixers)
+            if (type && type->kind == dc_json::STR && type->str == t.name) L.kind = t.kind, form = t.form;
         if (L.kind < 0 || !mixer || mixer->kind != dc_json::OBJ) {
             r.bad(where + ": unknown mixer type '" + (type ? type->str : "") + "'");
             break;
         }
         if (L.kind == DC_MIX_DELTA) read_delta(r, *mixer, p + "mix.", where + ".mixer", &L);
         else if (L.kind == DC_MIX_SSD) read_ssd(r, *mixer, p + "mix.", where + ".mixer", &L);
-        else if (L.kind == DC_MIX_GQA) read_gqa(r, *mixer, p + "mix.", where + ".mixer", &L);
+        else if (L.kind == DC_MIX_GQA) read_gqa(r, *mixer, p + "mix.", where + ".mixer", &L, form);
         else if (L.kind == DC_MIX_LIGHTNING) read_lightning(r, *mixer, p + "mix.", where + ".mixer", &L);
-        else read_latent(r, *mixer, p + "mix.", where + ".mixer", &L, i);
+        else read_latent(r, *mixer, p + "mix.", where + ".mixer", &L, i, form);
         r.vec(&L.norm1, p + "norm1", {H}, 1);
         if (mlp && !mlp->is_null()) {
             const dc_json* kind = mlp->get("kind");
-            if (!kind || kind->str != "dense") {
+            const bool pre = a->block == DC_BLOCK_PRE_NORM;
+            if (!kind || kind->str != (pre ? "moe" : "dense")) {
                 r.bad(where + ".mlp: unknown kind");
                 break;
             }
             if (a->block == DC_BLOCK_PARALLEL) {
                 read_dense_clamped(r, *mlp, p + "mlp.", where + ".mlp", &L);
             } else {
-                read_dense_gelu(r, *mlp, p + "mlp.", where + ".mlp", &L);
+                if (pre) read_moe(r, *mlp, p + "mlp.", where + ".mlp", &L);
+                else read_dense_gelu(r, *mlp, p + "mlp.", where + ".mlp", &L);
                 r.vec(&L.norm2, p + "norm2", {H}, 1);
             }
         }
     }
+    // the order in which layers run
+    const dc_stack_config& c = s->cfg;
+    auto run = [&](int from, int to, int pass) {
+        for (int i = from; i < to; ++i) {
+            dc_stack_run e;
+            e.layer = i;
+            e.step = i == from ? pass : -1;
+            s->runs.push_back(e);
+        }
+    };
+    const int stop = c.loop_times ? c.loop_stop : n, start = c.loop_times ? c.loop_start : n;
+    run(0, start, -1);
+    for (int t = 0; t < c.loop_times; ++t) run(start, stop, t);
+    run(stop, n, -1);
     r.vec(&s->final_norm, "final.norm", {H}, 1);
     if (!s->cfg.tied) r.matrix(&s->head, "head", s->cfg.vocab, H);
     if (!r.error.empty()) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "%s", r.error.c_str());
@@ -440,7 +562,7 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)&s->embed->dev, s->embed->bytes + 64), "weight memory"));
     }
     for (dc_stack_layer& L : s->layers) {
-        dc_lin* ls[] = {&L.dl.in, &L.dl.a2, &L.dl.g2, &L.dl.o, &L.ssd.in, &L.ssd.o, &L.la.in, &L.la.ukv, &L.la.o, &L.gate_up, &L.down, &L.in, &L.out};
+        dc_lin* ls[] = {&L.dl.in, &L.dl.a2, &L.dl.g2, &L.dl.o, &L.ssd.in, &L.ssd.o, &L.la.in, &L.la.ukv, &L.la.o, &L.gate_up, &L.down, &L.in, &L.out, &L.moe.router, &L.moe.up, &L.moe.down};
         for (dc_lin* l : ls) DC_TRY(alloc_lin(m, l));
         if (!L.li.decays.empty()) {
             const size_t bytes = L.li.decays.size() * 4;

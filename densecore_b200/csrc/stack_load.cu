@@ -58,7 +58,7 @@ int create(dc_ctx* ctx, const dc_json& config, const Shapes& shapes, int dtype, 
     if (st == DC_B200_OK) {
         m->stack->dtype = dtype;
         dc_model_config& c = m->cfg;
-        c.n_layer = (int)m->stack->layers.size();
+        c.n_layer = (int)m->stack->runs.size();
         c.hidden = m->stack->cfg.width;
         c.vocab = m->stack->cfg.vocab;
         c.rms_eps = m->stack->cfg.eps;
