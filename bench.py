@@ -384,6 +384,22 @@ def datasun_config(width: int, repeats: int, vocab: int = 32768):
     return {"architecture": "Datasun", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "layers": layers}
 
 
+def gomuzen_config(width: int, repeats: int, vocab: int = 32768):
+    """A Gomuzen decoder whose layers have the sizes of a real model of this width: per repeat one latent, one differential and two
+    windowed attention layers, each with 64 experts of which a token uses 8; the first four layers run twice.  4 * (repeats + 1) layer runs."""
+    h, g = width // 128, max(1, width // 512)
+    rot = {"base": 10000.0, "dims": 64}
+    latent = {"type": "latent_attention", "mixer": {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": rot}}
+    diff = {"type": "attention", "mixer": {"heads": h, "kv_heads": g, "dim": 64, "vdim": 128, "diff": 0.5, "scale": 0.125, "softcap": 30.0, "rot": rot}}
+    kept = {"type": "attention_2", "mixer": {"heads": h, "kv_heads": g, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                                             "mask": {"size": 1024, "keep_first": 4},
+                                             "rot": dict(rot, scaling={"factor": 2.0, "original": 2048, "fast": 32.0, "slow": 1.0})}}
+    mlp = {"kind": "moe", "expert": {"ff": 3 * width // 8, "limit": 7.0},
+           "router": {"experts": 64, "top": 8, "scale": 2.0, "groups": {"count": 8, "keep": 4}}}
+    return {"architecture": "Gomuzen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 4, "times": 2},
+            "layers": [dict(ly, mlp=mlp) for ly in (latent, diff, kept, kept) * repeats]}
+
+
 def time_decoder(m, vocab: int, prompt: int, streams, steps: int, reps: int = 5) -> dict:
     """Prompt throughput (host tokens in, first token out, best of reps on fresh sequences) and greedy decode after
     that prompt (device time of decode_run) of any decoder of the library."""
@@ -446,6 +462,26 @@ def bench_datasun(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), r
         r = {}
         for name, (cfg, shapes) in (("datasun_bf16", (datasun_config(w, repeats), {})), ("garilix_bf16", garilix_config(w, repeats))):
             m = dc.Model.from_config(ctx, cfg, shapes, max_seqs=4, max_ctx=prompt + 512)
+            m.init_synthetic(11, 0.02)
+            m.finalize()
+            r[name] = time_decoder(m, cfg["vocab"], prompt, (1, 4), steps)
+            m.close()
+            for v in r[name]["decode"].values():
+                v["hbm_fraction"] = v["weight_gbs"] / peak_gbs
+        out["sizes"][str(w)] = r
+    return out
+
+
+def bench_gomuzen(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), repeats: int = 2, prompt: int = 2048) -> dict:
+    """Gomuzen decoders (bf16, random weights) beside Datasun decoders of the same width, number of layer runs, vocabulary and
+    feed-forward size that a token uses.  Decode reads more weights than the L2 holds at the larger widths; no flush."""
+    import densecore_b200 as dc
+    runs = 4 * (repeats + 1)
+    out = {"vocab": 32768, "layer_runs": runs, "sizes": {}}
+    for w in widths:
+        r = {}
+        for name, cfg in (("gomuzen_bf16", gomuzen_config(w, repeats)), ("datasun_bf16", datasun_config(w, runs // 6))):
+            m = dc.Model.from_config(ctx, cfg, max_seqs=4, max_ctx=prompt + 512)
             m.init_synthetic(11, 0.02)
             m.finalize()
             r[name] = time_decoder(m, cfg["vocab"], prompt, (1, 4), steps)
@@ -533,6 +569,8 @@ def run_single_op(args) -> int:
         out = bench_garilix(ctx, args.steps, peak)
     elif args.op == "datasun":
         out = bench_datasun(ctx, args.steps, peak)
+    elif args.op == "gomuzen":
+        out = bench_gomuzen(ctx, args.steps, peak)
     elif args.op == "dense-0p8b":
         out = bench_dense_0p8b(ctx, peak)
     else:
@@ -565,7 +603,7 @@ def main():
     ap.add_argument("--profiler-range", action="store_true",
                     help="bracket the timed 1-stream decode run with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
     ap.add_argument("--no-extras", action="store_true", help="skip the other workloads (single ops, dense model, speculative sweep)")
-    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix", "datasun"],
+    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix", "datasun", "gomuzen"],
                     help="time one operator alone and print its own JSON line (not the benchmark line)")
     args = ap.parse_args()
     if args.warmup < 3:

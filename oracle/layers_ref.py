@@ -296,7 +296,8 @@ def mix_differential(h, P, m, eps, pos, st):
     q = rotate_halves(rms_norm(linear(h, P["q"]).reshape(T, H * 2, d), P["q.norm"], eps), pos, freq, mul).reshape(T, H, 2, d)
     k = rotate_halves(rms_norm(linear(h, P["k"]).reshape(T, G * 2, d), P["k.norm"], eps), pos, freq, mul).reshape(T, G, 2, d)
     k, v = grow(st, k=k, v=linear(h, P["v"]).reshape(T, G, e))
-    a1, a2 = (paged_attention(q[:, :, i], k[:, :, i], v, pos, m["scale"], m.get("softcap")) for i in range(2))
+    mask = m.get("mask") or {}
+    a1, a2 = (paged_attention(q[:, :, i], k[:, :, i], v, pos, m["scale"], m.get("softcap"), mask.get("size"), mask.get("keep_first", 0)) for i in range(2))
     lam = np.exp(np.sum(P["lq1"] * P["lk1"])) - np.exp(np.sum(P["lq2"] * P["lk2"])) + m["diff"]
     o = rms_norm(a1 - lam * a2, 1.0, eps) * (1.0 - m["diff"])
     return linear(o.reshape(T, H * e), P["o"])
