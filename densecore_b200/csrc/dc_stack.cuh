@@ -115,6 +115,27 @@ struct CacheRef {
     }
 };
 
+// One warp: what each of up to DC_MAX_SPLITS key splits, given as (largest score, sum of weights) pairs, counts in their join,
+// times mul.  sink: score of one more term of the denominator (-inf: none).
+__device__ __forceinline__ void join_weights(const float* ml, int splits, int lane, float sink, float mul, float* w) {
+    constexpr int PER = DC_MAX_SPLITS / 32;
+    float m[PER], l[PER], M = sink, L = 0.0f;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int s = lane + 32 * j;
+        const float2 v = s < splits ? *reinterpret_cast<const float2*>(ml + 2 * s) : make_float2(-INFINITY, 0.0f);
+        m[j] = v.x, l[j] = v.y;
+        M = fmaxf(M, m[j]);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+#pragma unroll
+    for (int j = 0; j < PER; ++j) m[j] = expf(m[j] - M), L += l[j] * m[j];
+    L = warp_sum(L) + expf(sink - M);
+#pragma unroll
+    for (int j = 0; j < PER; ++j) w[lane + 32 * j] = m[j] / L * mul;
+}
+
 // ---- copies, fragments and products of the attention and chunk kernels
 __device__ __forceinline__ void unpack16(const uint4& v, float (&f)[8], __nv_bfloat16) {
     const uint32_t u[4] = {v.x, v.y, v.z, v.w};

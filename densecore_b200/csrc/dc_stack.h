@@ -28,6 +28,8 @@ enum { DC_DTYPE_BF16 = 0, DC_DTYPE_F32 = 1 };
 enum { DC_BLOCK_POST_NORM = 0, DC_BLOCK_PARALLEL = 1, DC_BLOCK_PRE_NORM = 2 };
 enum { DC_PAIR_GELU = 0, DC_PAIR_CLAMPED = 1 };
 
+#define DC_MAX_SPLITS 64        // key splits of a decode step's attention
+
 static inline int dc_pad8(int n) { return (n + 7) & ~7; }
 
 // Rows of one or more weight matrices that share their input, bf16, every row padded with zeros to `ld`
@@ -320,7 +322,9 @@ int dc_launch_pre_norm(dc_ctx* ctx, float* x, const float* step, const dc_row_su
                        __nv_bfloat16* outb);
 
 // ---- ffn_moe.cu
-// up to DC_MAX_T tokens: norm of the residual (out / outb), router logits, choices (ids and weights [T][top])
+// norm of the residual (out / outb), router logits, choices (ids and weights [T][top]); where it fits: few tokens, or a bf16
+// model whose width and experts leave room in shared memory
+bool dc_moe_norm_route_fits(const dc_moe_ffn& f, bool b16, int T, int ld);
 int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const float* w, int T, int H, int ld, float eps, float* out,
                              __nv_bfloat16* outb, int32_t* ids, float* weights);
 // choices from logits [T][ldl]

@@ -3,9 +3,9 @@
 // Steps of up to DC_MAX_T tokens: k_moe_norm_route norms the residual and routes it (one cluster per token), k_moe_up_mma
 // streams the gate and up rows of the chosen experts, k_moe_down_mma streams their down rows, every distinct expert once,
 // and adds the sum over experts to the residual.  Hidden values carry the routing weight already, so the down products
-// of a token are one long sum.  Larger steps sort the assignments by expert (k_moe_order), gather the input rows and run
-// grouped tensor-core products (linear_tc.cu); f32 models use k_moe_f32 instead.  The rows of a token are then added up
-// by the norm that follows (norm_act.cu).
+// of a token are one long sum.  Larger steps (k_moe_norm_route_tile) sort the assignments by expert (k_moe_order), gather
+// the input rows and run grouped tensor-core products (linear_tc.cu); f32 models use k_moe_f32 instead.  The rows of a
+// token are then added up by the norm that follows (norm_act.cu).
 #include <algorithm>
 
 #include "dc_common.cuh"
@@ -31,75 +31,79 @@ __device__ __forceinline__ uint32_t ordered(float f) {      // order-preserving,
     return f != f ? 1u : (u & 0x80000000u) ? ~u : (u | 0x80000000u);
 }
 
-// One warp: the choices of a token whose scores are in shared memory.  Equal scores: the lower index first.
-__device__ __forceinline__ void choose(const RouteParams& p, const float* score, int t, int lane) {
-    constexpr int PER = DC_MOE_MAX_EXPERTS / 32;
+// One warp: the choices of a token.  score, correction: shared memory; PER: experts of a lane.  Equal scores: the lower index
+// first.
+template <int PER>
+__device__ __forceinline__ void choose(const RouteParams& p, const float* score, const float* correction, int t, int lane) {
     uint32_t c[PER];             // choice of expert lane + 32 j; 0: not available
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
         const int e = lane + 32 * j;
-        c[j] = e < p.experts ? ordered(score[e] + p.correction[e]) : 0u;
+        c[j] = e < p.experts ? ordered(score[e] + correction[e]) : 0u;
     }
     if (p.keep < p.groups) {
-        const int n = p.experts / p.groups;
-        float mine = -INFINITY;  // lane g: score of group g
-        for (int g = 0; g < p.groups; ++g) {
-            float a = -INFINITY, b = -INFINITY;             // the two best
-            for (int i = lane; i < n; i += 32) {
-                const float v = score[g * n + i] + p.correction[g * n + i];
+        int share = 32;          // lanes of a group
+        while (share * p.groups > 32) share >>= 1;
+        const int n = p.experts / p.groups, g = lane / share;
+        float a = -INFINITY, b = -INFINITY;                 // the group's two best
+        if (g < p.groups)
+            for (int i = lane % share; i < n; i += share) {
+                const float v = score[g * n + i] + correction[g * n + i];
                 b = fmaxf(b, fminf(a, v)), a = fmaxf(a, v);
             }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
-                b = fmaxf(fmaxf(b, ob), fminf(a, oa)), a = fmaxf(a, oa);
-            }
-            if (lane == g) mine = n > 1 ? a + b : a;
+        for (int o = share >> 1; o > 0; o >>= 1) {
+            const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+            b = fmaxf(fmaxf(b, ob), fminf(a, oa)), a = fmaxf(a, oa);
         }
-        uint32_t key = lane < p.groups ? ordered(mine) : 0u, kept = 0u;
+        uint32_t key = g < p.groups && lane % share == 0 ? ordered(n > 1 ? a + b : a) : 0u, kept = 0u;
         for (int k = 0; k < p.keep; ++k) {
             const uint32_t best = __reduce_max_sync(0xffffffffu, key);
-            const int g = __ffs(__ballot_sync(0xffffffffu, key == best)) - 1;
-            kept |= 1u << g;
-            if (lane == g) key = 0u;
+            const int at = __ffs(__ballot_sync(0xffffffffu, key == best)) - 1;
+            kept |= 1u << (at / share);
+            if (lane == at) key = 0u;
         }
 #pragma unroll
         for (int j = 0; j < PER; ++j)
             if (lane + 32 * j < p.experts && !(kept >> ((lane + 32 * j) / n) & 1)) c[j] = 0u;
     }
+    int id = 0;                  // lane k: the k-th choice
     for (int k = 0; k < p.top; ++k) {
         uint32_t best = 0u;
 #pragma unroll
         for (int j = 0; j < PER; ++j) best = max(best, c[j]);
         best = __reduce_max_sync(0xffffffffu, best);
-        int e = DC_MOE_MAX_EXPERTS;
+        int e = p.experts;
 #pragma unroll
         for (int j = PER - 1; j >= 0; --j)
             if (c[j] == best && lane + 32 * j < p.experts) e = lane + 32 * j;
-        e = __reduce_min_sync(0xffffffffu, e);
+        e = min(__reduce_min_sync(0xffffffffu, e), p.experts - 1);
 #pragma unroll
         for (int j = 0; j < PER; ++j)
             if (lane + 32 * j == e) c[j] = 0u;
-        if (lane == 0) {
-            p.ids[(size_t)t * p.top + k] = e;
-            p.weights[(size_t)t * p.top + k] = score[e] * p.scale;
-        }
+        if (lane == k) id = e;
+    }
+    if (lane < p.top) {
+        p.ids[(size_t)t * p.top + lane] = id;
+        p.weights[(size_t)t * p.top + lane] = score[id] * p.scale;
     }
 }
 
 // A warp per token.
+template <int PER>
 __global__ void __launch_bounds__(128) k_moe_route(const RouteParams p, const float* __restrict__ logits, int ldl, int T) {
-    __shared__ float score[4][DC_MOE_MAX_EXPERTS];
+    __shared__ float score[4][32 * PER], correction[32 * PER];
     pdl_launch_dependents();
+    for (int e = threadIdx.x; e < p.experts; e += 128) correction[e] = p.correction[e];
+    __syncthreads();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp;
     if (t >= T) return;
     for (int e = lane; e < p.experts; e += 32) score[warp][e] = sigmoid(logits[(size_t)t * ldl + e]);
     __syncwarp();
-    choose(p, score[warp], t, lane);
+    choose<PER>(p, score[warp], correction, t, lane);
 }
 
-// ---------------------------------------------------------------- norm and choices of few tokens
+// ---------------------------------------------------------------- norm and choices together
 struct NormRouteParams {
     RouteParams r;
     const float *x, *w;
@@ -113,9 +117,10 @@ struct NormRouteParams {
 constexpr int NR_CTAS = 8, NR_WARPS = 8, NR_AHEAD = 4;
 
 // A cluster per token: every CTA norms the row and takes its share of the experts, the first one chooses.
+template <int PER>
 __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRouteParams p) {
     extern __shared__ __align__(16) float h[];              // the normed row, padded with zeros to a multiple of 256
-    __shared__ float red[33], score[DC_MOE_MAX_EXPERTS];
+    __shared__ float red[33], score[32 * PER], correction[32 * PER];
     asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");       // waited for ahead of the first remote store
     pdl_launch_dependents();
     const int rank = blockIdx.x % NR_CTAS, t = blockIdx.x / NR_CTAS, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -130,6 +135,8 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
     for (int i = 0; i < NR_AHEAD; ++i) ahead[i] = fetch(e0 + warp, i);
     for (int e = e0 + warp; e < e1; e += NR_WARPS)          // the rest comes from L2
         for (int k = 64 * lane; k < K8; k += 64 * 32) prefetch_l2(p.router + (size_t)e * p.ldw + k);
+    if (rank == 0)
+        for (int e = tid; e < p.r.experts; e += NR_WARPS * 32) correction[e] = p.r.correction[e];
     pdl_wait();
     const int n4 = p.ld / 4;
     const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)t * p.ld);
@@ -185,17 +192,163 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
     }
     asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
     asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-    if (rank == 0 && warp == 0) choose(p.r, score, t, lane);
+    if (rank == 0 && warp == 0) choose<PER>(p.r, score, correction, t, lane);
+}
+
+// Prompts of bf16 models: sixteen tokens per CTA, a warp norms each; the router product takes the rounded rows (tensor cores,
+// f32 sums), sixteen experts and a share of the columns per warp; then a warp chooses for each token.
+constexpr int NT_WARPS = 16, NT_AHEAD = 4;
+struct TileSizes {
+    int tiles, shares, ldh;      // expert tiles, column shares, pitch of a normed row in shared memory
+    size_t part, score, bytes;   // offsets
+    __host__ __device__ static TileSizes of(int experts, int ld) {
+        TileSizes z;
+        z.tiles = (experts + 15) / 16;
+        z.shares = z.tiles < NT_WARPS ? NT_WARPS / z.tiles : 1;
+        z.ldh = (ld + 63) / 64 * 64 + 32;
+        z.part = (size_t)16 * z.ldh * 2;
+        z.score = z.part + (size_t)z.shares * z.tiles * 16 * 17 * 4;
+        z.bytes = z.score + (size_t)16 * z.tiles * 16 * 4;
+        return z;
+    }
+};
+
+template <int PER>
+__global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const NormRouteParams p, int rows, int T) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    __shared__ float correction[32 * PER];
+    const TileSizes z = TileSizes::of(p.r.experts, p.ld);
+    __nv_bfloat16* h = reinterpret_cast<__nv_bfloat16*>(sm);            // [16][ldh]
+    float* part = reinterpret_cast<float*>(sm + z.part);                // [shares][experts][17]
+    float* score = reinterpret_cast<float*>(sm + z.score);              // [16][experts]
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, t = blockIdx.x * 16 + warp, E = 16 * z.tiles;
+    const int runs = (p.ld + 31) / 32, n4 = p.ld / 4;
+    const int share = warp / z.tiles, per = (runs + z.shares - 1) / z.shares, begin = share * per, end = min(runs, begin + per);
+    uint4 a[NT_AHEAD][2];
+    auto fetch = [&](int j, int tile, int run) {
+        const int k = 32 * run + 8 * q;
+        const bool ok = run < end && k < p.ld;
+        const __nv_bfloat16* w = p.router + (ok ? k : 0);
+        a[j][0] = ok ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)min(16 * tile + g, rows - 1) * p.ldw)) : make_uint4(0, 0, 0, 0);
+        a[j][1] = ok ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)min(16 * tile + 8 + g, rows - 1) * p.ldw)) : make_uint4(0, 0, 0, 0);
+    };
+    const bool working = share < z.shares;
+    if (working)
+#pragma unroll
+        for (int j = 0; j < NT_AHEAD; ++j) fetch(j, warp % z.tiles, begin + j);
+    for (int e = tid; e < p.r.experts; e += NT_WARPS * 32) correction[e] = p.r.correction[e];
+    pdl_wait();
+    {
+        const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld);
+        const float4* w4 = reinterpret_cast<const float4*>(p.w);
+        uint2* to = reinterpret_cast<uint2*>(h + warp * z.ldh);
+        float ss = 0.0f;
+#pragma unroll 8
+        for (int i = lane; i < n4; i += 32) {
+            const float4 v = x4[i];
+            ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        }
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.H + p.eps);
+#pragma unroll 8
+        for (int i = lane; i < (z.ldh - 32) / 4; i += 32) {
+            uint2 v = make_uint2(0u, 0u);
+            if (i < n4) {
+                const float4 x = x4[i], w = w4[i];
+                v = make_uint2(pack_bf2(x.x * inv * w.x, x.y * inv * w.y), pack_bf2(x.z * inv * w.z, x.w * inv * w.w));
+                if (t < T) reinterpret_cast<uint2*>(p.outb + (size_t)t * p.ld)[i] = v;
+            }
+            to[i] = v;
+        }
+    }
+    __syncthreads();
+    for (int tile = warp % z.tiles; working && tile < z.tiles; tile += z.shares > 1 ? z.tiles : NT_WARPS) {
+        float acc[2][4] = {};
+        if (tile != warp % z.tiles)
+#pragma unroll
+            for (int j = 0; j < NT_AHEAD; ++j) fetch(j, tile, begin + j);
+        for (int rb = begin; rb < end; rb += NT_AHEAD) {
+#pragma unroll
+            for (int j = 0; j < NT_AHEAD; ++j) {
+                const int run = rb + j;
+                const uint4 a0 = a[j][0], a1 = a[j][1];
+                fetch(j, tile, run + NT_AHEAD);
+                if (run >= end) continue;
+                const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const uint4 b = *reinterpret_cast<const uint4*>(h + (8 * i + g) * z.ldh + 32 * run + 8 * q);
+                    mma_bf16(acc[i], lo, b.x, b.y);
+                    mma_bf16(acc[i], hi, b.z, b.w);
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) part[(size_t)(share * E + 16 * tile + g + 8 * (j >> 1)) * 17 + 8 * i + 2 * q + (j & 1)] = acc[i][j];
+    }
+    __syncthreads();
+    for (int i = tid; i < 16 * E; i += NT_WARPS * 32) {
+        const int e = i % E, tok = i / E;
+        float v = 0.0f;
+        for (int k = 0; k < z.shares; ++k) v += part[(size_t)(k * E + e) * 17 + tok];
+        score[tok * E + e] = sigmoid(v);
+    }
+    __syncthreads();
+    if (t < T) choose<PER>(p.r, score + warp * E, correction, t, lane);
 }
 
 // ---------------------------------------------------------------- few tokens: weights streamed once
-constexpr int ME_WARPS = 16;     // warps of a CTA; a CTA takes sixteen rows at a time
+constexpr int ME_WARPS = 16;     // warps of a CTA; a CTA takes sixteen rows at a time, column order within a run of 32 as in linear.cu
 
-// Gate and up rows of one assignment's expert for all its tokens: hidden value times routing weight.  Grid: row tiles x
-// assignments; only an expert's first assignment works.  Column order within a run of 32 as in linear.cu.
+// The distinct experts of a step and which of their assignments (-1: none) belongs to which token, in shared memory.
+template <int NT>
+struct Units {
+    static constexpr int CAP = 8 * NT * DC_MOE_MAX_TOP;
+    int16_t expert[CAP], asg[CAP][8 * NT];
+    int first[DC_MOE_MAX_EXPERTS], n;
+
+    __device__ __forceinline__ void clear(int T, int experts) {         // ahead of the dependency wait
+        if (T == 1) return;
+        for (int i = threadIdx.x; i < experts; i += ME_WARPS * 32) first[i] = 1 << 30;
+        for (int i = threadIdx.x; i < CAP * 8 * NT / 2; i += ME_WARPS * 32) reinterpret_cast<uint32_t*>(&asg[0][0])[i] = 0xffffffffu;
+        __syncthreads();
+    }
+    __device__ __forceinline__ void build(const int32_t* ids, int T, int top) {
+        const int tid = threadIdx.x, lane = tid & 31, A = T * top;
+        if (T == 1) {
+            if (tid < A) expert[tid] = (int16_t)ids[tid], asg[tid][0] = (int16_t)tid;
+            if (tid == 0) n = A;
+            __syncthreads();
+            return;
+        }
+        for (int i = tid; i < A; i += ME_WARPS * 32) atomicMin(&first[ids[i]], i);
+        __syncthreads();
+        if (tid < 32) {
+            int count = 0;
+            for (int i0 = 0; i0 < A; i0 += 32) {
+                const int i = i0 + lane, e = i < A ? ids[i] : 0;
+                const bool is = i < A && first[e] == i;
+                const unsigned hit = __ballot_sync(0xffffffffu, is);
+                const int u = count + __popc(hit & ((1u << lane) - 1));
+                if (is) expert[u] = (int16_t)e;
+                __syncwarp();
+                if (is) first[e] = -1 - u;
+                __syncwarp();
+                count += __popc(hit);
+            }
+            if (lane == 0) n = count;
+        }
+        __syncthreads();
+        for (int i = tid; i < A; i += ME_WARPS * 32) asg[-1 - first[ids[i]]][i / top] = (int16_t)i;
+        __syncthreads();
+    }
+};
+
 struct UpParams {
     const __nv_bfloat16* w;
-    int K, ldw, rows, top, T, ff;
+    int K, ldw, rows, top, T, ff, experts;
     float limit;
     const __nv_bfloat16* x;
     int ldx;
@@ -205,83 +358,79 @@ struct UpParams {
     int ldh;
 };
 
+// Gate and up rows of every distinct expert for its tokens: hidden value times routing weight.  A CTA walks over tiles of
+// sixteen rows and fetches the next tile's first runs ahead of a tile's sum.
 template <int NT>
-__global__ void __launch_bounds__(ME_WARPS * 32) k_moe_up_mma(const UpParams p) {
-    constexpr int AHEAD = 4;
-    __shared__ float red[ME_WARPS][16][8 * NT + 1];
-    __shared__ int s_asg[8 * NT], s_n;
+__global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_up_mma(const UpParams p) {
+    constexpr int AHEAD = 2, BUFS = NT > 1 ? 1 : 2;
+    __shared__ float red[BUFS][ME_WARPS][16][8 * NT + 1];
+    __shared__ Units<NT> units;
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, first = blockIdx.y, A = p.T * p.top;
-    const int K8 = (p.K + 7) & ~7, runs = (p.K + 31) / 32;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3;
+    const int K8 = (p.K + 7) & ~7, runs = (p.K + 31) / 32, row_tiles = p.rows / 16;
+    units.clear(p.T, p.experts);
     pdl_wait();
-    const int e = p.ids[first];
-    const __nv_bfloat16* w0 = p.w + ((size_t)e * p.rows + 16 * blockIdx.x + g) * p.ldw + 8 * q;
+    units.build(p.ids, p.T, p.top);
+    const int tiles = units.n * row_tiles;
     uint4 a[AHEAD][2];
-    auto fetch = [&](int j, int run) {
-        const bool ok = run < runs && 32 * run + 8 * q < K8;
-        a[j][0] = ok ? __ldg(reinterpret_cast<const uint4*>(w0 + 32 * run)) : make_uint4(0, 0, 0, 0);
-        a[j][1] = ok ? __ldg(reinterpret_cast<const uint4*>(w0 + (size_t)8 * p.ldw + 32 * run)) : make_uint4(0, 0, 0, 0);
+    auto rows_of = [&](int tile) {          // the lane's first row and column of a tile, null: no more tiles
+        const int u = tile / row_tiles;
+        return tile < tiles ? p.w + ((size_t)units.expert[u] * p.rows + 16 * (tile - u * row_tiles) + g) * p.ldw + 8 * q : nullptr;
     };
-    if (p.T > 1) {               // the expert's assignments (at most one a token), or nothing if an earlier one has it
-        if (warp == 0) {
-            int n = 0;
-            bool mine = true;
-            for (int i0 = 0; i0 < A && mine; i0 += 32) {
-                const int i = i0 + lane;
-                const unsigned hit = __ballot_sync(0xffffffffu, i < A && p.ids[min(i, A - 1)] == e);
-                if (hit && n == 0) mine = i0 + __ffs(hit) - 1 == first;
-                if (hit >> lane & 1) s_asg[n + __popc(hit & ((1u << lane) - 1))] = i;
-                n += __popc(hit);
-            }
-            if (lane == 0) s_n = mine ? n : 0;
-        }
-        __syncthreads();
-        if (!s_n) return;
-    } else if (tid == 0) {
-        s_asg[0] = first, s_n = 1;
-    }
+    auto fetch = [&](int j, const __nv_bfloat16* w, int run) {
+        const bool ok = w && run < runs && 32 * run + 8 * q < K8;
+        a[j][0] = ok ? __ldg(reinterpret_cast<const uint4*>(w + 32 * run)) : make_uint4(0, 0, 0, 0);
+        a[j][1] = ok ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)8 * p.ldw + 32 * run)) : make_uint4(0, 0, 0, 0);
+    };
+    int tile = blockIdx.x;
+    const __nv_bfloat16* w = rows_of(tile);
 #pragma unroll
-    for (int j = 0; j < AHEAD; ++j) fetch(j, warp * AHEAD + j);
-    if (p.T == 1) __syncthreads();
-    const int n = s_n;
-    const __nv_bfloat16* x[NT];
+    for (int j = 0; j < AHEAD; ++j) fetch(j, w, warp * AHEAD + j);
+    for (int buf = 0; tile < tiles; tile += gridDim.x, buf ^= BUFS - 1) {
+        const int u = tile / row_tiles;
+        const __nv_bfloat16* next = rows_of(tile + gridDim.x);
+        const __nv_bfloat16* x[NT];
 #pragma unroll
-    for (int i = 0; i < NT; ++i) x[i] = 8 * i + g < n ? p.x + (size_t)(s_asg[8 * i + g] / p.top) * p.ldx : nullptr;
-    float acc[NT][4];
+        for (int i = 0; i < NT; ++i) x[i] = units.asg[u][8 * i + g] >= 0 && 8 * i + g < p.T ? p.x + (size_t)(8 * i + g) * p.ldx : nullptr;
+        float acc[NT][4];
 #pragma unroll
-    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
-    for (int rb = warp * AHEAD; rb < runs; rb += ME_WARPS * AHEAD) {
+        for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+        for (int rb = warp * AHEAD; rb < runs; rb += ME_WARPS * AHEAD) {
+            const bool last = rb + ME_WARPS * AHEAD >= runs;
 #pragma unroll
-        for (int j = 0; j < AHEAD; ++j) {
-            const int run = rb + j, k = 32 * run + 8 * q;
-            const uint4 a0 = a[j][0], a1 = a[j][1];
-            fetch(j, run + ME_WARPS * AHEAD);
-            if (run >= runs) continue;
-#pragma unroll
-            for (int i = 0; i < NT; ++i) {
-                const uint4 b = x[i] && k < K8 ? *reinterpret_cast<const uint4*>(x[i] + k) : make_uint4(0, 0, 0, 0);
+            for (int j = 0; j < AHEAD; ++j) {
+                const int run = rb + j, k = 32 * run + 8 * q;
+                const uint4 a0 = a[j][0], a1 = a[j][1];
+                fetch(j, last ? next : w, last ? warp * AHEAD + j : run + ME_WARPS * AHEAD);
+                if (run >= runs) continue;
                 const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
-                mma_bf16(acc[i], lo, b.x, b.y);
-                mma_bf16(acc[i], hi, b.z, b.w);
+#pragma unroll
+                for (int i = 0; i < NT; ++i) {
+                    const uint4 b = x[i] && k < K8 ? *reinterpret_cast<const uint4*>(x[i] + k) : make_uint4(0, 0, 0, 0);
+                    mma_bf16(acc[i], lo, b.x, b.y);
+                    mma_bf16(acc[i], hi, b.z, b.w);
+                }
             }
         }
-    }
+        w = next;
+        if (BUFS == 1) __syncthreads();
 #pragma unroll
-    for (int i = 0; i < NT; ++i)
+        for (int i = 0; i < NT; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) red[warp][g + 8 * (j >> 1)][8 * i + 2 * q + (j & 1)] = acc[i][j];
-    __syncthreads();
-    const int r = tid & 15, t = tid >> 4, o = 8 * blockIdx.x + (r >> 1);
-    if (t >= 8 * NT) return;
-    float v = 0.0f;
+            for (int j = 0; j < 4; ++j) red[buf][warp][g + 8 * (j >> 1)][8 * i + 2 * q + (j & 1)] = acc[i][j];
+        __syncthreads();
+        const int r = tid & 15, t = tid >> 4, o = 8 * (tile - u * row_tiles) + (r >> 1);
+        if (tid >= 128 * NT) continue;
+        float v = 0.0f;
 #pragma unroll
-    for (int i = 0; i < ME_WARPS; ++i) v += red[i][r][t];
-    const float up = __shfl_down_sync(0xffffffffu, v, 1);
-    if (!(r & 1) && t < n && o < p.ff) {
-        const int as = s_asg[t];
-        dc_lin_epi epi;
-        epi.pair_kind = DC_PAIR_CLAMPED, epi.limit = p.limit;
-        p.hid[(size_t)as * p.ldh + o] = __float2bfloat16_rn(pair_value(epi, v, up) * p.weights[as]);
+        for (int i = 0; i < ME_WARPS; ++i) v += red[buf][i][r][t];
+        const float up = __shfl_down_sync(0xffffffffu, v, 1);
+        const int as = t < p.T ? units.asg[u][t] : -1;
+        if (!(r & 1) && as >= 0 && o < p.ff) {
+            dc_lin_epi epi;
+            epi.pair_kind = DC_PAIR_CLAMPED, epi.limit = p.limit;
+            p.hid[(size_t)as * p.ldh + o] = __float2bfloat16_rn(pair_value(epi, v, up) * p.weights[as]);
+        }
     }
 }
 
@@ -298,53 +447,24 @@ struct DownParams {
 // x[t] += sum over the token's assignments of W_down hid.  The distinct experts' columns are one long row: a token has
 // zeros where an expert is not its own.  KS: CTAs of a cluster that share sixteen rows, each with its part of that row.
 template <int NT, int KS>
-__global__ void __launch_bounds__(ME_WARPS * 32) k_moe_down_mma(const DownParams p) {
-    constexpr int AHEAD = 2, CAP = 8 * NT * DC_MOE_MAX_TOP;
+__global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_down_mma(const DownParams p) {
+    constexpr int AHEAD = NT > 1 ? 2 : 3;
     __shared__ float red[ME_WARPS][16][8 * NT + 1];
     __shared__ float other[KS > 1 ? KS - 1 : 1][KS > 1 ? 128 * NT : 1];
-    __shared__ int16_t s_expert[CAP], s_asg[CAP][8 * NT];       // distinct experts; their assignment of every token, -1: none
-    __shared__ int s_first[DC_MOE_MAX_EXPERTS], s_n;
+    __shared__ Units<NT> units;
     if (KS > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
     pdl_launch_dependents();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3, part = blockIdx.x % KS, row0 = blockIdx.x / KS * 16;
-    const int A = p.T * p.top, K8 = (p.K + 7) & ~7, per_expert = (p.K + 31) / 32;
-    if (p.T > 1) {
-        for (int i = tid; i < p.experts; i += ME_WARPS * 32) s_first[i] = 1 << 30;
-        for (int i = tid; i < CAP * 8 * NT / 2; i += ME_WARPS * 32) reinterpret_cast<uint32_t*>(&s_asg[0][0])[i] = 0xffffffffu;
-        __syncthreads();
-    }
+    const int K8 = (p.K + 7) & ~7, per_expert = (p.K + 31) / 32;
+    units.clear(p.T, p.experts);
     pdl_wait();
-    if (p.T > 1) {
-        for (int i = tid; i < A; i += ME_WARPS * 32) atomicMin(&s_first[p.ids[i]], i);
-        __syncthreads();
-        if (warp == 0) {
-            int n = 0;
-            for (int i0 = 0; i0 < A; i0 += 32) {
-                const int i = i0 + lane, e = i < A ? p.ids[i] : 0;
-                const bool is = i < A && s_first[e] == i;
-                const unsigned hit = __ballot_sync(0xffffffffu, is);
-                const int u = n + __popc(hit & ((1u << lane) - 1));
-                if (is) s_expert[u] = (int16_t)e;
-                __syncwarp();
-                if (is) s_first[e] = -1 - u;
-                __syncwarp();
-                n += __popc(hit);
-            }
-            if (lane == 0) s_n = n;
-        }
-        __syncthreads();
-        for (int i = tid; i < A; i += ME_WARPS * 32) s_asg[-1 - s_first[p.ids[i]]][i / p.top] = (int16_t)i;
-    } else {
-        if (tid < A) s_expert[tid] = (int16_t)p.ids[tid], s_asg[tid][0] = (int16_t)tid;
-        if (tid == 0) s_n = A;
-    }
-    __syncthreads();
-    const int all = s_n * per_expert, share = (all + KS - 1) / KS, begin = part * share, end = min(all, begin + share);
+    units.build(p.ids, p.T, p.top);
+    const int all = units.n * per_expert, share = (all + KS - 1) / KS, begin = part * share, end = min(all, begin + share);
     uint4 a[AHEAD][2];
     auto fetch = [&](int j, int run) {
         const int u = run / per_expert, k = 32 * (run - u * per_expert) + 8 * q;
         const bool ok = run < end && k < K8;
-        const __nv_bfloat16* w = p.w + ((size_t)s_expert[ok ? u : 0] * p.rows + row0 + g) * p.ldw + (ok ? k : 0);
+        const __nv_bfloat16* w = p.w + ((size_t)units.expert[ok ? u : 0] * p.rows + row0 + g) * p.ldw + (ok ? k : 0);
         a[j][0] = ok ? __ldg(reinterpret_cast<const uint4*>(w)) : make_uint4(0, 0, 0, 0);
         a[j][1] = ok ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)8 * p.ldw)) : make_uint4(0, 0, 0, 0);
     };
@@ -361,11 +481,11 @@ __global__ void __launch_bounds__(ME_WARPS * 32) k_moe_down_mma(const DownParams
             fetch(j, run + ME_WARPS * AHEAD);
             if (run >= end) continue;
             const int u = run / per_expert, k = 32 * (run - u * per_expert) + 8 * q;
+            const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
 #pragma unroll
             for (int i = 0; i < NT; ++i) {
-                const int t = 8 * i + g, as = t < p.T ? s_asg[u][t] : -1;
+                const int t = 8 * i + g, as = t < p.T ? units.asg[u][t] : -1;
                 const uint4 b = as >= 0 && k < K8 ? *reinterpret_cast<const uint4*>(p.hid + (size_t)as * p.ldh + k) : make_uint4(0, 0, 0, 0);
-                const uint32_t lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
                 mma_bf16(acc[i], lo, b.x, b.y);
                 mma_bf16(acc[i], hi, b.z, b.w);
             }
@@ -400,49 +520,63 @@ __global__ void __launch_bounds__(ME_WARPS * 32) k_moe_down_mma(const DownParams
 }
 
 // ---------------------------------------------------------------- many tokens: assignments sorted by expert
-// A CTA per expert: how many assignments go to lower experts, then its own in order.
+// A CTA per expert: how many assignments go to lower experts, then its own.  A warp has a run of assignments and reads 128 of
+// them at a time.
 __global__ void __launch_bounds__(256) k_moe_order(const int32_t* __restrict__ ids, const float* __restrict__ weights, int A, int top, int experts,
                                                    int32_t* __restrict__ off, int32_t* __restrict__ src, float* __restrict__ row_w,
                                                    int32_t* __restrict__ row) {
     __shared__ int s_mine[8], s_below[8];
     pdl_launch_dependents();
     pdl_wait();
-    const int e = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    // a thread's run of assignments
-    const int per = ((A + 255) / 256 + 3) & ~3, i0 = min(A, tid * per), i1 = min(A, i0 + per);
+    const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int per = (A + 1023) / 1024 * 128, begin = min(A, warp * per), end = min(A, begin + per);
+    auto four = [&](int i, int (&v)[4]) {                   // -1 beyond the run
+        if (i + 4 <= end) {
+            const int4 u = *reinterpret_cast<const int4*>(ids + i);
+            v[0] = u.x, v[1] = u.y, v[2] = u.z, v[3] = u.w;
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[j] = i + j < end ? ids[i + j] : -1;
+        }
+    };
     int mine = 0, below = 0;
 #pragma unroll 8
-    for (int i = i0; i < i1; ++i) {
-        const int v = ids[i];
-        mine += v == e;
-        below += v < e;
-    }
-    int before = mine;           // inclusive sum over the warp
+    for (int i = begin + 4 * lane; i < end; i += 128) {
+        int v[4];
+        four(i, v);
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-        const int v = __shfl_up_sync(0xffffffffu, before, o);
-        if (lane >= o) before += v;
+        for (int j = 0; j < 4; ++j) mine += v[j] == e, below += v[j] >= 0 && v[j] < e;
     }
-    below = __reduce_add_sync(0xffffffffu, below);
-    if (lane == 31) s_mine[warp] = before, s_below[warp] = below;
+    mine = __reduce_add_sync(0xffffffffu, mine), below = __reduce_add_sync(0xffffffffu, below);
+    if (lane == 0) s_mine[warp] = mine, s_below[warp] = below;
     __syncthreads();
-    int at = before - mine, total = 0;
+    int at = 0, total = 0;
 #pragma unroll
     for (int w = 0; w < 8; ++w) {
         at += s_below[w] + (w < warp ? s_mine[w] : 0);
         total += s_below[w];
     }
-    if (tid == 0) {
+    if (threadIdx.x == 0) {
         off[e] = total;
         if (e == experts - 1) off[experts] = A;
     }
-    for (int i = i0; i < i1 && mine; ++i)
-        if (ids[i] == e) {
-            src[at] = i / top;
-            row_w[at] = weights[i];
-            row[i] = at;
-            ++at, --mine;
+    if (!mine) return;
+#pragma unroll 4
+    for (int i0 = begin; i0 < end; i0 += 128) {
+        int v[4];
+        four(i0 + 4 * lane, v);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const unsigned hit = __ballot_sync(0xffffffffu, v[j] == e);
+            if (v[j] == e) {
+                const int i = i0 + 4 * lane + j, to = at + __popc(hit & ((1u << lane) - 1));
+                src[to] = i / top;
+                row_w[to] = weights[i];
+                row[i] = to;
+            }
+            at += __popc(hit);
         }
+    }
 }
 
 // out[r] = x[src[r]], rows of ld elements (a multiple of eight); a warp per row
@@ -542,14 +676,35 @@ int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, c
     if (f.experts > DC_MOE_MAX_EXPERTS || f.groups > DC_MOE_MAX_GROUPS || ld % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad operand");
     const NormRouteParams p = {route_params(f, ids, weights), x, w, f.router.w, f.router.ld, H, ld, eps, out, outb};
     const size_t smem = (size_t)(ld + 255) / 256 * 256 * 4;
-    const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route, (int)smem, "k_moe_norm_route");
-    if (st != DC_B200_OK) return st;
-    return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);
+    const TileSizes z = TileSizes::of(f.experts, ld);
+#define DC_ROUTE(PER)                                                                                                                            \
+    do {                                                                                                                                         \
+        if (T > DC_MAX_T) {                                                                                                                      \
+            const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route_tile<PER>, (int)z.bytes, "k_moe_norm_route_tile");                  \
+            if (st != DC_B200_OK) return st;                                                                                                     \
+            return dc_launch(ctx, "k_moe_norm_route_tile", k_moe_norm_route_tile<PER>, dim3((T + 15) / 16), dim3(NT_WARPS * 32), z.bytes, p,      \
+                             f.router.N, T);                                                                                                     \
+        }                                                                                                                                        \
+        const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route<PER>, (int)smem, "k_moe_norm_route");                                   \
+        if (st != DC_B200_OK) return st;                                                                                                         \
+        return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route<PER>, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);       \
+    } while (0)
+    if (f.experts <= 64) DC_ROUTE(2);
+    if (f.experts <= 128) DC_ROUTE(4);
+    if (f.experts <= 256) DC_ROUTE(8);
+    DC_ROUTE(16);
+#undef DC_ROUTE
+}
+
+bool dc_moe_norm_route_fits(const dc_moe_ffn& f, bool b16, int T, int ld) {
+    return T <= DC_MAX_T || (b16 && TileSizes::of(f.experts, ld).bytes <= 200 * 1024);
 }
 
 int dc_launch_moe_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* logits, int ldl, int T, int32_t* ids, float* weights) {
     if (f.experts > DC_MOE_MAX_EXPERTS || f.groups > DC_MOE_MAX_GROUPS) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_route: bad operand");
-    return dc_launch(ctx, "k_moe_route", k_moe_route, dim3((T + 3) / 4), dim3(128), 0, route_params(f, ids, weights), logits, ldl, T);
+    const dim3 grid((T + 3) / 4), block(128);
+    if (f.experts <= 128) return dc_launch(ctx, "k_moe_route", k_moe_route<4>, grid, block, 0, route_params(f, ids, weights), logits, ldl, T);
+    return dc_launch(ctx, "k_moe_route", k_moe_route<16>, grid, block, 0, route_params(f, ids, weights), logits, ldl, T);
 }
 
 int dc_launch_moe_order(dc_ctx* ctx, const dc_moe_ffn& f, const int32_t* ids, const float* weights, int T, int32_t* off, int32_t* src, float* row_w,
@@ -564,8 +719,9 @@ int dc_launch_moe_gather(dc_ctx* ctx, const __nv_bfloat16* x, int ldx, const int
 int dc_launch_moe_up_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* xb, int ldx, int T, const int32_t* ids, const float* weights,
                          __nv_bfloat16* hid, int ldh) {
     if (T < 1 || T > DC_MAX_T || ldx % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_up: bad operand");
-    const UpParams p = {f.up.w, f.up.K, f.up.ld, f.up_rows, f.top, T, f.ff, f.limit, xb, ldx, ids, weights, hid, ldh};
-    const dim3 grid(f.up_rows / 16, T * f.top), block(ME_WARPS * 32);
+    const UpParams p = {f.up.w, f.up.K, f.up.ld, f.up_rows, f.top, T, f.ff, f.experts, f.limit, xb, ldx, ids, weights, hid, ldh};
+    const int tiles = f.up_rows / 16 * std::min(f.experts, T * f.top), room = 2 * ctx->num_sms, rounds = (tiles + room - 1) / room;
+    const dim3 grid(T == 1 ? (tiles + rounds - 1) / rounds : std::min(tiles, room)), block(ME_WARPS * 32);
     if (T <= 8) return dc_launch(ctx, "k_moe_up_mma", k_moe_up_mma<1>, grid, block, 0, p);
     return dc_launch(ctx, "k_moe_up_mma", k_moe_up_mma<2>, grid, block, 0, p);
 }

@@ -171,6 +171,90 @@ __global__ void __launch_bounds__(256) k_gqa_prep_heads(const HeadsParams p) {
     }
 }
 
+__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w)); }
+
+// The same four dimensions at a time, for sizes that are multiples of four: a warp has U heads of a token in flight, a lane the
+// dimensions 4 lane .. 4 lane + 3 (and, with NV 2, those 128 further on).
+template <typename TC, int NV, int U>
+__global__ void __launch_bounds__(256) k_gqa_prep_heads4(const HeadsParams p) {
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31, u0 = blockIdx.y * 8 * U + (threadIdx.x >> 5), units = p.nq + p.nk + p.nv, half = p.rot / 2;
+    pdl_wait();
+    const int t = blockIdx.x, pos = min(max(p.positions[t], 0), p.max_pos - 1);
+    const float* row = p.proj + (size_t)t * p.ldp;
+    const float* cs = p.cos_sin + (size_t)pos * p.rot;
+    float4 v[U][NV], mate[U][NV];
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+        const int u = u0 + 8 * i;
+        const bool query = u < p.nq, value = u >= p.nq + p.nk;
+        const int head = query ? u : value ? u - p.nq - p.nk : u - p.nq, n = value ? p.vdim : p.dim;
+        const float* x = row + (query ? p.off_q : value ? p.off_v : p.off_k) + head * n;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int d = 4 * lane + 128 * j;
+            v[i][j] = u < units && d < n ? *reinterpret_cast<const float4*>(x + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+            mate[i][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (u < units && !value && p.halves && d < p.rot) mate[i][j] = *reinterpret_cast<const float4*>(x + (d < half ? d + half : d - half));
+        }
+    }
+    TC* cache = reinterpret_cast<TC*>(p.c.arena) + p.c.at(p.seq_ids[t], pos);
+    float4 c[NV], s[NV];         // of the lane's dimensions; the sine has the sign of the mate's share
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int d = 4 * lane + 128 * j;
+        c[j] = make_float4(1.f, 1.f, 1.f, 1.f), s[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d >= p.rot) continue;
+        if (p.halves) {
+            const bool first = d < half;
+            const float4* at = reinterpret_cast<const float4*>(cs + 2 * (first ? d : d - half));
+            const float4 a = at[0], b = at[1];
+            const float sign = first ? -1.0f : 1.0f;
+            c[j] = make_float4(a.x, a.z, b.x, b.z), s[j] = make_float4(sign * a.y, sign * a.w, sign * b.y, sign * b.w);
+        } else {
+            const float4 a = *reinterpret_cast<const float4*>(cs + d);
+            c[j] = make_float4(a.x, a.x, a.z, a.z), s[j] = make_float4(-a.y, a.y, -a.w, a.w);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+        const int u = u0 + 8 * i;
+        if (u >= units) break;
+        const bool query = u < p.nq, value = u >= p.nq + p.nk;
+        const int head = query ? u : value ? u - p.nq - p.nk : u - p.nq, pitch = query ? p.ldq : value ? p.vdim_p : p.dim_p;
+        const float* w = value ? nullptr : query ? p.q_norm : p.k_norm;
+        float inv = 1.0f;
+        if (w) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int j = 0; j < NV; ++j) ss += (v[i][j].x * v[i][j].x + v[i][j].y * v[i][j].y) + (v[i][j].z * v[i][j].z + v[i][j].w * v[i][j].w);
+            inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int d = 4 * lane + 128 * j;
+            if (d >= pitch) break;
+            float4 a = v[i][j], b = mate[i][j];
+            if (w && d < p.dim) {
+                const float4 f = *reinterpret_cast<const float4*>(w + d);
+                a = make_float4(a.x * f.x, a.y * f.y, a.z * f.z, a.w * f.w);
+                if (p.halves && d < p.rot) {
+                    const float4 m = *reinterpret_cast<const float4*>(w + (d < half ? d + half : d - half));
+                    b = make_float4(b.x * m.x, b.y * m.y, b.z * m.z, b.w * m.w);
+                }
+            }
+            if (!p.halves) b = make_float4(a.y, a.x, a.w, a.z);
+            const float4 r = value ? a : make_float4((a.x * c[j].x + b.x * s[j].x) * inv, (a.y * c[j].y + b.y * s[j].y) * inv,
+                                                     (a.z * c[j].z + b.z * s[j].z) * inv, (a.w * c[j].w + b.w * s[j].w) * inv);
+            const size_t at = ((size_t)t * p.nq + head) * pitch + d;
+            if (!query) store_four(cache + (value ? p.v_at : 0) + head * pitch + d, r);
+            else if (p.qb) store_four(p.qb + at, r);
+            else store_four(p.q + at, r);
+        }
+    }
+}
+
 // ---------------------------------------------------------------- every token alone
 // The keys that a token sees, in order: the kept first ones that its window has left behind, then the window.
 struct Keys {
@@ -290,20 +374,12 @@ template <int MAPS>
 __global__ void __launch_bounds__(128) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int vdim,
                                                   float sink, float lambda, float mul, float eps, float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb,
                                                   int ldm) {
-    __shared__ float sw[MAPS][32], red[33];
+    __shared__ float sw[MAPS][DC_MAX_SPLITS], red[33];
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t o = ((size_t)t * heads + h) * MAPS * splits;
-    if (warp < MAPS) {                  // splits <= 32
-        const size_t at = o + warp * splits + lane;
-        const float m = lane < splits ? part_ml[2 * at] : -INFINITY, l = lane < splits ? part_ml[2 * at + 1] : 0.0f;
-        float M = fmaxf(m, sink);
-#pragma unroll
-        for (int k = 16; k > 0; k >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, k));
-        const float w = expf(m - M), L = warp_sum(l * w) + expf(sink - M);
-        sw[warp][lane] = w / L * (warp ? -lambda : 1.0f);
-    }
+    if (warp < MAPS) join_weights(part_ml + 2 * (o + warp * splits), splits, lane, sink, warp ? -lambda : 1.0f, sw[warp]);
     __syncthreads();
     float v[2] = {0.0f, 0.0f}, ss = 0.0f;         // vdim <= 256
 #pragma unroll
@@ -598,11 +674,21 @@ int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, co
         if (m.off_v == m.off_k) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prep: values from the keys need the norm over all heads");
         HeadsParams p = {proj, ldp, m.off_q, m.off_k, m.off_v, m.heads * m.maps, m.kv_heads * m.maps, m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at,
                          dc_gqa_ldq(m), m.rot.dims, m.halves, max_pos, m.q_norm, m.k_norm, m.cos_sin, eps, st.seq_ids, st.positions, cache_ref(c, m.row), q, qb};
-        const dim3 grid(st.T, (p.nq + p.nk + p.nv + 7) / 8), block(256);
+        const int units = p.nq + p.nk + p.nv, most = std::max(std::max(p.ldq, p.dim_p), p.vdim_p);
+        const dim3 grid(st.T, (units + 7) / 8), block(256);
+        if (m.dim % 4 == 0 && m.vdim % 4 == 0 && m.rot.dims % (m.halves ? 8 : 4) == 0 && ldp % 4 == 0) {
+#define DC_HEADS4(TC, NV)                                                                                                                                    \
+    return st.T > DC_MAX_T ? dc_launch(ctx, "k_gqa_prep_heads4", k_gqa_prep_heads4<TC, NV, 3>, dim3(st.T, (units + 23) / 24), block, 0, p)                    \
+                           : dc_launch(ctx, "k_gqa_prep_heads4", k_gqa_prep_heads4<TC, NV, 1>, grid, block, 0, p)
+            if (c.f32 && most <= 128) DC_HEADS4(float, 1);
+            if (c.f32) DC_HEADS4(float, 2);
+            if (most <= 128) DC_HEADS4(__nv_bfloat16, 1);
+            DC_HEADS4(__nv_bfloat16, 2);
+#undef DC_HEADS4
+        }
 #define DC_HEADS(VP)                                                                                                          \
     return c.f32 ? dc_launch(ctx, "k_gqa_prep_heads", k_gqa_prep_heads<float, VP>, grid, block, 0, p)                          \
                  : dc_launch(ctx, "k_gqa_prep_heads", k_gqa_prep_heads<__nv_bfloat16, VP>, grid, block, 0, p)
-        const int most = std::max(std::max(p.ldq, p.dim_p), p.vdim_p);
         if (most <= 64) DC_HEADS(2);
         if (most <= 128) DC_HEADS(4);
         DC_HEADS(8);

@@ -244,7 +244,7 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
                                                     const float* __restrict__ gate, int ldg,
                                                     float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
     extern __shared__ __align__(16) float lat[];      // [rank padded to 8]
-    __shared__ float sw[32];
+    __shared__ float sw[DC_MAX_SPLITS];
     pdl_launch_dependents();
     const int h = blockIdx.x, t = blockIdx.y, e0 = blockIdx.z * OUT_ROWS, e1 = min(vdim, e0 + OUT_ROWS), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const char* rows = reinterpret_cast<const char*>(uv + (size_t)(h * vdim_p + e0) * ldw);
@@ -252,14 +252,7 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
     pdl_wait();
     const size_t o = ((size_t)t * heads + h) * splits;
     const float mul = gate ? sigmoid(gate[(size_t)t * ldg + h]) : 1.0f;
-    if (warp == 0) {             // splits <= 32
-        const float m = lane < splits ? part_ml[2 * (o + lane)] : -INFINITY, l = lane < splits ? part_ml[2 * (o + lane) + 1] : 0.0f;
-        float M = m;
-#pragma unroll
-        for (int k = 16; k > 0; k >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, k));
-        const float w = expf(m - M), L = warp_sum(l * w);
-        sw[lane] = w / L;
-    }
+    if (warp == 0) join_weights(part_ml + 2 * o, splits, lane, -INFINITY, 1.0f, sw);
     __syncthreads();
     const int rank8 = (rank + 7) & ~7;
     for (int r = threadIdx.x; r < rank8; r += 256) {

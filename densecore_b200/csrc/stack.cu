@@ -249,7 +249,7 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
         }
     }
     // key splits of a decode step: about 32 keys each at the longest span
-    s->splits = std::max(1, std::min(32, (span + 31) / 32));
+    s->splits = std::max(1, std::min(DC_MAX_SPLITS, (span + 31) / 32));
     const int per_seq = (c.max_ctx + DC_KV_BLOCK - 1) / DC_KV_BLOCK;
     const int blocks = pool_tokens > 0 ? (pool_tokens + DC_KV_BLOCK - 1) / DC_KV_BLOCK : per_seq * c.max_seqs;
     return dc_kv_init_planes(ctx, &m->kv, planes, state, blocks, c.max_seqs, per_seq);
@@ -582,7 +582,7 @@ int moe_layer(dc_model* m, const dc_step& st, dc_stack_layer& Ly, dc_row_sum* ow
     __nv_bfloat16* xb = st.b16 ? b.xb : nullptr;
     const double up_bytes = (double)f.up_rows * f.up.ld * 2, down_bytes = (double)f.down_rows * f.down.ld * 2;
     const double touched = std::min<double>(f.experts, rows);
-    if (T <= DC_MAX_T) {
+    if (dc_moe_norm_route_fits(f, st.b16, T, H)) {
         L(DC_K_ROUTER, lin_bytes(f.router, T), 1, dc_launch_moe_norm_route(ctx, f, b.x, Ly.norm2, T, W, H, s->cfg.eps, b.y, xb, b.moe_ids, b.moe_w));
     } else {
         L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, b.y, xb, H));
