@@ -243,23 +243,30 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
         const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld);
         const float4* w4 = reinterpret_cast<const float4*>(p.w);
         uint2* to = reinterpret_cast<uint2*>(h + warp * z.ldh);
+        constexpr int KEEP = 16;             // groups of four that a lane holds; wider rows are read twice
+        float4 x[KEEP];
         float ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) x[j] = lane + 32 * j < n4 ? x4[lane + 32 * j] : make_float4(0.f, 0.f, 0.f, 0.f);
+        auto square = [&](const float4& v) { ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); };
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) square(x[j]);
 #pragma unroll 8
-        for (int i = lane; i < n4; i += 32) {
-            const float4 v = x4[i];
-            ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
-        }
+        for (int i = lane + 32 * KEEP; i < n4; i += 32) square(x4[i]);
         const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.H + p.eps);
-#pragma unroll 8
-        for (int i = lane; i < (z.ldh - 32) / 4; i += 32) {
-            uint2 v = make_uint2(0u, 0u);
+        auto put = [&](int i, const float4& v) {
+            uint2 r = make_uint2(0u, 0u);
             if (i < n4) {
-                const float4 x = x4[i], w = w4[i];
-                v = make_uint2(pack_bf2(x.x * inv * w.x, x.y * inv * w.y), pack_bf2(x.z * inv * w.z, x.w * inv * w.w));
-                if (t < T) reinterpret_cast<uint2*>(p.outb + (size_t)t * p.ld)[i] = v;
+                const float4 w = w4[i];
+                r = make_uint2(pack_bf2(v.x * inv * w.x, v.y * inv * w.y), pack_bf2(v.z * inv * w.z, v.w * inv * w.w));
+                if (t < T) reinterpret_cast<uint2*>(p.outb + (size_t)t * p.ld)[i] = r;
             }
-            to[i] = v;
-        }
+            if (i < (z.ldh - 32) / 4) to[i] = r;
+        };
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) put(lane + 32 * j, x[j]);
+#pragma unroll 8
+        for (int i = lane + 32 * KEEP; i < (z.ldh - 32) / 4; i += 32) put(i, i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f));
     }
     __syncthreads();
     for (int tile = warp % z.tiles; working && tile < z.tiles; tile += z.shares > 1 ? z.tiles : NT_WARPS) {
@@ -523,8 +530,7 @@ __global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_down_mma(const DownPar
 // A CTA per expert: how many assignments go to lower experts, then its own.  A warp has a run of assignments and reads 128 of
 // them at a time.
 __global__ void __launch_bounds__(256) k_moe_order(const int32_t* __restrict__ ids, const float* __restrict__ weights, int A, int top, int experts,
-                                                   int32_t* __restrict__ off, int32_t* __restrict__ src, float* __restrict__ row_w,
-                                                   int32_t* __restrict__ row) {
+                                                   int32_t* __restrict__ off, int32_t* src, float* __restrict__ row_w, int32_t* __restrict__ row) {
     __shared__ int s_mine[8], s_below[8];
     pdl_launch_dependents();
     pdl_wait();
@@ -539,43 +545,49 @@ __global__ void __launch_bounds__(256) k_moe_order(const int32_t* __restrict__ i
             for (int j = 0; j < 4; ++j) v[j] = i + j < end ? ids[i + j] : -1;
         }
     };
+    constexpr int B = 8;         // loads in flight
     int mine = 0, below = 0;
-#pragma unroll 8
-    for (int i = begin + 4 * lane; i < end; i += 128) {
-        int v[4];
-        four(i, v);
+    for (int i0 = begin; i0 < end; i0 += 128 * B) {
+        int v[B][4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) mine += v[j] == e, below += v[j] >= 0 && v[j] < e;
+        for (int k = 0; k < B; ++k) four(i0 + 128 * k + 4 * lane, v[k]);
+#pragma unroll
+        for (int k = 0; k < B; ++k)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) mine += v[k][j] == e, below += v[k][j] >= 0 && v[k][j] < e;
     }
     mine = __reduce_add_sync(0xffffffffu, mine), below = __reduce_add_sync(0xffffffffu, below);
     if (lane == 0) s_mine[warp] = mine, s_below[warp] = below;
     __syncthreads();
-    int at = 0, total = 0;
+    int at = 0, total = 0, own = 0;
 #pragma unroll
     for (int w = 0; w < 8; ++w) {
         at += s_below[w] + (w < warp ? s_mine[w] : 0);
-        total += s_below[w];
+        total += s_below[w], own += s_mine[w];
     }
     if (threadIdx.x == 0) {
         off[e] = total;
         if (e == experts - 1) off[experts] = A;
     }
-    if (!mine) return;
-#pragma unroll 4
-    for (int i0 = begin; i0 < end; i0 += 128) {
-        int v[4];
-        four(i0 + 4 * lane, v);
+    for (int i0 = begin; i0 < end && mine; i0 += 128 * B) {
+        int v[B][4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const unsigned hit = __ballot_sync(0xffffffffu, v[j] == e);
-            if (v[j] == e) {
-                const int i = i0 + 4 * lane + j, to = at + __popc(hit & ((1u << lane) - 1));
-                src[to] = i / top;
-                row_w[to] = weights[i];
-                row[i] = to;
+        for (int k = 0; k < B; ++k) four(i0 + 128 * k + 4 * lane, v[k]);
+#pragma unroll
+        for (int k = 0; k < B; ++k)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const unsigned hit = __ballot_sync(0xffffffffu, v[k][j] == e);
+                if (v[k][j] == e) src[at + __popc(hit & ((1u << lane) - 1))] = i0 + 128 * k + 4 * lane + j;
+                at += __popc(hit);
             }
-            at += __popc(hit);
-        }
+    }
+    __syncthreads();
+    for (int r = total + threadIdx.x; r < total + own; r += 256) {       // the assignments are listed: rows side by side
+        const int i = src[r];
+        src[r] = i / top;
+        row_w[r] = weights[i];
+        row[i] = r;
     }
 }
 

@@ -6,12 +6,14 @@
 // a warp's stores of one token are 32 consecutive outputs.  Two CTAs share an SM: one's read-out overlaps the
 // other's products.  Large products use tiles of 128 x 256 instead (k_linear_tc_wide): one CTA per SM walks its share
 // of them, with two sets of accumulators, so that the loads and products of a tile run while the tile before is read
-// out; the wider tile reads shared memory less often per product.  Its grouped form multiplies runs of sorted tokens with
+// out by eight warps; the wider tile reads shared memory less often per product.  Its grouped form multiplies runs of sorted tokens with
 // a matrix of their own each (experts); the runs' ends are device data, so every CTA lists the tiles itself, and a tile
 // of few tokens takes narrower products.  All let the next kernel start only after every
 // CTA has its tensor memory.  Columns beyond K and rows beyond the matrix are the zeros that TMA fills in.  Every wait is
 // bounded; a CTA that gives up drains its copies, frees its tensor memory and leaves.
 #include <algorithm>
+#include <mutex>
+#include <set>
 
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
@@ -47,6 +49,7 @@ template <int COLS, typename F>
 __device__ __forceinline__ void each16(uint32_t tmem, int n, F f) {
     int v[2][16];
     tmem_ld16(tmem, v[0]);
+#pragma unroll 1
     for (int c0 = 0; c0 < COLS && c0 < n; c0 += 32) {
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -59,35 +62,68 @@ __device__ __forceinline__ void each16(uint32_t tmem, int n, F f) {
     }
 }
 
-// Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.
-template <int COLS>
+// Eight lanes (xor 1, 2, 4 times STEP) hold one row each, N pairs of tokens packed as bf16; afterwards a lane holds N / 4 tokens,
+// eight rows each in a row of four registers.  Token of set k: 2 (N / 2 b1 + N / 4 b2 + k) + b0, b: the lane's bits.
+template <int STEP, int N>
+__device__ __forceinline__ void transpose8(const uint32_t (&r)[N], uint32_t (&out)[N / 4][4], int lane) {
+    const bool b0 = lane & STEP, b1 = lane & 2 * STEP, b2 = lane & 4 * STEP;
+    const uint32_t give = b0 ? 0x5410u : 0x7632u, mine0 = b0 ? 0x3254u : 0x5410u, mine1 = b0 ? 0x3276u : 0x7610u;
+    uint32_t a[N];
+#pragma unroll
+    for (int j = 0; j < N; j += 2) {
+        const uint32_t got = __shfl_xor_sync(0xffffffffu, __byte_perm(r[j], r[j + 1], give), STEP);
+        a[j] = __byte_perm(r[j], got, mine0);
+        a[j + 1] = __byte_perm(r[j + 1], got, mine1);
+    }
+    uint32_t b[N / 2][2];
+#pragma unroll
+    for (int j = 0; j < N / 2; ++j) {
+        const uint32_t got = __shfl_xor_sync(0xffffffffu, b1 ? a[j] : a[j + N / 2], 2 * STEP), own = b1 ? a[j + N / 2] : a[j];
+        b[j][0] = b1 ? got : own, b[j][1] = b1 ? own : got;
+    }
+#pragma unroll
+    for (int j = 0; j < N / 4; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const uint32_t got = __shfl_xor_sync(0xffffffffu, b2 ? b[j][i] : b[j + N / 4][i], 4 * STEP), own = b2 ? b[j + N / 4][i] : b[j][i];
+            out[j][i] = b2 ? got : own, out[j][2 + i] = b2 ? own : got;
+        }
+}
+
+// Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.  Grouped
+// products end in clamped pairs with a factor per token or in bf16 rows.
+template <int COLS, bool GROUPED>
 __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int t1, int quarter, int lane) {
     const int row = row0 + 32 * quarter + lane, n = t1 - t0;
     const dc_lin_epi& e = p.e;
     tmem += (uint32_t)(32 * quarter) << 16;
     if (row0 + 32 * quarter >= e.pair0) {
         // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
-        const bool up = lane & 1, gelu = e.pair_kind == DC_PAIR_GELU;
+        const bool up = lane & 1, gelu = !GROUPED && e.pair_kind == DC_PAIR_GELU;
         const int o = (row - e.pair0) >> 1, first = up ? 8 : 0;
         const bool in = o < e.n_pairs;
         const size_t at = (size_t)(t0 + first) * e.ldp + o;
+        const bool wide = e.poutb && e.n_pairs % 8 == 0 && e.ldp % 8 == 0 && ((uintptr_t)e.poutb & 15) == 0;     // whole groups of eight outputs
         each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
-            float h[8];
+            float h[8], f[8];        // factors: asked for ahead of the arithmetic
+#pragma unroll
+            for (int i = 0; i < 8; ++i) f[i] = GROUPED ? e.tok_scale[min(t0 + c0 + first + i, t1 - 1)] : 1.0f;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
                 const float mine = __int_as_float(up ? v[i + 8] : v[i]);
                 const float gate = up ? got : mine, val = up ? mine : got;
-                h[i] = gelu ? gelu_tanh(gate) * val : quick_clamped(e.limit, gate, val);
+                h[i] = (gelu ? gelu_tanh(gate) * val : quick_clamped(e.limit, gate, val)) * f[i];
             }
             const int m = in ? n - c0 - first : 0;
-            if (e.tok_scale) {
-                const float* f = e.tok_scale + t0 + c0 + first;
+            if (wide) {
+                uint32_t r[4], v8[1][4];
 #pragma unroll
-                for (int i = 0; i < 8; ++i)
-                    if (i < m) h[i] *= f[i];
-            }
-            if (e.poutb) {
+                for (int i = 0; i < 4; ++i) r[i] = pack_bf2(h[2 * i], h[2 * i + 1]);
+                transpose8<2, 4>(r, v8, lane);
+                const int tok = 2 * ((lane & 4 ? 2 : 0) + (lane & 8 ? 1 : 0)) + (lane & 2 ? 1 : 0);
+                if (tok < m) *reinterpret_cast<uint4*>(e.poutb + at + (size_t)(c0 + tok) * e.ldp - ((lane >> 1) & 7)) = make_uint4(v8[0][0], v8[0][1], v8[0][2], v8[0][3]);
+            } else if (GROUPED || e.poutb) {
                 __nv_bfloat16* to = e.poutb + at + (size_t)c0 * e.ldp;
 #pragma unroll
                 for (int i = 0; i < 8; ++i, to += e.ldp)
@@ -102,10 +138,27 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
         return;
     }
     const bool in = row < e.n_store;
-    const float bias = in && e.bias ? e.bias[row] : 0.0f;
+    const float bias = !GROUPED && in && e.bias ? e.bias[row] : 0.0f;
     const size_t at = (size_t)t0 * e.ldo + row;
-    if (e.outb) {
-        const bool act = row < e.silu_rows;
+    if (e.outb && e.n_store % 8 == 0 && e.ldo % 8 == 0 && ((uintptr_t)e.outb & 15) == 0) {       // whole groups of eight rows
+        const bool act = !GROUPED && row < e.silu_rows;
+        const int tok = 2 * ((lane & 2 ? 4 : 0) + (lane & 4 ? 2 : 0)) + (lane & 1);
+        each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
+            uint32_t r[8], v8[2][4];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float a = __int_as_float(v[2 * i]) + bias, b = __int_as_float(v[2 * i + 1]) + bias;
+                r[i] = act ? pack_bf2(quick_silu(a), quick_silu(b)) : pack_bf2(a, b);
+            }
+            transpose8<1, 8>(r, v8, lane);
+            const int m = in ? n - c0 : 0;
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                if (tok + 2 * i < m)
+                    *reinterpret_cast<uint4*>(e.outb + at + (size_t)(c0 + tok + 2 * i) * e.ldo - (lane & 7)) = make_uint4(v8[i][0], v8[i][1], v8[i][2], v8[i][3]);
+        });
+    } else if (GROUPED || e.outb) {
+        const bool act = !GROUPED && row < e.silu_rows;
         each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
             const int m = in ? n - c0 : 0;
             __nv_bfloat16* to = e.outb + at + (size_t)c0 * e.ldo;
@@ -119,12 +172,17 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
         each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
             const int m = in ? n - c0 : 0;
             float* to = e.out + at + (size_t)c0 * e.ldo;
-            float old[16];
 #pragma unroll
-            for (int i = 0; i < 16; ++i) old[i] = i < m ? to[(size_t)i * e.ldo] : 0.0f;         // every load ahead of the stores
+            for (int i0 = 0; i0 < 16; i0 += 8, to += 8 * (size_t)e.ldo) {
+                float old[8];
+                float* at8 = to;
 #pragma unroll
-            for (int i = 0; i < 16; ++i, to += e.ldo)
-                if (i < m) *to = old[i] + (__int_as_float(v[i]) + bias);
+                for (int i = 0; i < 8; ++i, at8 += e.ldo) old[i] = i0 + i < m ? *at8 : 0.0f;          // loads ahead of the stores
+                at8 = to;
+#pragma unroll
+                for (int i = 0; i < 8; ++i, at8 += e.ldo)
+                    if (i0 + i < m) *at8 = old[i] + (__int_as_float(v[i0 + i]) + bias);
+            }
         });
     } else {
         each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
@@ -202,7 +260,7 @@ __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_consta
     } else {
         const bool ok = tc_wait_raw(acc, 0, give_up, p.err) && !*give_up;
         tc_fence_after();
-        if (__all_sync(0xffffffffu, ok)) read_out<128>(p, tmem, row0, t0, p.T, warp & 3, lane);
+        if (__all_sync(0xffffffffu, ok)) read_out<128, false>(p, tmem, row0, t0, p.T, warp & 3, lane);
     }
     tc_fence_before();
     __syncthreads();
@@ -212,6 +270,7 @@ __global__ void __launch_bounds__(LT_THREADS, 2) k_linear_tc(const __grid_consta
 
 // ---- 128 x 256 tiles, one CTA per SM over its share of them
 constexpr int LW_STAGES = 4, LW_STAGE = 3 * LT_TILE;       // 128 weight rows and 256 token rows of 64 columns
+constexpr int LW_READERS = 2, LW_THREADS = 64 + 128 * LW_READERS;     // warps of a quarter's lanes share its columns
 constexpr size_t LW_SMEM = (size_t)LW_STAGES * LW_STAGE + 1024;
 
 struct LwTiles {
@@ -221,7 +280,7 @@ struct LwTiles {
 };
 
 template <bool GROUPED>
-__global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_constant__ CUtensorMap wmap,
+__global__ void __launch_bounds__(LW_THREADS, 1) k_linear_tc_wide(const __grid_constant__ CUtensorMap wmap,
                                                                   const __grid_constant__ CUtensorMap xmap, const LtParams p, const LwTiles tl) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t s_bar[2 * LW_STAGES + 4];
@@ -245,7 +304,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_c
         }
         for (int i = 0; i < 2; ++i) {
             mbar_init(acc_full + 8 * i, 1);
-            mbar_init(acc_free + 8 * i, 128);
+            mbar_init(acc_free + 8 * i, 128 * LW_READERS);
         }
         mbar_fence_init();
     }
@@ -351,7 +410,8 @@ __global__ void __launch_bounds__(LT_THREADS, 1) k_linear_tc_wide(const __grid_c
             tc_fence_after();
             if (!__all_sync(0xffffffffu, ok)) break;
             const Place at = place(tile, group);
-            read_out<256>(p, tmem + 256 * set, at.row0, at.t0, at.t1, warp & 3, lane);
+            const int per = (at.cols() + 16 * LW_READERS - 1) / (16 * LW_READERS) * 16, c0 = (warp - 2) / 4 * per;
+            if (c0 < at.cols()) read_out<256 / LW_READERS, GROUPED>(p, tmem + 256 * set + c0, at.row0, at.t0 + c0, min(at.t1, at.t0 + c0 + per), warp & 3, lane);
             tc_fence_before();
             mbar_arrive(acc_free + 8 * set);
         }
@@ -377,6 +437,24 @@ EncodeFn encode_fn() {
 
 }  // namespace
 
+// Loads from tensor memory land in their registers some time after the instruction; each16 uses others meanwhile.  A build that
+// spills could store such a register too early and give it another use, which the load then overwrites: it may not run.
+static int setup_unspilled(dc_ctx* ctx, const void* f, int smem, const char* name) {
+    static std::mutex mu;
+    static std::set<const void*> good;
+    {
+        std::lock_guard<std::mutex> lk(mu);
+        if (!good.count(f)) {
+            cudaFuncAttributes a;
+            const int st = dc_check_cuda(ctx, cudaFuncGetAttributes(&a, f), name);
+            if (st != DC_B200_OK) return st;
+            if (a.localSizeBytes) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "%s was built with %d bytes of spilled registers", name, (int)a.localSizeBytes);
+            good.insert(f);
+        }
+    }
+    return dc_kernel_setup(ctx, f, smem, name);
+}
+
 // Tensor map of a bf16 matrix [rows][ld] whose first K columns count: boxes of 128 rows x 64 columns.
 int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int rows, int K, int ld) {
     EncodeFn f = encode_fn();
@@ -396,13 +474,13 @@ int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, 
     p.e.n_pairs = std::max(0, std::min(epi.n_pairs, (w.N - epi.pair0) / 2));
     const int row_tiles = (w.N + 127) / 128, tok_tiles = (T + 255) / 256, tiles = row_tiles * tok_tiles;
     if (T > 128 && tiles >= ctx->num_sms / 2) {
-        int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide<false>, (int)LW_SMEM, "k_linear_tc_wide");
+        int st = setup_unspilled(ctx, (const void*)k_linear_tc_wide<false>, (int)LW_SMEM, "k_linear_tc_wide");
         if (st != DC_B200_OK) return st;
         const LwTiles tl = {row_tiles, tok_tiles, 0, 0, nullptr};
-        return dc_launch(ctx, "k_linear_tc_wide", k_linear_tc_wide<false>, dim3(tiles < ctx->num_sms ? tiles : ctx->num_sms), dim3(LT_THREADS), LW_SMEM,
+        return dc_launch(ctx, "k_linear_tc_wide", k_linear_tc_wide<false>, dim3(tiles < ctx->num_sms ? tiles : ctx->num_sms), dim3(LW_THREADS), LW_SMEM,
                          w.map, x.map, p, tl);
     }
-    int st = dc_kernel_setup(ctx, (const void*)k_linear_tc, (int)LT_SMEM, "k_linear_tc");
+    int st = setup_unspilled(ctx, (const void*)k_linear_tc, (int)LT_SMEM, "k_linear_tc");
     if (st != DC_B200_OK) return st;
     return dc_launch(ctx, "k_linear_tc", k_linear_tc, dim3((w.N + 127) / 128, (T + 127) / 128), dim3(LT_THREADS), LT_SMEM, w.map, x.map, p);
 }
@@ -411,14 +489,15 @@ int dc_launch_linear_grouped_tc(dc_ctx* ctx, const dc_lin& w, int groups, int gr
                                 const dc_lin_epi& epi) {
     if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: inner sizes %d and %d differ", w.K, x.K);
     if (groups < 1 || groups > DC_MOE_MAX_EXPERTS || groups * group_rows != w.N || max_rows < 1) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: bad groups");
-    if (epi.keys || epi.add || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: epilogue not available");
+    const bool pairs = epi.pair0 == 0 && epi.pair_kind == DC_PAIR_CLAMPED && epi.poutb && epi.tok_scale, rows = epi.pair0 >= (1 << 30) && epi.outb && !epi.bias && !epi.silu_rows;
+    if (epi.keys || epi.add || !(pairs || rows) || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: epilogue not available");
     LtParams p = {w.K, max_rows, epi, ctx->d_err};
     p.e.n_store = std::min(epi.n_store, std::min(group_rows, epi.pair0));
     p.e.n_pairs = std::max(0, std::min(epi.n_pairs, (group_rows - epi.pair0) / 2));
     const LwTiles tl = {(group_rows + 127) / 128, 0, groups, group_rows, group_off};
-    const int st = dc_kernel_setup(ctx, (const void*)k_linear_tc_wide<true>, (int)LW_SMEM, "k_linear_tc_grouped");
+    const int st = setup_unspilled(ctx, (const void*)k_linear_tc_wide<true>, (int)LW_SMEM, "k_linear_tc_grouped");
     if (st != DC_B200_OK) return st;
     const long long most = (long long)tl.row_tiles * (max_rows / 256 + std::min(groups, max_rows));
-    return dc_launch(ctx, "k_linear_tc_grouped", k_linear_tc_wide<true>, dim3((int)std::min<long long>(most, ctx->num_sms)), dim3(LT_THREADS), LW_SMEM, w.map, x.map,
+    return dc_launch(ctx, "k_linear_tc_grouped", k_linear_tc_wide<true>, dim3((int)std::min<long long>(most, ctx->num_sms)), dim3(LW_THREADS), LW_SMEM, w.map, x.map,
                      p, tl);
 }

@@ -369,34 +369,49 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
         }
 }
 
-// Splits of one (head, token) and the sink joined; with two maps the second is taken off the first and the rest normed.
+// Splits of one (head, token) and the sink joined; with two maps the second is taken off the first and the rest normed.  Every
+// fourth split is a warpgroup's.
+constexpr int JOIN_PARTS = 4;
 template <int MAPS>
-__global__ void __launch_bounds__(128) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int vdim,
-                                                  float sink, float lambda, float mul, float eps, float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb,
-                                                  int ldm) {
-    __shared__ float sw[MAPS][DC_MAX_SPLITS], red[33];
+__global__ void __launch_bounds__(128 * JOIN_PARTS) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int vdim,
+                                                               float sink, float lambda, float mul, float eps, float* __restrict__ mix,
+                                                               __nv_bfloat16* __restrict__ mixb, int ldm) {
+    __shared__ float sw[MAPS][DC_MAX_SPLITS], red[33], sum[JOIN_PARTS - 1][256];
     pdl_launch_dependents();
     pdl_wait();
-    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, share = threadIdx.x >> 7, d0 = threadIdx.x & 127;
     const size_t o = ((size_t)t * heads + h) * MAPS * splits;
+    float x[2][MAPS][DC_MAX_SPLITS / JOIN_PARTS];         // vdim <= 256
     if (warp < MAPS) join_weights(part_ml + 2 * (o + warp * splits), splits, lane, sink, warp ? -lambda : 1.0f, sw[warp]);
+    float v[2] = {0.0f, 0.0f}, ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int i = 0; i < MAPS; ++i)
+#pragma unroll
+            for (int k = 0; k < DC_MAX_SPLITS / JOIN_PARTS; ++k) {
+                const int s = share + JOIN_PARTS * k, d = d0 + 128 * j;
+                x[j][i][k] = s < splits && d < vdim ? part[(o + i * splits + s) * vdim + d] : 0.0f;
+            }
     __syncthreads();
-    float v[2] = {0.0f, 0.0f}, ss = 0.0f;         // vdim <= 256
 #pragma unroll
-    for (int j = 0; j < 2; ++j) {
-        const int d = threadIdx.x + 128 * j;
-        if (d < vdim) {
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int i = 0; i < MAPS; ++i)
-#pragma unroll 16
-                for (int s = 0; s < splits; ++s) v[j] = fmaf(part[(o + i * splits + s) * vdim + d], sw[i][s], v[j]);
-        }
-        ss = fmaf(v[j], v[j], ss);
-    }
+        for (int i = 0; i < MAPS; ++i)
+#pragma unroll
+            for (int k = 0; k < DC_MAX_SPLITS / JOIN_PARTS; ++k) v[j] = fmaf(x[j][i][k], sw[i][share + JOIN_PARTS * k], v[j]);
+    if (share > 0) sum[share - 1][d0] = v[0], sum[share - 1][d0 + 128] = v[1];
+    __syncthreads();
+    if (share > 0) v[0] = v[1] = 0.0f;
+    else
+#pragma unroll
+        for (int k = 0; k < JOIN_PARTS - 1; ++k) v[0] += sum[k][d0], v[1] += sum[k][d0 + 128];
+    ss = v[0] * v[0] + v[1] * v[1];
     const float f = MAPS > 1 ? mul / sqrtf(block_sum(ss, red) / (float)vdim + eps) : 1.0f;
+    if (share > 0) return;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
-        const int d = threadIdx.x + 128 * j;
+        const int d = d0 + 128 * j;
         if (d >= vdim) break;
         const size_t at = (size_t)t * ldm + (size_t)h * vdim + d;
         if (mixb) mixb[at] = __float2bfloat16_rn(v[j] * f);
@@ -712,11 +727,11 @@ int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, 
                      m.scale, m.softcap, st.seq_ids, st.positions, cache_ref(c, m.row), part, part_ml};
     if (m.maps > 1) {
         DC_TRY((c.f32 ? launch_tokens<float, 2>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16, 2>(ctx, p, m.kv_heads, st.T)));
-        return dc_launch(ctx, "k_gqa_join", k_gqa_join<2>, dim3(m.heads, st.T), dim3(128), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), m.lambda,
+        return dc_launch(ctx, "k_gqa_join", k_gqa_join<2>, dim3(m.heads, st.T), dim3(128 * JOIN_PARTS), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), m.lambda,
                          1.0f - m.diff, eps, mix, mixb, ldm);
     }
     DC_TRY((c.f32 ? launch_tokens<float, 1>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16, 1>(ctx, p, m.kv_heads, st.T)));
-    return dc_launch(ctx, "k_gqa_join", k_gqa_join<1>, dim3(m.heads, st.T), dim3(128), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), 0.0f, 1.0f, eps, mix,
+    return dc_launch(ctx, "k_gqa_join", k_gqa_join<1>, dim3(m.heads, st.T), dim3(128 * JOIN_PARTS), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), 0.0f, 1.0f, eps, mix,
                      mixb, ldm);
 }
 

@@ -237,13 +237,154 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
         }
 }
 
+// The same on the tensor cores for bf16 caches: sixteen heads are the rows of the products.  One CTA per (key split, sixteen
+// heads, token), eight warps: a warp scores eight of a tile's 64 keys, then two warps' worth of heads turn scores into
+// weights, then a warp sums NV groups of eight latent columns.  The queries are rounded to bf16, as the weights are.
+constexpr int HD_KEYS = 64, HD_WARPS = 8;
+
+template <int NV>
+__global__ void __launch_bounds__(HD_WARPS * 32) k_latent_heads(const AbsorbedParams p) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    const int row = p.c.row, dk = (row + 15) & ~15, ldk = (dk + 63) / 64 * 64 + 8;
+    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(sm);          // [16][ldk]
+    __nv_bfloat16* sk = sq + 16 * ldk;                                 // [HD_KEYS][ldk]
+    __shared__ __align__(16) __nv_bfloat16 sp[16][HD_KEYS + 8];
+    __shared__ float ss[16][HD_KEYS + 1], s_corr[16];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int s = blockIdx.x, h0 = blockIdx.y * 16, t = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int pos = p.positions[t], seq = p.seq_ids[t], first = first_key(pos, p.window), nk = pos - first + 1;
+    const int per = ((nk + p.splits - 1) / p.splits + 15) / 16 * 16, kb = first + s * per, ke = min(first + nk, kb + per);
+    const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.c.arena);
+    auto load = [&](int k0) {            // a warp's keys: all rows asked for before any arrives; zeros beyond the split
+        const __nv_bfloat16* src[HD_KEYS / HD_WARPS];
+#pragma unroll
+        for (int i = 0; i < HD_KEYS / HD_WARPS; ++i) src[i] = cache + p.c.at(seq, max(first, min(k0 + warp * (HD_KEYS / HD_WARPS) + i, ke - 1)));
+        for (int c = lane; c < dk / 8; c += 32)
+#pragma unroll
+            for (int i = 0; i < HD_KEYS / HD_WARPS; ++i) {
+                const int key = warp * (HD_KEYS / HD_WARPS) + i;
+                const bool in = k0 + key < ke && 8 * c < row;
+                cp_async16z(smem_u32(sk + key * ldk + 8 * c), in ? src[i] + 8 * c : cache, in);
+            }
+        cp_async_commit();
+    };
+    if (kb < ke) load(kb);
+    for (int r = warp; r < 16; r += HD_WARPS) {        // the absorbed part, then the rotated part, zeros in the padding
+        const int h = min(h0 + r, p.heads - 1);
+        const float *qa = p.qa + ((size_t)t * p.heads + h) * p.ldq, *qr = p.proj + (size_t)t * p.ldp + p.off_q + h * (p.dim + p.rot) + p.dim - p.rank;
+#pragma unroll 8
+        for (int c = lane; c < dk; c += 32)
+            sq[r * ldk + c] = __float2bfloat16_rn((c < p.rank ? qa[c] : c < p.rank + p.rot ? qr[c] : 0.0f) * p.scale);
+    }
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};          // of heads 2 warp, 2 warp + 1
+    float acc[NV][4];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    const int mi = lane >> 3, r8 = lane & 7, g = lane >> 2, q = lane & 3;
+    for (int k0 = kb; k0 < ke; k0 += HD_KEYS) {
+        cp_async_wait<0>();
+        __syncthreads();
+        float sc[2][4] = {};
+        const uint32_t qa = smem_u32(sq + ((mi & 1) * 8 + r8) * ldk + (mi >> 1) * 8), ka = smem_u32(sk + (8 * warp + r8) * ldk + mi * 8);
+#pragma unroll 4
+        for (int kk = 0; kk < dk; kk += 32) {          // a row of keys is padded to whole groups of 32 columns
+            uint32_t a[4], b[4];
+            ldsm_x4(ka + 2 * kk, b);
+            ldsm_x4(qa + 2 * kk, a);
+            mma_bf16(sc[0], a, b[0], b[1]);
+            if (kk + 16 < dk) {
+                ldsm_x4(qa + 2 * (kk + 16), a);
+                mma_bf16(sc[1], a, b[2], b[3]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss[g + 8 * (i >> 1)][8 * warp + 2 * q + (i & 1)] = sc[0][i] + sc[1][i];
+        __syncthreads();
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int h = 2 * warp + r;
+            float v[2];
+#pragma unroll
+            for (int j = 0; j < 2; ++j) v[j] = k0 + lane + 32 * j < ke ? ss[h][lane + 32 * j] : -INFINITY;
+            float mx = fmaxf(v[0], v[1]);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float mn = fmaxf(m[r], mx), corr = expf(m[r] - mn), w0 = expf(v[0] - mn), w1 = expf(v[1] - mn);
+            m[r] = mn;
+            l[r] = l[r] * corr + warp_sum(w0 + w1);
+            sp[h][lane] = __float2bfloat16_rn(w0), sp[h][lane + 32] = __float2bfloat16_rn(w1);
+            if (lane == 0) s_corr[h] = corr;
+        }
+        __syncthreads();
+        const float c0 = s_corr[g], c1 = s_corr[g + 8];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) acc[i][0] *= c0, acc[i][1] *= c0, acc[i][2] *= c1, acc[i][3] *= c1;
+#pragma unroll
+        for (int ks = 0; ks < HD_KEYS / 16; ++ks) {
+            uint32_t a[4];
+            ldsm_x4(smem_u32(&sp[(mi & 1) * 8 + r8][16 * ks + (mi >> 1) * 8]), a);
+#pragma unroll
+            for (int i = 0; i < NV; i += 2) {
+                const int c = 8 * (NV * warp + i);
+                if (c >= p.rank) break;
+                uint32_t b[4];
+                ldsm_x4_t(smem_u32(sk + (16 * ks + (mi & 1) * 8 + r8) * ldk + c + (mi >> 1) * 8), b);
+                mma_bf16(acc[i], a, b[0], b[1]);
+                mma_bf16(acc[i + 1], a, b[2], b[3]);
+            }
+        }
+        if (k0 + HD_KEYS < ke) {
+            __syncthreads();                           // every warp is done with the tile
+            load(k0 + HD_KEYS);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const int h = h0 + 2 * warp + r;
+        if (lane == 0 && h < p.heads) {
+            float* to = p.part_ml + 2 * (((size_t)t * p.heads + h) * p.splits + s);
+            to[0] = m[r], to[1] = l[r];
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const int h = h0 + g + 8 * r;
+        if (h >= p.heads) continue;
+        float* to = p.part + (((size_t)t * p.heads + h) * p.splits + s) * p.rank;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const int c = 8 * (NV * warp + i) + 2 * q + j;
+                if (c < p.rank) to[c] = acc[i][2 * r + j];
+            }
+    }
+}
+
+int launch_heads(dc_ctx* ctx, const AbsorbedParams& p, int T) {
+    const int ldk = (((p.c.row + 15) & ~15) + 63) / 64 * 64 + 8;
+    const size_t smem = (size_t)(16 + HD_KEYS) * ldk * 2;
+    const dim3 grid(p.splits, (p.heads + 15) / 16, T), block(HD_WARPS * 32);
+#define DC_HD(NV)                                                                                                  \
+    do {                                                                                                           \
+        DC_TRY(dc_kernel_setup(ctx, (const void*)k_latent_heads<NV>, (int)smem, "k_latent_heads"));                \
+        return dc_launch(ctx, "k_latent_heads", k_latent_heads<NV>, grid, block, smem, p);                         \
+    } while (0)
+    if (p.rank <= 128) DC_HD(2);
+    if (p.rank <= 256) DC_HD(4);
+    if (p.rank <= 512) DC_HD(8);
+    DC_HD(16);
+#undef DC_HD
+}
+
 // Splits of one (head, token) joined, then taken through OUT_ROWS rows of the head's W_uv and multiplied by the head's gate.
 constexpr int OUT_ROWS = 64;
 __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits,
                                                     int rank, const __nv_bfloat16* __restrict__ uv, int ldw, int vdim_p, int vdim,
                                                     const float* __restrict__ gate, int ldg,
                                                     float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
-    extern __shared__ __align__(16) float lat[];      // [rank padded to 8]
+    extern __shared__ __align__(16) float lat[];      // twice [rank padded to 8]
     __shared__ float sw[DC_MAX_SPLITS];
     pdl_launch_dependents();
     const int h = blockIdx.x, t = blockIdx.y, e0 = blockIdx.z * OUT_ROWS, e1 = min(vdim, e0 + OUT_ROWS), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -255,13 +396,31 @@ __global__ void __launch_bounds__(256) k_latent_out(const float* __restrict__ pa
     if (warp == 0) join_weights(part_ml + 2 * o, splits, lane, -INFINITY, 1.0f, sw);
     __syncthreads();
     const int rank8 = (rank + 7) & ~7;
-    for (int r = threadIdx.x; r < rank8; r += 256) {
-        float v = 0.0f;
-        if (r < rank) {
+    if (rank % 4 == 0) {         // two threads share four values of a latent
+        float* half = lat + rank8;
+        const int n4 = rank8 / 4, share = threadIdx.x >> 7;
+        for (int i = threadIdx.x & 127; i < n4; i += 128) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (4 * i < rank) {
 #pragma unroll 16
-            for (int s = 0; s < splits; ++s) v = fmaf(part[(o + s) * rank + r], sw[s], v);
+                for (int s = share; s < splits; s += 2) {
+                    const float4 x = *reinterpret_cast<const float4*>(part + (o + s) * rank + 4 * i);
+                    v.x = fmaf(x.x, sw[s], v.x), v.y = fmaf(x.y, sw[s], v.y), v.z = fmaf(x.z, sw[s], v.z), v.w = fmaf(x.w, sw[s], v.w);
+                }
+            }
+            reinterpret_cast<float4*>(share ? half : lat)[i] = v;
         }
-        lat[r] = v;
+        __syncthreads();
+        for (int i = threadIdx.x; i < rank8; i += 256) lat[i] += half[i];
+    } else {
+        for (int r = threadIdx.x; r < rank8; r += 256) {
+            float v = 0.0f;
+            if (r < rank) {
+#pragma unroll 16
+                for (int s = 0; s < splits; ++s) v = fmaf(part[(o + s) * rank + r], sw[s], v);
+            }
+            lat[r] = v;
+        }
     }
     __syncthreads();
     constexpr int ROWS = OUT_ROWS / 8;                // of a warp, all in flight
@@ -544,8 +703,8 @@ int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_st
 #undef DC_ABSORB
     AbsorbedParams p = {qa, ldq, proj, ldp, m.off_q, m.heads, m.dim, m.rot_dim, m.kv_rank, m.window, splits, m.scale, st.seq_ids, st.positions,
                         cache_ref(c, m.row), part, part_ml};
-    DC_TRY(c.f32 ? launch_absorbed<float>(ctx, p, st.T) : launch_absorbed<__nv_bfloat16>(ctx, p, st.T));
-    return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T, (m.vdim + OUT_ROWS - 1) / OUT_ROWS), dim3(256), (size_t)dc_pad8(m.kv_rank) * 4, part, part_ml, m.heads, splits,
+    DC_TRY(c.f32 ? launch_absorbed<float>(ctx, p, st.T) : launch_heads(ctx, p, st.T));
+    return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T, (m.vdim + OUT_ROWS - 1) / OUT_ROWS), dim3(256), (size_t)dc_pad8(m.kv_rank) * 8, part, part_ml, m.heads, splits,
                      m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim,
                      m.off_g < 0 ? nullptr : proj + m.off_g, ldp, mix, mixb, ldm);
 }
