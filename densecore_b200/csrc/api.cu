@@ -37,15 +37,20 @@ static std::mutex g_kernel_mu;
 static std::map<std::pair<int, const void*>, int> g_kernel_smem;                    // opted-in bytes
 static std::map<std::tuple<int, const void*, int, size_t>, int> g_kernel_occupancy;
 
-int dc_kernel_setup(dc_ctx* ctx, const void* func, int max_dyn_smem, const char* name) {
+static int kernel_setup(dc_ctx* ctx, const void* func, int max_dyn_smem, const char* name, int carveout) {
     std::lock_guard<std::mutex> lk(g_kernel_mu);
     auto key = std::make_pair(ctx->device, func);
     auto it = g_kernel_smem.find(key);
     if (it != g_kernel_smem.end() && it->second >= max_dyn_smem) return DC_B200_OK;
     cudaError_t e = cudaFuncSetAttribute(func, cudaFuncAttributeMaxDynamicSharedMemorySize, max_dyn_smem);
+    if (e == cudaSuccess && carveout > 0) e = cudaFuncSetAttribute(func, cudaFuncAttributePreferredSharedMemoryCarveout, carveout);
     if (e != cudaSuccess) return dc_check_cuda(ctx, e, name);
     g_kernel_smem[key] = max_dyn_smem;
     return DC_B200_OK;
+}
+int dc_kernel_setup(dc_ctx* ctx, const void* func, int max_dyn_smem, const char* name) { return kernel_setup(ctx, func, max_dyn_smem, name, 0); }
+int dc_kernel_setup_small(dc_ctx* ctx, const void* func, int max_dyn_smem, const char* name) {
+    return kernel_setup(ctx, func, max_dyn_smem, name, max_dyn_smem <= 50 * 1024 ? 45 : 0);
 }
 
 int dc_kernel_occupancy(dc_ctx* ctx, const void* func, int threads, size_t dyn_smem) {

@@ -54,6 +54,8 @@ int dc_check_device_error(dc_ctx* ctx);            // reads d_err after a sync
 // One-time, per-device kernel set-up (thread-safe): opt `func` into max_dyn_smem bytes of dynamic shared
 // memory on ctx's device; cached occupancy (resident CTAs per SM) of `func` on that device.
 int dc_kernel_setup(dc_ctx* ctx, const void* func, int max_dyn_smem, const char* name);
+// the same, asking for a split that leaves more than half of an SM's memory to L1: kernels of a decode step that overlap share one split
+int dc_kernel_setup_small(dc_ctx* ctx, const void* func, int max_dyn_smem, const char* name);
 int dc_kernel_occupancy(dc_ctx* ctx, const void* func, int threads, size_t dyn_smem);
 
 // ---- launch helpers implemented in the kernel translation units ----

@@ -39,3 +39,15 @@ static inline int dc_launch(dc_ctx* ctx, const char* name, void (*kernel)(KArgs.
     cfg.numAttrs = ctx->use_pdl ? 1 : 0;
     return dc_check_cuda(ctx, cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...), name);
 }
+
+// The same without the attribute: the kernel starts once the one before has left the SMs.  For the successor of a kernel with
+// much shared memory: SMs that never drain keep its split between shared memory and L1, and streaming kernels need the L1.
+template <typename... KArgs, typename... Args>
+static inline int dc_launch_drained(dc_ctx* ctx, const char* name, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    return dc_check_cuda(ctx, cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...), name);
+}

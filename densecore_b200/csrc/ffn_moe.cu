@@ -697,7 +697,7 @@ int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, c
             return dc_launch(ctx, "k_moe_norm_route_tile", k_moe_norm_route_tile<PER>, dim3((T + 15) / 16), dim3(NT_WARPS * 32), z.bytes, p,      \
                              f.router.N, T);                                                                                                     \
         }                                                                                                                                        \
-        const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route<PER>, (int)smem, "k_moe_norm_route");                                   \
+        const int st = dc_kernel_setup_small(ctx, (const void*)k_moe_norm_route<PER>, (int)smem, "k_moe_norm_route");                                   \
         if (st != DC_B200_OK) return st;                                                                                                         \
         return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route<PER>, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);       \
     } while (0)

@@ -704,9 +704,15 @@ int dc_launch_latent_absorbed(dc_ctx* ctx, const dc_latent_mixer& m, const dc_st
     AbsorbedParams p = {qa, ldq, proj, ldp, m.off_q, m.heads, m.dim, m.rot_dim, m.kv_rank, m.window, splits, m.scale, st.seq_ids, st.positions,
                         cache_ref(c, m.row), part, part_ml};
     DC_TRY(c.f32 ? launch_absorbed<float>(ctx, p, st.T) : launch_heads(ctx, p, st.T));
-    return dc_launch(ctx, "k_latent_out", k_latent_out, dim3(m.heads, st.T, (m.vdim + OUT_ROWS - 1) / OUT_ROWS), dim3(256), (size_t)dc_pad8(m.kv_rank) * 8, part, part_ml, m.heads, splits,
-                     m.kv_rank, m.ukv.w + (size_t)m.uv_row * m.ukv.ld, m.ukv.ld, m.vdim_p, m.vdim,
-                     m.off_g < 0 ? nullptr : proj + m.off_g, ldp, mix, mixb, ldm);
+    const dim3 grid(m.heads, st.T, (m.vdim + OUT_ROWS - 1) / OUT_ROWS), block(256);
+    const size_t smem = (size_t)dc_pad8(m.kv_rank) * 8;
+    const __nv_bfloat16* uv = m.ukv.w + (size_t)m.uv_row * m.ukv.ld;
+    const float* gate = m.off_g < 0 ? nullptr : proj + m.off_g;
+    if (c.f32)
+        return dc_launch(ctx, "k_latent_out", k_latent_out, grid, block, smem, part, part_ml, m.heads, splits, m.kv_rank, uv, m.ukv.ld, m.vdim_p, m.vdim, gate, ldp,
+                         mix, mixb, ldm);
+    return dc_launch_drained(ctx, "k_latent_out", k_latent_out, grid, block, smem, part, part_ml, m.heads, splits, m.kv_rank, uv, m.ukv.ld, m.vdim_p, m.vdim, gate,
+                             ldp, mix, mixb, ldm);
 }
 
 int dc_launch_latent_gather(dc_ctx* ctx, const dc_latent_mixer& m, const dc_step& st, const dc_latent_cache& c, const int32_t* key_base,
