@@ -453,16 +453,6 @@ __device__ __forceinline__ float soft_cap(float z, float cap) {
     return cap - __fdividef(2.0f * cap, 1.0f + ex2(2.8853900817779268f * z));
 }
 
-// the same for |z| < 0.3 by the series of tanh
-constexpr float CAP_SERIES = 0.3f;
-__device__ __forceinline__ float soft_cap_small(float z, float cap) {
-    const float u = z * z;
-    float t = fmaf(u, 62.0f / 2835.0f, -17.0f / 315.0f);
-    t = fmaf(u, t, 2.0f / 15.0f);
-    t = fmaf(u, t, -1.0f / 3.0f);
-    return cap * fmaf(u * z, t, z);
-}
-
 // One CTA per (QT = PQ / MAPS queries of one entry, head), sixteen rows (queries of one map) a warp; key and value tiles in
 // a ring of ST stages, two CTAs an SM.  DP, VP: key and value size, padded.
 template <int DP, int VP, int PQ, int ST, int MAPS>
@@ -563,25 +553,10 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
             }
         }
         if (capped) {
-            float most = 0.0f;
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    s[nt][j] *= to_cap;
-                    most = fmaxf(most, fabsf(s[nt][j]));
-                }
-            if (__any_sync(0xffffffffu, most >= CAP_SERIES)) {
-#pragma unroll
-                for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-                    for (int j = 0; j < 4; ++j) s[nt][j] = soft_cap(s[nt][j], cap);
-            } else {
-#pragma unroll
-                for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-                    for (int j = 0; j < 4; ++j) s[nt][j] = soft_cap_small(s[nt][j], cap);
-            }
+                for (int j = 0; j < 4; ++j) s[nt][j] = soft_cap(s[nt][j] * to_cap, cap);
         }
         // the warp's sixteen queries see the whole tile, or the mask decides key by key
         if (!(k1 <= wq0 && wq0 + 15 - k0 < window)) {

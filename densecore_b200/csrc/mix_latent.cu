@@ -270,12 +270,37 @@ __global__ void __launch_bounds__(HD_WARPS * 32) k_latent_heads(const AbsorbedPa
         cp_async_commit();
     };
     if (kb < ke) load(kb);
-    for (int r = warp; r < 16; r += HD_WARPS) {        // the absorbed part, then the rotated part, zeros in the padding
-        const int h = min(h0 + r, p.heads - 1);
-        const float *qa = p.qa + ((size_t)t * p.heads + h) * p.ldq, *qr = p.proj + (size_t)t * p.ldp + p.off_q + h * (p.dim + p.rot) + p.dim - p.rank;
-#pragma unroll 8
-        for (int c = lane; c < dk; c += 32)
-            sq[r * ldk + c] = __float2bfloat16_rn((c < p.rank ? qa[c] : c < p.rank + p.rot ? qr[c] : 0.0f) * p.scale);
+    // a warp's two heads: the absorbed part, all loads in flight, then the rotated part, zeros in the padding
+    {
+        const float *qa[2], *qr[2];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int h = min(h0 + 2 * warp + r, p.heads - 1);
+            qa[r] = p.qa + ((size_t)t * p.heads + h) * p.ldq;
+            qr[r] = p.proj + (size_t)t * p.ldp + p.off_q + h * (p.dim + p.rot) + p.dim - p.rank;
+        }
+        const int whole = p.rank & ~3;
+        float4 v[2][NV / 2];             // 64 NV columns at most
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+            for (int j = 0; j < NV / 2; ++j) {
+                const int c = 4 * lane + 128 * j;
+                v[r][j] = c < whole ? *reinterpret_cast<const float4*>(qa[r] + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        for (int c = whole + lane; c < dk; c += 32)
+#pragma unroll
+            for (int r = 0; r < 2; ++r)
+                sq[(2 * warp + r) * ldk + c] = __float2bfloat16_rn((c < p.rank ? qa[r][c] : c < p.rank + p.rot ? qr[r][c] : 0.0f) * p.scale);
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+            for (int j = 0; j < NV / 2; ++j) {
+                const int c = 4 * lane + 128 * j;
+                if (c < whole)
+                    *reinterpret_cast<uint2*>(sq + (2 * warp + r) * ldk + c) = make_uint2(pack_bf2(v[r][j].x * p.scale, v[r][j].y * p.scale),
+                                                                                          pack_bf2(v[r][j].z * p.scale, v[r][j].w * p.scale));
+            }
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};          // of heads 2 warp, 2 warp + 1
     float acc[NV][4];
@@ -353,12 +378,16 @@ __global__ void __launch_bounds__(HD_WARPS * 32) k_latent_heads(const AbsorbedPa
         if (h >= p.heads) continue;
         float* to = p.part + (((size_t)t * p.heads + h) * p.splits + s) * p.rank;
 #pragma unroll
-        for (int i = 0; i < NV; ++i)
+        for (int i = 0; i < NV; ++i) {
+            const int c = 8 * (NV * warp + i) + 2 * q;
+            if (p.rank % 2 == 0) {
+                if (c < p.rank) *reinterpret_cast<float2*>(to + c) = make_float2(acc[i][2 * r], acc[i][2 * r + 1]);
+            } else {
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int c = 8 * (NV * warp + i) + 2 * q + j;
-                if (c < p.rank) to[c] = acc[i][2 * r + j];
+                for (int j = 0; j < 2; ++j)
+                    if (c + j < p.rank) to[c + j] = acc[i][2 * r + j];
             }
+        }
     }
 }
 
