@@ -238,8 +238,8 @@ __global__ void __launch_bounds__(AB_HEADS * 32) k_latent_absorbed(const Absorbe
 }
 
 // The same on the tensor cores for bf16 caches: sixteen heads are the rows of the products.  One CTA per (key split, sixteen
-// heads, token), eight warps: a warp scores eight of a tile's 64 keys, then two warps' worth of heads turn scores into
-// weights, then a warp sums NV groups of eight latent columns.  The queries are rounded to bf16, as the weights are.
+// heads, token), eight warps: a warp scores eight of a tile's 64 keys for all heads, then turns two heads' scores into
+// weights, then sums NV groups of eight latent columns for all heads.  The queries are rounded to bf16, as the weights are.
 constexpr int HD_KEYS = 64, HD_WARPS = 8;
 
 template <int NV>
