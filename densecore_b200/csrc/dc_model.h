@@ -13,7 +13,7 @@ enum {
     DC_K_EMBED = 0, DC_K_RMSNORM, DC_K_GEMV_QKV, DC_K_QKROPE, DC_K_ATTENTION, DC_K_GEMV_O, DC_K_ROUTER, DC_K_MOE_GATEUP,
     DC_K_QUANT_H, DC_K_MOE_DOWN, DC_K_COMBINE, DC_K_ALLREDUCE, DC_K_FFN_GATEUP, DC_K_FFN_DOWN, DC_K_LM_HEAD, DC_K_ARGMAX,
     DC_K_MIX_IN, DC_K_MIX_OUT, DC_K_MIX_DELTA, DC_K_MIX_SSD, DC_K_MIX_LATENT, DC_K_POST_NORM, DC_K_PRE_NORM,
-    DC_K_MIX_GQA, DC_K_MIX_LIGHTNING,
+    DC_K_MIX_GQA, DC_K_MIX_LIGHTNING, DC_K_MIX_GENERAL,
     DC_K_COUNT
 };
 

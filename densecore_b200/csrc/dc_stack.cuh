@@ -11,6 +11,10 @@ namespace dc {
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float relu2(float z) {
+    z = fmaxf(z, 0.0f);
+    return z * z;
+}
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float gelu_tanh(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -61,6 +65,7 @@ __device__ __forceinline__ float load_as(const __nv_bfloat16* p) { return __bflo
 // ---- epilogues of the products (dc_lin_epi)
 __device__ __forceinline__ float pair_value(const dc_lin_epi& e, float gate, float up) {
     if (e.pair_kind == DC_PAIR_GELU) return gelu_tanh(gate) * up;
+    if (e.pair_kind == DC_PAIR_SILU) return silu(gate) * up;
     gate = fminf(gate, e.limit);
     up = fminf(fmaxf(up, -e.limit), e.limit);
     return gate * sigmoid(1.702f * gate) * (up + 1.0f);
@@ -73,7 +78,8 @@ __device__ __forceinline__ void put_pair(const dc_lin_epi& e, int t, int pair, f
 // returns the stored value
 __device__ __forceinline__ float put_row(const dc_lin_epi& e, int t, int row, float v) {
     if (e.bias) v += e.bias[row];
-    if (row < e.silu_rows) v = silu(v);
+    if (row < e.act_rows) v = e.act == DC_ACT_SILU ? silu(v) : relu2(v);
+    if (e.tok_scale) v *= e.tok_scale[t];
     const size_t at = (size_t)t * e.ldo + row;
     if (e.outb) {
         e.outb[at] = __float2bfloat16_rn(v);
@@ -103,6 +109,107 @@ __device__ __forceinline__ BlockRef block_at(const int32_t* starts, int E, int b
     }
     return BlockRef{0, 0, 0};
 }
+// ---- short causal convolutions
+__device__ __forceinline__ int entry_of(const int32_t* starts, int E, int t) {
+    int e = 0;
+    while (e + 1 < E && starts[e + 1] <= t) ++e;
+    return e;
+}
+
+// Convolution of one channel at token t (local index i in its entry, position pos): weights w[j * ldw], the last tap for
+// the token itself; inputs before the entry come from the ring, before position 0 they are zero.
+__device__ __forceinline__ float conv_at(const float* __restrict__ proj, int ldp, const float* __restrict__ ring, int C, int rc, int taps,
+                                         const float* __restrict__ w, int ldw, int col, int t, int i, int pos) {
+    float s = 0.0f;
+    if (i >= taps - 1) {
+        const float* in = proj + (size_t)(t - taps + 1) * ldp + col;
+#pragma unroll 4
+        for (int j = 0; j < taps; ++j) s = fmaf(w[(size_t)j * ldw], in[(size_t)j * ldp], s);
+        return s;
+    }
+    for (int j0 = 0; j0 < taps; j0 += 4) {      // four taps' loads in flight, none behind a branch
+        float in[4], wj[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int j = min(j0 + k, taps - 1), back = taps - 1 - j;
+            const float* src = back <= i ? proj + (size_t)(t - back) * ldp + col : ring + (size_t)(max(pos - back, 0) % taps) * C + rc;
+            in[k] = *src;
+            wj[k] = w[(size_t)j * ldw];
+            if (j0 + k >= taps || pos < back) in[k] = 0.0f;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) s = fmaf(wj[k], in[k], s);
+    }
+    return s;
+}
+
+struct ConvRef {
+    uint8_t* base;
+    size_t slot_bytes, ring_off;
+    const int32_t *seq_ids, *positions, *starts;
+    int E, taps, C, ldw;     // C: channels of a ring row; ldw: pitch of the convolution weights [taps][ldw]
+    __device__ float* ring(int seq) const { return reinterpret_cast<float*>(base + (size_t)seq * slot_bytes + ring_off); }
+};
+
+// ---- a residual of several streams (dc_hyper)
+// Sixteen-byte groups of rows named by a sum, added up.
+__device__ __forceinline__ void add4(float4& a, float4 b) { a.x += b.x, a.y += b.y, a.z += b.z, a.w += b.w; }
+__device__ __forceinline__ float4 row_sum4(const dc_row_sum& sum, const int32_t* rows, int i) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int k = 0; k < sum.k; ++k) {
+        const size_t at = (size_t)rows[k] * sum.ld + 4 * i;
+        if (sum.yb) {
+            const uint2 u = *reinterpret_cast<const uint2*>(sum.yb + at);
+            add4(v, make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u)));
+        } else {
+            add4(v, *reinterpret_cast<const float4*>(sum.y + at));
+        }
+    }
+    return v;
+}
+// Coefficients in shared memory, padded with zeros to S streams: in [S] | out [S], times mul | mix [S][S].
+template <int S>
+__device__ __forceinline__ void hyper_coefficients(const dc_hyper& h, float* c) {
+    const int n = h.streams;
+    for (int i = threadIdx.x; i < S * (S + 2); i += blockDim.x) {
+        float v = 0.0f;
+        if (i < S) {
+            if (i < n) v = h.next ? h.next[i] : 1.0f;
+        } else if (i < 2 * S) {
+            if (i - S < n && h.done) v = h.mul * h.done[i];
+        } else {
+            const int s = (i - 2 * S) / S, t = (i - 2 * S) % S;
+            if (s < n && t < n) v = h.done ? h.done[2 * n + s * n + t] : s == t ? 1.0f : 0.0f;
+        }
+        c[i] = v;
+    }
+}
+// Group i of four columns of token t, whose sublayer output is y: the streams anew (to x_out if store) and u.
+template <int S>
+__device__ __forceinline__ float4 hyper_column(const dc_hyper& h, const float* c, int t, int i, int ld, float4 y, bool store) {
+    float4 v[S], u = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int n = h.streams;
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+        const size_t row = h.first ? t : (size_t)t * n + s;
+        v[s] = s < n ? *reinterpret_cast<const float4*>(h.x + row * ld + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int to = 0; to < S; ++to) {
+        const float o = c[S + to], in = c[to];
+        float4 r = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll
+        for (int s = 0; s < S; ++s) {
+            const float m = c[2 * S + s * S + to];
+            r.x = fmaf(m, v[s].x, r.x), r.y = fmaf(m, v[s].y, r.y), r.z = fmaf(m, v[s].z, r.z), r.w = fmaf(m, v[s].w, r.w);
+        }
+        if (store && to < n) *reinterpret_cast<float4*>(h.x_out + ((size_t)t * n + to) * ld + 4 * i) = r;
+        u.x = fmaf(in, r.x, u.x), u.y = fmaf(in, r.y, u.y), u.z = fmaf(in, r.z, u.z), u.w = fmaf(in, r.w, u.w);
+    }
+    return u;
+}
+
 // ---- cached rows of a sequence's tokens
 __device__ __forceinline__ int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
 

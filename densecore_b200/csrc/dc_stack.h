@@ -20,13 +20,14 @@
 
 struct dc_model;
 
-enum { DC_MIX_DELTA = 0, DC_MIX_LATENT = 1, DC_MIX_SSD = 2, DC_MIX_GQA = 3, DC_MIX_LIGHTNING = 4 };
+enum { DC_MIX_DELTA = 0, DC_MIX_LATENT = 1, DC_MIX_SSD = 2, DC_MIX_GQA = 3, DC_MIX_LIGHTNING = 4, DC_MIX_GENERAL = 5 };
 enum { DC_DTYPE_BF16 = 0, DC_DTYPE_F32 = 1 };
 // How a layer's sublayers meet the residual.  POST_NORM: x += norm1(mixer(x)), then x += norm2(ff(x)).  PARALLEL: with
 // h = norm1(x), x += mixer(h) + ff(h); the input matrices of both are one product, and so are the output matrices.
-// PRE_NORM: x += mixer(norm1(x)), then x += ff(norm2(x)).
-enum { DC_BLOCK_POST_NORM = 0, DC_BLOCK_PARALLEL = 1, DC_BLOCK_PRE_NORM = 2 };
-enum { DC_PAIR_GELU = 0, DC_PAIR_CLAMPED = 1 };
+// PRE_NORM: x += mixer(norm1(x)), then x += ff(norm2(x)).  HYPER: pre-norm over a residual of several streams, see dc_hyper.
+enum { DC_BLOCK_POST_NORM = 0, DC_BLOCK_PARALLEL = 1, DC_BLOCK_PRE_NORM = 2, DC_BLOCK_HYPER = 3 };
+enum { DC_PAIR_GELU = 0, DC_PAIR_CLAMPED = 1, DC_PAIR_SILU = 2 };
+enum { DC_ACT_SILU = 0, DC_ACT_RELU2 = 1 };     // of single rows
 
 #define DC_MAX_SPLITS 64        // key splits of a decode step's attention
 
@@ -41,23 +42,23 @@ struct dc_lin {
 };
 
 // What becomes of a product's rows.  Rows below pair0 are stored (to outb if given, else to out) after the bias and, for
-// the first silu_rows of them, silu; `add` adds to what out holds.  Rows from pair0 on are gate and up rows in turn
-// and each pair is one value of poutb / pout: gelu_tanh(gate) up, or with both clamped (gate from above only)
-// gate sigmoid(1.702 gate) (up + 1).
+// the first act_rows of them, silu or the square of relu; `add` adds to what out holds.  Rows from pair0 on are gate and
+// up rows in turn and each pair is one value of poutb / pout: gelu_tanh(gate) up, silu(gate) up, or with both clamped
+// (gate from above only) gate sigmoid(1.702 gate) (up + 1).
 #define DC_PAIR_ALIGN 32        // pair0 is a multiple of this
 struct dc_lin_epi {
     float* out = nullptr;
     __nv_bfloat16* outb = nullptr;
     int ldo = 0, n_store = 0;   // rows stored: at most n_store (launchers: also at most the matrix' rows)
     const float* bias = nullptr;
-    int silu_rows = 0;
+    int act_rows = 0, act = DC_ACT_SILU;
     bool add = false;
     int pair0 = 1 << 30, pair_kind = DC_PAIR_GELU;
     float limit = 0.0f;
     float* pout = nullptr;
     __nv_bfloat16* poutb = nullptr;
     int ldp = 0, n_pairs = 0;
-    const float* tok_scale = nullptr;        // factor of every pair value of a token (grouped products)
+    const float* tok_scale = nullptr;        // factor of every pair value, or of every row after its activation, of a token (grouped products)
     unsigned long long* keys = nullptr;      // packed greedy picks per token (products of up to DC_MAX_T tokens)
 
     static dc_lin_epi store(float* out, __nv_bfloat16* outb, int ldo, unsigned long long* keys = nullptr) {
@@ -125,7 +126,8 @@ struct dc_rotation {
 enum { DC_QK_PLAIN = 0, DC_QK_NORM_ALL = 1, DC_QK_NORM_HEAD = 2 };
 
 // Grouped-query attention.  maps 2: every head has two queries and keys over the same values; the second map's output is
-// taken off the first's, weighted by lambda, and the difference is normed per head and multiplied by 1 - diff.
+// taken off the first's, weighted by lambda, and the difference is normed per head and multiplied by 1 - diff.  score_bias:
+// no softmax, a visible key counts sigmoid(score + the head's bias), unnormalized.
 struct dc_gqa_mixer {
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0, maps = 1;
     int window = 0, keep = 0;   // window 0: every earlier token; else the last `window` and the sequence's first `keep`
@@ -138,7 +140,12 @@ struct dc_gqa_mixer {
     int off_q = 0, off_k = 0, off_v = 0;    // projection rows; off_v = off_k: the values are the keys before norm and rotation
     int dim_p = 0, vdim_p = 0;  // padded sizes in the cached rows
     float *bias = nullptr;      // of the projection rows
-    float *q_norm = nullptr, *k_norm = nullptr;             // [heads * dim] and [kv_heads * dim], or [dim]
+    float *q_norm = nullptr, *k_norm = nullptr;             // [heads * dim] and [kv_heads * dim], or [dim] (null: no weight)
+    bool v_norm = false;        // every head's value over its root mean square
+    int taps = 0;               // short causal convolution of the projections ahead of everything else (0: none)
+    float *conv = nullptr;      // [taps][projection columns up to the values' end]
+    float *score_bias = nullptr;            // [heads]
+    int off_g = -1;             // one gate per head: the head's output is multiplied by sigmoid of this row (-1: none)
     float diff = 0.0f, lambda = 0.0f;       // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
     float* lam[4] = {};         // lq1, lk1, lq2, lk2 [dim]
     const float* cos_sin = nullptr;
@@ -154,15 +161,28 @@ struct dc_lightning_mixer {     // linear attention with one constant decay per 
     float *norm = nullptr;      // [heads * vdim]: all heads are normed together, then gated by sigmoid(g)
 };
 
-// Mixture of clamped gated experts.  Scores are sigmoid(router); choices are made on score + correction, among the
-// experts of the `keep` groups whose two best choice scores sum up highest; an expert's weight is its score times scale.
+// Generalized delta rule: S <- diag(w) S - (a u)(u^T S) + k v^T, o = S^T r, with the unit key u, a removal rate a and a decay
+// w = exp(-e^(-1/2) sigmoid(W2 tanh(W1 h) + w0)) per key channel.  Heads are normed, weighted and gated by sigmoid(g).
+struct dc_general_mixer {
+    int heads = 0, dim = 0, rank = 0;       // values have the keys' size
+    float unit_eps = 1e-6f;
+    int off_r = 0, off_k = 0, off_v = 0, off_g = 0, off_a = 0, off_w = 0;   // projection rows; off_w: W1
+    dc_lin w2;
+    float *w0 = nullptr, *a_bias = nullptr, *norm = nullptr;                // [heads * dim]
+};
+
+// Mixture of experts.  Scores are sigmoid(router); choices are made on score + correction, among the experts of the `keep`
+// groups whose two best choice scores sum up highest; an expert's weight is its score times scale.  softmax: scores are the
+// softmax over all experts, and the chosen ones' are divided by their sum.  Experts are clamped and gated, or (plain) the
+// square of relu between two matrices.
 #define DC_MOE_MAX_EXPERTS 512
 #define DC_MOE_MAX_TOP 32
 #define DC_MOE_MAX_GROUPS 32
 struct dc_moe_ffn {
     int experts = 0, top = 0, groups = 1, keep = 1, ff = 0;
     float scale = 1.0f, limit = 0.0f;
-    dc_lin router, up, down;    // up: per expert up_rows rows (gate and up in turn), down: per expert down_rows
+    bool softmax = false, plain = false;
+    dc_lin router, up, down;    // up: per expert up_rows rows (gate and up in turn, or up alone), down: per expert down_rows
     int up_rows = 0, down_rows = 0;
     float* correction = nullptr;
 };
@@ -174,6 +194,7 @@ struct dc_stack_layer {
     dc_latent_mixer la;
     dc_gqa_mixer ga;
     dc_lightning_mixer li;
+    dc_general_mixer ge;
     // parallel blocks: mixer rows, then (from pair0) gate and up rows in turn; mixer columns, then (from out_ff) the
     // feed-forward's
     dc_lin in, out;
@@ -183,7 +204,9 @@ struct dc_stack_layer {
     int ff = 0;                 // 0: no dense feed-forward
     dc_moe_ffn moe;             // experts 0: none
     dc_lin gate_up, down;       // gate_up: rows 2i = gate row i, 2i + 1 = up row i
+    int ff_pair = DC_PAIR_GELU; // dense feed-forward of its own
     float *norm1 = nullptr, *norm2 = nullptr;
+    float* hyper[2] = {};       // coefficients of the sublayers: in [streams] | out [streams] | mix [from][to]
 };
 
 // One run of a layer: a looped layer has several, each with a cache or state of its own.
@@ -205,10 +228,11 @@ struct dc_stack_tensor {
     float** vec = nullptr;
     int64_t vec_off = 0, vec_len = 0;     // destination range and the vector's whole length
     bool neg_exp = false;       // stored as -exp(value)
+    float plus = 0.0f;          // added to what the file holds
     int64_t pitch = 0;          // a vector of shape [n, k] stored with rows of this many floats
     int64_t cols = 0;           // a vector of shape [n, taps] stored transposed: element (c, j) at j * cols + vec_off + c
     bool loaded = false;
-    int synth = 0;              // random-weight kind: 0 matrix, 1 norm weight, 2 decay exponent, 3 step bias, 4 small vector
+    int synth = 0;              // random-weight kind: 0 matrix, 1 norm weight, 2 decay exponent, 3 step bias, 4 small vector, 5 one over the streams
 };
 
 struct dc_stack_config {
@@ -217,6 +241,8 @@ struct dc_stack_config {
     int loop_start = 0, loop_stop = 0, loop_times = 0;      // layers start .. stop - 1 run `times` times in a row (0: no loop)
     float eps = 1e-5f, embed_scale = 1.0f;
     bool tied = false;          // the output matrix is the embedding table
+    int streams = 1;            // of the residual
+    float residual_mult = 1.0f;
 };
 
 // One step's tokens on the device.  Entry e is tokens starts[e] .. starts[e + 1] - 1, consecutive positions of one
@@ -236,7 +262,7 @@ struct dc_stack_buffers {
     int32_t* h_meta = nullptr;  // pinned, DC_STACK_META_SLOTS slots
     int meta_ints = 0, meta_slot = 0;
     int32_t *iota = nullptr, *chunk = nullptr;   // constant entry starts: one token each; one entry of n tokens at chunk + 2 n
-    float *x = nullptr, *y = nullptr, *proj = nullptr, *act = nullptr, *scan = nullptr, *low = nullptr, *gate = nullptr, *small = nullptr, *blk = nullptr;
+    float *x = nullptr, *x2 = nullptr, *h = nullptr, *y = nullptr, *proj = nullptr, *act = nullptr, *scan = nullptr, *low = nullptr, *gate = nullptr, *small = nullptr, *blk = nullptr;
     float *mix = nullptr, *ff = nullptr, *lm_x = nullptr;   // mix, ff, lm_x: f32 models
     __nv_bfloat16 *lm_xb = nullptr, *xb = nullptr, *mixb = nullptr, *ffb = nullptr, *lowb = nullptr;
     __nv_bfloat16 *keys_c = nullptr, *keys_r = nullptr, *keys_kv = nullptr;
@@ -258,6 +284,7 @@ struct dc_stack {
     int dtype = DC_DTYPE_BF16;
     std::vector<dc_stack_layer> layers;
     std::vector<dc_stack_run> runs;
+    float* hyper_sum = nullptr; // [streams]: ones
     float* loop_step = nullptr; // [loop_times][width padded to 8]
     dc_weight* embed = nullptr;
     dc_lin head;
@@ -321,11 +348,31 @@ struct dc_row_sum {
 int dc_launch_pre_norm(dc_ctx* ctx, float* x, const float* step, const dc_row_sum& sum, const float* w, int T, int H, int ld, float eps, float* out,
                        __nv_bfloat16* outb);
 
+// A residual of `streams` streams, [token][stream][ld], and what it still owes: the sublayer before left y (one row a token, or
+// the sum of rows) and its coefficients `done`; stream t becomes sum_s mix[s][t] x_s + mul out[t] y.  u = sum_t next[t] x_t is
+// what the next sublayer's norm takes.  Without `done` nothing is owed.  x_out (optional) is another buffer than x: several
+// CTAs of a token read x.
+#define DC_MAX_STREAMS 8
+struct dc_hyper {
+    int streams = 1;
+    bool first = false;         // x has one row per token that all streams share
+    const float* x = nullptr;
+    float* x_out = nullptr;
+    const float* y = nullptr;
+    dc_row_sum sum;
+    const float *done = nullptr, *next = nullptr;
+    float mul = 1.0f;
+};
+// out row r: u of token rows[r] (rows null: first + r), normed with w (w null: as it is)
+int dc_launch_hyper_norm(dc_ctx* ctx, const dc_hyper& hy, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps, float* out,
+                         __nv_bfloat16* outb);
+
 // ---- ffn_moe.cu
 // norm of the residual (out / outb), router logits, choices (ids and weights [T][top]); where it fits: few tokens, or a bf16
 // model whose width and experts leave room in shared memory
 bool dc_moe_norm_route_fits(const dc_moe_ffn& f, bool b16, int T, int ld);
-int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const float* w, int T, int H, int ld, float eps, float* out,
+// hy: the row that is normed comes from the streams instead of x
+int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const dc_hyper* hy, const float* w, int T, int H, int ld, float eps, float* out,
                              __nv_bfloat16* outb, int32_t* ids, float* weights);
 // choices from logits [T][ldl]
 int dc_launch_moe_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* logits, int ldl, int T, int32_t* ids, float* weights);
@@ -333,10 +380,11 @@ int dc_launch_moe_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* logits, i
 int dc_launch_moe_order(dc_ctx* ctx, const dc_moe_ffn& f, const int32_t* ids, const float* weights, int T, int32_t* off, int32_t* src, float* row_w,
                         int32_t* row);
 int dc_launch_moe_gather(dc_ctx* ctx, const __nv_bfloat16* x, int ldx, const int32_t* src, int rows, __nv_bfloat16* out);
-// up to DC_MAX_T tokens of bf16 models: hidden values of every assignment times its weight, then x += their products
+// up to DC_MAX_T tokens of bf16 models: hidden values of every assignment times its weight, then x = or += their products
 int dc_launch_moe_up_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* xb, int ldx, int T, const int32_t* ids, const float* weights,
                          __nv_bfloat16* hid, int ldh);
-int dc_launch_moe_down_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* hid, int ldh, int T, const int32_t* ids, int H, float* x, int ldx);
+int dc_launch_moe_down_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* hid, int ldh, int T, const int32_t* ids, int H, float* x, int ldx,
+                             bool add);
 // f32 models: sorted rows; src: input row of a row (null: itself)
 int dc_launch_moe_f32(dc_ctx* ctx, const dc_lin& w, int experts, int group_rows, const int32_t* off, int rows, const float* x, int ldx,
                       const int32_t* src, const dc_lin_epi& epi);
@@ -361,6 +409,14 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
                   int lda, float* small, float* blk, float* y, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ssd_decode(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* y, int ldy,
                          float eps, float* mix, __nv_bfloat16* mixb, int ldm);
+// generalized delta rule.  tanh: columns off_w .. of proj, to lowb or in place.  scan: entries of any length; low: decay
+// projections [T][ldd].  decode: one token per sequence, everything from the projections.
+size_t dc_general_block_floats(const dc_general_mixer& m);
+int dc_launch_general_tanh(dc_ctx* ctx, const dc_general_mixer& m, int T, float* proj, int ldp, __nv_bfloat16* lowb, int ldl);
+int dc_launch_general_scan(dc_ctx* ctx, const dc_general_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, const float* low,
+                           int ldd, float* blk, float eps, float* o, int ldo, float* mix, __nv_bfloat16* mixb, int ldm);
+int dc_launch_general_decode(dc_ctx* ctx, const dc_general_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
+                             float* mix, __nv_bfloat16* mixb, int ldm);
 int dc_launch_ring_update(dc_ctx* ctx, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, int off, int C, int taps);
 
 // lightning attention.  decode: one token per sequence.  scan: entries of any length in f32 (blocks of sixteen tokens).
@@ -386,15 +442,17 @@ struct dc_gqa_cache {
     int max_blocks = 0;
 };
 static inline int dc_gqa_ldq(const dc_gqa_mixer& m) { return (m.dim + 15) & ~15; }      // pitch of a turned query
-// norms, rotation, cache rows of the step's tokens; queries to q or qb [T][heads * maps][dc_gqa_ldq]
-int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
+// convolution, norms, rotation, cache rows of the step's tokens; queries to q or qb [T][heads * maps][dc_gqa_ldq].  sr: the
+// convolution's ring (null without one)
+int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const dc_state_ref* sr, const float* proj, int ldp, float eps,
                        int max_pos, float* q, __nv_bfloat16* qb);
-// every token alone: keys split over CTAs, then joined
-int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
-                         float* part_ml, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
+static inline int dc_gqa_conv_cols(const dc_gqa_mixer& m) { return m.off_v + m.kv_heads * m.vdim; }     // projection columns under the convolution
+// every token alone: keys split over CTAs, then joined.  proj: for the heads' gates
+int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, const float* proj, int ldp, int splits,
+                         float* part, float* part_ml, float eps, float* mix, __nv_bfloat16* mixb, int ldm);
 // prompts of bf16 models: tiles of queries over the cached rows
 int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const int32_t* tiles, int n_tiles,
-                         const __nv_bfloat16* qb, float eps, __nv_bfloat16* mixb, int ldm);
+                         const __nv_bfloat16* qb, const float* proj, int ldp, float eps, __nv_bfloat16* mixb, int ldm);
 
 // ---- mix_latent.cu
 struct dc_latent_cache {

@@ -1,4 +1,5 @@
-// Mixture of clamped gated experts with a sigmoid router whose choices are limited to groups of experts (dc_moe_ffn).
+// Mixture of experts (dc_moe_ffn): clamped gated ones, or the square of relu between two matrices, behind a sigmoid router whose
+// choices are limited to groups of experts, or a softmax router whose chosen scores are divided by their sum.
 //
 // Steps of up to DC_MAX_T tokens: k_moe_norm_route norms the residual and routes it (one cluster per token), k_moe_up_mma
 // streams the gate and up rows of the chosen experts, k_moe_down_mma streams their down rows, every distinct expert once,
@@ -21,7 +22,8 @@ namespace {
 struct RouteParams {
     int experts, top, groups, keep;
     float scale;
-    const float* correction;
+    bool softmax;
+    const float* correction;     // or null
     int32_t* ids;
     float* weights;
 };
@@ -31,8 +33,8 @@ __device__ __forceinline__ uint32_t ordered(float f) {      // order-preserving,
     return f != f ? 1u : (u & 0x80000000u) ? ~u : (u | 0x80000000u);
 }
 
-// One warp: the choices of a token.  score, correction: shared memory; PER: experts of a lane.  Equal scores: the lower index
-// first.
+// One warp: the choices of a token.  score (softmax: the logits), correction: shared memory; PER: experts of a lane.  Equal scores:
+// the lower index first.
 template <int PER>
 __device__ __forceinline__ void choose(const RouteParams& p, const float* score, const float* correction, int t, int lane) {
     uint32_t c[PER];             // choice of expert lane + 32 j; 0: not available
@@ -82,9 +84,19 @@ __device__ __forceinline__ void choose(const RouteParams& p, const float* score,
             if (lane + 32 * j == e) c[j] = 0u;
         if (lane == k) id = e;
     }
+    float w = score[id];
+    if (p.softmax) {
+        float m = -INFINITY, sum = 0.0f;
+        for (int e = lane; e < p.experts; e += 32) m = fmaxf(m, score[e]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        for (int e = lane; e < p.experts; e += 32) sum += expf(score[e] - m);
+        w = expf(w - m) / warp_sum(sum);
+        w /= warp_sum(lane < p.top ? w : 0.0f) + 1e-20f;
+    }
     if (lane < p.top) {
         p.ids[(size_t)t * p.top + lane] = id;
-        p.weights[(size_t)t * p.top + lane] = score[id] * p.scale;
+        p.weights[(size_t)t * p.top + lane] = w * p.scale;
     }
 }
 
@@ -93,12 +105,15 @@ template <int PER>
 __global__ void __launch_bounds__(128) k_moe_route(const RouteParams p, const float* __restrict__ logits, int ldl, int T) {
     __shared__ float score[4][32 * PER], correction[32 * PER];
     pdl_launch_dependents();
-    for (int e = threadIdx.x; e < p.experts; e += 128) correction[e] = p.correction[e];
+    for (int e = threadIdx.x; e < p.experts; e += 128) correction[e] = p.correction ? p.correction[e] : 0.0f;
     __syncthreads();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp;
     if (t >= T) return;
-    for (int e = lane; e < p.experts; e += 32) score[warp][e] = sigmoid(logits[(size_t)t * ldl + e]);
+    for (int e = lane; e < p.experts; e += 32) {
+        const float z = logits[(size_t)t * ldl + e];
+        score[warp][e] = p.softmax ? z : sigmoid(z);
+    }
     __syncwarp();
     choose<PER>(p, score[warp], correction, t, lane);
 }
@@ -106,6 +121,7 @@ __global__ void __launch_bounds__(128) k_moe_route(const RouteParams p, const fl
 // ---------------------------------------------------------------- norm and choices together
 struct NormRouteParams {
     RouteParams r;
+    dc_hyper hy;             // S > 0: where the row comes from
     const float *x, *w;
     const __nv_bfloat16* router;
     int ldw, H, ld;
@@ -116,11 +132,12 @@ struct NormRouteParams {
 
 constexpr int NR_CTAS = 8, NR_WARPS = 8, NR_AHEAD = 4;
 
-// A cluster per token: every CTA norms the row and takes its share of the experts, the first one chooses.
-template <int PER>
+// A cluster per token: every CTA norms the row and takes its share of the experts, the first one chooses.  S: streams at most
+// (0: the row is x).
+template <int PER, int S>
 __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRouteParams p) {
     extern __shared__ __align__(16) float h[];              // the normed row, padded with zeros to a multiple of 256
-    __shared__ float red[33], score[32 * PER], correction[32 * PER];
+    __shared__ float red[33], score[32 * PER], correction[32 * PER], coef[S ? S * (S + 2) : 1];
     asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");       // waited for ahead of the first remote store
     pdl_launch_dependents();
     const int rank = blockIdx.x % NR_CTAS, t = blockIdx.x / NR_CTAS, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -136,13 +153,19 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
     for (int e = e0 + warp; e < e1; e += NR_WARPS)          // the rest comes from L2
         for (int k = 64 * lane; k < K8; k += 64 * 32) prefetch_l2(p.router + (size_t)e * p.ldw + k);
     if (rank == 0)
-        for (int e = tid; e < p.r.experts; e += NR_WARPS * 32) correction[e] = p.r.correction[e];
+        for (int e = tid; e < p.r.experts; e += NR_WARPS * 32) correction[e] = p.r.correction ? p.r.correction[e] : 0.0f;
+    if constexpr (S > 0) {
+        hyper_coefficients<S>(p.hy, coef);
+        __syncthreads();
+    }
     pdl_wait();
     const int n4 = p.ld / 4;
     const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)t * p.ld);
     float ss = 0.0f;
     for (int i = tid; i < n4; i += NR_WARPS * 32) {
-        const float4 v = x4[i];
+        float4 v;
+        if constexpr (S > 0) v = hyper_column<S>(p.hy, coef, t, i, p.ld, reinterpret_cast<const float4*>(p.hy.y + (size_t)t * p.ld)[i], i % NR_CTAS == rank);
+        else v = x4[i];
         reinterpret_cast<float4*>(h)[i] = v;
         ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
     }
@@ -183,7 +206,8 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
                 a = fmaf(f[4], v.x, fmaf(f[5], v.y, fmaf(f[6], v.z, fmaf(f[7], v.w, a))));
             }
         }
-        a = sigmoid(warp_sum(a));
+        a = warp_sum(a);
+        if (!p.r.softmax) a = sigmoid(a);
         if (lane == 0) {
             uint32_t to;
             asm("mapa.shared::cluster.u32 %0, %1, 0;" : "=r"(to) : "r"(smem_u32(score + e)));
@@ -213,10 +237,10 @@ struct TileSizes {
     }
 };
 
-template <int PER>
+template <int PER, int S>
 __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const NormRouteParams p, int rows, int T) {
     extern __shared__ __align__(16) uint8_t sm[];
-    __shared__ float correction[32 * PER];
+    __shared__ float correction[32 * PER], coef[S ? S * (S + 2) : 1];
     const TileSizes z = TileSizes::of(p.r.experts, p.ld);
     __nv_bfloat16* h = reinterpret_cast<__nv_bfloat16*>(sm);            // [16][ldh]
     float* part = reinterpret_cast<float*>(sm + z.part);                // [shares][experts][17]
@@ -237,22 +261,33 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
     if (working)
 #pragma unroll
         for (int j = 0; j < NT_AHEAD; ++j) fetch(j, warp % z.tiles, begin + j);
-    for (int e = tid; e < p.r.experts; e += NT_WARPS * 32) correction[e] = p.r.correction[e];
+    for (int e = tid; e < p.r.experts; e += NT_WARPS * 32) correction[e] = p.r.correction ? p.r.correction[e] : 0.0f;
+    if constexpr (S > 0) {
+        hyper_coefficients<S>(p.hy, coef);
+        __syncthreads();
+    }
     pdl_wait();
     {
-        const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld);
+        auto row = [&](int i, bool store) {
+            if constexpr (S > 0) {
+                const int tc = min(t, T - 1);
+                return hyper_column<S>(p.hy, coef, tc, i, p.ld, reinterpret_cast<const float4*>(p.hy.y + (size_t)tc * p.ld)[i], store && t < T);
+            } else {
+                return reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld)[i];
+            }
+        };
         const float4* w4 = reinterpret_cast<const float4*>(p.w);
         uint2* to = reinterpret_cast<uint2*>(h + warp * z.ldh);
-        constexpr int KEEP = 16;             // groups of four that a lane holds; wider rows are read twice
+        constexpr int KEEP = S > 4 ? 4 : S > 2 ? 8 : 16;         // groups of four that a lane holds; wider rows are read twice
         float4 x[KEEP];
         float ss = 0.0f;
 #pragma unroll
-        for (int j = 0; j < KEEP; ++j) x[j] = lane + 32 * j < n4 ? x4[lane + 32 * j] : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int j = 0; j < KEEP; ++j) x[j] = lane + 32 * j < n4 ? row(lane + 32 * j, true) : make_float4(0.f, 0.f, 0.f, 0.f);
         auto square = [&](const float4& v) { ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); };
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) square(x[j]);
-#pragma unroll 8
-        for (int i = lane + 32 * KEEP; i < n4; i += 32) square(x4[i]);
+#pragma unroll (S > 0 ? 2 : 8)
+        for (int i = lane + 32 * KEEP; i < n4; i += 32) square(row(i, true));
         const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.H + p.eps);
         auto put = [&](int i, const float4& v) {
             uint2 r = make_uint2(0u, 0u);
@@ -265,8 +300,8 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
         };
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) put(lane + 32 * j, x[j]);
-#pragma unroll 8
-        for (int i = lane + 32 * KEEP; i < (z.ldh - 32) / 4; i += 32) put(i, i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f));
+#pragma unroll (S > 0 ? 2 : 8)
+        for (int i = lane + 32 * KEEP; i < (z.ldh - 32) / 4; i += 32) put(i, i < n4 ? row(i, false) : make_float4(0.f, 0.f, 0.f, 0.f));
     }
     __syncthreads();
     for (int tile = warp % z.tiles; working && tile < z.tiles; tile += z.shares > 1 ? z.tiles : NT_WARPS) {
@@ -300,7 +335,7 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
         const int e = i % E, tok = i / E;
         float v = 0.0f;
         for (int k = 0; k < z.shares; ++k) v += part[(size_t)(k * E + e) * 17 + tok];
-        score[tok * E + e] = sigmoid(v);
+        score[tok * E + e] = p.r.softmax ? v : sigmoid(v);
     }
     __syncthreads();
     if (t < T) choose<PER>(p.r, score + warp * E, correction, t, lane);
@@ -357,6 +392,7 @@ struct UpParams {
     const __nv_bfloat16* w;
     int K, ldw, rows, top, T, ff, experts;
     float limit;
+    bool plain;
     const __nv_bfloat16* x;
     int ldx;
     const int32_t* ids;
@@ -365,7 +401,7 @@ struct UpParams {
     int ldh;
 };
 
-// Gate and up rows of every distinct expert for its tokens: hidden value times routing weight.  A CTA walks over tiles of
+// Gate and up rows (plain: up rows) of every distinct expert for its tokens: hidden value times routing weight.  A CTA walks over tiles of
 // sixteen rows and fetches the next tile's first runs ahead of a tile's sum.
 template <int NT>
 __global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_up_mma(const UpParams p) {
@@ -433,7 +469,10 @@ __global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_up_mma(const UpParams 
         for (int i = 0; i < ME_WARPS; ++i) v += red[buf][i][r][t];
         const float up = __shfl_down_sync(0xffffffffu, v, 1);
         const int as = t < p.T ? units.asg[u][t] : -1;
-        if (!(r & 1) && as >= 0 && o < p.ff) {
+        if (p.plain) {
+            const int row = 16 * (tile - u * row_tiles) + r;
+            if (as >= 0 && row < p.ff) p.hid[(size_t)as * p.ldh + row] = __float2bfloat16_rn(relu2(v) * p.weights[as]);
+        } else if (!(r & 1) && as >= 0 && o < p.ff) {
             dc_lin_epi epi;
             epi.pair_kind = DC_PAIR_CLAMPED, epi.limit = p.limit;
             p.hid[(size_t)as * p.ldh + o] = __float2bfloat16_rn(pair_value(epi, v, up) * p.weights[as]);
@@ -449,9 +488,10 @@ struct DownParams {
     const int32_t* ids;
     float* x;
     int ldx;
+    bool add;
 };
 
-// x[t] += sum over the token's assignments of W_down hid.  The distinct experts' columns are one long row: a token has
+// x[t] = or += sum over the token's assignments of W_down hid.  The distinct experts' columns are one long row: a token has
 // zeros where an expert is not its own.  KS: CTAs of a cluster that share sixteen rows, each with its part of that row.
 template <int NT, int KS>
 __global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_down_mma(const DownParams p) {
@@ -523,7 +563,7 @@ __global__ void __launch_bounds__(ME_WARPS * 32, 2) k_moe_down_mma(const DownPar
 #pragma unroll
             for (int k = 0; k < KS - 1; ++k) v += other[k][tid];
     }
-    if (mine && t < p.T && row < p.H) p.x[(size_t)t * p.ldx + row] += v;
+    if (mine && t < p.T && row < p.H) p.x[(size_t)t * p.ldx + row] = p.add ? p.x[(size_t)t * p.ldx + row] + v : v;
 }
 
 // ---------------------------------------------------------------- many tokens: assignments sorted by expert
@@ -670,7 +710,7 @@ __global__ void __launch_bounds__(256) k_moe_f32(const F32Params p) {
 }
 
 RouteParams route_params(const dc_moe_ffn& f, int32_t* ids, float* weights) {
-    return RouteParams{f.experts, f.top, f.groups, f.keep, f.scale, f.correction, ids, weights};
+    return RouteParams{f.experts, f.top, f.groups, f.keep, f.scale, f.softmax, f.correction, ids, weights};
 }
 
 template <int NT, int KS>
@@ -683,29 +723,38 @@ int launch_down(dc_ctx* ctx, const DownParams& p) {
 
 }  // namespace
 
-int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const float* w, int T, int H, int ld, float eps, float* out,
+int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const dc_hyper* hy, const float* w, int T, int H, int ld, float eps, float* out,
                              __nv_bfloat16* outb, int32_t* ids, float* weights) {
     if (f.experts > DC_MOE_MAX_EXPERTS || f.groups > DC_MOE_MAX_GROUPS || ld % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad operand");
-    const NormRouteParams p = {route_params(f, ids, weights), x, w, f.router.w, f.router.ld, H, ld, eps, out, outb};
+    if (hy && (hy->streams > DC_MAX_STREAMS || hy->sum.k || !hy->y || !hy->x_out || hy->x == hy->x_out)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad streams");
+    const NormRouteParams p = {route_params(f, ids, weights), hy ? *hy : dc_hyper(), x, w, f.router.w, f.router.ld, H, ld, eps, out, outb};
     const size_t smem = (size_t)(ld + 255) / 256 * 256 * 4;
     const TileSizes z = TileSizes::of(f.experts, ld);
-#define DC_ROUTE(PER)                                                                                                                            \
+#define DC_ROUTE_S(PER, S)                                                                                                                       \
     do {                                                                                                                                         \
         if (T > DC_MAX_T) {                                                                                                                      \
-            const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route_tile<PER>, (int)z.bytes, "k_moe_norm_route_tile");                  \
+            const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route_tile<PER, S>, (int)z.bytes, "k_moe_norm_route_tile");               \
             if (st != DC_B200_OK) return st;                                                                                                     \
-            return dc_launch(ctx, "k_moe_norm_route_tile", k_moe_norm_route_tile<PER>, dim3((T + 15) / 16), dim3(NT_WARPS * 32), z.bytes, p,      \
+            return dc_launch(ctx, "k_moe_norm_route_tile", k_moe_norm_route_tile<PER, S>, dim3((T + 15) / 16), dim3(NT_WARPS * 32), z.bytes, p,   \
                              f.router.N, T);                                                                                                     \
         }                                                                                                                                        \
-        const int st = dc_kernel_setup_small(ctx, (const void*)k_moe_norm_route<PER>, (int)smem, "k_moe_norm_route");                                   \
+        const int st = dc_kernel_setup_small(ctx, (const void*)k_moe_norm_route<PER, S>, (int)smem, "k_moe_norm_route");                          \
         if (st != DC_B200_OK) return st;                                                                                                         \
-        return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route<PER>, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);       \
+        return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route<PER, S>, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);    \
+    } while (0)
+#define DC_ROUTE(PER)                                   \
+    do {                                                \
+        if (!hy) DC_ROUTE_S(PER, 0);                    \
+        if (hy->streams <= 2) DC_ROUTE_S(PER, 2);       \
+        if (hy->streams <= 4) DC_ROUTE_S(PER, 4);       \
+        DC_ROUTE_S(PER, DC_MAX_STREAMS);                \
     } while (0)
     if (f.experts <= 64) DC_ROUTE(2);
     if (f.experts <= 128) DC_ROUTE(4);
     if (f.experts <= 256) DC_ROUTE(8);
     DC_ROUTE(16);
 #undef DC_ROUTE
+#undef DC_ROUTE_S
 }
 
 bool dc_moe_norm_route_fits(const dc_moe_ffn& f, bool b16, int T, int ld) {
@@ -731,16 +780,17 @@ int dc_launch_moe_gather(dc_ctx* ctx, const __nv_bfloat16* x, int ldx, const int
 int dc_launch_moe_up_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* xb, int ldx, int T, const int32_t* ids, const float* weights,
                          __nv_bfloat16* hid, int ldh) {
     if (T < 1 || T > DC_MAX_T || ldx % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_up: bad operand");
-    const UpParams p = {f.up.w, f.up.K, f.up.ld, f.up_rows, f.top, T, f.ff, f.experts, f.limit, xb, ldx, ids, weights, hid, ldh};
+    const UpParams p = {f.up.w, f.up.K, f.up.ld, f.up_rows, f.top, T, f.ff, f.experts, f.limit, f.plain, xb, ldx, ids, weights, hid, ldh};
     const int tiles = f.up_rows / 16 * std::min(f.experts, T * f.top), room = 2 * ctx->num_sms, rounds = (tiles + room - 1) / room;
     const dim3 grid(T == 1 ? (tiles + rounds - 1) / rounds : std::min(tiles, room)), block(ME_WARPS * 32);
     if (T <= 8) return dc_launch(ctx, "k_moe_up_mma", k_moe_up_mma<1>, grid, block, 0, p);
     return dc_launch(ctx, "k_moe_up_mma", k_moe_up_mma<2>, grid, block, 0, p);
 }
 
-int dc_launch_moe_down_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* hid, int ldh, int T, const int32_t* ids, int H, float* x, int ldx) {
+int dc_launch_moe_down_mma(dc_ctx* ctx, const dc_moe_ffn& f, const __nv_bfloat16* hid, int ldh, int T, const int32_t* ids, int H, float* x, int ldx,
+                             bool add) {
     if (T < 1 || T > DC_MAX_T || ldh % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_down: bad operand");
-    const DownParams p = {f.down.w, f.down.K, f.down.ld, f.down_rows, f.top, T, H, f.experts, hid, ldh, ids, x, ldx};
+    const DownParams p = {f.down.w, f.down.K, f.down.ld, f.down_rows, f.top, T, H, f.experts, hid, ldh, ids, x, ldx, add};
     // fewer row tiles than SMs: the long rows are shared by a cluster
     const int tiles = f.down_rows / 16;
     if (2 * tiles <= ctx->num_sms) return T <= 8 ? launch_down<1, 4>(ctx, p) : launch_down<2, 4>(ctx, p);

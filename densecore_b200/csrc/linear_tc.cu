@@ -91,7 +91,7 @@ __device__ __forceinline__ void transpose8(const uint32_t (&r)[N], uint32_t (&ou
 }
 
 // Accumulators of a tile (rows: tensor-memory lanes, tokens: columns) to the output; a warp reads its quarter's lanes.  Grouped
-// products end in clamped pairs with a factor per token or in bf16 rows.
+// products end in clamped pairs or the rows' squares of relu, both with a factor per token, or in bf16 rows.
 template <int COLS, bool GROUPED>
 __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int row0, int t0, int t1, int quarter, int lane) {
     const int row = row0 + 32 * quarter + lane, n = t1 - t0;
@@ -99,7 +99,7 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
     tmem += (uint32_t)(32 * quarter) << 16;
     if (row0 + 32 * quarter >= e.pair0) {
         // lanes 2i (gate row) and 2i + 1 (up row) share one output row: each finishes eight tokens
-        const bool up = lane & 1, gelu = !GROUPED && e.pair_kind == DC_PAIR_GELU;
+        const bool up = lane & 1, gelu = !GROUPED && e.pair_kind == DC_PAIR_GELU, swish = !GROUPED && e.pair_kind == DC_PAIR_SILU;
         const int o = (row - e.pair0) >> 1, first = up ? 8 : 0;
         const bool in = o < e.n_pairs;
         const size_t at = (size_t)(t0 + first) * e.ldp + o;
@@ -113,7 +113,7 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
                 const float got = __int_as_float(__shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1));
                 const float mine = __int_as_float(up ? v[i + 8] : v[i]);
                 const float gate = up ? got : mine, val = up ? mine : got;
-                h[i] = (gelu ? gelu_tanh(gate) * val : quick_clamped(e.limit, gate, val)) * f[i];
+                h[i] = (gelu ? gelu_tanh(gate) * val : swish ? quick_silu(gate) * val : quick_clamped(e.limit, gate, val)) * f[i];
             }
             const int m = in ? n - c0 - first : 0;
             if (wide) {
@@ -141,10 +141,16 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
     const float bias = !GROUPED && in && e.bias ? e.bias[row] : 0.0f;
     const size_t at = (size_t)t0 * e.ldo + row;
     if (e.outb && e.n_store % 8 == 0 && e.ldo % 8 == 0 && ((uintptr_t)e.outb & 15) == 0) {       // whole groups of eight rows
-        const bool act = !GROUPED && row < e.silu_rows;
+        const bool act = !GROUPED && row < e.act_rows;
         const int tok = 2 * ((lane & 2 ? 4 : 0) + (lane & 4 ? 2 : 0)) + (lane & 1);
         each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
             uint32_t r[8], v8[2][4];
+            if (GROUPED && e.act_rows) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                    r[i] = pack_bf2(relu2(__int_as_float(v[2 * i])) * e.tok_scale[min(t0 + c0 + 2 * i, t1 - 1)],
+                                    relu2(__int_as_float(v[2 * i + 1])) * e.tok_scale[min(t0 + c0 + 2 * i + 1, t1 - 1)]);
+            } else
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const float a = __int_as_float(v[2 * i]) + bias, b = __int_as_float(v[2 * i + 1]) + bias;
@@ -158,14 +164,14 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
                     *reinterpret_cast<uint4*>(e.outb + at + (size_t)(c0 + tok + 2 * i) * e.ldo - (lane & 7)) = make_uint4(v8[i][0], v8[i][1], v8[i][2], v8[i][3]);
         });
     } else if (GROUPED || e.outb) {
-        const bool act = !GROUPED && row < e.silu_rows;
+        const bool act = row < e.act_rows;
         each16<COLS>(tmem, n, [&](int (&v)[16], int c0) {
             const int m = in ? n - c0 : 0;
             __nv_bfloat16* to = e.outb + at + (size_t)c0 * e.ldo;
 #pragma unroll
             for (int i = 0; i < 16; ++i, to += e.ldo) {
                 const float r = __int_as_float(v[i]) + bias;
-                if (i < m) *to = __float2bfloat16_rn(act ? quick_silu(r) : r);
+                if (i < m) *to = __float2bfloat16_rn(!act ? r : GROUPED ? relu2(r) * e.tok_scale[t0 + c0 + i] : quick_silu(r));
             }
         });
     } else if (e.add) {
@@ -468,7 +474,8 @@ int dc_lin_encode(dc_ctx* ctx, CUtensorMap* map, const __nv_bfloat16* base, int 
 
 int dc_launch_linear_tc(dc_ctx* ctx, const dc_lin& w, const dc_tc_in& x, int T, const dc_lin_epi& epi) {
     if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: inner sizes %d and %d differ", w.K, x.K);
-    if (epi.keys || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: epilogue not available");
+    if (epi.keys || epi.tok_scale || (epi.act_rows && epi.act != DC_ACT_SILU) || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN))
+        return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_tc: epilogue not available");
     LtParams p = {w.K, T, epi, ctx->d_err};
     p.e.n_store = std::min(epi.n_store, std::min(w.N, epi.pair0));
     p.e.n_pairs = std::max(0, std::min(epi.n_pairs, (w.N - epi.pair0) / 2));
@@ -489,7 +496,7 @@ int dc_launch_linear_grouped_tc(dc_ctx* ctx, const dc_lin& w, int groups, int gr
                                 const dc_lin_epi& epi) {
     if (w.K != x.K) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: inner sizes %d and %d differ", w.K, x.K);
     if (groups < 1 || groups > DC_MOE_MAX_EXPERTS || groups * group_rows != w.N || max_rows < 1) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: bad groups");
-    const bool pairs = epi.pair0 == 0 && epi.pair_kind == DC_PAIR_CLAMPED && epi.poutb && epi.tok_scale, rows = epi.pair0 >= (1 << 30) && epi.outb && !epi.bias && !epi.silu_rows;
+    const bool pairs = epi.pair0 == 0 && epi.pair_kind == DC_PAIR_CLAMPED && epi.poutb && epi.tok_scale, rows = epi.pair0 >= (1 << 30) && epi.outb && !epi.bias && (epi.act_rows ? epi.act == DC_ACT_RELU2 && epi.act_rows >= group_rows && epi.tok_scale : !epi.tok_scale);
     if (epi.keys || epi.add || !(pairs || rows) || (epi.pair0 < (1 << 30) && epi.pair0 % DC_PAIR_ALIGN)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "linear_grouped_tc: epilogue not available");
     LtParams p = {w.K, max_rows, epi, ctx->d_err};
     p.e.n_store = std::min(epi.n_store, std::min(group_rows, epi.pair0));

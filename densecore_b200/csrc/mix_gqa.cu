@@ -1,7 +1,8 @@
 // Grouped-query attention with its variants: a sliding window with or without the sequence's first tokens kept in sight, a
-// soft cap on the scores, a sink in the softmax' denominator, norms of queries and keys over the whole projection or per
-// head, rotation of neighbouring or of half-distant pairs, values of their own or the key projection before norm and
-// rotation, and two maps per head whose outputs are subtracted.
+// soft cap on the scores, a sink in the softmax' denominator, unnormalized sigmoid weights instead of a softmax, short
+// convolutions ahead of everything, norms of queries and keys over the whole projection or per head, norms of values, rotation of
+// neighbouring or of half-distant pairs, values of their own or the key projection before norm and rotation, two maps per head
+// whose outputs are subtracted, and a gate per head.
 //
 // A cached token is one row: the turned keys of all key heads (and maps), then the values.  Steps of up to DC_MAX_T tokens
 // and f32 models take every token alone (k_gqa_tokens: keys split over CTAs, k_gqa_join); prompt-sized steps of bf16
@@ -255,6 +256,118 @@ __global__ void __launch_bounds__(256) k_gqa_prep_heads4(const HeadsParams p) {
     }
 }
 
+// Convolution and norms, no rotation: a warp takes a head of the queries, keys or values through a few tokens of an entry, a lane the
+// dimensions lane, lane + 32, ...  The inputs ahead of the portion come from the sequence's ring.  TAPS: taps at most, 0: any number.
+struct ConvParams {
+    HeadsParams h;
+    ConvRef cr;
+    const float* conv;       // [taps][cr.ldw]
+    bool q_unit, k_unit, v_unit, put_ring;      // put_ring: every entry is one token, whose input goes into the ring here
+};
+constexpr int conv_portion(int vp) { return vp <= 4 ? 8 : 4; }
+
+template <typename TC, int VP, int TAPS>
+__global__ void __launch_bounds__(256) k_gqa_prep_conv(const ConvParams p) {
+    pdl_launch_dependents();
+    const HeadsParams& a = p.h;
+    const int lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5), taps = p.cr.taps;
+    if (u >= a.nq + a.nk + a.nv) return;
+    const bool query = u < a.nq, value = u >= a.nq + a.nk;
+    const int head = query ? u : value ? u - a.nq - a.nk : u - a.nq, n = value ? a.vdim : a.dim;
+    const int col0 = (query ? a.off_q : value ? a.off_v : a.off_k) + head * n;
+    const float* nw = value ? nullptr : query ? a.q_norm : a.k_norm;
+    const bool unit = query ? p.q_unit : value ? p.v_unit : p.k_unit;
+    constexpr int WN = TAPS > 0 ? TAPS : 1, PB = conv_portion(VP);
+    float w[VP][WN];             // the last taps first: w[j][WN - 1] is the token's own
+#pragma unroll
+    for (int j = 0; j < VP; ++j)
+#pragma unroll
+        for (int k = 0; k < WN; ++k) {
+            const int tap = taps - WN + k;
+            w[j][k] = TAPS > 0 && tap >= 0 && lane + 32 * j < n ? p.conv[(size_t)tap * p.cr.ldw + col0 + lane + 32 * j] : 0.0f;
+        }
+    pdl_wait();
+    const BlockRef br = block_at<PB>(p.cr.starts, p.cr.E, blockIdx.x);
+    if (br.n <= 0) return;
+    const int i0 = br.t0 - p.cr.starts[br.e], pos0 = p.cr.positions[br.t0], seq = p.cr.seq_ids[br.t0];
+    float* ring = p.cr.ring(seq);
+    float x[PB][VP], h[VP][WN > 1 ? WN - 1 : 1];
+#pragma unroll
+    for (int i = 0; i < PB; ++i)
+#pragma unroll
+        for (int j = 0; j < VP; ++j) {
+            const int d = lane + 32 * j;
+            x[i][j] = i < br.n && d < n ? a.proj[(size_t)(br.t0 + i) * a.ldp + col0 + d] : 0.0f;
+        }
+    if (TAPS > 1) {
+#pragma unroll
+        for (int j = 0; j < VP; ++j)
+#pragma unroll
+            for (int k = 0; k < WN - 1; ++k) {
+                const int back = WN - 1 - k, d = lane + 32 * j;
+                h[j][k] = 0.0f;
+                if (back < taps && pos0 >= back && d < n)
+                    h[j][k] = back <= i0 ? a.proj[(size_t)(br.t0 - back) * a.ldp + col0 + d] : ring[(size_t)((pos0 - back) % taps) * p.cr.C + col0 + d];
+            }
+    }
+    if (p.put_ring)              // a row that no tap of this token reads
+#pragma unroll
+        for (int j = 0; j < VP; ++j)
+            if (lane + 32 * j < n) ring[(size_t)(pos0 % taps) * p.cr.C + col0 + lane + 32 * j] = x[0][j];
+    float y[PB][VP], ss[PB];
+#pragma unroll
+    for (int i = 0; i < PB; ++i) {
+        ss[i] = 0.0f;
+#pragma unroll
+        for (int j = 0; j < VP; ++j) {
+            const int d = lane + 32 * j;
+            if (TAPS > 0) {
+                float s = 0.0f;
+#pragma unroll
+                for (int k = 0; k < WN - 1; ++k) s = fmaf(w[j][k], h[j][k], s);
+                y[i][j] = fmaf(w[j][WN - 1], x[i][j], s);
+#pragma unroll
+                for (int k = 0; k + 1 < WN - 1; ++k) h[j][k] = h[j][k + 1];
+                if (TAPS > 1) h[j][WN > 1 ? WN - 2 : 0] = x[i][j];
+            } else {
+                y[i][j] = i < br.n && d < n ? conv_at(a.proj, a.ldp, ring, p.cr.C, col0 + d, taps, p.conv + col0 + d, p.cr.ldw, col0 + d, br.t0 + i, i0 + i, pos0 + i) : 0.0f;
+            }
+            ss[i] = fmaf(y[i][j], y[i][j], ss[i]);
+        }
+    }
+    if (unit) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int i = 0; i < PB; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+    }
+    const int pitch = query ? a.ldq : value ? a.vdim_p : a.dim_p;
+#pragma unroll
+    for (int i = 0; i < PB; ++i) {
+        if (i >= br.n) break;
+        const float inv = unit ? 1.0f / sqrtf(ss[i] / (float)n + a.eps) : 1.0f;
+        const int t = br.t0 + i, pos = min(pos0 + i, a.max_pos - 1);
+        TC* cache = query ? nullptr : reinterpret_cast<TC*>(a.c.arena) + a.c.at(seq, pos) + (value ? a.v_at + head * a.vdim_p : head * a.dim_p);
+#pragma unroll
+        for (int j = 0; j < VP; ++j) {
+            const int d = lane + 32 * j;
+            if (d >= pitch) break;
+            const float r = y[i][j] * inv * (nw && d < n ? nw[d] : 1.0f);       // zero in the padding
+            const size_t at = ((size_t)t * a.nq + head) * pitch + d;
+            if (!query) store_as(cache + d, r);
+            else if (a.qb) store_as(a.qb + at, r);
+            else a.q[at] = r;
+        }
+    }
+}
+
+template <typename TC, int VP>
+int launch_prep_conv(dc_ctx* ctx, const ConvParams& p, const dc_step& st) {
+    const dim3 grid(st.single ? st.T : st.T / conv_portion(VP) + st.E, (p.h.nq + p.h.nk + p.h.nv + 7) / 8);
+    if (p.cr.taps <= 4) return dc_launch(ctx, "k_gqa_prep_conv", k_gqa_prep_conv<TC, VP, 4>, grid, dim3(256), 0, p);
+    return dc_launch(ctx, "k_gqa_prep_conv", k_gqa_prep_conv<TC, VP, 0>, grid, dim3(256), 0, p);
+}
+
 // ---------------------------------------------------------------- every token alone
 // The keys that a token sees, in order: the kept first ones that its window has left behind, then the window.
 struct Keys {
@@ -275,6 +388,7 @@ struct TokenParams {
     float scale, softcap;
     const int32_t *seq_ids, *positions;
     CacheRef c;
+    const float* score_bias; // sigmoid weights; or null: softmax
     float *part, *part_ml;   // [T][heads * MAPS][splits][vdim], [T][heads * MAPS][splits][2]
 };
 
@@ -295,6 +409,7 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
     const int s = blockIdx.x, g = blockIdx.y / p.groups, t = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int unit = (blockIdx.y % p.groups) * TK_HEADS + warp, map = unit % MAPS, h = g * p.per * MAPS + unit, pos = p.positions[t], seq = p.seq_ids[t];
     const bool live = unit < p.per * MAPS;
+    const float bias = p.score_bias && live ? p.score_bias[h] : 0.0f;
     const Keys keys = keys_of(pos, pos, p.window, p.keep);
     const int per = ((keys.n + p.splits - 1) / p.splits + TK_KEYS - 1) / TK_KEYS * TK_KEYS;
     const int kb = s * per, ke = min(keys.n, kb + per);
@@ -335,14 +450,20 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
         for (int i = 0; i < EPC; ++i) sc += part[i];
         if (p.softcap > 0.0f) sc = p.softcap * tanhf(sc / p.softcap);
         if (k0 + lane >= ke) sc = -INFINITY;
-        float mx = sc;
+        float pr;
+        if (p.score_bias) {
+            pr = k0 + lane < ke ? sigmoid(sc + bias) : 0.0f;
+        } else {
+            float mx = sc;
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        const float mn = fmaxf(m, mx), corr = expf(m - mn), pr = expf(sc - mn);
-        m = mn;
-        l = l * corr + warp_sum(pr);
+            for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float mn = fmaxf(m, mx), corr = expf(m - mn);
+            pr = expf(sc - mn);
+            m = mn;
+            l = l * corr + warp_sum(pr);
 #pragma unroll
-        for (int j = 0; j < VP; ++j) acc[j][0] *= corr, acc[j][1] *= corr;
+            for (int j = 0; j < VP; ++j) acc[j][0] *= corr, acc[j][1] *= corr;
+        }
 #pragma unroll 8
         for (int kk = 0; kk < TK_KEYS; ++kk) {
             const float w = __shfl_sync(0xffffffffu, pr, kk);
@@ -356,7 +477,7 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
     }
     if (!live) return;
     const size_t o = ((size_t)t * p.heads * MAPS + h) * p.splits + s;
-    if (lane == 0) {
+    if (lane == 0 && !p.score_bias) {
         p.part_ml[2 * o] = m;
         p.part_ml[2 * o + 1] = l;
     }
@@ -369,20 +490,22 @@ __global__ void __launch_bounds__(TK_HEADS * 32) k_gqa_tokens(const TokenParams 
         }
 }
 
-// Splits of one (head, token) and the sink joined; with two maps the second is taken off the first and the rest normed.  Every
-// fourth split is a warpgroup's.
+// Splits of one (head, token) and the sink joined; with two maps the second is taken off the first and the rest normed.  part_ml
+// null: the splits' plain sum.  gate: the head's, or null.  Every fourth split is a warpgroup's.
 constexpr int JOIN_PARTS = 4;
 template <int MAPS>
 __global__ void __launch_bounds__(128 * JOIN_PARTS) k_gqa_join(const float* __restrict__ part, const float* __restrict__ part_ml, int heads, int splits, int vdim,
-                                                               float sink, float lambda, float mul, float eps, float* __restrict__ mix,
-                                                               __nv_bfloat16* __restrict__ mixb, int ldm) {
+                                                               float sink, float lambda, float mul, float eps, const float* __restrict__ gate, int ldg,
+                                                               float* __restrict__ mix, __nv_bfloat16* __restrict__ mixb, int ldm) {
     __shared__ float sw[MAPS][DC_MAX_SPLITS], red[33], sum[JOIN_PARTS - 1][256];
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, share = threadIdx.x >> 7, d0 = threadIdx.x & 127;
     const size_t o = ((size_t)t * heads + h) * MAPS * splits;
     float x[2][MAPS][DC_MAX_SPLITS / JOIN_PARTS];         // vdim <= 256
-    if (warp < MAPS) join_weights(part_ml + 2 * (o + warp * splits), splits, lane, sink, warp ? -lambda : 1.0f, sw[warp]);
+    if (!part_ml) {
+        if (threadIdx.x < DC_MAX_SPLITS) sw[0][threadIdx.x] = 1.0f;
+    } else if (warp < MAPS) join_weights(part_ml + 2 * (o + warp * splits), splits, lane, sink, warp ? -lambda : 1.0f, sw[warp]);
     float v[2] = {0.0f, 0.0f}, ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < 2; ++j)
@@ -407,7 +530,8 @@ __global__ void __launch_bounds__(128 * JOIN_PARTS) k_gqa_join(const float* __re
 #pragma unroll
         for (int k = 0; k < JOIN_PARTS - 1; ++k) v[0] += sum[k][d0], v[1] += sum[k][d0 + 128];
     ss = v[0] * v[0] + v[1] * v[1];
-    const float f = MAPS > 1 ? mul / sqrtf(block_sum(ss, red) / (float)vdim + eps) : 1.0f;
+    float f = MAPS > 1 ? mul / sqrtf(block_sum(ss, red) / (float)vdim + eps) : 1.0f;
+    if (gate) f *= sigmoid(gate[(size_t)t * ldg + h]);
     if (share > 0) return;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -440,6 +564,9 @@ struct PromptParams {
     int ldq, heads, per, dim, vdim, dim_p, vdim_p, v_at, window, keep;
     float scale, softcap, sink;
     float lambda, mul, eps;  // two maps
+    const float* score_bias; // sigmoid weights
+    const float* gate;       // [T][ldg] per head, or null
+    int ldg;
     const int32_t *seq_ids, *positions, *starts, *tiles;     // tiles: (entry, first query of the entry) pairs
     CacheRef c;
     __nv_bfloat16* out;
@@ -454,8 +581,8 @@ __device__ __forceinline__ float soft_cap(float z, float cap) {
 }
 
 // One CTA per (QT = PQ / MAPS queries of one entry, head), sixteen rows (queries of one map) a warp; key and value tiles in
-// a ring of ST stages, two CTAs an SM.  DP, VP: key and value size, padded.
-template <int DP, int VP, int PQ, int ST, int MAPS>
+// a ring of ST stages, two CTAs an SM.  DP, VP: key and value size, padded.  SIGMOID: sigmoid weights, no denominator.
+template <int DP, int VP, int PQ, int ST, int MAPS, bool SIGMOID>
 __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const PromptParams p) {
     constexpr int LD = DP + 8, LDK = MAPS * DP + 8, LDV = VP + 8, NT = 2 * PQ, CH = DP / 8, VCH = VP / 8, QT = PQ / MAPS;
     extern __shared__ __align__(16) uint8_t smem[];
@@ -521,6 +648,7 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
     float o[VCH][4];
 #pragma unroll
     for (int i = 0; i < VCH; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    const float bias2 = SIGMOID ? p.score_bias[head] * 1.4426950408889634f : 0.0f;
     // the sink is the first term of the sum (one lane of a row's four counts it)
     const bool sink = p.sink > -INFINITY;
     float m_run[2], l_run[2];
@@ -558,6 +686,12 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
 #pragma unroll
                 for (int j = 0; j < 4; ++j) s[nt][j] = soft_cap(s[nt][j] * to_cap, cap);
         }
+        if constexpr (SIGMOID) {
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) s[nt][j] = __fdividef(1.0f, 1.0f + ex2(-fmaf(s[nt][j], sl2, bias2)));
+        }
         // the warp's sixteen queries see the whole tile, or the mask decides key by key
         if (!(k1 <= wq0 && wq0 + 15 - k0 < window)) {
 #pragma unroll
@@ -565,43 +699,45 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     const int kp = keys.at(tile * PK + 8 * nt + 2 * t4 + (j & 1)), qp = qpos0 + (j >> 1) * 8;
-                    if (!(kp <= qp && (qp - kp < window || kp < p.keep))) s[nt][j] = -INFINITY;
+                    if (!(kp <= qp && (qp - kp < window || kp < p.keep))) s[nt][j] = SIGMOID ? 0.0f : -INFINITY;
                 }
         }
-        float mx[2] = {-1e30f, -1e30f};
+        if constexpr (!SIGMOID) {
+            float mx[2] = {-1e30f, -1e30f};
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) {
-            mx[0] = fmaxf(mx[0], fmaxf(s[nt][0], s[nt][1]));
-            mx[1] = fmaxf(mx[1], fmaxf(s[nt][2], s[nt][3]));
-        }
-        float m_new[2];
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-            m_new[h] = fmaxf(m_run[h], mx[h] * sl2);
-        }
-        if (__any_sync(0xffffffffu, m_new[0] > m_run[0] || m_new[1] > m_run[1])) {
+            for (int nt = 0; nt < 8; ++nt) {
+                mx[0] = fmaxf(mx[0], fmaxf(s[nt][0], s[nt][1]));
+                mx[1] = fmaxf(mx[1], fmaxf(s[nt][2], s[nt][3]));
+            }
+            float m_new[2];
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
-                const float corr = ex2(m_run[h] - m_new[h]);
-                m_run[h] = m_new[h];
-                l_run[h] *= corr;
+                mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+                mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+                m_new[h] = fmaxf(m_run[h], mx[h] * sl2);
+            }
+            if (__any_sync(0xffffffffu, m_new[0] > m_run[0] || m_new[1] > m_run[1])) {
 #pragma unroll
-                for (int i = 0; i < VCH; ++i) {
-                    o[i][2 * h] *= corr;
-                    o[i][2 * h + 1] *= corr;
+                for (int h = 0; h < 2; ++h) {
+                    const float corr = ex2(m_run[h] - m_new[h]);
+                    m_run[h] = m_new[h];
+                    l_run[h] *= corr;
+#pragma unroll
+                    for (int i = 0; i < VCH; ++i) {
+                        o[i][2 * h] *= corr;
+                        o[i][2 * h + 1] *= corr;
+                    }
                 }
             }
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float w = ex2(fmaf(s[nt][j], sl2, -m_run[j >> 1]));
+                    s[nt][j] = w;
+                    l_run[j >> 1] += w;
+                }
         }
-#pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const float w = ex2(fmaf(s[nt][j], sl2, -m_run[j >> 1]));
-                s[nt][j] = w;
-                l_run[j >> 1] += w;
-            }
         const uint32_t va = smem_u32(sV + (buf * PK + (mi & 1) * 8 + r8) * LDV + (mi >> 1) * 8);
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks) {
@@ -624,7 +760,8 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
         l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
         l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
     }
-    float mul[2] = {1.0f / l_run[0], 1.0f / l_run[1]};
+    float mul[2] = {1.0f, 1.0f};
+    if (!SIGMOID) mul[0] = 1.0f / l_run[0], mul[1] = 1.0f / l_run[1];
     if (MAPS > 1) {
         constexpr int LDX = VP + 4;
         float* other = reinterpret_cast<float*>(smem);              // [QT][LDX]: the second map's answers
@@ -658,6 +795,7 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
     for (int h = 0; h < 2; ++h) {
         const int row = q0 + qrow + g + 8 * h;
         if (row >= n) continue;
+        if (p.gate) mul[h] *= sigmoid(p.gate[(size_t)(t0 + row) * p.ldg + head]);
         __nv_bfloat16* dst = p.out + (size_t)(t0 + row) * p.ldm + (size_t)head * p.vdim;
 #pragma unroll
         for (int nt = 0; nt < VCH; ++nt)
@@ -669,13 +807,13 @@ __global__ void __launch_bounds__(2 * PQ, PQ == 128 ? 2 : 1) k_gqa_prompt(const 
     }
 }
 
-template <int DP, int VP, int PQ, int ST, int MAPS>
+template <int DP, int VP, int PQ, int ST, int MAPS, bool SIGMOID>
 int launch_prompt(dc_ctx* ctx, const PromptParams& p, int n_tiles) {
     constexpr int QT = PQ / MAPS, bytes = (PQ * (DP + 8) + ST * PK * (MAPS * DP + VP + 16)) * 2;
     static_assert(bytes <= 227 * 1024 && (MAPS == 1 || QT * (VP + 4) * 4 <= bytes), "shared memory");
-    DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_prompt<DP, VP, PQ, ST, MAPS>, bytes, "k_gqa_prompt"));
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_gqa_prompt<DP, VP, PQ, ST, MAPS, SIGMOID>, bytes, "k_gqa_prompt"));
     const dim3 grid(n_tiles, p.heads, QT < DC_LATENT_QTILE ? DC_LATENT_QTILE / QT : 1);
-    return dc_launch(ctx, "k_gqa_prompt", k_gqa_prompt<DP, VP, PQ, ST, MAPS>, grid, dim3(2 * PQ), (size_t)bytes, p);
+    return dc_launch(ctx, "k_gqa_prompt", k_gqa_prompt<DP, VP, PQ, ST, MAPS, SIGMOID>, grid, dim3(2 * PQ), (size_t)bytes, p);
 }
 
 CacheRef cache_ref(const dc_gqa_cache& c, int row) { return CacheRef{c.arena, c.tables, c.max_blocks, row}; }
@@ -683,8 +821,23 @@ float sink_of(const dc_gqa_mixer& m) { return m.sink ? m.sink_score : -INFINITY;
 
 }  // namespace
 
-int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* proj, int ldp, float eps,
-                       int max_pos, float* q, __nv_bfloat16* qb) {
+int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const dc_state_ref* sr, const float* proj,
+                       int ldp, float eps, int max_pos, float* q, __nv_bfloat16* qb) {
+    if (m.taps > 0) {
+        if (!sr || m.rot.dims || m.qk_norm == DC_QK_NORM_ALL || m.off_v == m.off_k) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prep: form not available with convolutions");
+        const int C = dc_gqa_conv_cols(m);
+        ConvParams p = {{proj, ldp, m.off_q, m.off_k, m.off_v, m.heads * m.maps, m.kv_heads * m.maps, m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at,
+                         dc_gqa_ldq(m), 0, 0, max_pos, m.q_norm, m.k_norm, nullptr, eps, st.seq_ids, st.positions, cache_ref(c, m.row), q, qb},
+                        {sr->base, sr->slot_bytes, sr->ring_off, st.seq_ids, st.positions, st.starts, st.E, m.taps, C, C}, m.conv,
+                        m.qk_norm == DC_QK_NORM_HEAD, m.qk_norm == DC_QK_NORM_HEAD, m.v_norm, st.single};
+        const int most = std::max(std::max(p.h.ldq, p.h.dim_p), p.h.vdim_p);
+#define DC_CONV(VP) DC_TRY((c.f32 ? launch_prep_conv<float, VP>(ctx, p, st) : launch_prep_conv<__nv_bfloat16, VP>(ctx, p, st)))
+        if (most <= 64) DC_CONV(2);
+        else if (most <= 128) DC_CONV(4);
+        else DC_CONV(8);
+#undef DC_CONV
+        return st.single ? DC_B200_OK : dc_launch_ring_update(ctx, st, *sr, proj, ldp, 0, C, m.taps);
+    }
     if (m.qk_norm != DC_QK_NORM_ALL) {
         if (m.off_v == m.off_k) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prep: values from the keys need the norm over all heads");
         HeadsParams p = {proj, ldp, m.off_q, m.off_k, m.off_v, m.heads * m.maps, m.kv_heads * m.maps, m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at,
@@ -720,28 +873,33 @@ int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, co
     return dc_launch(ctx, "k_gqa_prep", k_gqa_prep<__nv_bfloat16>, grid, block, 0, p);
 }
 
-int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, int splits, float* part,
-                         float* part_ml, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
+int dc_launch_gqa_tokens(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const float* q, const float* proj, int ldp, int splits,
+                         float* part, float* part_ml, float eps, float* mix, __nv_bfloat16* mixb, int ldm) {
+    const float* gate = m.off_g < 0 ? nullptr : proj + m.off_g;
+    const float* ml = m.score_bias ? nullptr : part_ml;
+    if (m.score_bias && (m.maps > 1 || m.sink)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_tokens: form not available with sigmoid weights");
     const int per = m.heads / m.kv_heads;
     TokenParams p = {q, dc_gqa_ldq(m), m.heads, per, (per * m.maps + TK_HEADS - 1) / TK_HEADS, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at, m.window, m.keep, splits,
-                     m.scale, m.softcap, st.seq_ids, st.positions, cache_ref(c, m.row), part, part_ml};
+                     m.scale, m.softcap, st.seq_ids, st.positions, cache_ref(c, m.row), m.score_bias, part, part_ml};
     if (m.maps > 1) {
         DC_TRY((c.f32 ? launch_tokens<float, 2>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16, 2>(ctx, p, m.kv_heads, st.T)));
-        return dc_launch(ctx, "k_gqa_join", k_gqa_join<2>, dim3(m.heads, st.T), dim3(128 * JOIN_PARTS), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), m.lambda,
-                         1.0f - m.diff, eps, mix, mixb, ldm);
+        return dc_launch(ctx, "k_gqa_join", k_gqa_join<2>, dim3(m.heads, st.T), dim3(128 * JOIN_PARTS), 0, part, ml, m.heads, splits, m.vdim, sink_of(m), m.lambda,
+                         1.0f - m.diff, eps, gate, ldp, mix, mixb, ldm);
     }
     DC_TRY((c.f32 ? launch_tokens<float, 1>(ctx, p, m.kv_heads, st.T) : launch_tokens<__nv_bfloat16, 1>(ctx, p, m.kv_heads, st.T)));
-    return dc_launch(ctx, "k_gqa_join", k_gqa_join<1>, dim3(m.heads, st.T), dim3(128 * JOIN_PARTS), 0, part, part_ml, m.heads, splits, m.vdim, sink_of(m), 0.0f, 1.0f, eps, mix,
-                     mixb, ldm);
+    return dc_launch(ctx, "k_gqa_join", k_gqa_join<1>, dim3(m.heads, st.T), dim3(128 * JOIN_PARTS), 0, part, ml, m.heads, splits, m.vdim, sink_of(m), 0.0f, 1.0f, eps,
+                     gate, ldp, mix, mixb, ldm);
 }
 
 int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, const dc_gqa_cache& c, const int32_t* tiles, int n_tiles,
-                         const __nv_bfloat16* qb, float eps, __nv_bfloat16* mixb, int ldm) {
+                         const __nv_bfloat16* qb, const float* proj, int ldp, float eps, __nv_bfloat16* mixb, int ldm) {
     PromptParams p = {qb, dc_gqa_ldq(m), m.heads, m.heads / m.kv_heads, m.dim, m.vdim, m.dim_p, m.vdim_p, m.v_at, m.window, m.keep, m.scale, m.softcap, sink_of(m),
-                      m.lambda, 1.0f - m.diff, eps, st.seq_ids, st.positions, st.starts, tiles, cache_ref(c, m.row), mixb, ldm};
+                      m.lambda, 1.0f - m.diff, eps, m.score_bias, m.off_g < 0 ? nullptr : proj + m.off_g, ldp, st.seq_ids, st.positions, st.starts, tiles, cache_ref(c, m.row), mixb, ldm};
     // the smallest pair of padded key and value sizes that holds the head
 #define DC_PROMPT(DP, VP, PQ, ST, MAPS)                                                                  \
-    if (m.maps == MAPS && m.dim <= DP && m.vdim <= VP) return launch_prompt<DP, VP, PQ, ST, MAPS>(ctx, p, n_tiles)
+    if (m.maps == MAPS && !m.score_bias && m.dim <= DP && m.vdim <= VP) return launch_prompt<DP, VP, PQ, ST, MAPS, false>(ctx, p, n_tiles)
+#define DC_PROMPT_SIGMOID(DP, VP, PQ, ST)                                                                \
+    if (m.maps == 1 && m.score_bias && m.dim <= DP && m.vdim <= VP) return launch_prompt<DP, VP, PQ, ST, 1, true>(ctx, p, n_tiles)
     DC_PROMPT(32, 32, 128, 3, 1);
     DC_PROMPT(32, 64, 128, 3, 1);
     DC_PROMPT(64, 64, 128, 3, 1);
@@ -755,6 +913,13 @@ int dc_launch_gqa_prompt(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, 
     DC_PROMPT(64, 128, 128, 2, 2);
     DC_PROMPT(128, 128, 128, 2, 2);
     DC_PROMPT(128, 256, 64, 2, 2);
+    DC_PROMPT_SIGMOID(32, 32, 128, 3);
+    DC_PROMPT_SIGMOID(64, 32, 128, 3);
+    DC_PROMPT_SIGMOID(64, 64, 128, 3);
+    DC_PROMPT_SIGMOID(96, 96, 128, 2);
+    DC_PROMPT_SIGMOID(128, 128, 128, 2);
+    DC_PROMPT_SIGMOID(256, 256, 64, 2);
+#undef DC_PROMPT_SIGMOID
 #undef DC_PROMPT
     return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "gqa_prompt: head sizes %d and %d", m.dim, m.vdim);
 }

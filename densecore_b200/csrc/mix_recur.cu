@@ -1,5 +1,6 @@
-// Recurrent mixers: short causal convolution, gated delta rule with one decay per key channel, Mamba-2 state-space
-// scan, linear attention with a constant decay per head, and their gated output norms.
+// Recurrent mixers: short causal convolution, gated delta rule with one decay per key channel, generalized delta rule whose
+// removed part is read from the old state, Mamba-2 state-space scan, linear attention with a constant decay per head, and
+// their gated output norms.
 //
 // Per-sequence state (f32) lives in the cache manager's state slots: the matrix S as [head][value column][key
 // channel], and the convolution's last inputs as a ring [position % taps][channel].  A sequence at position 0 starts
@@ -24,47 +25,6 @@
 using namespace dc;
 
 namespace {
-
-__device__ __forceinline__ int entry_of(const int32_t* starts, int E, int t) {
-    int e = 0;
-    while (e + 1 < E && starts[e + 1] <= t) ++e;
-    return e;
-}
-
-// Convolution of one channel at token t (local index i in its entry, position pos): weights w[j * ldw], the last tap for
-// the token itself; inputs before the entry come from the ring, before position 0 they are zero.
-__device__ __forceinline__ float conv_at(const float* __restrict__ proj, int ldp, const float* __restrict__ ring, int C, int rc, int taps,
-                                         const float* __restrict__ w, int ldw, int col, int t, int i, int pos) {
-    float s = 0.0f;
-    if (i >= taps - 1) {
-        const float* in = proj + (size_t)(t - taps + 1) * ldp + col;
-#pragma unroll 4
-        for (int j = 0; j < taps; ++j) s = fmaf(w[(size_t)j * ldw], in[(size_t)j * ldp], s);
-        return s;
-    }
-    for (int j0 = 0; j0 < taps; j0 += 4) {      // four taps' loads in flight, none behind a branch
-        float in[4], wj[4];
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-            const int j = min(j0 + k, taps - 1), back = taps - 1 - j;
-            const float* src = back <= i ? proj + (size_t)(t - back) * ldp + col : ring + (size_t)(max(pos - back, 0) % taps) * C + rc;
-            in[k] = *src;
-            wj[k] = w[(size_t)j * ldw];
-            if (j0 + k >= taps || pos < back) in[k] = 0.0f;
-        }
-#pragma unroll
-        for (int k = 0; k < 4; ++k) s = fmaf(wj[k], in[k], s);
-    }
-    return s;
-}
-
-struct ConvRef {
-    uint8_t* base;
-    size_t slot_bytes, ring_off;
-    const int32_t *seq_ids, *positions, *starts;
-    int E, taps, C, ldw;     // C: channels of a ring row; ldw: pitch of the convolution weights [taps][ldw]
-    __device__ float* ring(int seq) const { return reinterpret_cast<float*>(base + (size_t)seq * slot_bytes + ring_off); }
-};
 
 constexpr int BT = 16, BROW = 20;                       // tokens of a block; pitch of a 16 x 16 factor (conflict-free rows)
 
@@ -398,6 +358,168 @@ __global__ void __launch_bounds__(128) k_delta_blocks(const DeltaBlock p) {
     }
 }
 
+// The generalized delta rule, S <- diag(w) S - (a u)(u^T S) + k v^T, with W_t and P_ti products of w as above, c_t = -a_t u_t:
+//   z_t = u_t . S_(t-1) = d_t + sum_{i<t} (A_ti z_i + K_ti v_i),   d_t = S0 . (W_(t-1) u_t),
+//   A_ti = sum_d P_(t-1,i) c_i u_t,   K_ti = sum_d P_(t-1,i) k_i u_t,   so that z = X d + M v with X = (I - A)^-1, M = X K
+//   o_t = S0 . (W_t r_t) + sum_{i<=t} (C_ti z_i + B_ti v_i),   C_ti = sum_d P_ti c_i r_t,   B_ti = sum_d P_ti k_i r_t
+//   S   = W_15 S0 + sum_i (P_15,i c_i z_i + P_15,i k_i v_i)
+// z is eliminated: with N = C X and N' = B + C M, o = S0 . W r + N d + N' v; with D = P c X and E = P c M + P k (over the block's
+// tokens), S = W_15 S0 + D d + E v.  A block leaves W_(t-1) u, W r, D, E, W_15, N and N'.
+// Floats of one (block, head): W u, W r, D, E (each [16][dp]), W_15 [dp], N and N' [16][20].
+__host__ __device__ constexpr int general_block_floats(int dp) { return 4 * BT * dp + dp + 2 * BT * BROW; }
+
+// exp(-e^(-1/2) sigmoid(z))
+__device__ __forceinline__ float decay_below_one(float z) { return expf(-0.6065306597126334f * sigmoid(z)); }
+
+struct GeneralBlock {
+    const float* proj;
+    int ldp, off_r, off_k, off_a, heads, dim, dp;
+    const float* low;            // decay projection [T][ldd]
+    int ldd;
+    const float *w0, *a_bias;
+    float unit_eps;
+    const int32_t* starts;
+    int E;
+    float* out;
+};
+
+__global__ void __launch_bounds__(128) k_general_blocks(const GeneralBlock p) {
+    extern __shared__ __align__(16) float sm[];         // k, r, w, c: [16][dim] each
+    __shared__ float sA[BT][BT + 1], sK[BT][BT + 1], sC[BT][BT + 1], sB[BT][BT + 1], sX[BT][BT + 1], sM[BT][BT + 1], s_unit[BT];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim, dp = p.dp;
+    const BlockRef br = block_at<BT>(p.starts, p.E, blockIdx.x);
+    if (br.n <= 0) return;
+    float *sk = sm, *sr = sm + BT * dim, *sw = sm + 2 * BT * dim, *sc = sm + 3 * BT * dim;
+    float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * general_block_floats(dp);
+    for (int d = tid; d < dim; d += 128) {              // every load before the arithmetic
+        float k[BT], r[BT], a[BT], w[BT];
+        const float w0 = p.w0[h * dim + d], ab = p.a_bias[h * dim + d];
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+            const int tc = br.t0 + min(t, br.n - 1);
+            const float* row = p.proj + (size_t)tc * p.ldp + h * dim + d;
+            k[t] = row[p.off_k], r[t] = row[p.off_r], a[t] = row[p.off_a];
+            w[t] = p.low[(size_t)tc * p.ldd + h * dim + d];
+        }
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+            const bool ok = t < br.n;
+            sk[t * dim + d] = ok ? k[t] : 0.0f;
+            sr[t * dim + d] = ok ? r[t] : 0.0f;
+            sw[t * dim + d] = ok ? decay_below_one(w[t] + w0) : 1.0f;
+            sc[t * dim + d] = ok ? -sigmoid(a[t] + ab) * k[t] : 0.0f;      // the unit key's length is still to come
+        }
+    }
+    __syncthreads();
+    {
+        float ss[4] = {};
+        for (int d = lane; d < dim; d += 32)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) ss[j] = fmaf(sk[(4 * warp + j) * dim + d], sk[(4 * warp + j) * dim + d], ss[j]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            ss[j] = warp_sum(ss[j]);
+            if (lane == 0) s_unit[4 * warp + j] = 1.0f / sqrtf(ss[j] + p.unit_eps);
+        }
+    }
+    __syncthreads();
+    // the products of the source tokens i = warp, warp + 4, ...: c, k run over P_ti c_i, P_ti k_i (c without the lengths)
+#pragma unroll 1
+    for (int i = warp; i < BT; i += 4) {
+        float v[2][32];
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[0][j] = v[1][j] = 0.0f;
+        for (int d = lane; d < dim; d += 32) {
+            float c = 0.0f, k = 0.0f;
+#pragma unroll
+            for (int t = 0; t < BT; ++t) {
+                const float kt = sk[t * dim + d], rt = sr[t * dim + d], wt = sw[t * dim + d];
+                v[0][t] = fmaf(c, kt, v[0][t]);
+                v[1][t] = fmaf(k, kt, v[1][t]);
+                c = t == i ? sc[t * dim + d] : c * wt;
+                k = t == i ? kt : k * wt;
+                v[0][BT + t] = fmaf(c, rt, v[0][BT + t]);
+                v[1][BT + t] = fmaf(k, rt, v[1][BT + t]);
+            }
+        }
+        const float ui = s_unit[i], ut = s_unit[lane & 15];
+        const float a = transpose_sum32(v[0], lane) * ui, b = transpose_sum32(v[1], lane);
+        if (lane < BT) sA[lane][i] = a * ut, sK[lane][i] = b * ut;
+        else sC[lane - BT][i] = a, sB[lane - BT][i] = b;
+    }
+    __syncthreads();
+    if (tid < BT) {                                     // column tid of (I - A)^-1
+        float x[BT];
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+            float a[2] = {};
+#pragma unroll
+            for (int i = 0; i < t; ++i) a[i & 1] = fmaf(sA[t][i], x[i], a[i & 1]);
+            x[t] = t < tid ? 0.0f : t == tid ? 1.0f : a[0] + a[1];
+            sX[t][tid] = x[t];
+        }
+    }
+    __syncthreads();
+    float* N = out + 4 * BT * dp + dp;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int t = (tid + 128 * j) / BT, i = tid % BT;
+        float m = 0.0f, n = 0.0f;
+#pragma unroll
+        for (int q = 0; q < BT; ++q) {
+            m = fmaf(sX[t][q], sK[q][i], m);            // factors are zero above the diagonal
+            n = fmaf(sC[t][q], sX[q][i], n);
+        }
+        sM[t][i] = m;
+        N[t * BROW + i] = n;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int t = (tid + 128 * j) / BT, i = tid % BT;
+        float n = sB[t][i];
+#pragma unroll
+        for (int q = 0; q < BT; ++q) n = fmaf(sC[t][q], sM[q][i], n);
+        N[(BT + t) * BROW + i] = n;
+    }
+    // per channel: one thread the decayed vectors and D, another one E
+    for (int i = tid; i < 2 * dp; i += 128) {
+        const bool second = i >= dp;
+        const int d = second ? i - dp : i;
+        const bool in = d < dim;
+        float w[BT], c[BT];
+#pragma unroll
+        for (int t = 0; t < BT; ++t) w[t] = in ? sw[t * dim + d] : 1.0f, c[t] = in ? sc[t * dim + d] * s_unit[t] : 0.0f;
+        if (!second) {
+            float cum = 1.0f;
+#pragma unroll
+            for (int t = 0; t < BT; ++t) {
+                out[t * dp + d] = in ? cum * sk[t * dim + d] * s_unit[t] : 0.0f;
+                cum *= w[t];
+                out[(BT + t) * dp + d] = in ? cum * sr[t * dim + d] : 0.0f;
+            }
+            out[4 * BT * dp + d] = cum;
+        }
+        float suffix = 1.0f, k[BT];
+#pragma unroll
+        for (int t = BT - 1; t >= 0; --t) {
+            c[t] *= suffix;
+            k[t] = second && in ? suffix * sk[t * dim + d] : 0.0f;
+            suffix *= w[t];
+        }
+        const float (*F)[BT + 1] = second ? sM : sX;
+#pragma unroll
+        for (int j = 0; j < BT; ++j) {
+            float a[2] = {k[j], 0.0f};
+#pragma unroll
+            for (int t = j; t < BT; ++t) a[t & 1] = fmaf(c[t], F[t][j], a[t & 1]);
+            out[((second ? 3 : 2) * BT + j) * dp + d] = a[0] + a[1];
+        }
+    }
+}
+
 // Floats of one (block, head) of the state-space scan: M [16][20], cumulative decays [16], update factors [16].
 constexpr int SSD_BLOCK = BT * BROW + 2 * BT;
 
@@ -459,9 +581,10 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
 
 // ---------------------------------------------------------------- the scan over blocks
 constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp
+enum { SCAN_SSD = 0, SCAN_DELTA = 1, SCAN_GENERAL = 2 };
 
 struct ScanParams {
-    const float* blocks;           // k_delta_blocks / k_ssd_blocks
+    const float* blocks;           // k_delta_blocks / k_general_blocks / k_ssd_blocks
     const float *k, *q;            // ssd: B and C of group 0
     const float* v;                // values of head 0
     int ld, heads, per, dim, vdim;
@@ -546,9 +669,12 @@ __device__ __forceinline__ void column_dots(const float* rows, int dp, const flo
 }
 
 // EPL: key channels per lane (the key size, padded to 32 EPL).
-template <int EPL, bool DELTA>
+constexpr int scan_block_floats(int kind, int dp) { return kind == SCAN_DELTA ? delta_block_floats(dp) : kind == SCAN_GENERAL ? general_block_floats(dp) : 2 * BT * dp + SSD_BLOCK; }
+
+template <int EPL, int KIND>
 __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
-    constexpr int DP = 32 * EPL, BLK = DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK, BUF = BLK + BT * SC_COLS;
+    constexpr bool GENERAL = KIND == SCAN_GENERAL, DELTA = KIND != SCAN_SSD;         // the delta rules' factors come whole from memory
+    constexpr int DP = 32 * EPL, BLK = scan_block_floats(KIND, DP), BUF = BLK + BT * SC_COLS;
     extern __shared__ __align__(16) float sm[];
     __shared__ __align__(16) float s_d[4][4][BT], s_u[4][4][BT];
     pdl_launch_dependents();
@@ -623,7 +749,8 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             v[k] = x[BLK + (lt + 8 * k) * SC_COLS + warp * 4 + lc];
-            s_d[warp][lc][lt + 8 * k] = DELTA ? v[k] - r[0][k] : v[k];
+            s_d[warp][lc][lt + 8 * k] = GENERAL ? r[0][k] : DELTA ? v[k] - r[0][k] : v[k];
+            if (GENERAL) s_u[warp][lc][lt + 8 * k] = v[k];
         }
         __syncwarp();
         auto row_dot = [&](const float* row, const float* vals) {      // rows of W, B, M are zero above the diagonal
@@ -638,9 +765,13 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             }
             return (a[0] + a[1]) + (a[2] + a[3]);
         };
-        const float* scal = x + (DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
+        const float* scal = x + (GENERAL ? 4 * BT * DP + DP : DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
         float out[2];
-        if (DELTA) {
+        if (GENERAL) {
+#pragma unroll
+            for (int k = 0; k < 2; ++k)
+                out[k] = rq[k] + row_dot(scal + (lt + 8 * k) * BROW, s_d[warp][lc]) + row_dot(scal + (BT + lt + 8 * k) * BROW, s_u[warp][lc]);
+        } else if (DELTA) {
 #pragma unroll
             for (int k = 0; k < 2; ++k) s_u[warp][lc][lt + 8 * k] = row_dot(scal + (lt + 8 * k) * BROW, s_d[warp][lc]);
             __syncwarp();
@@ -665,7 +796,7 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         const float* keys = x + (DELTA ? 2 * BT * DP : BT * DP);
         {
             float g[EPL];
-            if (DELTA) Chan<EPL>::load(x + 3 * BT * DP, lane, g);
+            if (DELTA) Chan<EPL>::load(x + (GENERAL ? 4 : 3) * BT * DP, lane, g);
 #pragma unroll
             for (int c = 0; c < 4; ++c)
 #pragma unroll
@@ -673,15 +804,17 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
         constexpr int G = EPL <= 4 ? 8 : 4;
 #pragma unroll
-        for (int t = 0; t < BT; t += G) {
+        for (int row = 0; row < (GENERAL ? 2 : 1) * BT; row += G) {
+            const int t = row % BT;
+            float (*vals)[BT] = GENERAL && row < BT ? s_d[warp] : s_u[warp];
             float w[G][EPL], u[4][G];
 #pragma unroll
-            for (int g = 0; g < G; ++g) Chan<EPL>::load(keys + (t + g) * DP, lane, w[g]);
+            for (int g = 0; g < G; ++g) Chan<EPL>::load(keys + (row + g) * DP, lane, w[g]);
 #pragma unroll
             for (int c = 0; c < 4; ++c)
 #pragma unroll
                 for (int g = 0; g < G; g += 4) {
-                    const float4 f = *reinterpret_cast<const float4*>(&s_u[warp][c][t + g]);
+                    const float4 f = *reinterpret_cast<const float4*>(&vals[c][t + g]);
                     u[c][g] = f.x, u[c][g + 1] = f.y, u[c][g + 2] = f.z, u[c][g + 3] = f.w;
                 }
 #pragma unroll
@@ -702,21 +835,20 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
 }
 
-template <int EPL, bool DELTA>
+template <int EPL, int KIND>
 int launch_scan_epl(dc_ctx* ctx, const ScanParams& p, int E) {
-    constexpr int DP = 32 * EPL;
-    const size_t smem = (size_t)2 * ((DELTA ? delta_block_floats(DP) : 2 * BT * DP + SSD_BLOCK) + BT * SC_COLS) * 4;
-    DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, DELTA>, (int)smem, "k_state_scan"));
-    return dc_launch(ctx, "k_state_scan", k_state_scan<EPL, DELTA>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_THREADS), smem, p);
+    const size_t smem = (size_t)2 * (scan_block_floats(KIND, 32 * EPL) + BT * SC_COLS) * 4;
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, KIND>, (int)smem, "k_state_scan"));
+    return dc_launch(ctx, "k_state_scan", k_state_scan<EPL, KIND>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_THREADS), smem, p);
 }
 int key_pad(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
-template <bool DELTA>
+template <int KIND>
 int launch_scan(dc_ctx* ctx, const ScanParams& p, int E) {
     switch (key_pad(p.dim)) {
-    case 32: return launch_scan_epl<1, DELTA>(ctx, p, E);
-    case 64: return launch_scan_epl<2, DELTA>(ctx, p, E);
-    case 128: return launch_scan_epl<4, DELTA>(ctx, p, E);
-    default: return launch_scan_epl<8, DELTA>(ctx, p, E);
+    case 32: return launch_scan_epl<1, KIND>(ctx, p, E);
+    case 64: return launch_scan_epl<2, KIND>(ctx, p, E);
+    case 128: return launch_scan_epl<4, KIND>(ctx, p, E);
+    default: return launch_scan_epl<8, KIND>(ctx, p, E);
     }
 }
 
@@ -987,6 +1119,119 @@ __global__ void __launch_bounds__(256) k_delta_decode(const DeltaDecode p) {
     }
 }
 
+struct GeneralDecode {
+    const float* proj;
+    int ldp, heads, dim, rank, off_r, off_k, off_v, off_g, off_a, off_w;
+    float unit_eps, eps;
+    const __nv_bfloat16* w2;
+    int ldw2;
+    const float *w0, *a_bias, *norm;
+    uint8_t* base;
+    size_t slot_bytes, state_off;
+    const int32_t *seq_ids, *positions;
+    float* mix;
+    __nv_bfloat16* mixb;         // instead of mix
+    int ldm;
+};
+
+// Generalized delta rule, one CTA per (head, sequence): decays and removal rates, the state's step, the gated norm.
+template <int EPL>
+__global__ void __launch_bounds__(256) k_general_decode(const GeneralDecode p) {
+    constexpr int DP = 32 * EPL, NC = 8;            // columns of a warp at a time
+    extern __shared__ __align__(16) float sm[];     // r, k, removal rate, decay, v, gate: [DP]; answers [DP]; low-rank inputs
+    __shared__ float red[33];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, t = blockIdx.y, dim = p.dim, rank = (p.rank + 127) & ~127;
+    float *sr = sm, *sk = sr + DP, *sa = sk + DP, *sw = sa + DP, *sv = sw + DP, *sg = sv + DP, *so = sg + DP, *sl = so + DP;
+    pdl_launch_dependents();
+    // the weights do not depend on the kernel before: on their way to L2 while this one still waits
+    const char* pw = (const char*)(p.w2 + (size_t)h * dim * p.ldw2);
+    for (int i = tid * 128; i < dim * p.ldw2 * 2; i += 256 * 128) prefetch_l2(pw + i);
+    pdl_wait();
+    const int pos = p.positions[t];
+    float* S = reinterpret_cast<float*>(p.base + (size_t)p.seq_ids[t] * p.slot_bytes + p.state_off) + (size_t)h * dim * dim;
+    for (int i = tid * 32; i < dim * dim; i += 256 * 32) prefetch_l2(S + i);
+    const float* row = p.proj + (size_t)t * p.ldp;
+    for (int c = tid; c < rank; c += 256) sl[c] = c < p.rank ? tanhf(row[p.off_w + c]) : 0.0f;
+    for (int i = tid; i < 5 * DP; i += 256) {
+        const int part = i / DP, d = i - part * DP, off = part == 0 ? p.off_r : part == 1 ? p.off_k : part == 2 ? p.off_a : part == 3 ? p.off_v : p.off_g;
+        float v = d < dim ? row[off + h * dim + d] : 0.0f;
+        if (part == 2) v = d < dim ? sigmoid(v + p.a_bias[h * dim + d]) : 0.0f;
+        (part < 3 ? sm + part * DP : sv + (part - 3) * DP)[d] = v;
+    }
+    __syncthreads();
+    low_rank_rows(p.w2 + (size_t)h * dim * p.ldw2, p.ldw2, dim, sl, p.rank, sw);
+    float rr[EPL], kr[EPL], ur[EPL], cr[EPL], wr[EPL], ss = 0.0f, kq = 0.0f, cq = 0.0f;
+    Chan<EPL>::load(sr, lane, rr);
+    Chan<EPL>::load(sk, lane, kr);
+    Chan<EPL>::load(sa, lane, cr);
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) ss = fmaf(kr[i], kr[i], ss);
+    const float unit = 1.0f / sqrtf(warp_sum(ss) + p.unit_eps);
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+        ur[i] = kr[i] * unit;
+        cr[i] *= -ur[i];
+        kq = fmaf(kr[i], rr[i], kq);
+        cq = fmaf(cr[i], rr[i], cq);
+    }
+    kq = warp_sum(kq);
+    cq = warp_sum(cq);
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+        const int d = Chan<EPL>::at(lane, i);
+        wr[i] = d < dim ? decay_below_one(sw[d] + p.w0[h * dim + d]) : 0.0f;
+        rr[i] *= wr[i];
+    }
+    for (int c0 = NC * warp; c0 < dim; c0 += 8 * NC) {
+        float s[NC][EPL], a[NC], b[NC];
+        load_columns<NC, EPL>(S, c0, dim, dim, lane, pos == 0, s);
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            a[c] = b[c] = 0.0f;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) {
+                a[c] = fmaf(s[c][i], ur[i], a[c]);
+                b[c] = fmaf(s[c][i], rr[i], b[c]);
+            }
+        }
+        // lane l works for column l / 4
+        const float z = transpose_sum8(a, lane), q = transpose_sum8(b, lane);
+        const int mine = c0 + (lane >> 2);
+        const float v = mine < dim ? sv[mine] : 0.0f;
+        if ((lane & 3) == 0 && mine < dim) so[mine] = fmaf(kq, v, fmaf(cq, z, q));
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            const float zc = __shfl_sync(0xffffffffu, z, 4 * c), vc = __shfl_sync(0xffffffffu, v, 4 * c);
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(kr[i], vc, fmaf(cr[i], zc, s[c][i] * wr[i]));
+        }
+        store_columns<NC, EPL>(S, c0, dim, dim, lane, s);
+    }
+    __syncthreads();
+    float sq = 0.0f;
+    for (int c = tid; c < dim; c += 256) sq = fmaf(so[c], so[c], sq);
+    const float inv = 1.0f / sqrtf(block_sum(sq, red) / (float)dim + p.eps);
+    for (int c = tid; c < dim; c += 256) {
+        const float v = so[c] * inv * p.norm[h * dim + c] * sigmoid(sg[c]);
+        const size_t o = (size_t)t * p.ldm + (size_t)h * dim + c;
+        if (p.mixb) p.mixb[o] = __float2bfloat16_rn(v);
+        else p.mix[o] = v;
+    }
+}
+
+// tanh of n columns, to lowb or in place
+__global__ void __launch_bounds__(256) k_tanh_columns(float* proj, int ldp, int n, int T, __nv_bfloat16* __restrict__ lowb, int ldl) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+    if (i >= (long long)T * n) return;
+    const int t = (int)(i / n), c = (int)(i % n);
+    const float v = tanhf(proj[(size_t)t * ldp + c]);
+    if (lowb) lowb[(size_t)t * ldl + c] = __float2bfloat16_rn(v);
+    else proj[(size_t)t * ldp + c] = v;
+}
+
 struct SsdDecode {
     ConvRef cr;
     const float* proj;
@@ -1049,10 +1294,10 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
 }
 
 // ---------------------------------------------------------------- output norms
-// delta: one warp per (token, head): o / rms(o) * w * sigmoid(gate)
+// delta rules: one warp per (token, head): o / rms(o) * w * sigmoid(gate).  ws: pitch of the heads' weights, 0: they share them
 template <typename TO>
 __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg,
-                                                        const float* __restrict__ w, int heads, int vdim, int T, float eps,
+                                                        const float* __restrict__ w, int ws, int heads, int vdim, int T, float eps,
                                                         TO* __restrict__ out, int ldm) {
     pdl_launch_dependents();
     pdl_wait();
@@ -1065,7 +1310,14 @@ __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict_
     for (int c = lane; c < vdim; c += 32) ss = fmaf(r[c], r[c], ss);
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
     for (int c = lane; c < vdim; c += 32)
-        store_as(out + (size_t)t * ldm + (size_t)h * vdim + c, r[c] * inv * w[c] * sigmoid(gate[(size_t)t * ldg + (size_t)h * vdim + c]));
+        store_as(out + (size_t)t * ldm + (size_t)h * vdim + c, r[c] * inv * w[h * ws + c] * sigmoid(gate[(size_t)t * ldg + (size_t)h * vdim + c]));
+}
+
+int launch_head_norm_gate(dc_ctx* ctx, const float* o, int ldo, const float* gate, int ldg, const float* w, int ws, int heads, int vdim, int T, float eps,
+                          float* mix, __nv_bfloat16* mixb, int ldm) {
+    const dim3 grid((unsigned)(((long long)T * heads + 7) / 8)), block(256);
+    if (mixb) return dc_launch(ctx, "k_head_norm_gate", k_head_norm_gate<__nv_bfloat16>, grid, block, 0, o, ldo, gate, ldg, w, ws, heads, vdim, T, eps, mixb, ldm);
+    return dc_launch(ctx, "k_head_norm_gate", k_head_norm_gate<float>, grid, block, 0, o, ldo, gate, ldg, w, ws, heads, vdim, T, eps, mix, ldm);
 }
 
 // ssd: one CTA per (token, norm group): y silu(z) (unless gated already), over its root mean square, times w
@@ -1341,13 +1593,45 @@ int dc_launch_delta_scan(dc_ctx* ctx, const dc_delta_mixer& m, const dc_step& st
     p.o = o, p.ldo = lda;
     p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
     p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
-    DC_TRY(launch_scan<true>(ctx, p, st.E));
-    const unsigned blocks = (unsigned)(((long long)st.T * m.heads + 7) / 8);
-    if (mixb)
-        return dc_launch(ctx, "k_head_norm_gate", k_head_norm_gate<__nv_bfloat16>, dim3(blocks), dim3(256), 0, o, lda, raw_g, ldg, m.norm, m.heads,
-                         m.vdim, st.T, eps, mixb, ldm);
-    return dc_launch(ctx, "k_head_norm_gate", k_head_norm_gate<float>, dim3(blocks), dim3(256), 0, o, lda, raw_g, ldg, m.norm, m.heads, m.vdim, st.T,
-                     eps, mix, ldm);
+    DC_TRY(launch_scan<SCAN_DELTA>(ctx, p, st.E));
+    return launch_head_norm_gate(ctx, o, lda, raw_g, ldg, m.norm, 0, m.heads, m.vdim, st.T, eps, mix, mixb, ldm);
+}
+
+size_t dc_general_block_floats(const dc_general_mixer& m) { return (size_t)m.heads * general_block_floats(key_pad(m.dim)); }
+
+int dc_launch_general_tanh(dc_ctx* ctx, const dc_general_mixer& m, int T, float* proj, int ldp, __nv_bfloat16* lowb, int ldl) {
+    const int n = dc_pad8(m.rank);
+    return dc_launch(ctx, "k_tanh_columns", k_tanh_columns, dim3((unsigned)(((long long)T * n + 255) / 256)), dim3(256), 0, proj + m.off_w, ldp, n, T, lowb, ldl);
+}
+
+int dc_launch_general_scan(dc_ctx* ctx, const dc_general_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, const float* low,
+                           int ldd, float* blk, float eps, float* o, int ldo, float* mix, __nv_bfloat16* mixb, int ldm) {
+    const GeneralBlock b = {proj, ldp, m.off_r, m.off_k, m.off_a, m.heads, m.dim, key_pad(m.dim), low, ldd, m.w0, m.a_bias, m.unit_eps, st.starts, st.E, blk};
+    const size_t smem = (size_t)4 * BT * m.dim * 4;
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_general_blocks, (int)smem, "k_general_blocks"));
+    DC_TRY(dc_launch(ctx, "k_general_blocks", k_general_blocks, dim3(dc_scan_blocks(st.T, st.E), m.heads), dim3(128), smem, b));
+    ScanParams p = {};
+    p.blocks = blk, p.v = proj + m.off_v;
+    p.ld = ldp, p.heads = m.heads, p.per = 1, p.dim = m.dim, p.vdim = m.dim;
+    p.o = o, p.ldo = ldo;
+    p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
+    p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
+    DC_TRY(launch_scan<SCAN_GENERAL>(ctx, p, st.E));
+    return launch_head_norm_gate(ctx, o, ldo, proj + m.off_g, ldp, m.norm, m.dim, m.heads, m.dim, st.T, eps, mix, mixb, ldm);
+}
+
+int dc_launch_general_decode(dc_ctx* ctx, const dc_general_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float eps,
+                             float* mix, __nv_bfloat16* mixb, int ldm) {
+    const GeneralDecode p = {proj, ldp, m.heads, m.dim, m.rank, m.off_r, m.off_k, m.off_v, m.off_g, m.off_a, m.off_w, m.unit_eps, eps, m.w2.w, m.w2.ld, m.w0,
+                             m.a_bias, m.norm, sr.base, sr.slot_bytes, sr.state_off, st.seq_ids, st.positions, mix, mixb, ldm};
+    const int dp = key_pad(m.dim);
+    const size_t smem = (size_t)(7 * dp + ((m.rank + 127) & ~127)) * 4;
+    const dim3 grid(m.heads, st.T), block(256);
+    if (smem > 48 * 1024) return dc_fail(ctx, DC_B200_UNSUPPORTED, "generalized delta rule: decay rank %d is too large", m.rank);
+    if (dp == 32) return dc_launch(ctx, "k_general_decode", k_general_decode<1>, grid, block, smem, p);
+    if (dp == 64) return dc_launch(ctx, "k_general_decode", k_general_decode<2>, grid, block, smem, p);
+    if (dp == 128) return dc_launch(ctx, "k_general_decode", k_general_decode<4>, grid, block, smem, p);
+    return dc_launch(ctx, "k_general_decode", k_general_decode<8>, grid, block, smem, p);
 }
 
 int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, float* act,
@@ -1366,7 +1650,7 @@ int dc_launch_ssd(dc_ctx* ctx, const dc_ssd_mixer& m, const dc_step& st, const d
     p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
     p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
     p.vec = m.state % 4 == 0 && lda % 4 == 0 && inner % 4 == 0;
-    DC_TRY(launch_scan<false>(ctx, p, st.E));
+    DC_TRY(launch_scan<SCAN_SSD>(ctx, p, st.E));
     const int n = inner / m.norm_groups;
     const float* z = proj + m.off_z;
     return mixb ? launch_group_norm(ctx, y, lda, z, ldp, m.norm, n, m.norm_groups, st.T, eps, mixb, ldm)
@@ -1420,7 +1704,7 @@ int dc_launch_lightning_scan(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_
     p.base = sr.base, p.slot_bytes = sr.slot_bytes, p.state_off = sr.state_off;
     p.seq_ids = st.seq_ids, p.positions = st.positions, p.starts = st.starts;
     p.vec = m.dim % 4 == 0 && lda % 4 == 0;
-    return launch_scan<false>(ctx, p, st.E);
+    return launch_scan<SCAN_SSD>(ctx, p, st.E);
 }
 
 int dc_launch_lightning_decode(dc_ctx* ctx, const dc_lightning_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* act,

@@ -858,7 +858,7 @@ static const char* kClassNames[DC_K_COUNT] = {"embed", "rmsnorm_q8k", "gemv_qkv"
                                                "moe_down", "moe_combine", "ep_allreduce", "ffn_gate_up_swiglu",
                                                "ffn_down", "lm_head_argmax", "argmax_finish", "mixer_in", "mixer_out",
                                                "mixer_delta", "mixer_ssd", "mixer_latent", "post_norm", "pre_norm",
-                                               "mixer_gqa", "mixer_lightning"};
+                                               "mixer_gqa", "mixer_lightning", "mixer_general_delta"};
 
 const char* dc_b200_kernel_class_name(int cls) { return (cls >= 0 && cls < DC_K_COUNT) ? kClassNames[cls] : nullptr; }
 

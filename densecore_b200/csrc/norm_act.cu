@@ -1,6 +1,6 @@
 // Norms around the sublayers of a layer-list decoder: RMS norm of a sublayer's output added to the f32 residual;
 // RMS norm of residual rows (ahead of a layer's products, and the output norm on the rows whose logits are wanted), with
-// what a step still owes the residual added on the way.
+// what a step still owes the residual added on the way; the same over a residual of several streams.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
 #include "dc_stack.h"
@@ -115,34 +115,20 @@ __global__ void __launch_bounds__(256) k_pre_norm(float* __restrict__ x, const f
         const int i = threadIdx.x + 256 * j;
         xv[j] = i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    auto add = [&](float4& a, float4 b) { a.x += b.x, a.y += b.y, a.z += b.z, a.w += b.w; };
     if (sum.k) {
         if (threadIdx.x < (unsigned)sum.k) s_rows[threadIdx.x] = sum.rows[blockIdx.x * sum.k + threadIdx.x];
         __syncthreads();
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) {
             const int i = threadIdx.x + 256 * j;
-            if (i >= n4) continue;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-            for (int k = 0; k < sum.k; ++k) {
-                const size_t at = (size_t)s_rows[k] * sum.ld + 4 * i;
-                if (sum.yb) {
-                    const uint2 u = *reinterpret_cast<const uint2*>(sum.yb + at);
-                    add(v, make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
-                                       __uint_as_float(u.y & 0xffff0000u)));
-                } else {
-                    add(v, *reinterpret_cast<const float4*>(sum.y + at));
-                }
-            }
-            add(xv[j], v);
+            if (i < n4) dc::add4(xv[j], dc::row_sum4(sum, s_rows, i));
         }
     }
     if (step)
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) {
             const int i = threadIdx.x + 256 * j;
-            if (i < n4) add(xv[j], reinterpret_cast<const float4*>(step)[i]);
+            if (i < n4) dc::add4(xv[j], reinterpret_cast<const float4*>(step)[i]);
         }
     if (sum.k || step)
 #pragma unroll
@@ -169,7 +155,68 @@ __global__ void __launch_bounds__(256) k_pre_norm(float* __restrict__ x, const f
     }
 }
 
+// S: streams at most.  Rows as above.
+template <int S, int KEEP>
+__global__ void __launch_bounds__(256) k_hyper_norm(const dc_hyper hy, const float* __restrict__ w, const int32_t* __restrict__ rows, int first, int H, int ld,
+                                                    float eps, float* __restrict__ out, __nv_bfloat16* __restrict__ outb) {
+    __shared__ float red[33], coef[S * (S + 2)];
+    __shared__ int32_t s_rows[DC_MOE_MAX_TOP];
+    dc::pdl_launch_dependents();
+    const int n4 = ld / 4;
+    float4 wv[KEEP], u[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        wv[j] = w && i < n4 ? reinterpret_cast<const float4*>(w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    dc::hyper_coefficients<S>(hy, coef);
+    dc::pdl_wait();
+    const int t = rows ? rows[blockIdx.x] : first + (int)blockIdx.x;
+    if (threadIdx.x < (unsigned)hy.sum.k) s_rows[threadIdx.x] = hy.sum.rows[t * hy.sum.k + threadIdx.x];
+    __syncthreads();
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i >= n4) continue;
+        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (hy.sum.k) y = dc::row_sum4(hy.sum, s_rows, i);
+        else if (hy.y) y = *reinterpret_cast<const float4*>(hy.y + (size_t)t * ld + 4 * i);
+        u[j] = dc::hyper_column<S>(hy, coef, t, i, ld, y, hy.x_out != nullptr);
+        ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
+    }
+    const float inv = w ? 1.0f / sqrtf(dc::block_sum(ss, red) / (float)H + eps) : 1.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        if (i >= n4) continue;
+        float4 v = u[j];
+        if (w) v = make_float4(v.x * inv * wv[j].x, v.y * inv * wv[j].y, v.z * inv * wv[j].z, v.w * inv * wv[j].w);
+        if (outb) reinterpret_cast<uint2*>(outb + (size_t)blockIdx.x * ld)[i] = make_uint2(dc::pack_bf2(v.x, v.y), dc::pack_bf2(v.z, v.w));
+        else reinterpret_cast<float4*>(out + (size_t)blockIdx.x * ld)[i] = v;
+    }
+}
+
+template <int S>
+int launch_hyper(dc_ctx* ctx, const dc_hyper& hy, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps, float* out, __nv_bfloat16* outb) {
+    const dim3 grid(R), block(256);
+    if (ld <= 1024) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 1>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
+    if (ld <= 2048) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 2>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
+    if (ld <= 4096) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 4>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
+    return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 8>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
+}
+
 }  // namespace
+
+int dc_launch_hyper_norm(dc_ctx* ctx, const dc_hyper& hy, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps, float* out,
+                         __nv_bfloat16* outb) {
+    if (ld % 8 || ld > 8192 || hy.streams < 1 || hy.streams > DC_MAX_STREAMS || hy.sum.k > DC_MOE_MAX_TOP || (hy.sum.k && hy.sum.ld != ld) || hy.x == hy.x_out)
+        return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "hyper_norm: bad operand");
+    if (hy.streams <= 2) return launch_hyper<2>(ctx, hy, w, rows, first, R, H, ld, eps, out, outb);
+    if (hy.streams <= 4) return launch_hyper<4>(ctx, hy, w, rows, first, R, H, ld, eps, out, outb);
+    return launch_hyper<DC_MAX_STREAMS>(ctx, hy, w, rows, first, R, H, ld, eps, out, outb);
+}
 
 int dc_launch_pre_norm(dc_ctx* ctx, float* x, const float* step, const dc_row_sum& sum, const float* w, int T, int H, int ld, float eps, float* out,
                        __nv_bfloat16* outb) {

@@ -92,6 +92,7 @@ int dc_stack_set_tensor(dc_model* m, const char* name, int type, const int64_t n
         for (int64_t i = 0; i < n; ++i) {
             v[i] = type == DC_TYPE_F32 ? ((const float*)data)[i] : bf16_value(((const uint16_t*)data)[i]);
             if (t.neg_exp) v[i] = (float)-exp((double)v[i]);
+            v[i] += t.plus;
         }
         e = put_vector(t, v);
     } else if (!t.lin) {
@@ -121,7 +122,7 @@ int dc_stack_init_synthetic(dc_model* m, uint64_t seed, float sigma) {
         if (t.loaded || st != DC_B200_OK) continue;
         const int64_t n = elems(t);
         // norm weights around 1, decay exponents and step biases in a useful range, convolution taps not tiny
-        const float sg = t.synth == 4 ? 0.4f : t.synth == 2 ? 0.5f : sigma, off = t.synth == 1 ? 1.0f : t.synth == 3 ? -2.0f : 0.0f;
+        const float sg = t.synth == 4 ? 0.4f : t.synth == 2 ? 0.5f : sigma, off = t.synth == 1 ? 1.0f : t.synth == 3 ? -2.0f : t.synth == 5 ? 1.0f / s->cfg.streams : 0.0f;
         st = dc_launch_synth_f32(ctx, seed + fnv1a64(t.name.c_str()), n, sg, off, tmp);
         if (st != DC_B200_OK) break;
         if (t.vec) {
@@ -130,6 +131,7 @@ int dc_stack_init_synthetic(dc_model* m, uint64_t seed, float sigma) {
             cudaMemcpy(v.data(), tmp, (size_t)n * 4, cudaMemcpyDeviceToHost);
             if (t.neg_exp)
                 for (float& x : v) x = (float)-exp((double)x);
+            for (float& x : v) x += t.plus;
             st = dc_check_cuda(ctx, put_vector(t, v), "init_synthetic");
         } else {
             const int K = (int)t.shape[1];
@@ -229,10 +231,13 @@ int dc_stack_create_cache(dc_model* m, int pool_tokens) {
         dc_stack_layer& L = s->layers[r.layer];
         if (L.kind == DC_MIX_LIGHTNING) {
             r.state_off = carve((size_t)L.li.heads * L.li.vdim * L.li.dim);
+        } else if (L.kind == DC_MIX_GENERAL) {
+            r.state_off = carve((size_t)L.ge.heads * L.ge.dim * L.ge.dim);
         } else if (L.kind == DC_MIX_GQA) {
             r.plane = plane(L.ga.row);
             L.ga.range = key_range(L.ga.window, L.ga.keep);
-            DC_TRY(rotation_table(m, L.ga.rot, &L.ga.cos_sin));
+            if (L.ga.taps) r.ring_off = carve((size_t)L.ga.taps * dc_gqa_conv_cols(L.ga));
+            if (L.ga.rot.dims) DC_TRY(rotation_table(m, L.ga.rot, &L.ga.cos_sin));
         } else if (L.kind == DC_MIX_DELTA) {
             r.state_off = carve((size_t)L.dl.heads * L.dl.vdim * L.dl.dim);
             r.ring_off = carve((size_t)L.dl.taps * (L.dl.off_v + L.dl.heads * L.dl.vdim));
@@ -269,6 +274,9 @@ static int map_weight(dc_model* m, dc_gqa_mixer* d) {
     return DC_B200_OK;
 }
 
+// rows of a layer's input product that are the mixer's
+static int mixer_rows(const dc_stack_layer& L) { return L.pair0 ? L.pair0 : L.in.N; }
+
 static constexpr int ENTRY_INTS = DC_MAX_T + 1;
 
 int dc_stack_finalize(dc_model* m) {
@@ -300,14 +308,18 @@ int dc_stack_finalize(dc_model* m) {
             span = std::max(span, window > 0 ? std::min(window, m->cfg.max_ctx) : m->cfg.max_ctx);
         };
         if (s->cfg.block == DC_BLOCK_PARALLEL) up(mix, L.out.K);
-        if (L.kind == DC_MIX_GQA) {
-            up(proj, L.ff ? L.pair0 : L.in.N);
+        if (L.kind == DC_MIX_GENERAL) {
+            const dc_general_mixer& d = L.ge;
+            up(proj, L.in.N), up(act, d.heads * d.dim), up(low, d.w2.N), up(lowb, d.rank), up(mix, L.out.K);
+            blk = std::max(blk, dc_general_block_floats(d));
+        } else if (L.kind == DC_MIX_GQA) {
+            up(proj, mixer_rows(L));
             up(mix, L.out.K);
             q = std::max(q, (size_t)L.ga.heads * L.ga.maps * dc_gqa_ldq(L.ga));
             attention(L.ga.heads * L.ga.maps, L.ga.vdim, L.ga.window);
             if (L.ga.maps > 1) DC_TRY(map_weight(m, &L.ga));
         } else if (L.kind == DC_MIX_LIGHTNING) {
-            up(f32 ? proj : actb, L.ff ? L.pair0 : L.in.N);
+            up(f32 ? proj : actb, mixer_rows(L));
             up(act, L.li.heads * L.li.vdim);
             if (f32) blk = std::max(blk, dc_lightning_block_floats(L.li));
             else head_state = std::max(head_state, (size_t)L.li.heads * L.li.dim * L.li.vdim);
@@ -330,7 +342,12 @@ int dc_stack_finalize(dc_model* m) {
     }
     b.key_cap = (int)std::min<long long>((long long)C + (long long)m->cfg.max_seqs * (span - 1), all);
     b.key_cap = std::max(b.key_cap, DC_MAX_T);
-    DC_TRY(alloc(m, &b.x, C * H));
+    const bool hyper = s->cfg.block == DC_BLOCK_HYPER;
+    DC_TRY(alloc(m, &b.x, C * H * s->cfg.streams));
+    if (hyper) {
+        DC_TRY(alloc(m, &b.x2, C * H * s->cfg.streams));
+        DC_TRY(alloc(m, &b.h, F * H));
+    }
     DC_TRY(alloc(m, &b.y, C * H));
     DC_TRY(alloc(m, &b.proj, C * proj));
     DC_TRY(alloc(m, &b.act, C * act));
@@ -467,6 +484,8 @@ dc_lin_epi to(float* out, int ld) { return dc_lin_epi::store(out, nullptr, ld); 
         m->last_launches += (n);                                         \
     } while (0)
 
+// a stream norm's: the streams in and out, y and the normed row
+double hyper_bytes(const dc_model* m, int T) { return 8.0 * T * m->stack->cfg.width * (m->stack->cfg.streams + 1); }
 double lin_bytes(const dc_lin& w, int T) { return (double)w.N * w.ld * 2 + (double)T * (w.N + w.K) * 4; }
 
 int mix_delta(dc_model* m, const dc_step& st, const dc_stack_run& run, dc_stack_layer& Ly) {
@@ -530,17 +549,31 @@ int mix_gqa(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_stack_r
     c.f32 = m->stack->dtype == DC_DTYPE_F32;
     c.tables = m->kv.d_tables;
     c.max_blocks = m->kv.max_blocks_per_seq;
-    const int ldp = Ly.ff ? Ly.pair0 : Ly.in.N, ldm = dc_pad8(Ly.out.K);
-    DC_TRY(dc_launch_gqa_prep(m->ctx, d, st, c, b.proj, ldp, m->stack->cfg.eps, m->cfg.max_ctx, b.q, st.tc ? b.qb : nullptr));
-    if (st.tc) return dc_launch_gqa_prompt(m->ctx, d, st, c, sk.tiles, sk.n_tiles, b.qb, m->stack->cfg.eps, b.mixb, ldm);
-    return dc_launch_gqa_tokens(m->ctx, d, st, c, b.q, st.T <= DC_MAX_T ? m->stack->splits : 1, b.part, b.part_ml, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, ldm);
+    const int ldp = mixer_rows(Ly), ldm = dc_pad8(Ly.out.K);
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, run.state_off, run.ring_off};
+    DC_TRY(dc_launch_gqa_prep(m->ctx, d, st, c, d.taps ? &sr : nullptr, b.proj, ldp, m->stack->cfg.eps, m->cfg.max_ctx, b.q, st.tc ? b.qb : nullptr));
+    if (st.tc) return dc_launch_gqa_prompt(m->ctx, d, st, c, sk.tiles, sk.n_tiles, b.qb, b.proj, ldp, m->stack->cfg.eps, b.mixb, ldm);
+    return dc_launch_gqa_tokens(m->ctx, d, st, c, b.q, b.proj, ldp, st.T <= DC_MAX_T ? m->stack->splits : 1, b.part, b.part_ml, m->stack->cfg.eps, b.mix, st.b16 ? b.mixb : nullptr, ldm);
+}
+
+int mix_general(dc_model* m, const dc_step& st, const dc_stack_run& run, dc_stack_layer& Ly) {
+    const dc_general_mixer& d = Ly.ge;
+    const dc_stack_buffers& b = m->stack->b;
+    const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, run.state_off, 0};
+    const int ldp = Ly.in.N, ldo = dc_pad8(d.heads * d.dim), ldl = dc_pad8(d.rank), ldm = dc_pad8(Ly.out.K);
+    const float eps = m->stack->cfg.eps;
+    __nv_bfloat16 *lowb = st.b16 ? b.lowb : nullptr, *mixb = st.b16 ? b.mixb : nullptr;
+    if (st.single && st.T <= DC_MAX_T) return dc_launch_general_decode(m->ctx, d, st, sr, b.proj, ldp, eps, b.mix, mixb, ldm);
+    DC_TRY(dc_launch_general_tanh(m->ctx, d, st.T, b.proj, ldp, lowb, ldl));
+    DC_TRY(linear(m, st, d.w2, b.proj + d.off_w, lowb, st.b16 ? ldl : ldp, to(b.low, d.w2.N)));
+    return dc_launch_general_scan(m->ctx, d, st, sr, b.proj, ldp, b.low, d.w2.N, b.blk, eps, b.scan, ldo, b.mix, mixb, ldm);
 }
 
 int mix_lightning(dc_model* m, const dc_step& st, const dc_stack_run& run, dc_stack_layer& Ly) {
     const dc_lightning_mixer& d = Ly.li;
     const dc_stack_buffers& b = m->stack->b;
     const dc_state_ref sr = {m->kv.state, m->kv.state_bytes, run.state_off, 0};
-    const int lda = Ly.ff ? Ly.pair0 : Ly.in.N, ldy = dc_pad8(d.heads * d.vdim), ldm = dc_pad8(Ly.out.K);
+    const int lda = mixer_rows(Ly), ldy = dc_pad8(d.heads * d.vdim), ldm = dc_pad8(Ly.out.K);
     const __nv_bfloat16* actb = st.b16 ? b.actb : nullptr;
     if (st.single && st.T <= DC_MAX_T) DC_TRY(dc_launch_lightning_decode(m->ctx, d, st, sr, b.proj, actb, lda, b.scan, ldy));
     else if (st.b16) DC_TRY(dc_launch_lightning_chunks(m->ctx, d, st, sr, b.actb, lda, b.chunk_state, b.scan, ldy));
@@ -554,11 +587,11 @@ int parallel_layer(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_
     dc_stack* s = m->stack;
     dc_ctx* ctx = m->ctx;
     dc_stack_buffers& b = s->b;
-    const int W = s->cfg.width, H = dc_pad8(W), T = st.T, rows = Ly.ff ? Ly.pair0 : Ly.in.N, ldm = dc_pad8(Ly.out.K);
+    const int W = s->cfg.width, H = dc_pad8(W), T = st.T, rows = mixer_rows(Ly), ldm = dc_pad8(Ly.out.K);
     L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm1, nullptr, 0, T, W, H, s->cfg.eps, b.y, st.b16 ? b.xb : nullptr, H));
     const bool light = Ly.kind == DC_MIX_LIGHTNING;
     dc_lin_epi in = dc_lin_epi::store(b.proj, light && st.b16 ? b.actb : nullptr, rows);
-    if (light) in.silu_rows = Ly.li.off_g;
+    if (light) in.act_rows = Ly.li.off_g;
     else in.bias = Ly.ga.bias;
     if (Ly.ff) in.pairs(Ly.pair0, DC_PAIR_CLAMPED, Ly.limit, b.mix + Ly.out_ff, st.b16 ? b.mixb + Ly.out_ff : nullptr, ldm, Ly.ff);
     L(DC_K_MIX_IN, lin_bytes(Ly.in, T), 1, linear(m, st, Ly.in, b.y, b.xb, H, in));
@@ -571,31 +604,35 @@ int parallel_layer(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_
     return DC_B200_OK;
 }
 
-// x += the layer's experts on norm2(x).  Steps of up to DC_MAX_T tokens of bf16 models add to x at once; the others leave
-// a row of every chosen expert behind, which *owed names.
-int moe_layer(dc_model* m, const dc_step& st, dc_stack_layer& Ly, dc_row_sum* owed) {
+// The layer's experts on norm2 of the residual: of x, or (hy) of its streams, which are brought up to date on the way.  Steps of
+// up to DC_MAX_T tokens of bf16 models add to x at once, with streams they leave y in b.y; the others leave a row of every chosen
+// expert behind, which *owed names.
+int moe_layer(dc_model* m, const dc_step& st, dc_stack_layer& Ly, const dc_hyper* hy, dc_row_sum* owed) {
     dc_stack* s = m->stack;
     dc_ctx* ctx = m->ctx;
     dc_stack_buffers& b = s->b;
     const dc_moe_ffn& f = Ly.moe;
     const int W = s->cfg.width, H = dc_pad8(W), T = st.T, rows = T * f.top, F = dc_pad8(f.ff);
     __nv_bfloat16* xb = st.b16 ? b.xb : nullptr;
+    float* h = hy ? b.h : b.y;
     const double up_bytes = (double)f.up_rows * f.up.ld * 2, down_bytes = (double)f.down_rows * f.down.ld * 2;
     const double touched = std::min<double>(f.experts, rows);
     if (dc_moe_norm_route_fits(f, st.b16, T, H)) {
-        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, dc_launch_moe_norm_route(ctx, f, b.x, Ly.norm2, T, W, H, s->cfg.eps, b.y, xb, b.moe_ids, b.moe_w));
+        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, dc_launch_moe_norm_route(ctx, f, b.x, hy, Ly.norm2, T, W, H, s->cfg.eps, h, xb, b.moe_ids, b.moe_w));
     } else {
-        L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, b.y, xb, H));
-        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, linear(m, st, f.router, b.y, b.xb, H, to(b.moe_logits, f.router.N)));
+        if (hy) L(DC_K_PRE_NORM, hyper_bytes(m, T), 1, dc_launch_hyper_norm(ctx, *hy, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, h, xb));
+        else L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, h, xb, H));
+        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, linear(m, st, f.router, h, b.xb, H, to(b.moe_logits, f.router.N)));
         L(DC_K_ROUTER, 4.0 * T * f.experts, 1, dc_launch_moe_route(ctx, f, b.moe_logits, f.router.N, T, b.moe_ids, b.moe_w));
     }
     if (st.b16 && T <= DC_MAX_T) {
         L(DC_K_MOE_GATEUP, touched * up_bytes, 1, dc_launch_moe_up_mma(ctx, f, b.xb, H, T, b.moe_ids, b.moe_w, b.moe_hidb, F));
-        L(DC_K_MOE_DOWN, touched * down_bytes, 1, dc_launch_moe_down_mma(ctx, f, b.moe_hidb, F, T, b.moe_ids, W, b.x, H));
+        L(DC_K_MOE_DOWN, touched * down_bytes, 1, dc_launch_moe_down_mma(ctx, f, b.moe_hidb, F, T, b.moe_ids, W, hy ? b.y : b.x, H, !hy));
         return DC_B200_OK;
     }
     L(DC_K_ROUTER, 16.0 * rows, 1, dc_launch_moe_order(ctx, f, b.moe_ids, b.moe_w, T, b.moe_off, b.moe_src, b.moe_row_w, b.moe_row));
-    dc_lin_epi hid = dc_lin_epi().pairs(0, DC_PAIR_CLAMPED, f.limit, b.moe_hid, b.moe_hidb, F, f.ff);
+    dc_lin_epi hid = f.plain ? dc_lin_epi::store(b.moe_hid, b.moe_hidb, F) : dc_lin_epi().pairs(0, DC_PAIR_CLAMPED, f.limit, b.moe_hid, b.moe_hidb, F, f.ff);
+    if (f.plain) hid.act_rows = f.up_rows, hid.act = DC_ACT_RELU2;
     hid.tok_scale = b.moe_row_w;
     const dc_lin_epi y = dc_lin_epi::store(b.moe_y, b.moe_yb, H);
     if (st.b16) {
@@ -606,7 +643,7 @@ int moe_layer(dc_model* m, const dc_step& st, dc_stack_layer& Ly, dc_row_sum* ow
         DC_TRY(tc_in(m, &in, b.moe_hidb, f.ff, F, b.moe_rows));
         L(DC_K_MOE_DOWN, touched * down_bytes + 2.0 * rows * (W + f.ff), 1, dc_launch_linear_grouped_tc(ctx, f.down, f.experts, f.down_rows, b.moe_off, in, rows, y));
     } else {
-        L(DC_K_MOE_GATEUP, touched * up_bytes, 1, dc_launch_moe_f32(ctx, f.up, f.experts, f.up_rows, b.moe_off, rows, b.y, H, b.moe_src, hid));
+        L(DC_K_MOE_GATEUP, touched * up_bytes, 1, dc_launch_moe_f32(ctx, f.up, f.experts, f.up_rows, b.moe_off, rows, h, H, b.moe_src, hid));
         L(DC_K_MOE_DOWN, touched * down_bytes, 1, dc_launch_moe_f32(ctx, f.down, f.experts, f.down_rows, b.moe_off, rows, b.moe_hid, F, nullptr, y));
     }
     owed->y = b.moe_y, owed->yb = b.moe_yb, owed->rows = b.moe_row, owed->k = f.top, owed->ld = H;
@@ -632,24 +669,65 @@ int pre_norm_layer(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_
     dc_lin_epi out = to(b.x, H);
     out.add = true;
     L(DC_K_MIX_OUT, lin_bytes(o, T), 1, linear(m, st, o, b.mix, b.mixb, dc_pad8(o.K), out));
-    return Ly.moe.experts ? moe_layer(m, st, Ly, owed) : DC_B200_OK;
+    return Ly.moe.experts ? moe_layer(m, st, Ly, nullptr, owed) : DC_B200_OK;
 }
 
-// Embedding and every layer; the residual ends in b.x.
-int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
+// The streams as the next sublayer (coefficients next) finds them; afterwards they lie in the other buffer and owe y.
+dc_hyper hyper_next(dc_model* m, dc_hyper* hy, const float* next) {
+    const dc_stack_buffers& b = m->stack->b;
+    dc_hyper now = *hy;
+    now.next = next;
+    now.x_out = hy->x == b.x ? b.x2 : b.x;
+    hy->x = now.x_out, hy->first = false, hy->done = next, hy->y = b.y, hy->sum = dc_row_sum();
+    return now;
+}
+
+// Hyper-connected sublayers, mixer and feed-forward: u from the streams, y = f(norm(u)), which the streams then owe.
+int hyper_layer(dc_model* m, const dc_step& st, const StepKeys& sk, const dc_stack_run& run, dc_stack_layer& Ly, dc_hyper* hy) {
+    dc_stack* s = m->stack;
+    dc_ctx* ctx = m->ctx;
+    dc_stack_buffers& b = s->b;
+    const int W = s->cfg.width, H = dc_pad8(W), T = st.T;
+    __nv_bfloat16* xb = st.b16 ? b.xb : nullptr;
+    L(DC_K_PRE_NORM, hyper_bytes(m, T), 1, dc_launch_hyper_norm(ctx, hyper_next(m, hy, Ly.hyper[0]), Ly.norm1, nullptr, 0, T, W, H, s->cfg.eps, b.h, xb));
+    L(DC_K_MIX_IN, lin_bytes(Ly.in, T), 1, linear(m, st, Ly.in, b.h, b.xb, H, to(b.proj, Ly.in.N)));
+    if (Ly.kind == DC_MIX_GENERAL) L(DC_K_MIX_GENERAL, 8.0 * st.E * Ly.ge.heads * Ly.ge.dim * Ly.ge.dim, st.single && !st.tc ? 1 : 5, mix_general(m, st, run, Ly));
+    else L(DC_K_MIX_GQA, 4.0 * T * Ly.in.N, st.tc ? 2 : 3, mix_gqa(m, st, sk, run, Ly));
+    L(DC_K_MIX_OUT, lin_bytes(Ly.out, T), 1, linear(m, st, Ly.out, b.mix, b.mixb, dc_pad8(Ly.out.K), to(b.y, H)));
+    if (Ly.moe.experts) {
+        const dc_hyper now = hyper_next(m, hy, Ly.hyper[1]);
+        return moe_layer(m, st, Ly, &now, &hy->sum);
+    }
+    if (!Ly.ff) return DC_B200_OK;
+    const int F = dc_pad8(Ly.ff);
+    L(DC_K_PRE_NORM, hyper_bytes(m, T), 1, dc_launch_hyper_norm(ctx, hyper_next(m, hy, Ly.hyper[1]), Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, b.h, xb));
+    L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.h, b.xb, H, dc_lin_epi().pairs(0, Ly.ff_pair, 0.0f, b.ff, st.b16 ? b.ffb : nullptr, F, F)));
+    L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, to(b.y, H)));
+    return DC_B200_OK;
+}
+
+// Embedding and every layer; the residual ends in b.x, several streams in *hy.
+int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk, dc_hyper* hy) {
     dc_stack* s = m->stack;
     dc_ctx* ctx = m->ctx;
     dc_stack_buffers& b = s->b;
     const int W = s->cfg.width, H = dc_pad8(W), T = st.T;
     const float eps = s->cfg.eps;
     __nv_bfloat16* xb = st.b16 ? b.xb : nullptr;
+    const bool hyper = s->cfg.block == DC_BLOCK_HYPER;
     auto capture = [&](int il) -> int {     // parity aid: what enters layer il (the last slot: the output norm)
         if (!m->dbg_x || T > DC_MAX_T) return DC_B200_OK;
-        return dc_check_cuda(ctx, cudaMemcpy2DAsync(m->dbg_x + (size_t)il * DC_MAX_T * W, (size_t)W * 4, b.x, (size_t)H * 4, (size_t)W * 4, T,
+        const float* x = b.x;
+        if (hyper) {                        // the streams' sum
+            DC_TRY(dc_launch_hyper_norm(ctx, *hy, nullptr, nullptr, 0, T, W, H, eps, b.h, nullptr));
+            x = b.h;
+        }
+        return dc_check_cuda(ctx, cudaMemcpy2DAsync(m->dbg_x + (size_t)il * DC_MAX_T * W, (size_t)W * 4, x, (size_t)H * 4, (size_t)W * 4, T,
                                                     cudaMemcpyDeviceToDevice, ctx->stream), "capture");
     };
     m->last_launches = 0;
-    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, b.x, H, s->cfg.block == DC_BLOCK_POST_NORM ? xb : nullptr, s->cfg.embed_scale));
+    L(DC_K_EMBED, (double)T * W * 6, 1, dc_launch_embed(ctx, s->embed, st.tokens, T, hyper ? b.y : b.x, H, s->cfg.block == DC_BLOCK_POST_NORM ? xb : nullptr, s->cfg.embed_scale));
+    if (hyper) hy->streams = s->cfg.streams, hy->mul = s->cfg.residual_mult, hy->x = b.y, hy->first = true;
     dc_row_sum owed;
     auto settle = [&]() -> int {
         if (!owed.k) return DC_B200_OK;
@@ -662,6 +740,10 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
         dc_stack_layer& Ly = s->layers[run.layer];
         if (m->dbg_x) DC_TRY(settle());
         DC_TRY(capture((int)il));
+        if (hyper) {
+            DC_TRY(hyper_layer(m, st, sk, run, Ly, hy));
+            continue;
+        }
         if (s->cfg.block == DC_BLOCK_PARALLEL) {
             DC_TRY(parallel_layer(m, st, sk, run, Ly));
             continue;
@@ -680,7 +762,7 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm1, T, W, H, eps, xb));
         if (!Ly.ff) continue;
         const int F = dc_pad8(Ly.ff);
-        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, dc_lin_epi().pairs(0, DC_PAIR_GELU, 0.0f, b.ff, st.b16 ? b.ffb : nullptr, F, F)));
+        L(DC_K_FFN_GATEUP, lin_bytes(Ly.gate_up, T), 1, linear(m, st, Ly.gate_up, b.x, xb, H, dc_lin_epi().pairs(0, Ly.ff_pair, 0.0f, b.ff, st.b16 ? b.ffb : nullptr, F, F)));
         L(DC_K_FFN_DOWN, lin_bytes(Ly.down, T), 1, linear(m, st, Ly.down, b.ff, b.ffb, F, to(b.y, H)));
         L(DC_K_POST_NORM, 12.0 * T * W, 1, dc_launch_post_norm(ctx, b.x, b.y, Ly.norm2, T, W, H, eps, xb));
     }
@@ -689,12 +771,13 @@ int run_layers(dc_model* m, const dc_step& st, const StepKeys& sk) {
 }
 
 // Logits and greedy picks of R <= DC_MAX_T rows (rows: device list, or first, first + 1, ...).
-int run_head(dc_model* m, const int32_t* rows, int first, int R, bool feedback) {
+int run_head(dc_model* m, const dc_hyper& hy, const int32_t* rows, int first, int R, bool feedback) {
     dc_stack* s = m->stack;
     dc_ctx* ctx = m->ctx;
     const int W = s->cfg.width, H = dc_pad8(W);
     dc_step_buffers& g = m->buf;
-    L(DC_K_POST_NORM, 8.0 * R * W, 1, dc_launch_norm_rows(ctx, s->b.x, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, s->b.lm_xb, H));
+    if (hy.x) L(DC_K_PRE_NORM, hyper_bytes(m, R), 1, dc_launch_hyper_norm(ctx, hy, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, s->b.lm_xb));
+    else L(DC_K_POST_NORM, 8.0 * R * W, 1, dc_launch_norm_rows(ctx, s->b.x, s->final_norm, rows, first, R, W, H, s->cfg.eps, s->b.lm_x, s->b.lm_xb, H));
     L(DC_K_LM_HEAD, lin_bytes(s->head, R), 1,
       s->b.lm_xb ? dc_launch_linear_mma(ctx, s->head, s->b.lm_xb, H, R, dc_lin_epi::store(g.logits, nullptr, s->cfg.vocab, g.argmax_keys))
                  : dc_launch_linear_rows(ctx, s->head, s->b.lm_x, H, R, dc_lin_epi::store(g.logits, nullptr, s->cfg.vocab, g.argmax_keys)));
@@ -714,9 +797,10 @@ int dc_stack_enqueue_small(dc_model* m, int T, bool chunk, int lm_mode, bool fee
     st.starts = chunk ? m->stack->b.chunk + 2 * T : m->stack->b.iota;
     st.single = !chunk || T == 1;
     st.b16 = m->stack->dtype == DC_DTYPE_BF16;
-    DC_TRY(run_layers(m, st, StepKeys()));
-    if (lm_mode == 1) return run_head(m, nullptr, T - 1, 1, feedback);
-    return lm_mode ? run_head(m, nullptr, 0, T, feedback) : DC_B200_OK;
+    dc_hyper hy;
+    DC_TRY(run_layers(m, st, StepKeys(), &hy));
+    if (lm_mode == 1) return run_head(m, hy, nullptr, T - 1, 1, feedback);
+    return lm_mode ? run_head(m, hy, nullptr, 0, T, feedback) : DC_B200_OK;
 }
 
 int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* counts, const int32_t* tokens, int n_rows, const int32_t* rows,
@@ -780,10 +864,11 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
         sk.tiles = b.meta + (h_tiles - h);
         st.b16 = s->dtype == DC_DTYPE_BF16;
         st.tc = st.b16 && st.T > DC_MAX_T;
-        DC_TRY(run_layers(m, st, sk));
+        dc_hyper hy;
+        DC_TRY(run_layers(m, st, sk, &hy));
         for (int r = 0; r < R; r += DC_MAX_T) {
             const int n = std::min(DC_MAX_T, R - r);
-            DC_TRY(run_head(m, b.meta + 3 * C + r, 0, n, false));
+            DC_TRY(run_head(m, hy, b.meta + 3 * C + r, 0, n, false));
             if (logits_host)
                 DC_TRY(dc_check_cuda(ctx, cudaMemcpyAsync(logits_host + (size_t)(next_row + r) * V, m->buf.logits, (size_t)n * V * 4, cudaMemcpyDeviceToHost,
                                                           ctx->stream), "D2H logits"));
@@ -799,13 +884,15 @@ int dc_stack_batch(dc_model* m, int E, const int32_t* seqs, const int32_t* count
 void dc_stack_stats(dc_model* m, double* weight_bytes, double* kv_bytes_per_token) {
     dc_stack* s = m->stack;
     double w = (double)s->head.N * s->head.ld * 2 + (s->cfg.tied ? 0.0 : (double)s->embed->row_bytes), kv = 0.0;
-    if (s->cfg.block != DC_BLOCK_PRE_NORM) {
+    bool experts = false;
+    for (const dc_stack_layer& L : s->layers) experts |= L.moe.experts > 0;
+    if (!experts) {
         w = (double)s->weight_bytes - (double)s->embed->bytes + (s->cfg.tied ? 0.0 : (double)s->embed->row_bytes);
     } else {
         for (const dc_stack_run& r : s->runs) {         // every run reads its layer; of the experts, those that a token chooses
             const dc_stack_layer& L = s->layers[r.layer];
             const dc_moe_ffn& f = L.moe;
-            for (const dc_lin* l : {&L.la.in, &L.la.ukv, &L.la.o, &L.in, &L.out, &f.router}) w += (double)l->N * l->ld * 2;
+            for (const dc_lin* l : {&L.la.in, &L.la.ukv, &L.la.o, &L.in, &L.out, &L.ge.w2, &L.gate_up, &L.down, &f.router}) w += (double)l->N * l->ld * 2;
             if (f.experts) w += ((double)f.up.N * f.up.ld + (double)f.down.N * f.down.ld) * 2 * f.top / f.experts;
         }
     }

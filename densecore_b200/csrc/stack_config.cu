@@ -24,6 +24,7 @@ struct Reader {
     dc_stack* s;
     const Shapes* shapes;
     std::string error;      // first problem found
+    float norm_plus = 0.0f; // norm weights are stored as their distance from this
 
     void bad(const std::string& what) {
         if (error.empty()) error = what;
@@ -108,6 +109,11 @@ struct Reader {
         t.neg_exp = neg_exp;
         t.synth = synth;
         tensor(t);
+    }
+    // a norm's weight over the residual
+    void norm(float** p, const std::string& name) {
+        vec(p, name, {s->cfg.width}, norm_plus > 0.0f ? 0 : 1);
+        s->tensors.back().plus = norm_plus;
     }
     // convolution weights [n, taps], kept as [taps][cols]
     void conv(float** p, const std::string& name, int n, int taps, int off, int cols) {
@@ -251,6 +257,11 @@ enum {
     GQA_HALVES = 32,        // rotated pairs (i, i + dims / 2)
     GQA_SINK = 64,          // a sink of score 0
     GQA_TWO_MAPS = 128,     // differential attention
+    GQA_UNTURNED = 256,     // no rotation
+    GQA_CONV = 512,         // short convolutions behind the projections
+    GQA_UNIT = 1024,        // queries, keys and values over their root mean square per head, no weights
+    GQA_SIGMOID = 2048,     // sigmoid weights with a bias per head
+    GQA_GATE = 4096,        // a gate per head
 };
 
 void read_gqa(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L, unsigned form) {
@@ -264,7 +275,8 @@ void read_gqa(Reader& r, const dc_json& j, const std::string& p, const std::stri
     if (form & GQA_KEY_VALUES && d.vdim != d.dim) r.bad(where + ": the values are the keys, so vdim must equal dim");
     if (d.heads % d.kv_heads) r.bad(where + ": heads is not a multiple of kv_heads");
     d.scale = (float)r.number(j, "scale", where);
-    if (const dc_json* rot = r.object(j, "rot", where)) r.rotation(*rot, where + ".rot", &d.rot);
+    if (!(form & GQA_UNTURNED))
+        if (const dc_json* rot = r.object(j, "rot", where)) r.rotation(*rot, where + ".rot", &d.rot);
     if (d.rot.dims > d.dim) r.bad(where + ".rot: dims is larger than the head");
     d.halves = form & GQA_HALVES;
     r.mask(j, where, &d.window, &d.keep);
@@ -287,11 +299,22 @@ void read_gqa(Reader& r, const dc_json& j, const std::string& p, const std::stri
         r.vec(&d.bias, p + "k.b", {K}, 4, d.off_k, rows);
         if (own_values) r.vec(&d.bias, p + "v.b", {V}, 4, d.off_v, rows);
     }
-    if (d.qk_norm != DC_QK_PLAIN) {
+    if (form & GQA_UNIT) {
+        d.qk_norm = DC_QK_NORM_HEAD, d.v_norm = true;
+    } else if (d.qk_norm != DC_QK_PLAIN) {
         const bool all = d.qk_norm == DC_QK_NORM_ALL;
         r.vec(&d.q_norm, p + "q.norm", {all ? Q : d.dim}, 1);
         r.vec(&d.k_norm, p + "k.norm", {all ? K : d.dim}, 1);
     }
+    if (form & GQA_CONV) {       // weights sit at the channels' projection columns, so that one index serves both
+        d.taps = r.size(j, "conv", where, 1, 16);
+        const int C = dc_gqa_conv_cols(d);
+        r.conv(&d.conv, p + "q.conv", Q, d.taps, d.off_q, C);
+        r.conv(&d.conv, p + "k.conv", K, d.taps, d.off_k, C);
+        r.conv(&d.conv, p + "v.conv", V, d.taps, d.off_v, C);
+    }
+    if (form & GQA_SIGMOID) r.vec(&d.score_bias, p + "pb", {d.heads}, 3);
+    if (form & GQA_GATE) d.off_g = r.matrix(&L->in, p + "g", d.heads, H);
     if (d.maps > 1) {
         const char* names[] = {"lq1", "lk1", "lq2", "lk2"};
         for (int i = 0; i < 4; ++i) r.vec(&d.lam[i], p + names[i], {d.dim}, 0);
@@ -324,6 +347,34 @@ void read_lightning(Reader& r, const dc_json& j, const std::string& p, const std
     out_columns(r, p + "o", L, V);
 }
 
+void read_general(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+    dc_general_mixer& d = L->ge;
+    const int H = r.s->cfg.width;
+    d.heads = r.size(j, "heads", where);
+    d.dim = r.size(j, "dim", where, 1, 256);
+    d.rank = r.from_shape(p + "w1", 0);
+    const int Q = d.heads * d.dim;
+    d.off_r = r.matrix(&L->in, p + "r", Q, H);
+    d.off_k = r.matrix(&L->in, p + "k", Q, H);
+    d.off_v = r.matrix(&L->in, p + "v", Q, H);
+    d.off_g = r.matrix(&L->in, p + "g", Q, H);
+    d.off_a = r.matrix(&L->in, p + "a", Q, H);
+    d.off_w = r.matrix(&L->in, p + "w1", d.rank, H);
+    r.matrix(&d.w2, p + "w2", Q, d.rank);
+    r.vec(&d.w0, p + "w0", {Q}, 4);
+    r.vec(&d.a_bias, p + "a.b", {Q}, 4);
+    r.vec(&d.norm, p + "norm", {Q}, 1);
+    out_columns(r, p + "o", L, Q);
+}
+
+// Coefficients of a sublayer's hyper-connections
+void read_hyper(Reader& r, const std::string& p, float** to) {
+    const int n = r.s->cfg.streams, all = n * (n + 2);
+    r.vec(to, p + "in", {n}, 5, 0, all);
+    r.vec(to, p + "out", {n}, 1, n, all);
+    r.vec(to, p + "mix", {n, n}, 5, 2 * n, all);
+}
+
 // Gate and up rows in turn from L->pair0 of the input matrix, the down matrix beside the mixer's output matrix.
 void read_dense_clamped(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
     const int H = r.s->cfg.width;
@@ -344,8 +395,9 @@ void read_dense_clamped(Reader& r, const dc_json& j, const std::string& p, const
     out_columns(r, p + "down", L, L->ff);
 }
 
-void read_dense_gelu(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+void read_dense(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L, int pair) {
     const int H = r.s->cfg.width;
+    L->ff_pair = pair;
     L->ff = r.size(j, "ff", where);
     L->gate_up.N = 2 * dc_pad8(L->ff);
     L->gate_up.K = H;
@@ -361,15 +413,23 @@ void read_dense_gelu(Reader& r, const dc_json& j, const std::string& p, const st
     r.matrix(&L->down, p + "down", H, L->ff);
 }
 
-void read_moe(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L) {
+// What a design fixes of its experts
+enum {
+    MOE_CLAMPED = 1,        // clamped gated experts behind a sigmoid router
+    MOE_SOFTMAX = 2,        // softmax router, chosen scores divided by their sum
+    MOE_PLAIN = 4,          // square of relu between two matrices
+};
+
+void read_moe(Reader& r, const dc_json& j, const std::string& p, const std::string& where, dc_stack_layer* L, unsigned form) {
     dc_moe_ffn& f = L->moe;
     const int H = r.s->cfg.width;
     const dc_json *router = r.object(j, "router", where), *expert = r.object(j, "expert", where);
     if (!router || !expert) return;
     f.experts = r.size(*router, "experts", where + ".router", 1, DC_MOE_MAX_EXPERTS);
     f.top = r.size(*router, "top", where + ".router", 1, DC_MOE_MAX_TOP);
-    f.scale = (float)r.number(*router, "scale", where + ".router");
-    const dc_json* groups = router->get("groups");
+    f.softmax = form & MOE_SOFTMAX, f.plain = form & MOE_PLAIN;
+    if (!f.softmax) f.scale = (float)r.number(*router, "scale", where + ".router");
+    const dc_json* groups = f.softmax ? nullptr : router->get("groups");
     if (groups && !groups->is_null()) {
         f.groups = r.size(*groups, "count", where + ".router.groups", 1, DC_MOE_MAX_GROUPS);
         f.keep = r.size(*groups, "keep", where + ".router.groups");
@@ -377,24 +437,24 @@ void read_moe(Reader& r, const dc_json& j, const std::string& p, const std::stri
     if (f.experts % f.groups) r.bad(where + ".router: experts is not a multiple of groups.count");
     else if (f.keep > f.groups || f.top > f.experts / f.groups * f.keep) r.bad(where + ".router: fewer experts than 'top' in the kept groups");
     f.ff = r.size(*expert, "ff", where + ".expert");
-    f.limit = (float)r.number(*expert, "limit", where + ".expert");
+    if (!f.plain) f.limit = (float)r.number(*expert, "limit", where + ".expert");
     if (!r.error.empty()) return;
-    f.up_rows = 2 * dc_pad8(f.ff);
+    f.up_rows = f.plain ? (f.ff + 15) & ~15 : 2 * dc_pad8(f.ff);
     f.down_rows = (H + 15) & ~15;
     r.matrix(&f.router, p + "router", f.experts, H);
-    r.vec(&f.correction, p + "correction", {f.experts}, 4);
+    if (!f.softmax) r.vec(&f.correction, p + "correction", {f.experts}, 4);
     f.up.N = f.experts * f.up_rows, f.up.K = H;
     f.down.N = f.experts * f.down_rows, f.down.K = f.ff;
     for (int e = 0; e < f.experts; ++e) {
         const std::string in = p + "e" + std::to_string(e) + ".";
-        for (int i = 0; i < 3; ++i) {
+        for (int i = f.plain ? 1 : 0; i < 3; ++i) {
             const bool down = i == 2;
             dc_stack_tensor t;
             t.name = in + (down ? "down" : i ? "up" : "gate");
             t.shape = {down ? H : f.ff, down ? f.ff : H};
             t.lin = down ? &f.down : &f.up;
-            t.row0 = down ? e * f.down_rows : e * f.up_rows + i;
-            t.row_step = down ? 1 : 2;
+            t.row0 = down ? e * f.down_rows : e * f.up_rows + (f.plain ? 0 : i);
+            t.row_step = down || f.plain ? 1 : 2;
             r.tensor(t);
         }
     }
@@ -420,23 +480,30 @@ struct MixerType {
 };
 struct Arch {
     const char* name;
-    int block;              // DC_BLOCK_*: post-norm blocks have the tanh-gelu feed-forward, parallel ones the clamped one, pre-norm ones experts
+    int block;              // DC_BLOCK_*
     bool embed_scale;       // config.embedding.scale
     bool tied;
     bool loops;             // config.loop
+    float norm_plus;        // norm weights are stored as their distance from this
+    int dense;              // pairs of the dense feed-forward (-1: none)
+    unsigned moe;           // form of the experts (0: none)
     std::vector<MixerType> mixers;
 };
 const Arch kArchs[] = {
     // Garilix: RMS norms on the sublayers' outputs only (x += norm(f(x))), tanh-gelu gated feed-forward
-    {"Garilix", DC_BLOCK_POST_NORM, false, false, false,
+    {"Garilix", DC_BLOCK_POST_NORM, false, false, false, 0.0f, DC_PAIR_GELU, 0,
      {{"channel_delta", DC_MIX_DELTA, 0}, {"latent_attention", DC_MIX_LATENT, 0}, {"mamba2", DC_MIX_SSD, 0}}},
     // Datasun: mixer and clamped feed-forward side by side on one normed input, embedding table as output matrix
-    {"Datasun", DC_BLOCK_PARALLEL, true, true, false,
+    {"Datasun", DC_BLOCK_PARALLEL, true, true, false, 0.0f, DC_PAIR_CLAMPED, 0,
      {{"attention", DC_MIX_GQA, GQA_KEY_VALUES | GQA_BIAS | GQA_OUT_BIAS | GQA_NORM_ALL | GQA_SINK}, {"lightning", DC_MIX_LIGHTNING, 0}}},
     // Gomuzen: norms ahead of the sublayers, looped layers, gated latent attention, differential attention, biased attention over
     // a window and the first tokens, experts in groups
-    {"Gomuzen", DC_BLOCK_PRE_NORM, false, false, true,
+    {"Gomuzen", DC_BLOCK_PRE_NORM, false, false, true, 0.0f, -1, MOE_CLAMPED,
      {{"latent_attention", DC_MIX_LATENT, 1}, {"attention", DC_MIX_GQA, GQA_NORM_HEAD | GQA_HALVES | GQA_TWO_MAPS}, {"attention_2", DC_MIX_GQA, GQA_BIAS | GQA_HALVES}}},
+    // Vepitar: hyper-connections over several streams, generalized delta rule, attention with sigmoid weights and short
+    // convolutions, dense layers or experts behind a softmax router, embedding table as output matrix
+    {"Vepitar", DC_BLOCK_HYPER, false, true, false, 1.0f, DC_PAIR_SILU, MOE_SOFTMAX | MOE_PLAIN,
+     {{"general_delta", DC_MIX_GENERAL, 0}, {"attention", DC_MIX_GQA, GQA_UNTURNED | GQA_CONV | GQA_UNIT | GQA_SIGMOID | GQA_GATE}}},
 };
 
 int alloc_lin(dc_model* m, dc_lin* l) {
@@ -454,7 +521,7 @@ int alloc_lin(dc_model* m, dc_lin* l) {
 
 int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
     dc_stack* s = m->stack = new dc_stack();
-    Reader r{m, s, &shapes, ""};
+    Reader r{m, s, &shapes, "", 0.0f};
     const dc_json* arch = cj.get("architecture");
     const Arch* a = nullptr;
     for (const Arch& e : kArchs)
@@ -471,6 +538,11 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
     const dc_json* norm = cj.get("norm");
     if (norm && norm->kind == dc_json::OBJ) s->cfg.eps = (float)r.number(*norm, "eps", "config.norm");
     else r.bad("config: 'norm' is missing");
+    r.norm_plus = a->norm_plus;
+    if (a->block == DC_BLOCK_HYPER) {
+        s->cfg.streams = r.size(cj, "streams", "config", 1, DC_MAX_STREAMS);
+        s->cfg.residual_mult = (float)r.number(cj, "residual_mult", "config");
+    }
     const dc_json* layers = cj.get("layers");
     if (!layers || layers->kind != dc_json::ARR || layers->arr.empty()) r.bad("config: 'layers' is missing");
     if (!r.error.empty()) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "%s", r.error.c_str());
@@ -508,23 +580,24 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         if (L.kind == DC_MIX_DELTA) read_delta(r, *mixer, p + "mix.", where + ".mixer", &L);
         else if (L.kind == DC_MIX_SSD) read_ssd(r, *mixer, p + "mix.", where + ".mixer", &L);
         else if (L.kind == DC_MIX_GQA) read_gqa(r, *mixer, p + "mix.", where + ".mixer", &L, form);
+        else if (L.kind == DC_MIX_GENERAL) read_general(r, *mixer, p + "mix.", where + ".mixer", &L);
         else if (L.kind == DC_MIX_LIGHTNING) read_lightning(r, *mixer, p + "mix.", where + ".mixer", &L);
         else read_latent(r, *mixer, p + "mix.", where + ".mixer", &L, i, form);
-        r.vec(&L.norm1, p + "norm1", {H}, 1);
+        const bool hyper = a->block == DC_BLOCK_HYPER;
+        r.norm(&L.norm1, p + "norm1");
+        if (hyper) read_hyper(r, p + "hc1.", &L.hyper[0]);
         if (mlp && !mlp->is_null()) {
             const dc_json* kind = mlp->get("kind");
-            const bool pre = a->block == DC_BLOCK_PRE_NORM;
-            if (!kind || kind->str != (pre ? "moe" : "dense")) {
+            const std::string name = kind && kind->kind == dc_json::STR ? kind->str : "";
+            if (!(name == "dense" && a->dense >= 0) && !(name == "moe" && a->moe)) {
                 r.bad(where + ".mlp: unknown kind");
                 break;
             }
-            if (a->block == DC_BLOCK_PARALLEL) {
-                read_dense_clamped(r, *mlp, p + "mlp.", where + ".mlp", &L);
-            } else {
-                if (pre) read_moe(r, *mlp, p + "mlp.", where + ".mlp", &L);
-                else read_dense_gelu(r, *mlp, p + "mlp.", where + ".mlp", &L);
-                r.vec(&L.norm2, p + "norm2", {H}, 1);
-            }
+            if (name == "moe") read_moe(r, *mlp, p + "mlp.", where + ".mlp", &L, a->moe);
+            else if (a->block == DC_BLOCK_PARALLEL) read_dense_clamped(r, *mlp, p + "mlp.", where + ".mlp", &L);
+            else read_dense(r, *mlp, p + "mlp.", where + ".mlp", &L, a->dense);
+            if (a->block != DC_BLOCK_PARALLEL) r.norm(&L.norm2, p + "norm2");
+            if (hyper) read_hyper(r, p + "hc2.", &L.hyper[1]);
         }
     }
     // the order in which layers run
@@ -541,7 +614,7 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
     run(0, start, -1);
     for (int t = 0; t < c.loop_times; ++t) run(start, stop, t);
     run(stop, n, -1);
-    r.vec(&s->final_norm, "final.norm", {H}, 1);
+    r.norm(&s->final_norm, "final.norm");
     if (!s->cfg.tied) r.matrix(&s->head, "head", s->cfg.vocab, H);
     if (!r.error.empty()) return dc_fail(m->ctx, DC_B200_INVALID_ARGUMENT, "%s", r.error.c_str());
 
@@ -562,7 +635,7 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
         DC_TRY(dc_check_cuda(m->ctx, cudaMalloc((void**)&s->embed->dev, s->embed->bytes + 64), "weight memory"));
     }
     for (dc_stack_layer& L : s->layers) {
-        dc_lin* ls[] = {&L.dl.in, &L.dl.a2, &L.dl.g2, &L.dl.o, &L.ssd.in, &L.ssd.o, &L.la.in, &L.la.ukv, &L.la.o, &L.gate_up, &L.down, &L.in, &L.out, &L.moe.router, &L.moe.up, &L.moe.down};
+        dc_lin* ls[] = {&L.dl.in, &L.dl.a2, &L.dl.g2, &L.dl.o, &L.ssd.in, &L.ssd.o, &L.la.in, &L.la.ukv, &L.la.o, &L.gate_up, &L.down, &L.in, &L.out, &L.moe.router, &L.moe.up, &L.moe.down, &L.ge.w2};
         for (dc_lin* l : ls) DC_TRY(alloc_lin(m, l));
         if (!L.li.decays.empty()) {
             const size_t bytes = L.li.decays.size() * 4;

@@ -338,6 +338,96 @@ def moe_mlp(h, P, mlp):
     return out
 
 
+def mix_general_delta(h, P, m, eps, st):
+    """S <- diag(w) S - (a u)(u^T S) + k v^T with the unit key u, o = S^T r; both terms read the old state."""
+    T, H, d = h.shape[0], m["heads"], m["dim"]
+    r, k, v = (linear(h, P[n]).reshape(T, H, d) for n in "rkv")
+    w = decay_below_one(linear(np.tanh(linear(h, P["w1"])), P["w2"]) + P["w0"].reshape(-1)).reshape(T, H, d)
+    a = sigmoid(linear(h, P["a"]) + P["a.b"].reshape(-1)).reshape(T, H, d)
+    if "S" not in st:
+        st["S"] = np.zeros((H, d, d), F)
+    o = removal_rule(r, k, v, w, a, unit_vectors(k), st["S"])
+    o = rms_norm(o, 1.0, eps).reshape(T, H * d) * P["norm"].reshape(-1)
+    return linear(o * sigmoid(linear(h, P["g"])), P["o"])
+
+
+def decay_below_one(z):
+    """exp(-e^(-1/2) sigmoid(z)): between 0.545 and 1."""
+    return np.exp(-np.exp(-0.5) * sigmoid(z))
+
+
+def removal_rule(r, k, v, w, a, u, S):
+    """All [T, H, d]; S [H, d, d] (changed in place).  Returns o [T, H, d]."""
+    o = np.zeros_like(v)
+    for t in range(r.shape[0]):
+        for h in range(r.shape[1]):
+            old = S[h].copy()
+            S[h] = w[t, h][:, None] * old - np.outer(a[t, h] * u[t, h], u[t, h] @ old) + np.outer(k[t, h], v[t, h])
+            o[t, h] = S[h].T @ r[t, h]
+    return o
+
+
+def sigmoid_attention(q, k, v, pos, scale, bias, window=None):
+    """q [T, H, d], k [n, G, d], v [n, G, e]: every visible key counts sigmoid(score + bias of the head), unnormalized."""
+    T, H, _ = q.shape
+    of = np.arange(H) // (H // k.shape[1])
+    out = np.zeros((T, H, v.shape[2]), F)
+    for t in range(T):
+        n = int(pos[t]) + 1
+        lo = max(0, n - window) if window else 0
+        s = np.einsum("hd,nhd->hn", q[t], k[lo:n, of]) * scale + bias[:, None]
+        out[t] = np.einsum("hn,nhe->he", sigmoid(s), v[lo:n, of])
+    return out
+
+
+def mix_sigmoid_attention(h, P, m, eps, pos, st):
+    """Grouped-query attention without rotation: short convolutions, norms of queries, keys and values per head, sigmoid weights,
+    a gate per head."""
+    T, H, G, d, e = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    z = {}
+    for n in "qkv":
+        z[n], st["conv." + n] = short_conv(linear(h, P[n]), P[n + ".conv"], None, st.get("conv." + n))
+    q = rms_norm(z["q"].reshape(T, H, d), 1.0, eps)
+    k, v = grow(st, k=rms_norm(z["k"].reshape(T, G, d), 1.0, eps), v=rms_norm(z["v"].reshape(T, G, e), 1.0, eps))
+    o = sigmoid_attention(q, k, v, pos, m["scale"], P["pb"].reshape(-1), (m.get("mask") or {}).get("size"))
+    o = o * sigmoid(linear(h, P["g"]))[:, :, None]
+    return linear(o.reshape(T, H * e), P["o"])
+
+
+def silu_mlp(h, P):
+    return linear(silu(linear(h, P["gate"])) * linear(h, P["up"]), P["down"])
+
+
+def softmax_route(z, top):
+    """Router logits of one token -> (chosen experts, their weights): the largest softmax scores, divided by their sum."""
+    s = np.exp(z - z.max())
+    s = s / s.sum()
+    ids = np.argsort(-s, kind="stable")[:top]
+    return ids, s[ids] / (s[ids].sum() + 1e-20)
+
+
+def squared_relu_mlp(h, P):
+    return linear(np.maximum(linear(h, P["up"]), 0.0) ** 2, P["down"])
+
+
+def softmax_moe_mlp(h, P, mlp):
+    out, z = np.zeros_like(h), linear(h, P["router"])
+    for t in range(h.shape[0]):
+        for i, wi in zip(*softmax_route(z[t], mlp["router"]["top"])):
+            out[t] += wi * squared_relu_mlp(h[t:t + 1], {n: P[f"e{i}.{n}"] for n in ("up", "down")})[0]
+    return out
+
+
+def hyper_input(x, hc):
+    """x [streams, T, W] -> the sublayer's input."""
+    return np.einsum("s,stw->tw", hc["in"].reshape(-1), x)
+
+
+def hyper_update(x, y, hc, mul):
+    """Every stream anew from all old ones (mix: [from, to]) and the sublayer's output."""
+    return np.einsum("st,snw->tnw", hc["mix"], x) + mul * hc["out"].reshape(-1)[:, None, None] * y
+
+
 # ---------------------------------------------------------------- the decoder
 def layer_runs(config):
     """(layer, pass that starts here or None) in the order in which layers run."""
@@ -365,16 +455,23 @@ class Stepper:
         residual after every layer."""
         tokens = np.asarray(tokens)
         pos = self.pos + np.arange(tokens.size)
-        layer = {"Garilix": self.garilix_layer, "Datasun": self.datasun_layer, "Gomuzen": self.gomuzen_layer}[self.c["architecture"]]
+        layer = {"Garilix": self.garilix_layer, "Datasun": self.datasun_layer, "Gomuzen": self.gomuzen_layer,
+                 "Vepitar": self.vepitar_layer}[self.c["architecture"]]
         x = self.w["embed"][tokens] * self.c.get("embedding", {}).get("scale", 1.0)
+        streams = self.c.get("streams")
+        plus = 1.0 if streams else 0.0          # norm weights stored around zero
+        if streams:
+            x = np.stack([x] * streams)
         for st, (i, t) in zip(self.state, self.runs):
             if t is not None:
                 x = x + self.w["loop.step"][t]
             x = layer(i, x, pos, st)
             if trace is not None:
-                trace.append(x.copy())
+                trace.append(x.sum(axis=0) if streams else x.copy())
         self.pos += tokens.size
-        return linear(rms_norm(x, self.w["final.norm"], self.c["norm"]["eps"]), self.w["head" if "head" in self.w else "embed"])
+        if streams:
+            x = x.sum(axis=0)
+        return linear(rms_norm(x, self.w["final.norm"] + plus, self.c["norm"]["eps"]), self.w["head" if "head" in self.w else "embed"])
 
     def garilix_layer(self, i, x, pos, st):
         L, P, eps = self.c["layers"][i], self.part(f"l{i}.mix."), self.c["norm"]["eps"]
@@ -422,6 +519,23 @@ class Stepper:
             raise ValueError(L["type"])
         if L.get("mlp"):
             x = x + moe_mlp(rms_norm(x, self.w[f"l{i}.norm2"], eps), self.part(f"l{i}.mlp."), L["mlp"])
+        return x
+
+    def vepitar_layer(self, i, x, pos, st):
+        L, P, eps, mul = self.c["layers"][i], self.part(f"l{i}.mix."), self.c["norm"]["eps"], self.c["residual_mult"]
+        hc = self.part(f"l{i}.hc1.")
+        h = rms_norm(hyper_input(x, hc), 1.0 + self.w[f"l{i}.norm1"], eps)
+        if L["type"] == "general_delta":
+            y = mix_general_delta(h, P, L["mixer"], eps, st)
+        elif L["type"] == "attention":
+            y = mix_sigmoid_attention(h, P, L["mixer"], eps, pos, st)
+        else:
+            raise ValueError(L["type"])
+        x = hyper_update(x, y, hc, mul)
+        if L.get("mlp"):
+            hc, P = self.part(f"l{i}.hc2."), self.part(f"l{i}.mlp.")
+            h = rms_norm(hyper_input(x, hc), 1.0 + self.w[f"l{i}.norm2"], eps)
+            x = hyper_update(x, softmax_moe_mlp(h, P, L["mlp"]) if L["mlp"]["kind"] == "moe" else silu_mlp(h, P), hc, mul)
         return x
 
 
