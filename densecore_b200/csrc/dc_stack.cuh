@@ -177,7 +177,7 @@ __device__ __forceinline__ void hyper_coefficients(const dc_hyper& h, float* c) 
         if (i < S) {
             if (i < n) v = h.next ? h.next[i] : 1.0f;
         } else if (i < 2 * S) {
-            if (i - S < n && h.done) v = h.mul * h.done[i];
+            if (i - S < n && h.done) v = h.mul * h.done[n + i - S];
         } else {
             const int s = (i - 2 * S) / S, t = (i - 2 * S) % S;
             if (s < n && t < n) v = h.done ? h.done[2 * n + s * n + t] : s == t ? 1.0f : 0.0f;
