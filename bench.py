@@ -400,6 +400,19 @@ def gomuzen_config(width: int, repeats: int, vocab: int = 32768):
             "layers": [dict(ly, mlp=mlp) for ly in (latent, diff, kept, kept) * repeats]}
 
 
+def vepitar_config(width: int, layers: int, vocab: int = 32768):
+    """A Vepitar decoder whose layers have the sizes of a real model of this width: one windowed attention layer to two recurrent
+    ones, a dense feed-forward in the first layer, then 64 experts of which a token uses 8 (as many weights as Gomuzen's), four
+    residual streams; and the shapes that its config does not give."""
+    att = {"type": "attention", "mixer": {"heads": width // 128, "kv_heads": max(1, width // 512), "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** -0.5,
+                                          "mask": {"size": 1024}}}
+    rec = {"type": "general_delta", "mixer": {"heads": width // 64, "dim": 64}}
+    moe = {"kind": "moe", "expert": {"ff": 9 * width // 16}, "router": {"experts": 64, "top": 8}}
+    out = [dict((rec, rec, att)[i % 3], mlp=moe if i else {"kind": "dense", "ff": 3 * width}) for i in range(layers)]
+    shapes = {f"l{i}.mix.w1": [max(32, width // 32), width] for i in range(layers) if i % 3 < 2}
+    return {"architecture": "Vepitar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 4, "residual_mult": 0.5, "layers": out}, shapes
+
+
 def time_decoder(m, vocab: int, prompt: int, streams, steps: int, reps: int = 5) -> dict:
     """Prompt throughput (host tokens in, first token out, best of reps on fresh sequences) and greedy decode after
     that prompt (device time of decode_run) of any decoder of the library."""
@@ -492,6 +505,26 @@ def bench_gomuzen(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), r
     return out
 
 
+def bench_vepitar(ctx, steps: int, peak_gbs: float, widths=(1024, 2048, 4096), runs: int = 12, prompt: int = 2048) -> dict:
+    """Vepitar decoders (bf16, random weights) beside Gomuzen and Garilix decoders of the same width, number of layer runs,
+    vocabulary and feed-forward size that a token uses.  Decode reads more weights than the L2 holds at the larger widths; no flush."""
+    import densecore_b200 as dc
+    out = {"vocab": 32768, "layer_runs": runs, "sizes": {}}
+    for w in widths:
+        r = {}
+        for name, (cfg, shapes) in (("vepitar_bf16", vepitar_config(w, runs)), ("gomuzen_bf16", (gomuzen_config(w, runs // 4 - 1), {})),
+                                    ("garilix_bf16", garilix_config(w, runs // 6))):
+            m = dc.Model.from_config(ctx, cfg, shapes, max_seqs=4, max_ctx=prompt + 512)
+            m.init_synthetic(11, 0.02)
+            m.finalize()
+            r[name] = time_decoder(m, cfg["vocab"], prompt, (1, 4), steps)
+            m.close()
+            for v in r[name]["decode"].values():
+                v["hbm_fraction"] = v["weight_gbs"] / peak_gbs
+        out["sizes"][str(w)] = r
+    return out
+
+
 def spec_sweep(ctx, model, cfg, rng, seqs_to_free) -> dict:
     """Config 5: target = the benchmark model, draft = the dense 0.8B-class model, gamma 4, 1024-token prompt,
     128 output tokens; greedy accept with synthetic drafts at forced 0 / 50 / 100 % acceptance, and the
@@ -571,6 +604,8 @@ def run_single_op(args) -> int:
         out = bench_datasun(ctx, args.steps, peak)
     elif args.op == "gomuzen":
         out = bench_gomuzen(ctx, args.steps, peak)
+    elif args.op == "vepitar":
+        out = bench_vepitar(ctx, args.steps, peak)
     elif args.op == "dense-0p8b":
         out = bench_dense_0p8b(ctx, peak)
     else:
@@ -603,7 +638,7 @@ def main():
     ap.add_argument("--profiler-range", action="store_true",
                     help="bracket the timed 1-stream decode run with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
     ap.add_argument("--no-extras", action="store_true", help="skip the other workloads (single ops, dense model, speculative sweep)")
-    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix", "datasun", "gomuzen"],
+    ap.add_argument("--op", default=None, choices=["gemv-config1", "gemv-lm-head", "gemv-q4-big", "gemm-q4", "gemm-q6", "moe-layer", "dense-0p8b", "garilix", "datasun", "gomuzen", "vepitar"],
                     help="time one operator alone and print its own JSON line (not the benchmark line)")
     args = ap.parse_args()
     if args.warmup < 3:

@@ -185,16 +185,19 @@ __device__ __forceinline__ void hyper_coefficients(const dc_hyper& h, float* c) 
         c[i] = v;
     }
 }
-// Group i of four columns of token t, whose sublayer output is y: the streams anew (to x_out if store) and u.
+// Group i of four columns of token t: the streams,
 template <int S>
-__device__ __forceinline__ float4 hyper_column(const dc_hyper& h, const float* c, int t, int i, int ld, float4 y, bool store) {
-    float4 v[S], u = make_float4(0.f, 0.f, 0.f, 0.f);
-    const int n = h.streams;
+__device__ __forceinline__ void hyper_load(const dc_hyper& h, int t, int i, int ld, float4 (&v)[S]) {
 #pragma unroll
     for (int s = 0; s < S; ++s) {
-        const size_t row = h.first ? t : (size_t)t * n + s;
-        v[s] = s < n ? *reinterpret_cast<const float4*>(h.x + row * ld + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const size_t row = h.first ? t : (size_t)t * h.streams + s;
+        v[s] = s < h.streams ? *reinterpret_cast<const float4*>(h.x + row * ld + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+}
+// the streams anew with the sublayer's output y (to x_out if store), and u.
+template <int S>
+__device__ __forceinline__ float4 hyper_mix(const dc_hyper& h, const float* c, int t, int i, int ld, const float4 (&v)[S], float4 y, bool store) {
+    float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int to = 0; to < S; ++to) {
         const float o = c[S + to], in = c[to];
@@ -204,7 +207,7 @@ __device__ __forceinline__ float4 hyper_column(const dc_hyper& h, const float* c
             const float m = c[2 * S + s * S + to];
             r.x = fmaf(m, v[s].x, r.x), r.y = fmaf(m, v[s].y, r.y), r.z = fmaf(m, v[s].z, r.z), r.w = fmaf(m, v[s].w, r.w);
         }
-        if (store && to < n) *reinterpret_cast<float4*>(h.x_out + ((size_t)t * n + to) * ld + 4 * i) = r;
+        if (store && to < h.streams) *reinterpret_cast<float4*>(h.x_out + ((size_t)t * h.streams + to) * ld + 4 * i) = r;
         u.x = fmaf(in, r.x, u.x), u.y = fmaf(in, r.y, u.y), u.z = fmaf(in, r.z, u.z), u.w = fmaf(in, r.w, u.w);
     }
     return u;

@@ -164,8 +164,13 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
     float ss = 0.0f;
     for (int i = tid; i < n4; i += NR_WARPS * 32) {
         float4 v;
-        if constexpr (S > 0) v = hyper_column<S>(p.hy, coef, t, i, p.ld, reinterpret_cast<const float4*>(p.hy.y + (size_t)t * p.ld)[i], i % NR_CTAS == rank);
-        else v = x4[i];
+        if constexpr (S > 0) {
+            float4 streams[S];
+            hyper_load<S>(p.hy, t, i, p.ld, streams);
+            v = hyper_mix<S>(p.hy, coef, t, i, p.ld, streams, reinterpret_cast<const float4*>(p.hy.y + (size_t)t * p.ld)[i], i % NR_CTAS == rank);
+        } else {
+            v = x4[i];
+        }
         reinterpret_cast<float4*>(h)[i] = v;
         ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
     }
@@ -271,18 +276,23 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
         auto row = [&](int i, bool store) {
             if constexpr (S > 0) {
                 const int tc = min(t, T - 1);
-                return hyper_column<S>(p.hy, coef, tc, i, p.ld, reinterpret_cast<const float4*>(p.hy.y + (size_t)tc * p.ld)[i], store && t < T);
+                float4 streams[S];
+                hyper_load<S>(p.hy, tc, i, p.ld, streams);
+                return hyper_mix<S>(p.hy, coef, tc, i, p.ld, streams, reinterpret_cast<const float4*>(p.hy.y + (size_t)tc * p.ld)[i], store && t < T);
             } else {
                 return reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld)[i];
             }
         };
         const float4* w4 = reinterpret_cast<const float4*>(p.w);
         uint2* to = reinterpret_cast<uint2*>(h + warp * z.ldh);
-        constexpr int KEEP = S > 4 ? 4 : S > 2 ? 8 : 16;         // groups of four that a lane holds; wider rows are read twice
+        constexpr int KEEP = S > 4 ? 8 : 16;         // groups of four that a lane holds; wider rows are read twice
         float4 x[KEEP];
         float ss = 0.0f;
 #pragma unroll
-        for (int j = 0; j < KEEP; ++j) x[j] = lane + 32 * j < n4 ? row(lane + 32 * j, true) : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int j = 0; j < KEEP; ++j) {
+            x[j] = lane + 32 * j < n4 ? row(lane + 32 * j, true) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (S > 2 || (S > 0 && j % 2)) asm volatile("" ::: "memory");        // as many loads in flight as there are registers
+        }
         auto square = [&](const float4& v) { ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); };
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) square(x[j]);

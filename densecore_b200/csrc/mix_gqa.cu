@@ -28,6 +28,9 @@ namespace {
 __device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
 __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf2(a, b); }
 
+__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w)); }
+
 // ---------------------------------------------------------------- norms, rotation, cache write
 struct PrepParams {
     const float* proj;
@@ -171,9 +174,6 @@ __global__ void __launch_bounds__(256) k_gqa_prep_heads(const HeadsParams p) {
         else p.q[at] = r;
     }
 }
-
-__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store_four(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w)); }
 
 // The same four dimensions at a time, for sizes that are multiples of four: a warp has U heads of a token in flight, a lane the
 // dimensions 4 lane .. 4 lane + 3 (and, with NV 2, those 128 further on).
@@ -359,6 +359,79 @@ __global__ void __launch_bounds__(256) k_gqa_prep_conv(const ConvParams p) {
             else a.q[at] = r;
         }
     }
+}
+
+// The same for up to four taps and head sizes that are multiples of four up to 128: a lane has the dimensions 4 lane .. 4 lane + 3.
+// PB: tokens of a warp; 1: every entry is one token.
+template <typename TC, int PB>
+__global__ void __launch_bounds__(256) k_gqa_prep_conv4(const ConvParams p) {
+    pdl_launch_dependents();
+    const HeadsParams& a = p.h;
+    const int lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5), taps = p.cr.taps, d = 4 * lane;
+    if (u >= a.nq + a.nk + a.nv) return;
+    const bool query = u < a.nq, value = u >= a.nq + a.nk;
+    const int head = query ? u : value ? u - a.nq - a.nk : u - a.nq, n = value ? a.vdim : a.dim;
+    const int col = (query ? a.off_q : value ? a.off_v : a.off_k) + head * n + min(d, n - 4);
+    const bool unit = query ? p.q_unit : value ? p.v_unit : p.k_unit, in = d < n;
+    const float* nw = value ? nullptr : query ? a.q_norm : a.k_norm;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto at4 = [](const float* q) { return *reinterpret_cast<const float4*>(q); };
+    float4 w[4];                 // w[3] is the token's own
+#pragma unroll
+    for (int k = 0; k < 4; ++k) w[k] = in && taps - 4 + k >= 0 ? at4(p.conv + (size_t)(taps - 4 + k) * p.cr.ldw + col) : zero;
+    const float4 nv = nw && in ? at4(nw + d) : make_float4(1.f, 1.f, 1.f, 1.f);
+    pdl_wait();
+    BlockRef br = {(int)blockIdx.x, (int)blockIdx.x, 1};
+    if (PB > 1) br = block_at<PB>(p.cr.starts, p.cr.E, blockIdx.x);
+    if (br.n <= 0) return;
+    const int i0 = PB > 1 ? br.t0 - p.cr.starts[br.e] : 0, pos0 = p.cr.positions[br.t0], seq = p.cr.seq_ids[br.t0];
+    float* ring = p.cr.ring(seq) + col;
+    const float* x0 = a.proj + (size_t)br.t0 * a.ldp + col;
+    float4 x[PB], h[3];
+#pragma unroll
+    for (int i = 0; i < PB; ++i) x[i] = i < br.n ? at4(x0 + (size_t)i * a.ldp) : zero;
+#pragma unroll
+    for (int k = 0; k < 3; ++k) {
+        const int back = 3 - k;
+        h[k] = back >= taps || pos0 < back ? zero : back <= i0 ? at4(x0 - (size_t)back * a.ldp) : at4(ring + (size_t)((pos0 - back) % taps) * p.cr.C);
+    }
+    if (p.put_ring && in) *reinterpret_cast<float4*>(ring + (size_t)(pos0 % taps) * p.cr.C) = x[0];       // a row that no tap of this token reads
+    float ss[PB];
+#pragma unroll
+    for (int i = 0; i < PB; ++i) {
+        float4 y;
+#define DC_TAPS(e) y.e = fmaf(w[3].e, x[i].e, fmaf(w[2].e, h[2].e, fmaf(w[1].e, h[1].e, w[0].e * h[0].e)))
+        DC_TAPS(x), DC_TAPS(y), DC_TAPS(z), DC_TAPS(w);
+#undef DC_TAPS
+        h[0] = h[1], h[1] = h[2], h[2] = x[i];
+        x[i] = y;
+        ss[i] = (y.x * y.x + y.y * y.y) + (y.z * y.z + y.w * y.w);       // zero beyond the head: its weights are
+    }
+    if (unit) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int i = 0; i < PB; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+    }
+    const int pitch = query ? a.ldq : value ? a.vdim_p : a.dim_p;
+    if (d >= pitch) return;
+#pragma unroll
+    for (int i = 0; i < PB; ++i) {
+        if (i >= br.n) break;
+        const float inv = unit ? 1.0f / sqrtf(ss[i] / (float)n + a.eps) : 1.0f;
+        const float4 r = make_float4(x[i].x * inv * nv.x, x[i].y * inv * nv.y, x[i].z * inv * nv.z, x[i].w * inv * nv.w);
+        const size_t q = ((size_t)(br.t0 + i) * a.nq + head) * pitch + d;
+        if (!query) store_four(reinterpret_cast<TC*>(a.c.arena) + a.c.at(seq, min(pos0 + i, a.max_pos - 1)) + (value ? a.v_at + head * a.vdim_p : head * a.dim_p) + d, r);
+        else if (a.qb) store_four(a.qb + q, r);
+        else store_four(a.q + q, r);
+    }
+}
+
+template <typename TC>
+int launch_prep_conv4(dc_ctx* ctx, const ConvParams& p, const dc_step& st) {
+    const int parts = (p.h.nq + p.h.nk + p.h.nv + 7) / 8;
+    if (st.single) return dc_launch(ctx, "k_gqa_prep_conv4", k_gqa_prep_conv4<TC, 1>, dim3(st.T, parts), dim3(256), 0, p);
+    return dc_launch(ctx, "k_gqa_prep_conv4", k_gqa_prep_conv4<TC, 8>, dim3(st.T / 8 + st.E, parts), dim3(256), 0, p);
 }
 
 template <typename TC, int VP>
@@ -832,7 +905,9 @@ int dc_launch_gqa_prep(dc_ctx* ctx, const dc_gqa_mixer& m, const dc_step& st, co
                         m.qk_norm == DC_QK_NORM_HEAD, m.qk_norm == DC_QK_NORM_HEAD, m.v_norm, st.single};
         const int most = std::max(std::max(p.h.ldq, p.h.dim_p), p.h.vdim_p);
 #define DC_CONV(VP) DC_TRY((c.f32 ? launch_prep_conv<float, VP>(ctx, p, st) : launch_prep_conv<__nv_bfloat16, VP>(ctx, p, st)))
-        if (most <= 64) DC_CONV(2);
+        if (m.taps <= 4 && m.dim % 4 == 0 && m.vdim % 4 == 0 && most <= 128 && ldp % 4 == 0)
+            DC_TRY((c.f32 ? launch_prep_conv4<float>(ctx, p, st) : launch_prep_conv4<__nv_bfloat16>(ctx, p, st)));
+        else if (most <= 64) DC_CONV(2);
         else if (most <= 128) DC_CONV(4);
         else DC_CONV(8);
 #undef DC_CONV

@@ -9,7 +9,7 @@
 // Value columns of S never mix: a column c obeys S_c <- g S_c; u = beta (v_c - S_c . k); S_c <- S_c + u k;
 // o_c = S_c . q.  A single token (decode) is done as written, by one kernel per mixer from projections to normed
 // output.  Longer entries go through blocks of sixteen tokens (see "blocks of sixteen tokens" below): what a head's
-// columns share is computed once per block, and k_state_scan walks the blocks with four columns in the registers of
+// columns share is computed once per block, and k_state_scan walks the blocks with two or four columns in the registers of
 // each warp.  All of it is f32 on the CUDA cores.
 #include "dc_common.cuh"
 #include "dc_launch.cuh"
@@ -373,7 +373,7 @@ __device__ __forceinline__ float decay_below_one(float z) { return expf(-0.60653
 
 struct GeneralBlock {
     const float* proj;
-    int ldp, off_r, off_k, off_a, heads, dim, dp;
+    int ldp, off_r, off_k, off_a, heads, dim;
     const float* low;            // decay projection [T][ldd]
     int ldd;
     const float *w0, *a_bias;
@@ -383,71 +383,109 @@ struct GeneralBlock {
     float* out;
 };
 
+// The decays are never below 0.545, so a block's cumulative ones W_t stay above 6e-5 and their quotients keep their bits:
+// P_ti = W_t / W_i.  One 32 x 32 product of the rows W_(t-1) u_t, W_t r_t with the rows c_i / W_i, k_i / W_i holds A, K, C and B.
+// EPL: key channels of a lane.
+template <int EPL>
 __global__ void __launch_bounds__(128) k_general_blocks(const GeneralBlock p) {
-    extern __shared__ __align__(16) float sm[];         // k, r, w, c: [16][dim] each
-    __shared__ float sA[BT][BT + 1], sK[BT][BT + 1], sC[BT][BT + 1], sB[BT][BT + 1], sX[BT][BT + 1], sM[BT][BT + 1], s_unit[BT];
+    constexpr int DP = 32 * EPL, LD = DP + 4, TW = BT / 4;      // tokens of a warp
+    extern __shared__ __align__(16) float sm[];                 // u, r | c, k: [16][LD] each, then the decays
+    __shared__ float sA[BT][BT + 1], sK[BT][BT + 1], sC[BT][BT + 1], sB[BT][BT + 1];
+    __shared__ __align__(16) float sF[2][BT][BROW];             // X, M
     pdl_launch_dependents();
+    float *su = sm, *sr = su + BT * LD, *sc = sr + BT * LD, *sk = sc + BT * LD, *sw = sk + BT * LD;
+    const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim;
+    float w0[EPL], ab[EPL];
+#pragma unroll
+    for (int j = 0; j < EPL; ++j) {
+        const int d = min(lane + 32 * j, dim - 1);
+        w0[j] = p.w0[h * dim + d], ab[j] = p.a_bias[h * dim + d];
+    }
     pdl_wait();
-    const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim, dp = p.dp;
     const BlockRef br = block_at<BT>(p.starts, p.E, blockIdx.x);
     if (br.n <= 0) return;
-    float *sk = sm, *sr = sm + BT * dim, *sw = sm + 2 * BT * dim, *sc = sm + 3 * BT * dim;
-    float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * general_block_floats(dp);
-    for (int d = tid; d < dim; d += 128) {              // every load before the arithmetic
-        float k[BT], r[BT], a[BT], w[BT];
-        const float w0 = p.w0[h * dim + d], ab = p.a_bias[h * dim + d];
+    float* out = p.out + ((size_t)blockIdx.x * p.heads + h) * general_block_floats(DP);
+    constexpr int AT = EPL <= 4 ? TW : 2;                       // tokens whose inputs are in flight
 #pragma unroll
-        for (int t = 0; t < BT; ++t) {
-            const int tc = br.t0 + min(t, br.n - 1);
-            const float* row = p.proj + (size_t)tc * p.ldp + h * dim + d;
-            k[t] = row[p.off_k], r[t] = row[p.off_r], a[t] = row[p.off_a];
-            w[t] = p.low[(size_t)tc * p.ldd + h * dim + d];
+    for (int i0 = 0; i0 < TW; i0 += AT) {
+        float k[AT][EPL], r[AT][EPL], a[AT][EPL], w[AT][EPL];
+#pragma unroll
+        for (int i = 0; i < AT; ++i) {
+            const int tc = br.t0 + min(TW * warp + i0 + i, br.n - 1);
+            const float *row = p.proj + (size_t)tc * p.ldp + h * dim, *low = p.low + (size_t)tc * p.ldd + h * dim;
+#pragma unroll
+            for (int j = 0; j < EPL; ++j) {
+                const int d = min(lane + 32 * j, dim - 1);
+                k[i][j] = row[p.off_k + d], r[i][j] = row[p.off_r + d], a[i][j] = row[p.off_a + d], w[i][j] = low[d];
+            }
         }
 #pragma unroll
-        for (int t = 0; t < BT; ++t) {
-            const bool ok = t < br.n;
-            sk[t * dim + d] = ok ? k[t] : 0.0f;
-            sr[t * dim + d] = ok ? r[t] : 0.0f;
-            sw[t * dim + d] = ok ? decay_below_one(w[t] + w0) : 1.0f;
-            sc[t * dim + d] = ok ? -sigmoid(a[t] + ab) * k[t] : 0.0f;      // the unit key's length is still to come
+        for (int i = 0; i < AT; ++i) {
+            const int t = TW * warp + i0 + i;
+            float ss = 0.0f;
+#pragma unroll
+            for (int j = 0; j < EPL; ++j) {
+                if (t >= br.n || lane + 32 * j >= dim) k[i][j] = r[i][j] = 0.0f;
+                ss = fmaf(k[i][j], k[i][j], ss);
+            }
+            const float unit = 1.0f / sqrtf(warp_sum(ss) + p.unit_eps);
+#pragma unroll
+            for (int j = 0; j < EPL; ++j) {
+                const int at = t * LD + lane + 32 * j;
+                const float u = k[i][j] * unit;
+                su[at] = u, sr[at] = r[i][j], sk[at] = k[i][j];
+                sc[at] = -sigmoid(a[i][j] + ab[j]) * u;
+                sw[at] = t < br.n ? decay_below_one(w[i][j] + w0[j]) : 1.0f;
+            }
         }
+    }
+    __syncthreads();
+    for (int i = tid; i < 2 * DP; i += 128) {           // a channel's u and c, or its r and k
+        const bool second = i >= DP;
+        const int d = second ? i - DP : i;
+        float *x = (second ? sr : su) + d, *y = (second ? sk : sc) + d, *to = out + (second ? BT * DP : 0) + d;
+        float w[BT], cum = 1.0f;
+#pragma unroll
+        for (int t = 0; t < BT; ++t) w[t] = sw[t * LD + d];
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+            const float before = cum;
+            cum *= w[t];
+            const float v = x[t * LD] * (second ? cum : before);
+            x[t * LD] = v;
+            to[t * DP] = v;
+            y[t * LD] = __fdividef(y[t * LD], cum);
+        }
+        if (second) out[4 * BT * DP + d] = cum;
     }
     __syncthreads();
     {
-        float ss[4] = {};
-        for (int d = lane; d < dim; d += 32)
+        // rows 2 ty, 2 ty + 1 of (u | r) with rows tx, tx + 8, .. of (c | k)
+        const int tx = tid & 7, ty = tid >> 3;
+        uint64_t acc[2][4] = {};
+        const float *xa = sm + 2 * ty * LD, *ya = sc + tx * LD;
+#pragma unroll 4
+        for (int d = 0; d < DP; d += 4) {
+            ulonglong2 x[2], y[4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) ss[j] = fmaf(sk[(4 * warp + j) * dim + d], sk[(4 * warp + j) * dim + d], ss[j]);
+            for (int i = 0; i < 2; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(xa + i * LD + d);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            ss[j] = warp_sum(ss[j]);
-            if (lane == 0) s_unit[4 * warp + j] = 1.0f / sqrtf(ss[j] + p.unit_eps);
+            for (int j = 0; j < 4; ++j) y[j] = *reinterpret_cast<const ulonglong2*>(ya + 8 * j * LD + d);
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fma2(x[i].y, y[j].y, fma2(x[i].x, y[j].x, acc[i][j]));
         }
-    }
-    __syncthreads();
-    // the products of the source tokens i = warp, warp + 4, ...: c, k run over P_ti c_i, P_ti k_i (c without the lengths)
-#pragma unroll 1
-    for (int i = warp; i < BT; i += 4) {
-        float v[2][32];
 #pragma unroll
-        for (int j = 0; j < 32; ++j) v[0][j] = v[1][j] = 0.0f;
-        for (int d = lane; d < dim; d += 32) {
-            float c = 0.0f, k = 0.0f;
+        for (int i = 0; i < 2; ++i)
 #pragma unroll
-            for (int t = 0; t < BT; ++t) {
-                const float kt = sk[t * dim + d], rt = sr[t * dim + d], wt = sw[t * dim + d];
-                v[0][t] = fmaf(c, kt, v[0][t]);
-                v[1][t] = fmaf(k, kt, v[1][t]);
-                c = t == i ? sc[t * dim + d] : c * wt;
-                k = t == i ? kt : k * wt;
-                v[0][BT + t] = fmaf(c, rt, v[0][BT + t]);
-                v[1][BT + t] = fmaf(k, rt, v[1][BT + t]);
+            for (int j = 0; j < 4; ++j) {
+                const float2 f = unpair(acc[i][j]);
+                const int t = (2 * ty + i) % BT, s = (tx + 8 * j) % BT;
+                const bool answer = 2 * ty >= BT;
+                float(*to)[BT + 1] = answer ? (j < 2 ? sC : sB) : (j < 2 ? sA : sK);
+                to[t][s] = s < t || (answer && s == t) ? f.x + f.y : 0.0f;
             }
-        }
-        const float ui = s_unit[i], ut = s_unit[lane & 15];
-        const float a = transpose_sum32(v[0], lane) * ui, b = transpose_sum32(v[1], lane);
-        if (lane < BT) sA[lane][i] = a * ut, sK[lane][i] = b * ut;
-        else sC[lane - BT][i] = a, sB[lane - BT][i] = b;
     }
     __syncthreads();
     if (tid < BT) {                                     // column tid of (I - A)^-1
@@ -458,66 +496,62 @@ __global__ void __launch_bounds__(128) k_general_blocks(const GeneralBlock p) {
 #pragma unroll
             for (int i = 0; i < t; ++i) a[i & 1] = fmaf(sA[t][i], x[i], a[i & 1]);
             x[t] = t < tid ? 0.0f : t == tid ? 1.0f : a[0] + a[1];
-            sX[t][tid] = x[t];
+            sF[0][t][tid] = x[t];
         }
     }
     __syncthreads();
-    float* N = out + 4 * BT * dp + dp;
-#pragma unroll
-    for (int j = 0; j < 2; ++j) {
-        const int t = (tid + 128 * j) / BT, i = tid % BT;
-        float m = 0.0f, n = 0.0f;
+    float* N = out + 4 * BT * DP + DP;
+    {
+        const int t = tid >> 3, i = 2 * (tid & 7);      // two neighbouring elements
+        float m[2] = {}, n[2] = {};
 #pragma unroll
         for (int q = 0; q < BT; ++q) {
-            m = fmaf(sX[t][q], sK[q][i], m);            // factors are zero above the diagonal
-            n = fmaf(sC[t][q], sX[q][i], n);
+            const float x = sF[0][t][q], c = sC[t][q];
+            const float2 f = *reinterpret_cast<const float2*>(&sF[0][q][i]);
+            m[0] = fmaf(x, sK[q][i], m[0]), m[1] = fmaf(x, sK[q][i + 1], m[1]);
+            n[0] = fmaf(c, f.x, n[0]), n[1] = fmaf(c, f.y, n[1]);
         }
-        sM[t][i] = m;
-        N[t * BROW + i] = n;
+        *reinterpret_cast<float2*>(&sF[1][t][i]) = make_float2(m[0], m[1]);
+        *reinterpret_cast<float2*>(N + t * BROW + i) = make_float2(n[0], n[1]);
+        __syncthreads();
+        n[0] = sB[t][i], n[1] = sB[t][i + 1];
+#pragma unroll
+        for (int q = 0; q < BT; ++q) {
+            const float c = sC[t][q];
+            const float2 f = *reinterpret_cast<const float2*>(&sF[1][q][i]);
+            n[0] = fmaf(c, f.x, n[0]), n[1] = fmaf(c, f.y, n[1]);
+        }
+        *reinterpret_cast<float2*>(N + (BT + t) * BROW + i) = make_float2(n[0], n[1]);
     }
-    __syncthreads();
+    for (int i = tid; i < 2 * DP; i += 128) {           // a channel of D or of E
+        const bool second = i >= DP;
+        const int d = second ? i - DP : i;
+        float last = 1.0f, a[BT];
 #pragma unroll
-    for (int j = 0; j < 2; ++j) {
-        const int t = (tid + 128 * j) / BT, i = tid % BT;
-        float n = sB[t][i];
+        for (int t = 0; t < BT; ++t) {
+            last *= sw[t * LD + d];
+            a[t] = second ? sk[t * LD + d] : 0.0f;
+        }
+        const float (*F)[BROW] = sF[second];
 #pragma unroll
-        for (int q = 0; q < BT; ++q) n = fmaf(sC[t][q], sM[q][i], n);
-        N[(BT + t) * BROW + i] = n;
-    }
-    // per channel: one thread the decayed vectors and D, another one E
-    for (int i = tid; i < 2 * dp; i += 128) {
-        const bool second = i >= dp;
-        const int d = second ? i - dp : i;
-        const bool in = d < dim;
-        float w[BT], c[BT];
+        for (int t = 0; t < BT; ++t) {
+            const float c = sc[t * LD + d];
 #pragma unroll
-        for (int t = 0; t < BT; ++t) w[t] = in ? sw[t * dim + d] : 1.0f, c[t] = in ? sc[t * dim + d] * s_unit[t] : 0.0f;
-        if (!second) {
-            float cum = 1.0f;
-#pragma unroll
-            for (int t = 0; t < BT; ++t) {
-                out[t * dp + d] = in ? cum * sk[t * dim + d] * s_unit[t] : 0.0f;
-                cum *= w[t];
-                out[(BT + t) * dp + d] = in ? cum * sr[t * dim + d] : 0.0f;
+            for (int j = 0; j <= t; j += 4) {           // zero above the diagonal
+                const float4 f = *reinterpret_cast<const float4*>(&F[t][j]);
+                a[j] = fmaf(c, f.x, a[j]), a[j + 1] = fmaf(c, f.y, a[j + 1]), a[j + 2] = fmaf(c, f.z, a[j + 2]), a[j + 3] = fmaf(c, f.w, a[j + 3]);
             }
-            out[4 * BT * dp + d] = cum;
         }
-        float suffix = 1.0f, k[BT];
 #pragma unroll
-        for (int t = BT - 1; t >= 0; --t) {
-            c[t] *= suffix;
-            k[t] = second && in ? suffix * sk[t * dim + d] : 0.0f;
-            suffix *= w[t];
-        }
-        const float (*F)[BT + 1] = second ? sM : sX;
-#pragma unroll
-        for (int j = 0; j < BT; ++j) {
-            float a[2] = {k[j], 0.0f};
-#pragma unroll
-            for (int t = j; t < BT; ++t) a[t & 1] = fmaf(c[t], F[t][j], a[t & 1]);
-            out[((second ? 3 : 2) * BT + j) * dp + d] = a[0] + a[1];
-        }
+        for (int j = 0; j < BT; ++j) out[((second ? 3 : 2) * BT + j) * DP + d] = last * a[j];
     }
+}
+
+template <int EPL>
+int launch_general_blocks(dc_ctx* ctx, const GeneralBlock& p, dim3 grid) {
+    constexpr int bytes = 5 * BT * (32 * EPL + 4) * 4;
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_general_blocks<EPL>, bytes, "k_general_blocks"));
+    return dc_launch(ctx, "k_general_blocks", k_general_blocks<EPL>, grid, dim3(128), (size_t)bytes, p);
 }
 
 // Floats of one (block, head) of the state-space scan: M [16][20], cumulative decays [16], update factors [16].
@@ -580,7 +614,7 @@ __global__ void __launch_bounds__(256) k_ssd_blocks(const SsdBlock p) {
 }
 
 // ---------------------------------------------------------------- the scan over blocks
-constexpr int SC_COLS = 16, SC_THREADS = 128;           // value columns per CTA: four per warp
+constexpr int SC_COLS = 16;                             // value columns per CTA
 enum { SCAN_SSD = 0, SCAN_DELTA = 1, SCAN_GENERAL = 2 };
 
 struct ScanParams {
@@ -619,12 +653,13 @@ struct Chan {
     }
 };
 
-// Dot products of the warp's four columns (s: this lane's channels of each) with NS sets of sixteen rows of shared
-// memory, eight rows in flight ahead of the arithmetic.  Lane 8 c + j gets column c's products with rows j and j + 8.
-template <int EPL, int NS>
-__device__ __forceinline__ void column_dots(const float* rows, int dp, const float (&s)[4][EPL], int lane, float (&out)[NS][2]) {
-    constexpr int G = EPL <= 4 ? 8 : 4;
-    float r[NS][64], w[2][G][EPL];
+// Dot products of the warp's NC columns (s: this lane's channels of each) with NS sets of sixteen rows of shared memory, eight
+// rows in flight ahead of the arithmetic.  L = 32 / NC lanes work for a column: lane L c + j gets column c's products with rows
+// j, j + L, ...
+template <int EPL, int NS, int NC>
+__device__ __forceinline__ void column_dots(const float* rows, int dp, const float (&s)[NC][EPL], int lane, float (&out)[NS][NC / 2]) {
+    constexpr int G = EPL <= 4 ? 8 : 4, L = 32 / NC, PER = NC / 2;
+    float r[NS][BT * NC], w[2][G][EPL];
 #pragma unroll
     for (int t = 0; t < G; ++t) Chan<EPL>::load(rows + t * dp, lane, w[0][t]);
 #pragma unroll
@@ -637,8 +672,8 @@ __device__ __forceinline__ void column_dots(const float* rows, int dp, const flo
         for (int u = 0; u < G; ++u) {
             const int row = G * g + u, t = row % BT;
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                float& dst = r[row / BT][16 * c + 2 * (t & 7) + (t >> 3)];
+            for (int c = 0; c < NC; ++c) {
+                float& dst = r[row / BT][BT * c + PER * (t % L) + t / L];
                 if (EPL == 1) {
                     dst = s[c][0] * w[g & 1][u][0];
                 } else {
@@ -655,32 +690,36 @@ __device__ __forceinline__ void column_dots(const float* rows, int dp, const flo
     for (int o = 16; o > 0; o >>= 1) {                           // each step halves the sums a lane carries
         const bool up = lane & o;
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
-            if (i < 2 * o) {
+        for (int i = 0; i < BT * NC / 2; ++i)
+            if (i < PER * o) {
 #pragma unroll
                 for (int k = 0; k < NS; ++k) {
-                    const float send = up ? r[k][i] : r[k][i + 2 * o], keep = up ? r[k][i + 2 * o] : r[k][i];
+                    const float send = up ? r[k][i] : r[k][i + PER * o], keep = up ? r[k][i + PER * o] : r[k][i];
                     r[k][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
                 }
             }
     }
 #pragma unroll
-    for (int k = 0; k < NS; ++k) out[k][0] = r[k][0], out[k][1] = r[k][1];
+    for (int k = 0; k < NS; ++k)
+#pragma unroll
+        for (int i = 0; i < PER; ++i) out[k][i] = r[k][i];
 }
 
 // EPL: key channels per lane (the key size, padded to 32 EPL).
 constexpr int scan_block_floats(int kind, int dp) { return kind == SCAN_DELTA ? delta_block_floats(dp) : kind == SCAN_GENERAL ? general_block_floats(dp) : 2 * BT * dp + SSD_BLOCK; }
 
-template <int EPL, int KIND>
-__global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
+// NC: columns of a warp.
+template <int EPL, int KIND, int NC>
+__global__ void __launch_bounds__(SC_COLS / NC * 32) k_state_scan(const ScanParams p) {
     constexpr bool GENERAL = KIND == SCAN_GENERAL, DELTA = KIND != SCAN_SSD;         // the delta rules' factors come whole from memory
     constexpr int DP = 32 * EPL, BLK = scan_block_floats(KIND, DP), BUF = BLK + BT * SC_COLS;
+    constexpr int SC_THREADS = SC_COLS / NC * 32, LANES = 32 / NC, PER = NC / 2;
     extern __shared__ __align__(16) float sm[];
-    __shared__ __align__(16) float s_d[4][4][BT], s_u[4][4][BT];
+    __shared__ __align__(16) float s_d[SC_COLS / NC][NC][BT], s_u[SC_COLS / NC][NC][BT];
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lt = lane & 7, lc = lane >> 3;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lt = lane % LANES, lc = lane / LANES;
     const int c0 = blockIdx.x * SC_COLS, h = blockIdx.y, e = blockIdx.z, kh = h / p.per;
-    const int col = c0 + warp * 4 + lc;
+    const int col = c0 + warp * NC + lc;
     if (!DELTA) {
         for (int i = tid; i < 2 * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels stay zero
         __syncthreads();
@@ -691,15 +730,15 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
     const int seq = p.seq_ids[t0], blocks = (t1 - t0 + BT - 1) / BT;
     const float* bsrc = p.blocks + ((size_t)block_base<BT>(p.starts, e) * p.heads + h) * (DELTA ? BLK : SSD_BLOCK);
     const size_t bstep = (size_t)p.heads * (DELTA ? BLK : SSD_BLOCK);
-    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * 4) * p.dim;
-    float s[4][EPL];             // channels Chan::at of the warp's four columns
+    float* S = reinterpret_cast<float*>(p.base + (size_t)seq * p.slot_bytes + p.state_off) + ((size_t)h * p.vdim + c0 + warp * NC) * p.dim;
+    float s[NC][EPL];            // channels Chan::at of the warp's columns
     const bool fresh = p.positions[t0] == 0, live = col < p.vdim;
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int i = 0; i < EPL; ++i) {
             const int d = Chan<EPL>::at(lane, i);
-            s[c][i] = !fresh && c0 + warp * 4 + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
+            s[c][i] = !fresh && c0 + warp * NC + c < p.vdim && d < p.dim ? S[(size_t)c * p.dim + d] : 0.0f;
         }
 
     auto load = [&](int b, int buf) {
@@ -710,16 +749,16 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             for (int i = tid; i < BLK / 4; i += SC_THREADS) cp_async16z(smem_u32(dst + 4 * i), src + 4 * i, true);
         } else {
             for (int i = tid; i < SSD_BLOCK / 4; i += SC_THREADS) cp_async16z(smem_u32(dst + 2 * BT * DP + 4 * i), src + 4 * i, true);
-            const int t = tid >> 3;                  // eight threads per token
+            const int t = tid / (SC_THREADS / BT), part = tid % (SC_THREADS / BT);
             const bool ok = tb + t < t1;
 #pragma unroll
             for (int a = 0; a < 2; ++a) {
                 const float* row = (a ? p.k : p.q) + (size_t)kh * p.dim + (size_t)(ok ? tb + t : tb) * p.ld;
                 const uint32_t to = smem_u32(dst + (a * BT + t) * DP);
                 if (p.vec) {
-                    for (int d = 4 * (tid & 7); d < p.dim; d += 32) cp_async16z(to + 4 * d, row + d, ok);
+                    for (int d = 4 * part; d < p.dim; d += SC_THREADS / BT * 4) cp_async16z(to + 4 * d, row + d, ok);
                 } else {
-                    for (int d = tid & 7; d < p.dim; d += 8) cp_async4z(to + 4 * d, row + d, ok);
+                    for (int d = part; d < p.dim; d += SC_THREADS / BT) cp_async4z(to + 4 * d, row + d, ok);
                 }
             }
         }
@@ -741,16 +780,16 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         }
         __syncthreads();
         const float* x = sm + (b & 1) * BUF;
-        // ---- the columns against the block's (decayed) keys and queries; lane 8 c + j works for column c, tokens j, j + 8
-        float r[DELTA ? 2 : 1][2];
-        column_dots<EPL, DELTA ? 2 : 1>(x, DP, s, lane, r);
+        // ---- the columns against the block's (decayed) keys and queries; see column_dots for who works for whom
+        float r[DELTA ? 2 : 1][PER];
+        column_dots<EPL, DELTA ? 2 : 1, NC>(x, DP, s, lane, r);
         const float* rq = r[DELTA ? 1 : 0];
-        float v[2];
+        float v[PER];
 #pragma unroll
-        for (int k = 0; k < 2; ++k) {
-            v[k] = x[BLK + (lt + 8 * k) * SC_COLS + warp * 4 + lc];
-            s_d[warp][lc][lt + 8 * k] = GENERAL ? r[0][k] : DELTA ? v[k] - r[0][k] : v[k];
-            if (GENERAL) s_u[warp][lc][lt + 8 * k] = v[k];
+        for (int k = 0; k < PER; ++k) {
+            v[k] = x[BLK + (lt + LANES * k) * SC_COLS + warp * NC + lc];
+            s_d[warp][lc][lt + LANES * k] = GENERAL ? r[0][k] : DELTA ? v[k] - r[0][k] : v[k];
+            if (GENERAL) s_u[warp][lc][lt + LANES * k] = v[k];
         }
         __syncwarp();
         auto row_dot = [&](const float* row, const float* vals) {      // rows of W, B, M are zero above the diagonal
@@ -766,30 +805,30 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             return (a[0] + a[1]) + (a[2] + a[3]);
         };
         const float* scal = x + (GENERAL ? 4 * BT * DP + DP : DELTA ? 3 * BT * DP + DP : 2 * BT * DP);
-        float out[2];
+        float out[PER];
         if (GENERAL) {
 #pragma unroll
-            for (int k = 0; k < 2; ++k)
-                out[k] = rq[k] + row_dot(scal + (lt + 8 * k) * BROW, s_d[warp][lc]) + row_dot(scal + (BT + lt + 8 * k) * BROW, s_u[warp][lc]);
+            for (int k = 0; k < PER; ++k)
+                out[k] = rq[k] + row_dot(scal + (lt + LANES * k) * BROW, s_d[warp][lc]) + row_dot(scal + (BT + lt + LANES * k) * BROW, s_u[warp][lc]);
         } else if (DELTA) {
 #pragma unroll
-            for (int k = 0; k < 2; ++k) s_u[warp][lc][lt + 8 * k] = row_dot(scal + (lt + 8 * k) * BROW, s_d[warp][lc]);
+            for (int k = 0; k < PER; ++k) s_u[warp][lc][lt + LANES * k] = row_dot(scal + (lt + LANES * k) * BROW, s_d[warp][lc]);
             __syncwarp();
 #pragma unroll
-            for (int k = 0; k < 2; ++k) out[k] = rq[k] + row_dot(scal + (BT + lt + 8 * k) * BROW, s_u[warp][lc]);
+            for (int k = 0; k < PER; ++k) out[k] = rq[k] + row_dot(scal + (BT + lt + LANES * k) * BROW, s_u[warp][lc]);
         } else {
             const float* cd = scal + BT * BROW;
 #pragma unroll
-            for (int k = 0; k < 2; ++k) {
-                const int t = lt + 8 * k;
+            for (int k = 0; k < PER; ++k) {
+                const int t = lt + LANES * k;
                 s_u[warp][lc][t] = v[k] * cd[BT + t];
                 out[k] = fmaf(cd[t], rq[k], row_dot(scal + t * BROW, s_d[warp][lc])) + Dh * v[k];
             }
             __syncwarp();
         }
 #pragma unroll
-        for (int k = 0; k < 2; ++k) {
-            const int t = t0 + b * BT + lt + 8 * k;
+        for (int k = 0; k < PER; ++k) {
+            const int t = t0 + b * BT + lt + LANES * k;
             if (t < t1 && live) p.o[(size_t)t * p.ldo + (size_t)h * p.vdim + col] = out[k];
         }
         // ---- the state after the block
@@ -798,7 +837,7 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
             float g[EPL];
             if (DELTA) Chan<EPL>::load(x + (GENERAL ? 4 : 3) * BT * DP, lane, g);
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
+            for (int c = 0; c < NC; ++c)
 #pragma unroll
                 for (int i = 0; i < EPL; ++i) s[c][i] *= DELTA ? g[i] : scal[BT * BROW + BT - 1];
         }
@@ -807,11 +846,11 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
         for (int row = 0; row < (GENERAL ? 2 : 1) * BT; row += G) {
             const int t = row % BT;
             float (*vals)[BT] = GENERAL && row < BT ? s_d[warp] : s_u[warp];
-            float w[G][EPL], u[4][G];
+            float w[G][EPL], u[NC][G];
 #pragma unroll
             for (int g = 0; g < G; ++g) Chan<EPL>::load(keys + (row + g) * DP, lane, w[g]);
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
+            for (int c = 0; c < NC; ++c)
 #pragma unroll
                 for (int g = 0; g < G; g += 4) {
                     const float4 f = *reinterpret_cast<const float4*>(&vals[c][t + g]);
@@ -820,35 +859,42 @@ __global__ void __launch_bounds__(SC_THREADS) k_state_scan(const ScanParams p) {
 #pragma unroll
             for (int g = 0; g < G; ++g)
 #pragma unroll
-                for (int c = 0; c < 4; ++c)
+                for (int c = 0; c < NC; ++c)
 #pragma unroll
                     for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(w[g][i], u[c][g], s[c][i]);
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int i = 0; i < EPL; ++i) {
             const int d = Chan<EPL>::at(lane, i);
-            if (c0 + warp * 4 + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
+            if (c0 + warp * NC + c < p.vdim && d < p.dim) S[(size_t)c * p.dim + d] = s[c][i];
         }
 }
 
-template <int EPL, int KIND>
+template <int EPL, int KIND, int NC>
 int launch_scan_epl(dc_ctx* ctx, const ScanParams& p, int E) {
+    // a few CTAs that run long: started while the many of the kernel before still leave, they would crowd on the first free SMs
     const size_t smem = (size_t)2 * (scan_block_floats(KIND, 32 * EPL) + BT * SC_COLS) * 4;
-    DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, KIND>, (int)smem, "k_state_scan"));
-    return dc_launch(ctx, "k_state_scan", k_state_scan<EPL, KIND>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_THREADS), smem, p);
+    DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, KIND, NC>, (int)smem, "k_state_scan"));
+    return dc_launch_drained(ctx, "k_state_scan", k_state_scan<EPL, KIND, NC>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_COLS / NC * 32), smem, p);
 }
 int key_pad(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+// Few columns in the whole step: fewer of them for each warp.
+template <int EPL, int KIND>
+int launch_scan_columns(dc_ctx* ctx, const ScanParams& p, int E) {
+    const int ctas = (p.vdim + SC_COLS - 1) / SC_COLS * p.heads * E;
+    return ctas <= 2 * ctx->num_sms ? launch_scan_epl<EPL, KIND, 2>(ctx, p, E) : launch_scan_epl<EPL, KIND, 4>(ctx, p, E);
+}
 template <int KIND>
 int launch_scan(dc_ctx* ctx, const ScanParams& p, int E) {
     switch (key_pad(p.dim)) {
-    case 32: return launch_scan_epl<1, KIND>(ctx, p, E);
-    case 64: return launch_scan_epl<2, KIND>(ctx, p, E);
-    case 128: return launch_scan_epl<4, KIND>(ctx, p, E);
-    default: return launch_scan_epl<8, KIND>(ctx, p, E);
+    case 32: return launch_scan_columns<1, KIND>(ctx, p, E);
+    case 64: return launch_scan_columns<2, KIND>(ctx, p, E);
+    case 128: return launch_scan_columns<4, KIND>(ctx, p, E);
+    default: return launch_scan_columns<8, KIND>(ctx, p, E);
     }
 }
 
@@ -1294,6 +1340,15 @@ __global__ void __launch_bounds__(128) k_ssd_decode(const SsdDecode p) {
 }
 
 // ---------------------------------------------------------------- output norms
+// Four neighbouring values as f32.
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w)); }
+
 // delta rules: one warp per (token, head): o / rms(o) * w * sigmoid(gate).  ws: pitch of the heads' weights, 0: they share them
 template <typename TO>
 __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg,
@@ -1313,9 +1368,49 @@ __global__ void __launch_bounds__(256) k_head_norm_gate(const float* __restrict_
         store_as(out + (size_t)t * ldm + (size_t)h * vdim + c, r[c] * inv * w[h * ws + c] * sigmoid(gate[(size_t)t * ldg + (size_t)h * vdim + c]));
 }
 
+// The same for value sizes that are a power of two from 4 to 128: vdim / 4 lanes a head, each with four units of (token, head).
+template <typename TO>
+__global__ void __launch_bounds__(256) k_head_norm_gate4(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg,
+                                                         const float* __restrict__ w, int ws, int heads, int vdim, int T, float eps,
+                                                         TO* __restrict__ out, int ldm) {
+    constexpr int U = 4;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lanes = vdim / 4, per = 256 / lanes, c = 4 * (threadIdx.x % lanes);
+    const long long id0 = (long long)blockIdx.x * per * U + threadIdx.x / lanes, all = (long long)T * heads;
+    float4 v[U], g[U], f[U];
+    float ss[U];
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+        const long long id = min(id0 + per * i, all - 1);
+        const int t = (int)(id / heads), h = (int)(id % heads);
+        v[i] = load4(o + (size_t)t * ldo + h * vdim + c), g[i] = load4(gate + (size_t)t * ldg + h * vdim + c), f[i] = load4(w + h * ws + c);
+    }
+#pragma unroll
+    for (int i = 0; i < U; ++i) ss[i] = (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+    for (int x = lanes >> 1; x > 0; x >>= 1)
+#pragma unroll
+        for (int i = 0; i < U; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], x);
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+        const long long id = id0 + per * i;
+        if (id >= all) break;
+        const int t = (int)(id / heads), h = (int)(id % heads);
+        const float inv = 1.0f / sqrtf(ss[i] / (float)vdim + eps);
+        store4(out + (size_t)t * ldm + h * vdim + c, make_float4(v[i].x * inv * f[i].x * sigmoid(g[i].x), v[i].y * inv * f[i].y * sigmoid(g[i].y),
+                                                                 v[i].z * inv * f[i].z * sigmoid(g[i].z), v[i].w * inv * f[i].w * sigmoid(g[i].w)));
+    }
+}
+
 int launch_head_norm_gate(dc_ctx* ctx, const float* o, int ldo, const float* gate, int ldg, const float* w, int ws, int heads, int vdim, int T, float eps,
                           float* mix, __nv_bfloat16* mixb, int ldm) {
     const dim3 grid((unsigned)(((long long)T * heads + 7) / 8)), block(256);
+    if (vdim >= 4 && vdim <= 128 && !(vdim & (vdim - 1)) && ldo % 4 == 0 && ldg % 4 == 0 && ldm % 4 == 0 && ((uintptr_t)gate & 15) == 0) {
+        const int units = 4 * 256 / (vdim / 4);
+        const dim3 grid4((unsigned)(((long long)T * heads + units - 1) / units));
+        if (mixb) return dc_launch(ctx, "k_head_norm_gate4", k_head_norm_gate4<__nv_bfloat16>, grid4, block, 0, o, ldo, gate, ldg, w, ws, heads, vdim, T, eps, mixb, ldm);
+        return dc_launch(ctx, "k_head_norm_gate4", k_head_norm_gate4<float>, grid4, block, 0, o, ldo, gate, ldg, w, ws, heads, vdim, T, eps, mix, ldm);
+    }
     if (mixb) return dc_launch(ctx, "k_head_norm_gate", k_head_norm_gate<__nv_bfloat16>, grid, block, 0, o, ldo, gate, ldg, w, ws, heads, vdim, T, eps, mixb, ldm);
     return dc_launch(ctx, "k_head_norm_gate", k_head_norm_gate<float>, grid, block, 0, o, ldo, gate, ldg, w, ws, heads, vdim, T, eps, mix, ldm);
 }
@@ -1359,15 +1454,6 @@ int launch_group_norm(dc_ctx* ctx, const float* y, int ldy, const float* z, int 
     if (n <= 512) return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 64>, grid, dim3(64), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
     return dc_launch(ctx, "k_gate_group_norm", k_gate_group_norm<TO, 256>, grid, dim3(256), 0, y, ldy, z, ldz, w, n, eps, out, ldm);
 }
-
-// Four neighbouring values as f32.
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w)); }
 
 // lightning: one CTA per token: y over its root mean square, times w, times sigmoid(gate).  Rows are padded to multiples of
 // eight (what the padding holds does not matter); KEEP: groups of four values of a thread.
@@ -1606,10 +1692,14 @@ int dc_launch_general_tanh(dc_ctx* ctx, const dc_general_mixer& m, int T, float*
 
 int dc_launch_general_scan(dc_ctx* ctx, const dc_general_mixer& m, const dc_step& st, const dc_state_ref& sr, const float* proj, int ldp, const float* low,
                            int ldd, float* blk, float eps, float* o, int ldo, float* mix, __nv_bfloat16* mixb, int ldm) {
-    const GeneralBlock b = {proj, ldp, m.off_r, m.off_k, m.off_a, m.heads, m.dim, key_pad(m.dim), low, ldd, m.w0, m.a_bias, m.unit_eps, st.starts, st.E, blk};
-    const size_t smem = (size_t)4 * BT * m.dim * 4;
-    DC_TRY(dc_kernel_setup(ctx, (const void*)k_general_blocks, (int)smem, "k_general_blocks"));
-    DC_TRY(dc_launch(ctx, "k_general_blocks", k_general_blocks, dim3(dc_scan_blocks(st.T, st.E), m.heads), dim3(128), smem, b));
+    const GeneralBlock b = {proj, ldp, m.off_r, m.off_k, m.off_a, m.heads, m.dim, low, ldd, m.w0, m.a_bias, m.unit_eps, st.starts, st.E, blk};
+    const dim3 grid(dc_scan_blocks(st.T, st.E), m.heads);
+    switch (key_pad(m.dim)) {
+    case 32: DC_TRY(launch_general_blocks<1>(ctx, b, grid)); break;
+    case 64: DC_TRY(launch_general_blocks<2>(ctx, b, grid)); break;
+    case 128: DC_TRY(launch_general_blocks<4>(ctx, b, grid)); break;
+    default: DC_TRY(launch_general_blocks<8>(ctx, b, grid));
+    }
     ScanParams p = {};
     p.blocks = blk, p.v = proj + m.off_v;
     p.ld = ldp, p.heads = m.heads, p.per = 1, p.dim = m.dim, p.vdim = m.dim;

@@ -155,41 +155,54 @@ __global__ void __launch_bounds__(256) k_pre_norm(float* __restrict__ x, const f
     }
 }
 
-// S: streams at most.  Rows as above.
-template <int S, int KEEP>
-__global__ void __launch_bounds__(256) k_hyper_norm(const dc_hyper hy, const float* __restrict__ w, const int32_t* __restrict__ rows, int first, int H, int ld,
-                                                    float eps, float* __restrict__ out, __nv_bfloat16* __restrict__ outb) {
+// S: streams at most.  Rows as above; NT threads, KEEP groups of four columns each.
+template <int S, int KEEP, int NT>
+__global__ void __launch_bounds__(NT) k_hyper_norm(const dc_hyper hy, const float* __restrict__ w, const int32_t* __restrict__ rows, int first, int H, int ld,
+                                                   float eps, float* __restrict__ out, __nv_bfloat16* __restrict__ outb) {
     __shared__ float red[33], coef[S * (S + 2)];
     __shared__ int32_t s_rows[DC_MOE_MAX_TOP];
+    constexpr int AHEAD = S * KEEP <= 8 ? KEEP : S >= 8 ? 1 : 8 / S;      // groups whose streams are in flight together
     dc::pdl_launch_dependents();
     const int n4 = ld / 4;
     float4 wv[KEEP], u[KEEP];
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-        const int i = threadIdx.x + 256 * j;
+        const int i = threadIdx.x + NT * j;
         wv[j] = w && i < n4 ? reinterpret_cast<const float4*>(w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     dc::hyper_coefficients<S>(hy, coef);
     dc::pdl_wait();
     const int t = rows ? rows[blockIdx.x] : first + (int)blockIdx.x;
-    if (threadIdx.x < (unsigned)hy.sum.k) s_rows[threadIdx.x] = hy.sum.rows[t * hy.sum.k + threadIdx.x];
-    __syncthreads();
     float ss = 0.0f;
 #pragma unroll
-    for (int j = 0; j < KEEP; ++j) {
-        const int i = threadIdx.x + 256 * j;
-        u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i >= n4) continue;
-        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (hy.sum.k) y = dc::row_sum4(hy.sum, s_rows, i);
-        else if (hy.y) y = *reinterpret_cast<const float4*>(hy.y + (size_t)t * ld + 4 * i);
-        u[j] = dc::hyper_column<S>(hy, coef, t, i, ld, y, hy.x_out != nullptr);
-        ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
+    for (int j0 = 0; j0 < KEEP; j0 += AHEAD) {
+        float4 v[AHEAD][S], y[AHEAD];
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int i = threadIdx.x + NT * (j0 + j);
+            y[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i >= n4) continue;
+            dc::hyper_load<S>(hy, t, i, ld, v[j]);
+            if (hy.y && !hy.sum.k) y[j] = *reinterpret_cast<const float4*>(hy.y + (size_t)t * ld + 4 * i);
+        }
+        if (j0 == 0) {
+            if (threadIdx.x < (unsigned)hy.sum.k) s_rows[threadIdx.x] = hy.sum.rows[t * hy.sum.k + threadIdx.x];
+            __syncthreads();
+        }
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int i = threadIdx.x + NT * (j0 + j);
+            u[j0 + j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i >= n4) continue;
+            if (hy.sum.k) y[j] = dc::row_sum4(hy.sum, s_rows, i);
+            const float4 r = u[j0 + j] = dc::hyper_mix<S>(hy, coef, t, i, ld, v[j], y[j], hy.x_out != nullptr);
+            ss += (r.x * r.x + r.y * r.y) + (r.z * r.z + r.w * r.w);
+        }
     }
     const float inv = w ? 1.0f / sqrtf(dc::block_sum(ss, red) / (float)H + eps) : 1.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-        const int i = threadIdx.x + 256 * j;
+        const int i = threadIdx.x + NT * j;
         if (i >= n4) continue;
         float4 v = u[j];
         if (w) v = make_float4(v.x * inv * wv[j].x, v.y * inv * wv[j].y, v.z * inv * wv[j].z, v.w * inv * wv[j].w);
@@ -200,11 +213,18 @@ __global__ void __launch_bounds__(256) k_hyper_norm(const dc_hyper hy, const flo
 
 template <int S>
 int launch_hyper(dc_ctx* ctx, const dc_hyper& hy, const float* w, const int32_t* rows, int first, int R, int H, int ld, float eps, float* out, __nv_bfloat16* outb) {
-    const dim3 grid(R), block(256);
-    if (ld <= 1024) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 1>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
-    if (ld <= 2048) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 2>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
-    if (ld <= 4096) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 4>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
-    return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, 8>, grid, block, 0, hy, w, rows, first, H, ld, eps, out, outb);
+#define DC_HYPER(KEEP, NT) return dc_launch(ctx, "k_hyper_norm", k_hyper_norm<S, KEEP, NT>, dim3(R), dim3(NT), 0, hy, w, rows, first, H, ld, eps, out, outb)
+    if (R <= DC_MAX_T) {         // few tokens: a group a thread
+        if (ld <= 1024) DC_HYPER(1, 256);
+        if (ld <= 2048) DC_HYPER(1, 512);
+        if (ld <= 4096) DC_HYPER(1, 1024);
+        DC_HYPER(2, 1024);
+    }
+    if (ld <= 1024) DC_HYPER(1, 256);
+    if (ld <= 2048) DC_HYPER(2, 256);
+    if (ld <= 4096) DC_HYPER(4, 256);
+    DC_HYPER(8, 256);
+#undef DC_HYPER
 }
 
 }  // namespace
