@@ -168,22 +168,15 @@ __device__ __forceinline__ float4 row_sum4(const dc_row_sum& sum, const int32_t*
     }
     return v;
 }
-// Coefficients in shared memory, padded with zeros to S streams: in [S] | out [S], times mul | mix [S][S].
+// Coefficient i of the table that hyper_mix reads, padded with zeros to S streams: in [S] | out [S], times mul | mix [S][S].  A
+// thread below S (S + 2) has one and puts it there.
 template <int S>
-__device__ __forceinline__ void hyper_coefficients(const dc_hyper& h, float* c) {
+__device__ __forceinline__ float hyper_coefficient(const dc_hyper& h, int i) {
     const int n = h.streams;
-    for (int i = threadIdx.x; i < S * (S + 2); i += blockDim.x) {
-        float v = 0.0f;
-        if (i < S) {
-            if (i < n) v = h.next ? h.next[i] : 1.0f;
-        } else if (i < 2 * S) {
-            if (i - S < n && h.done) v = h.mul * h.done[n + i - S];
-        } else {
-            const int s = (i - 2 * S) / S, t = (i - 2 * S) % S;
-            if (s < n && t < n) v = h.done ? h.done[2 * n + s * n + t] : s == t ? 1.0f : 0.0f;
-        }
-        c[i] = v;
-    }
+    if (i < S) return i >= n ? 0.0f : h.next ? h.next[i] : 1.0f;
+    if (i < 2 * S) return i - S < n && h.done ? h.mul * h.done[n + i - S] : 0.0f;
+    const int s = (i - 2 * S) / S, t = (i - 2 * S) % S;
+    return s >= n || t >= n ? 0.0f : h.done ? h.done[2 * n + s * n + t] : s == t ? 1.0f : 0.0f;
 }
 // Group i of four columns of token t: the streams,
 template <int S>

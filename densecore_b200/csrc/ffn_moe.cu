@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
     if (rank == 0)
         for (int e = tid; e < p.r.experts; e += NR_WARPS * 32) correction[e] = p.r.correction ? p.r.correction[e] : 0.0f;
     if constexpr (S > 0) {
-        hyper_coefficients<S>(p.hy, coef);
+        if (tid < S * (S + 2)) coef[tid] = hyper_coefficient<S>(p.hy, tid);
         __syncthreads();
     }
     pdl_wait();
@@ -225,7 +225,8 @@ __global__ void __launch_bounds__(NR_WARPS * 32) k_moe_norm_route(const NormRout
 }
 
 // Prompts of bf16 models: sixteen tokens per CTA, a warp norms each; the router product takes the rounded rows (tensor cores,
-// f32 sums), sixteen experts and a share of the columns per warp; then a warp chooses for each token.
+// f32 sums), sixteen experts and a share of the columns per warp; then a warp chooses for each token.  Without NORM the rounded rows
+// are there already.
 constexpr int NT_WARPS = 16, NT_AHEAD = 4;
 struct TileSizes {
     int tiles, shares, ldh;      // expert tiles, column shares, pitch of a normed row in shared memory
@@ -242,10 +243,10 @@ struct TileSizes {
     }
 };
 
-template <int PER, int S>
+template <int PER, bool NORM>
 __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const NormRouteParams p, int rows, int T) {
     extern __shared__ __align__(16) uint8_t sm[];
-    __shared__ float correction[32 * PER], coef[S ? S * (S + 2) : 1];
+    __shared__ float correction[32 * PER];
     const TileSizes z = TileSizes::of(p.r.experts, p.ld);
     __nv_bfloat16* h = reinterpret_cast<__nv_bfloat16*>(sm);            // [16][ldh]
     float* part = reinterpret_cast<float*>(sm + z.part);                // [shares][experts][17]
@@ -267,37 +268,26 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
 #pragma unroll
         for (int j = 0; j < NT_AHEAD; ++j) fetch(j, warp % z.tiles, begin + j);
     for (int e = tid; e < p.r.experts; e += NT_WARPS * 32) correction[e] = p.r.correction ? p.r.correction[e] : 0.0f;
-    if constexpr (S > 0) {
-        hyper_coefficients<S>(p.hy, coef);
-        __syncthreads();
-    }
     pdl_wait();
-    {
-        auto row = [&](int i, bool store) {
-            if constexpr (S > 0) {
-                const int tc = min(t, T - 1);
-                float4 streams[S];
-                hyper_load<S>(p.hy, tc, i, p.ld, streams);
-                return hyper_mix<S>(p.hy, coef, tc, i, p.ld, streams, reinterpret_cast<const float4*>(p.hy.y + (size_t)tc * p.ld)[i], store && t < T);
-            } else {
-                return reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld)[i];
-            }
-        };
+    if constexpr (!NORM) {
+        const uint4* from = reinterpret_cast<const uint4*>(p.outb + (size_t)min(t, T - 1) * p.ld);
+        uint4* to = reinterpret_cast<uint4*>(h + warp * z.ldh);
+#pragma unroll 8
+        for (int i = lane; i < (z.ldh - 32) / 8; i += 32) to[i] = i < p.ld / 8 ? from[i] : make_uint4(0, 0, 0, 0);
+    } else {
+        const float4* x4 = reinterpret_cast<const float4*>(p.x + (size_t)min(t, T - 1) * p.ld);
         const float4* w4 = reinterpret_cast<const float4*>(p.w);
         uint2* to = reinterpret_cast<uint2*>(h + warp * z.ldh);
-        constexpr int KEEP = S > 4 ? 8 : 16;         // groups of four that a lane holds; wider rows are read twice
+        constexpr int KEEP = 16;             // groups of four that a lane holds; wider rows are read twice
         float4 x[KEEP];
         float ss = 0.0f;
 #pragma unroll
-        for (int j = 0; j < KEEP; ++j) {
-            x[j] = lane + 32 * j < n4 ? row(lane + 32 * j, true) : make_float4(0.f, 0.f, 0.f, 0.f);
-            if (S > 2 || (S > 0 && j % 2)) asm volatile("" ::: "memory");        // as many loads in flight as there are registers
-        }
+        for (int j = 0; j < KEEP; ++j) x[j] = lane + 32 * j < n4 ? x4[lane + 32 * j] : make_float4(0.f, 0.f, 0.f, 0.f);
         auto square = [&](const float4& v) { ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); };
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) square(x[j]);
-#pragma unroll (S > 0 ? 2 : 8)
-        for (int i = lane + 32 * KEEP; i < n4; i += 32) square(row(i, true));
+#pragma unroll 8
+        for (int i = lane + 32 * KEEP; i < n4; i += 32) square(x4[i]);
         const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.H + p.eps);
         auto put = [&](int i, const float4& v) {
             uint2 r = make_uint2(0u, 0u);
@@ -310,8 +300,8 @@ __global__ void __launch_bounds__(NT_WARPS * 32) k_moe_norm_route_tile(const Nor
         };
 #pragma unroll
         for (int j = 0; j < KEEP; ++j) put(lane + 32 * j, x[j]);
-#pragma unroll (S > 0 ? 2 : 8)
-        for (int i = lane + 32 * KEEP; i < (z.ldh - 32) / 4; i += 32) put(i, i < n4 ? row(i, false) : make_float4(0.f, 0.f, 0.f, 0.f));
+#pragma unroll 8
+        for (int i = lane + 32 * KEEP; i < (z.ldh - 32) / 4; i += 32) put(i, i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f));
     }
     __syncthreads();
     for (int tile = warp % z.tiles; working && tile < z.tiles; tile += z.shares > 1 ? z.tiles : NT_WARPS) {
@@ -731,29 +721,39 @@ int launch_down(dc_ctx* ctx, const DownParams& p) {
     return dc_launch(ctx, "k_moe_down_mma", k_moe_down_mma<NT, 1>, dim3(tiles), block, 0, p);
 }
 
+template <int PER>
+int launch_route_tile(dc_ctx* ctx, const NormRouteParams& p, const dc_moe_ffn& f, int T, bool normed) {
+    const TileSizes z = TileSizes::of(f.experts, p.ld);
+    const void* k = normed ? (const void*)k_moe_norm_route_tile<PER, false> : (const void*)k_moe_norm_route_tile<PER, true>;
+    const int st = dc_kernel_setup(ctx, k, (int)z.bytes, "k_moe_norm_route_tile");
+    if (st != DC_B200_OK) return st;
+    const dim3 grid((T + 15) / 16), block(NT_WARPS * 32);
+    if (normed) return dc_launch(ctx, "k_moe_route_tile", k_moe_norm_route_tile<PER, false>, grid, block, z.bytes, p, f.router.N, T);
+    return dc_launch(ctx, "k_moe_norm_route_tile", k_moe_norm_route_tile<PER, true>, grid, block, z.bytes, p, f.router.N, T);
+}
+
 }  // namespace
 
 int dc_launch_moe_norm_route(dc_ctx* ctx, const dc_moe_ffn& f, const float* x, const dc_hyper* hy, const float* w, int T, int H, int ld, float eps, float* out,
                              __nv_bfloat16* outb, int32_t* ids, float* weights) {
     if (f.experts > DC_MOE_MAX_EXPERTS || f.groups > DC_MOE_MAX_GROUPS || ld % 8) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad operand");
-    if (hy && (hy->streams > DC_MAX_STREAMS || hy->sum.k || !hy->y || !hy->x_out || hy->x == hy->x_out)) return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad streams");
+    // prompt-sized steps bring the streams up to date in a kernel of their own: what this one reads of a row it would read twice
+    if (hy && T > DC_MAX_T) {
+        const int st = dc_launch_hyper_norm(ctx, *hy, w, nullptr, 0, T, H, ld, eps, out, outb);
+        if (st != DC_B200_OK) return st;
+    } else if (hy && (hy->streams > DC_MAX_STREAMS || hy->sum.k || !hy->y || !hy->x_out || hy->x == hy->x_out))
+        return dc_fail(ctx, DC_B200_INTERNAL_ERROR, "moe_norm_route: bad streams");
     const NormRouteParams p = {route_params(f, ids, weights), hy ? *hy : dc_hyper(), x, w, f.router.w, f.router.ld, H, ld, eps, out, outb};
     const size_t smem = (size_t)(ld + 255) / 256 * 256 * 4;
-    const TileSizes z = TileSizes::of(f.experts, ld);
 #define DC_ROUTE_S(PER, S)                                                                                                                       \
     do {                                                                                                                                         \
-        if (T > DC_MAX_T) {                                                                                                                      \
-            const int st = dc_kernel_setup(ctx, (const void*)k_moe_norm_route_tile<PER, S>, (int)z.bytes, "k_moe_norm_route_tile");               \
-            if (st != DC_B200_OK) return st;                                                                                                     \
-            return dc_launch(ctx, "k_moe_norm_route_tile", k_moe_norm_route_tile<PER, S>, dim3((T + 15) / 16), dim3(NT_WARPS * 32), z.bytes, p,   \
-                             f.router.N, T);                                                                                                     \
-        }                                                                                                                                        \
         const int st = dc_kernel_setup_small(ctx, (const void*)k_moe_norm_route<PER, S>, (int)smem, "k_moe_norm_route");                          \
         if (st != DC_B200_OK) return st;                                                                                                         \
         return dc_launch_cluster(ctx, "k_moe_norm_route", k_moe_norm_route<PER, S>, dim3(T * NR_CTAS), dim3(NR_WARPS * 32), smem, NR_CTAS, p);    \
     } while (0)
 #define DC_ROUTE(PER)                                   \
     do {                                                \
+        if (T > DC_MAX_T) return launch_route_tile<PER>(ctx, p, f, T, hy != nullptr); \
         if (!hy) DC_ROUTE_S(PER, 0);                    \
         if (hy->streams <= 2) DC_ROUTE_S(PER, 2);       \
         if (hy->streams <= 4) DC_ROUTE_S(PER, 4);       \

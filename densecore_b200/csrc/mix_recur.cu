@@ -708,12 +708,18 @@ __device__ __forceinline__ void column_dots(const float* rows, int dp, const flo
 // EPL: key channels per lane (the key size, padded to 32 EPL).
 constexpr int scan_block_floats(int kind, int dp) { return kind == SCAN_DELTA ? delta_block_floats(dp) : kind == SCAN_GENERAL ? general_block_floats(dp) : 2 * BT * dp + SSD_BLOCK; }
 
+// Blocks in flight or at work: a block takes less time than its way from L2.
+constexpr int scan_stages(int kind, int dp) {
+    const int bytes = (scan_block_floats(kind, dp) + BT * SC_COLS) * 4;
+    return 4 * bytes <= 160 * 1024 ? 4 : 3 * bytes <= 220 * 1024 ? 3 : 2;
+}
+
 // NC: columns of a warp.
 template <int EPL, int KIND, int NC>
 __global__ void __launch_bounds__(SC_COLS / NC * 32) k_state_scan(const ScanParams p) {
     constexpr bool GENERAL = KIND == SCAN_GENERAL, DELTA = KIND != SCAN_SSD;         // the delta rules' factors come whole from memory
     constexpr int DP = 32 * EPL, BLK = scan_block_floats(KIND, DP), BUF = BLK + BT * SC_COLS;
-    constexpr int SC_THREADS = SC_COLS / NC * 32, LANES = 32 / NC, PER = NC / 2;
+    constexpr int SC_THREADS = SC_COLS / NC * 32, LANES = 32 / NC, PER = NC / 2, STAGES = scan_stages(KIND, DP);
     extern __shared__ __align__(16) float sm[];
     __shared__ __align__(16) float s_d[SC_COLS / NC][NC][BT], s_u[SC_COLS / NC][NC][BT];
     pdl_launch_dependents();
@@ -721,7 +727,7 @@ __global__ void __launch_bounds__(SC_COLS / NC * 32) k_state_scan(const ScanPara
     const int c0 = blockIdx.x * SC_COLS, h = blockIdx.y, e = blockIdx.z, kh = h / p.per;
     const int col = c0 + warp * NC + lc;
     if (!DELTA) {
-        for (int i = tid; i < 2 * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels stay zero
+        for (int i = tid; i < STAGES * BUF; i += SC_THREADS) sm[i] = 0.0f;    // padded channels stay zero
         __syncthreads();
     }
     pdl_wait();
@@ -770,16 +776,15 @@ __global__ void __launch_bounds__(SC_COLS / NC * 32) k_state_scan(const ScanPara
         cp_async_commit();
     };
     const float Dh = DELTA || !p.D ? 0.0f : p.D[h];
-    load(0, 0);
+    for (int b = 0; b < STAGES - 1; ++b)
+        if (b < blocks) load(b, b);
+        else cp_async_commit();
     for (int b = 0; b < blocks; ++b) {
-        if (b + 1 < blocks) {
-            load(b + 1, (b + 1) & 1);
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
-        const float* x = sm + (b & 1) * BUF;
+        cp_async_wait<STAGES - 2>();
+        __syncthreads();         // the block has landed; every warp is done with the stage that the next load fills
+        if (b + STAGES - 1 < blocks) load(b + STAGES - 1, (b + STAGES - 1) % STAGES);
+        else cp_async_commit();
+        const float* x = sm + b % STAGES * BUF;
         // ---- the columns against the block's (decayed) keys and queries; see column_dots for who works for whom
         float r[DELTA ? 2 : 1][PER];
         column_dots<EPL, DELTA ? 2 : 1, NC>(x, DP, s, lane, r);
@@ -863,7 +868,7 @@ __global__ void __launch_bounds__(SC_COLS / NC * 32) k_state_scan(const ScanPara
 #pragma unroll
                     for (int i = 0; i < EPL; ++i) s[c][i] = fmaf(w[g][i], u[c][g], s[c][i]);
         }
-        __syncthreads();
+        __syncwarp();
     }
 #pragma unroll
     for (int c = 0; c < NC; ++c)
@@ -877,16 +882,16 @@ __global__ void __launch_bounds__(SC_COLS / NC * 32) k_state_scan(const ScanPara
 template <int EPL, int KIND, int NC>
 int launch_scan_epl(dc_ctx* ctx, const ScanParams& p, int E) {
     // a few CTAs that run long: started while the many of the kernel before still leave, they would crowd on the first free SMs
-    const size_t smem = (size_t)2 * (scan_block_floats(KIND, 32 * EPL) + BT * SC_COLS) * 4;
+    const size_t smem = (size_t)scan_stages(KIND, 32 * EPL) * (scan_block_floats(KIND, 32 * EPL) + BT * SC_COLS) * 4;
     DC_TRY(dc_kernel_setup(ctx, (const void*)k_state_scan<EPL, KIND, NC>, (int)smem, "k_state_scan"));
     return dc_launch_drained(ctx, "k_state_scan", k_state_scan<EPL, KIND, NC>, dim3((p.vdim + SC_COLS - 1) / SC_COLS, p.heads, E), dim3(SC_COLS / NC * 32), smem, p);
 }
 int key_pad(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
-// Few columns in the whole step: fewer of them for each warp.
+// Few columns in the whole step: the delta rules' warps, which work on more rows, take fewer of them each.
 template <int EPL, int KIND>
 int launch_scan_columns(dc_ctx* ctx, const ScanParams& p, int E) {
     const int ctas = (p.vdim + SC_COLS - 1) / SC_COLS * p.heads * E;
-    return ctas <= 2 * ctx->num_sms ? launch_scan_epl<EPL, KIND, 2>(ctx, p, E) : launch_scan_epl<EPL, KIND, 4>(ctx, p, E);
+    return KIND != SCAN_SSD && ctas <= 2 * ctx->num_sms ? launch_scan_epl<EPL, KIND, 2>(ctx, p, E) : launch_scan_epl<EPL, KIND, 4>(ctx, p, E);
 }
 template <int KIND>
 int launch_scan(dc_ctx* ctx, const ScanParams& p, int E) {

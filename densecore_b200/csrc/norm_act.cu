@@ -170,7 +170,7 @@ __global__ void __launch_bounds__(NT) k_hyper_norm(const dc_hyper hy, const floa
         const int i = threadIdx.x + NT * j;
         wv[j] = w && i < n4 ? reinterpret_cast<const float4*>(w)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    dc::hyper_coefficients<S>(hy, coef);
+    const float own = threadIdx.x < S * (S + 2) ? dc::hyper_coefficient<S>(hy, threadIdx.x) : 0.0f;
     dc::pdl_wait();
     const int t = rows ? rows[blockIdx.x] : first + (int)blockIdx.x;
     float ss = 0.0f;
@@ -187,6 +187,7 @@ __global__ void __launch_bounds__(NT) k_hyper_norm(const dc_hyper hy, const floa
         }
         if (j0 == 0) {
             if (threadIdx.x < (unsigned)hy.sum.k) s_rows[threadIdx.x] = hy.sum.rows[t * hy.sum.k + threadIdx.x];
+            if (threadIdx.x < S * (S + 2)) coef[threadIdx.x] = own;
             __syncthreads();
         }
 #pragma unroll

@@ -618,7 +618,7 @@ int moe_layer(dc_model* m, const dc_step& st, dc_stack_layer& Ly, const dc_hyper
     const double up_bytes = (double)f.up_rows * f.up.ld * 2, down_bytes = (double)f.down_rows * f.down.ld * 2;
     const double touched = std::min<double>(f.experts, rows);
     if (dc_moe_norm_route_fits(f, st.b16, T, H)) {
-        L(DC_K_ROUTER, lin_bytes(f.router, T), 1, dc_launch_moe_norm_route(ctx, f, b.x, hy, Ly.norm2, T, W, H, s->cfg.eps, h, xb, b.moe_ids, b.moe_w));
+        L(DC_K_ROUTER, lin_bytes(f.router, T), hy && T > DC_MAX_T ? 2 : 1, dc_launch_moe_norm_route(ctx, f, b.x, hy, Ly.norm2, T, W, H, s->cfg.eps, h, xb, b.moe_ids, b.moe_w));
     } else {
         if (hy) L(DC_K_PRE_NORM, hyper_bytes(m, T), 1, dc_launch_hyper_norm(ctx, *hy, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, h, xb));
         else L(DC_K_PRE_NORM, 8.0 * T * W, 1, dc_launch_norm_rows(ctx, b.x, Ly.norm2, nullptr, 0, T, W, H, s->cfg.eps, h, xb, H));
