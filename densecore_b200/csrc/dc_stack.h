@@ -10,6 +10,7 @@
 #include <cuda_bf16.h>
 
 #include <map>
+#include <set>
 #include <string>
 #include <tuple>
 #include <vector>
@@ -291,6 +292,7 @@ struct dc_stack {
     float* final_norm = nullptr;
     std::vector<dc_stack_tensor> tensors;
     std::map<std::string, int> index;
+    std::set<std::string> unused;        // files may hold these too: norms and coefficients of sublayers that a layer does not have
     std::vector<void*> owned;   // weight memory
     size_t weight_bytes = 0;
     std::map<dc_rotation, float*> rot;   // cos/sin tables [max_ctx][dims / 2][2]

@@ -598,6 +598,8 @@ int dc_stack_parse(dc_model* m, const dc_json& cj, const Shapes& shapes) {
             else read_dense(r, *mlp, p + "mlp.", where + ".mlp", &L, a->dense);
             if (a->block != DC_BLOCK_PARALLEL) r.norm(&L.norm2, p + "norm2");
             if (hyper) read_hyper(r, p + "hc2.", &L.hyper[1]);
+        } else if (hyper) {
+            for (const char* t : {"norm2", "hc2.in", "hc2.out", "hc2.mix"}) s->unused.insert(p + t);
         }
     }
     // the order in which layers run

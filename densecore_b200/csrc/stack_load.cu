@@ -125,6 +125,7 @@ int load_dir(dc_ctx* ctx, const std::string& dir, int dtype, int max_seqs, int m
     DC_TRY(create(ctx, config, shapes, dtype, max_seqs, max_ctx, pool_tokens, out));
     dc_model* m = *out;
     for (const Entry& e : entries) {
+        if (m->stack->unused.count(e.name)) continue;
         auto it = m->stack->index.find(e.name);
         int rc = DC_B200_OK;
         if (it == m->stack->index.end()) {

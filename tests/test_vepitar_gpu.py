@@ -32,7 +32,7 @@ ALONE = {
     "general_one_head": [general(heads=1, dim=8)],
     "general_of_one": [general(heads=4, dim=1)],
     "general_odd_sizes": [general(heads=5, dim=19)],
-    "general_32": [general(heads=4, dim=32)],
+    "general_32": [general(heads=5, dim=32)],
     "general_64": [general(heads=3, dim=64)],
     "general_100": [general(heads=2, dim=100)],
     "general_128": [general(heads=2, dim=128)],
@@ -452,6 +452,8 @@ def test_loading_errors(ctx, tmp_path):
         return c
     load("good")
     load("f32_vectors", f32=("l0.norm1", "l1.mix.w0", "l0.mix.pb", "l0.hc1.mix", "l0.mix.q.conv"))
+    none = dict(cfg, layers=[dict(cfg["layers"][0], mlp=None), cfg["layers"][1]])
+    load("unused", none, {k: v for k, v in t.items() if not k.startswith("l0.mlp.")})      # the second sublayer's norm and coefficients stay
     without = lambda *names: {k: v for k, v in t.items() if k not in names}
     for name, c, tensors, msg in (
             ("missing", cfg, without("l0.mlp.e3.up"), "l0.mlp.e3.up"),
