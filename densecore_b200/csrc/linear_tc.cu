@@ -150,11 +150,12 @@ __device__ __forceinline__ void read_out(const LtParams& p, uint32_t tmem, int r
                 for (int i = 0; i < 8; ++i)
                     r[i] = pack_bf2(relu2(__int_as_float(v[2 * i])) * e.tok_scale[min(t0 + c0 + 2 * i, t1 - 1)],
                                     relu2(__int_as_float(v[2 * i + 1])) * e.tok_scale[min(t0 + c0 + 2 * i + 1, t1 - 1)]);
-            } else
+            } else {
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const float a = __int_as_float(v[2 * i]) + bias, b = __int_as_float(v[2 * i + 1]) + bias;
-                r[i] = act ? pack_bf2(quick_silu(a), quick_silu(b)) : pack_bf2(a, b);
+                for (int i = 0; i < 8; ++i) {
+                    const float a = __int_as_float(v[2 * i]) + bias, b = __int_as_float(v[2 * i + 1]) + bias;
+                    r[i] = act ? pack_bf2(quick_silu(a), quick_silu(b)) : pack_bf2(a, b);
+                }
             }
             transpose8<1, 8>(r, v8, lane);
             const int m = in ? n - c0 : 0;
